@@ -26,8 +26,10 @@ OBJ = ROOT / "csrc" / "build"
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
-    "--use_fast_math", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr", "-Xptxas", "-v",
+    "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr", "-Xptxas", "-v",
 ]
+# Files whose arithmetic also serves 32-bit models keep the exact divide, square root and exponential; all others use the fast forms.
+EXACT_MATH = {"linear_attention", "recurrent_scan", "residual32", "gemm_simt", "attention_general"}
 
 
 def _stamp(paths, extra=""):
@@ -67,32 +69,62 @@ def nvcc_path() -> str:
     return shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
 
 
-def build_kernels(force: bool = False) -> Path:
-    out = ROOT / "_kernels.so"
+def _kernel_sources(only=None):
+    """``[(source, compile flags, stamp of everything the object depends on)]`` of all kernels, or of the files named in ``only``."""
     srcs = sorted((CSRC / "kernels").glob("*.cu"))
+    if only is not None:
+        missing = set(only) - {s.stem for s in srcs}
+        if missing:
+            raise ValueError(f"no kernel source named {sorted(missing)}")
+        srcs = [s for s in srcs if s.stem in only]
     hdrs = sorted((CSRC / "kernels").glob("*.cuh")) + sorted((CSRC / "kernels").glob("*.h"))
+    hdr_stamp = _stamp(hdrs, " ".join(NVCC_FLAGS))
+    out = []
+    for src in srcs:
+        flags = NVCC_FLAGS + ([] if src.stem in EXACT_MATH else ["--use_fast_math"])
+        out.append((src, flags, _stamp([src], hdr_stamp + " ".join(flags))))
+    return out
+
+
+def build_kernels(force: bool = False, only=None) -> Path:
+    """Compile and link every kernel into ``_kernels.so``, or the sources named in ``only`` into ``_kernels_part.so``."""
+    out = ROOT / ("_kernels.so" if only is None else "_kernels_part.so")
     OBJ.mkdir(parents=True, exist_ok=True)
     nvcc = nvcc_path()
-    hdr_stamp = _stamp(hdrs, " ".join(NVCC_FLAGS))
 
-    def compile_one(src: Path):
+    def compile_one(item):
+        src, flags, stamp = item
         obj = OBJ / (src.stem + ".o")
         sf = OBJ / (src.stem + ".stamp")
-        stamp = _stamp([src], hdr_stamp)
         if obj.exists() and not force and sf.exists() and sf.read_text() == stamp:
             return obj, False
-        _run([nvcc] + NVCC_FLAGS + ["-I", str(CSRC / "kernels"), "-c", str(src), "-o", str(obj)],
+        _run([nvcc] + flags + ["-I", str(CSRC / "kernels"), "-c", str(src), "-o", str(obj)],
              log=OBJ / (src.stem + ".ptxas.log"))
         sf.write_text(stamp)
         return obj, True
 
+    items = _kernel_sources(only)
     with cf.ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 2)) as ex:
-        res = list(ex.map(compile_one, srcs))
+        res = list(ex.map(compile_one, items))
     objs = [str(o) for o, _ in res]
-    if out.exists() and not force and not any(ch for _, ch in res):
+    linked = OBJ / (out.name + ".stamp")
+    stamp = _stamp([], " ".join(s for _, _, s in items))
+    if out.exists() and not force and linked.exists() and linked.read_text() == stamp:
         return out
-    _run([nvcc, "-shared", "-o", str(out)] + objs + ["-gencode", "arch=compute_100a,code=sm_100a", "-lcudart"])
+    tmp = out.with_suffix(f".{os.getpid()}.tmp")           # renamed into place: another process never loads a half-written library
+    _run([nvcc, "-shared", "-o", str(tmp)] + objs + ["-gencode", "arch=compute_100a,code=sm_100a", "-lcudart"])
+    os.replace(tmp, out)
+    linked.write_text(stamp)
     return out
+
+
+def ensure_kernels(only) -> Path:
+    """A library that holds at least the sources named in ``only``: the full one when it has been built from the sources as they are,
+    else a partial one, compiled now if need be."""
+    full, stamp_file = ROOT / "_kernels.so", OBJ / "_kernels.so.stamp"
+    if full.exists() and (not stamp_file.exists() or stamp_file.read_text() == _stamp([], " ".join(s for _, _, s in _kernel_sources()))):
+        return full
+    return build_kernels(only=only)
 
 
 def build_all(force: bool = False):

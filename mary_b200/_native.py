@@ -39,6 +39,17 @@ def kernels() -> ctypes.CDLL:
         return _kernels
 
 
+def require_kernels(sources) -> None:
+    """Load a kernel library that holds the named sources, compiling them first where the checkout has none (the entry points of a
+    fresh checkout call this; everything else expects the full library to be built)."""
+    global _kernels
+    from . import _build
+    path = _build.ensure_kernels(sources)
+    with _lock:
+        if _kernels is None:
+            _kernels = ctypes.CDLL(str(path))
+
+
 def kernels_available() -> bool:
     return (_ROOT / "_kernels.so").exists()
 

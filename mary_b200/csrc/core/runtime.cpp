@@ -7,6 +7,8 @@
 // `kv_truncate` rolls back, and the scheduler packs prefill chunks and decode rows of many sequences into one
 // flattened batch under a token budget, admitting requests only while pages are available (the admission
 // idea of src/models/inkling/budget.rs:677).
+// Models with recurrent layers keep a fixed-size state per sequence beside the pages: the allocator also owns `num_slots` state
+// slots, a sequence takes one when it is created and gives it back with its pages, so admission covers both resources.
 #include <algorithm>
 #include <cstdint>
 #include <cstring>
@@ -19,6 +21,7 @@ namespace {
 struct Seq {
   std::vector<int32_t> pages;
   int64_t len = 0;  // tokens whose K/V are in the cache
+  int32_t slot = -1;  // recurrent-state slot (allocators without slots leave it at -1)
 };
 
 struct KvAlloc {
@@ -26,6 +29,8 @@ struct KvAlloc {
   std::vector<int32_t> free_list;  // stack
   std::unordered_map<int64_t, Seq> seqs;
   int64_t peak_used = 0;
+  int32_t num_slots = 0;           // 0: no recurrent state, any number of sequences
+  std::vector<int32_t> free_slots; // stack
 };
 
 struct Request {
@@ -78,16 +83,41 @@ int64_t kv_seq_len(void* h, int64_t seq) {
   return it == a->seqs.end() ? -1 : it->second.len;
 }
 
-// Grow `seq` by `tokens`; allocates pages as needed.  Returns the new length, or -1 when out of pages
-// (nothing is changed in that case).
+// Give the allocator `n` recurrent-state slots (before the first sequence is created).  Returns 0, or -1 when sequences exist.
+int32_t kv_set_slots(void* h, int32_t n) {
+  auto* a = (KvAlloc*)h;
+  if (!a->seqs.empty() || n < 0) return -1;
+  a->num_slots = n;
+  a->free_slots.resize(n);
+  for (int32_t i = 0; i < n; ++i) a->free_slots[i] = n - 1 - i;  // pop gives 0,1,2,...
+  return 0;
+}
+int32_t kv_free_slots(void* h) { return (int32_t)((KvAlloc*)h)->free_slots.size(); }
+
+// State slots of a list of sequences; -1 for an unknown sequence or an allocator without slots.  Returns how many were unknown.
+int32_t kv_seq_slots(void* h, const int64_t* seqs, int32_t n, int32_t* out) {
+  auto* a = (KvAlloc*)h;
+  int32_t missing = 0;
+  for (int32_t i = 0; i < n; ++i) {
+    auto it = a->seqs.find(seqs[i]);
+    out[i] = it == a->seqs.end() ? -1 : it->second.slot;
+    missing += it == a->seqs.end();
+  }
+  return missing;
+}
+
+// Grow `seq` by `tokens`; allocates pages (and, for a new sequence, its state slot) as needed.  Returns the new length, or -1 when
+// out of pages or slots (nothing is changed in that case).
 int64_t kv_extend(void* h, int64_t seq, int64_t tokens) {
   auto* a = (KvAlloc*)h;
   Seq& s = a->seqs[seq];
   int32_t need = pages_for(a, s.len + tokens) - (int32_t)s.pages.size();
-  if (need > (int32_t)a->free_list.size()) {
+  const bool no_slot = a->num_slots > 0 && s.slot < 0 && a->free_slots.empty();
+  if (need > (int32_t)a->free_list.size() || no_slot) {
     if (s.pages.empty() && s.len == 0) a->seqs.erase(seq);
     return -1;
   }
+  if (a->num_slots > 0 && s.slot < 0) { s.slot = a->free_slots.back(); a->free_slots.pop_back(); }
   for (int32_t i = 0; i < need; ++i) { s.pages.push_back(a->free_list.back()); a->free_list.pop_back(); }
   s.len += tokens;
   a->peak_used = std::max<int64_t>(a->peak_used, a->num_pages - (int64_t)a->free_list.size());
@@ -112,6 +142,7 @@ void kv_release(void* h, int64_t seq) {
   auto it = a->seqs.find(seq);
   if (it == a->seqs.end()) return;
   for (auto p = it->second.pages.rbegin(); p != it->second.pages.rend(); ++p) a->free_list.push_back(*p);
+  if (it->second.slot >= 0) a->free_slots.push_back(it->second.slot);
   a->seqs.erase(it);
 }
 
@@ -169,9 +200,11 @@ int32_t sched_add(void* h, int64_t id, const int32_t* prompt, int32_t n, int32_t
 int32_t sched_num_waiting(void* h) { return (int32_t)((Sched*)h)->waiting.size(); }
 int32_t sched_num_running(void* h) { return (int32_t)((Sched*)h)->running.size(); }
 
-// Attach draft tokens to a running sequence: its next decode step feeds [pending, drafts...] (k+1 rows).
+// Attach draft tokens to a running sequence: its next decode step feeds [pending, drafts...] (k+1 rows).  Refused for models with
+// recurrent state, which cannot be rolled back over rejected rows.
 int32_t sched_set_drafts(void* h, int64_t id, const int32_t* drafts, int32_t k) {
   Sched* s = (Sched*)h;
+  if (s->kv->num_slots > 0 && k > 0) return -1;
   auto it = s->reqs.find(id);
   if (it == s->reqs.end() || k > 8) return -1;
   it->second.spec = k;

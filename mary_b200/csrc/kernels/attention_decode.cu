@@ -29,6 +29,7 @@ struct DecParams {
   int64_t k_tok, k_page, v_tok, v_page;
   int Hq, Hkv, G, RQ, nsplit, window;
   float scale, softcap;
+  int64_t out_ld;              // elements between the output rows of two tokens
   // 8-bit cache: kc / vc hold one unsigned code per element and the strides count codes; k_sz / v_sz hold (scale, zero) of every
   // (slot, kv head) as two floats, slot-major; element = code * scale + zero
   const float* k_sz; const float* v_sz;
@@ -239,7 +240,7 @@ attn_decode_kernel(const DecParams p) {
     }
     if (p.nsplit == 1) {
       const int tq = row0 + r / p.G, h = kvh * p.G + r % p.G;
-      p.out[((int64_t)tq * p.Hq + h) * D + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+      p.out[(int64_t)tq * p.out_ld + (int64_t)h * D + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
     } else {
       const int64_t pi = (((int64_t)nb * p.Hkv + kvh) * p.nsplit + split) * MAXR + r;
       p.part_o[pi * D + d] = acc;
@@ -268,7 +269,7 @@ __global__ void attn_decode_combine_kernel(const DecParams p, int D) {
       acc += p.part_o[pi * D + d] * c;
     }
     const int tq = row0 + r / p.G, h = kvh * p.G + r % p.G;
-    p.out[((int64_t)tq * p.Hq + h) * D + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+    p.out[(int64_t)tq * p.out_ld + (int64_t)h * D + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
   }
 }
 
@@ -295,7 +296,7 @@ static int decode_run(const void* q, const void* kc, const void* vc, const float
                       const int* kv_len, const int* q_start, const int* blk_seq, const int* blk_q0, int NB,
                       int max_pages, int page_size, int64_t k_tok, int64_t k_page, int64_t v_tok, int64_t v_page,
                       int Hq, int Hkv, int D, int RQ, int nsplit, int window, float scale, float softcap,
-                      float* scratch, cudaStream_t s) {
+                      float* scratch, cudaStream_t s, int64_t out_ld = 0) {
   if (NB <= 0) return MARY_OK;
   DecParams p;
   p.k_sz = k_sz; p.v_sz = v_sz;
@@ -304,6 +305,7 @@ static int decode_run(const void* q, const void* kc, const void* vc, const float
   p.max_pages = max_pages; p.page_size = page_size; p.k_tok = k_tok; p.k_page = k_page; p.v_tok = v_tok; p.v_page = v_page;
   p.Hq = Hq; p.Hkv = Hkv; p.G = Hq / Hkv; p.RQ = RQ; p.nsplit = nsplit < 1 ? 1 : nsplit; p.window = window; p.scale = scale;
   p.softcap = softcap;
+  p.out_ld = out_ld > 0 ? out_ld : (int64_t)Hq * D;
   if (p.G * Hkv != Hq) return MARY_ERR_BAD_ARG;
   if (p.nsplit > 1 && !scratch) return MARY_ERR_BAD_ARG;
   p.part_o = scratch;
@@ -315,13 +317,14 @@ static int decode_run(const void* q, const void* kc, const void* vc, const float
   return MARY_ERR_BAD_ARG;
 }
 
+// out_ld: elements between the output rows of two tokens (0: Hq * D, contiguous).
 MARY_API int mary_paged_attention_decode(const void* q, const void* kc, const void* vc, void* out, const int* page_table,
                                          const int* kv_len, const int* q_start, const int* blk_seq, const int* blk_q0, int NB,
                                          int max_pages, int page_size, int64_t k_tok, int64_t k_page, int64_t v_tok, int64_t v_page,
                                          int Hq, int Hkv, int D, int RQ, int nsplit, int window, float scale, float softcap,
-                                         float* scratch, cudaStream_t s) {
+                                         float* scratch, int64_t out_ld, cudaStream_t s) {
   return decode_run(q, kc, vc, nullptr, nullptr, out, page_table, kv_len, q_start, blk_seq, blk_q0, NB, max_pages, page_size, k_tok, k_page,
-                    v_tok, v_page, Hq, Hkv, D, RQ, nsplit, window, scale, softcap, scratch, s);
+                    v_tok, v_page, Hq, Hkv, D, RQ, nsplit, window, scale, softcap, scratch, s, out_ld);
 }
 
 // The same over an 8-bit cache: kc / vc are code pages [pages, page, Hkv, D] of unsigned bytes (strides in bytes), k_sz / v_sz the

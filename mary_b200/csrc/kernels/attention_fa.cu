@@ -25,12 +25,14 @@ using namespace mary;
 namespace {
 
 constexpr int PAGE = 16, KB = 64, TR = 128, CHUNK = 64;
-constexpr int NSBUF = 2, NPBUF = 2;
+constexpr int NSBUF = 2;
 constexpr int P_BYTES = TR * KB * 2;              // 16 KB
 constexpr int NTHREADS = 224;
 constexpr float RESCALE_THRESHOLD = 8.0f;
 
-template <int DK, int DV>
+// SPLITP: P is handed to the tensor cores as the sum of two bf16 values (rounded value and rounding error), so that the softmax
+// weights keep 16 significant bits; two P V products per block.
+template <int DK, int DV, bool SPLITP>
 struct FaCfg {
   static constexpr int NCK = DK / CHUNK, NCV = DV / CHUNK;
   static constexpr int Q_CHUNK_BYTES = TR * 128;
@@ -38,7 +40,9 @@ struct FaCfg {
   static constexpr int K_CHUNK_BYTES = KB * 128, V_CHUNK_BYTES = KB * 128;
   static constexpr int K_STAGE = NCK * K_CHUNK_BYTES, V_STAGE = NCV * V_CHUNK_BYTES;
   static constexpr int STAGES = (DK + DV > 384) ? 2 : 3;
-  static constexpr int SMEM = Q_BYTES + STAGES * (K_STAGE + V_STAGE) + NPBUF * P_BYTES + 1024 + 256;
+  static constexpr int NPBUF = (SPLITP && DK + DV > 384) ? 1 : 2;
+  static constexpr int P_STAGE = SPLITP ? 2 * P_BYTES : P_BYTES;
+  static constexpr int SMEM = Q_BYTES + STAGES * (K_STAGE + V_STAGE) + NPBUF * P_STAGE + 1024 + 256;
   static constexpr int TMEM_COLS = DV <= 128 ? 256 : 512;     // S: 2 x 64 columns at 0..127, O: DV columns at 128..
   static_assert(DK % CHUNK == 0 && DV % CHUNK == 0 && DV <= 256 && DK <= 256, "head dims: multiples of 64 up to 256");
   static_assert(SMEM <= 232448, "shared memory budget");
@@ -46,7 +50,8 @@ struct FaCfg {
 
 struct FaParams {
   const int* page_table; const int* kv_len; const int* q_start; const int* blk_seq; const int* blk_tok0;
-  __nv_bfloat16* out;      // [T, Hq, DV]
+  __nv_bfloat16* out;      // rows of out_ld elements, head h at h * DV
+  int64_t out_ld;          // elements between the output rows of two tokens
   int max_pages, Hq, Hkv, window, page;
   float scale_log2;
   int* status;
@@ -60,19 +65,19 @@ __device__ __forceinline__ uint64_t fa_desc_mnmajor_sw128(uint32_t addr, uint32_
          (2ull << 61);
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool SPLITP>
 __global__ void __launch_bounds__(NTHREADS, 1)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                   const __grid_constant__ CUtensorMap tm_v, const FaParams p) {
-  using C = FaCfg<DK, DV>;
-  constexpr int STAGES = C::STAGES;
+  using C = FaCfg<DK, DV, SPLITP>;
+  constexpr int STAGES = C::STAGES, NPBUF = C::NPBUF;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
   uint8_t* sK = sQ + C::Q_BYTES;
   uint8_t* sV = sK + STAGES * C::K_STAGE;
   uint8_t* sP = sV + STAGES * C::V_STAGE;
-  uint64_t* bars = (uint64_t*)(sP + NPBUF * P_BYTES);
+  uint64_t* bars = (uint64_t*)(sP + NPBUF * C::P_STAGE);
   uint64_t* q_full = bars;                 // 1
   uint64_t* k_full = q_full + 1;           // [STAGES]
   uint64_t* k_empty = k_full + STAGES;
@@ -187,17 +192,23 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       if (!issue_qk(0)) goto done;
       if (nblk > 1 && !issue_qk(1)) goto done;
       for (int i = 0; i < nblk; ++i) {
-        const int pb = i & 1, stage = i % STAGES;
+        const int pb = i % NPBUF, stage = i % STAGES;
         if (!mbar_wait(&v_full[stage], (i / STAGES) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_TMA)) goto done;
-        if (!mbar_wait(&p_full[pb], (i >> 1) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+        if (!mbar_wait(&p_full[pb], (i / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
         tc_fence_after();
         const uint32_t vb_addr = smem_u32(sV + stage * C::V_STAGE);
 #pragma unroll
         for (int kk = 0; kk < KB / 16; ++kk) {
           // A = P[:, 16 keys] (K-major, no swizzle: the two 16-byte key chunks of one MMA TR*16 bytes apart, 8-row groups
           // 128 bytes apart); B = V^T of those keys (MN-major, 128B swizzle: 64-dim groups one chunk apart, 8-key groups 1 KB apart)
-          umma_f16(tmem_O, fa_desc_kmajor_noswz(p_addr + pb * P_BYTES + kk * 2 * (TR * 16), TR * 16, 128),
+          umma_f16(tmem_O, fa_desc_kmajor_noswz(p_addr + pb * C::P_STAGE + kk * 2 * (TR * 16), TR * 16, 128),
                    fa_desc_mnmajor_sw128(vb_addr + kk * 16 * 128, C::V_CHUNK_BYTES, 1024), idesc_o, (i > 0 || kk > 0) ? 1u : 0u);
+        }
+        if constexpr (SPLITP) {
+#pragma unroll
+          for (int kk = 0; kk < KB / 16; ++kk)
+            umma_f16(tmem_O, fa_desc_kmajor_noswz(p_addr + pb * C::P_STAGE + P_BYTES + kk * 2 * (TR * 16), TR * 16, 128),
+                     fa_desc_mnmajor_sw128(vb_addr + kk * 16 * 128, C::V_CHUNK_BYTES, 1024), idesc_o, 1u);
         }
         umma_commit(&v_empty[stage]);
         umma_commit(&pv_done[pb]);
@@ -214,7 +225,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
     const uint32_t lane_off = (uint32_t)(q4 * 32) << 16;
     float m_ref = -INFINITY, l = 0.f;
     for (int i = 0; i < nblk; ++i) {
-      const int sb = i % NSBUF, pb = i & 1;
+      const int sb = i % NSBUF, pb = i % NPBUF;
       if (!mbar_wait(&s_full[sb], (i / NSBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
       tc_fence_after();
       uint32_t sr[KB];
@@ -251,7 +262,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       const bool first = (m_ref == -INFINITY);
       float corr = 1.f;
       if (need) { corr = first ? 0.f : exp2f(m_ref - mx); m_ref = mx; }
-      uint32_t pw[KB / 2];
+      uint32_t pw[KB / 2], pl[SPLITP ? KB / 2 : 1];
       float psum = 0.f;
       if (full_blk) {
         const float nm = -m_ref;
@@ -261,6 +272,11 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
           const float b = exp2f(fmaf(sf[2 * j + 1], p.scale_log2, nm));
           __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
           pw[j] = *(uint32_t*)&h;
+          if constexpr (SPLITP) {
+            const float2 back = __bfloat1622float2(h);
+            __nv_bfloat162 lo = __floats2bfloat162_rn(a - back.x, b - back.y);
+            pl[j] = *(uint32_t*)&lo;
+          }
           psum += a + b;
         }
       } else {
@@ -271,13 +287,19 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
           __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
           pw[j] = *(uint32_t*)&h;
           float2 back = __bfloat1622float2(h);
-          psum += back.x + back.y;
+          if constexpr (SPLITP) {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(a - back.x, b - back.y);
+            pl[j] = *(uint32_t*)&lo;
+            psum += a + b;
+          } else {
+            psum += back.x + back.y;
+          }
         }
       }
       l = l * corr + psum;
       if (__any_sync(0xffffffffu, need && !first) && i > 0) {
         // O may only be touched once the previous P V has completed
-        if (!mbar_wait(&pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+        if (!mbar_wait(&pv_done[(i - 1) % NPBUF], ((i - 1) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
         tc_fence_after();
 #pragma unroll 1
         for (int c0 = 0; c0 < DV; c0 += 32) {
@@ -292,20 +314,25 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
         tmem_st_wait();
       }
       if (i >= NPBUF) {
-        // this P buffer was last read by the P V of block i - 2
-        if (!mbar_wait(&pv_done[pb], ((i - NPBUF) >> 1) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+        // this P buffer was last read by the P V of block i - NPBUF
+        if (!mbar_wait(&pv_done[pb], ((i - NPBUF) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
       }
       // P (bf16) -> shared memory: chunk c holds keys 8c..8c+7 of every row, 16 bytes per row
 #pragma unroll
       for (int c = 0; c < KB / 8; ++c)
-        *(uint4*)(sP + pb * P_BYTES + c * (TR * 16) + r * 16) = make_uint4(pw[4 * c], pw[4 * c + 1], pw[4 * c + 2], pw[4 * c + 3]);
+        *(uint4*)(sP + pb * C::P_STAGE + c * (TR * 16) + r * 16) = make_uint4(pw[4 * c], pw[4 * c + 1], pw[4 * c + 2], pw[4 * c + 3]);
+      if constexpr (SPLITP) {
+#pragma unroll
+        for (int c = 0; c < KB / 8; ++c)
+          *(uint4*)(sP + pb * C::P_STAGE + P_BYTES + c * (TR * 16) + r * 16) = make_uint4(pl[4 * c], pl[4 * c + 1], pl[4 * c + 2], pl[4 * c + 3]);
+      }
       fence_proxy_async();       // make the generic-proxy writes of P visible to the tensor core
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&p_full[pb]);
     }
     // ------------------------------------------------------------------ write out
-    if (!mbar_wait(&pv_done[(nblk - 1) & 1], ((nblk - 1) >> 1) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+    if (!mbar_wait(&pv_done[(nblk - 1) % NPBUF], ((nblk - 1) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
     tc_fence_after();
     const float inv_l = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll 1
@@ -314,7 +341,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       tmem_ld_32x32b_x32(tmem_O + lane_off + c0, o);
       tmem_ld_wait();
       if (row_ok) {
-        __nv_bfloat16* dst = p.out + ((int64_t)(tok0 + r) * p.Hq + head) * DV + c0;
+        __nv_bfloat16* dst = p.out + (int64_t)(tok0 + r) * p.out_ld + head * DV + c0;
         uint4 w[4];
         uint32_t* wp = (uint32_t*)w;
 #pragma unroll
@@ -357,11 +384,12 @@ int make_cache_map(CUtensorMap* m, const void* cache, int heads, int hd, int num
   return r == CUDA_SUCCESS ? MARY_OK : MARY_ERR_CUDA;
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool SPLITP>
 int launch_fa(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const FaParams& p, int NB, cudaStream_t s) {
   static MarySmemSlots smem_set = {};
-  if (int rc = mary_ensure_dyn_smem((const void*)fa_prefill_kernel<DK, DV>, FaCfg<DK, DV>::SMEM, &smem_set)) return rc;
-  fa_prefill_kernel<DK, DV><<<dim3(NB, p.Hq), NTHREADS, FaCfg<DK, DV>::SMEM, s>>>(tq, tk, tv, p);
+  constexpr int SMEM = FaCfg<DK, DV, SPLITP>::SMEM;
+  if (int rc = mary_ensure_dyn_smem((const void*)fa_prefill_kernel<DK, DV, SPLITP>, SMEM, &smem_set)) return rc;
+  fa_prefill_kernel<DK, DV, SPLITP><<<dim3(NB, p.Hq), NTHREADS, SMEM, s>>>(tq, tk, tv, p);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }
@@ -378,12 +406,13 @@ MARY_API int mary_attention_prefill_supported(int DK, int DV) {
 // q [T, Hq, DK] bf16 contiguous; kcache [pages, page_size (16 or 64), Hkv, DK] and vcache [.., Hkv, DV] bf16 with element strides per token
 // and per page (heads contiguous inside a token row); out [T, Hq, DV] bf16.  blk_seq / blk_tok0: NB tiles of at most 128 query
 // tokens that never cross a sequence.  Causal with the last query token of a sequence at position kv_len - 1; window > 0 keeps
-// keys (pos - window, pos].  Returns MARY_ERR_BAD_ARG for head dims without an instantiation.
+// keys (pos - window, pos].  out_ld: elements between the output rows of two tokens (0: Hq * DV; a multiple of 8).  split_p: softmax
+// weights with 16 significant bits (equal key and value widths only).  Returns MARY_ERR_BAD_ARG for head dims without an instantiation.
 MARY_API int mary_attention_prefill(const void* q, const void* kcache, const void* vcache, void* out, const int* page_table,
                                     const int* kv_len, const int* q_start, const int* blk_seq, const int* blk_tok0, int NB, int T, int Hq,
                                     int Hkv, int DK, int DV, int num_pages, int max_pages, int64_t k_tok_stride, int64_t k_page_stride,
                                     int64_t v_tok_stride, int64_t v_page_stride, int window, float scale, int page_size,
-                                    cudaStream_t s) {
+                                    int64_t out_ld, int split_p, cudaStream_t s) {
   if (NB <= 0) return MARY_OK;
   if (!mary_attention_prefill_supported(DK, DV) || Hkv < 1 || Hq % Hkv || (page_size != PAGE && page_size != KB)) return MARY_ERR_BAD_ARG;
   if ((k_tok_stride * 2) % 16 || (k_page_stride * 2) % 16 || (v_tok_stride * 2) % 16 || (v_page_stride * 2) % 16) return MARY_ERR_BAD_ARG;
@@ -395,9 +424,16 @@ MARY_API int mary_attention_prefill(const void* q, const void* kcache, const voi
   FaParams p;
   p.page_table = page_table; p.kv_len = kv_len; p.q_start = q_start; p.blk_seq = blk_seq; p.blk_tok0 = blk_tok0;
   p.out = (__nv_bfloat16*)out; p.max_pages = max_pages; p.Hq = Hq; p.Hkv = Hkv; p.window = window; p.page = page_size;
+  p.out_ld = out_ld > 0 ? out_ld : (int64_t)Hq * DV;
+  if (p.out_ld % 8 || ((uintptr_t)out & 15) || (split_p && DK != DV)) return MARY_ERR_BAD_ARG;
   p.scale_log2 = scale * 1.4426950408889634f; p.status = mary_status_ptr();
-  if (DK == 64) return launch_fa<64, 64>(tq, tk, tv, p, NB, s);
-  if (DK == 128) return launch_fa<128, 128>(tq, tk, tv, p, NB, s);
-  if (DK == 192) return launch_fa<192, 128>(tq, tk, tv, p, NB, s);
-  return launch_fa<256, 256>(tq, tk, tv, p, NB, s);
+  if (split_p) {
+    if (DK == 64) return launch_fa<64, 64, true>(tq, tk, tv, p, NB, s);
+    if (DK == 128) return launch_fa<128, 128, true>(tq, tk, tv, p, NB, s);
+    return launch_fa<256, 256, true>(tq, tk, tv, p, NB, s);
+  }
+  if (DK == 64) return launch_fa<64, 64, false>(tq, tk, tv, p, NB, s);
+  if (DK == 128) return launch_fa<128, 128, false>(tq, tk, tv, p, NB, s);
+  if (DK == 192) return launch_fa<192, 128, false>(tq, tk, tv, p, NB, s);
+  return launch_fa<256, 256, false>(tq, tk, tv, p, NB, s);
 }

@@ -353,6 +353,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tm_r, const __grid_constant
                 for (int j = 0; j < 32; ++j)
                   if (j0 + j < p.rows_c) dst[j] = __float2bfloat16(v[j] + (p.bias ? p.bias[j0 + j] : 0.f));
               }
+            } else if (epi == EPI_STORE_F32 && j0 + 32 <= p.rows_c && ((uintptr_t)((float*)p.out + o) & 15) == 0) {
+              float4* dst = (float4*)((float*)p.out + o);
+#pragma unroll
+              for (int j = 0; j < 8; ++j) {
+                const float* b = p.bias ? p.bias + j0 + 4 * j : nullptr;
+                dst[j] = make_float4(v[4 * j] + (b ? b[0] : 0.f), v[4 * j + 1] + (b ? b[1] : 0.f), v[4 * j + 2] + (b ? b[2] : 0.f), v[4 * j + 3] + (b ? b[3] : 0.f));
+              }
             } else if (epi == EPI_STORE_F32) {
               for (int j = 0; j < 32; ++j)
                 if (j0 + j < p.rows_c) ((float*)p.out)[o + j] = v[j] + (p.bias ? p.bias[j0 + j] : 0.f);

@@ -1,0 +1,85 @@
+// General matrix product on the CUDA cores with 32-bit accumulation: out[M, N] = alpha * X[M, K] W[N, K]^T (+ out).  It serves 32-bit
+// models (no reduced-precision tensor-core mode is involved) and the shapes that TMA addressing excludes (row pitches that are not
+// multiples of 16 bytes); everything else belongs to gemm_bf16.cu.  64 x 64 tile, 256 threads, 4 x 4 outputs each, register prefetch.
+#include "host_utils.h"
+#include "typed.cuh"
+
+using namespace mary;
+
+namespace {
+
+constexpr int BM = 64, BN = 64, BK = 16, NT = 256;
+
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(NT) gemm_simt_kernel(const TI* __restrict__ X, const TI* __restrict__ W, TO* __restrict__ out, int M, int N, int K,
+                                                       int64_t ldx, int64_t ldw, int64_t ldo, float alpha, int accumulate) {
+  pdl_sync();
+  __shared__ float sx[2][BK][BM + 4], sw[2][BK][BN + 4];
+  const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
+  const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
+  const int lk = threadIdx.x % BK, lr = threadIdx.x / BK;          // loader: one k, rows lr, lr + 16, ...
+  float acc[4][4] = {};
+  float px[4], pw[4];
+  auto fetch = [&](int k0) {
+    const int k = k0 + lk;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int m = m0 + lr + 16 * i, n = n0 + lr + 16 * i;
+      px[i] = (k < K && m < M) ? to_f<TI>(X[(int64_t)m * ldx + k]) : 0.f;
+      pw[i] = (k < K && n < N) ? to_f<TI>(W[(int64_t)n * ldw + k]) : 0.f;
+    }
+  };
+  auto stash = [&](int b) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { sx[b][lk][lr + 16 * i] = px[i]; sw[b][lk][lr + 16 * i] = pw[i]; }
+  };
+  fetch(0);
+  stash(0);
+  __syncthreads();
+  const int nk = (K + BK - 1) / BK;
+  for (int kb = 0; kb < nk; ++kb) {
+    const int b = kb & 1;
+    if (kb + 1 < nk) fetch((kb + 1) * BK);
+#pragma unroll
+    for (int k = 0; k < BK; ++k) {
+      const float4 a = *(const float4*)&sx[b][k][ty * 4], c = *(const float4*)&sw[b][k][tx * 4];
+      const float av[4] = {a.x, a.y, a.z, a.w}, cv[4] = {c.x, c.y, c.z, c.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], cv[j], acc[i][j]);
+    }
+    if (kb + 1 < nk) stash(b ^ 1);
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= M) continue;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= N) continue;
+      TO* o = out + (int64_t)m * ldo + n;
+      const float v = alpha * acc[i][j];
+      *o = from_f<TO>(accumulate ? to_f<TO>(*o) + v : v);
+    }
+  }
+}
+
+}  // namespace
+
+// x_f32: X and W are f32 (else both bf16); out_f32: out is f32 (else bf16)
+MARY_API int mary_gemm_simt(const void* X, const void* W, void* out, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldo, float alpha,
+                            int accumulate, int x_f32, int out_f32, cudaStream_t s) {
+  if (M <= 0) return MARY_OK;
+  if (N <= 0 || K <= 0 || (M + BM - 1) / BM > 65535) return MARY_ERR_BAD_ARG;
+  const dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
+  using B = __nv_bfloat16;
+  if (x_f32 && out_f32) MARY_LAUNCH((gemm_simt_kernel<float, float>), grid, NT, 0, s, (const float*)X, (const float*)W, (float*)out, M, N, K, ldx, ldw, ldo, alpha, accumulate);
+  else if (x_f32) return MARY_ERR_BAD_ARG;
+  else if (out_f32) MARY_LAUNCH((gemm_simt_kernel<B, float>), grid, NT, 0, s, (const B*)X, (const B*)W, (float*)out, M, N, K, ldx, ldw, ldo, alpha, accumulate);
+  else MARY_LAUNCH((gemm_simt_kernel<B, B>), grid, NT, 0, s, (const B*)X, (const B*)W, (B*)out, M, N, K, ldx, ldw, ldo, alpha, accumulate);
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
+}

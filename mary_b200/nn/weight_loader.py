@@ -39,6 +39,11 @@ class WeightLoader:
             raise LookupError("leaf views exist only for pile-backed loaders")
         return self.index.leaf(name)
 
+    def shape(self, name: str) -> tuple[int, ...]:
+        if self.index is not None:
+            return tuple(int(d) for d in self.index.leaf(name).dims)
+        return self._file_of[name].info(name)[1]
+
     def load_host_f32(self, name: str) -> np.ndarray:
         if self.index is not None:
             l = self.index.leaf(name)

@@ -39,11 +39,12 @@ def linear(x, w, bias=None):
     return _k().linear(x, w, bias) if _cuda(x) else ref.linear(x, w, bias)
 
 
-def linear_f32(x, w):
-    """``x @ w^T`` with an f32 result (router logits, row-parallel partial sums)."""
+def linear_f32(x, w, alpha: float = 1.0):
+    """``alpha * x @ w^T`` with an f32 result (router logits, row-parallel partial sums, inputs of a post-norm)."""
     if _cuda(x):
-        return _k().linear_f32(x, w)
-    return ref.linear(x.float(), w.float())
+        return _k().linear_f32(x, w, alpha=alpha)
+    y = ref.linear(x.float(), w.float())
+    return y if alpha == 1.0 else y * alpha
 
 
 def qk_norm_rope_append(qkv, n_q, n_kv, head_dim, q_norm, k_norm, v_norm: bool, inv_freq, meta, kcache, vcache, eps):
@@ -233,3 +234,65 @@ def quantize_nvfp4(x):
 
 def short_conv(x, w, history=None):
     return _k().short_conv(x, w, history) if _cuda(x) else ref.short_conv(x, w, history)
+
+
+# --------------------------------------------------------------------------- 32-bit residual stream, exact attention, recurrent layers
+def _h():
+    from . import cuda_hybrid
+    return cuda_hybrid
+
+
+def rows_buffer(T: int, n: int, like):
+    """An uninitialised ``[T, n]`` row view whose pitch keeps every row 16-byte aligned."""
+    return torch.empty(T, (n + 7) // 8 * 8, dtype=like.dtype, device=like.device)[:, :n]
+
+
+def embed32(ids, table, scale=1.0):
+    """Rows of the embedding table as ``(residual stream f32, activations)``."""
+    return _h().embed32(ids, table, scale) if _cuda(table) else ref.embed32(ids, table, scale)
+
+
+def post_norm_add(a, w_post, h, w_next, eps):
+    """Post-norm residual step on a 32-bit stream: ``h += rms(a) * w_post`` in place; returns the next sublayer's input in the
+    activation type: ``rms(h) * w_next``, or ``h`` itself with ``w_next=None``."""
+    return _h().post_norm_add(a, w_post, h, w_next, eps) if _cuda(h) else ref.post_norm_add(a, w_post, h, w_next, eps)
+
+
+def rmsnorm32(h, w, eps):
+    """RMS norm of a 32-bit stream into the activation type."""
+    return _h().rmsnorm32(h, w, eps) if _cuda(h) else ref.rmsnorm32(h, w, eps)
+
+
+def qk_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps):
+    """Per-head RMS norm of queries and keys (no rotation), keys and values appended to the cache; ``q``, ``k``, ``v`` are row views of
+    one projection, keys ``dk`` and values ``dv`` wide.  Returns ``q [T, n_q, dk]``."""
+    f = _h().qk_norm_append if _cuda(q) else ref.qk_norm_append
+    return f(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps)
+
+
+def attention_exact(q, kcache, vcache, meta, scale, out=None):
+    """Causal paged attention whose scores, softmax weights and sums stay in 32 bits, for any head widths: ``[T, Hq * DV]``."""
+    if _cuda(q):
+        return _h().attention_exact(q, kcache, vcache, meta, scale, out)
+    o = ref.paged_attention(q, kcache, vcache, meta, scale).reshape(q.shape[0], -1)
+    if out is None:
+        return o
+    out.copy_(o)
+    return out
+
+
+def decayed_linear_attention(q, k, v, gate, low, a2, a2_bias, inv_tau, gain, state, meta, H, dk, dv, eps, out_scale, out):
+    """``S <- diag(alpha) S + k v^T``, ``o = S^T q`` per head with ``alpha = sigmoid(low a2^T + a2_bias) ** inv_tau`` per key channel and
+    ``q`` scaled by ``dk ** -0.5``; then ``rms(o) * gain * silu(gate) * out_scale`` into ``out [T, H * dv]``.  Continues from and updates
+    ``state [slots, H, dv, pitch]`` (f32, one column of key channels per value channel)."""
+    f = _h().decayed_linear_attention if _cuda(q) else ref.decayed_linear_attention
+    return f(q, k, v, gate, low, a2, a2_bias, inv_tau, gain, state, meta, H, dk, dv, eps, out_scale, out)
+
+
+def gated_delta_attention(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, ring, state, meta, HK, H, dk, dv, eps, out_scale, out):
+    """Gated delta rule with short convolutions: ``x [T, 2 HK dk + H dv]`` holds the q, k, v inputs; ``silu(conv(x))``, unit q and k per
+    head, ``beta = sigmoid(b_in)``, ``g = exp(-exp(a_log) softplus(a_in + dt_bias))``; ``S <- g S``, ``S <- S + k (beta (v - S^T k))^T``,
+    ``o = S^T q``; then ``rms(o) * gain * silu(gate) * out_scale`` into ``out``.  ``ring [slots, taps, channels]`` keeps the last inputs of
+    the convolutions by absolute position, ``state`` is laid out as above."""
+    f = _h().gated_delta_attention if _cuda(x) else ref.gated_delta_attention
+    return f(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, ring, state, meta, HK, H, dk, dv, eps, out_scale, out)

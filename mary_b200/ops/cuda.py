@@ -54,8 +54,8 @@ def declare(name: str, sig: str, ret64: bool = False):
     if ret64:
         _RET64.add(name)
     global _lib
-    if _lib is not None:
-        fn = getattr(_lib, name)
+    fn = getattr(_lib, name, None) if _lib is not None else None
+    if fn is not None:
         fn.argtypes = [_CT[c] for c in sig]
         fn.restype = ctypes.c_int64 if ret64 else ctypes.c_int32
 
@@ -168,7 +168,7 @@ def _sk_workspace(dev):
     return _SK_WS[key]
 
 
-def gemm_splitk(x, w, split_k: int, out=None, f32: bool = False, bias=None, swap: int = -1):
+def gemm_splitk(x, w, split_k: int, out=None, f32: bool = False, bias=None, swap: int = -1, alpha: float = 1.0):
     """``x @ w^T`` with K cut into ``split_k`` slices reduced inside the kernel (every slice adds into an f32 accumulator tile in
     scratch; the slice that finishes last converts and stores it and leaves the scratch zero): no zero-fill, no cast pass.  ``split_k=0`` is stream-K: the K-blocks of all tiles are dealt out in
     equal contiguous runs, one per SM, so every SM streams the same share of the weights whatever the tile count.  Falls back
@@ -181,10 +181,10 @@ def gemm_splitk(x, w, split_k: int, out=None, f32: bool = False, bias=None, swap
     ws, cnt = _sk_workspace(x.device)
     if out is None:
         out = _empty(M, N, dtype=torch.float32 if f32 else torch.bfloat16, device=x.device)
-    rc = lib().mary_gemm_bf16_splitk(_p(x), _p(w), _p(out), M, N, K, x.stride(0), w.stride(0), out.stride(0), _p(bias), 1.0, int(f32),
+    rc = lib().mary_gemm_bf16_splitk(_p(x), _p(w), _p(out), M, N, K, x.stride(0), w.stride(0), out.stride(0), _p(bias), alpha, int(f32),
                                      split_k, swap, _p(ws), ws.numel(), _p(cnt), cnt.numel(), _stream())
     if rc == 4:                                             # scratch too small for this shape
-        red = gemm(x, w, epi="red", split_k=split_k or _auto_split_k(M, N, K))
+        red = gemm(x, w, alpha=alpha, epi="red", split_k=split_k or _auto_split_k(M, N, K))
         if bias is not None:
             red += bias
         out.copy_(red)
@@ -231,6 +231,11 @@ def _linear(x, w, bias=None):
     if x2.stride(-1) != 1:
         x2 = x2.contiguous()
     M, K = x2.shape
+    if x2.dtype == torch.float32 or K % 8 or x2.stride(0) % 8 or w.stride(0) % 8:
+        # 32-bit models, and row pitches that TMA cannot address: the CUDA-core product
+        from .cuda_hybrid import gemm_simt
+        out = gemm_simt(x2, w)
+        return (out if bias is None else out + bias.to(out.dtype)).reshape(*shp[:-1], w.shape[0])
     if (M == 1 and bias is None and K % 8 == 0 and K <= 8192 and w.shape[0] * K * 2 <= MATVEC_MAX_BYTES and w.stride(1) == 1
             and w.stride(0) % 8 == 0 and x2.dtype == torch.bfloat16 and w.dtype == torch.bfloat16):
         return step_matvec(x2, w).reshape(*shp[:-1], w.shape[0])
@@ -239,16 +244,22 @@ def _linear(x, w, bias=None):
     return out.reshape(*shp[:-1], w.shape[0])
 
 
-def linear_f32(x, w, split_k: int | None = None):
+def linear_f32(x, w, split_k: int | None = None, alpha: float = 1.0):
     """Row-parallel style GEMM whose f32 result feeds a norm kernel directly (no bf16 rounding in between)."""
     M, K = x.shape
+    if x.dtype == torch.float32 or K % 8 or x.stride(0) % 8 or w.stride(0) % 8:
+        from .cuda_hybrid import gemm_simt
+        return gemm_simt(x, w, alpha=alpha, out_f32=True)
     sk = split_k or _auto_split_k(M, w.shape[0], K)
     with static_weights:
-        return gemm_splitk(x, w, 0 if split_k is None else sk, f32=True) if sk > 1 else gemm(x, w, epi="f32")
+        return gemm_splitk(x, w, 0 if split_k is None else sk, f32=True, alpha=alpha) if sk > 1 else gemm(x, w, alpha=alpha, epi="f32")
 
 
 def linear_glu(x, w_gu, act: str = "geglu"):
     M = x.shape[0]
+    if x.dtype == torch.float32 or x.shape[1] % 8 or w_gu.shape[0] % 16:
+        from .cuda_hybrid import glu_any
+        return glu_any(linear(x, w_gu), act)
     with static_weights:
         if M <= 128:
             return gemm(x, w_gu, glu=act)
@@ -314,15 +325,20 @@ def short_conv(x, w, history=None):
 
 
 # --------------------------------------------------------------------------- attention
-def _q_blocks(meta, rq: int):
-    key = ("qblk", rq)
+DECODE_GROUP_ROWS = 8
+
+
+def _q_blocks(meta, rq: int, group: str | None = None):
+    """Blocks of at most ``rq`` query tokens of one sequence: ``(sequence, first row, number of blocks)``.  ``group``: only the sequences
+    that bring more (``"prefill"``) or at most (``"decode"``) ``DECODE_GROUP_ROWS`` tokens."""
+    key = ("qblk", rq, group)
     cache = meta.__dict__.setdefault("_cache", {})
     if key not in cache:
         import numpy as np
         seqs, q0 = [], []
         start = 0
         for s, n in enumerate(meta.q_lens_host.tolist()):
-            for b in range(0, n, rq):
+            for b in range(0, n if group is None or (group == "prefill") == (n > DECODE_GROUP_ROWS) else 0, rq):
                 seqs.append(s)
                 q0.append(start + b)
             start += n
@@ -332,32 +348,36 @@ def _q_blocks(meta, rq: int):
     return cache[key]
 
 
-declare("mary_paged_attention_decode", "ppppppppp" + "iii" + "llll" + "iiiiii" + "ff" + "ps")
+declare("mary_paged_attention_decode", "ppppppppp" + "iii" + "llll" + "iiiiii" + "ff" + "pls")
 
 
 DECODE_TARGET_CTAS = 2368      # CTAs the decode attention kernel aims for when it picks the number of kv splits (16 per SM)
 
 
-def _paged_attention_decode(q, kcache, vcache, meta, scale, window, softcap, nsplit):
+def _paged_attention_decode(q, kcache, vcache, meta, scale, window, softcap, nsplit, out=None, group=None):
     """Decode-shaped batches (few rows per kv head, equal K and V widths of 64/128/256): the bandwidth-oriented kernel."""
     T, Hq, D = q.shape
     Hkv = kcache.shape[2]
     G = Hq // Hkv
     cap = 4 if D == 256 else 8
     rq = max(1, min(cap // G, meta.max_q_len))
-    blk_seq, blk_q0, NB = _q_blocks(meta, rq)
+    blk_seq, blk_q0, NB = _q_blocks(meta, rq, group)
     if nsplit is None:
         want = max(1, DECODE_TARGET_CTAS // max(1, NB * Hkv))
         span = meta.max_kv_len if window <= 0 else min(meta.max_kv_len, window + rq)
         nsplit = max(1, min(want, 32, span // 64))
-    out = _empty(T, Hq, D, dtype=torch.bfloat16, device=q.device)
+    ld = 0                                        # ``out``: a row view [T, Hq * D] of any pitch
+    if out is None:
+        out = _empty(T, Hq, D, dtype=torch.bfloat16, device=q.device)
+    else:
+        ld = out.stride(0)
     scratch = None
     if nsplit > 1:
         scratch = _empty(lib().mary_paged_attention_scratch_floats(NB, Hkv, nsplit, D), dtype=torch.float32, device=q.device)
     check(lib().mary_paged_attention_decode(_p(q.contiguous()), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len),
                                             _p(meta.q_start), _p(blk_seq), _p(blk_q0), NB, meta.page_table.shape[1], meta.page_size,
                                             kcache.stride(1), kcache.stride(0), vcache.stride(1), vcache.stride(0), Hq, Hkv, D, rq,
-                                            nsplit, window, scale, softcap, _p(scratch), _stream()), "paged_attention_decode")
+                                            nsplit, window, scale, softcap, _p(scratch), ld, _stream()), "paged_attention_decode")
     return out
 
 
@@ -446,16 +466,17 @@ def gqa_decode_tc(q, kcache, vcache, meta, scale, window=0, softcap=0.0, nsplit=
     return out
 
 
-declare("mary_attention_prefill", "ppppppppp" + "iiiiiiii" + "llll" + "ifis")
+declare("mary_attention_prefill", "ppppppppp" + "iiiiiiii" + "llll" + "ifi" + "lis")
 declare("mary_attention_prefill_supported", "ii")
 PREFILL_MIN_ROWS = 48     # mean query tokens per sequence from which the 128-row tensor-core tiles pay off
 
 
-def attention_prefill(q, kcache, vcache, meta, scale, window=0):
+def attention_prefill(q, kcache, vcache, meta, scale, window=0, out=None, split_p: bool = False, group=None):
     """Causal / sliding-window attention of whole query blocks on the tensor cores (``csrc/kernels/attention_fa.cu``):
     ``q[T, Hq, DK]``, caches ``[pages, page, Hkv, D]``; 128 query tokens of one head per CTA.  A cache with 64-token pages is
     streamed with one TMA operation per 64-key stage; a cache with smaller pages is first regrouped into 64-token pages (one
-    gather, small beside the attention arithmetic) when the host knows the sequence lengths."""
+    gather, small beside the attention arithmetic) when the host knows the sequence lengths.
+    ``split_p`` keeps 16 significant bits of the softmax weights; ``out`` may be a row view ``[T, Hq * DV]``; ``group``: see ``_q_blocks``."""
     T, Hq, DK = q.shape
     Hkv, DV = kcache.shape[2], vcache.shape[-1]
     ps = meta.page_size
@@ -466,12 +487,16 @@ def attention_prefill(q, kcache, vcache, meta, scale, window=0):
         vcache = vcache[pick].view(-1, 64, Hkv, DV)
         ps = 64
     assert ps in (16, 64)
-    blk_seq, blk_tok0, NB = _q_blocks(meta, 128)
-    out = _empty(T, Hq, DV, dtype=torch.bfloat16, device=q.device)
+    blk_seq, blk_tok0, NB = _q_blocks(meta, 128, group)
+    ld = 0
+    if out is None:
+        out = _empty(T, Hq, DV, dtype=torch.bfloat16, device=q.device)
+    else:
+        ld = out.stride(0)
     check(lib().mary_attention_prefill(_p(q.contiguous()), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len),
                                        _p(meta.q_start), _p(blk_seq), _p(blk_tok0), NB, T, Hq, Hkv, DK, DV, kcache.shape[0],
                                        meta.page_table.shape[1], kcache.stride(1), kcache.stride(0), vcache.stride(1), vcache.stride(0),
-                                       int(window), float(scale), ps, _stream()), "attention_prefill")
+                                       int(window), float(scale), ps, ld, int(split_p), _stream()), "attention_prefill")
     return out
 
 
@@ -573,7 +598,7 @@ def sample_top_k_top_p(logits, temperature: float, top_k: int = 0, top_p: float 
 
 
 def lm_head_argmax(h, table, softcap=0.0, vocab_limit=None):
-    logits = gemm(h.contiguous(), table, epi="f32")
+    logits = linear_f32(h.contiguous(), table, split_k=1)
     if vocab_limit:
         logits = logits[:, :vocab_limit]
     return argmax(logits, softcap)

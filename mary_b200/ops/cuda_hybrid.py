@@ -1,0 +1,241 @@
+"""CUDA wrappers of the ops that decoders with a 32-bit residual stream, exact attention and recurrent layers are made of.
+
+Each wrapper serves bf16 and 32-bit activations (the kernels are instantiated for both): the storage type follows the tensors it is
+given.  Nothing here converts a 32-bit product to a reduced-precision mode."""
+from __future__ import annotations
+
+import torch
+
+from ..utils.canary import empty as _empty
+from . import cuda as K
+from .cuda import _p, _stream, check, declare, lib
+
+declare("mary_gemm_simt", "pppiiilllfiiis")
+declare("mary_embed32", "ppppiifiis")
+declare("mary_post_norm_add", "plppppiifis")
+declare("mary_rmsnorm32", "pppiifis")
+declare("mary_glu_any", "ppiiiis")
+declare("mary_qk_norm_append", "ppp" + "liiii" + "pppppp" + "fil" + "is")
+declare("mary_attention_general", "ppppppppp" + "iii" + "lllll" + "iiiiiii" + "fpis")
+declare("mary_attention_general_rows", "i")
+declare("mary_attention_general_scratch_floats", "iiiii", ret64=True)
+declare("mary_channel_decay", "pli" + "ppp" + "iifis")
+declare("mary_delta_prep", "pl" + "pppppp" + "pppp" + "ppppp" + "iiiiii" + "is")
+declare("mary_conv_history", "plpppp" + "iiiis")
+declare("mary_gated_head_norm", "pplppl" + "iiiffis")
+declare("mary_decay_scan", "pppppp" + "ppp" + "illl" + "iiifis")
+declare("mary_delta_scan", "ppppppp" + "ppp" + "illl" + "iiiifs")
+declare("mary_decay_step", "ppppp" + "li" + "ppfp" + "plfp" + "ppp" + "iiiiffis")
+declare("mary_delta_step", "plppi" + "pppppp" + "plp" + "ppp" + "iiiiiffis")
+
+
+def _f32(t) -> int:
+    if t.dtype not in (torch.float32, torch.bfloat16):
+        raise TypeError(f"expected a bf16 or f32 tensor, got {t.dtype}")
+    return int(t.dtype == torch.float32)
+
+
+def _rows(t):
+    """``(tensor, pitch)`` of a row view ``[T, n]`` whose last dimension is contiguous."""
+    assert t.dim() == 2 and t.stride(1) == 1
+    return _p(t), t.stride(0)
+
+
+def tensor_core_ok(x, w) -> bool:
+    """Whether the TMA-fed tensor-core GEMM can address ``x [M, K]`` and ``w [N, K]``."""
+    return (x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.shape[1] % 8 == 0 and x.stride(0) % 8 == 0 and w.stride(0) % 8 == 0
+            and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
+
+
+def gemm_simt(x, w, out=None, alpha: float = 1.0, accumulate: bool = False, out_f32: bool = False):
+    """``alpha * x @ w^T`` (added to ``out`` when ``accumulate``) with 32-bit products and sums, any shape."""
+    M, Kd = x.shape
+    N = w.shape[0]
+    assert x.dtype == w.dtype and w.shape[1] == Kd and x.stride(1) == 1 and w.stride(1) == 1
+    if out is None:
+        out = _empty(M, N, dtype=torch.float32 if out_f32 else x.dtype, device=x.device)
+    check(lib().mary_gemm_simt(_p(x), _p(w), _p(out), M, N, Kd, x.stride(0), w.stride(0), out.stride(0), alpha, int(accumulate), _f32(x), _f32(out),
+                               _stream()), "gemm_simt")
+    return out
+
+
+def embed32(ids, table, scale: float = 1.0):
+    """``(h f32, x)``: the rows of the embedding table as the residual stream and in the activation type."""
+    ids = ids.to(torch.int32)
+    T, H = ids.shape[0], table.shape[1]
+    h = _empty(T, H, dtype=torch.float32, device=table.device)
+    x = _empty(T, H, dtype=table.dtype, device=table.device)
+    check(lib().mary_embed32(_p(ids), _p(table), _p(h), _p(x), T, H, scale, table.shape[0], _f32(table), _stream()), "embed32")
+    return h, x
+
+
+def post_norm_add(a, w_post, h, w_next, eps):
+    x = _empty(h.shape, dtype=w_post.dtype, device=h.device)
+    pa, lda = _rows(a)
+    assert a.dtype == torch.float32 and h.dtype == torch.float32 and h.is_contiguous()
+    check(lib().mary_post_norm_add(pa, lda, _p(w_post), _p(h), _p(w_next), _p(x), h.shape[0], h.shape[1], eps, _f32(w_post), _stream()), "post_norm_add")
+    return x
+
+
+def rmsnorm32(h, w, eps):
+    y = _empty(h.shape, dtype=w.dtype, device=h.device)
+    check(lib().mary_rmsnorm32(_p(h), _p(w), _p(y), h.shape[0], h.shape[1], eps, _f32(w), _stream()), "rmsnorm32")
+    return y
+
+
+def glu_any(gate_up, act: str):
+    T, F2 = gate_up.shape
+    out = _empty(T, F2 // 2, dtype=gate_up.dtype, device=gate_up.device)
+    check(lib().mary_glu_any(_p(gate_up.contiguous()), _p(out), T, F2 // 2, {"geglu": 0, "swiglu": 1}[act], _f32(gate_up), _stream()), "glu_any")
+    return out
+
+
+def qk_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps):
+    T = q.shape[0]
+    qo = _empty(T, n_q, dk, dtype=q.dtype, device=q.device)
+    (pq, ld), (pk, l2), (pv, l3) = _rows(q), _rows(k), _rows(v)
+    assert ld == l2 == l3 and kcache.is_contiguous() and vcache.is_contiguous() and kcache.dtype == q.dtype
+    check(lib().mary_qk_norm_append(pq, pk, pv, ld, n_q, n_kv, dk, dv, _p(q_gain), _p(k_gain), _p(meta.slot_mapping), _p(qo), _p(kcache), _p(vcache),
+                                    eps, T, kcache.shape[0] * kcache.shape[1], _f32(q), _stream()), "qk_norm_append")
+    return qo
+
+
+# --------------------------------------------------------------------------- exact attention
+DECODE_ROWS = K.DECODE_GROUP_ROWS         # sequences with at most this many query tokens take the decode kernel, the others the prefill kernel
+
+
+def attention_general(q, kcache, vcache, meta, scale, out, group=None, nsplit=None, window: int = 0):
+    """Any head widths, group size and storage type; ``group`` restricts the call to ``"prefill"`` or ``"decode"`` sequences."""
+    T, Hq, DK = q.shape
+    Hkv, DV = kcache.shape[2], vcache.shape[3]
+    G = Hq // Hkv
+    rq = max(1, min(lib().mary_attention_general_rows(G), meta.max_q_len))
+    blk_seq, blk_q0, NB = K._q_blocks(meta, rq, group)
+    if NB == 0:
+        return out
+    if nsplit is None:
+        want = max(1, 296 // max(1, NB * Hkv * ((G + 15) // 16)))
+        span = meta.max_kv_len if window <= 0 else min(meta.max_kv_len, window + rq)
+        nsplit = max(1, min(want, 32, span // 128))
+    scratch = None
+    if nsplit > 1:
+        scratch = _empty(lib().mary_attention_general_scratch_floats(NB, Hq, Hkv, nsplit, DV), dtype=torch.float32, device=q.device)
+    check(lib().mary_attention_general(_p(q), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len), _p(meta.q_start), _p(blk_seq),
+                                       _p(blk_q0), NB, meta.page_table.shape[1], meta.page_size, kcache.stride(1), kcache.stride(0), vcache.stride(1),
+                                       vcache.stride(0), out.stride(0), Hq, Hkv, DK, DV, rq, nsplit, window, scale, _p(scratch), _f32(q), _stream()),
+          "attention_general")
+    return out
+
+
+def attention_exact(q, kcache, vcache, meta, scale, out=None):
+    """Causal attention with scores, softmax weights and sums in 32 bits: the tensor-core prefill kernel with two-term weights for
+    sequences that bring more than ``DECODE_ROWS`` tokens, the bandwidth-oriented decode kernel for the others, the general kernel for
+    32-bit tensors and for head shapes those have no instantiation for.  ``out`` may be a row view ``[T, Hq * DV]``."""
+    T, Hq, DK = q.shape
+    Hkv, DV = kcache.shape[2], vcache.shape[3]
+    assert q.is_contiguous() and kcache.is_contiguous() and vcache.is_contiguous() and kcache.shape[1] == meta.page_size
+    if out is None:
+        out = _empty(T, Hq * DV, dtype=q.dtype, device=q.device)
+    assert out.stride(1) == 1
+    bf16 = q.dtype == torch.bfloat16 and DK == DV
+    fast_prefill = bf16 and DK in (64, 128, 256) and meta.page_size in (16, 64) and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
+    fast_decode = bf16 and DK in (64, 128, 256) and Hq // Hkv <= (4 if DK == 256 else 8)
+    if not (fast_prefill or fast_decode):
+        return attention_general(q, kcache, vcache, meta, scale, out)
+    if meta.max_q_len > DECODE_ROWS:
+        if fast_prefill:
+            K.attention_prefill(q, kcache, vcache, meta, scale, out=out, split_p=True, group="prefill")
+        else:
+            attention_general(q, kcache, vcache, meta, scale, out, "prefill")
+    if K._q_blocks(meta, 1, "decode")[2]:
+        if fast_decode:
+            K._paged_attention_decode(q, kcache, vcache, meta, scale, 0, 0.0, None, out=out, group="decode")
+        else:
+            attention_general(q, kcache, vcache, meta, scale, out, "decode")
+    return out
+
+
+# --------------------------------------------------------------------------- recurrent layers
+def channel_decay(low, a2, bias, inv_tau: float):
+    """``sigmoid(low @ a2^T + bias) ** inv_tau`` in f32 ``[T, C]``."""
+    T, C = low.shape[0], a2.shape[0]
+    out = _empty(T, C, dtype=torch.float32, device=low.device)
+    pl, ld = _rows(low)
+    assert a2.is_contiguous() and a2.dtype == low.dtype
+    check(lib().mary_channel_decay(pl, ld, a2.shape[1], _p(a2), _p(bias), _p(out), T, C, inv_tau, _f32(low), _stream()), "channel_decay")
+    return out
+
+
+def decay_scan(q, k, v, decay, state, meta, H, dk, dv, q_scale):
+    """Decayed linear attention over the portions of a batch; the state of every sequence's slot is read and updated.  f32 ``[T, H, dv]``."""
+    T = q.shape[0]
+    out = _empty(T, H, dv, dtype=torch.float32, device=q.device)
+    (pq, lq), (pk, lk), (pv, lv) = _rows(q), _rows(k), _rows(v)
+    check(lib().mary_decay_scan(pq, pk, pv, _p(decay), _p(out), _p(state), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots), meta.num_seqs,
+                                lq, lk, lv, H, dk, dv, q_scale, _f32(q), _stream()), "decay_scan")
+    return out
+
+
+def delta_prep(x, taps_w, ring, b_in, a_in, a_log, dt_bias, meta, HK, H, dk, dv):
+    """Short convolutions, unit norms and gates of a gated-delta-rule layer: f32 ``q, k [T, HK * dk]``, ``v [T, H * dv]``, ``g, beta [T, H]``."""
+    T = x.shape[0]
+    f = dict(dtype=torch.float32, device=x.device)
+    q, k, v = _empty(T, HK * dk, **f), _empty(T, HK * dk, **f), _empty(T, H * dv, **f)
+    g, beta = _empty(T, H, **f), _empty(T, H, **f)
+    px, ldx = _rows(x)
+    assert b_in.stride(0) == ldx and a_in.stride(0) == ldx
+    check(lib().mary_delta_prep(px, ldx, _p(taps_w), _p(ring), _p(b_in), _p(a_in), _p(a_log), _p(dt_bias), _p(meta.positions), _p(meta.seq_index),
+                                _p(meta.q_start), _p(meta.state_slots), _p(q), _p(k), _p(v), _p(g), _p(beta), T, HK, H, dk, dv, taps_w.shape[1],
+                                _f32(x), _stream()), "delta_prep")
+    return q, k, v, g, beta
+
+
+def conv_history(x, ring, meta, taps, C):
+    px, ldx = _rows(x)
+    check(lib().mary_conv_history(px, ldx, _p(ring), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots), meta.num_seqs, taps, C, _f32(x),
+                                  _stream()), "conv_history")
+
+
+def delta_scan(q, k, v, g, beta, state, meta, HK, H, dk, dv, q_scale: float = 1.0):
+    T = q.shape[0]
+    out = _empty(T, H, dv, dtype=torch.float32, device=q.device)
+    (pq, lq), (pk, lk), (pv, lv) = _rows(q), _rows(k), _rows(v)
+    check(lib().mary_delta_scan(pq, pk, pv, _p(g), _p(beta), _p(out), _p(state), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots),
+                                meta.num_seqs, lq, lk, lv, HK, H, dk, dv, q_scale, _stream()), "delta_scan")
+    return out
+
+
+def gated_head_norm(o, gate, gain, eps, scale, out):
+    T, H, dv = o.shape
+    (pg, ldg), (po, ldo) = _rows(gate), _rows(out)
+    check(lib().mary_gated_head_norm(_p(o), pg, ldg, _p(gain), po, ldo, T, H, dv, eps, scale, _f32(gate), _stream()), "gated_head_norm")
+    return out
+
+
+def decayed_linear_attention(q, k, v, gate, low, a2, a2_bias, inv_tau, gain, state, meta, H, dk, dv, eps, out_scale, out):
+    q_scale = dk ** -0.5
+    if meta.max_q_len == 1:
+        po, ldo = _rows(out)
+        ld = q.stride(0)
+        assert all(t.stride(0) == ld for t in (k, v, gate, low)) and a2.is_contiguous()
+        check(lib().mary_decay_step(_p(q), _p(k), _p(v), _p(gate), _p(low), ld, a2.shape[1], _p(a2), _p(a2_bias), inv_tau, _p(gain), po, ldo, q_scale,
+                                    _p(state), _p(meta.q_start), _p(meta.positions), _p(meta.state_slots), meta.num_seqs, H, dk, dv, eps, out_scale,
+                                    _f32(q), _stream()), "decay_step")
+        return out
+    o = decay_scan(q, k, v, channel_decay(low, a2, a2_bias, inv_tau), state, meta, H, dk, dv, q_scale)
+    return gated_head_norm(o, gate, gain, eps, out_scale, out)
+
+
+def gated_delta_attention(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, ring, state, meta, HK, H, dk, dv, eps, out_scale, out):
+    taps = taps_w.shape[1]
+    if meta.max_q_len == 1:
+        (px, ldx), (po, ldo) = _rows(x), _rows(out)
+        assert b_in.stride(0) == ldx and a_in.stride(0) == ldx and gate.stride(0) == ldx
+        check(lib().mary_delta_step(px, ldx, _p(taps_w), _p(ring), taps, _p(b_in), _p(a_in), _p(a_log), _p(dt_bias), _p(gate), _p(gain), po, ldo,
+                                    _p(state), _p(meta.q_start), _p(meta.positions), _p(meta.state_slots), meta.num_seqs, HK, H, dk, dv, eps,
+                                    out_scale, _f32(x), _stream()), "delta_step")
+        return out
+    q, k, v, g, beta = delta_prep(x, taps_w, ring, b_in, a_in, a_log, dt_bias, meta, HK, H, dk, dv)
+    conv_history(x, ring, meta, taps, taps_w.shape[0])
+    o = delta_scan(q, k, v, g, beta, state, meta, HK, H, dk, dv)
+    return gated_head_norm(o, gate, gain, eps, out_scale, out)

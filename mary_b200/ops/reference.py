@@ -247,3 +247,89 @@ def short_conv(x, w, history=None):
     for j in range(k):
         y += xp[j:j + T] * w[:, j].float()[None, :]
     return y.to(x.dtype), xp[-(k - 1):].to(x.dtype)
+
+
+# --------------------------------------------------------------------------- 32-bit residual stream, exact attention, recurrent layers
+def embed32(ids, table, scale: float = 1.0):
+    h = table[ids.long()].float() * scale
+    return h, h.to(table.dtype, copy=True)
+
+
+def post_norm_add(a, w_post, h, w_next, eps: float):
+    """``h += rms(a) * w_post`` (in place, f32); returns ``rms(h) * w_next``, or a copy of ``h``, in the weights' type."""
+    af = a.float()
+    h += af / torch.sqrt(af.pow(2).mean(-1, keepdim=True) + eps) * w_post.float()
+    return rmsnorm32(h, w_next, eps) if w_next is not None else h.to(w_post.dtype, copy=True)
+
+
+def rmsnorm32(h, w, eps: float):
+    return (h / torch.sqrt(h.pow(2).mean(-1, keepdim=True) + eps) * w.float()).to(w.dtype)
+
+
+def qk_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps):
+    T = q.shape[0]
+    q, k = q.reshape(T, n_q, dk), k.reshape(T, n_kv, dk)
+    q = rmsnorm(q, q_gain, eps) if q_gain is not None else q
+    k = rmsnorm(k, k_gain, eps) if k_gain is not None else k
+    kv_append(k, v.reshape(T, n_kv, dv), kcache, vcache, meta.slot_mapping)
+    return q
+
+
+def _portions(meta):
+    """``(rows, state slot, position of the first row)`` of every sequence of the batch."""
+    qs, kl, sl = meta.q_start.tolist(), meta.kv_len.tolist(), meta.state_slots.tolist()
+    return [(slice(qs[s], qs[s + 1]), sl[s], kl[s] - (qs[s + 1] - qs[s])) for s in range(meta.num_seqs)]
+
+
+def head_norm_gate(o, gate, gain, eps: float, scale: float):
+    """``rms(o) * gain * silu(gate) * scale`` for ``o [T, H, dv]`` f32, ``gate [T, H * dv]``."""
+    T, H, dv = o.shape
+    y = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * gain.float() * F.silu(gate.float()).view(T, H, dv) * scale
+    return y.reshape(T, H * dv).to(gate.dtype)
+
+
+def decayed_linear_attention(q, k, v, gate, low, a2, a2_bias, inv_tau, gain, state, meta, H, dk, dv, eps, out_scale, out):
+    T = q.shape[0]
+    qf, kf, vf = q.float().view(T, H, dk) * dk ** -0.5, k.float().view(T, H, dk), v.float().view(T, H, dv)
+    alpha = torch.exp(F.logsigmoid(low.float() @ a2.float().T + a2_bias.float()) * inv_tau).view(T, H, dk)
+    o = torch.empty(T, H, dv)
+    for rows, slot, pos in _portions(meta):
+        S = state[slot, :, :, :dk] * (0.0 if pos == 0 else 1.0)                 # [H, dv, dk]
+        for t in range(rows.start, rows.stop):
+            S = S * alpha[t][:, None, :] + vf[t][:, :, None] * kf[t][:, None, :]
+            o[t] = (S * qf[t][:, None, :]).sum(-1)
+        state[slot, :, :, :dk] = S
+    out.copy_(head_norm_gate(o, gate, gain, eps, out_scale))
+    return out
+
+
+def gated_delta_attention(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, ring, state, meta, HK, H, dk, dv, eps, out_scale, out):
+    T, taps = x.shape[0], taps_w.shape[1]
+    w = taps_w.float()
+    y = torch.empty(T, taps_w.shape[0])
+    for rows, slot, pos in _portions(meta):
+        n = rows.stop - rows.start
+        hist = [ring[slot, (pos - d) % taps].float() if pos - d >= 0 else torch.zeros(w.shape[0]) for d in range(taps - 1, 0, -1)]
+        ext = torch.cat([torch.stack(hist), x[rows].float()]) if hist else x[rows].float()
+        y[rows] = F.silu(sum(ext[j:j + n] * w[:, j] for j in range(taps)))
+        for d in range(min(taps, n)):
+            ring[slot, (pos + n - 1 - d) % taps] = x[rows.stop - 1 - d].to(ring.dtype)
+    q, k, v = y.split([HK * dk, HK * dk, H * dv], -1)
+    unit = lambda z: z / torch.sqrt(z.pow(2).sum(-1, keepdim=True) + 1e-6)  # noqa: E731
+    rep = H // HK
+    q = (unit(q.view(T, HK, dk)) * dk ** -0.5).repeat_interleave(rep, 1)
+    k = unit(k.view(T, HK, dk)).repeat_interleave(rep, 1)
+    v = v.view(T, H, dv)
+    beta = torch.sigmoid(b_in.float())
+    g = torch.exp(-torch.exp(a_log) * F.softplus(a_in.float() + dt_bias))
+    o = torch.empty(T, H, dv)
+    for rows, slot, pos in _portions(meta):
+        S = state[slot, :, :, :dk] * (0.0 if pos == 0 else 1.0)
+        for t in range(rows.start, rows.stop):
+            S = S * g[t][:, None, None]
+            u = beta[t][:, None] * (v[t] - (S * k[t][:, None, :]).sum(-1))
+            S = S + u[:, :, None] * k[t][:, None, :]
+            o[t] = (S * q[t][:, None, :]).sum(-1)
+        state[slot, :, :, :dk] = S
+    out.copy_(head_norm_gate(o, gate, gain, eps, out_scale))
+    return out

@@ -49,9 +49,10 @@ class BatchMeta:
     # host copies (no device sync needed to read them)
     q_lens_host: np.ndarray | None = None
     kv_lens_host: np.ndarray | None = None
+    state_slots: torch.Tensor | None = None      # int32 [S] recurrent-state slot of every sequence (models with recurrent layers)
 
     @staticmethod
-    def build(q_lens, kv_lens, page_table: np.ndarray, page_size: int, device="cpu") -> "BatchMeta":
+    def build(q_lens, kv_lens, page_table: np.ndarray, page_size: int, device="cpu", state_slots=None) -> "BatchMeta":
         q_lens = np.asarray(q_lens, dtype=np.int32)
         kv_lens = np.asarray(kv_lens, dtype=np.int32)
         S, T = len(q_lens), int(q_lens.sum())
@@ -72,7 +73,8 @@ class BatchMeta:
                          kv_len=t(kv_lens, torch.int32), page_table=t(page_table, torch.int32),
                          slot_mapping=t(slots, torch.int64), page_size=page_size, max_q_len=int(q_lens.max()) if S else 0,
                          max_kv_len=int(kv_lens.max()) if S else 0, num_seqs=S, num_tokens=T,
-                         all_decode=bool(S and q_lens.max() == 1), q_lens_host=q_lens, kv_lens_host=kv_lens)
+                         all_decode=bool(S and q_lens.max() == 1), q_lens_host=q_lens, kv_lens_host=kv_lens,
+                         state_slots=None if state_slots is None else t(np.asarray(state_slots), torch.int32))
 
     def repage(self, target: int = 64):
         """Regroup every sequence's pages into ``target``-token pages: returns ``(pick, meta)`` where ``cache[pick]`` viewed as

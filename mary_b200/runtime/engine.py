@@ -66,6 +66,59 @@ class Engine:
     def pending(self) -> int:
         return self.lib.sched_num_waiting(self.h) + self.lib.sched_num_running(self.h)
 
+    # ------------------------------------------------------------------ the model on one batch
+    def _run_batch(self, seq_ids, q_lens, tokens, rows, logits: bool):
+        """Run ``tokens`` (host int32, the rows of all sequences concatenated; their cache rows already reserved) through the model:
+        the logits or the arg-max tokens of ``rows``, or ``None`` when no row is asked for."""
+        table, kv_lens = self.cache.alloc.page_table(seq_ids)
+        meta = BatchMeta.build(q_lens, kv_lens, table, self.cache.page_size, self.device, self.cache.alloc.slots(seq_ids))
+        ids = tokens.to(self.device, non_blocking=True)
+        with torch.no_grad():
+            if not rows:
+                self.model.hidden(ids, meta, self.cache)
+                return None
+            rows_t = torch.tensor(rows, dtype=torch.long).to(self.device)
+            return (self.model if logits else self.model.greedy)(ids, meta, self.cache, rows_t)
+
+    # ------------------------------------------------------------------ externally scheduled steps
+    def open_sequence(self) -> int:
+        """A sequence whose tokens the caller feeds itself (``feed``) instead of the scheduler; ``close_sequence`` ends it."""
+        rid = self._next_id
+        self._next_id += 1
+        return rid
+
+    def close_sequence(self, rid: int) -> None:
+        """Give back the pages and the state slot of a fed sequence."""
+        self.cache.alloc.release(rid)
+
+    def feed(self, entries):
+        """One step of a batch the caller composed: ``entries`` = ``(sequence, its next tokens, the places among them whose logits are
+        wanted)``.  Continues from what the cache and the state slots hold; returns f32 logits ``[wanted, vocab]`` (on the model's
+        device, in the order of the entries) or ``None``.  Nothing is reserved when the batch does not fit."""
+        entries = [(rid, np.asarray(t, dtype=np.int32), list(want)) for rid, t, want in entries]
+        if len({e[0] for e in entries}) != len(entries) or any(len(t) == 0 for _, t, _ in entries):
+            raise ValueError("a step takes every sequence at most once, with at least one token")
+        if any(not 0 <= w < len(t) for _, t, want in entries for w in want):
+            raise ValueError("a wanted place lies outside the entry's tokens")
+        if not entries:
+            return None
+        alloc = self.cache.alloc
+        before = {rid: alloc.seq_len(rid) for rid, _, _ in entries}
+        done = []
+        try:
+            for rid, t, _ in entries:
+                alloc.extend(rid, len(t))
+                done.append(rid)
+        except Exception:
+            for rid in done:
+                alloc.truncate(rid, before[rid]) if before[rid] > 0 else alloc.release(rid)
+            raise
+        q_lens = np.array([len(t) for _, t, _ in entries], dtype=np.int32)
+        start = np.concatenate([[0], np.cumsum(q_lens)])
+        rows = [int(start[i]) + w for i, (_, _, want) in enumerate(entries) for w in want]
+        tokens = torch.from_numpy(np.concatenate([t for _, t, _ in entries]))
+        return self._run_batch(np.array([e[0] for e in entries], dtype=np.int64), q_lens, tokens, rows, logits=True)
+
     # ------------------------------------------------------------------ one step
     def step(self) -> StepStats:
         t0 = time.perf_counter()
@@ -77,9 +130,6 @@ class Engine:
             return StepStats()
         seq_ids = self._ids[:ns].numpy()
         q_lens = self._ql[:ns].numpy()
-        table, kv_lens = self.cache.alloc.page_table(seq_ids)
-        meta = BatchMeta.build(q_lens, kv_lens, table, self.cache.page_size, self.device)
-        ids = self._tok[:nt].to(self.device, non_blocking=True)
         srow = self._srow[:ns].numpy()
         is_dec = self._dec[:ns].numpy()
         # rows whose logits are needed: every row of a decode group (for draft verification), the last prefill row
@@ -92,17 +142,11 @@ class Engine:
                 rows.append(int(srow[i]) + j)
                 owner.append(i)
         out = StepStats(tokens_in=nt, seqs=ns)
-        with torch.no_grad():
-            if rows:
-                rows_t = torch.tensor(rows, dtype=torch.long).to(self.device)
-                if self.sampler is None:
-                    toks = self.model.greedy(ids, meta, self.cache, rows_t)
-                else:
-                    toks = self.sampler(self.model(ids, meta, self.cache, rows_t))
-                toks = toks.to("cpu").numpy()
-            else:
-                self.model.hidden(ids, meta, self.cache)
-                toks = np.zeros(0, dtype=np.int64)
+        res = self._run_batch(seq_ids, q_lens, self._tok[:nt], rows, logits=self.sampler is not None)
+        if res is None:
+            toks = np.zeros(0, dtype=np.int64)
+        else:
+            toks = (res if self.sampler is None else self.sampler(res)).to("cpu").numpy()
         now = time.perf_counter()
         # commit
         k = 0

@@ -31,6 +31,9 @@ def _declare(lib):
     lib.kv_truncate.argtypes = [c.c_void_p, c.c_int64, c.c_int64]
     lib.kv_release.argtypes = [c.c_void_p, c.c_int64]
     lib.kv_pages.argtypes = [c.c_void_p, c.c_int64, c.c_void_p, c.c_int32]
+    lib.kv_set_slots.argtypes = [c.c_void_p, c.c_int32]
+    lib.kv_free_slots.argtypes = [c.c_void_p]
+    lib.kv_seq_slots.argtypes = [c.c_void_p, c.c_void_p, c.c_int32, c.c_void_p]
     lib.kv_page_table.argtypes = [c.c_void_p, c.c_void_p, c.c_int32, c.c_void_p, c.c_int32, c.c_void_p]
     lib.sched_create.restype = c.c_void_p
     lib.sched_create.argtypes = [c.c_void_p, c.c_int32, c.c_int32, c.c_int32]
@@ -52,18 +55,37 @@ class OutOfPages(RuntimeError):
 
 
 class PageAllocator:
-    def __init__(self, num_pages: int, page_size: int = 16):
+    """Pages, and for models with recurrent layers one state slot per sequence (``num_slots`` of them): a sequence takes its slot
+    when it is created and returns it with its pages."""
+
+    def __init__(self, num_pages: int, page_size: int = 16, num_slots: int = 0):
         self.lib = _native.core()
         _declare(self.lib)
-        self.num_pages, self.page_size = num_pages, page_size
+        self.num_pages, self.page_size, self.num_slots = num_pages, page_size, num_slots
         self.h = self.lib.kv_create(num_pages, page_size)
+        if num_slots:
+            self.lib.kv_set_slots(self.h, num_slots)
 
     def extend(self, seq: int, tokens: int) -> int:
         n = self.lib.kv_extend(self.h, seq, tokens)
         if n < 0:
-            raise OutOfPages(f"sequence {seq}: no free pages for {tokens} more tokens "
-                             f"({self.free_pages} of {self.num_pages} pages free)")
+            raise OutOfPages(f"sequence {seq}: no room for {tokens} more tokens ({self.free_pages} of {self.num_pages} pages free"
+                             + (f", {self.free_slots} of {self.num_slots} state slots free)" if self.num_slots else ")"))
         return n
+
+    def slots(self, seqs):
+        """State slots of the sequences as an int32 NumPy array, or ``None`` for an allocator without slots."""
+        if not self.num_slots:
+            return None
+        s = np.asarray(seqs, dtype=np.int64)
+        out = np.empty(len(s), dtype=np.int32)
+        if self.lib.kv_seq_slots(self.h, s.ctypes.data, len(s), out.ctypes.data):
+            raise KeyError(f"unknown sequence among {s.tolist()}")
+        return out
+
+    @property
+    def free_slots(self) -> int:
+        return self.lib.kv_free_slots(self.h)
 
     def truncate(self, seq: int, new_len: int) -> None:
         if self.lib.kv_truncate(self.h, seq, new_len) < 0:
@@ -154,20 +176,30 @@ class Q8Pages:
 
 
 class PagedKVCache:
-    """Device storage for the pages of every layer.  ``kv_dtype="int8"`` keeps K and V as :class:`Q8Pages`."""
+    """Device storage for the pages of every layer.  ``kv_dtype="int8"`` keeps K and V as :class:`Q8Pages`.  ``v_head_dim`` gives
+    values a width of their own.  ``state_spec`` (one ``{name: (shape, dtype)}`` per recurrent layer) adds ``state[layer][name]``
+    tensors ``[num_slots, *shape]``: the per-sequence recurrent state, addressed by ``BatchMeta.state_slots``.  A slot is never
+    cleared: the kernels take a sequence whose rows start at position 0 to have zero state."""
 
     def __init__(self, num_layers: int, num_pages: int, page_size: int, kv_heads: int | list[int], head_dim: int | list[int],
-                 dtype=torch.bfloat16, device="cpu", latent_dim: int | None = None, alias_v_to_k: bool = False, kv_dtype: str | None = None):
-        self.alloc = PageAllocator(num_pages, page_size)
+                 dtype=torch.bfloat16, device="cpu", latent_dim: int | None = None, alias_v_to_k: bool = False, kv_dtype: str | None = None,
+                 v_head_dim: int | list[int] | None = None, state_spec: list[dict] | None = None, num_slots: int = 0):
+        if state_spec and num_slots < 1:
+            raise ValueError("recurrent layers need at least one state slot")
+        self.alloc = PageAllocator(num_pages, page_size, num_slots if state_spec else 0)
+        self.num_slots = num_slots if state_spec else 0
+        self.state = [{n: torch.zeros(num_slots, *shape, dtype=dt, device=device) for n, (shape, dt) in spec.items()}
+                      for spec in (state_spec or [])]
         self.page_size, self.num_pages, self.num_layers = page_size, num_pages, num_layers
         self.latent = latent_dim is not None
         heads = kv_heads if isinstance(kv_heads, list) else [kv_heads] * num_layers
         dims = head_dim if isinstance(head_dim, list) else [head_dim] * num_layers
+        vdims = dims if v_head_dim is None else v_head_dim if isinstance(v_head_dim, list) else [v_head_dim] * num_layers
         self.kv_dtype = kv_dtype
         if kv_dtype not in (None, "int8"):
             raise ValueError(f"kv_dtype {kv_dtype!r}: only None (the activation dtype) and 'int8' are implemented")
         if kv_dtype == "int8":
-            if self.latent or alias_v_to_k:
+            if self.latent or alias_v_to_k or vdims != dims:
                 raise ValueError("the 8-bit cache holds separate K and V pages of attention heads, not a latent or aliased cache")
             self.k = [Q8Pages(num_pages, page_size, heads[i], dims[i], device) for i in range(num_layers)]
             self.v = [Q8Pages(num_pages, page_size, heads[i], dims[i], device) for i in range(num_layers)]
@@ -176,10 +208,33 @@ class PagedKVCache:
             self.v = self.k
         else:
             self.k = [torch.zeros(num_pages, page_size, heads[i], dims[i], dtype=dtype, device=device) for i in range(num_layers)]
-            self.v = self.k if alias_v_to_k else [torch.zeros_like(t) for t in self.k]
+            self.v = self.k if alias_v_to_k else [torch.zeros(num_pages, page_size, heads[i], vdims[i], dtype=dtype, device=device)
+                                                  for i in range(num_layers)]
+
+    @staticmethod
+    def for_model(model, num_pages: int, page_size: int, device="cpu", num_slots: int = 0, **kw) -> "PagedKVCache":
+        """The cache a model asks for through ``kv_spec()`` (attention layers) and, where it has one, ``state_spec()``."""
+        spec = dict(model.kv_spec())
+        if hasattr(model, "state_spec"):
+            spec.update(state_spec=model.state_spec(), num_slots=num_slots)
+        return PagedKVCache(num_pages=num_pages, page_size=page_size, dtype=model.dtype, device=device, **spec, **kw)
+
+    def state_bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for layer in self.state for t in layer.values())
+
+    def save_state(self):
+        """Copy of every recurrent state (a step that is run twice, such as a warm-up before a capture, has to start from it again)."""
+        return [{n: t.clone() for n, t in layer.items()} for layer in self.state]
+
+    def restore_state(self, saved) -> None:
+        for layer, old in zip(self.state, saved):
+            for n, t in layer.items():
+                t.copy_(old[n])
 
     def bytes(self) -> int:
         if self.kv_dtype == "int8":
             return sum(t.nbytes() for t in self.k) + sum(t.nbytes() for t in self.v)
         n = sum(t.numel() * t.element_size() for t in self.k)
-        return n if (self.latent or self.v is self.k) else 2 * n
+        if not (self.latent or self.v is self.k):
+            n += sum(t.numel() * t.element_size() for t in self.v)
+        return n + self.state_bytes()

@@ -25,6 +25,8 @@ from .kv_cache import PagedKVCache
 class SpecDecoder:
     def __init__(self, model, cache: PagedKVCache, batch: int, spec_k: int = 0, max_len: int = 8192, device="cuda",
                  use_graph: bool = True):
+        if spec_k and getattr(cache, "num_slots", 0):
+            raise ValueError("speculative rows cannot be rolled back over a recurrent state: spec_k must be 0 for this model")
         self.model, self.cache, self.B, self.k = model, cache, batch, spec_k
         self.dev = torch.device(device)
         self.use_graph = use_graph and self.dev.type == "cuda"
@@ -36,6 +38,7 @@ class SpecDecoder:
             cache.alloc.extend(s, max_len)
         table, _ = cache.alloc.page_table(list(range(B)), self.max_pages)
         self.page_table = torch.from_numpy(table).to(self.dev)
+        self.slots = cache.alloc.slots(list(range(B)))
         i32 = dict(dtype=torch.int32, device=self.dev)
         self.kv_before = torch.zeros(B, **i32)           # committed cache length per sequence
         self.fed = torch.zeros(B, R, **i32)              # [pending, drafts...]
@@ -59,7 +62,7 @@ class SpecDecoder:
                       page_table=self.page_table, slot_mapping=torch.zeros(B * q_len, dtype=torch.int64, device=dev),
                       page_size=self.cache.page_size, max_q_len=q_len, max_kv_len=self.max_len, num_seqs=B,
                       num_tokens=B * q_len, all_decode=(q_len == 1), q_lens_host=np.full(B, q_len, dtype=np.int32),
-                      kv_lens_host=None)
+                      kv_lens_host=None, state_slots=None if self.slots is None else torch.from_numpy(self.slots).to(dev))
         return m
 
     def _set_meta(self, m: BatchMeta, pos0, q_len: int):
@@ -92,7 +95,7 @@ class SpecDecoder:
         with torch.no_grad():
             for c0 in range(0, L, chunk):
                 n = min(chunk, L - c0)
-                meta = BatchMeta.build([n] * B, [c0 + n] * B, table, self.cache.page_size, self.dev)
+                meta = BatchMeta.build([n] * B, [c0 + n] * B, table, self.cache.page_size, self.dev, self.slots)
                 flat = ids[:, c0:c0 + n].reshape(-1)
                 last = torch.arange(B, device=self.dev) * n + (n - 1)
                 if self.k == 0:
@@ -163,6 +166,7 @@ class SpecDecoder:
         if not self.use_graph:
             return
         saved = (self.kv_before.clone(), self.fed.clone())
+        state = self.cache.save_state()
         s = torch.cuda.Stream()
         s.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(s), torch.no_grad():
@@ -171,6 +175,7 @@ class SpecDecoder:
         torch.cuda.current_stream().wait_stream(s)
         torch.cuda.synchronize()
         self.kv_before.copy_(saved[0]); self.fed.copy_(saved[1])
+        self.cache.restore_state(state)
         self.graph = torch.cuda.CUDAGraph()
         with torch.no_grad(), torch.cuda.graph(self.graph):
             self._step_device()
