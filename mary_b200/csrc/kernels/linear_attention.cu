@@ -20,14 +20,15 @@ __global__ void __launch_bounds__(NT) channel_decay_kernel(const T* __restrict__
                                                            const T* __restrict__ bias, float* __restrict__ decay, int n_tok, int C, float inv_tau) {
   pdl_sync();
   constexpr int TT = 16, RC = 16;
-  __shared__ float sx[TT][RC], sw[NT][RC + 1];
+  __shared__ __align__(16) float sx[RC][TT];
+  __shared__ float sw[NT][RC + 1];
   const int c = blockIdx.x * NT + threadIdx.x, t0 = blockIdx.y * TT;
   float acc[TT] = {};
   for (int r0 = 0; r0 < rank; r0 += RC) {
     __syncthreads();
     {
       const int t = threadIdx.x / RC, r = threadIdx.x % RC;
-      sx[t][r] = (t0 + t < n_tok && r0 + r < rank) ? to_f<T>(x[(int64_t)(t0 + t) * ldx + r0 + r]) : 0.f;
+      sx[r][t] = (t0 + t < n_tok && r0 + r < rank) ? to_f<T>(x[(int64_t)(t0 + t) * ldx + r0 + r]) : 0.f;
     }
     for (int i = threadIdx.x; i < NT * RC; i += NT) {
       const int cc = blockIdx.x * NT + i / RC, r = r0 + i % RC;
@@ -38,14 +39,18 @@ __global__ void __launch_bounds__(NT) channel_decay_kernel(const T* __restrict__
     for (int r = 0; r < RC; ++r) {
       const float w = sw[threadIdx.x][r];
 #pragma unroll
-      for (int t = 0; t < TT; ++t) acc[t] = fmaf(w, sx[t][r], acc[t]);
+      for (int t = 0; t < TT; t += 4) {
+        const float4 x4 = *(const float4*)&sx[r][t];
+        acc[t] = fmaf(w, x4.x, acc[t]); acc[t + 1] = fmaf(w, x4.y, acc[t + 1]);
+        acc[t + 2] = fmaf(w, x4.z, acc[t + 2]); acc[t + 3] = fmaf(w, x4.w, acc[t + 3]);
+      }
     }
   }
   if (c >= C) return;
   const float b = to_f<T>(bias[c]);
 #pragma unroll
   for (int t = 0; t < TT; ++t)
-    if (t0 + t < n_tok) decay[(int64_t)(t0 + t) * C + c] = expf(log_sigmoid_x(acc[t] + b) * inv_tau);
+    if (t0 + t < n_tok) decay[(int64_t)(t0 + t) * C + c] = exp_t<T>(log_sigmoid_t<T>(acc[t] + b) * inv_tau);
 }
 
 struct ConvIn {
@@ -63,47 +68,152 @@ __device__ __forceinline__ float conv_silu(const T* __restrict__ x, int64_t ldx,
     else if (pos - d >= 0) v = to_f<T>(ring[(int64_t)((pos - d) % taps) * C + c]);
     acc = fmaf(to_f<T>(w[(int64_t)c * taps + taps - 1 - d]), v, acc);
   }
-  return silu_x(acc);
+  return silu_t<T>(acc);
 }
 
-// One warp per (token, item); items: HK query heads, HK key heads (both made unit vectors), H value heads (with their gates).
-template <typename T>
-__global__ void delta_prep_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, const T* __restrict__ ring_all,
-                                  const T* __restrict__ b_in, const T* __restrict__ a_in, const float* __restrict__ a_log,
-                                  const float* __restrict__ dt_bias, const int* __restrict__ positions, const int* __restrict__ seq_index,
-                                  const int* __restrict__ q_start, const int* __restrict__ slots, float* __restrict__ q, float* __restrict__ k,
-                                  float* __restrict__ v, float* __restrict__ g, float* __restrict__ beta, int n_tok, ConvIn ci) {
-  pdl_sync();
-  const int items = 2 * ci.HK + ci.H;
-  const int64_t gw = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (gw >= (int64_t)n_tok * items) return;
-  const int t = (int)(gw / items), it = (int)(gw % items), lane = threadIdx.x & 31;
-  const int seq = seq_index[t], first = q_start[seq], pos = positions[t];
-  const T* ring = ring_all + (int64_t)slots[seq] * ci.taps * ci.C;
-  if (it < 2 * ci.HK) {
-    const bool is_q = it < ci.HK;
-    const int c0 = it * ci.DK;                         // q channels first, then k channels
-    float y[8], ss = 0.f;                              // DK <= 256
+// silu(conv) of E channels from c on for the four tokens of a block: rows rb .. rb + 3 (a sequence's portion is rows first .. end - 1),
+// the block's first token at position pos.  Rows before the portion come from the ring, positions before 0 are zero.
+template <typename T, int TAPS, int E>
+__device__ __forceinline__ void conv_block(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, const T* __restrict__ ring, int n_taps, int C,
+                                           int c, int rb, int first, int end, int pos, float (&y)[4][E]) {
+  const int taps = TAPS > 0 ? TAPS : n_taps;
+  float wr[E][TAPS > 0 ? TAPS : 1];
+  if constexpr (TAPS > 0) {
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int c = lane + 32 * i;
-      y[i] = c < ci.DK ? conv_silu<T>(x, ldx, w, ring, ci.taps, ci.C, c0 + c, t, first, pos) : 0.f;
-      ss += y[i] * y[i];
+    for (int e = 0; e < E; ++e) {
+      if constexpr (TAPS == 4 && E == 4) {
+        load_e<T, 4>(w + (int64_t)(c + e) * 4, wr[e]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) wr[e][j] = to_f<T>(w[(int64_t)(c + e) * TAPS + j]);
+      }
     }
-    const float inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f) * (is_q ? 1.0f / sqrtf((float)ci.DK) : 1.0f);
-    float* dst = (is_q ? q : k) + ((int64_t)t * ci.HK + (is_q ? it : it - ci.HK)) * ci.DK;
+  }
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
-      if (lane + 32 * i < ci.DK) dst[lane + 32 * i] = y[i] * inv;
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int e = 0; e < E; ++e) y[i][e] = 0.f;
+#pragma unroll
+  for (int r = 1 - taps; r < 4; ++r) {
+    float v[E] = {};
+    if (rb + r >= end) break;
+    if (rb + r >= first) load_e<T, E>(x + (int64_t)(rb + r) * ldx + c, v);
+    else if (pos + r >= 0) load_e<T, E>(ring + (int64_t)((pos + r) % taps) * C + c, v);
+    else continue;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int d = i - r;
+      if (d < 0 || d >= taps) continue;
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        float wv;
+        if constexpr (TAPS > 0) wv = wr[e][TAPS - 1 - d];
+        else wv = to_f<T>(w[(int64_t)(c + e) * taps + taps - 1 - d]);
+        y[i][e] = fmaf(wv, v[e], y[i][e]);
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int e = 0; e < E; ++e) y[i][e] = silu_t<T>(y[i][e]);
+}
+
+// One warp per (sequence, block of four tokens, item); items: HK query / key heads (unit vectors, and the products of the block's keys
+// with its keys and queries), H value heads (with their gates).  VEC: widths, pitch and addresses allow accesses of four values.
+template <typename T, int TAPS, bool VEC>
+__global__ void __launch_bounds__(256) delta_prep_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, const T* __restrict__ ring_all,
+                                                         const T* __restrict__ b_in, const T* __restrict__ a_in, const float* __restrict__ a_log,
+                                                         const float* __restrict__ dt_bias, const int* __restrict__ q_start,
+                                                         const int* __restrict__ kv_len, const int* __restrict__ slots, float* __restrict__ q,
+                                                         float* __restrict__ k, float* __restrict__ v, float* __restrict__ g, float* __restrict__ beta,
+                                                         float* __restrict__ pairs, ConvIn ci) {
+  pdl_sync();
+  constexpr int E = VEC ? 4 : 1, NI = 8 / E;          // DK <= 256: eight channels per lane
+  const int items = ci.HK + ci.H;
+  const int gw = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int blk = gw / items, it = gw % items, lane = threadIdx.x & 31, seq = blockIdx.y;
+  const int first = q_start[seq], end = q_start[seq + 1], rb = first + blk * 4;
+  if (rb >= end) return;
+  const int nt = min(4, end - rb);
+  const int pos = kv_len[seq] - (end - first) + blk * 4;
+  const T* ring = ring_all + (int64_t)slots[seq] * ci.taps * ci.C;
+  if (it < ci.HK) {
+    float yq[NI][4][E], yk[NI][4][E];
+    float ss[8] = {};                                  // sums of squares: 4 queries, 4 keys
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = i * 32 * E + lane * E;
+      if (c < ci.DK) {
+        conv_block<T, TAPS, E>(x, ldx, w, ring, ci.taps, ci.C, it * ci.DK + c, rb, first, end, pos, yq[i]);
+        conv_block<T, TAPS, E>(x, ldx, w, ring, ci.taps, ci.C, (ci.HK + it) * ci.DK + c, rb, first, end, pos, yk[i]);
+      } else {
+#pragma unroll
+        for (int t = 0; t < 4; ++t)
+#pragma unroll
+          for (int e = 0; e < E; ++e) yq[i][t][e] = yk[i][t][e] = 0.f;
+      }
+#pragma unroll
+      for (int t = 0; t < 4; ++t)
+#pragma unroll
+        for (int e = 0; e < E; ++e) { ss[t] = fmaf(yq[i][t][e], yq[i][t][e], ss[t]); ss[4 + t] = fmaf(yk[i][t][e], yk[i][t][e], ss[4 + t]); }
+    }
+    const float qs = 1.0f / sqrtf((float)ci.DK);
+#pragma unroll
+    for (int t = 0; t < 8; ++t) ss[t] = 1.0f / sqrtf(warp_sum(ss[t]) + 1e-6f) * (t < 4 ? qs : 1.0f);
+    float pr[16] = {};                                 // k_j . k_i (j < i) in slots i * 4 + j below the diagonal, the diagonal unused
+    float pq[16] = {};
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = i * 32 * E + lane * E;
+#pragma unroll
+      for (int t = 0; t < 4; ++t)
+#pragma unroll
+        for (int e = 0; e < E; ++e) { yq[i][t][e] *= ss[t]; yk[i][t][e] *= ss[4 + t]; }
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+#pragma unroll
+        for (int j = 0; j <= t; ++j)
+#pragma unroll
+          for (int e = 0; e < E; ++e) {
+            if (j < t) pr[t * 4 + j] = fmaf(yk[i][j][e], yk[i][t][e], pr[t * 4 + j]);
+            pq[t * 4 + j] = fmaf(yk[i][j][e], yq[i][t][e], pq[t * 4 + j]);
+          }
+        if (t < nt && c < ci.DK) {
+          const int64_t o = ((int64_t)(rb + t) * ci.HK + it) * ci.DK + c;
+          store_e<float, E>(q + o, yq[i][t]);
+          store_e<float, E>(k + o, yk[i][t]);
+        }
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < 4; ++t) {
+      float r[8];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        r[j] = j < t ? warp_sum(pr[t * 4 + j]) : 0.f;
+        r[4 + j] = j <= t ? warp_sum(pq[t * 4 + j]) : 0.f;
+      }
+      if (t < nt && lane < 2) {
+        float4* dst = (float4*)(pairs + ((int64_t)(rb + t) * ci.HK + it) * 8) + lane;
+        *dst = lane == 0 ? make_float4(r[0], r[1], r[2], r[3]) : make_float4(r[4], r[5], r[6], r[7]);
+      }
+    }
     return;
   }
-  const int h = it - 2 * ci.HK;
+  const int h = it - ci.HK;
   const int c0 = 2 * ci.HK * ci.DK + h * ci.DV;
-  for (int c = lane; c < ci.DV; c += 32)
-    v[((int64_t)t * ci.H + h) * ci.DV + c] = conv_silu<T>(x, ldx, w, ring, ci.taps, ci.C, c0 + c, t, first, pos);
-  if (lane == 0) {
-    beta[(int64_t)t * ci.H + h] = sigmoid_x(to_f<T>(b_in[(int64_t)t * ldx + h]));
-    g[(int64_t)t * ci.H + h] = expf(-expf(a_log[h]) * softplus_x(to_f<T>(a_in[(int64_t)t * ldx + h]) + dt_bias[h]));
+  for (int c = lane * E; c < ci.DV; c += 32 * E) {
+    float y[4][E];
+    conv_block<T, TAPS, E>(x, ldx, w, ring, ci.taps, ci.C, c0 + c, rb, first, end, pos, y);
+#pragma unroll
+    for (int t = 0; t < 4; ++t)
+      if (t < nt) store_e<float, E>(v + ((int64_t)(rb + t) * ci.H + h) * ci.DV + c, y[t]);
+  }
+  if (lane < nt) {
+    const int64_t t = rb + lane;
+    beta[t * ci.H + h] = sigmoid_x(to_f<T>(b_in[t * ldx + h]));
+    g[t * ci.H + h] = expf(-expf(a_log[h]) * softplus_x(to_f<T>(a_in[t * ldx + h]) + dt_bias[h]));
   }
 }
 
@@ -119,8 +229,8 @@ __global__ void conv_history_kernel(const T* __restrict__ x, int64_t ldx, T* __r
   for (int d = 0; d < taps && end - 1 - d >= first; ++d) ring[(int64_t)((kv_len[seq] - 1 - d) % taps) * C + c] = x[(int64_t)(end - 1 - d) * ldx + c];
 }
 
-// y[t, h, :] = rms(o[t, h, :]) * gain * silu(gate[t, h, :]) * scale, one warp per (token, head)
-template <typename T>
+// y[t, h, :] = rms(o[t, h, :]) * gain * silu(gate[t, h, :]) * scale, one warp per (token, head); E values per access
+template <typename T, int E>
 __global__ void gated_head_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int64_t ldg, const T* __restrict__ gain,
                                        T* __restrict__ y, int64_t ldy, int n_tok, int H, int DV, float eps, float scale) {
   pdl_sync();
@@ -128,11 +238,25 @@ __global__ void gated_head_norm_kernel(const float* __restrict__ o, const T* __r
   if (gw >= (int64_t)n_tok * H) return;
   const int t = (int)(gw / H), h = (int)(gw % H), lane = threadIdx.x & 31;
   const float* src = o + gw * DV;
+  const T* gr = gate + (int64_t)t * ldg + (int64_t)h * DV;
+  T* yr = y + (int64_t)t * ldy + (int64_t)h * DV;
   float ss = 0.f;
-  for (int c = lane; c < DV; c += 32) ss += src[c] * src[c];
+  for (int c = lane * E; c < DV; c += 32 * E) {
+    float f[E];
+    load_e<float, E>(src + c, f);
+#pragma unroll
+    for (int e = 0; e < E; ++e) ss = fmaf(f[e], f[e], ss);
+  }
   const float inv = 1.0f / sqrtf(warp_sum(ss) / DV + eps) * scale;
-  for (int c = lane; c < DV; c += 32)
-    y[(int64_t)t * ldy + (int64_t)h * DV + c] = from_f<T>(src[c] * inv * to_f<T>(gain[c]) * silu_x(to_f<T>(gate[(int64_t)t * ldg + (int64_t)h * DV + c])));
+  for (int c = lane * E; c < DV; c += 32 * E) {
+    float f[E], gt[E], gn[E];
+    load_e<float, E>(src + c, f);
+    load_e<T, E>(gr + c, gt);
+    load_e<T, E>(gain + c, gn);
+#pragma unroll
+    for (int e = 0; e < E; ++e) f[e] *= inv * gn[e] * silu_t<T>(gt[e]);
+    store_e<T, E>(yr + c, f);
+  }
 }
 
 // ----------------------------------------------------------------------------------------------- fused one-token steps
@@ -198,7 +322,7 @@ __device__ __forceinline__ void finish_head(const float* so, float* red, const T
   float ss = 0.f;
   for (int c = threadIdx.x; c < DV; c += NT) ss += so[c] * so[c];
   const float inv = 1.0f / sqrtf(block_sum_x(ss, red) / DV + eps) * scale;
-  for (int c = threadIdx.x; c < DV; c += NT) y[c] = from_f<T>(so[c] * inv * to_f<T>(gain[c]) * silu_x(to_f<T>(gate[c])));
+  for (int c = threadIdx.x; c < DV; c += NT) y[c] = from_f<T>(so[c] * inv * to_f<T>(gain[c]) * silu_t<T>(to_f<T>(gate[c])));
 }
 
 struct StepIo {
@@ -230,7 +354,7 @@ __global__ void __launch_bounds__(NT) decay_step_kernel(const T* __restrict__ q,
       const int ch = h * io.DK + c;
       float z = to_f<T>(a2_bias[ch]);
       for (int r = 0; r < rank; ++r) z = fmaf(to_f<T>(a2[(int64_t)ch * rank + r]), to_f<T>(low[row + r]), z);
-      a = expf(log_sigmoid_x(z) * inv_tau);
+      a = exp_t<T>(log_sigmoid_t<T>(z) * inv_tau);
       qv = to_f<T>(q[row + ch]) * q_scale;
       kv = to_f<T>(k[row + ch]);
     }
@@ -313,17 +437,25 @@ MARY_API int mary_channel_decay(const void* x, int64_t ldx, int rank, const void
   return MARY_OK;
 }
 
-// x: projection rows whose first 2 HK DK + H DV columns are the q, k, v inputs; b_in / a_in: columns of the same rows
+// x: projection rows whose first 2 HK DK + H DV columns are the q, k, v inputs; b_in / a_in: columns of the same rows.  S sequences of at
+// most max_q rows each.  pairs [T, HK, 8] as mary_delta_scan takes it.
 MARY_API int mary_delta_prep(const void* x, int64_t ldx, const void* taps_w, const void* ring, const void* b_in, const void* a_in,
-                             const float* a_log, const float* dt_bias, const int* positions, const int* seq_index, const int* q_start,
-                             const int* slots, float* q, float* k, float* v, float* g, float* beta, int n_tok, int HK, int H, int DK, int DV,
-                             int taps, int f32, cudaStream_t s) {
-  if (n_tok <= 0) return MARY_OK;
-  if (HK < 1 || H < 1 || H % HK || DK < 1 || DK > 256 || DV < 1 || taps < 1) return MARY_ERR_BAD_ARG;
+                             const float* a_log, const float* dt_bias, const int* q_start, const int* kv_len, const int* slots, float* q, float* k,
+                             float* v, float* g, float* beta, float* pairs, int S, int max_q, int HK, int H, int DK, int DV, int taps, int f32,
+                             cudaStream_t s) {
+  if (S <= 0 || max_q <= 0) return MARY_OK;
+  if (HK < 1 || H < 1 || H % HK || DK < 1 || DK > 256 || DV < 1 || taps < 1 || S > 65535 || ((uintptr_t)pairs & 15)) return MARY_ERR_BAD_ARG;
   const ConvIn ci = {HK, H, DK, DV, taps, 2 * HK * DK + H * DV};
-  const int64_t warps = (int64_t)n_tok * (2 * HK + H);
-  BY_TYPE(f32, MARY_LAUNCH((delta_prep_kernel<T>), (unsigned)((warps + 7) / 8), 256, 0, s, (const T*)x, ldx, (const T*)taps_w, (const T*)ring, (const T*)b_in,
-                           (const T*)a_in, a_log, dt_bias, positions, seq_index, q_start, slots, q, k, v, g, beta, n_tok, ci));
+  const int64_t warps = (int64_t)((max_q + 3) / 4) * (HK + H);
+  const dim3 grid((unsigned)((warps + 7) / 8), S);
+  BY_TYPE(f32, {
+    const uintptr_t mask = 4 * sizeof(T) - 1;
+    const bool vec = DK % 4 == 0 && DV % 4 == 0 && ldx % 4 == 0 && !(((uintptr_t)x | (uintptr_t)ring | (uintptr_t)taps_w) & mask);
+    auto fn = taps == 4 ? (vec ? delta_prep_kernel<T, 4, true> : delta_prep_kernel<T, 4, false>)
+                        : (vec ? delta_prep_kernel<T, 0, true> : delta_prep_kernel<T, 0, false>);
+    MARY_LAUNCH(fn, grid, 256, 0, s, (const T*)x, ldx, (const T*)taps_w, (const T*)ring, (const T*)b_in, (const T*)a_in, a_log, dt_bias, q_start, kv_len,
+                slots, q, k, v, g, beta, pairs, ci);
+  });
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }
@@ -341,8 +473,12 @@ MARY_API int mary_gated_head_norm(const float* o, const void* gate, int64_t ldg,
                                   float eps, float scale, int f32, cudaStream_t s) {
   if (n_tok <= 0) return MARY_OK;
   const int64_t warps = (int64_t)n_tok * H;
-  BY_TYPE(f32, MARY_LAUNCH((gated_head_norm_kernel<T>), (unsigned)((warps + 7) / 8), 256, 0, s, o, (const T*)gate, ldg, (const T*)gain, (T*)y, ldy, n_tok, H, DV,
-                           eps, scale));
+  BY_TYPE(f32, {
+    const uintptr_t mask = 4 * sizeof(T) - 1;
+    const bool vec = DV % 4 == 0 && ldg % 4 == 0 && ldy % 4 == 0 && !(((uintptr_t)gate | (uintptr_t)gain | (uintptr_t)y) & mask) && !((uintptr_t)o & 15);
+    auto fn = vec ? gated_head_norm_kernel<T, 4> : gated_head_norm_kernel<T, 1>;
+    MARY_LAUNCH(fn, (unsigned)((warps + 7) / 8), 256, 0, s, o, (const T*)gate, ldg, (const T*)gain, (T*)y, ldy, n_tok, H, DV, eps, scale);
+  });
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }

@@ -34,11 +34,55 @@ __device__ __forceinline__ uint4 pack16(const float (&f)[8]) {
   return v;
 }
 
+// E consecutive values (E = 4: one 8- or 16-byte access, aligned) as floats.
+template <typename T, int E> __device__ __forceinline__ void load_e(const T* p, float (&f)[E]) {
+  if constexpr (E == 4 && sizeof(T) == 2) {
+    const uint2 v = *(const uint2*)p;
+    const __nv_bfloat162* h = (const __nv_bfloat162*)&v;
+    const float2 a = __bfloat1622float2(h[0]), b = __bfloat1622float2(h[1]);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else if constexpr (E == 4) {
+    const float4 v = *(const float4*)p;
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+  } else {
+#pragma unroll
+    for (int j = 0; j < E; ++j) f[j] = to_f<T>(p[j]);
+  }
+}
+template <typename T, int E> __device__ __forceinline__ void store_e(T* p, const float (&f)[E]) {
+  if constexpr (E == 4 && sizeof(T) == 2) {
+    uint2 v;
+    __nv_bfloat162* h = (__nv_bfloat162*)&v;
+    h[0] = __floats2bfloat162_rn(f[0], f[1]); h[1] = __floats2bfloat162_rn(f[2], f[3]);
+    *(uint2*)p = v;
+  } else if constexpr (E == 4) {
+    *(float4*)p = make_float4(f[0], f[1], f[2], f[3]);
+  } else {
+#pragma unroll
+    for (int j = 0; j < E; ++j) p[j] = from_f<T>(f[j]);
+  }
+}
+
 // Exact forms (these files are compiled without fast math): logistic function, SiLU, softplus and the log of the logistic function.
 __device__ __forceinline__ float sigmoid_x(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float silu_x(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus_x(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float log_sigmoid_x(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
+
+// The same by storage type: exact for 32-bit models, the hardware's fast exponential / logarithm / divide (a few units in the last place
+// of a 32-bit result) for bf16 models.
+template <typename T> __device__ __forceinline__ float exp_t(float x) {
+  if constexpr (sizeof(T) == 4) return expf(x);
+  else return __expf(x);
+}
+template <typename T> __device__ __forceinline__ float silu_t(float x) {
+  if constexpr (sizeof(T) == 4) return silu_x(x);
+  else return __fdividef(x, 1.0f + __expf(-x));
+}
+template <typename T> __device__ __forceinline__ float log_sigmoid_t(float x) {
+  if constexpr (sizeof(T) == 4) return log_sigmoid_x(x);
+  else return fminf(x, 0.f) - __logf(1.0f + __expf(-fabsf(x)));
+}
 
 __device__ __forceinline__ float block_sum_x(float v, float* red) {      // red: 32 floats of shared memory
   v = warp_sum(v);

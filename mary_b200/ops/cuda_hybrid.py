@@ -20,11 +20,11 @@ declare("mary_attention_general", "ppppppppp" + "iii" + "lllll" + "iiiiiii" + "f
 declare("mary_attention_general_rows", "i")
 declare("mary_attention_general_scratch_floats", "iiiii", ret64=True)
 declare("mary_channel_decay", "pli" + "ppp" + "iifis")
-declare("mary_delta_prep", "pl" + "pppppp" + "pppp" + "ppppp" + "iiiiii" + "is")
+declare("mary_delta_prep", "pl" + "pppppp" + "ppp" + "pppppp" + "iiiiiii" + "is")
 declare("mary_conv_history", "plpppp" + "iiiis")
 declare("mary_gated_head_norm", "pplppl" + "iiiffis")
 declare("mary_decay_scan", "pppppp" + "ppp" + "illl" + "iiifis")
-declare("mary_delta_scan", "ppppppp" + "ppp" + "illl" + "iiiifs")
+declare("mary_delta_scan", "pppppppp" + "ppp" + "illl" + "iiiifs")
 declare("mary_decay_step", "ppppp" + "li" + "ppfp" + "plfp" + "ppp" + "iiiiffis")
 declare("mary_delta_step", "plppi" + "pppppp" + "plp" + "ppp" + "iiiiiffis")
 
@@ -177,17 +177,18 @@ def decay_scan(q, k, v, decay, state, meta, H, dk, dv, q_scale):
 
 
 def delta_prep(x, taps_w, ring, b_in, a_in, a_log, dt_bias, meta, HK, H, dk, dv):
-    """Short convolutions, unit norms and gates of a gated-delta-rule layer: f32 ``q, k [T, HK * dk]``, ``v [T, H * dv]``, ``g, beta [T, H]``."""
+    """Short convolutions, unit norms and gates of a gated-delta-rule layer: f32 ``q, k [T, HK * dk]``, ``v [T, H * dv]``, ``g, beta [T, H]``
+    and the products ``pairs [T, HK, 8]`` of every four tokens' keys with their keys and queries (what ``delta_scan`` takes)."""
     T = x.shape[0]
     f = dict(dtype=torch.float32, device=x.device)
     q, k, v = _empty(T, HK * dk, **f), _empty(T, HK * dk, **f), _empty(T, H * dv, **f)
-    g, beta = _empty(T, H, **f), _empty(T, H, **f)
+    g, beta, pairs = _empty(T, H, **f), _empty(T, H, **f), _empty(T, HK, 8, **f)
     px, ldx = _rows(x)
     assert b_in.stride(0) == ldx and a_in.stride(0) == ldx
-    check(lib().mary_delta_prep(px, ldx, _p(taps_w), _p(ring), _p(b_in), _p(a_in), _p(a_log), _p(dt_bias), _p(meta.positions), _p(meta.seq_index),
-                                _p(meta.q_start), _p(meta.state_slots), _p(q), _p(k), _p(v), _p(g), _p(beta), T, HK, H, dk, dv, taps_w.shape[1],
-                                _f32(x), _stream()), "delta_prep")
-    return q, k, v, g, beta
+    check(lib().mary_delta_prep(px, ldx, _p(taps_w), _p(ring), _p(b_in), _p(a_in), _p(a_log), _p(dt_bias), _p(meta.q_start), _p(meta.kv_len),
+                                _p(meta.state_slots), _p(q), _p(k), _p(v), _p(g), _p(beta), _p(pairs), meta.num_seqs, meta.max_q_len, HK, H, dk, dv,
+                                taps_w.shape[1], _f32(x), _stream()), "delta_prep")
+    return q, k, v, g, beta, pairs
 
 
 def conv_history(x, ring, meta, taps, C):
@@ -196,11 +197,11 @@ def conv_history(x, ring, meta, taps, C):
                                   _stream()), "conv_history")
 
 
-def delta_scan(q, k, v, g, beta, state, meta, HK, H, dk, dv, q_scale: float = 1.0):
+def delta_scan(q, k, v, g, beta, pairs, state, meta, HK, H, dk, dv, q_scale: float = 1.0):
     T = q.shape[0]
     out = _empty(T, H, dv, dtype=torch.float32, device=q.device)
     (pq, lq), (pk, lk), (pv, lv) = _rows(q), _rows(k), _rows(v)
-    check(lib().mary_delta_scan(pq, pk, pv, _p(g), _p(beta), _p(out), _p(state), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots),
+    check(lib().mary_delta_scan(pq, pk, pv, _p(g), _p(beta), _p(pairs), _p(out), _p(state), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots),
                                 meta.num_seqs, lq, lk, lv, HK, H, dk, dv, q_scale, _stream()), "delta_scan")
     return out
 
@@ -235,7 +236,7 @@ def gated_delta_attention(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, rin
                                     _p(state), _p(meta.q_start), _p(meta.positions), _p(meta.state_slots), meta.num_seqs, HK, H, dk, dv, eps,
                                     out_scale, _f32(x), _stream()), "delta_step")
         return out
-    q, k, v, g, beta = delta_prep(x, taps_w, ring, b_in, a_in, a_log, dt_bias, meta, HK, H, dk, dv)
+    q, k, v, g, beta, pairs = delta_prep(x, taps_w, ring, b_in, a_in, a_log, dt_bias, meta, HK, H, dk, dv)
     conv_history(x, ring, meta, taps, taps_w.shape[0])
-    o = delta_scan(q, k, v, g, beta, state, meta, HK, H, dk, dv)
+    o = delta_scan(q, k, v, g, beta, pairs, state, meta, HK, H, dk, dv)
     return gated_head_norm(o, gate, gain, eps, out_scale, out)
