@@ -93,7 +93,30 @@ __device__ __forceinline__ void conv_block(const T* __restrict__ x, int64_t ldx,
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int e = 0; e < E; ++e) y[i][e] = 0.f;
+  if constexpr (TAPS > 0) {
+    // all rows are requested before the first is used
+    float v[TAPS + 3][E];
 #pragma unroll
+    for (int r = 1 - TAPS; r < 4; ++r) {
+      const bool here = rb + r >= first;
+      const T* src = here ? x + (int64_t)(rb + r) * ldx + c : ring + (int64_t)((pos + r + TAPS) % TAPS) * C + c;
+      if (rb + r < end && pos + r >= 0) load_e<T, E>(src, v[r + TAPS - 1]);
+      else
+#pragma unroll
+        for (int e = 0; e < E; ++e) v[r + TAPS - 1][e] = 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int d = 0; d < TAPS; ++d)
+#pragma unroll
+        for (int e = 0; e < E; ++e) y[i][e] = fmaf(wr[e][TAPS - 1 - d], v[i - d + TAPS - 1][e], y[i][e]);
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int e = 0; e < E; ++e) y[i][e] = silu_t<T>(y[i][e]);
+    return;
+  }
   for (int r = 1 - taps; r < 4; ++r) {
     float v[E] = {};
     if (rb + r >= end) break;
@@ -106,10 +129,7 @@ __device__ __forceinline__ void conv_block(const T* __restrict__ x, int64_t ldx,
       if (d < 0 || d >= taps) continue;
 #pragma unroll
       for (int e = 0; e < E; ++e) {
-        float wv;
-        if constexpr (TAPS > 0) wv = wr[e][TAPS - 1 - d];
-        else wv = to_f<T>(w[(int64_t)(c + e) * taps + taps - 1 - d]);
-        y[i][e] = fmaf(wv, v[e], y[i][e]);
+        y[i][e] = fmaf(to_f<T>(w[(int64_t)(c + e) * taps + taps - 1 - d]), v[e], y[i][e]);
       }
     }
   }
@@ -140,7 +160,12 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const T* __restrict__ x
   const T* ring = ring_all + (int64_t)slots[seq] * ci.taps * ci.C;
   if (it < ci.HK) {
     float yq[NI][4][E], yk[NI][4][E];
-    float ss[8] = {};                                  // sums of squares: 4 queries, 4 keys
+    // 32 sums in the places of the output rows: dot[8 t + j] = k_j . k_t for j < t, dot[8 t + 4 + j] = k_j . q_t for j <= t,
+    // dot[8 t + 3] = k_t . k_t, and q_t . q_t in four of the places that no product takes
+    constexpr int QQ[4] = {0, 1, 2, 5};
+    float dot[32];
+#pragma unroll
+    for (int i = 0; i < 32; ++i) dot[i] = 0.f;
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
       const int c = i * 32 * E + lane * E;
@@ -156,29 +181,36 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const T* __restrict__ x
 #pragma unroll
       for (int t = 0; t < 4; ++t)
 #pragma unroll
-        for (int e = 0; e < E; ++e) { ss[t] = fmaf(yq[i][t][e], yq[i][t][e], ss[t]); ss[4 + t] = fmaf(yk[i][t][e], yk[i][t][e], ss[4 + t]); }
-    }
-    const float qs = 1.0f / sqrtf((float)ci.DK);
+        for (int e = 0; e < E; ++e) {
+          const float qv = yq[i][t][e], kv = yk[i][t][e];
+          dot[QQ[t]] = fmaf(qv, qv, dot[QQ[t]]);
+          dot[8 * t + 3] = fmaf(kv, kv, dot[8 * t + 3]);
 #pragma unroll
-    for (int t = 0; t < 8; ++t) ss[t] = 1.0f / sqrtf(warp_sum(ss[t]) + 1e-6f) * (t < 4 ? qs : 1.0f);
-    float pr[16] = {};                                 // k_j . k_i (j < i) in slots i * 4 + j below the diagonal, the diagonal unused
-    float pq[16] = {};
+          for (int j = 0; j <= t; ++j) {
+            if (j < t) dot[8 * t + j] = fmaf(yk[i][j][e], kv, dot[8 * t + j]);
+            dot[8 * t + 4 + j] = fmaf(yk[i][j][e], qv, dot[8 * t + 4 + j]);
+          }
+        }
+    }
+    halve<32>(dot, lane, 16);
+    halve<16>(dot, lane, 8);
+    halve<8>(dot, lane, 4);
+    halve<4>(dot, lane, 2);
+    halve<2>(dot, lane, 1);                            // lane i holds sum i
+    const float r = 1.0f / sqrtf(dot[0] + 1e-6f), qs = 1.0f / sqrtf((float)ci.DK);
+    float iq[4], ik[4];
+#pragma unroll
+    for (int t = 0; t < 4; ++t) {
+      iq[t] = __shfl_sync(0xffffffffu, r, QQ[t]) * qs;
+      ik[t] = __shfl_sync(0xffffffffu, r, 8 * t + 3);
+    }
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
       const int c = i * 32 * E + lane * E;
 #pragma unroll
-      for (int t = 0; t < 4; ++t)
-#pragma unroll
-        for (int e = 0; e < E; ++e) { yq[i][t][e] *= ss[t]; yk[i][t][e] *= ss[4 + t]; }
-#pragma unroll
       for (int t = 0; t < 4; ++t) {
 #pragma unroll
-        for (int j = 0; j <= t; ++j)
-#pragma unroll
-          for (int e = 0; e < E; ++e) {
-            if (j < t) pr[t * 4 + j] = fmaf(yk[i][j][e], yk[i][t][e], pr[t * 4 + j]);
-            pq[t * 4 + j] = fmaf(yk[i][j][e], yq[i][t][e], pq[t * 4 + j]);
-          }
+        for (int e = 0; e < E; ++e) { yq[i][t][e] *= iq[t]; yk[i][t][e] *= ik[t]; }
         if (t < nt && c < ci.DK) {
           const int64_t o = ((int64_t)(rb + t) * ci.HK + it) * ci.DK + c;
           store_e<float, E>(q + o, yq[i][t]);
@@ -186,19 +218,14 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const T* __restrict__ x
         }
       }
     }
+    const int pt = lane >> 3, pj = lane & 3;
+    float si = 0.f, sj = 0.f;
 #pragma unroll
     for (int t = 0; t < 4; ++t) {
-      float r[8];
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        r[j] = j < t ? warp_sum(pr[t * 4 + j]) : 0.f;
-        r[4 + j] = j <= t ? warp_sum(pq[t * 4 + j]) : 0.f;
-      }
-      if (t < nt && lane < 2) {
-        float4* dst = (float4*)(pairs + ((int64_t)(rb + t) * ci.HK + it) * 8) + lane;
-        *dst = lane == 0 ? make_float4(r[0], r[1], r[2], r[3]) : make_float4(r[4], r[5], r[6], r[7]);
-      }
+      if (t == pt) si = (lane & 4) ? iq[t] : ik[t];
+      if (t == pj) sj = ik[t];
     }
+    if (pt < nt) pairs[((int64_t)(rb + pt) * ci.HK + it) * 8 + (lane & 7)] = dot[0] * si * sj;
     return;
   }
   const int h = it - ci.HK;
@@ -240,6 +267,20 @@ __global__ void gated_head_norm_kernel(const float* __restrict__ o, const T* __r
   const float* src = o + gw * DV;
   const T* gr = gate + (int64_t)t * ldg + (int64_t)h * DV;
   T* yr = y + (int64_t)t * ldy + (int64_t)h * DV;
+  if (E == 4 && DV == 128) {                 // one access per lane, all of them requested before the reduction
+    float f[E], gt[E], gn[E];
+    load_e<float, E>(src + lane * E, f);
+    load_e<T, E>(gr + lane * E, gt);
+    load_e<T, E>(gain + lane * E, gn);
+    float s2 = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e) s2 = fmaf(f[e], f[e], s2);
+    const float r = 1.0f / sqrtf(warp_sum(s2) / DV + eps) * scale;
+#pragma unroll
+    for (int e = 0; e < E; ++e) f[e] *= r * gn[e] * silu_t<T>(gt[e]);
+    store_e<T, E>(yr + lane * E, f);
+    return;
+  }
   float ss = 0.f;
   for (int c = lane * E; c < DV; c += 32 * E) {
     float f[E];

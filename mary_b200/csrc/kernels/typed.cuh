@@ -84,6 +84,17 @@ template <typename T> __device__ __forceinline__ float log_sigmoid_t(float x) {
   else return fminf(x, 0.f) - __logf(1.0f + __expf(-fabsf(x)));
 }
 
+// One halving step of a reduction over lanes: of N values a lane keeps the half its lane bit selects and adds what its partner sends.
+template <int N>
+__device__ __forceinline__ void halve(float* v, int lane, int bit) {
+  const bool up = (lane & bit) != 0;
+#pragma unroll
+  for (int i = 0; i < N / 2; ++i) {
+    const float send = up ? v[i] : v[i + N / 2], keep = up ? v[i + N / 2] : v[i];
+    v[i] = keep + __shfl_xor_sync(0xffffffffu, send, bit);
+  }
+}
+
 __device__ __forceinline__ float block_sum_x(float v, float* red) {      // red: 32 floats of shared memory
   v = warp_sum(v);
   const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
