@@ -91,12 +91,14 @@ def decode_step(m, cache, batch: int, ctx: int, tokens: int, dev):
 def run(sizes, cases, steps: int, warmup: int, trace: bool = False) -> dict:
     from ...ops import cuda as K
     dev = torch.device("cuda", 0)
-    K.set_pdl(True)                       # chains of dense products and small kernels: dependent launch gains for both models
     out = []
     for size in sizes:
         for kind in ("tatizen", "dense"):
             m = make_model(kind, size, dev)
             for what, batch, n in cases:
+                # dependent launch: a decode step is a chain of short kernels and gains from it; a prefill step loses (the waiting blocks of
+                # the next kernel take room beside the long scans)
+                K.set_pdl(what == "decode")
                 tokens = n if what == "prefill" else n + max(steps, 1) + max(warmup, 3) + 64
                 tokens = (tokens + PAGE - 1) // PAGE * PAGE
                 cache = make_cache(m, batch, tokens, dev)

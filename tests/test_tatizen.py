@@ -359,6 +359,23 @@ def test_mixed_batches_pages_and_slots_reused(target, name):
     assert eng.cache.alloc.free_pages == 8 and eng.cache.alloc.free_slots == 3
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("dt", [torch.float32, torch.bfloat16], ids=str)
+def test_long_prompts(dt):
+    """Prompts of more than a thousand tokens, whole and in long portions, time after time over the same pages and slots."""
+    target = ("cuda", dt)
+    cfg, w, eng = engine(config([parallel((8, 2, 64, 64), (2, 64, 64), ff=192)] * 2, vocab=64, width=128), target, tokens=6400)
+    ids = prompt(cfg, 1500, 2)
+    logits, _ = oracle.run(cfg, w, ids)
+    for sizes in ([1500], [1100, 400], [1500], [1024, 1, 475]):
+        s, at, got = eng.open_sequence(), 0, []
+        for n in sizes:
+            got.append(eng.feed([(s, ids[at:at + n], range(n))]))
+            at += n
+        assert error(torch.cat(got), logits) < tol(target, **LOGIT_TOL)
+        eng.close_sequence(s)
+
+
 def test_long_decoding(target):
     cfg = config([delta(4, 2, 32, 16, 4, 64), parallel((4, 2, 64, 64), (2, 16, 16), ff=64, tau=20.0)], vocab=97, width=64)
     cfg, w, eng = engine(cfg, target)
