@@ -565,6 +565,9 @@ if __name__ == "__main__":
     nums = [int(v) for v in sys.argv[2:]]
     if what == "membw":
         bench_membw(*nums)
+    if what == "hybrid":
+        from .bench_hybrid import run as bench_hybrid
+        bench_hybrid(*nums)
     if what == "moeprefill":
         bench_moeprefill(*nums)
     if what == "bf16moe":

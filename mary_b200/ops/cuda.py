@@ -222,6 +222,7 @@ def linear(x, w, bias=None):
         return _linear(x, w, bias)
 
 
+MATVEC_GLU_MAX_BYTES = 24 << 20  # the same for gate / up products (two rows per output: twice the bytes per launch)
 MATVEC_MAX_BYTES = 8 << 20       # one-token products up to this weight size take the SIMT matrix-vector stage (4 us against 6 us per launch)
 
 
@@ -250,6 +251,8 @@ def linear_f32(x, w, split_k: int | None = None, alpha: float = 1.0):
     if x.dtype == torch.float32 or K % 8 or x.stride(0) % 8 or w.stride(0) % 8:
         from .cuda_hybrid import gemm_simt
         return gemm_simt(x, w, alpha=alpha, out_f32=True)
+    if M == 1 and split_k is None and K <= 8192 and w.shape[0] * K * 2 <= MATVEC_MAX_BYTES and w.stride(1) == 1:
+        return step_matvec(x, w, mode="f32", alpha=alpha)
     sk = split_k or _auto_split_k(M, w.shape[0], K)
     with static_weights:
         return gemm_splitk(x, w, 0 if split_k is None else sk, f32=True, alpha=alpha) if sk > 1 else gemm(x, w, alpha=alpha, epi="f32")
@@ -260,6 +263,8 @@ def linear_glu(x, w_gu, act: str = "geglu"):
     if x.dtype == torch.float32 or x.shape[1] % 8 or w_gu.shape[0] % 16:
         from .cuda_hybrid import glu_any
         return glu_any(linear(x, w_gu), act)
+    if M == 1 and act in ("geglu", "swiglu") and x.shape[1] <= 8192 and w_gu.numel() * 2 <= MATVEC_GLU_MAX_BYTES and w_gu.stride(0) % 8 == 0:
+        return step_matvec(x, w_gu, mode=act)
     with static_weights:
         if M <= 128:
             return gemm(x, w_gu, glu=act)
@@ -729,19 +734,19 @@ def mla_unabsorb_o(o_lat, w_uv, H):
 
 
 # ------------------------------------------------------------------------------------------------- one-token decoder layer step
-declare("mary_step_matvec", "ppfpliippi" + "s")
+declare("mary_step_matvec", "ppfpliippi" + "fs")
 declare("mary_step_attention", "pppppppppp" + "iiiilffp" + "s")
 
 
-def step_matvec(h, w, gain=None, eps: float = 1e-6, res=None, mode: str = "plain"):
-    """One-token matrix-vector stage of the fused layer step: ``W x`` (``plain``), ``res + W x`` (``residual``) or
-    ``silu(W_gate x) * (W_up x)`` over ``w = [gate; up]`` (``swiglu``), with ``x = rms(h) * gain`` when ``gain`` is given,
+def step_matvec(h, w, gain=None, eps: float = 1e-6, res=None, mode: str = "plain", alpha: float = 1.0):
+    """One-token matrix-vector stage of the fused layer step: ``W x`` (``plain``), ``res + W x`` (``residual``), ``act(W_gate x) * (W_up x)``
+    over ``w = [gate; up]`` (``swiglu`` / ``geglu``) or ``alpha * W x`` as f32 (``f32``), with ``x = rms(h) * gain`` when ``gain`` is given,
     else ``x = h``.  ``h [1, K]`` -> ``[1, N]``."""
-    m = {"plain": 0, "residual": 1, "swiglu": 2}[mode]
+    m = {"plain": 0, "residual": 1, "swiglu": 2, "f32": 3, "geglu": 4}[mode]
     K = h.shape[-1]
-    N = w.shape[0] // 2 if m == 2 else w.shape[0]
-    y = _empty(1, N, dtype=torch.bfloat16, device=h.device)
-    check(lib().mary_step_matvec(_p(h), _p(gain), eps, _p(w), w.stride(0), N, K, _p(res), _p(y), m, _stream()), "step_matvec")
+    N = w.shape[0] // 2 if m in (2, 4) else w.shape[0]
+    y = _empty(1, N, dtype=torch.float32 if m == 3 else torch.bfloat16, device=h.device)
+    check(lib().mary_step_matvec(_p(h), _p(gain), eps, _p(w), w.stride(0), N, K, _p(res), _p(y), m, alpha, _stream()), "step_matvec")
     return y
 
 

@@ -264,7 +264,7 @@ def test_residual_ops(target, width):
     assert torch.equal(hd.cpu(), table[ids]) and torch.equal(x.float().cpu(), table[ids])
 
 
-@pytest.mark.parametrize("mkn", [(1, 72, 50), (7, 50, 33), (130, 64, 200), (70, 333, 65), (300, 128, 96)], ids=str)
+@pytest.mark.parametrize("mkn", [(1, 72, 50), (1, 256, 512), (7, 50, 33), (130, 64, 200), (70, 333, 65), (300, 128, 96)], ids=str)
 def test_linear_any_shape(target, mkn):
     dev, dt = target
     M, K, N = mkn
