@@ -22,9 +22,9 @@ CASES = [("prefill", 1, 4096), ("prefill", 8, 512), ("decode", 1, 2048), ("decod
 
 def tatizen_config(size: str) -> TatizenConfig:
     W, F, (H, G), L, (DH, DK) = SIZES[size]
-    par = LayerSpec(ParallelSpec(AttentionSpec(H, G, 128, 128, 128 ** -0.5), DecayedLinearSpec(L, 128, 128, 16.0), 0.8, 1.1), F)
+    par = LayerSpec(ParallelSpec(AttentionSpec(H, G, 128, 128, 128 ** -0.5), DecayedLinearSpec(L, 128, 128, 8.0), 0.9, 0.6), F)
     dlt = LayerSpec(DeltaSpec(DH, DK, 128, 128, 4), F)
-    return TatizenConfig(VOCAB, W, 1e-5, [par, dlt] * (LAYERS // 2), name=f"tatizen-{size}")
+    return TatizenConfig(VOCAB, W, 1e-6, [par, dlt] * (LAYERS // 2), name=f"tatizen-{size}")
 
 
 def dense_config(size: str):

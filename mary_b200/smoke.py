@@ -46,6 +46,22 @@ def _gemma_engine(dev):
     return m, out
 
 
+def _recurrent_engine(dev):
+    """A Tatizen decoder (attention beside decayed linear attention, gated delta rule) generating through the scheduler, two sequences."""
+    from .models.registry import family_of, make_engine
+    from .models.tatizen import TatizenConfig, TatizenModel, init_random_
+    layers = [{"type": "parallel", "mlp": {"kind": "dense", "ff": 512}, "mixer": {
+        "left": dict(heads=8, kv_heads=2, dim=64, vdim=64, scale=0.1), "right": dict(heads=4, dim=64, vdim=64, tau=8.0),
+        "left_scale": 0.9, "right_scale": 0.7}},
+        {"type": "delta", "mlp": {"kind": "dense", "ff": 512}, "mixer": dict(heads=4, kv_heads=2, dim=64, vdim=64, conv=4)}]
+    d = {"architecture": "Tatizen", "vocab": 1024, "width": 512, "norm": {"eps": 1e-6}, "layers": layers}
+    m = TatizenModel(TatizenConfig.from_json(d), dtype=torch.bfloat16, device=dev)
+    init_random_(m, 0)
+    out = make_engine(m, family_of(d), 512, 2, dev).generate([list(range(90)), [5, 4, 3]], 4)
+    assert all(len(o) == 4 for o in out)
+    return out
+
+
 def _lora_step(m, dev):
     from .train.trainer import LoraTrainer
     tr = LoraTrainer(m, rank=8, alpha=16.0, lr=1e-3)
@@ -63,9 +79,10 @@ def run_smoke() -> None:
     torch.cuda.set_device(0)
     n = _flagship(dev)
     m, out = _gemma_engine(dev)
+    rec = _recurrent_engine(dev)
     losses = _lora_step(m, dev)
     torch.cuda.synchronize()
     st = cuda.last_status()
     assert st == 0, f"kernel status {st}"
-    print(f"smoke ok: flagship emitted {n} tokens in 4 speculative steps; gemma {out}; lora loss {losses[0]:.3f} -> {losses[1]:.3f}; "
+    print(f"smoke ok: flagship emitted {n} tokens in 4 speculative steps; gemma {out}; tatizen {rec}; lora loss {losses[0]:.3f} -> {losses[1]:.3f}; "
           f"{cuda.LAUNCHES} kernel launches")

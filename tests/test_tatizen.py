@@ -70,7 +70,7 @@ def schedule(lengths: dict, rng, sizes=(1, 1, 2, 3, 5, 17, 40, 70)):
 
 
 # --------------------------------------------------------------------------- mechanisms alone
-ATTENTION = [(6, 3, 64, 64), (4, 4, 32, 48), (8, 1, 128, 128), (12, 2, 96, 40), (2, 2, 256, 256), (20, 1, 16, 24), (3, 1, 17, 33), (4, 2, 64, 128),
+ATTENTION = [(6, 2, 64, 64), (4, 4, 32, 48), (8, 1, 128, 128), (12, 2, 96, 40), (2, 2, 256, 256), (20, 1, 16, 24), (3, 1, 17, 33), (4, 2, 64, 128),
              (16, 2, 128, 128), (10, 1, 64, 64)]
 
 
@@ -141,7 +141,7 @@ def test_attention_finds_one_far_key(target, heads, decoded):
         assert error(out, want) < tol(target, 2e-5, 2e-2), j
 
 
-LINEAR = [(2, 32, 32), (3, 48, 40), (1, 128, 64), (2, 200, 24), (2, 20, 17), (2, 256, 8), (1, 9, 130)]
+LINEAR = [(2, 32, 64), (3, 48, 40), (1, 128, 64), (2, 200, 24), (2, 20, 17), (2, 256, 8), (1, 9, 130)]
 
 
 @pytest.mark.parametrize("shape", LINEAR, ids=str)
@@ -175,7 +175,7 @@ def test_decayed_linear_attention(target, shape, tau):
         assert error(out, torch.cat([want[s][a:a + n] for s, (a, n) in step.items()])) < tol(target, 5e-5, 1e-2)
 
 
-DELTA = [(4, 2, 64, 32, 4), (3, 3, 48, 40, 1), (6, 2, 128, 128, 3), (2, 1, 20, 17, 5), (2, 2, 200, 16, 2), (5, 1, 32, 70, 9)]
+DELTA = [(4, 2, 64, 48, 4), (3, 3, 48, 40, 1), (6, 2, 128, 128, 3), (2, 1, 20, 17, 5), (2, 2, 200, 16, 2), (5, 1, 32, 70, 9)]
 
 
 @pytest.mark.parametrize("shape", DELTA, ids=str)
