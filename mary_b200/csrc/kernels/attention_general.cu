@@ -21,7 +21,15 @@ struct GenParams {
   int max_pages, page_size, Hq, Hkv, G, GC, gchunks, DK, DV, RQ, nsplit, window;
   int64_t k_tok, k_page, v_tok, v_page, out_ld;
   float scale;
+  const float* bias;                     // [Hq][window], by distance, or null
+  const void* gate; int64_t gate_ld;     // rows of gate_ld elements, head h at h * DV: the output times its logistic function; or null
 };
+
+template <typename T>
+__device__ __forceinline__ T gated(const GenParams& p, float v, int64_t row, int col) {
+  if (p.gate) v *= sigmoid_x(to_f<T>(((const T*)p.gate)[row * p.gate_ld + col]));
+  return from_f<T>(v);
+}
 
 template <typename T, int NV>      // NV: value dims per lane
 __global__ void __launch_bounds__(WARPS * 32) attn_general_kernel(const GenParams p) {
@@ -85,7 +93,11 @@ __global__ void __launch_bounds__(WARPS * 32) attn_general_kernel(const GenParam
       const int rr = warp * RPW + r;
       const int qp = pos0 + rr / gc;
       const bool ok = rr < R && lane < nk && kp <= qp && (p.window <= 0 || qp - kp < p.window);
-      const float sv_ = ok ? s[r] * p.scale : -INFINITY;
+      float sv_ = -INFINITY;
+      if (ok) {
+        sv_ = s[r] * p.scale;
+        if (p.bias) sv_ += p.bias[(int64_t)(kvh * p.G + g0 + rr % gc) * p.window + (qp - kp)];
+      }
       const float mx = fmaxf(m[r], warp_max(sv_));
       pr[r] = 0.f;
       if (mx == -INFINITY) continue;                // warp-uniform: nothing visible to this row yet
@@ -113,11 +125,13 @@ __global__ void __launch_bounds__(WARPS * 32) attn_general_kernel(const GenParam
     const int rr = warp * RPW + r;
     if (rr >= R) continue;
     if (p.nsplit == 1) {
-      T* dst = (T*)p.out + (int64_t)(row0 + rr / gc) * p.out_ld + (int64_t)(kvh * p.G + g0 + rr % gc) * p.DV;
+      const int64_t row = row0 + rr / gc;
+      const int col = (kvh * p.G + g0 + rr % gc) * p.DV;
+      T* dst = (T*)p.out + row * p.out_ld + col;
       const float inv = l[r] > 0.f ? 1.0f / l[r] : 0.f;
 #pragma unroll
       for (int v = 0; v < NV; ++v)
-        if (lane + 32 * v < p.DV) dst[lane + 32 * v] = from_f<T>(o[r][v] * inv);
+        if (lane + 32 * v < p.DV) dst[lane + 32 * v] = gated<T>(p, o[r][v] * inv, row, col + lane + 32 * v);
     } else {
       const int64_t pi = (((int64_t)nb * gridDim.y + blockIdx.y) * p.nsplit + split) * ROWS + rr;
 #pragma unroll
@@ -148,7 +162,9 @@ __global__ void attn_general_combine_kernel(const GenParams p) {
       ll += p.part_ml[pi * 2 + 1] * c;
       acc += p.part_o[pi * p.DV + d] * c;
     }
-    ((T*)p.out)[(int64_t)(row0 + r / gc) * p.out_ld + (int64_t)(kvh * p.G + g0 + r % gc) * p.DV + d] = from_f<T>(ll > 0.f ? acc / ll : 0.f);
+    const int64_t row = row0 + r / gc;
+    const int col = (kvh * p.G + g0 + r % gc) * p.DV + d;
+    ((T*)p.out)[row * p.out_ld + col] = gated<T>(p, ll > 0.f ? acc / ll : 0.f, row, col);
   }
 }
 
@@ -184,17 +200,19 @@ MARY_API int64_t mary_attention_general_scratch_floats(int NB, int Hq, int Hkv, 
 }
 
 // q [T, Hq, DK] contiguous; caches with element strides per token and per page, heads contiguous inside a token row; out rows of
-// out_ld elements, head h at h * DV.  blk_seq / blk_q0: NB blocks of at most RQ query tokens that never cross a sequence.
+// out_ld elements, head h at h * DV.  bias [Hq][window] (or null) is added to the scaled score by distance, gate (or null) multiplies the
+// output by its logistic function.  blk_seq / blk_q0: NB blocks of at most RQ query tokens that never cross a sequence.
 MARY_API int mary_attention_general(const void* q, const void* kc, const void* vc, void* out, const int* page_table, const int* kv_len,
                                     const int* q_start, const int* blk_seq, const int* blk_q0, int NB, int max_pages, int page_size, int64_t k_tok,
                                     int64_t k_page, int64_t v_tok, int64_t v_page, int64_t out_ld, int Hq, int Hkv, int DK, int DV, int RQ,
-                                    int nsplit, int window, float scale, float* scratch, int f32, cudaStream_t s) {
+                                    int nsplit, int window, float scale, const float* bias, const void* gate, int64_t gate_ld,
+                                    float* scratch, int f32, cudaStream_t s) {
   if (NB <= 0) return MARY_OK;
-  if (Hkv < 1 || Hq % Hkv || DK < 1 || DV < 1 || DK > 512 || DV > 512 || nsplit < 1) return MARY_ERR_BAD_ARG;
+  if (Hkv < 1 || Hq % Hkv || DK < 1 || DV < 1 || DK > 640 || DV > 512 || nsplit < 1 || (bias && window < 1)) return MARY_ERR_BAD_ARG;
   GenParams p;
   p.q = q; p.kc = kc; p.vc = vc; p.out = out; p.page_table = page_table; p.kv_len = kv_len; p.q_start = q_start; p.blk_seq = blk_seq; p.blk_q0 = blk_q0;
   p.max_pages = max_pages; p.page_size = page_size; p.Hq = Hq; p.Hkv = Hkv; p.G = Hq / Hkv; p.DK = DK; p.DV = DV; p.RQ = RQ; p.nsplit = nsplit;
-  p.window = window; p.k_tok = k_tok; p.k_page = k_page; p.v_tok = v_tok; p.v_page = v_page; p.out_ld = out_ld; p.scale = scale;
+  p.window = window; p.k_tok = k_tok; p.k_page = k_page; p.v_tok = v_tok; p.v_page = v_page; p.out_ld = out_ld; p.scale = scale; p.bias = bias; p.gate = gate; p.gate_ld = gate_ld;
   p.GC = p.G < ROWS ? p.G : ROWS;
   p.gchunks = (p.G + p.GC - 1) / p.GC;
   if (RQ < 1 || RQ * p.GC > ROWS || (nsplit > 1 && !scratch)) return MARY_ERR_BAD_ARG;

@@ -12,8 +12,10 @@ constexpr int BM = 64, BN = 64, BK = 16, NT = 256;
 
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(NT) gemm_simt_kernel(const TI* __restrict__ X, const TI* __restrict__ W, TO* __restrict__ out, int M, int N, int K,
-                                                       int64_t ldx, int64_t ldw, int64_t ldo, float alpha, int accumulate) {
+                                                       int64_t ldx, int64_t ldw, int64_t ldo, float alpha, int accumulate, int64_t bsx, int64_t bsw,
+                                                       int64_t bso) {
   pdl_sync();
+  X += blockIdx.z * bsx; W += blockIdx.z * bsw; out += blockIdx.z * bso;
   __shared__ float sx[2][BK][BM + 4], sw[2][BK][BN + 4];
   const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
   const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
@@ -69,17 +71,25 @@ __global__ void __launch_bounds__(NT) gemm_simt_kernel(const TI* __restrict__ X,
 
 }  // namespace
 
-// x_f32: X and W are f32 (else both bf16); out_f32: out is f32 (else bf16)
-MARY_API int mary_gemm_simt(const void* X, const void* W, void* out, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldo, float alpha,
-                            int accumulate, int x_f32, int out_f32, cudaStream_t s) {
+// `batch` products over strided views (element strides bsx / bsw / bso).  x_f32: X and W are f32 (else both bf16); out_f32: out is f32 (else bf16)
+MARY_API int mary_gemm_simt_batched(const void* X, const void* W, void* out, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldo, int batch,
+                                    int64_t bsx, int64_t bsw, int64_t bso, float alpha, int accumulate, int x_f32, int out_f32, cudaStream_t s) {
   if (M <= 0) return MARY_OK;
-  if (N <= 0 || K <= 0 || (M + BM - 1) / BM > 65535) return MARY_ERR_BAD_ARG;
-  const dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
+  if (N <= 0 || K <= 0 || (M + BM - 1) / BM > 65535 || batch < 1 || batch > 65535) return MARY_ERR_BAD_ARG;
+  const dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM, batch);
   using B = __nv_bfloat16;
-  if (x_f32 && out_f32) MARY_LAUNCH((gemm_simt_kernel<float, float>), grid, NT, 0, s, (const float*)X, (const float*)W, (float*)out, M, N, K, ldx, ldw, ldo, alpha, accumulate);
+  if (x_f32 && out_f32)
+    MARY_LAUNCH((gemm_simt_kernel<float, float>), grid, NT, 0, s, (const float*)X, (const float*)W, (float*)out, M, N, K, ldx, ldw, ldo, alpha, accumulate, bsx, bsw, bso);
   else if (x_f32) return MARY_ERR_BAD_ARG;
-  else if (out_f32) MARY_LAUNCH((gemm_simt_kernel<B, float>), grid, NT, 0, s, (const B*)X, (const B*)W, (float*)out, M, N, K, ldx, ldw, ldo, alpha, accumulate);
-  else MARY_LAUNCH((gemm_simt_kernel<B, B>), grid, NT, 0, s, (const B*)X, (const B*)W, (B*)out, M, N, K, ldx, ldw, ldo, alpha, accumulate);
+  else if (out_f32)
+    MARY_LAUNCH((gemm_simt_kernel<B, float>), grid, NT, 0, s, (const B*)X, (const B*)W, (float*)out, M, N, K, ldx, ldw, ldo, alpha, accumulate, bsx, bsw, bso);
+  else
+    MARY_LAUNCH((gemm_simt_kernel<B, B>), grid, NT, 0, s, (const B*)X, (const B*)W, (B*)out, M, N, K, ldx, ldw, ldo, alpha, accumulate, bsx, bsw, bso);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
+}
+
+MARY_API int mary_gemm_simt(const void* X, const void* W, void* out, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldo, float alpha,
+                            int accumulate, int x_f32, int out_f32, cudaStream_t s) {
+  return mary_gemm_simt_batched(X, W, out, M, N, K, ldx, ldw, ldo, 1, 0, 0, 0, alpha, accumulate, x_f32, out_f32, s);
 }

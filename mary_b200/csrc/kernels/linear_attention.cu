@@ -2,17 +2,14 @@
 // low-rank projection, the short convolutions with their unit norms and gates, the convolution history, the gated norm of the
 // read-out, and the fused one-token steps that do all of it in one launch per layer.  Decays, gates, unit norms and the state are in
 // exact 32-bit arithmetic.
-//
-// Convolution history: the last `taps` inputs of every channel in a ring addressed by absolute position, [slot][taps][channels].  A
-// token at position p reads the entries of p - 1 .. p - (taps - 1) and writes the entry of p, which none of those reads touches.
 #include "host_utils.h"
-#include "typed.cuh"
+#include "recurrent.cuh"
 
 using namespace mary;
 
 namespace {
 
-constexpr int NT = 256;
+constexpr int NT = STEP_THREADS;
 
 // decay[t, c] = sigmoid(a2[c] . x[t] + bias[c]) ^ inv_tau, x[t] of `rank` values
 template <typename T>
@@ -57,88 +54,6 @@ struct ConvIn {
   int HK, H, DK, DV, taps, C;      // C = 2 HK DK + H DV channels, in the order q, k, v; taps [C][taps], last one the current token's
 };
 
-// silu of the depthwise causal convolution of channel c at row t (position pos of its sequence, whose portion starts at row first)
-template <typename T>
-__device__ __forceinline__ float conv_silu(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, const T* __restrict__ ring, int taps, int C,
-                                           int c, int t, int first, int pos) {
-  float acc = 0.f;
-  for (int d = 0; d < taps; ++d) {                     // d tokens back
-    float v = 0.f;
-    if (t - d >= first) v = to_f<T>(x[(int64_t)(t - d) * ldx + c]);
-    else if (pos - d >= 0) v = to_f<T>(ring[(int64_t)((pos - d) % taps) * C + c]);
-    acc = fmaf(to_f<T>(w[(int64_t)c * taps + taps - 1 - d]), v, acc);
-  }
-  return silu_t<T>(acc);
-}
-
-// silu(conv) of E channels from c on for the four tokens of a block: rows rb .. rb + 3 (a sequence's portion is rows first .. end - 1),
-// the block's first token at position pos.  Rows before the portion come from the ring, positions before 0 are zero.
-template <typename T, int TAPS, int E>
-__device__ __forceinline__ void conv_block(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, const T* __restrict__ ring, int n_taps, int C,
-                                           int c, int rb, int first, int end, int pos, float (&y)[4][E]) {
-  const int taps = TAPS > 0 ? TAPS : n_taps;
-  float wr[E][TAPS > 0 ? TAPS : 1];
-  if constexpr (TAPS > 0) {
-#pragma unroll
-    for (int e = 0; e < E; ++e) {
-      if constexpr (TAPS == 4 && E == 4) {
-        load_e<T, 4>(w + (int64_t)(c + e) * 4, wr[e]);
-      } else {
-#pragma unroll
-        for (int j = 0; j < TAPS; ++j) wr[e][j] = to_f<T>(w[(int64_t)(c + e) * TAPS + j]);
-      }
-    }
-  }
-#pragma unroll
-  for (int i = 0; i < 4; ++i)
-#pragma unroll
-    for (int e = 0; e < E; ++e) y[i][e] = 0.f;
-  if constexpr (TAPS > 0) {
-    // all rows are requested before the first is used
-    float v[TAPS + 3][E];
-#pragma unroll
-    for (int r = 1 - TAPS; r < 4; ++r) {
-      const bool here = rb + r >= first;
-      const T* src = here ? x + (int64_t)(rb + r) * ldx + c : ring + (int64_t)((pos + r + TAPS) % TAPS) * C + c;
-      if (rb + r < end && pos + r >= 0) load_e<T, E>(src, v[r + TAPS - 1]);
-      else
-#pragma unroll
-        for (int e = 0; e < E; ++e) v[r + TAPS - 1][e] = 0.f;
-    }
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int d = 0; d < TAPS; ++d)
-#pragma unroll
-        for (int e = 0; e < E; ++e) y[i][e] = fmaf(wr[e][TAPS - 1 - d], v[i - d + TAPS - 1][e], y[i][e]);
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int e = 0; e < E; ++e) y[i][e] = silu_t<T>(y[i][e]);
-    return;
-  }
-  for (int r = 1 - taps; r < 4; ++r) {
-    float v[E] = {};
-    if (rb + r >= end) break;
-    if (rb + r >= first) load_e<T, E>(x + (int64_t)(rb + r) * ldx + c, v);
-    else if (pos + r >= 0) load_e<T, E>(ring + (int64_t)((pos + r) % taps) * C + c, v);
-    else continue;
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int d = i - r;
-      if (d < 0 || d >= taps) continue;
-#pragma unroll
-      for (int e = 0; e < E; ++e) {
-        y[i][e] = fmaf(to_f<T>(w[(int64_t)(c + e) * taps + taps - 1 - d]), v[e], y[i][e]);
-      }
-    }
-  }
-#pragma unroll
-  for (int i = 0; i < 4; ++i)
-#pragma unroll
-    for (int e = 0; e < E; ++e) y[i][e] = silu_t<T>(y[i][e]);
-}
-
 // One warp per (sequence, block of four tokens, item); items: HK query / key heads (unit vectors, and the products of the block's keys
 // with its keys and queries), H value heads (with their gates).  VEC: widths, pitch and addresses allow accesses of four values.
 template <typename T, int TAPS, bool VEC>
@@ -170,8 +85,8 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const T* __restrict__ x
     for (int i = 0; i < NI; ++i) {
       const int c = i * 32 * E + lane * E;
       if (c < ci.DK) {
-        conv_block<T, TAPS, E>(x, ldx, w, ring, ci.taps, ci.C, it * ci.DK + c, rb, first, end, pos, yq[i]);
-        conv_block<T, TAPS, E>(x, ldx, w, ring, ci.taps, ci.C, (ci.HK + it) * ci.DK + c, rb, first, end, pos, yk[i]);
+        conv_block<T, TAPS, E>(x, ldx, w, (const T*)nullptr, ring, ci.taps, ci.C, it * ci.DK + c, rb, first, end, pos, yq[i]);
+        conv_block<T, TAPS, E>(x, ldx, w, (const T*)nullptr, ring, ci.taps, ci.C, (ci.HK + it) * ci.DK + c, rb, first, end, pos, yk[i]);
       } else {
 #pragma unroll
         for (int t = 0; t < 4; ++t)
@@ -232,7 +147,7 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const T* __restrict__ x
   const int c0 = 2 * ci.HK * ci.DK + h * ci.DV;
   for (int c = lane * E; c < ci.DV; c += 32 * E) {
     float y[4][E];
-    conv_block<T, TAPS, E>(x, ldx, w, ring, ci.taps, ci.C, c0 + c, rb, first, end, pos, y);
+    conv_block<T, TAPS, E>(x, ldx, w, (const T*)nullptr, ring, ci.taps, ci.C, c0 + c, rb, first, end, pos, y);
 #pragma unroll
     for (int t = 0; t < 4; ++t)
       if (t < nt) store_e<float, E>(v + ((int64_t)(rb + t) * ci.H + h) * ci.DV + c, y[t]);
@@ -301,63 +216,6 @@ __global__ void gated_head_norm_kernel(const float* __restrict__ o, const T* __r
 }
 
 // ----------------------------------------------------------------------------------------------- fused one-token steps
-// One CTA per (sequence, head): 8 lanes per state column, 32 columns at a time, the next columns' state in flight while the
-// current ones are updated.  The read-out of all columns meets in shared memory for the head norm.
-template <int NR4>
-__device__ __forceinline__ void load_cols(float4 (&st)[NR4], const float* state, int col, int DV, int DKS, bool fresh, int lane8) {
-#pragma unroll
-  for (int r = 0; r < NR4; ++r) {
-    const int c = (r * 8 + lane8) * 4;
-    st[r] = (!fresh && col < DV && c < DKS) ? __ldcs((const float4*)(state + (int64_t)col * DKS + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
-  }
-}
-
-__device__ __forceinline__ float sum8(float v) {
-#pragma unroll
-  for (int o = 4; o >= 1; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
-
-// sq / sk [NR4 * 32] (zero beyond DK), sa [NR4 * 32] channel decays (DELTA: the scalars g and b instead), sv [DV]; leaves o in so[DV].
-template <int NR4, bool DELTA>
-__device__ __forceinline__ void step_columns(float4 (&st)[NR4], float* state, int DV, int DKS, bool fresh, const float* sq, const float* sk,
-                                             const float* sa, float g, float b, const float* sv, float* so) {
-  const int lane8 = threadIdx.x & 7;
-  for (int col = threadIdx.x >> 3, c0 = 0; c0 < DV; c0 += NT / 8, col += NT / 8) {
-    float4 nx[NR4];
-    if (c0 + NT / 8 < DV) load_cols<NR4>(nx, state, col + NT / 8, DV, DKS, fresh, lane8);
-    const float vt = col < DV ? sv[col] : 0.f;
-    float w = vt;
-    if constexpr (DELTA) {
-      float pred = 0.f;
-#pragma unroll
-      for (int r = 0; r < NR4; ++r) {
-        const float4 k4 = *(const float4*)(sk + (r * 8 + lane8) * 4);
-        st[r].x *= g; st[r].y *= g; st[r].z *= g; st[r].w *= g;
-        pred = fmaf(k4.x, st[r].x, fmaf(k4.y, st[r].y, fmaf(k4.z, st[r].z, fmaf(k4.w, st[r].w, pred))));
-      }
-      w = b * (vt - sum8(pred));
-    }
-    float acc = 0.f;
-#pragma unroll
-    for (int r = 0; r < NR4; ++r) {
-      const int c = (r * 8 + lane8) * 4;
-      const float4 k4 = *(const float4*)(sk + c), q4 = *(const float4*)(sq + c);
-      if constexpr (!DELTA) {
-        const float4 a4 = *(const float4*)(sa + c);
-        st[r].x *= a4.x; st[r].y *= a4.y; st[r].z *= a4.z; st[r].w *= a4.w;
-      }
-      st[r].x = fmaf(k4.x, w, st[r].x); st[r].y = fmaf(k4.y, w, st[r].y); st[r].z = fmaf(k4.z, w, st[r].z); st[r].w = fmaf(k4.w, w, st[r].w);
-      acc = fmaf(q4.x, st[r].x, fmaf(q4.y, st[r].y, fmaf(q4.z, st[r].z, fmaf(q4.w, st[r].w, acc))));
-      if (col < DV && c < DKS) __stcs((float4*)(state + (int64_t)col * DKS + c), st[r]);
-    }
-    acc = sum8(acc);
-    if (lane8 == 0 && col < DV) so[col] = acc;
-#pragma unroll
-    for (int r = 0; r < NR4; ++r) st[r] = nx[r];
-  }
-}
-
 template <typename T>
 __device__ __forceinline__ void finish_head(const float* so, float* red, const T* gate, const T* gain, T* y, int DV, float eps, float scale) {
   float ss = 0.f;
@@ -403,7 +261,7 @@ __global__ void __launch_bounds__(NT) decay_step_kernel(const T* __restrict__ q,
   }
   for (int c = threadIdx.x; c < io.DV; c += NT) sv[c] = to_f<T>(v[row + (int64_t)h * io.DV + c]);
   __syncthreads();
-  step_columns<NR4, false>(st, state, io.DV, io.DKS, fresh, sq, sk, sa, 0.f, 0.f, sv, so);
+  step_columns<NR4, DECAY_CHANNEL>(st, state, io.DV, io.DKS, fresh, sq, sk, sa, 0.f, 0.f, sv, so);
   __syncthreads();
   finish_head<T>(so, red, gate + row + (int64_t)h * io.DV, gain, y + (int64_t)t * ldy + (int64_t)h * io.DV, io.DV, io.eps, io.out_scale);
 }
@@ -435,7 +293,7 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(const T* __restrict__ x,
     float f = 0.f;
     if (part == 2 || c < io.DK) {
       const int ch = part == 2 ? 2 * io.HK * io.DK + h * io.DV + c : (part * io.HK + hk) * io.DK + c;
-      f = conv_silu<T>(x, ldx, w, ring, taps, C, ch, t, t, pos);
+      f = conv_silu<T>(x, ldx, w, (const T*)nullptr, ring, taps, C, ch, t, t, pos);
       if (part == 2 || h % rep == 0) ring[(int64_t)(pos % taps) * C + ch] = x[row + ch];   // one head of the group records the shared channels
     }
     if (part == 0) { sq[c] = f; sq2 += f * f; }
@@ -448,7 +306,7 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(const T* __restrict__ x,
   const float b = sigmoid_x(to_f<T>(b_in[row + h]));
   const float g = expf(-expf(a_log[h]) * softplus_x(to_f<T>(a_in[row + h]) + dt_bias[h]));
   __syncthreads();
-  step_columns<NR4, true>(st, state, io.DV, io.DKS, fresh, sq, sk, nullptr, g, b, sv, so);
+  step_columns<NR4, DECAY_DELTA>(st, state, io.DV, io.DKS, fresh, sq, sk, nullptr, g, b, sv, so);
   __syncthreads();
   finish_head<T>(so, red, gate + row + (int64_t)h * io.DV, gain, y + (int64_t)t * ldy + (int64_t)h * io.DV, io.DV, io.eps, io.out_scale);
 }

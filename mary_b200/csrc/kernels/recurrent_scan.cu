@@ -1,6 +1,7 @@
 // Linear recurrences over the tokens of a batch, with the state in 32-bit registers:
 //
 //   decayed linear attention   S_t = diag(a_t) S_{t-1} + k_t v_t^T                       o_t = S_t^T q_t    (a decay per key channel)
+//   decay per head             S_t = g_t S_{t-1} + b_t k_t v_t^T                         o_t = S_t^T q_t + skip v_t
 //   gated delta rule           S' = g_t S_{t-1};  u_t = b_t (v_t - S'^T k_t);  S_t = S' + k_t u_t^T;  o_t = S_t^T q_t   (a decay per head)
 //
 // The columns of S (one per value channel) are independent, so the grid is (column block, head, sequence) and every CTA walks the
@@ -16,9 +17,9 @@
 //   u_i = b_i (v_i - G_i S_0^T k_i - sum_{j<i} w_ij (k_j . k_i) u_j),   o_i = G_i S_0^T q_i + sum_{j<=i} w_ij (k_j . q_i) u_j,
 //   S_4 = G_4 S_0 + sum_j w_4j k_j u_j^T,
 // which needs one round of reductions per four tokens; the products k.k and k.q do not depend on the column and are precomputed
-// (mary_delta_prep).  The weights w are products of decays, never quotients, so a decay of zero is exact.
+// (mary_delta_prep).  A decay per head without the delta rule is the same with u_i = b_i v_i: half the reads, no chain.  The weights w are products of decays, never quotients, so a decay of zero is exact.
 #include "host_utils.h"
-#include "typed.cuh"
+#include "recurrent.cuh"
 
 using namespace mary;
 
@@ -52,8 +53,10 @@ __device__ __forceinline__ f2 mul2(f2 a, f2 b) {
 struct ScanParams {
   const void* q; const void* k; const void* v;      // token rows of ldq / ldk / ldv elements; q, k head h / rep, v head h
   const float* decay;                               // [T, H * DK] per channel, or [T, H] per head
-  const float* beta;                                // [T, H] (delta rule)
-  const float* pairs;                               // [T, HK, 8] (delta rule): k_j . k_i and k_j . q_i of the row's block of four
+  const float* beta;                                // [T, H] (decay per head, delta rule)
+  const float* pairs;                               // [T, HK, 8] (delta rule): k_j . k_i and k_j . q_i of the row's block of four;
+                                                    // [T, HK, 4] (decay per head): k_j . q_i
+  const float* skip;                                // [H] (decay per head)
   float* out;                                       // [T, H * DV]
   float* state;                                     // [slots][H][DV][DKS]
   const int* q_start; const int* kv_len; const int* slots;
@@ -66,13 +69,14 @@ template <typename TI, int E> struct Reg { uint4 v; };             // one 16-byt
 template <typename TI> struct Reg<TI, 1> { TI v; };
 
 // LN lanes share a group of CN columns: 16, or 32 when the grid is small.
-template <typename TI, int NR4, bool DELTA, bool VEC, int NT, int LN>
+template <typename TI, int NR4, int MODE, bool VEC, int NT, int LN>
 __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
   pdl_sync();
+  constexpr bool BLOCKS = MODE != DECAY_CHANNEL, DELTA = MODE == DECAY_DELTA;
   constexpr int COLS = NT / LN * CN, DKP = NR4 * LN * 4;
   constexpr int TPT = NT / CT;                                     // staging threads per token
   constexpr int E = VEC ? Pack<TI>::N : 1, NVQ = (DKP / E + TPT - 1) / TPT;
-  constexpr int EA = VEC ? 4 : 1, NVA = DELTA ? 1 : (DKP / EA + TPT - 1) / TPT;
+  constexpr int EA = VEC ? 4 : 1, NVA = BLOCKS ? 1 : (DKP / EA + TPT - 1) / TPT;
   constexpr int NVV = COLS / TPT;
   typedef float Rows[CT][DKP];
   extern __shared__ __align__(16) float sm[];
@@ -97,7 +101,7 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
       st[c][r][0] = v.x; st[c][r][1] = v.y;
     }
   if (p.DK < DKP) {                       // channels beyond DK stay zero in both buffers
-    for (int i = tid; i < (DELTA ? 4 : 6) * CT * DKP; i += NT) sm[i] = 0.f;
+    for (int i = tid; i < (BLOCKS ? 4 : 6) * CT * DKP; i += NT) sm[i] = 0.f;
     __syncthreads();
   }
   // staging: this thread's token of a chunk and its channels
@@ -105,10 +109,12 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
   const TI* qp = (const TI*)p.q + (int64_t)(row0 + my_t) * p.ldq + (int64_t)hk * p.DK + my_c * E;
   const TI* kp = (const TI*)p.k + (int64_t)(row0 + my_t) * p.ldk + (int64_t)hk * p.DK + my_c * E;
   const TI* vp = (const TI*)p.v + (int64_t)(row0 + my_t) * p.ldv + (int64_t)h * p.DV + blockIdx.x * COLS + my_c;
-  const float* ap = DELTA ? p.decay + (int64_t)(row0 + lane) * p.H + h : p.decay + ((int64_t)(row0 + my_t) * p.H + h) * p.DK + my_c * EA;
-  const float* bp = DELTA ? p.beta + (int64_t)(row0 + lane) * p.H + h : nullptr;
-  const float4* pp = DELTA ? (const float4*)p.pairs + ((int64_t)(row0 + lane) * p.HK + hk) * 2 : nullptr;
-  const int64_t step_q = CT * p.ldq, step_k = CT * p.ldk, step_v = CT * p.ldv, step_a = (int64_t)CT * p.H * (DELTA ? 1 : p.DK);
+  const float* ap = BLOCKS ? p.decay + (int64_t)(row0 + lane) * p.H + h : p.decay + ((int64_t)(row0 + my_t) * p.H + h) * p.DK + my_c * EA;
+  const float* bp = BLOCKS ? p.beta + (int64_t)(row0 + lane) * p.H + h : nullptr;
+  constexpr int NP = DELTA ? 2 : 1;
+  const float4* pp = BLOCKS ? (const float4*)p.pairs + ((int64_t)(row0 + lane) * p.HK + hk) * NP : nullptr;
+  const float skip = MODE == DECAY_HEAD ? p.skip[h] : 0.f;
+  const int64_t step_q = CT * p.ldq, step_k = CT * p.ldk, step_v = CT * p.ldv, step_a = (int64_t)CT * p.H * (BLOCKS ? 1 : p.DK);
   const int ch_left = p.DK - my_c * E, ch_left_a = p.DK - my_c * EA, col_left = p.DV - blockIdx.x * COLS - my_c;
 
   Reg<TI, E> rq[NVQ], rk[NVQ];
@@ -128,7 +134,7 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
     }
 #pragma unroll
     for (int i = 0; i < NVV; ++i) rv[i] = (in && i * TPT < col_left) ? vp[i * TPT] : from_f<TI>(0.f);
-    if constexpr (!DELTA) {
+    if constexpr (!BLOCKS) {
 #pragma unroll
       for (int i = 0; i < NVA; ++i) {
         if (in && i * TPT * EA < ch_left_a) ra[i].v = *(const decltype(ra[i].v)*)(ap + i * TPT * EA);
@@ -139,10 +145,10 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
       const bool mine = t0 + tid < n;
       rg = mine ? *ap : 1.f;
       rb = mine ? *bp : 0.f;
-      rkk = mine ? pp[0] : make_float4(0.f, 0.f, 0.f, 0.f);
-      rkq = mine ? pp[1] : make_float4(0.f, 0.f, 0.f, 0.f);
+      if constexpr (DELTA) rkk = mine ? pp[0] : make_float4(0.f, 0.f, 0.f, 0.f);
+      rkq = mine ? pp[NP - 1] : make_float4(0.f, 0.f, 0.f, 0.f);
       bp += step_a;
-      pp += CT * p.HK * 2;
+      pp += CT * p.HK * NP;
     }
     qp += step_q; kp += step_k; vp += step_v; ap += step_a;
   };
@@ -168,7 +174,7 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
     }
 #pragma unroll
     for (int i = 0; i < NVV; ++i) sv[b][my_t][my_c + i * TPT] = to_f<TI>(rv[i]);
-    if constexpr (!DELTA) {
+    if constexpr (!BLOCKS) {
 #pragma unroll
       for (int i = 0; i < NVA; ++i) {
         if (i * TPT * EA < ch_left_a) {
@@ -194,7 +200,7 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
         else suffix *= g[j];
       }
       if (lane < CT) {
-        *(float4*)s_kk[b][lane] = make_float4(w[0] * rkk.x, w[1] * rkk.y, w[2] * rkk.z, w[3] * rkk.w);
+        if constexpr (DELTA) *(float4*)s_kk[b][lane] = make_float4(w[0] * rkk.x, w[1] * rkk.y, w[2] * rkk.z, w[3] * rkk.w);
         *(float4*)s_kq[b][lane] = make_float4(w[0] * rkq.x * p.q_scale, w[1] * rkq.y * p.q_scale, w[2] * rkq.z * p.q_scale, w[3] * rkq.w * p.q_scale);
         *(float4*)s_row[b][lane] = make_float4(G, suffix, rb, 0.f);
       }
@@ -207,7 +213,7 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
   for (int t0 = 0, b = 0; t0 < n; t0 += CT, b ^= 1) {
     const bool more = t0 + CT < n;
     if (more) fetch(t0 + CT);
-    if constexpr (!DELTA) {
+    if constexpr (!BLOCKS) {
       float o[CT * CN];                              // index token * 4 + column
 #pragma unroll
       for (int t = 0; t < CT; ++t) {
@@ -245,19 +251,20 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
 #pragma unroll
       for (int blk = 0; blk < 2; ++blk) {
         const int tb = blk * 4, my_col = ln / (LN / 4);
-        float d[CN * 8];                             // index column * 8 + {S_0^T k_0 .. k_3, S_0^T q_0 .. q_3}
+        constexpr int ND = DELTA ? 8 : 4;            // S_0^T k_0 .. k_3 (delta rule), S_0^T q_0 .. q_3
+        float d[CN * ND];                            // index column * ND + product
         {
-          f2 acc[CN][8];
+          f2 acc[CN][ND];
 #pragma unroll
           for (int c = 0; c < CN; ++c)
 #pragma unroll
-            for (int i = 0; i < 8; ++i) acc[c][i] = 0ull;
+            for (int i = 0; i < ND; ++i) acc[c][i] = 0ull;
 #pragma unroll
           for (int r = 0; r < NR4; ++r) {
             const int row = (r * LN + ln) * 4;
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-              const ulonglong2 x = *(const ulonglong2*)(i < 4 ? &sk[b][tb + i][row] : &sq[b][tb + i - 4][row]);
+            for (int i = 0; i < ND; ++i) {
+              const ulonglong2 x = *(const ulonglong2*)(i < ND - 4 ? &sk[b][tb + i][row] : &sq[b][tb + i - (ND - 4)][row]);
 #pragma unroll
               for (int c = 0; c < CN; ++c) acc[c][i] = fma2(x.y, st[c][r][1], fma2(x.x, st[c][r][0], acc[c][i]));
             }
@@ -265,24 +272,33 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
 #pragma unroll
           for (int c = 0; c < CN; ++c)
 #pragma unroll
-            for (int i = 0; i < 8; ++i) d[c * 8 + i] = sum2(acc[c][i]);
+            for (int i = 0; i < ND; ++i) d[c * ND + i] = sum2(acc[c][i]);
         }
-        halve<32>(d, lane, LN / 2);
-        halve<16>(d, lane, LN / 4);                  // the lane's column is my_col
+        halve<CN * ND>(d, lane, LN / 2);
+        halve<CN * ND / 2>(d, lane, LN / 4);         // the lane's column is my_col
 #pragma unroll
         for (int bit = LN / 8; bit >= 1; bit >>= 1)
 #pragma unroll
-          for (int i = 0; i < 8; ++i) d[i] += __shfl_xor_sync(0xffffffffu, d[i], bit);
+          for (int i = 0; i < ND; ++i) d[i] += __shfl_xor_sync(0xffffffffu, d[i], bit);
         float u[4], mine = 0.f, G4 = 1.f;
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const float4 row = *(const float4*)s_row[b][tb + i];
-          const float4 kk = *(const float4*)s_kk[b][tb + i], kq = *(const float4*)s_kq[b][tb + i];
-          const float kkv[4] = {kk.x, kk.y, kk.z, kk.w}, kqv[4] = {kq.x, kq.y, kq.z, kq.w};
-          float pred = row.x * d[i], oi = row.x * d[4 + i];
+          const float4 kq = *(const float4*)s_kq[b][tb + i];
+          const float kqv[4] = {kq.x, kq.y, kq.z, kq.w};
+          const float vt = sv[b][tb + i][gcol + my_col];
+          float oi = row.x * d[ND - 4 + i];
+          if constexpr (DELTA) {
+            const float4 kk = *(const float4*)s_kk[b][tb + i];
+            const float kkv[4] = {kk.x, kk.y, kk.z, kk.w};
+            float pred = row.x * d[i];
 #pragma unroll
-          for (int j = 0; j < i; ++j) pred = fmaf(kkv[j], u[j], pred);
-          u[i] = row.z * (sv[b][tb + i][gcol + my_col] - pred);
+            for (int j = 0; j < i; ++j) pred = fmaf(kkv[j], u[j], pred);
+            u[i] = row.z * (vt - pred);
+          } else {
+            u[i] = row.z * vt;
+            oi = fmaf(skip, vt, oi);
+          }
 #pragma unroll
           for (int j = 0; j <= i; ++j) oi = fmaf(kqv[j], u[j], oi);
           if ((ln & 3) == i) mine = oi;
@@ -334,35 +350,35 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
     }
 }
 
-template <typename TI, int NR4, bool DELTA, bool VEC, int LN>
+template <typename TI, int NR4, int MODE, bool VEC, int LN>
 int launch(const ScanParams& p, int S, cudaStream_t s) {
-  constexpr int NT = (DELTA ? 8 : 4) * LN, COLS = NT / LN * CN;
-  constexpr size_t SM = (size_t)(DELTA ? 4 : 6) * CT * NR4 * LN * 4 * 4;
+  constexpr int NT = (MODE == DECAY_CHANNEL ? 4 : 8) * LN, COLS = NT / LN * CN;
+  constexpr size_t SM = (size_t)(MODE == DECAY_CHANNEL ? 6 : 4) * CT * NR4 * LN * 4 * 4;
   static MarySmemSlots slots = {};
-  if (int rc = mary_ensure_dyn_smem((const void*)scan_kernel<TI, NR4, DELTA, VEC, NT, LN>, SM, &slots)) return rc;
-  MARY_LAUNCH((scan_kernel<TI, NR4, DELTA, VEC, NT, LN>), dim3((p.DV + COLS - 1) / COLS, p.H, S), NT, SM, s, p);
+  if (int rc = mary_ensure_dyn_smem((const void*)scan_kernel<TI, NR4, MODE, VEC, NT, LN>, SM, &slots)) return rc;
+  MARY_LAUNCH((scan_kernel<TI, NR4, MODE, VEC, NT, LN>), dim3((p.DV + COLS - 1) / COLS, p.H, S), NT, SM, s, p);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }
 
-template <typename TI, bool DELTA, bool VEC>
+template <typename TI, int MODE, bool VEC>
 int dispatch(const ScanParams& p, int S, cudaStream_t s) {
-  if constexpr (!DELTA) {
+  if constexpr (MODE == DECAY_CHANNEL) {
     // twice the warps per column where 16 lanes would leave most of the machine without work (the delta rule loses more to the longer
     // reductions than it gains: 924 against 763 us for 4096 tokens of 32 heads)
     if (p.DK > 64 && (int64_t)((p.DV + 15) / 16) * p.H * S <= 3 * mary_num_sms())
-      return p.DK <= 128 ? launch<TI, 1, DELTA, VEC, 32>(p, S, s) : launch<TI, 2, DELTA, VEC, 32>(p, S, s);
+      return p.DK <= 128 ? launch<TI, 1, MODE, VEC, 32>(p, S, s) : launch<TI, 2, MODE, VEC, 32>(p, S, s);
   }
-  if (p.DK <= 64) return launch<TI, 1, DELTA, VEC, 16>(p, S, s);
-  if (p.DK <= 128) return launch<TI, 2, DELTA, VEC, 16>(p, S, s);
-  return launch<TI, 4, DELTA, VEC, 16>(p, S, s);
+  if (p.DK <= 64) return launch<TI, 1, MODE, VEC, 16>(p, S, s);
+  if (p.DK <= 128) return launch<TI, 2, MODE, VEC, 16>(p, S, s);
+  return launch<TI, 4, MODE, VEC, 16>(p, S, s);
 }
 
-template <typename TI, bool DELTA>
+template <typename TI, int MODE>
 int entry(const ScanParams& p, int S, cudaStream_t s) {
   constexpr int E = Pack<TI>::N;
   const bool vec = p.DK % E == 0 && p.DK % 4 == 0 && p.ldq % E == 0 && p.ldk % E == 0 && !(((uintptr_t)p.q | (uintptr_t)p.k | (uintptr_t)p.decay) & 15);
-  return vec ? dispatch<TI, DELTA, true>(p, S, s) : dispatch<TI, DELTA, false>(p, S, s);
+  return vec ? dispatch<TI, MODE, true>(p, S, s) : dispatch<TI, MODE, false>(p, S, s);
 }
 
 }  // namespace
@@ -374,8 +390,8 @@ MARY_API int mary_decay_scan(const void* q, const void* k, const void* v, const 
                              float q_scale, int x_f32, cudaStream_t s) {
   if (S <= 0) return MARY_OK;
   if (H < 1 || DK < 1 || DK > 256 || DV < 1 || S > 65535 || H > 65535) return MARY_ERR_BAD_ARG;
-  ScanParams p = {q, k, v, decay, nullptr, nullptr, out, state, q_start, kv_len, slots, ldq, ldk, ldv, H, H, 1, DK, DV, (DK + 3) / 4 * 4, q_scale};
-  return x_f32 ? entry<float, false>(p, S, s) : entry<__nv_bfloat16, false>(p, S, s);
+  ScanParams p = {q, k, v, decay, nullptr, nullptr, nullptr, out, state, q_start, kv_len, slots, ldq, ldk, ldv, H, H, 1, DK, DV, (DK + 3) / 4 * 4, q_scale};
+  return x_f32 ? entry<float, DECAY_CHANNEL>(p, S, s) : entry<__nv_bfloat16, DECAY_CHANNEL>(p, S, s);
 }
 
 // f32 inputs; value head h reads query / key head h / (H / HK).  pairs [T, HK, 8]: for row i of a block of four tokens (counted from the
@@ -385,6 +401,17 @@ MARY_API int mary_delta_scan(const float* q, const float* k, const float* v, con
                              int HK, int H, int DK, int DV, float q_scale, cudaStream_t s) {
   if (S <= 0) return MARY_OK;
   if (HK < 1 || H < 1 || H % HK || DK < 1 || DK > 256 || DV < 1 || S > 65535 || H > 65535 || ((uintptr_t)pairs & 15)) return MARY_ERR_BAD_ARG;
-  ScanParams p = {q, k, v, decay, beta, pairs, out, state, q_start, kv_len, slots, ldq, ldk, ldv, H, HK, H / HK, DK, DV, (DK + 3) / 4 * 4, q_scale};
-  return entry<float, true>(p, S, s);
+  ScanParams p = {q, k, v, decay, beta, pairs, nullptr, out, state, q_start, kv_len, slots, ldq, ldk, ldv, H, HK, H / HK, DK, DV, (DK + 3) / 4 * 4, q_scale};
+  return entry<float, DECAY_DELTA>(p, S, s);
+}
+
+// f32 inputs; head h reads q / k of group h / (H / G).  pairs [T, G, 4]: k_j . q_i of the row's block of four tokens (used for j <= i);
+// out = S^T q + skip v.
+MARY_API int mary_head_decay_scan(const float* q, const float* k, const float* v, const float* decay, const float* beta, const float* pairs,
+                                  const float* skip, float* out, float* state, const int* q_start, const int* kv_len, const int* slots, int S,
+                                  int64_t ldq, int64_t ldk, int64_t ldv, int G, int H, int DK, int DV, cudaStream_t s) {
+  if (S <= 0) return MARY_OK;
+  if (G < 1 || H < 1 || H % G || DK < 1 || DK > 256 || DV < 1 || S > 65535 || H > 65535 || ((uintptr_t)pairs & 15)) return MARY_ERR_BAD_ARG;
+  ScanParams p = {q, k, v, decay, beta, pairs, skip, out, state, q_start, kv_len, slots, ldq, ldk, ldv, H, G, H / G, DK, DV, (DK + 3) / 4 * 4, 1.f};
+  return entry<float, DECAY_HEAD>(p, S, s);
 }

@@ -1,7 +1,8 @@
 // Row kernels of decoders that keep the residual stream in 32-bit floats, for bf16 and for 32-bit activations: embedding into the
 // stream, norm of a sublayer's output added to the stream (with the following pre-norm or the stream's copy for the next
 // projection), plain RMS norm, gated activation, per-head query / key norm with cache append for heads whose keys and values have
-// widths of their own.  One CTA per row (or one warp per head); any width; norms, sums and activations in exact 32-bit arithmetic.
+// widths of their own; dynamic tanh around the stream, and query / key norm over whole projection rows.  One CTA per row (or one warp per
+// head); any width; norms, sums and activations in exact 32-bit arithmetic.
 #include "host_utils.h"
 #include "typed.cuh"
 
@@ -148,6 +149,113 @@ __global__ void qk_norm_append_kernel(const T* __restrict__ q, const T* __restri
   for (int i = lane; i < DK; i += 32) dst[i] = from_f<T>(to_f<T>(src[i]) * inv * (gain ? to_f<T>(gain[i]) : 1.f));
 }
 
+// E values of storage type T, 16-byte aligned when E > 1 (E = 8, or 4 for f32).
+template <typename T, int E> __device__ __forceinline__ void load_v(const T* p, float (&f)[E]) {
+  if constexpr (E == 8 && sizeof(T) == 2) unpack16(*(const uint4*)p, f);
+  else if constexpr (E == 8) {
+    *(float4*)f = *(const float4*)p;
+    *(float4*)(f + 4) = *(const float4*)(p + 4);
+  } else load_e<T, E>(p, f);
+}
+template <typename T, int E> __device__ __forceinline__ void store_v(T* p, const float (&f)[E]) {
+  if constexpr (E == 8 && sizeof(T) == 2) *(uint4*)p = pack16(f);
+  else if constexpr (E == 8) {
+    *(float4*)p = *(const float4*)f;
+    *(float4*)(p + 4) = *(const float4*)(f + 4);
+  } else store_e<T, E>(p, f);
+}
+
+template <typename T> struct Dyt {               // tanh(alpha x) * w + b
+  const T* w; const T* b; const float* alpha;
+};
+
+// h[t] = table[ids[t]] * scale;  x = n(h)
+template <typename T>
+__global__ void embed_dyt_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ h, T* __restrict__ x, int H, float scale,
+                                 Dyt<T> n, int vocab, int* __restrict__ status) {
+  pdl_sync();
+  int id = ids[blockIdx.x];
+  if (id < 0 || id >= vocab) {                 // recorded, and redirected to row 0: no read outside the table
+    if (threadIdx.x == 0) atomicCAS(status, 0, (int)MARY_ERR_BOUNDS);
+    id = 0;
+  }
+  const T* src = table + (int64_t)id * H;
+  const int64_t o = (int64_t)blockIdx.x * H;
+  const float alpha = *n.alpha;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float v = to_f<T>(src[i]) * scale;
+    h[o + i] = v;
+    x[o + i] = from_f<T>(fmaf(tanhf(alpha * v), to_f<T>(n.w[i]), to_f<T>(n.b[i])));
+  }
+}
+
+// h += post(a);  x = next(h).  blockIdx.y: row.
+template <typename T, int E>
+__global__ void __launch_bounds__(NT) dyt_add_kernel(const float* __restrict__ a, int64_t lda, Dyt<T> post, float* __restrict__ h, Dyt<T> next,
+                                                     T* __restrict__ x, int H) {
+  pdl_sync();
+  const int i = (blockIdx.x * NT + threadIdx.x) * E;
+  if (i >= H) return;
+  const int64_t row = blockIdx.y;
+  const float al = *post.alpha, an = *next.alpha;
+  float av[E], hv[E], w[E], b[E];
+  load_v<float, E>(a + row * lda + i, av);
+  load_v<float, E>(h + row * H + i, hv);
+  load_v<T, E>(post.w + i, w);
+  load_v<T, E>(post.b + i, b);
+#pragma unroll
+  for (int j = 0; j < E; ++j) hv[j] += fmaf(tanhf(al * av[j]), w[j], b[j]);
+  store_v<float, E>(h + row * H + i, hv);
+  load_v<T, E>(next.w + i, w);
+  load_v<T, E>(next.b + i, b);
+#pragma unroll
+  for (int j = 0; j < E; ++j) hv[j] = fmaf(tanhf(an * hv[j]), w[j], b[j]);
+  store_v<T, E>(x + row * H + i, hv);
+}
+
+// One CTA per token: RMS norm of the whole query row (nq values) and of the whole key row (nk), queries to qo, keys and values to their
+// cache slot.  k null: queries only.
+template <typename T, int E>
+__global__ void __launch_bounds__(NT) row_norm_append_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int64_t ld, int nq,
+                                                             int nk, int nv, const T* __restrict__ q_gain, const T* __restrict__ k_gain,
+                                                             const int64_t* __restrict__ slots, T* __restrict__ qo, T* __restrict__ kc,
+                                                             T* __restrict__ vc, float eps, int64_t n_slots, int* __restrict__ status) {
+  pdl_sync();
+  __shared__ float red[32];
+  const int64_t t = blockIdx.x;
+  auto norm = [&](const T* src, const T* gain, T* dst, int n) {
+    float ss = 0.f, f[E], g[E];
+    for (int i = threadIdx.x * E; i < n; i += NT * E) {
+      load_v<T, E>(src + i, f);
+#pragma unroll
+      for (int j = 0; j < E; ++j) ss = fmaf(f[j], f[j], ss);
+    }
+    const float inv = 1.0f / sqrtf(block_sum_x(ss, red) / n + eps);
+    for (int i = threadIdx.x * E; i < n; i += NT * E) {
+      load_v<T, E>(src + i, f);
+      load_v<T, E>(gain + i, g);
+#pragma unroll
+      for (int j = 0; j < E; ++j) f[j] *= inv * g[j];
+      store_v<T, E>(dst + i, f);
+    }
+  };
+  if (blockIdx.y == 0) {
+    norm(q + t * ld, q_gain, qo + t * nq, nq);
+    return;
+  }
+  const int64_t slot = slots[t];
+  if (slot < 0 || slot >= n_slots) {           // a cache slot outside the cache: record it, skip the write
+    if (threadIdx.x == 0) atomicCAS(status, 0, (int)MARY_ERR_BOUNDS);
+    return;
+  }
+  for (int i = threadIdx.x * E; i < nv; i += NT * E) {
+    float f[E];
+    load_v<T, E>(v + t * ld + i, f);
+    store_v<T, E>(vc + slot * nv + i, f);
+  }
+  norm(k + t * ld, k_gain, kc + slot * nk, nk);
+}
+
 }  // namespace
 
 #define BY_TYPE(f32, ...)                                      \
@@ -204,6 +312,53 @@ MARY_API int mary_qk_norm_append(const void* q, const void* k, const void* v, in
   const int64_t warps = (int64_t)n_tok * (n_q + 2 * n_kv);
   BY_TYPE(f32, MARY_LAUNCH((qk_norm_append_kernel<T>), (unsigned)((warps + 7) / 8), 256, 0, s, (const T*)q, (const T*)k, (const T*)v, ld, n_q, n_kv, DK,
                            DV, (const T*)q_gain, (const T*)k_gain, slots, (T*)qo, (T*)kc, (T*)vc, eps, n_tok, n_slots, mary_status_ptr()));
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
+}
+
+MARY_API int mary_embed_dyt(const int* ids, const void* table, float* h, void* x, int T_, int H, float scale, const void* w, const void* b,
+                            const float* alpha, int vocab, int f32, cudaStream_t s) {
+  if (T_ <= 0) return MARY_OK;
+  BY_TYPE(f32, {
+    const Dyt<T> n = {(const T*)w, (const T*)b, alpha};
+    MARY_LAUNCH((embed_dyt_kernel<T>), T_, NT, 0, s, ids, (const T*)table, h, (T*)x, H, scale, n, vocab, mary_status_ptr());
+  });
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
+}
+
+// h[T, H] (f32) += tanh(alpha a) w + b, then x[T, H] = tanh(alpha_n h) w_n + b_n.  `a` is f32, rows of `lda`.
+MARY_API int mary_dyt_add(const float* a, int64_t lda, const void* w, const void* b, const float* alpha, float* h, const void* w_n, const void* b_n,
+                          const float* alpha_n, void* x, int T_, int H, int f32, cudaStream_t s) {
+  if (T_ <= 0) return MARY_OK;
+  if (T_ > 65535 * 16) return MARY_ERR_BAD_ARG;
+  const bool vec = H % 8 == 0 && lda % 4 == 0 &&
+                   !(((uintptr_t)a | (uintptr_t)h | (uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)w_n | (uintptr_t)b_n) & 15);
+  const int E = vec ? 8 : 1;
+  BY_TYPE(f32, {
+    const Dyt<T> post = {(const T*)w, (const T*)b, alpha}, next = {(const T*)w_n, (const T*)b_n, alpha_n};
+    auto fn = vec ? dyt_add_kernel<T, 8> : dyt_add_kernel<T, 1>;
+    for (int t = 0; t < T_; t += 65535)
+      MARY_LAUNCH(fn, dim3((H + NT * E - 1) / (NT * E), T_ - t < 65535 ? T_ - t : 65535), NT, 0, s, a + (int64_t)t * lda, lda, post, h + (int64_t)t * H, next,
+                  (T*)x + (int64_t)t * H, H);
+  });
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
+}
+
+// q / k / v: columns of projection rows with pitch ld, nq / nk / nv values each; k null: queries only.
+MARY_API int mary_row_norm_append(const void* q, const void* k, const void* v, int64_t ld, int nq, int nk, int nv, const void* q_gain,
+                                  const void* k_gain, const int64_t* slots, void* qo, void* kc, void* vc, float eps, int n_tok, int64_t n_slots,
+                                  int f32, cudaStream_t s) {
+  if (n_tok <= 0) return MARY_OK;
+  if (nq < 1 || (k && (nk < 1 || nv < 1))) return MARY_ERR_BAD_ARG;
+  BY_TYPE(f32, {
+    const bool vec = nq % 8 == 0 && nk % 8 == 0 && nv % 8 == 0 && ld % 8 == 0 &&
+                     !(((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)qo | (uintptr_t)kc | (uintptr_t)vc) & 15);
+    auto fn = vec ? row_norm_append_kernel<T, 8> : row_norm_append_kernel<T, 1>;
+    MARY_LAUNCH(fn, dim3(n_tok, k ? 2 : 1), NT, 0, s, (const T*)q, (const T*)k, (const T*)v, ld, nq, nk, nv, (const T*)q_gain, (const T*)k_gain, slots,
+                (T*)qo, (T*)kc, (T*)vc, eps, n_slots, mary_status_ptr());
+  });
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }

@@ -6,6 +6,8 @@ declare their cache pages through ``kv_spec()`` and are given their layer index 
 declare their per-sequence state through ``state_spec(dtype)`` (``{name: (shape, dtype)}``) and get ``state_index``."""
 from __future__ import annotations
 
+import math
+
 import torch
 from torch import nn
 
@@ -50,6 +52,25 @@ class DenseGLU(nn.Module):
 
     def forward(self, x):
         return ops.linear_f32(ops.linear_glu(x, self.w_gu, self.act), self.w_down)
+
+    def load(self, get, p: str) -> None:
+        self.w_gu.data[:self.ff].copy_(get(p + "gate"))
+        self.w_gu.data[self.ff:].copy_(get(p + "up"))
+        self.w_down.data.copy_(get(p + "down"))
+
+
+class DynamicTanh(nn.Module):
+    """``tanh(alpha x) * w + b``: the elementwise stand-in for a norm.  Applied by the op that produces or consumes the residual stream."""
+
+    def __init__(self, width: int, dtype, device):
+        super().__init__()
+        self.w, self.b = param(width, dtype=dtype, device=device), param(width, dtype=dtype, device=device)
+        self.alpha = param(1, dtype=torch.float32, device=device)
+
+    def load(self, get, name: str) -> None:
+        self.w.data.copy_(get(name))
+        self.b.data.copy_(get(name + ".b"))
+        self.alpha.data.copy_(get(name + ".alpha").reshape(1))
 
 
 def state_shape(heads: int, dk: int, dv: int):
@@ -149,4 +170,170 @@ class GatedDeltaMixer(nn.Module):
             self.proj.fill(self.w_in, n, get(p + n))
         self.w_taps.data.copy_(torch.cat([get(p + n + ".conv") for n in "qkv"], 0))
         for mine, theirs in ((self.w_out, "o"), (self.gain, "norm"), (self.a_log, "A_log"), (self.dt_bias, "dt_bias")):
+            mine.data.copy_(get(p + theirs))
+
+
+def distance_buckets(window: int, rows: int, far: float):
+    """Row of a bias table with ``rows`` rows for the distances ``0 .. window - 1``: one row each up to half of the table, from there
+    logarithmic steps that reach the last row at distance ``far``."""
+    half = rows // 2
+    if rows < 2 or far <= half:
+        raise ValueError(f"a table of {rows} rows cannot reach to distance {far}")
+    step = math.log(far / half)
+    return torch.tensor([n if n < half else min(rows - 1, half + math.floor(math.log(n / half) / step * (rows - half))) for n in range(window)])
+
+
+def yarn_frequencies(dims: int, base: float, factor: float | None = None, original: float = 0.0, fast: float = 0.0, slow: float = 0.0):
+    """``(rotation frequencies [dims / 2] in f64, gain of cosine and sine)``.  With a ``factor``, dimensions that turn fewer than ``slow``
+    times over ``original`` positions are slowed down by it, those that turn more than ``fast`` times are kept, with a ramp between."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = base ** (-2.0 * i / dims)
+    if factor is None:
+        return f, 1.0
+    turn = lambda t: dims * math.log(original / (2.0 * math.pi * t)) / (2.0 * math.log(base))  # noqa: E731
+    lo, hi = max(math.floor(turn(fast)), 0), min(math.ceil(turn(slow)), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return f / factor * ramp + f * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
+class BiasedAttentionMixer(nn.Module):
+    """Sliding-window attention without rotation: queries and keys normed over their whole projection, a learned bias by distance added to the
+    scaled score, the heads' output multiplied by a sigmoid gate of the input before the output projection.  ``kv_from``: the layer whose
+    cached keys and values are read instead of own ones."""
+
+    def __init__(self, width, heads, kv_heads, dk, dv, scale, window, bias_rows, bias_far, kv_from, eps, dtype, device):
+        super().__init__()
+        if dk > 640 or dv > 512:
+            raise ValueError(f"head widths {dk}/{dv} exceed what the kernels hold (640/512)")
+        self.heads, self.kv_heads, self.dk, self.dv, self.scale, self.window, self.eps = heads, kv_heads, dk, dv, scale, window, eps
+        self.kv_from, self.bias_far = kv_from, bias_far
+        kw = dict(dtype=dtype, device=device)
+        own = dict(k=kv_heads * dk, v=kv_heads * dv) if kv_from is None else {}
+        self.proj = FusedProjection(dict(q=heads * dk, **own, g=heads * dv))
+        self.w_in, self.w_out = param(self.proj.rows, width, **kw), param(width, heads * dv, **kw)
+        self.q_gain = param(heads * dk, **kw)
+        self.k_gain = param(kv_heads * dk, **kw) if kv_from is None else None
+        self.rel = param(bias_rows, heads, dtype=torch.float32, device=device)
+        self.register_buffer("bias", torch.zeros(heads, window, dtype=torch.float32, device=device), persistent=False)      # by distance
+        self.kv_index = self.state_index = -1
+
+    def kv_spec(self):
+        return (self.kv_heads, self.dk, self.dv) if self.kv_from is None else None
+
+    def state_spec(self, dtype):
+        return None
+
+    def finish(self) -> None:
+        """Spread the bias table over the distances of the window (after the parameters have been set)."""
+        at = distance_buckets(self.window, self.rel.shape[0], self.bias_far).to(self.rel.device)
+        self.bias.copy_(self.rel.data[at].T)
+
+    def forward(self, x, meta, cache):
+        y = ops.linear(x, self.w_in)
+        part = lambda n: self.proj.part(y, n)  # noqa: E731
+        kc, vc = cache.k[self.kv_index], cache.v[self.kv_index]
+        k, v = (part("k"), part("v")) if self.kv_from is None else (None, None)
+        q = ops.row_norm_append(part("q"), k, v, self.heads, self.kv_heads, self.dk, self.dv, self.q_gain, self.k_gain, meta, kc, vc, self.eps)
+        o = ops.rows_buffer(x.shape[0], self.heads * self.dv, x)
+        ops.attention_exact(q, kc, vc, meta, self.scale, out=o, window=self.window, bias=self.bias, gate=part("g"))
+        return ops.linear_f32(o, self.w_out)
+
+    def load(self, get, p: str) -> None:
+        for n in self.proj.at:
+            self.proj.fill(self.w_in, n, get(p + n))
+        for mine, theirs in ((self.w_out, "o"), (self.q_gain, "q.norm"), (self.k_gain, "k.norm"), (self.rel, "rel")):
+            if mine is not None:
+                mine.data.copy_(get(p + theirs))
+
+
+class LatentAttentionMixer(nn.Module):
+    """Sliding-window attention over a latent: the cache row of a token is ``[normed latent | rotated key part shared by all heads]``; per-head
+    keys and values are linear in the latent, so one-token steps attend in latent space (the key matrix applied to the query, the value
+    matrix to the read-out) and prompts attend over expanded keys and values where that is the smaller work."""
+
+    kv_from = None
+
+    def __init__(self, width, heads, dim, rot, dv, q_rank, rank, scale, window, freq, rot_gain, eps, dtype, device):
+        super().__init__()
+        if rank + rot > 640 or rank > 512:
+            raise ValueError(f"latent width {rank} + {rot} exceeds what the kernels hold (512, 640 with the rotated part)")
+        self.heads, self.dim, self.rot, self.dv, self.rank, self.q_rank = heads, dim, rot, dv, rank, q_rank
+        self.scale, self.window, self.rot_gain, self.eps = scale, window, rot_gain, eps
+        kw = dict(dtype=dtype, device=device)
+        self.proj = FusedProjection(dict(dq=q_rank, dkv=rank + rot))
+        self.w_in, self.w_out = param(self.proj.rows, width, **kw), param(width, heads * dv, **kw)
+        self.q_gain, self.kv_gain = param(q_rank, **kw), param(rank, **kw)
+        self.w_q, self.w_k, self.w_v = param(heads * (dim + rot), q_rank, **kw), param(heads * dim, rank, **kw), param(heads * dv, rank, **kw)
+        self.register_buffer("w_k_t", torch.zeros(heads, rank, dim, **kw), persistent=False)      # the key matrices, applied to queries
+        self.register_buffer("freq", freq.to(torch.float32).to(device), persistent=False)
+        self.kv_index = self.state_index = -1
+
+    def kv_spec(self):
+        return 1, self.rank + self.rot, 0           # the values are part of the key row
+
+    def state_spec(self, dtype):
+        return None
+
+    def finish(self) -> None:
+        self.w_k_t.copy_(self.w_k.data.view(self.heads, self.dim, self.rank).transpose(1, 2))
+
+    def forward(self, x, meta, cache):
+        y = ops.linear(x, self.w_in)
+        rows = cache.k[self.kv_index]
+        c = ops.latent_prep(self.proj.part(y, "dq"), self.proj.part(y, "dkv"), self.q_gain, self.kv_gain, self.freq, self.rot_gain, meta, rows, self.eps)
+        o = ops.latent_attention(ops.linear(c, self.w_q), rows, meta, self)
+        return ops.linear_f32(o, self.w_out)
+
+    def load(self, get, p: str) -> None:
+        for n in self.proj.at:
+            self.proj.fill(self.w_in, n, get(p + n))
+        for mine, theirs in ((self.w_out, "o"), (self.q_gain, "dq.norm"), (self.kv_gain, "dkv.norm"), (self.w_q, "uq"), (self.w_k, "uk"), (self.w_v, "uv")):
+            mine.data.copy_(get(p + theirs))
+
+
+class StateSpaceMixer(nn.Module):
+    """Mamba-2 (state-space duality): short convolutions with bias on ``x``, ``B``, ``C``, one step size and decay per head, ``B`` and ``C``
+    shared by the heads of a group, a skip per head, the read-out gated and then normed in equal parts."""
+
+    kv_from = None
+
+    def __init__(self, width, heads, dv, state, groups, taps, norm_parts, eps, dtype, device):
+        super().__init__()
+        if state > 256:
+            raise ValueError(f"state width {state} exceeds what the kernels hold (256)")
+        self.heads, self.dv, self.state, self.groups, self.taps, self.norm_parts, self.eps = heads, dv, state, groups, taps, norm_parts, eps
+        kw, f32 = dict(dtype=dtype, device=device), dict(dtype=torch.float32, device=device)
+        self.inner = heads * dv
+        self.channels = self.inner + 2 * groups * state
+        self.proj = FusedProjection(dict(z=self.inner, xbc=self.channels, dt=heads))
+        self.w_in, self.w_out = param(self.proj.rows, width, **kw), param(width, self.inner, **kw)
+        self.w_taps, self.b_taps, self.gain = param(self.channels, taps, **kw), param(self.channels, **kw), param(self.inner, **kw)
+        self.a_log, self.dt_bias, self.skip = param(heads, **f32), param(heads, **f32), param(heads, **f32)
+        self.kv_index = self.state_index = -1
+
+    def kv_spec(self):
+        return None
+
+    def state_spec(self, dtype):
+        return {"S": (state_shape(self.heads, self.state, self.dv), torch.float32), "conv": ((self.taps, self.channels), dtype)}
+
+    def finish(self) -> None:
+        pass
+
+    def forward(self, x, meta, cache):
+        y = ops.linear(x, self.w_in)
+        part = lambda n: self.proj.part(y, n)  # noqa: E731
+        st = cache.state[self.state_index]
+        o = ops.rows_buffer(x.shape[0], self.inner, x)
+        ops.state_space(part("xbc"), self.w_taps, self.b_taps, part("dt"), self.dt_bias, self.a_log, self.skip, part("z"), self.gain, self.norm_parts,
+                        st["conv"], st["S"], meta, self.groups, self.heads, self.state, self.dv, self.eps, o)
+        return ops.linear_f32(o, self.w_out)
+
+    def load(self, get, p: str) -> None:
+        w, at = get(p + "in"), 0
+        for n, (_, rows) in self.proj.at.items():
+            self.proj.fill(self.w_in, n, w[at:at + rows])
+            at += rows
+        for mine, theirs in ((self.w_out, "o"), (self.w_taps, "conv"), (self.b_taps, "conv.b"), (self.gain, "norm"), (self.a_log, "A_log"),
+                             (self.dt_bias, "dt_bias"), (self.skip, "D")):
             mine.data.copy_(get(p + theirs))

@@ -36,6 +36,15 @@ def _load_tatizen(d, loader, device, dtype):
     return model
 
 
+def _load_rokarax(d, loader, device, dtype):
+    from .rokarax.config import RokaraxConfig
+    from .rokarax.model import RokaraxModel, bias_rows, load_into
+    cfg = RokaraxConfig.from_json(d)
+    model = RokaraxModel(cfg, bias_rows(cfg, loader.shape), dtype=dtype, device=device)
+    load_into(model, loader)
+    return model
+
+
 def _load_mistral(d, loader, device, dtype):
     from .mistral.model import MistralConfig, MistralModel, load_into
     model = MistralModel(MistralConfig.from_hf(d), dtype=dtype, device=device)
@@ -54,6 +63,8 @@ def _load_gemma4(d, loader, device, dtype):
 FAMILIES = [
     Family("tatizen", lambda d: d.get("architecture") == "Tatizen", _load_tatizen, page_size=64, f32_on_gpu=True,
            kernels=_DENSE_KERNELS + ("attention_general", "residual32", "linear_attention", "recurrent_scan")),
+    Family("rokarax", lambda d: d.get("architecture") == "Rokarax", _load_rokarax, page_size=64, f32_on_gpu=True,
+           kernels=_DENSE_KERNELS + ("attention_general", "attention_mla", "residual32", "linear_attention", "recurrent_scan", "latent", "state_space")),
     Family("gemma4", lambda d: str(d.get("model_type", "")).startswith("gemma4"), _load_gemma4),
     Family("mistral", lambda d: d.get("model_type") in ("mistral", "ministral", "qwen3", "mistral3"), _load_mistral),
 ]

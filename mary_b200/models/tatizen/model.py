@@ -133,7 +133,4 @@ def load_into(model: TatizenModel, loader) -> None:
         layer.mixer.load(get, f"l{i}.mix.")
         if layer.mlp is not None:
             layer.norm2.data.copy_(get(f"l{i}.norm2"))
-            F = layer.mlp.ff
-            layer.mlp.w_gu.data[:F].copy_(get(f"l{i}.mlp.gate"))
-            layer.mlp.w_gu.data[F:].copy_(get(f"l{i}.mlp.up"))
-            layer.mlp.w_down.data.copy_(get(f"l{i}.mlp.down"))
+            layer.mlp.load(get, f"l{i}.mlp.")

@@ -270,15 +270,56 @@ def qk_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vca
     return f(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps)
 
 
-def attention_exact(q, kcache, vcache, meta, scale, out=None):
-    """Causal paged attention whose scores, softmax weights and sums stay in 32 bits, for any head widths: ``[T, Hq * DV]``."""
+def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, bias=None, gate=None):
+    """Causal paged attention whose scores, softmax weights and sums stay in 32 bits, for any head widths: ``[T, Hq * DV]``.  ``window``: keys
+    at most ``window - 1`` positions back (0: all); ``bias [Hq, window]`` f32 is added to the scaled score by distance; ``gate [T, Hq * DV]``
+    multiplies the result by its logistic function before it is rounded."""
     if _cuda(q):
-        return _h().attention_exact(q, kcache, vcache, meta, scale, out)
-    o = ref.paged_attention(q, kcache, vcache, meta, scale).reshape(q.shape[0], -1)
+        return _h().attention_exact(q, kcache, vcache, meta, scale, out, window, bias, gate)
+    o = ref.attention_exact(q, kcache, vcache, meta, scale, window, bias, gate)
     if out is None:
         return o
     out.copy_(o)
     return out
+
+
+def embed_dyt(ids, table, scale, norm):
+    """Scaled rows of the embedding table as the 32-bit residual stream, and the stream through the dynamic tanh ``norm``: ``(h, x)``."""
+    return _h().embed_dyt(ids, table, scale, norm) if _cuda(table) else ref.embed_dyt(ids, table, scale, norm)
+
+
+def dyt_add(a, post, h, following):
+    """Residual step between dynamic tanhs (objects with ``w``, ``b``, ``alpha``): ``h += post(a)`` in place; returns ``following(h)`` in the
+    activation type."""
+    return _h().dyt_add(a, post, h, following) if _cuda(h) else ref.dyt_add(a, post, h, following)
+
+
+def row_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps):
+    """RMS norm over the whole query row and the whole key row (gains of those sizes), keys and values appended to the cache; ``k`` and ``v``
+    are None for a layer that reads another layer's cache.  Returns ``q [T, n_q, dk]``."""
+    f = _h().row_norm_append if _cuda(q) else ref.row_norm_append
+    return f(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps)
+
+
+def latent_prep(y_q, y_kv, q_gain, kv_gain, freq, rot_gain, meta, cache, eps):
+    """RMS norm of the query latent (returned) and of the key/value latent, rotation of the shared key part (pairs ``2i, 2i + 1``, cosine and
+    sine times ``rot_gain``); ``[latent | rotated part]`` goes to the cache."""
+    f = _h().latent_prep if _cuda(y_q) else ref.latent_prep
+    return f(y_q, y_kv, q_gain, kv_gain, freq, rot_gain, meta, cache, eps)
+
+
+def latent_attention(q, cache, meta, m):
+    """Sliding-window latent attention of ``q [T, heads * (dim + rot)]`` (not yet rotated) over cached rows ``[latent | rotated part]``;
+    ``m``: a ``LatentAttentionMixer``.  Returns ``[T, heads * dv]``."""
+    return (_h() if _cuda(q) else ref).latent_attention(q, cache, meta, m)
+
+
+def state_space(xbc, taps_w, taps_b, dt_in, dt_bias, a_log, skip, z, gain, norm_parts, ring, state, meta, G, H, N, P, eps, out):
+    """Mamba-2 mixer between its projections: ``silu(conv(xbc) + taps_b) = [x [H, P] | B [G, N] | C [G, N]]``, ``dt = softplus(dt_in + dt_bias)``,
+    ``S <- exp(-exp(a_log) dt) S + dt B x^T``, ``y = S^T C + skip x``; then ``y * silu(z)`` normed in ``norm_parts`` equal parts times ``gain``
+    into ``out [T, H * P]``.  ``ring`` and ``state`` as above."""
+    f = _h().state_space if _cuda(xbc) else ref.state_space
+    return f(xbc, taps_w, taps_b, dt_in, dt_bias, a_log, skip, z, gain, norm_parts, ring, state, meta, G, H, N, P, eps, out)
 
 
 def decayed_linear_attention(q, k, v, gate, low, a2, a2_bias, inv_tau, gain, state, meta, H, dk, dv, eps, out_scale, out):

@@ -16,7 +16,7 @@ declare("mary_post_norm_add", "plppppiifis")
 declare("mary_rmsnorm32", "pppiifis")
 declare("mary_glu_any", "ppiiiis")
 declare("mary_qk_norm_append", "ppp" + "liiii" + "pppppp" + "fil" + "is")
-declare("mary_attention_general", "ppppppppp" + "iii" + "lllll" + "iiiiiii" + "fpis")
+declare("mary_attention_general", "ppppppppp" + "iii" + "lllll" + "iiiiiii" + "fpplpis")
 declare("mary_attention_general_rows", "i")
 declare("mary_attention_general_scratch_floats", "iiiii", ret64=True)
 declare("mary_channel_decay", "pli" + "ppp" + "iifis")
@@ -27,6 +27,18 @@ declare("mary_decay_scan", "pppppp" + "ppp" + "illl" + "iiifis")
 declare("mary_delta_scan", "pppppppp" + "ppp" + "illl" + "iiiifs")
 declare("mary_decay_step", "ppppp" + "li" + "ppfp" + "plfp" + "ppp" + "iiiiffis")
 declare("mary_delta_step", "plppi" + "pppppp" + "plp" + "ppp" + "iiiiiffis")
+
+
+declare("mary_gemm_simt_batched", "pppiiilll" + "illl" + "fiiis")
+declare("mary_embed_dyt", "ppppiif" + "ppp" + "iis")
+declare("mary_dyt_add", "pl" + "ppp" + "p" + "ppp" + "piiis")
+declare("mary_row_norm_append", "ppp" + "liii" + "pppppp" + "filis")
+declare("mary_latent_prep", "pp" + "liii" + "ppp" + "f" + "pppp" + "filis")
+declare("mary_rotate_heads", "pppfp" + "iiiiii" + "is")
+declare("mary_ss_prep", "pl" + "pppppp" + "ppp" + "pppppp" + "iiiiiii" + "is")
+declare("mary_head_decay_scan", "pppppppp" + "p" + "ppp" + "illl" + "iiiis")
+declare("mary_gated_part_norm", "pplppl" + "iiifis")
+declare("mary_ss_step", "plppp" + "pppp" + "pp" + "ipl" + "ppp" + "ppp" + "iiiiiifis")
 
 
 def _f32(t) -> int:
@@ -104,8 +116,13 @@ def qk_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vca
 DECODE_ROWS = K.DECODE_GROUP_ROWS         # sequences with at most this many query tokens take the decode kernel, the others the prefill kernel
 
 
-def attention_general(q, kcache, vcache, meta, scale, out, group=None, nsplit=None, window: int = 0):
-    """Any head widths, group size and storage type; ``group`` restricts the call to ``"prefill"`` or ``"decode"`` sequences."""
+def _gate(gate):
+    return (None, 0) if gate is None else _rows(gate)
+
+
+def attention_general(q, kcache, vcache, meta, scale, out, group=None, nsplit=None, window: int = 0, bias=None, gate=None):
+    """Any head widths, group size and storage type; ``group`` restricts the call to ``"prefill"`` or ``"decode"`` sequences.  ``bias``,
+    ``gate``: see ``ops.attention_exact``."""
     T, Hq, DK = q.shape
     Hkv, DV = kcache.shape[2], vcache.shape[3]
     G = Hq // Hkv
@@ -122,36 +139,39 @@ def attention_general(q, kcache, vcache, meta, scale, out, group=None, nsplit=No
         scratch = _empty(lib().mary_attention_general_scratch_floats(NB, Hq, Hkv, nsplit, DV), dtype=torch.float32, device=q.device)
     check(lib().mary_attention_general(_p(q), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len), _p(meta.q_start), _p(blk_seq),
                                        _p(blk_q0), NB, meta.page_table.shape[1], meta.page_size, kcache.stride(1), kcache.stride(0), vcache.stride(1),
-                                       vcache.stride(0), out.stride(0), Hq, Hkv, DK, DV, rq, nsplit, window, scale, _p(scratch), _f32(q), _stream()),
-          "attention_general")
+                                       vcache.stride(0), out.stride(0), Hq, Hkv, DK, DV, rq, nsplit, window, scale, _p(bias), *_gate(gate), _p(scratch),
+                                       _f32(q), _stream()), "attention_general")
     return out
 
 
-def attention_exact(q, kcache, vcache, meta, scale, out=None):
+def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, bias=None, gate=None):
     """Causal attention with scores, softmax weights and sums in 32 bits: the tensor-core prefill kernel with two-term weights for
     sequences that bring more than ``DECODE_ROWS`` tokens, the bandwidth-oriented decode kernel for the others, the general kernel for
     32-bit tensors and for head shapes those have no instantiation for.  ``out`` may be a row view ``[T, Hq * DV]``."""
     T, Hq, DK = q.shape
     Hkv, DV = kcache.shape[2], vcache.shape[3]
-    assert q.is_contiguous() and kcache.is_contiguous() and vcache.is_contiguous() and kcache.shape[1] == meta.page_size
+    assert q.is_contiguous() and kcache.is_contiguous() and vcache.stride(3) == 1 and kcache.shape[1] == meta.page_size
+    assert bias is None or (bias.is_contiguous() and bias.shape == (Hq, window) and bias.dtype == torch.float32)
+    assert gate is None or gate.dtype == q.dtype
     if out is None:
         out = _empty(T, Hq * DV, dtype=q.dtype, device=q.device)
     assert out.stride(1) == 1
-    bf16 = q.dtype == torch.bfloat16 and DK == DV
+    bf16 = q.dtype == torch.bfloat16 and DK == DV and vcache.is_contiguous() and bias is None and gate is None
+    kw = dict(window=window, bias=bias, gate=gate)
     fast_prefill = bf16 and DK in (64, 128, 256) and meta.page_size in (16, 64) and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
     fast_decode = bf16 and DK in (64, 128, 256) and Hq // Hkv <= (4 if DK == 256 else 8)
     if not (fast_prefill or fast_decode):
-        return attention_general(q, kcache, vcache, meta, scale, out)
+        return attention_general(q, kcache, vcache, meta, scale, out, **kw)
     if meta.max_q_len > DECODE_ROWS:
         if fast_prefill:
-            K.attention_prefill(q, kcache, vcache, meta, scale, out=out, split_p=True, group="prefill")
+            K.attention_prefill(q, kcache, vcache, meta, scale, window, out=out, split_p=True, group="prefill")
         else:
-            attention_general(q, kcache, vcache, meta, scale, out, "prefill")
+            attention_general(q, kcache, vcache, meta, scale, out, "prefill", **kw)
     if K._q_blocks(meta, 1, "decode")[2]:
         if fast_decode:
-            K._paged_attention_decode(q, kcache, vcache, meta, scale, 0, 0.0, None, out=out, group="decode")
+            K._paged_attention_decode(q, kcache, vcache, meta, scale, window, 0.0, None, out=out, group="decode")
         else:
-            attention_general(q, kcache, vcache, meta, scale, out, "decode")
+            attention_general(q, kcache, vcache, meta, scale, out, "decode", **kw)
     return out
 
 
@@ -240,3 +260,137 @@ def gated_delta_attention(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, rin
     conv_history(x, ring, meta, taps, taps_w.shape[0])
     o = delta_scan(q, k, v, g, beta, pairs, state, meta, HK, H, dk, dv)
     return gated_head_norm(o, gate, gain, eps, out_scale, out)
+
+
+# --------------------------------------------------------------------------- dynamic tanh around the stream, whole-row norms
+def embed_dyt(ids, table, scale, norm):
+    ids = ids.to(torch.int32)
+    T, H = ids.shape[0], table.shape[1]
+    h = _empty(T, H, dtype=torch.float32, device=table.device)
+    x = _empty(T, H, dtype=table.dtype, device=table.device)
+    check(lib().mary_embed_dyt(_p(ids), _p(table), _p(h), _p(x), T, H, scale, _p(norm.w), _p(norm.b), _p(norm.alpha), table.shape[0], _f32(table),
+                               _stream()), "embed_dyt")
+    return h, x
+
+
+def dyt_add(a, post, h, following):
+    x = _empty(h.shape, dtype=post.w.dtype, device=h.device)
+    pa, lda = _rows(a)
+    assert a.dtype == torch.float32 and h.dtype == torch.float32 and h.is_contiguous()
+    check(lib().mary_dyt_add(pa, lda, _p(post.w), _p(post.b), _p(post.alpha), _p(h), _p(following.w), _p(following.b), _p(following.alpha), _p(x),
+                             h.shape[0], h.shape[1], _f32(x), _stream()), "dyt_add")
+    return x
+
+
+def row_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps):
+    T = q.shape[0]
+    qo = _empty(T, n_q, dk, dtype=q.dtype, device=q.device)
+    pq, ld = _rows(q)
+    pk = pv = None
+    if k is not None:
+        (pk, l2), (pv, l3) = _rows(k), _rows(v)
+        assert ld == l2 == l3 and kcache.is_contiguous() and vcache.is_contiguous() and kcache.dtype == q.dtype
+    check(lib().mary_row_norm_append(pq, pk, pv, ld, n_q * dk, n_kv * dk, n_kv * dv, _p(q_gain), _p(k_gain), _p(meta.slot_mapping), _p(qo), _p(kcache),
+                                     _p(vcache), eps, T, kcache.shape[0] * kcache.shape[1], _f32(q), _stream()), "row_norm_append")
+    return qo
+
+
+# --------------------------------------------------------------------------- latent attention
+def latent_prep(y_q, y_kv, q_gain, kv_gain, freq, rot_gain, meta, cache, eps):
+    T, rank = y_q.shape[0], kv_gain.shape[0]
+    (pq, ld), (pk, l2) = _rows(y_q), _rows(y_kv)
+    assert ld == l2 and cache.is_contiguous() and cache.dtype == y_q.dtype
+    c = _empty(T, q_gain.shape[0], dtype=y_q.dtype, device=y_q.device)
+    check(lib().mary_latent_prep(pq, pk, ld, q_gain.shape[0], rank, cache.shape[-1] - rank, _p(q_gain), _p(kv_gain), _p(freq), rot_gain,
+                                 _p(meta.positions), _p(meta.slot_mapping), _p(c), _p(cache), eps, T, cache.shape[0] * cache.shape[1], _f32(y_q),
+                                 _stream()), "latent_prep")
+    return c
+
+
+def rotate_heads(src, dst, dst_off, rot, freq, rot_gain, meta):
+    """The last ``rot`` values of every head of ``src [T, H, w]`` rotated into ``dst [T, H, w']`` from ``dst_off`` on (``src`` itself allowed)."""
+    T, H, w = src.shape
+    check(lib().mary_rotate_heads(_p(src), _p(dst), _p(freq), rot_gain, _p(meta.positions), T, H, w, dst.shape[2], dst_off, rot, _f32(src), _stream()),
+          "rotate_heads")
+    return dst
+
+
+def head_matmul(x, w, out):
+    """Per head ``out[t, h] = w[h] x[t, h]``: ``x [T, H, k]``, ``out [T, H, n]`` (views whose rows may be wider), ``w [H, n, k]``."""
+    T, H, k = x.shape
+    n = w.shape[1]
+    (ldx, bx), (ldo, bo) = x.stride()[:2], out.stride()[:2]
+    if x.dtype == torch.bfloat16 and k % 8 == 0 and n % 8 == 0 and ldx % 8 == 0 and bx % 8 == 0 and x.data_ptr() % 16 == 0 and bo % 8 == 0 and ldo % 8 == 0:
+        with K.static_weights:
+            return K.gemm_batched(x, w, out, T, n, k, ldx, k, ldo, H, bx, n * k, bo)
+    check(lib().mary_gemm_simt_batched(_p(x), _p(w), _p(out), T, n, k, ldx, k, ldo, H, bx, n * k, bo, 1.0, 0, _f32(x), _f32(out), _stream()),
+          "gemm_simt_batched")
+    return out
+
+
+def latent_attention(q, cache, meta, m):
+    T, H = q.shape[0], m.heads
+    q = q.view(T, H, m.dim + m.rot)
+    qf = _empty(T, H, m.rank + m.rot, dtype=q.dtype, device=q.device)
+    head_matmul(q[..., :m.dim], m.w_k_t, qf[..., :m.rank])
+    rotate_heads(q, qf, m.rank, m.rot, m.freq, m.rot_gain, meta)
+    lat = attention_exact(qf, cache, cache[..., :m.rank], meta, m.scale, window=m.window)
+    out = _empty(T, H * m.dv, dtype=q.dtype, device=q.device)
+    head_matmul(lat.view(T, H, m.rank), m.w_v.view(H, m.dv, m.rank), out.view(T, H, m.dv))
+    return out
+
+
+# --------------------------------------------------------------------------- state space layers
+_ARRIVED: dict = {}
+
+
+def _arrival_counters(dev, n: int):
+    """Counters of the one-token kernel, zero between launches; never freed, since a captured graph may hold them."""
+    pool = _ARRIVED.setdefault(dev, [])
+    if not pool or pool[-1].numel() < n:
+        pool.append(torch.zeros(max(n, 4096), dtype=torch.int32, device=dev))
+    return pool[-1]
+
+
+def ss_prep(xbc, taps_w, taps_b, ring, dt_in, dt_bias, a_log, meta, G, H, N, P):
+    """Convolutions, step sizes and decays of a Mamba-2 layer: f32 ``x [T, H * P]``, ``B, C [T, G * N]``, ``dt, decay [T, H]`` and the products
+    ``pairs [T, G, 4]`` of every four tokens' ``B`` and ``C`` (what ``head_decay_scan`` takes)."""
+    T = xbc.shape[0]
+    f = dict(dtype=torch.float32, device=xbc.device)
+    x, b, c, dt, decay, pairs = _empty(T, H * P, **f), _empty(T, G * N, **f), _empty(T, G * N, **f), _empty(T, H, **f), _empty(T, H, **f), _empty(T, G, 4, **f)
+    px, ldx = _rows(xbc)
+    assert dt_in.stride(0) == ldx
+    check(lib().mary_ss_prep(px, ldx, _p(taps_w), _p(taps_b), _p(ring), _p(dt_in), _p(dt_bias), _p(a_log), _p(meta.q_start), _p(meta.kv_len),
+                             _p(meta.state_slots), _p(x), _p(b), _p(c), _p(dt), _p(decay), _p(pairs), meta.num_seqs, meta.max_q_len, G, H, N, P,
+                             taps_w.shape[1], _f32(xbc), _stream()), "ss_prep")
+    return x, b, c, dt, decay, pairs
+
+
+def head_decay_scan(x, b, c, dt, decay, pairs, skip, state, meta, G, H, N, P):
+    out = _empty(x.shape[0], H * P, dtype=torch.float32, device=x.device)
+    check(lib().mary_head_decay_scan(_p(c), _p(b), _p(x), _p(decay), _p(dt), _p(pairs), _p(skip), _p(out), _p(state), _p(meta.q_start), _p(meta.kv_len),
+                                     _p(meta.state_slots), meta.num_seqs, c.stride(0), b.stride(0), x.stride(0), G, H, N, P, _stream()), "head_decay_scan")
+    return out
+
+
+def gated_part_norm(y, z, gain, parts, eps, out):
+    (pz, ldz), (po, ldo) = _rows(z), _rows(out)
+    check(lib().mary_gated_part_norm(_p(y), pz, ldz, _p(gain), po, ldo, y.shape[0], y.shape[1], parts, eps, _f32(z), _stream()), "gated_part_norm")
+    return out
+
+
+def state_space(xbc, taps_w, taps_b, dt_in, dt_bias, a_log, skip, z, gain, norm_parts, ring, state, meta, G, H, N, P, eps, out):
+    taps = taps_w.shape[1]
+    if meta.max_q_len == 1:
+        (px, ldx), (po, ldo) = _rows(xbc), _rows(out)
+        assert dt_in.stride(0) == ldx and z.stride(0) == ldx
+        S = meta.num_seqs
+        row = _empty(S, H * P, dtype=torch.float32, device=xbc.device)
+        cnt = _arrival_counters(xbc.device, S * norm_parts)
+        check(lib().mary_ss_step(px, ldx, _p(taps_w), _p(taps_b), _p(ring), _p(dt_in), _p(dt_bias), _p(a_log), _p(skip), _p(z), _p(gain), norm_parts, po, ldo,
+                                 _p(state), _p(row), _p(cnt), _p(meta.q_start), _p(meta.positions), _p(meta.state_slots), S, G, H, N, P, taps, eps,
+                                 _f32(xbc), _stream()), "ss_step")
+        return out
+    x, b, c, dt, decay, pairs = ss_prep(xbc, taps_w, taps_b, ring, dt_in, dt_bias, a_log, meta, G, H, N, P)
+    conv_history(xbc, ring, meta, taps, taps_w.shape[0])
+    return gated_part_norm(head_decay_scan(x, b, c, dt, decay, pairs, skip, state, meta, G, H, N, P), z, gain, norm_parts, eps, out)

@@ -303,17 +303,23 @@ def decayed_linear_attention(q, k, v, gate, low, a2, a2_bias, inv_tau, gain, sta
     return out
 
 
-def gated_delta_attention(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, ring, state, meta, HK, H, dk, dv, eps, out_scale, out):
-    T, taps = x.shape[0], taps_w.shape[1]
-    w = taps_w.float()
-    y = torch.empty(T, taps_w.shape[0])
+def _causal_conv(x, taps_w, bias, ring, meta):
+    """Depthwise convolution of every sequence's rows, continued from and recorded in its history ring."""
+    taps, w = taps_w.shape[1], taps_w.float()
+    y = torch.empty(x.shape[0], taps_w.shape[0])
     for rows, slot, pos in _portions(meta):
         n = rows.stop - rows.start
         hist = [ring[slot, (pos - d) % taps].float() if pos - d >= 0 else torch.zeros(w.shape[0]) for d in range(taps - 1, 0, -1)]
         ext = torch.cat([torch.stack(hist), x[rows].float()]) if hist else x[rows].float()
-        y[rows] = F.silu(sum(ext[j:j + n] * w[:, j] for j in range(taps)))
+        y[rows] = sum(ext[j:j + n] * w[:, j] for j in range(taps))
         for d in range(min(taps, n)):
             ring[slot, (pos + n - 1 - d) % taps] = x[rows.stop - 1 - d].to(ring.dtype)
+    return y if bias is None else y + bias.float()
+
+
+def gated_delta_attention(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, ring, state, meta, HK, H, dk, dv, eps, out_scale, out):
+    T = x.shape[0]
+    y = F.silu(_causal_conv(x, taps_w, None, ring, meta))
     q, k, v = y.split([HK * dk, HK * dk, H * dv], -1)
     unit = lambda z: z / torch.sqrt(z.pow(2).sum(-1, keepdim=True) + 1e-6)  # noqa: E731
     rep = H // HK
@@ -332,4 +338,74 @@ def gated_delta_attention(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, rin
             o[t] = (S * q[t][:, None, :]).sum(-1)
         state[slot, :, :, :dk] = S
     out.copy_(head_norm_gate(o, gate, gain, eps, out_scale))
+    return out
+
+
+def attention_exact(q, kcache, vcache, meta, scale, window: int = 0, bias=None, gate=None):
+    rel = None if bias is None else bias[None].expand(q.shape[0], -1, -1)
+    o = paged_attention(q.float(), kcache, vcache, meta, scale, window, rel_bias=rel).reshape(q.shape[0], -1)
+    return (o if gate is None else o * torch.sigmoid(gate.float())).to(q.dtype)
+
+
+def _dyt(x, norm):
+    return torch.tanh(norm.alpha * x) * norm.w.float() + norm.b.float()
+
+
+def embed_dyt(ids, table, scale: float, norm):
+    h = table[ids.long()].float() * scale
+    return h, _dyt(h, norm).to(table.dtype)
+
+
+def dyt_add(a, post, h, following):
+    h += _dyt(a.float(), post)
+    return _dyt(h, following).to(following.w.dtype)
+
+
+def row_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps):
+    T = q.shape[0]
+    if k is not None:
+        kv_append(rmsnorm(k, k_gain, eps).reshape(T, n_kv, dk), v.reshape(T, n_kv, dv), kcache, vcache, meta.slot_mapping)
+    return rmsnorm(q, q_gain, eps).reshape(T, n_q, dk)
+
+
+def rotate_pairs(x, positions, freq, gain: float):
+    """``x [T, ..., D]``: the pair ``(2i, 2i + 1)`` turns by ``position * freq[i]``; cosine and sine times ``gain``."""
+    ang = (positions.float()[:, None] * freq[None]).view(x.shape[0], *[1] * (x.dim() - 2), -1)
+    c, s = ang.cos() * gain, ang.sin() * gain
+    u, v = x[..., 0::2].float(), x[..., 1::2].float()
+    return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2).to(x.dtype)
+
+
+def latent_prep(y_q, y_kv, q_gain, kv_gain, freq, rot_gain, meta, cache, eps):
+    rank = kv_gain.shape[0]
+    row = torch.cat([rmsnorm(y_kv[:, :rank], kv_gain, eps), rotate_pairs(y_kv[:, rank:], meta.positions, freq, rot_gain)], -1)
+    cache.view(-1, cache.shape[-1])[meta.slot_mapping] = row.to(cache.dtype)
+    return rmsnorm(y_q, q_gain, eps)
+
+
+def latent_attention(q, cache, meta, m):
+    T = q.shape[0]
+    q = q.view(T, m.heads, m.dim + m.rot)
+    lat = torch.einsum("thd,hrd->thr", q[..., :m.dim].float(), m.w_k_t.float()).to(q.dtype)
+    qf = torch.cat([lat, rotate_pairs(q[..., m.dim:], meta.positions, m.freq, m.rot_gain)], -1)
+    o = attention_exact(qf, cache, cache[..., :m.rank], meta, m.scale, m.window).view(T, m.heads, m.rank)
+    return torch.einsum("thr,hvr->thv", o.float(), m.w_v.view(m.heads, m.dv, m.rank).float()).to(q.dtype).reshape(T, -1)
+
+
+def state_space(xbc, taps_w, taps_b, dt_in, dt_bias, a_log, skip, z, gain, norm_parts, ring, state, meta, G, H, N, P, eps, out):
+    T = xbc.shape[0]
+    x, B, C = F.silu(_causal_conv(xbc, taps_w, taps_b, ring, meta)).split([H * P, G * N, G * N], -1)
+    x = x.view(T, H, P)
+    B, C = (v.view(T, G, N).repeat_interleave(H // G, 1) for v in (B, C))
+    dt = F.softplus(dt_in.float() + dt_bias)
+    g = torch.exp(-torch.exp(a_log) * dt)
+    y = torch.empty(T, H, P)
+    for rows, slot, pos in _portions(meta):
+        S = state[slot, :, :, :N] * (0.0 if pos == 0 else 1.0)                  # [H, P, N]
+        for t in range(rows.start, rows.stop):
+            S = S * g[t][:, None, None] + (dt[t][:, None] * x[t])[:, :, None] * B[t][:, None, :]
+            y[t] = (S * C[t][:, None, :]).sum(-1)
+        state[slot, :, :, :N] = S
+    y = ((y + skip[:, None] * x).reshape(T, H * P) * F.silu(z.float())).view(T, norm_parts, -1)
+    out.copy_((y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, H * P) * gain.float())
     return out

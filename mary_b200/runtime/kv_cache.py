@@ -177,7 +177,7 @@ class Q8Pages:
 
 class PagedKVCache:
     """Device storage for the pages of every layer.  ``kv_dtype="int8"`` keeps K and V as :class:`Q8Pages`.  ``v_head_dim`` gives
-    values a width of their own.  ``state_spec`` (one ``{name: (shape, dtype)}`` per recurrent layer) adds ``state[layer][name]``
+    values a width of their own; a layer with width 0 stores none (its values are part of its key rows, ``v[layer] is k[layer]``).  ``state_spec`` (one ``{name: (shape, dtype)}`` per recurrent layer) adds ``state[layer][name]``
     tensors ``[num_slots, *shape]``: the per-sequence recurrent state, addressed by ``BatchMeta.state_slots``.  A slot is never
     cleared: the kernels take a sequence whose rows start at position 0 to have zero state."""
 
@@ -208,8 +208,8 @@ class PagedKVCache:
             self.v = self.k
         else:
             self.k = [torch.zeros(num_pages, page_size, heads[i], dims[i], dtype=dtype, device=device) for i in range(num_layers)]
-            self.v = self.k if alias_v_to_k else [torch.zeros(num_pages, page_size, heads[i], vdims[i], dtype=dtype, device=device)
-                                                  for i in range(num_layers)]
+            self.v = self.k if alias_v_to_k else [torch.zeros(num_pages, page_size, heads[i], vdims[i], dtype=dtype, device=device) if vdims[i]
+                                                  else self.k[i] for i in range(num_layers)]
 
     @staticmethod
     def for_model(model, num_pages: int, page_size: int, device="cpu", num_slots: int = 0, **kw) -> "PagedKVCache":
@@ -236,5 +236,5 @@ class PagedKVCache:
             return sum(t.nbytes() for t in self.k) + sum(t.nbytes() for t in self.v)
         n = sum(t.numel() * t.element_size() for t in self.k)
         if not (self.latent or self.v is self.k):
-            n += sum(t.numel() * t.element_size() for t in self.v)
+            n += sum(t.numel() * t.element_size() for i, t in enumerate(self.v) if t is not self.k[i])
         return n + self.state_bytes()
