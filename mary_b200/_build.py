@@ -29,13 +29,13 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr", "-Xptxas", "-v",
 ]
 # Files whose arithmetic also serves 32-bit models keep the exact divide, square root and exponential; all others use the fast forms.
-EXACT_MATH = {"linear_attention", "recurrent_scan", "residual32", "gemm_simt", "attention_general", "latent", "state_space"}
+EXACT_MATH = {"linear_attention", "recurrent_scan", "residual32", "gemm_simt", "attention_general", "latent", "state_space", "ssd_chunk"}
 
 
 def _stamp(paths, extra=""):
     h = hashlib.sha256(extra.encode())
     for p in sorted(paths):
-        h.update(str(p).encode())
+        h.update(Path(p).name.encode())
         h.update(Path(p).read_bytes())
     return h.hexdigest()
 

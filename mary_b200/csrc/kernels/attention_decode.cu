@@ -33,7 +33,15 @@ struct DecParams {
   // 8-bit cache: kc / vc hold one unsigned code per element and the strides count codes; k_sz / v_sz hold (scale, zero) of every
   // (slot, kv head) as two floats, slot-major; element = code * scale + zero
   const float* k_sz; const float* v_sz;
+  const float* bias;           // [Hq][window] by distance, added to the scaled score; or null
+  const __nv_bfloat16* gate;   // rows of gate_ld elements, head h at h * D: the output times its logistic function; or null
+  int64_t gate_ld;
 };
+
+__device__ __forceinline__ __nv_bfloat16 gated(const DecParams& p, float v, int64_t row, int col) {
+  if (p.gate) v = __fdividef(v, 1.0f + __expf(-__bfloat162float(p.gate[row * p.gate_ld + col])));
+  return __float2bfloat16(v);
+}
 
 template <int E> struct Vec;                       // E bf16 elements per lane
 template <> struct Vec<2> { using T = uint32_t; };
@@ -62,8 +70,9 @@ __device__ __forceinline__ void unpack_q8(const typename QVec<E>::T& v, float sc
 // Sums V values (a power of two, at most 32) over the 32 lanes and leaves ALL V totals in every lane.  Instead of one
 // five-step butterfly per value (5 V shuffles) the values are halved between the lanes at every step (a lane keeps the half its
 // lane bit selects and adds what its partner sends), which costs V - 1 shuffles, and the V totals are then broadcast (V more).
+// `extra` is added to the total of value lane % V.
 template <int V>
-__device__ __forceinline__ void warp_sum_vec(float* v, int lane) {
+__device__ __forceinline__ void warp_sum_vec(float* v, int lane, float extra) {
 #pragma unroll
   for (int o = 16; o >= V; o >>= 1) {
 #pragma unroll
@@ -81,7 +90,7 @@ __device__ __forceinline__ void warp_sum_vec(float* v, int lane) {
     }
     (void)n;
   }
-  const float t = v[0];                                   // the total of value (lane % V)
+  const float t = v[0] + extra;                           // the total of value (lane % V)
 #pragma unroll
   for (int i = 0; i < V; ++i) v[i] = __shfl_sync(0xffffffffu, t, (lane & ~(V - 1)) | i);
 }
@@ -153,6 +162,17 @@ attn_decode_kernel(const DecParams p) {
         vv[j] = *(const KV*)(p.vc + (int64_t)page * p.v_page + tok * p.v_tok + (int64_t)kvh * D + lane * E);
       }
     }
+    constexpr int NV = KG * RMAX, NB = (NV + 31) / 32;
+    float bias[NB];                                     // of the values lane, lane + 32, ..
+#pragma unroll
+    for (int b = 0; b < NB; ++b) {
+      bias[b] = 0.f;
+      if (p.bias) {
+        const int val = b * 32 + (lane & (NV < 32 ? NV - 1 : 31)), r = val % RMAX;
+        const int dist = pos0 + r / p.G - (kb + val / RMAX);
+        if (r < R && dist >= 0 && dist < p.window) bias[b] = p.bias[(int64_t)(kvh * p.G + r % p.G) * p.window + dist];
+      }
+    }
     float s[KG][RMAX];
 #pragma unroll
     for (int j = 0; j < KG; ++j) {
@@ -171,13 +191,12 @@ attn_decode_kernel(const DecParams p) {
     }
     // finish the dot products over the 32 lanes: all KG * RMAX totals end up in every lane
     {
-      constexpr int NV = KG * RMAX;
       float* flat = &s[0][0];
       if constexpr (NV <= 32) {
-        warp_sum_vec<NV>(flat, lane);
+        warp_sum_vec<NV>(flat, lane, bias[0]);
       } else {
 #pragma unroll
-        for (int h = 0; h < NV / 32; ++h) warp_sum_vec<32>(flat + 32 * h, lane);
+        for (int h = 0; h < NV / 32; ++h) warp_sum_vec<32>(flat + 32 * h, lane, bias[h]);
       }
     }
 #pragma unroll
@@ -240,7 +259,7 @@ attn_decode_kernel(const DecParams p) {
     }
     if (p.nsplit == 1) {
       const int tq = row0 + r / p.G, h = kvh * p.G + r % p.G;
-      p.out[(int64_t)tq * p.out_ld + (int64_t)h * D + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+      p.out[(int64_t)tq * p.out_ld + (int64_t)h * D + d] = gated(p, ll > 0.f ? acc / ll : 0.f, tq, h * D + d);
     } else {
       const int64_t pi = (((int64_t)nb * p.Hkv + kvh) * p.nsplit + split) * MAXR + r;
       p.part_o[pi * D + d] = acc;
@@ -269,7 +288,7 @@ __global__ void attn_decode_combine_kernel(const DecParams p, int D) {
       acc += p.part_o[pi * D + d] * c;
     }
     const int tq = row0 + r / p.G, h = kvh * p.G + r % p.G;
-    p.out[(int64_t)tq * p.out_ld + (int64_t)h * D + d] = __float2bfloat16(ll > 0.f ? acc / ll : 0.f);
+    p.out[(int64_t)tq * p.out_ld + (int64_t)h * D + d] = gated(p, ll > 0.f ? acc / ll : 0.f, tq, h * D + d);
   }
 }
 
@@ -296,9 +315,12 @@ static int decode_run(const void* q, const void* kc, const void* vc, const float
                       const int* kv_len, const int* q_start, const int* blk_seq, const int* blk_q0, int NB,
                       int max_pages, int page_size, int64_t k_tok, int64_t k_page, int64_t v_tok, int64_t v_page,
                       int Hq, int Hkv, int D, int RQ, int nsplit, int window, float scale, float softcap,
-                      float* scratch, cudaStream_t s, int64_t out_ld = 0) {
+                      float* scratch, cudaStream_t s, int64_t out_ld = 0, const float* bias = nullptr, const void* gate = nullptr,
+                      int64_t gate_ld = 0) {
   if (NB <= 0) return MARY_OK;
+  if (bias && window < 1) return MARY_ERR_BAD_ARG;
   DecParams p;
+  p.bias = bias; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld;
   p.k_sz = k_sz; p.v_sz = v_sz;
   p.q = (const __nv_bfloat16*)q; p.kc = (const __nv_bfloat16*)kc; p.vc = (const __nv_bfloat16*)vc; p.out = (__nv_bfloat16*)out;
   p.page_table = page_table; p.kv_len = kv_len; p.q_start = q_start; p.blk_seq = blk_seq; p.blk_q0 = blk_q0;
@@ -317,14 +339,15 @@ static int decode_run(const void* q, const void* kc, const void* vc, const float
   return MARY_ERR_BAD_ARG;
 }
 
-// out_ld: elements between the output rows of two tokens (0: Hq * D, contiguous).
+// out_ld: elements between the output rows of two tokens (0: Hq * D, contiguous).  bias [Hq][window] (or null) is added to the scaled score
+// by distance, gate (or null) multiplies the output by its logistic function.
 MARY_API int mary_paged_attention_decode(const void* q, const void* kc, const void* vc, void* out, const int* page_table,
                                          const int* kv_len, const int* q_start, const int* blk_seq, const int* blk_q0, int NB,
                                          int max_pages, int page_size, int64_t k_tok, int64_t k_page, int64_t v_tok, int64_t v_page,
                                          int Hq, int Hkv, int D, int RQ, int nsplit, int window, float scale, float softcap,
-                                         float* scratch, int64_t out_ld, cudaStream_t s) {
+                                         float* scratch, int64_t out_ld, const float* bias, const void* gate, int64_t gate_ld, cudaStream_t s) {
   return decode_run(q, kc, vc, nullptr, nullptr, out, page_table, kv_len, q_start, blk_seq, blk_q0, NB, max_pages, page_size, k_tok, k_page,
-                    v_tok, v_page, Hq, Hkv, D, RQ, nsplit, window, scale, softcap, scratch, s, out_ld);
+                    v_tok, v_page, Hq, Hkv, D, RQ, nsplit, window, scale, softcap, scratch, s, out_ld, bias, gate, gate_ld);
 }
 
 // The same over an 8-bit cache: kc / vc are code pages [pages, page, Hkv, D] of unsigned bytes (strides in bytes), k_sz / v_sz the

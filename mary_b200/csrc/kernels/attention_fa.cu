@@ -40,7 +40,7 @@ struct FaCfg {
   static constexpr int K_CHUNK_BYTES = KB * 128, V_CHUNK_BYTES = KB * 128;
   static constexpr int K_STAGE = NCK * K_CHUNK_BYTES, V_STAGE = NCV * V_CHUNK_BYTES;
   static constexpr int STAGES = (DK + DV > 384) ? 2 : 3;
-  static constexpr int NPBUF = (SPLITP && DK + DV > 384) ? 1 : 2;
+  static constexpr int NPBUF = (SPLITP && DK + DV > 256) ? 1 : 2;
   static constexpr int P_STAGE = SPLITP ? 2 * P_BYTES : P_BYTES;
   static constexpr int SMEM = Q_BYTES + STAGES * (K_STAGE + V_STAGE) + NPBUF * P_STAGE + 1024 + 256;
   static constexpr int TMEM_COLS = DV <= 128 ? 256 : 512;     // S: 2 x 64 columns at 0..127, O: DV columns at 128..
@@ -54,6 +54,9 @@ struct FaParams {
   int64_t out_ld;          // elements between the output rows of two tokens
   int max_pages, Hq, Hkv, window, page;
   float scale_log2;
+  const float* bias;       // BIAS: [Hq][window] by distance, added to the scaled score
+  const __nv_bfloat16* gate;   // rows of gate_ld elements, head h at h * DV: the output times its logistic function; or null
+  int64_t gate_ld;
   int* status;
 };
 
@@ -65,7 +68,7 @@ __device__ __forceinline__ uint64_t fa_desc_mnmajor_sw128(uint32_t addr, uint32_
          (2ull << 61);
 }
 
-template <int DK, int DV, bool SPLITP>
+template <int DK, int DV, bool SPLITP, bool BIAS>
 __global__ void __launch_bounds__(NTHREADS, 1)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                   const __grid_constant__ CUtensorMap tm_v, const FaParams p) {
@@ -242,7 +245,19 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       const bool full_blk = key0 + KB - 1 <= pos_first && (p.window <= 0 || key0 >= pos_first + TR - p.window);
       const float* sf = (const float*)sr;
       float mx;
-      if (full_blk) {
+      if (BIAS) {
+        constexpr float LOG2E = 1.4426950408889634f;
+        const float* br = p.bias + (int64_t)head * p.window + (qpos - key0);      // br[-j]: bias of key j of the block
+        mx = -INFINITY;
+#pragma unroll
+        for (int j = 0; j < KB; ++j) {
+          const int kj = key0 + j;
+          const bool ok = full_blk || (row_ok && kj <= qpos && kj >= lo_key);
+          const float v = ok ? fmaf(br[-j], LOG2E, __uint_as_float(sr[j]) * p.scale_log2) : -INFINITY;
+          sr[j] = __float_as_uint(v);
+          mx = fmaxf(mx, v);
+        }
+      } else if (full_blk) {
         mx = sf[0];
 #pragma unroll
         for (int j = 1; j < KB; ++j) mx = fmaxf(mx, sf[j]);
@@ -264,7 +279,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       if (need) { corr = first ? 0.f : exp2f(m_ref - mx); m_ref = mx; }
       uint32_t pw[KB / 2], pl[SPLITP ? KB / 2 : 1];
       float psum = 0.f;
-      if (full_blk) {
+      if (full_blk && !BIAS) {
         const float nm = -m_ref;
 #pragma unroll
         for (int j = 0; j < KB / 2; ++j) {
@@ -344,6 +359,21 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
         __nv_bfloat16* dst = p.out + (int64_t)(tok0 + r) * p.out_ld + head * DV + c0;
         uint4 w[4];
         uint32_t* wp = (uint32_t*)w;
+        if (p.gate) {
+          const uint4* src = (const uint4*)(p.gate + (int64_t)(tok0 + r) * p.gate_ld + head * DV + c0);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const uint4 g = src[j];
+            const __nv_bfloat162* gh = (const __nv_bfloat162*)&g;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const float2 f = __bfloat1622float2(gh[i]);
+              float &a = *(float*)&o[8 * j + 2 * i], &b = *(float*)&o[8 * j + 2 * i + 1];
+              a = __fdividef(a, 1.0f + __expf(-f.x));
+              b = __fdividef(b, 1.0f + __expf(-f.y));
+            }
+          }
+        }
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           __nv_bfloat162 h = __floats2bfloat162_rn(__uint_as_float(o[2 * j]) * inv_l, __uint_as_float(o[2 * j + 1]) * inv_l);
@@ -384,12 +414,12 @@ int make_cache_map(CUtensorMap* m, const void* cache, int heads, int hd, int num
   return r == CUDA_SUCCESS ? MARY_OK : MARY_ERR_CUDA;
 }
 
-template <int DK, int DV, bool SPLITP>
+template <int DK, int DV, bool SPLITP, bool BIAS>
 int launch_fa(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const FaParams& p, int NB, cudaStream_t s) {
   static MarySmemSlots smem_set = {};
   constexpr int SMEM = FaCfg<DK, DV, SPLITP>::SMEM;
-  if (int rc = mary_ensure_dyn_smem((const void*)fa_prefill_kernel<DK, DV, SPLITP>, SMEM, &smem_set)) return rc;
-  fa_prefill_kernel<DK, DV, SPLITP><<<dim3(NB, p.Hq), NTHREADS, SMEM, s>>>(tq, tk, tv, p);
+  if (int rc = mary_ensure_dyn_smem((const void*)fa_prefill_kernel<DK, DV, SPLITP, BIAS>, SMEM, &smem_set)) return rc;
+  fa_prefill_kernel<DK, DV, SPLITP, BIAS><<<dim3(NB, p.Hq), NTHREADS, SMEM, s>>>(tq, tk, tv, p);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }
@@ -407,12 +437,13 @@ MARY_API int mary_attention_prefill_supported(int DK, int DV) {
 // and per page (heads contiguous inside a token row); out [T, Hq, DV] bf16.  blk_seq / blk_tok0: NB tiles of at most 128 query
 // tokens that never cross a sequence.  Causal with the last query token of a sequence at position kv_len - 1; window > 0 keeps
 // keys (pos - window, pos].  out_ld: elements between the output rows of two tokens (0: Hq * DV; a multiple of 8).  split_p: softmax
-// weights with 16 significant bits (equal key and value widths only).  Returns MARY_ERR_BAD_ARG for head dims without an instantiation.
+// weights with 16 significant bits.  bias [Hq][window] (or null; with split_p and equal widths only) is added to the scaled score by
+// distance, gate (or null; 16-byte aligned rows) multiplies the output by its logistic function.  Returns MARY_ERR_BAD_ARG for head dims without an instantiation.
 MARY_API int mary_attention_prefill(const void* q, const void* kcache, const void* vcache, void* out, const int* page_table,
                                     const int* kv_len, const int* q_start, const int* blk_seq, const int* blk_tok0, int NB, int T, int Hq,
                                     int Hkv, int DK, int DV, int num_pages, int max_pages, int64_t k_tok_stride, int64_t k_page_stride,
                                     int64_t v_tok_stride, int64_t v_page_stride, int window, float scale, int page_size,
-                                    int64_t out_ld, int split_p, cudaStream_t s) {
+                                    int64_t out_ld, int split_p, const float* bias, const void* gate, int64_t gate_ld, cudaStream_t s) {
   if (NB <= 0) return MARY_OK;
   if (!mary_attention_prefill_supported(DK, DV) || Hkv < 1 || Hq % Hkv || (page_size != PAGE && page_size != KB)) return MARY_ERR_BAD_ARG;
   if ((k_tok_stride * 2) % 16 || (k_page_stride * 2) % 16 || (v_tok_stride * 2) % 16 || (v_page_stride * 2) % 16) return MARY_ERR_BAD_ARG;
@@ -425,15 +456,23 @@ MARY_API int mary_attention_prefill(const void* q, const void* kcache, const voi
   p.page_table = page_table; p.kv_len = kv_len; p.q_start = q_start; p.blk_seq = blk_seq; p.blk_tok0 = blk_tok0;
   p.out = (__nv_bfloat16*)out; p.max_pages = max_pages; p.Hq = Hq; p.Hkv = Hkv; p.window = window; p.page = page_size;
   p.out_ld = out_ld > 0 ? out_ld : (int64_t)Hq * DV;
-  if (p.out_ld % 8 || ((uintptr_t)out & 15) || (split_p && DK != DV)) return MARY_ERR_BAD_ARG;
+  p.bias = bias; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld;
+  if (p.out_ld % 8 || ((uintptr_t)out & 15) || gate_ld % 8 || ((uintptr_t)gate & 15)) return MARY_ERR_BAD_ARG;
+  if (bias && (!split_p || DK != DV || window < 1)) return MARY_ERR_BAD_ARG;
   p.scale_log2 = scale * 1.4426950408889634f; p.status = mary_status_ptr();
-  if (split_p) {
-    if (DK == 64) return launch_fa<64, 64, true>(tq, tk, tv, p, NB, s);
-    if (DK == 128) return launch_fa<128, 128, true>(tq, tk, tv, p, NB, s);
-    return launch_fa<256, 256, true>(tq, tk, tv, p, NB, s);
+  if (bias) {
+    if (DK == 64) return launch_fa<64, 64, true, true>(tq, tk, tv, p, NB, s);
+    if (DK == 128) return launch_fa<128, 128, true, true>(tq, tk, tv, p, NB, s);
+    return launch_fa<256, 256, true, true>(tq, tk, tv, p, NB, s);
   }
-  if (DK == 64) return launch_fa<64, 64, false>(tq, tk, tv, p, NB, s);
-  if (DK == 128) return launch_fa<128, 128, false>(tq, tk, tv, p, NB, s);
-  if (DK == 192) return launch_fa<192, 128, false>(tq, tk, tv, p, NB, s);
-  return launch_fa<256, 256, false>(tq, tk, tv, p, NB, s);
+  if (split_p) {
+    if (DK == 64) return launch_fa<64, 64, true, false>(tq, tk, tv, p, NB, s);
+    if (DK == 128) return launch_fa<128, 128, true, false>(tq, tk, tv, p, NB, s);
+    if (DK == 192) return launch_fa<192, 128, true, false>(tq, tk, tv, p, NB, s);
+    return launch_fa<256, 256, true, false>(tq, tk, tv, p, NB, s);
+  }
+  if (DK == 64) return launch_fa<64, 64, false, false>(tq, tk, tv, p, NB, s);
+  if (DK == 128) return launch_fa<128, 128, false, false>(tq, tk, tv, p, NB, s);
+  if (DK == 192) return launch_fa<192, 128, false, false>(tq, tk, tv, p, NB, s);
+  return launch_fa<256, 256, false, false>(tq, tk, tv, p, NB, s);
 }

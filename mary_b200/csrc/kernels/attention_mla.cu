@@ -42,9 +42,9 @@ constexpr int K_CHUNK_BYTES = KB * 128;           // 4 KB: 32 keys of one 64-dim
 constexpr int STAGE_BYTES = NCHUNK * K_CHUNK_BYTES;   // 36 KB
 constexpr int STAGES = 4;
 constexpr int NSBUF = 3;                          // S accumulators in TMEM
-constexpr int NPBUF = 2;                          // P tiles in shared memory
+constexpr int P_TILES = 2;                        // P tiles in shared memory: two buffers, or value and rounding error of one
 constexpr int P_BYTES = TR * KB * 2;              // 4 KB
-constexpr int SMEM = Q_BYTES + STAGES * STAGE_BYTES + NPBUF * P_BYTES + 1024 + 256;
+constexpr int SMEM = Q_BYTES + STAGES * STAGE_BYTES + P_TILES * P_BYTES + 1024 + 256;
 constexpr int TMEM_COLS = 512;                    // S 3 x 32 at columns 0..95, O 256 at columns 128..383
 constexpr int NTHREADS = 192;
 constexpr float RESCALE_THRESHOLD = 8.0f;
@@ -55,7 +55,7 @@ struct MlaParams {
   __nv_bfloat16* out;      // [T * Hq, 512]
   float* part_o;           // [NB, nsplit, 64, 512] when nsplit > 1
   float* part_ml;          // [NB, nsplit, 64, 2]
-  int max_pages, Hq, nsplit, page;
+  int max_pages, Hq, nsplit, page, window;
   float scale_log2;        // softmax scale * log2(e)
   int* status;
 };
@@ -72,15 +72,19 @@ __device__ __forceinline__ uint64_t desc_mnmajor_sw128(uint32_t addr, uint32_t l
          (2ull << 61);
 }
 
+// SPLITP: P is handed to the tensor cores as the sum of two bf16 values (rounded value and rounding error), so that the softmax weights
+// keep 16 significant bits; one P buffer then, and two P V products per block.
+template <bool SPLITP>
 __global__ void __launch_bounds__(NTHREADS, 1)
 mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv, const MlaParams p) {
   pdl_sync();
+  constexpr int NPBUF = SPLITP ? 1 : P_TILES;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
   uint8_t* sK = smem + Q_BYTES;
   uint8_t* sP = sK + STAGES * STAGE_BYTES;
-  uint64_t* bars = (uint64_t*)(sP + NPBUF * P_BYTES);
+  uint64_t* bars = (uint64_t*)(sP + P_TILES * P_BYTES);
   uint64_t* q_full = bars;                 // 1
   uint64_t* k_full = q_full + 1;           // [STAGES]
   uint64_t* k_empty = k_full + STAGES;     // [STAGES]
@@ -101,9 +105,11 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
   const int pos_first = kvlen - qlen;                             // position of the sequence's first query token
   const int tok_hi = (row0 - seq_row0 + nrows - 1) / p.Hq;
   const int k_hi = pos_first + tok_hi + 1;                        // keys [0, k_hi) are visible to some row of the tile
-  const int nblk_total = (k_hi + KB - 1) / KB;
-  const int per = (nblk_total + p.nsplit - 1) / p.nsplit;
-  const int b_lo = split * per, b_hi = min(nblk_total, b_lo + per);
+  const int tok_lo = (row0 - seq_row0) / p.Hq;
+  const int first_blk = p.window > 0 ? max(0, pos_first + tok_lo - p.window + 1) / KB : 0;      // blocks before it are outside every window
+  const int end_blk = (k_hi + KB - 1) / KB;
+  const int per = (end_blk - first_blk + p.nsplit - 1) / p.nsplit;
+  const int b_lo = first_blk + split * per, b_hi = min(end_blk, b_lo + per);
   const int nblk = max(0, b_hi - b_lo);
 
   if (threadIdx.x == 0) {
@@ -141,12 +147,12 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
         }
         ok = __shfl_sync(0xffffffffu, ok, 0);
         if (!ok) goto done;
-        if (p.page == KB) {
-          // one operation brings the whole stage: box [64 dims, 32 tokens, 9 chunks] of one page
+        if (p.page >= KB) {
+          // one operation brings the whole stage: box [64 dims, 32 tokens, 9 chunks] of one page (half of a 64-token page)
           if (lane == 0) {
             const int key0 = b * KB;
-            const int page = (key0 < kvlen) ? pt[key0 / KB] : pt[0];
-            tma_load_4d(sK + stage * STAGE_BYTES, &tm_kv, &k_full[stage], 0, 0, 0, page);
+            const int page = (key0 < kvlen) ? pt[key0 / p.page] : pt[0];
+            tma_load_4d(sK + stage * STAGE_BYTES, &tm_kv, &k_full[stage], 0, key0 % p.page, 0, page);
           }
         } else if (lane < (KB / PAGE) * NCHUNK) {
           // 2 pages x 9 chunks = 18 operations of [16 tokens x 64 dims] (2 KB each)
@@ -190,8 +196,8 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
         if (a < nblk && !issue_qk(a)) goto done;
       for (int i = 0; i < nblk; ++i) {
         if (i + AHEAD < nblk && !issue_qk(i + AHEAD)) goto done;
-        const int pb = i & 1;
-        if (!mbar_wait(&p_full[pb], (i >> 1) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+        const int pb = i % NPBUF;
+        if (!mbar_wait(&p_full[pb], (i / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
         tc_fence_after();
         const int stage = i % STAGES;
         const uint32_t kb_addr = smem_u32(sK + stage * STAGE_BYTES);
@@ -205,6 +211,9 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
             umma_f16(tmem_O + ((uint32_t)(half * 16) << 16), desc_kmajor_noswz(p_addr + pb * P_BYTES + kk * 2 * (TR * 16), TR * 16, 128),
                      desc_mnmajor_sw128(kb_addr + half * 4 * K_CHUNK_BYTES + kk * 16 * 128, K_CHUNK_BYTES, 1024), idesc_o,
                      (i > 0 || kk > 0) ? 1u : 0u);
+            if constexpr (SPLITP)
+              umma_f16(tmem_O + ((uint32_t)(half * 16) << 16), desc_kmajor_noswz(p_addr + P_BYTES + kk * 2 * (TR * 16), TR * 16, 128),
+                       desc_mnmajor_sw128(kb_addr + half * 4 * K_CHUNK_BYTES + kk * 16 * 128, K_CHUNK_BYTES, 1024), idesc_o, 1u);
           }
         }
         umma_commit(&k_empty[stage]);       // the stage may be overwritten once PV has read it
@@ -217,11 +226,13 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
     const int r = q4 * 16 + (lane & 15);            // accumulator row held by this lane (lanes 16-31 hold nothing)
     const bool row_ok = lane < 16 && r < nrows;
     const int qpos = pos_first + (row0 - seq_row0 + r) / p.Hq;
-    const int qpos_min = pos_first + (row0 - seq_row0) / p.Hq;      // the tile's first row sees the fewest keys
+    const int qpos_min = pos_first + tok_lo;                        // the tile's first row sees the fewest keys
+    const int lo_key = p.window > 0 ? qpos - p.window + 1 : 0;
+    const int lo_max = p.window > 0 ? pos_first + tok_hi - p.window + 1 : 0;      // and its last row's window starts latest
     const uint32_t lane_off = (uint32_t)(q4 * 32) << 16;
     float m_ref = -INFINITY, l = 0.f;
     for (int i = 0; i < nblk; ++i) {
-      const int sb = i % NSBUF, pb = i & 1;
+      const int sb = i % NSBUF, pb = i % NPBUF;
       if (!mbar_wait(&s_full[sb], (i / NSBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
       tc_fence_after();
       uint32_t sr[KB];
@@ -234,7 +245,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
       // A block that every row of the tile sees entirely (all but the last one or two of a decode step) takes the short path:
       // no per-element mask, the maximum on the raw scores, one fused multiply-add and one exponential per element.  A row's
       // 32 scores are processed by ONE lane in sequence, so the instruction count of this loop is the kernel's cycle time.
-      const bool full_blk = key0 + KB - 1 <= qpos_min;
+      const bool full_blk = key0 + KB - 1 <= qpos_min && key0 >= lo_max;
       const float* sf = (const float*)sr;
       float sv[KB];
       float mx;
@@ -247,7 +258,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
         mx = -INFINITY;
 #pragma unroll
         for (int j = 0; j < KB; ++j) {
-          const bool ok = row_ok && (key0 + j) <= qpos;
+          const bool ok = row_ok && (key0 + j) <= qpos && (key0 + j) >= lo_key;
           sv[j] = ok ? sf[j] * p.scale_log2 : -INFINITY;
           mx = fmaxf(mx, sv[j]);
         }
@@ -259,7 +270,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
       float corr = 1.f;
       if (need) { corr = first ? 0.f : exp2f(m_ref - mx); m_ref = mx; }
       // probabilities in registers first: the waits below then overlap this arithmetic of the other warps
-      uint32_t pw[KB / 2];
+      uint32_t pw[KB / 2], pl[SPLITP ? KB / 2 : 1];
       float psum = 0.f;
       if (full_blk) {
         const float nm = -m_ref;
@@ -269,6 +280,11 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
           const float b = exp2f(fmaf(sf[2 * j + 1], p.scale_log2, nm));
           __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
           pw[j] = *(uint32_t*)&h;
+          if constexpr (SPLITP) {
+            const float2 back = __bfloat1622float2(h);
+            __nv_bfloat162 lo = __floats2bfloat162_rn(a - back.x, b - back.y);
+            pl[j] = *(uint32_t*)&lo;
+          }
           psum += a + b;
         }
       } else {
@@ -279,7 +295,13 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
           __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
           pw[j] = *(uint32_t*)&h;
           float2 back = __bfloat1622float2(h);
-          psum += back.x + back.y;
+          if constexpr (SPLITP) {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(a - back.x, b - back.y);
+            pl[j] = *(uint32_t*)&lo;
+            psum += a + b;
+          } else {
+            psum += back.x + back.y;
+          }
         }
       }
       l = l * corr + psum;
@@ -287,7 +309,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
       const float corr_o = __shfl_sync(0xffffffffu, corr, lane & 15);
       if (__any_sync(0xffffffffu, need && !first) && i > 0) {
         // O may only be touched once the previous P V has completed
-        if (!mbar_wait(&pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+        if (!mbar_wait(&pv_done[(i - 1) % NPBUF], ((i - 1) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
         tc_fence_after();
 #pragma unroll 1
         for (int c0 = 0; c0 < DVH; c0 += 32) {
@@ -302,14 +324,19 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
         tmem_st_wait();
       }
       if (i >= NPBUF) {
-        // this P buffer was last read by the P V of block i - 2
-        if (!mbar_wait(&pv_done[pb], ((i - NPBUF) >> 1) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+        // this P buffer was last read by the P V of block i - NPBUF
+        if (!mbar_wait(&pv_done[pb], ((i - NPBUF) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
       }
       // P (bf16) -> shared memory: chunk c holds keys 8c..8c+7 of every row, 16 bytes per row
       if (lane < 16) {
 #pragma unroll
         for (int c = 0; c < KB / 8; ++c)
           *(uint4*)(sP + pb * P_BYTES + c * (TR * 16) + r * 16) = make_uint4(pw[4 * c], pw[4 * c + 1], pw[4 * c + 2], pw[4 * c + 3]);
+        if constexpr (SPLITP) {
+#pragma unroll
+          for (int c = 0; c < KB / 8; ++c)
+            *(uint4*)(sP + P_BYTES + c * (TR * 16) + r * 16) = make_uint4(pl[4 * c], pl[4 * c + 1], pl[4 * c + 2], pl[4 * c + 3]);
+        }
       }
       fence_proxy_async();       // make the generic-proxy writes of P visible to the tensor core
       tc_fence_before();
@@ -317,7 +344,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
       if (lane == 0) mbar_arrive(&p_full[pb]);
     }
     // ------------------------------------------------------------------ write out
-    if (!mbar_wait(&pv_done[(nblk - 1) & 1], ((nblk - 1) >> 1) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+    if (!mbar_wait(&pv_done[(nblk - 1) % NPBUF], ((nblk - 1) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
     tc_fence_after();
     const float l_row = __shfl_sync(0xffffffffu, l, lane & 15);
     const float inv_l = l_row > 0.f ? 1.f / l_row : 0.f;
@@ -399,25 +426,26 @@ typedef CUresult (*PFN_encode)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, vo
 MARY_API int64_t mary_mla_scratch_floats(int NB, int nsplit) { return nsplit > 1 ? (int64_t)NB * nsplit * TR * (DV + 2) : 0; }
 MARY_API int mary_mla_tile_rows() { return TR; }
 
-// q [T * Hq, 576] bf16 (rows = token-major, head-minor); cache [pages, page_size (16 or 32), 576] bf16 with element strides
+// q [T * Hq, 576] bf16 (rows = token-major, head-minor); cache [pages, page_size (16, 32 or 64), 576] bf16 with element strides
 // tok_stride / page_stride; out [T * Hq, 512] bf16.  blk_seq / blk_row0: NB tiles of query rows (row0 is a global
-// row index; a tile never crosses a sequence).  Tiles hold at most mary_mla_tile_rows() rows.
+// row index; a tile never crosses a sequence).  Tiles hold at most mary_mla_tile_rows() rows.  window > 0
+// keeps keys (pos - window, pos]; split_p: softmax weights with 16 significant bits.
 MARY_API int mary_mla_attention(const void* q, const void* cache, void* out, const int* page_table, const int* kv_len, const int* q_start,
                                 const int* blk_seq, const int* blk_row0, int NB, int total_rows, int num_pages, int max_pages,
                                 int64_t tok_stride, int64_t page_stride, int Hq, int nsplit, float scale, float* scratch,
-                                int page_size, cudaStream_t s) {
+                                int page_size, int window, int split_p, cudaStream_t s) {
   if (NB <= 0) return MARY_OK;
   if (nsplit < 1) nsplit = 1;
   if (nsplit > 1 && !scratch) return MARY_ERR_BAD_ARG;
-  if ((tok_stride * 2) % 16 || (page_stride * 2) % 16 || (page_size != PAGE && page_size != KB)) return MARY_ERR_BAD_ARG;
+  if ((tok_stride * 2) % 16 || (page_stride * 2) % 16 || (page_size != PAGE && page_size != KB && page_size != 2 * KB)) return MARY_ERR_BAD_ARG;
   PFN_encode enc = (PFN_encode)mary_encode_fn();
   if (!enc) return MARY_ERR_CUDA;
   CUtensorMap tq, tkv;
   int rc = mary_make_tmap_2d(&tq, q, 4, (uint64_t)total_rows, DK, DK, TR, CHUNK, 1);
   if (rc) return rc;
-  if (page_size == KB) {
-    // dims: 64 elements of a chunk, 32 tokens of a page, 9 chunks of a token row, pages; box = one whole page, chunk-major
-    cuuint64_t dims[4] = {CHUNK, KB, NCHUNK, (cuuint64_t)num_pages};
+  if (page_size >= KB) {
+    // dims: 64 elements of a chunk, tokens of a page, 9 chunks of a token row, pages; box = 32 tokens of one page, chunk-major
+    cuuint64_t dims[4] = {CHUNK, (cuuint64_t)page_size, NCHUNK, (cuuint64_t)num_pages};
     cuuint64_t strides[3] = {(cuuint64_t)tok_stride * 2, CHUNK * 2, (cuuint64_t)page_stride * 2};
     cuuint32_t box[4] = {CHUNK, KB, NCHUNK, 1};
     cuuint32_t estr[4] = {1, 1, 1, 1};
@@ -434,13 +462,14 @@ MARY_API int mary_mla_attention(const void* q, const void* cache, void* out, con
             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
       return MARY_ERR_CUDA;
   }
-  static MarySmemSlots smem_set = {};
-  if (int rc = mary_ensure_dyn_smem((const void*)mla_attn_kernel, SMEM, &smem_set)) return rc;
+  static MarySmemSlots smem_set[2] = {};
+  auto fn = split_p ? mla_attn_kernel<true> : mla_attn_kernel<false>;
+  if (int rc = mary_ensure_dyn_smem((const void*)fn, SMEM, &smem_set[split_p ? 1 : 0])) return rc;
   MlaParams p;
   p.page_table = page_table; p.kv_len = kv_len; p.q_start = q_start; p.blk_seq = blk_seq; p.blk_row0 = blk_row0;
   p.out = (__nv_bfloat16*)out; p.part_o = scratch; p.part_ml = scratch ? scratch + (int64_t)NB * nsplit * TR * DV : nullptr;
-  p.max_pages = max_pages; p.Hq = Hq; p.nsplit = nsplit; p.page = page_size; p.scale_log2 = scale * 1.4426950408889634f; p.status = mary_status_ptr();
-  MARY_LAUNCH(mla_attn_kernel, dim3(NB, nsplit), NTHREADS, SMEM, s, tq, tkv, p);
+  p.max_pages = max_pages; p.Hq = Hq; p.nsplit = nsplit; p.page = page_size; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.status = mary_status_ptr();
+  MARY_LAUNCH(fn, dim3(NB, nsplit), NTHREADS, SMEM, s, tq, tkv, p);
   MARY_CHECK_LAUNCH();
   if (nsplit > 1) {
     MARY_LAUNCH(mla_combine_kernel, dim3(NB, TR), 128, 0, s, p, NB);

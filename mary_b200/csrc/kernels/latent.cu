@@ -71,6 +71,18 @@ __global__ void __launch_bounds__(NT) rotate_heads_kernel(const T* src, T* dst, 
   d[1] = from_f<T>(v);
 }
 
+// Keys of an expanded prompt: the rotated part of cache row n behind the own dims of every head, k [n_rows, H, dim + rot].
+template <typename T>
+__global__ void __launch_bounds__(NT) fill_shared_part_kernel(const T* __restrict__ rows, int64_t ld, int rank, T* __restrict__ k, int64_t n, int H, int dim,
+                                                              int rot) {
+  pdl_sync();
+  const int64_t i = (int64_t)blockIdx.x * NT + threadIdx.x;
+  if (i >= n) return;
+  const int d = (int)(i % rot);
+  const int64_t nh = i / rot;
+  k[nh * (dim + rot) + dim + d] = rows[(nh / H) * ld + rank + d];
+}
+
 }  // namespace
 
 #define BY_TYPE(f32, ...)                                      \
@@ -98,6 +110,16 @@ MARY_API int mary_rotate_heads(const void* src, void* dst, const float* freq, fl
   const int64_t n = (int64_t)n_tok * H * (rot / 2);
   BY_TYPE(f32, MARY_LAUNCH((rotate_heads_kernel<T>), (unsigned)((n + NT - 1) / NT), NT, 0, s, (const T*)src, (T*)dst, freq, rot_gain, positions, n, H, src_w,
                            dst_w, dst_off, rot));
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
+}
+
+MARY_API int mary_fill_shared_part(const void* rows, int64_t ld, int rank, void* k, int64_t n_rows, int H, int dim, int rot, int f32, cudaStream_t s) {
+  if (n_rows <= 0 || rot == 0) return MARY_OK;
+  if (H < 1 || rot < 0 || dim < 1) return MARY_ERR_BAD_ARG;
+  const int64_t n = n_rows * H * rot;
+  if ((n + NT - 1) / NT > 0x7fffffff) return MARY_ERR_BAD_ARG;
+  BY_TYPE(f32, MARY_LAUNCH((fill_shared_part_kernel<T>), (unsigned)((n + NT - 1) / NT), NT, 0, s, (const T*)rows, ld, rank, (T*)k, n, H, dim, rot));
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }

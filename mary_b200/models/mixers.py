@@ -177,7 +177,7 @@ def distance_buckets(window: int, rows: int, far: float):
     """Row of a bias table with ``rows`` rows for the distances ``0 .. window - 1``: one row each up to half of the table, from there
     logarithmic steps that reach the last row at distance ``far``."""
     half = rows // 2
-    if rows < 2 or far <= half:
+    if window > half and (rows < 2 or far <= half):
         raise ValueError(f"a table of {rows} rows cannot reach to distance {far}")
     step = math.log(far / half)
     return torch.tensor([n if n < half else min(rows - 1, half + math.floor(math.log(n / half) / step * (rows - half))) for n in range(window)])

@@ -64,7 +64,7 @@ FAMILIES = [
     Family("tatizen", lambda d: d.get("architecture") == "Tatizen", _load_tatizen, page_size=64, f32_on_gpu=True,
            kernels=_DENSE_KERNELS + ("attention_general", "residual32", "linear_attention", "recurrent_scan")),
     Family("rokarax", lambda d: d.get("architecture") == "Rokarax", _load_rokarax, page_size=64, f32_on_gpu=True,
-           kernels=_DENSE_KERNELS + ("attention_general", "attention_mla", "residual32", "linear_attention", "recurrent_scan", "latent", "state_space")),
+           kernels=_DENSE_KERNELS + ("attention_general", "attention_mla", "residual32", "linear_attention", "recurrent_scan", "latent", "state_space", "ssd_chunk")),
     Family("gemma4", lambda d: str(d.get("model_type", "")).startswith("gemma4"), _load_gemma4),
     Family("mistral", lambda d: d.get("model_type") in ("mistral", "ministral", "qwen3", "mistral3"), _load_mistral),
 ]

@@ -353,14 +353,20 @@ def _q_blocks(meta, rq: int, group: str | None = None):
     return cache[key]
 
 
-declare("mary_paged_attention_decode", "ppppppppp" + "iii" + "llll" + "iiiiii" + "ff" + "pls")
+declare("mary_paged_attention_decode", "ppppppppp" + "iii" + "llll" + "iiiiii" + "ff" + "pl" + "ppls")
 
 
 DECODE_TARGET_CTAS = 2368      # CTAs the decode attention kernel aims for when it picks the number of kv splits (16 per SM)
 
 
-def _paged_attention_decode(q, kcache, vcache, meta, scale, window, softcap, nsplit, out=None, group=None):
-    """Decode-shaped batches (few rows per kv head, equal K and V widths of 64/128/256): the bandwidth-oriented kernel."""
+def _gate(gate):
+    """Pointer and pitch of an optional gate ``[T, n]`` (a row view)."""
+    return (None, 0) if gate is None else (_p(gate), gate.stride(0))
+
+
+def _paged_attention_decode(q, kcache, vcache, meta, scale, window, softcap, nsplit, out=None, group=None, bias=None, gate=None):
+    """Decode-shaped batches (few rows per kv head, equal K and V widths of 64/128/256): the bandwidth-oriented kernel.  ``bias``, ``gate``: see
+    ``ops.attention_exact``."""
     T, Hq, D = q.shape
     Hkv = kcache.shape[2]
     G = Hq // Hkv
@@ -382,7 +388,7 @@ def _paged_attention_decode(q, kcache, vcache, meta, scale, window, softcap, nsp
     check(lib().mary_paged_attention_decode(_p(q.contiguous()), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len),
                                             _p(meta.q_start), _p(blk_seq), _p(blk_q0), NB, meta.page_table.shape[1], meta.page_size,
                                             kcache.stride(1), kcache.stride(0), vcache.stride(1), vcache.stride(0), Hq, Hkv, D, rq,
-                                            nsplit, window, scale, softcap, _p(scratch), ld, _stream()), "paged_attention_decode")
+                                            nsplit, window, scale, softcap, _p(scratch), ld, _p(bias), *_gate(gate), _stream()), "paged_attention_decode")
     return out
 
 
@@ -471,17 +477,18 @@ def gqa_decode_tc(q, kcache, vcache, meta, scale, window=0, softcap=0.0, nsplit=
     return out
 
 
-declare("mary_attention_prefill", "ppppppppp" + "iiiiiiii" + "llll" + "ifi" + "lis")
+declare("mary_attention_prefill", "ppppppppp" + "iiiiiiii" + "llll" + "ifi" + "li" + "ppls")
 declare("mary_attention_prefill_supported", "ii")
 PREFILL_MIN_ROWS = 48     # mean query tokens per sequence from which the 128-row tensor-core tiles pay off
 
 
-def attention_prefill(q, kcache, vcache, meta, scale, window=0, out=None, split_p: bool = False, group=None):
+def attention_prefill(q, kcache, vcache, meta, scale, window=0, out=None, split_p: bool = False, group=None, bias=None, gate=None):
     """Causal / sliding-window attention of whole query blocks on the tensor cores (``csrc/kernels/attention_fa.cu``):
     ``q[T, Hq, DK]``, caches ``[pages, page, Hkv, D]``; 128 query tokens of one head per CTA.  A cache with 64-token pages is
     streamed with one TMA operation per 64-key stage; a cache with smaller pages is first regrouped into 64-token pages (one
     gather, small beside the attention arithmetic) when the host knows the sequence lengths.
-    ``split_p`` keeps 16 significant bits of the softmax weights; ``out`` may be a row view ``[T, Hq * DV]``; ``group``: see ``_q_blocks``."""
+    ``split_p`` keeps 16 significant bits of the softmax weights; ``out`` may be a row view ``[T, Hq * DV]``; ``group``: see ``_q_blocks``; ``bias`` (with
+    ``split_p``), ``gate``: see ``ops.attention_exact``."""
     T, Hq, DK = q.shape
     Hkv, DV = kcache.shape[2], vcache.shape[-1]
     ps = meta.page_size
@@ -501,7 +508,7 @@ def attention_prefill(q, kcache, vcache, meta, scale, window=0, out=None, split_
     check(lib().mary_attention_prefill(_p(q.contiguous()), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len),
                                        _p(meta.q_start), _p(blk_seq), _p(blk_tok0), NB, T, Hq, Hkv, DK, DV, kcache.shape[0],
                                        meta.page_table.shape[1], kcache.stride(1), kcache.stride(0), vcache.stride(1), vcache.stride(0),
-                                       int(window), float(scale), ps, ld, int(split_p), _stream()), "attention_prefill")
+                                       int(window), float(scale), ps, ld, int(split_p), _p(bias), *_gate(gate), _stream()), "attention_prefill")
     return out
 
 
@@ -626,13 +633,13 @@ def quantize_nvfp4(x):
 
 
 # --------------------------------------------------------------------------- MLA
-declare("mary_mla_attention", "pppppppp" + "iiii" + "ll" + "ii" + "f" + "pis")
+declare("mary_mla_attention", "pppppppp" + "iiii" + "ll" + "ii" + "f" + "pi" + "iis")
 declare("mary_mla_scratch_floats", "ii", ret64=True)
 declare("mary_mla_tile_rows", "")
 
 
-def _row_tiles(meta, hq: int):
-    key = ("rowtiles", hq)
+def _row_tiles(meta, hq: int, group: str | None = None):
+    key = ("rowtiles", hq, group)
     cache = meta.__dict__.setdefault("_cache", {})
     if key not in cache:
         seqs, r0 = [], []
@@ -640,7 +647,7 @@ def _row_tiles(meta, hq: int):
         tr = lib().mary_mla_tile_rows()
         for s, n in enumerate(meta.q_lens_host.tolist()):
             rows = n * hq
-            for b in range(0, rows, tr):
+            for b in range(0, rows if group is None or (group == "prefill") == (n > DECODE_GROUP_ROWS) else 0, tr):
                 seqs.append(s)
                 r0.append(start * hq + b)
             start += n
@@ -650,15 +657,17 @@ def _row_tiles(meta, hq: int):
     return cache[key]
 
 
-def mla_attention(q, cache, meta, scale, nsplit: int | None = None):
-    """``q[T, Hq, 576]`` bf16, ``cache[pages, page (16 or 32), 576]`` bf16 (finite everywhere) -> ``[T, Hq, 512]``.  With
-    32-token pages the kernel fetches a whole 32-key stage with one TMA operation."""
+def mla_attention(q, cache, meta, scale, nsplit: int | None = None, window: int = 0, split_p: bool = False, group: str | None = None):
+    """``q[T, Hq, 576]`` bf16, ``cache[pages, page (16, 32 or 64), 576]`` bf16 (finite everywhere) -> ``[T, Hq, 512]``.  With 32- and
+    64-token pages the kernel fetches a whole 32-key stage with one TMA operation.  ``split_p``: softmax weights with 16 significant bits;
+    ``group``: see ``_q_blocks`` (rows of the other sequences are not written)."""
     T, Hq, DK = q.shape
     ps = meta.page_size
-    assert DK == 576 and ps in (16, 32) and cache.shape[1] == ps and cache.shape[-1] == 576
-    blk_seq, blk_r0, NB = _row_tiles(meta, Hq)
+    assert DK == 576 and ps in (16, 32, 64) and cache.shape[1] == ps and cache.shape[-1] == 576
+    blk_seq, blk_r0, NB = _row_tiles(meta, Hq, group)
     if nsplit is None:
-        nsplit = max(1, min(8, 148 // max(1, NB), meta.max_kv_len // 512))
+        span = meta.max_kv_len if window <= 0 else min(meta.max_kv_len, window + 64)
+        nsplit = max(1, min(8, 148 // max(1, NB), span // (512 if window <= 0 else 256)))
     out = _empty(T, Hq, 512, dtype=torch.bfloat16, device=q.device)
     scratch = None
     if nsplit > 1:
@@ -666,7 +675,7 @@ def mla_attention(q, cache, meta, scale, nsplit: int | None = None):
     c = cache.view(cache.shape[0], ps, 576)
     check(lib().mary_mla_attention(_p(q.contiguous()), _p(c), _p(out), _p(meta.page_table), _p(meta.kv_len), _p(meta.q_start),
                                    _p(blk_seq), _p(blk_r0), NB, T * Hq, c.shape[0], meta.page_table.shape[1], c.stride(1),
-                                   c.stride(0), Hq, nsplit, scale, _p(scratch), ps, _stream()), "mla_attention")
+                                   c.stride(0), Hq, nsplit, scale, _p(scratch), ps, window, int(split_p), _stream()), "mla_attention")
     return out
 
 

@@ -35,7 +35,11 @@ declare("mary_dyt_add", "pl" + "ppp" + "p" + "ppp" + "piiis")
 declare("mary_row_norm_append", "ppp" + "liii" + "pppppp" + "filis")
 declare("mary_latent_prep", "pp" + "liii" + "ppp" + "f" + "pppp" + "filis")
 declare("mary_rotate_heads", "pppfp" + "iiiiii" + "is")
+declare("mary_fill_shared_part", "pliplii" + "iis")
 declare("mary_ss_prep", "pl" + "pppppp" + "ppp" + "pppppp" + "iiiiiii" + "is")
+declare("mary_ss_conv_decay", "pl" + "pppppp" + "ppp" + "pppp" + "iiiiiis")
+declare("mary_ssd_chunk", "ppppppp" + "ppp" + "iiiiiis")
+declare("mary_ssd_chunk_supported", "ii")
 declare("mary_head_decay_scan", "pppppppp" + "p" + "ppp" + "illl" + "iiiis")
 declare("mary_gated_part_norm", "pplppl" + "iiifis")
 declare("mary_ss_step", "plppp" + "pppp" + "pp" + "ipl" + "ppp" + "ppp" + "iiiiiifis")
@@ -116,10 +120,6 @@ def qk_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vca
 DECODE_ROWS = K.DECODE_GROUP_ROWS         # sequences with at most this many query tokens take the decode kernel, the others the prefill kernel
 
 
-def _gate(gate):
-    return (None, 0) if gate is None else _rows(gate)
-
-
 def attention_general(q, kcache, vcache, meta, scale, out, group=None, nsplit=None, window: int = 0, bias=None, gate=None):
     """Any head widths, group size and storage type; ``group`` restricts the call to ``"prefill"`` or ``"decode"`` sequences.  ``bias``,
     ``gate``: see ``ops.attention_exact``."""
@@ -139,7 +139,7 @@ def attention_general(q, kcache, vcache, meta, scale, out, group=None, nsplit=No
         scratch = _empty(lib().mary_attention_general_scratch_floats(NB, Hq, Hkv, nsplit, DV), dtype=torch.float32, device=q.device)
     check(lib().mary_attention_general(_p(q), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len), _p(meta.q_start), _p(blk_seq),
                                        _p(blk_q0), NB, meta.page_table.shape[1], meta.page_size, kcache.stride(1), kcache.stride(0), vcache.stride(1),
-                                       vcache.stride(0), out.stride(0), Hq, Hkv, DK, DV, rq, nsplit, window, scale, _p(bias), *_gate(gate), _p(scratch),
+                                       vcache.stride(0), out.stride(0), Hq, Hkv, DK, DV, rq, nsplit, window, scale, _p(bias), *K._gate(gate), _p(scratch),
                                        _f32(q), _stream()), "attention_general")
     return out
 
@@ -156,20 +156,21 @@ def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, b
     if out is None:
         out = _empty(T, Hq * DV, dtype=q.dtype, device=q.device)
     assert out.stride(1) == 1
-    bf16 = q.dtype == torch.bfloat16 and DK == DV and vcache.is_contiguous() and bias is None and gate is None
+    bf16 = q.dtype == torch.bfloat16 and DK == DV and vcache.is_contiguous()
     kw = dict(window=window, bias=bias, gate=gate)
-    fast_prefill = bf16 and DK in (64, 128, 256) and meta.page_size in (16, 64) and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
+    aligned = all(t is None or (t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0) for t in (out, gate))
+    fast_prefill = bf16 and DK in (64, 128, 256) and meta.page_size in (16, 64) and aligned
     fast_decode = bf16 and DK in (64, 128, 256) and Hq // Hkv <= (4 if DK == 256 else 8)
     if not (fast_prefill or fast_decode):
         return attention_general(q, kcache, vcache, meta, scale, out, **kw)
     if meta.max_q_len > DECODE_ROWS:
         if fast_prefill:
-            K.attention_prefill(q, kcache, vcache, meta, scale, window, out=out, split_p=True, group="prefill")
+            K.attention_prefill(q, kcache, vcache, meta, scale, out=out, split_p=True, group="prefill", **kw)
         else:
             attention_general(q, kcache, vcache, meta, scale, out, "prefill", **kw)
     if K._q_blocks(meta, 1, "decode")[2]:
         if fast_decode:
-            K._paged_attention_decode(q, kcache, vcache, meta, scale, window, 0.0, None, out=out, group="decode")
+            K._paged_attention_decode(q, kcache, vcache, meta, scale, window, 0.0, None, out=out, group="decode", bias=bias, gate=gate)
         else:
             attention_general(q, kcache, vcache, meta, scale, out, "decode", **kw)
     return out
@@ -328,15 +329,85 @@ def head_matmul(x, w, out):
     return out
 
 
+EXPAND_ROWS = DECODE_ROWS        # sequences with more query tokens than this attend over expanded keys and values
+
+
+def _visible_pages(meta, window: int):
+    """The pages that the sequences with a prompt portion can see, as a cache of their own: ``(pick, meta2)`` where ``cache[pick]`` holds them
+    and ``meta2`` addresses them, positions shifted by whole pages (only differences of positions enter the masks).  Memoised: every layer
+    with the same window asks for the same."""
+    import dataclasses
+    memo = meta.__dict__.setdefault("_cache", {})
+    key = ("visible", window)
+    if key not in memo:
+        ps = meta.page_size
+        shift, spans = [0] * meta.num_seqs, []
+        for s, (n, kv) in enumerate(zip(meta.q_lens_host.tolist(), meta.kv_lens_host.tolist())):
+            lo = max(0, kv - n - window + 1) // ps
+            spans.append((lo, (kv + ps - 1) // ps) if n > EXPAND_ROWS else (0, 0))
+            shift[s] = spans[-1][0] * ps
+        dev = meta.page_table.device
+        width = max(b - a for a, b in spans)
+        table, at, picks = torch.zeros(meta.num_seqs, width, dtype=torch.int32), 0, []
+        for s, (a, b) in enumerate(spans):
+            table[s, :b - a] = torch.arange(at, at + b - a, dtype=torch.int32)
+            at += b - a
+            picks.append(meta.page_table[s, a:b])
+        host = meta.kv_lens_host - torch.tensor(shift).numpy().astype(meta.kv_lens_host.dtype)
+        memo[key] = (torch.cat(picks).long(), dataclasses.replace(meta, page_table=table.to(dev, non_blocking=True), kv_lens_host=host,
+                                                                  kv_len=torch.from_numpy(host).to(dev, non_blocking=True)))
+    return memo[key]
+
+
+def expand_latent(rows, m):
+    """Keys ``[N, H, dim + rot]`` and values ``[N, H, dv]`` of cache rows ``[N, rank + rot]``, written straight into their final layout."""
+    N, H, w = rows.shape[0], m.heads, m.dim + m.rot
+    k = _empty(N, H, w, dtype=rows.dtype, device=rows.device)
+    with K.static_weights:
+        K.gemm_batched(rows, m.w_k, k, N, m.dim, m.rank, rows.stride(0), m.rank, H * w, H, 0, m.dim * m.rank, w)
+        v = K.gemm(rows[:, :m.rank], m.w_v)
+    check(lib().mary_fill_shared_part(_p(rows), rows.stride(0), m.rank, _p(k), N, H, m.dim, m.rot, _f32(rows), _stream()), "fill_shared_part")
+    return k, v.view(N, H, m.dv)
+
+
+def _latent_prompts(q, cache, meta, m, out):
+    """Sequences with a prompt portion: keys and values expanded from the visible rows, then ordinary attention, a third of the arithmetic of
+    attending in latent space."""
+    T, H, ps = q.shape[0], m.heads, meta.page_size
+    pick, meta2 = _visible_pages(meta, m.window)
+    rows = cache[pick].view(-1, m.rank + m.rot)
+    k, v = expand_latent(rows, m)
+    q = rotate_heads(q, q, m.dim, m.rot, m.freq, m.rot_gain, meta)
+    K.attention_prefill(q, k.view(-1, ps, H, m.dim + m.rot), v.view(-1, ps, H, m.dv), meta2, m.scale, m.window, out=out, split_p=True, group="prefill")
+
+
 def latent_attention(q, cache, meta, m):
     T, H = q.shape[0], m.heads
     q = q.view(T, H, m.dim + m.rot)
+    out = _empty(T, H * m.dv, dtype=q.dtype, device=q.device)
+    bf16 = q.dtype == torch.bfloat16
+    group = None
+    if (bf16 and meta.max_q_len > EXPAND_ROWS and meta.page_size == 64 and m.rank % 8 == 0 and m.rot % 8 == 0
+            and lib().mary_attention_prefill_supported(m.dim + m.rot, m.dv)):
+        decoded = bool((meta.q_lens_host <= EXPAND_ROWS).any())
+        _latent_prompts(q.clone() if decoded else q, cache, meta, m, out)
+        if not decoded:
+            return out
+        group = "decode"
+    prompts = out
     qf = _empty(T, H, m.rank + m.rot, dtype=q.dtype, device=q.device)
     head_matmul(q[..., :m.dim], m.w_k_t, qf[..., :m.rank])
     rotate_heads(q, qf, m.rank, m.rot, m.freq, m.rot_gain, meta)
-    lat = attention_exact(qf, cache, cache[..., :m.rank], meta, m.scale, window=m.window)
-    out = _empty(T, H * m.dv, dtype=q.dtype, device=q.device)
+    if bf16 and (m.rank, m.rot) == (512, 64) and meta.page_size in (16, 32, 64):
+        lat = K.mla_attention(qf, cache.view(cache.shape[0], meta.page_size, 576), meta, m.scale, window=m.window, split_p=True, group=group)
+    else:
+        lat = _empty(T, H * m.rank, dtype=q.dtype, device=q.device)
+        attention_general(qf, cache, cache[..., :m.rank], meta, m.scale, lat, group, window=m.window)
+    out = _empty(T, H * m.dv, dtype=q.dtype, device=q.device) if group else prompts
     head_matmul(lat.view(T, H, m.rank), m.w_v.view(H, m.dv, m.rank), out.view(T, H, m.dv))
+    if group:                                  # rows of the prompt portions keep what the expanded attention gave
+        rows = torch.from_numpy(meta.q_lens_host > EXPAND_ROWS).to(q.device).repeat_interleave(torch.from_numpy(meta.q_lens_host).to(q.device).long())
+        out = torch.where(rows[:, None], prompts, out)
     return out
 
 
@@ -373,6 +444,28 @@ def head_decay_scan(x, b, c, dt, decay, pairs, skip, state, meta, G, H, N, P):
     return out
 
 
+def ssd_chunk_prep(xbc, taps_w, taps_b, ring, dt_in, dt_bias, a_log, meta, H):
+    """bf16 models: convolved rows ``[T, C]`` and, per head and token, step size and summed log2 decay of the chunk as two floats."""
+    T, C = xbc.shape
+    rows = _empty(T, C, dtype=xbc.dtype, device=xbc.device)
+    dt, hi, lo = (_empty(H, T, dtype=torch.float32, device=xbc.device) for _ in range(3))
+    px, ldx = _rows(xbc)
+    assert dt_in.stride(0) == ldx
+    check(lib().mary_ss_conv_decay(px, ldx, _p(taps_w), _p(taps_b), _p(ring), _p(dt_in), _p(dt_bias), _p(a_log), _p(meta.q_start), _p(meta.kv_len),
+                                   _p(meta.state_slots), _p(rows), _p(dt), _p(hi), _p(lo), meta.num_seqs, meta.max_q_len, T, H, C, taps_w.shape[1],
+                                   _stream()), "ss_conv_decay")
+    return rows, dt, hi, lo
+
+
+def ssd_chunk(rows, dt, hi, lo, skip, state, meta, G, H, N, P):
+    """The recurrence on the tensor cores, 64 tokens at a time: f32 ``[T, H * P]``."""
+    T = rows.shape[0]
+    y = _empty(T, H * P, dtype=torch.float32, device=rows.device)
+    check(lib().mary_ssd_chunk(_p(rows), _p(dt), _p(hi), _p(lo), _p(skip), _p(y), _p(state), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots),
+                               meta.num_seqs, T, G, H, N, P, _stream()), "ssd_chunk")
+    return y
+
+
 def gated_part_norm(y, z, gain, parts, eps, out):
     (pz, ldz), (po, ldo) = _rows(z), _rows(out)
     check(lib().mary_gated_part_norm(_p(y), pz, ldz, _p(gain), po, ldo, y.shape[0], y.shape[1], parts, eps, _f32(z), _stream()), "gated_part_norm")
@@ -391,6 +484,11 @@ def state_space(xbc, taps_w, taps_b, dt_in, dt_bias, a_log, skip, z, gain, norm_
                                  _p(state), _p(row), _p(cnt), _p(meta.q_start), _p(meta.positions), _p(meta.state_slots), S, G, H, N, P, taps, eps,
                                  _f32(xbc), _stream()), "ss_step")
         return out
+    if (xbc.dtype == torch.bfloat16 and lib().mary_ssd_chunk_supported(N, P) and xbc.stride(0) % 4 == 0
+            and all(t.data_ptr() % 8 == 0 for t in (xbc, taps_w, ring))):
+        pre = ssd_chunk_prep(xbc, taps_w, taps_b, ring, dt_in, dt_bias, a_log, meta, H)
+        conv_history(xbc, ring, meta, taps, taps_w.shape[0])
+        return gated_part_norm(ssd_chunk(*pre, skip, state, meta, G, H, N, P), z, gain, norm_parts, eps, out)
     x, b, c, dt, decay, pairs = ss_prep(xbc, taps_w, taps_b, ring, dt_in, dt_bias, a_log, meta, G, H, N, P)
     conv_history(xbc, ring, meta, taps, taps_w.shape[0])
     return gated_part_norm(head_decay_scan(x, b, c, dt, decay, pairs, skip, state, meta, G, H, N, P), z, gain, norm_parts, eps, out)

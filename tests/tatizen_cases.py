@@ -1,14 +1,13 @@
-"""Small Tatizen models for the tests: configurations, random weights (bf16-representable, so every storage type holds them exactly), a
-checkpoint folder writer, and comparison helpers."""
+"""Small Tatizen models for the tests: configurations, random weights (bf16-representable, so every storage type holds them exactly)
+and the model built from them."""
 from __future__ import annotations
 
-import json
-
-import numpy as np
 import torch
 
 from mary_b200.models.tatizen.config import TatizenConfig
 from mary_b200.models.tatizen.model import TatizenModel, decay_ranks, load_into
+
+from paged_cases import DictLoader, bf16
 
 
 def parallel(left=(4, 2, 32, 48), right=(3, 24, 40), scale=0.2, tau=4.0, ls=0.6, rs=-0.7, ff=88):
@@ -37,10 +36,6 @@ CONFIGS = {
     "group": config([parallel((20, 1, 16, 24), (2, 8, 64), ls=0.0, ff=72), parallel((9, 1, 64, 64), (1, 256, 16), rs=0.0, ff=72)], vocab=90, width=64),
     "recurrent": config([delta(ff=None), delta(2, 2, 32, 32, 4, 64)], vocab=64, width=40),
 }
-
-
-def bf16(x):
-    return x.to(torch.bfloat16).float()
 
 
 def random_weights(cfg: dict, seed: int = 0, ranks=(16, 5)) -> dict:
@@ -77,35 +72,9 @@ def random_weights(cfg: dict, seed: int = 0, ranks=(16, 5)) -> dict:
     return {k: bf16(v) for k, v in w.items()}
 
 
-class DictLoader:
-    def __init__(self, w):
-        self.w = w
-
-    def load_tensor(self, name, dtype=None, device=None):
-        t = self.w[name]
-        return t if dtype is None else t.to(dtype)
-
-    def shape(self, name):
-        return tuple(self.w[name].shape)
-
-
 def build(cfg: dict, w: dict, device="cpu", dtype=torch.float32) -> TatizenModel:
     c = TatizenConfig.from_json(cfg)
     loader = DictLoader(w)
     m = TatizenModel(c, decay_ranks(c, loader.shape), dtype=dtype, device=device)
     load_into(m, loader)
     return m
-
-
-def write_folder(path, cfg: dict, w: dict) -> None:
-    from mary_b200.format.safetensors import save_file
-    bits = {k: v.to(torch.bfloat16).view(torch.int16).numpy().view(np.uint16) for k, v in w.items()}
-    save_file(bits, str(path / "model.safetensors"), bf16=set(bits))
-    (path / "config.json").write_text(json.dumps(cfg))
-
-
-def error(got, want) -> float:
-    """Largest rms difference of a row relative to the rms of all wanted values."""
-    got, want = torch.as_tensor(got).double().cpu(), want.double()
-    d = (got - want).flatten(1) if got.dim() > 1 else (got - want)[None]
-    return float(d.pow(2).mean(-1).sqrt().max() / want.pow(2).mean().sqrt())

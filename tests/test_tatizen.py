@@ -2,7 +2,6 @@
 bf16): each mechanism alone, whole prompts, token-by-token decoding, portions, mixed batches, reuse of pages and state slots."""
 import random
 
-import numpy as np
 import pytest
 import torch
 
@@ -12,7 +11,8 @@ from mary_b200.oracle import tatizen as oracle
 from mary_b200.runtime.batch import BatchMeta
 from mary_b200.runtime.kv_cache import PagedKVCache
 
-from tatizen_cases import CONFIGS, bf16, build, config, delta, error, parallel, random_weights
+from paged_cases import Paged, bf16, error, prompt, schedule
+from tatizen_cases import CONFIGS, build, config, delta, parallel, random_weights
 
 FAMILY = next(f for f in FAMILIES if f.name == "tatizen")
 TARGETS = [pytest.param(("cpu", torch.float32), id="cpu"), pytest.param(("cuda", torch.float32), id="cuda-f32", marks=pytest.mark.gpu),
@@ -26,47 +26,6 @@ def target(request):
 
 def tol(target, f32=2e-5, b16=1.5e-2):
     return f32 if target[1] == torch.float32 else b16
-
-
-class Paged:
-    """Sequences over one shuffled page pool and shuffled state slots, stepped by hand."""
-
-    def __init__(self, page=16, pages=96, slots=6, device="cpu", seed=0):
-        self.rng = random.Random(seed)
-        self.page, self.device = page, device
-        self.free = list(range(pages))
-        self.rng.shuffle(self.free)
-        self.slots = list(range(slots))
-        self.rng.shuffle(self.slots)
-        self.rows, self.len, self.slot = {}, {}, {}
-
-    def step(self, counts: dict):
-        for s, n in counts.items():
-            if s not in self.rows:
-                self.rows[s], self.len[s], self.slot[s] = [], 0, self.slots.pop()
-            self.len[s] += n
-            while len(self.rows[s]) * self.page < self.len[s]:
-                self.rows[s].append(self.free.pop())
-        width = max(len(self.rows[s]) for s in counts)
-        table = np.array([self.rows[s] + [-1] * (width - len(self.rows[s])) for s in counts], dtype=np.int32)
-        return BatchMeta.build(list(counts.values()), [self.len[s] for s in counts], table, self.page, self.device,
-                               [self.slot[s] for s in counts])
-
-    def drop(self, s):
-        self.free.extend(self.rows.pop(s))
-        self.slots.append(self.slot.pop(s))
-        del self.len[s]
-
-
-def schedule(lengths: dict, rng, sizes=(1, 1, 2, 3, 5, 17, 40, 70)):
-    """Steps of unequal portions: every step takes a random subset of the unfinished sequences."""
-    at = {s: 0 for s in lengths}
-    while any(at[s] < n for s, n in lengths.items()):
-        live = [s for s in lengths if at[s] < lengths[s]]
-        step = {s: min(rng.choice(sizes), lengths[s] - at[s]) for s in live if rng.random() < 0.7} or {live[0]: 1}
-        yield {s: (at[s], n) for s, n in step.items()}
-        for s, n in step.items():
-            at[s] += n
 
 
 # --------------------------------------------------------------------------- mechanisms alone
@@ -286,10 +245,6 @@ def engine(name, target, tokens=1024, seqs=4, seed=0, **kw):
     w = random_weights(cfg, seed)
     m = build(cfg, w, *target)
     return cfg, w, make_engine(m, FAMILY, tokens, seqs, target[0], **kw)
-
-
-def prompt(cfg, n, seed=0):
-    return np.random.default_rng(seed).integers(0, cfg["vocab"], n).tolist()
 
 
 LOGIT_TOL = dict(f32=1e-4, b16=8e-2)

@@ -15,14 +15,11 @@ from mary_b200.models.tatizen.config import TatizenConfig
 from mary_b200.oracle import tatizen as oracle
 from mary_b200.runtime.engine import Engine
 from mary_b200.runtime.kv_cache import OutOfPages, PageAllocator, PagedKVCache
-from tatizen_cases import CONFIGS, build, config, delta, error, parallel, random_weights, write_folder
+from paged_cases import TRACE, error, prompt, trace_case, write_folder
+from tatizen_cases import CONFIGS, build, config, delta, parallel, random_weights
 
 ROOT = Path(__file__).resolve().parents[1]
 DEVICES = [pytest.param("cpu", id="cpu"), pytest.param("cuda", id="cuda", marks=pytest.mark.gpu)]
-
-
-def prompt(cfg, n, seed=0):
-    return np.random.default_rng(seed).integers(0, cfg["vocab"], n).tolist()
 
 
 # --------------------------------------------------------------------------- configuration and registry
@@ -203,35 +200,6 @@ def test_text_gen(tmp_path, capsys, device):
     assert capsys.readouterr().out == first and len(first.splitlines()) == 3
 
 
-TRACE = [{"step": 0, "entries": [{"id": "a", "tokens": 50, "want": [0, 49]}], "end": []},
-         {"step": 1, "entries": [{"id": "b", "tokens": 30, "want": []}], "end": []},
-         {"step": 2, "entries": [{"id": "a", "tokens": 1, "want": [0]}, {"id": "c", "tokens": 2, "want": [1]}], "end": ["c"]},
-         {"step": 7, "entries": [{"id": "b", "tokens": 25, "want": [3, 24]}, {"id": "d", "tokens": 64, "want": [63]}], "end": ["b"]},
-         {"step": 8, "entries": [{"id": "d", "tokens": 1, "want": [0]}, {"id": "a", "tokens": 20, "want": [19]}, {"id": "c", "tokens": 9, "want": [8]}],
-          "end": ["a", "c", "d"]}]
-
-
-def trace_case(cfg, w):
-    """The trace with tokens filled in and the logits it asks for (an id that comes again after its end is a new request)."""
-    rng, hist, lines, want = np.random.default_rng(3), {}, [], {}
-    for s in TRACE:
-        entries, rows = [], []
-        for e in s["entries"]:
-            t = rng.integers(0, cfg["vocab"], e["tokens"]).tolist()
-            entries.append({"id": e["id"], "tokens": t, "want": e["want"]})
-            h = hist.setdefault(e["id"], [])
-            at = len(h)
-            h += t
-            if e["want"]:
-                rows.append(oracle.run(cfg, w, h)[0][[at + k for k in e["want"]]])
-        for i in s["end"]:
-            del hist[i]
-        lines.append(json.dumps({"step": s["step"], "entries": entries, "end": s["end"]}))
-        if rows:
-            want[s["step"]] = torch.cat(rows)
-    return lines, want
-
-
 @pytest.mark.parametrize("device", DEVICES)
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_trace_run(tmp_path, monkeypatch, capsys, device, dtype):
@@ -239,7 +207,7 @@ def test_trace_run(tmp_path, monkeypatch, capsys, device, dtype):
     cfg = CONFIGS["mixed"]
     w = random_weights(cfg, 2)
     write_folder(tmp_path, cfg, w)
-    lines, want = trace_case(cfg, w)
+    lines, want = trace_case(cfg, w, oracle.run)
     out = tmp_path / "out"
     out.mkdir()
     monkeypatch.setattr(sys, "stdin", io.StringIO("\n".join(lines) + "\n"))
