@@ -104,12 +104,12 @@ def reference_arm(args):
                       "not in the tree and no cargo/rustc exists in this image; pip cannot install it (no setup.py/pyproject.toml)"}))
 
 
-def tatizen_bench(args, warmup):
-    from mary_b200.models.tatizen import bench as tb
+def hybrid_bench(args, warmup):
+    from mary_b200.models import bench_hybrid as tb
     cases = [c for c in tb.CASES if args.batch in (None, c[1])]
     sampler = ClockSampler(0)
     sampler.start()
-    line = tb.run(list(tb.SIZES), cases, args.steps, warmup, trace=args.trace)
+    line = tb.run(args.model, list(tb.SIZES), cases, args.steps, warmup, trace=args.trace)
     line.update(n_gpus=1, clocks=sampler.stop(), higher_is_better=True)
     print(json.dumps(line))
 
@@ -125,8 +125,8 @@ def main():
                          "of this package's kernels); both: the product arm, then the library arm on the same GPUs, and vs_baseline = ours / library")
     ap.add_argument("--library-steps", type=int, default=4, help="timed steps of the library arm (after 2 warm-up steps)")
     ap.add_argument("--library-limit", type=float, default=240.0, help="seconds after which a stalled library arm is abandoned")
-    ap.add_argument("--model", default="k3", choices=["k3", "inkling", "gemma12b", "tiny", "tatizen"],
-                    help="k3 is the headline; the others time the remaining workload configurations with the same harness; tatizen: prefill and "
+    ap.add_argument("--model", default="k3", choices=["k3", "inkling", "gemma12b", "tiny", "tatizen", "rokarax"],
+                    help="k3 is the headline; the others time the remaining workload configurations with the same harness; tatizen, rokarax: prefill and "
                          "decode of that decoder beside the dense decoder of equal size, at two sizes, on one GPU")
     ap.add_argument("--ep", default="auto", choices=["auto", "replicated", "a2a"],
                     help="expert parallel layout for N > 1: replicated tokens + tensor-parallel attention + reduction, or home-rank "
@@ -158,8 +158,8 @@ def main():
     if args.impl == "reference":
         return reference_arm(args)
     W = max(args.warmup, 3)
-    if args.model == "tatizen":
-        return tatizen_bench(args, W)
+    if args.model in ("tatizen", "rokarax"):
+        return hybrid_bench(args, W)
     # a benchmark that stops making progress must end by itself: dump the stacks and exit after the limit
     import faulthandler
     from mary_b200.utils import flags

@@ -1,4 +1,5 @@
-"""Throughput of the Tatizen decoder beside the dense decoder of equal size (the Mistral shell), prefill and decode, on one GPU.
+"""Throughput of the hybrid decoders (Tatizen, Rokarax) beside the dense decoder of equal size (the Mistral shell), prefill and decode, on
+one GPU.
 
 Random weights of the named sizes; every step streams weights and caches far larger than L2.  Prefill: whole prompts through
 ``model.greedy`` (logits of the last rows).  Decode: the fixed-batch decoder replaying one CUDA graph per step over caches and states
@@ -8,27 +9,37 @@ from __future__ import annotations
 import numpy as np
 import torch
 
-from ...runtime.batch import BatchMeta
-from ...runtime.kv_cache import PagedKVCache
-from ...runtime.spec_decode import SpecDecoder
-from .config import AttentionSpec, DecayedLinearSpec, DeltaSpec, LayerSpec, ParallelSpec, TatizenConfig
+from ..runtime.batch import BatchMeta
+from ..runtime.kv_cache import PagedKVCache
+from ..runtime.spec_decode import SpecDecoder
 
 PAGE = 64
-# width, feed-forward, attention (heads, kv heads), linear heads, delta (value heads, q/k heads); head widths 128
+# width, feed-forward, attention (heads, kv heads), linear heads, delta (value heads, q/k heads); head widths 128.  Rokarax: the same attention
+# heads with windows of 1024 positions, state space layers of twice the width in heads of 64 with 128 state rows, latents of 512 + 64
 SIZES = {"2k": (2048, 8192, (16, 4), 8, (16, 8)), "4k": (4096, 12288, (32, 8), 16, (32, 16))}
-LAYERS, VOCAB = 8, 32768
+LAYERS, VOCAB, WINDOW = 8, 32768, 1024
 CASES = [("prefill", 1, 4096), ("prefill", 8, 512), ("decode", 1, 2048), ("decode", 32, 2048), ("decode", 128, 2048)]
 
 
-def tatizen_config(size: str) -> TatizenConfig:
+def tatizen_config(size: str):
+    from .tatizen.config import AttentionSpec, DecayedLinearSpec, DeltaSpec, LayerSpec, ParallelSpec, TatizenConfig
     W, F, (H, G), L, (DH, DK) = SIZES[size]
     par = LayerSpec(ParallelSpec(AttentionSpec(H, G, 128, 128, 128 ** -0.5), DecayedLinearSpec(L, 128, 128, 8.0), 0.9, 0.6), F)
     dlt = LayerSpec(DeltaSpec(DH, DK, 128, 128, 4), F)
     return TatizenConfig(VOCAB, W, 1e-6, [par, dlt] * (LAYERS // 2), name=f"tatizen-{size}")
 
 
+def rokarax_config(size: str):
+    from .rokarax.config import AttentionSpec, LatentSpec, LayerSpec, RokaraxConfig, RotationSpec, StateSpaceSpec
+    W, F, (H, G), _, _ = SIZES[size]
+    att = lambda src: LayerSpec(AttentionSpec(H, G, 128, 128, 128 ** -0.5, WINDOW, 800.0, src), F)  # noqa: E731
+    ssm = LayerSpec(StateSpaceSpec(2 * W // 64, 64, 128, 1, 4, 8), F)
+    lat = LayerSpec(LatentSpec(H, 128, 64, 128, 768, 512, 192 ** -0.5, WINDOW, RotationSpec(64, 1e4, 4.0, 4096.0, 32.0, 1.0)), F)
+    return RokaraxConfig(VOCAB, W, 1e-6, W ** 0.5, [att(None), ssm, lat, ssm, att(0), ssm, lat, ssm], name=f"rokarax-{size}")
+
+
 def dense_config(size: str):
-    from ..mistral.model import MistralConfig
+    from .mistral.model import MistralConfig
     W, F, (H, G), _, _ = SIZES[size]
     return MistralConfig(LAYERS, W, F, H, G, 128, VOCAB, qk_norm=True, name=f"dense-{size}")
 
@@ -36,10 +47,13 @@ def dense_config(size: str):
 def make_model(kind: str, size: str, dev):
     kw = dict(dtype=torch.bfloat16, device=dev)
     if kind == "tatizen":
-        from .model import TatizenModel, init_random_
+        from .tatizen.model import TatizenModel, init_random_
         m = TatizenModel(tatizen_config(size), **kw)
+    elif kind == "rokarax":
+        from .rokarax.model import RokaraxModel, init_random_
+        m = RokaraxModel(rokarax_config(size), **kw)
     else:
-        from ..mistral.model import MistralModel, init_random_
+        from .mistral.model import MistralModel, init_random_
         m = MistralModel(dense_config(size), **kw)
         m.trunk = m.hidden
     init_random_(m, seed=1)
@@ -88,12 +102,12 @@ def decode_step(m, cache, batch: int, ctx: int, tokens: int, dev):
     return dec.step
 
 
-def run(sizes, cases, steps: int, warmup: int, trace: bool = False) -> dict:
-    from ...ops import cuda as K
+def run(design: str, sizes, cases, steps: int, warmup: int, trace: bool = False) -> dict:
+    from ..ops import cuda as K
     dev = torch.device("cuda", 0)
     out = []
     for size in sizes:
-        for kind in ("tatizen", "dense"):
+        for kind in (design, "dense"):
             m = make_model(kind, size, dev)
             for what, batch, n in cases:
                 # dependent launch: a decode step is a chain of short kernels and gains from it; a prefill step loses (the waiting blocks of
@@ -103,7 +117,7 @@ def run(sizes, cases, steps: int, warmup: int, trace: bool = False) -> dict:
                 tokens = (tokens + PAGE - 1) // PAGE * PAGE
                 cache = make_cache(m, batch, tokens, dev)
                 if trace:
-                    from ...utils.trace import Tracer
+                    from ..utils.trace import Tracer
                     step = prefill_step(m, cache, batch, n, dev) if what == "prefill" else None
                     if step is None:
                         dec = SpecDecoder(m, cache, batch, max_len=tokens, device=dev, use_graph=False)
@@ -126,5 +140,5 @@ def run(sizes, cases, steps: int, warmup: int, trace: bool = False) -> dict:
     status = K.last_status()
     if status:
         raise RuntimeError(f"kernel status {status}")
-    return {"metric": "tokens/s, Tatizen beside the dense decoder of equal size", "unit": "tokens/s", "layers": LAYERS, "dtype": "bf16",
+    return {"metric": f"tokens/s, {design} beside the dense decoder of equal size", "unit": "tokens/s", "layers": LAYERS, "dtype": "bf16",
             "data": "synthetic", "steps": steps, "warmup": max(warmup, 3), "cases": out}

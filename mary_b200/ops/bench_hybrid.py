@@ -1,5 +1,5 @@
 """Micro-benchmarks of the kernels of decoders with recurrent layers, beside the like kernels of the dense decoders
-(``python -m mary_b200.ops.bench_kernels hybrid``).  Fractions: bytes against the measured copy bandwidth, tensor-core products against
+(``python -m mary_b200.ops.bench_kernels hybrid`` and ``rokarax``).  Fractions: bytes against the measured copy bandwidth, tensor-core products against
 the measured cuBLAS rate, the recurrences (32-bit multiply-adds on the CUDA cores) against the nominal 128 multiply-adds per SM and clock."""
 from __future__ import annotations
 
@@ -15,20 +15,30 @@ def _meta(B, q, ctx, page=64):
     return BatchMeta.build([q] * B, [ctx] * B, np.arange(B * n, dtype=np.int32).reshape(B, n), page, "cuda", np.arange(B, dtype=np.int32))
 
 
+class _Table:
+    """Times calls and prints them against the measured peaks."""
+
+    def __init__(self):
+        from .bench_kernels import peaks
+        self.hbm, self.tf, self.tag = peaks()
+        self.rows: list[dict] = []
+
+    def __call__(self, name, case, fn, flops=0.0, peak=None, nbytes=0.0, like=None):
+        from .bench_kernels import time_op
+        us = time_op(fn) * 1e3
+        frac = max(flops / us / 1e6 / peak if peak else 0.0, nbytes / us / 1e3 / self.hbm)
+        self.rows.append(dict(kernel=name, case=case, us=round(us, 1), tflops=round(flops / us / 1e6, 1), gbs=round(nbytes / us / 1e3), frac=round(frac, 3),
+                              like=like))
+        print(f"{name:<30}{case:<18}{us:>9.1f} us {flops / us / 1e6:>8.1f} TFLOP/s {nbytes / us / 1e3:>7.0f} GB/s  {frac:.3f} {self.tag}"
+              + (f"  (like: {like})" if like else ""))
+
+
 def run(width: int = 4096, heads: int = 32, kv_heads: int = 8, l_heads: int = 16, d_heads: int = 32, d_kv: int = 16, D: int = 128) -> list[dict]:
     from . import cuda as K
     from . import cuda_hybrid as H
-    from .bench_kernels import peaks, time_op
-    hbm, tf, tag = peaks()
+    add = _Table()
+    tf, rows = add.tf, add.rows
     bf = dict(dtype=torch.bfloat16, device="cuda")
-    rows: list[dict] = []
-
-    def add(name, case, fn, flops=0.0, peak=None, nbytes=0.0, like=None):
-        us = time_op(fn) * 1e3
-        frac = max(flops / us / 1e6 / peak if peak else 0.0, nbytes / us / 1e3 / hbm)
-        rows.append(dict(kernel=name, case=case, us=round(us, 1), tflops=round(flops / us / 1e6, 1), gbs=round(nbytes / us / 1e3), frac=round(frac, 3),
-                         like=like))
-        print(f"{name:<28}{case:<18}{us:>9.1f} us {flops / us / 1e6:>8.1f} TFLOP/s {nbytes / us / 1e3:>7.0f} GB/s  {frac:.3f} {tag}" + (f"  (like: {like})" if like else ""))
 
     for B, q in ((1, 4096), (8, 512)):
         case, T = f"{B} x {q} tokens", B * q
@@ -104,3 +114,105 @@ def run(width: int = 4096, heads: int = 32, kv_heads: int = 8, l_heads: int = 16
             add(name, case, fn, 2.0 * T * N * Kd, tf, 2.0 * (N * Kd + T * Kd + T * N))
     assert K.last_status() == 0
     return rows
+
+
+def run_rokarax(width: int = 4096, heads: int = 32, kv_heads: int = 8, window: int = 1024) -> list[dict]:
+    """The kernels of the Rokarax decoder: attention with a distance bias, a window and a gate beside the dense decoder's, latent attention
+    beside the expanded and the absorbed form without a window, the state space layer, the row kernels."""
+    from types import SimpleNamespace
+
+    from . import cuda as K
+    from . import cuda_hybrid as H
+    add = _Table()
+    tf = add.tf
+    bf = dict(dtype=torch.bfloat16, device="cuda")
+    D, P, N, G, taps = 128, 64, 128, 1, 4
+    SH = 2 * width // P
+    inner = SH * P
+    C = inner + 2 * G * N
+    bias = torch.randn(heads, window, device="cuda")
+    lat = SimpleNamespace(heads=heads, dim=128, rot=64, dv=128, rank=512, scale=0.07, window=window, rot_gain=1.0, freq=torch.rand(32, device="cuda"),
+                          w_k=torch.randn(heads * 128, 512, **bf) * 0.04, w_v=torch.randn(heads * 128, 512, **bf) * 0.04)
+    lat.w_k_t = lat.w_k.view(heads, 128, 512).transpose(1, 2).contiguous()
+    w, wb, gain = torch.randn(C, taps, **bf), torch.randn(C, **bf), torch.ones(inner, **bf)
+    one = torch.ones(SH, device="cuda")
+    norm = SimpleNamespace(w=torch.ones(width, **bf), b=torch.ones(width, **bf), alpha=torch.ones(1, device="cuda"))
+    pad = (SH + 7) // 8 * 8
+    for B, q in ((1, 4096), (8, 512)):
+        case, T = f"{B} x {q} tokens", B * q
+        m = _meta(B, q, q)
+        kc = torch.randn(m.page_table.numel(), 64, kv_heads, D, **bf)
+        vc, Q, gate = torch.randn_like(kc), torch.randn(T, heads, D, **bf), torch.randn(T, heads * D, **bf)
+        out = torch.empty(T, heads * D, **bf)
+        keys = sum(min(i + 1, window) for i in range(q)) / q
+        add("attention_prefill", case, lambda: K.attention_prefill(Q, kc, vc, m, 0.1), 4.0 * heads * D * T * (q + 1) / 2, tf, like="dense decoder")
+        fl = 4.0 * heads * D * T * keys
+        add("  windowed", case, lambda: K.attention_prefill(Q, kc, vc, m, 0.1, window), fl, tf, like="dense decoder")
+        add("  windowed split_p", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1, out=out, window=window), fl, tf)
+        add("  windowed split_p bias gate", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1, out=out, window=window, bias=bias, gate=gate), fl, tf)
+        cache = torch.randn(m.page_table.numel(), 64, 1, 576, **bf) * 0.1
+        ql = torch.randn(T, heads * 192, **bf)
+        k, v = H.expand_latent(cache.view(-1, 576), lat)
+        k, v = k.view(-1, 64, heads, 192), v.view(-1, 64, heads, 128)
+        fl = 2.0 * heads * (192 + 128) * T * keys
+        add("attention 192/128 windowed", case, lambda: K.attention_prefill(ql.view(T, heads, 192), k, v, m, 0.1, window), fl, tf, like="latent decoder")
+        add("  split_p", case, lambda: K.attention_prefill(ql.view(T, heads, 192), k, v, m, 0.1, window, split_p=True), fl, tf)
+        add("expand_latent", case, lambda: H.expand_latent(cache.view(-1, 576), lat), 2.0 * T * heads * 256 * 512, tf, T * heads * 320 * 2)
+        add("latent_attention (all)", case, lambda: H.latent_attention(ql, cache, m, lat), fl + 2.0 * T * heads * 256 * 512, tf)
+        del k, v, ql, Q, kc, vc
+        y = torch.randn(T, inner + C + pad, **bf)
+        z, xbc, dt = y[:, :inner], y[:, inner:inner + C], y[:, inner + C:inner + C + SH]
+        S, ring, o = torch.zeros(B, SH, P, N, device="cuda"), torch.zeros(B, taps, C, **bf), torch.empty(T, inner, **bf)
+        pre = H.ssd_chunk_prep(xbc, w, wb, ring, dt, one, one, m, SH)
+        yy = H.ssd_chunk(*pre, one, S, m, G, SH, N, P)
+        add("ss_conv_decay", case, lambda: H.ssd_chunk_prep(xbc, w, wb, ring, dt, one, one, m, SH), nbytes=T * C * 4)
+        # 64-token chunks: products of the chunk (lower half), read and update of the state
+        add("ssd_chunk", case, lambda: H.ssd_chunk(*pre, one, S, m, G, SH, N, P), 2.0 * T * SH * (32 * P + 32 * N + 2 * N * P), tf, T * (C * 2 + inner * 4))
+        add("gated_part_norm", case, lambda: H.gated_part_norm(yy, z, gain, 8, 1e-5, o), nbytes=T * inner * 8)
+        sp = H.ss_prep(xbc, w, wb, ring, dt, one, one, m, G, SH, N, P)
+        add("ss_prep (32-bit models)", case, lambda: H.ss_prep(xbc, w, wb, ring, dt, one, one, m, G, SH, N, P), nbytes=T * C * 6)
+        add("head_decay_scan (32-bit)", case, lambda: H.head_decay_scan(*sp, one, S, m, G, SH, N, P), 5.0 * T * SH * N * P, F32_TFLOPS)
+        del y, z, xbc, dt, pre, yy, sp
+        kc = torch.randn(m.page_table.numel(), 64, kv_heads, D, **bf)
+        vc = torch.randn_like(kc)
+        n_in = (heads + 2 * kv_heads) * D
+        y, g1 = torch.randn(T, n_in, **bf), torch.ones(D, **bf)
+        parts = y.split([heads * D, kv_heads * D, kv_heads * D], 1)
+        gq, gk = torch.ones(heads * D, **bf), torch.ones(kv_heads * D, **bf)
+        inv = torch.ones(D // 2, device="cuda")
+        add("qk_norm_rope_append", case, lambda: K.qk_norm_rope_append(y, heads, kv_heads, D, g1, g1, False, inv, m, kc, vc, 1e-5), nbytes=T * n_in * 4,
+            like="dense decoder")
+        add("row_norm_append", case, lambda: H.row_norm_append(*parts, heads, kv_heads, D, D, gq, gk, m, kc, vc, 1e-5), nbytes=T * n_in * 4)
+        yl = torch.randn(T, 768 + 576, **bf)
+        add("latent_prep", case, lambda: H.latent_prep(yl[:, :768], yl[:, 768:], torch.ones(768, **bf), torch.ones(512, **bf), lat.freq, 1.0, m, cache, 1e-5),
+            nbytes=T * 1344 * 4)
+        ar, h, hb, xb = torch.randn(T, width, device="cuda"), torch.randn(T, width, device="cuda"), torch.randn(T, width, **bf), torch.randn(T, width, **bf)
+        add("add_rmsnorm", case, lambda: K.add_rmsnorm(xb, hb, norm.w, 1e-5), nbytes=T * width * 8, like="dense decoder")
+        add("dyt_add", case, lambda: H.dyt_add(ar, norm, h, norm), nbytes=T * width * 14)
+    for B in (1, 32, 128):
+        case, ctx = f"{B} x 1 token", 2048
+        m = _meta(B, 1, ctx)
+        kc = torch.randn(m.page_table.numel(), 64, kv_heads, D, **bf)
+        vc, Q, gate = torch.randn_like(kc), torch.randn(B, heads, D, **bf), torch.randn(B, heads * D, **bf)
+        out = torch.empty(B, heads * D, **bf)
+        add("paged_attention_decode", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1), nbytes=2.0 * B * ctx * kv_heads * D * 2, like="dense decoder")
+        nb = 2.0 * B * window * kv_heads * D * 2
+        add("  windowed", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1, window=window), nbytes=nb, like="dense decoder")
+        add("  windowed bias gate", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1, out=out, window=window, bias=bias, gate=gate), nbytes=nb)
+        cache = torch.randn(m.page_table.numel(), 64, 1, 576, **bf) * 0.1
+        qf, ql = torch.randn(B, heads, 576, **bf), torch.randn(B, heads * 192, **bf)
+        cv = cache.view(-1, 64, 576)
+        add("mla_attention", case, lambda: K.mla_attention(qf, cv, m, 0.1), 2.0 * B * ctx * heads * 1088, tf, B * ctx * 1152.0, like="latent decoder")
+        fl, nb = 2.0 * B * window * heads * 1088, B * window * 1152.0
+        add("  windowed", case, lambda: K.mla_attention(qf, cv, m, 0.1, window=window), fl, tf, nb, like="latent decoder")
+        add("  windowed split_p", case, lambda: K.mla_attention(qf, cv, m, 0.1, window=window, split_p=True), fl, tf, nb)
+        add("latent_attention (all)", case, lambda: H.latent_attention(ql, cache, m, lat), fl, tf, nb + heads * 256 * 512 * 2)
+        y = torch.randn(B, inner + C + pad, **bf)
+        S, ring, o = torch.zeros(B, SH, P, N, device="cuda"), torch.zeros(B, taps, C, **bf), torch.empty(B, inner, **bf)
+        add("ss_step", case, lambda: H.state_space(y[:, inner:inner + C], w, wb, y[:, inner + C:inner + C + SH], one, one, one, y[:, :inner], gain, 8, ring, S, m,
+                                                   G, SH, N, P, 1e-5, o), nbytes=B * SH * P * N * 8.0)
+        ar, h, hb, xb = torch.randn(B, width, device="cuda"), torch.randn(B, width, device="cuda"), torch.randn(B, width, **bf), torch.randn(B, width, **bf)
+        add("add_rmsnorm", case, lambda: K.add_rmsnorm(xb, hb, norm.w, 1e-5), nbytes=B * width * 8, like="dense decoder")
+        add("dyt_add", case, lambda: H.dyt_add(ar, norm, h, norm), nbytes=B * width * 14)
+    assert K.last_status() == 0
+    return add.rows

@@ -568,6 +568,9 @@ if __name__ == "__main__":
     if what == "hybrid":
         from .bench_hybrid import run as bench_hybrid
         bench_hybrid(*nums)
+    if what == "rokarax":
+        from .bench_hybrid import run_rokarax
+        run_rokarax(*nums)
     if what == "moeprefill":
         bench_moeprefill(*nums)
     if what == "bf16moe":
