@@ -32,7 +32,9 @@ constexpr float RESCALE_THRESHOLD = 8.0f;
 
 // SPLITP: P is handed to the tensor cores as the sum of two bf16 values (rounded value and rounding error), so that the softmax
 // weights keep 16 significant bits; two P V products per block.
-template <int DK, int DV, bool SPLITP>
+// BIAS: a bias by distance is added to the scaled score.  Every softmax warp copies the 95 values that its rows can meet in a block to
+// shared memory, minus infinity outside the window and after the query, so the bias is the mask as well.
+template <int DK, int DV, bool SPLITP, bool BIAS>
 struct FaCfg {
   static constexpr int NCK = DK / CHUNK, NCV = DV / CHUNK;
   static constexpr int Q_CHUNK_BYTES = TR * 128;
@@ -41,8 +43,9 @@ struct FaCfg {
   static constexpr int K_STAGE = NCK * K_CHUNK_BYTES, V_STAGE = NCV * V_CHUNK_BYTES;
   static constexpr int STAGES = (DK + DV > 384) ? 2 : 3;
   static constexpr int NPBUF = (SPLITP && DK + DV > 256) ? 1 : 2;
+  static constexpr int BIAS_BYTES = BIAS ? 4 * 96 * 4 : 0;
   static constexpr int P_STAGE = SPLITP ? 2 * P_BYTES : P_BYTES;
-  static constexpr int SMEM = Q_BYTES + STAGES * (K_STAGE + V_STAGE) + NPBUF * P_STAGE + 1024 + 256;
+  static constexpr int SMEM = Q_BYTES + STAGES * (K_STAGE + V_STAGE) + NPBUF * P_STAGE + BIAS_BYTES + 1024 + 256;
   static constexpr int TMEM_COLS = DV <= 128 ? 256 : 512;     // S: 2 x 64 columns at 0..127, O: DV columns at 128..
   static_assert(DK % CHUNK == 0 && DV % CHUNK == 0 && DV <= 256 && DK <= 256, "head dims: multiples of 64 up to 256");
   static_assert(SMEM <= 232448, "shared memory budget");
@@ -72,7 +75,7 @@ template <int DK, int DV, bool SPLITP, bool BIAS>
 __global__ void __launch_bounds__(NTHREADS, 1)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                   const __grid_constant__ CUtensorMap tm_v, const FaParams p) {
-  using C = FaCfg<DK, DV, SPLITP>;
+  using C = FaCfg<DK, DV, SPLITP, BIAS>;
   constexpr int STAGES = C::STAGES, NPBUF = C::NPBUF;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~uintptr_t(1023));
@@ -80,7 +83,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
   uint8_t* sK = sQ + C::Q_BYTES;
   uint8_t* sV = sK + STAGES * C::K_STAGE;
   uint8_t* sP = sV + STAGES * C::V_STAGE;
-  uint64_t* bars = (uint64_t*)(sP + NPBUF * C::P_STAGE);
+  uint64_t* bars = (uint64_t*)(sP + NPBUF * C::P_STAGE + C::BIAS_BYTES);
   uint64_t* q_full = bars;                 // 1
   uint64_t* k_full = q_full + 1;           // [STAGES]
   uint64_t* k_empty = k_full + STAGES;
@@ -227,8 +230,21 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
     const int lo_key = p.window > 0 ? qpos - p.window + 1 : 0;
     const uint32_t lane_off = (uint32_t)(q4 * 32) << 16;
     float m_ref = -INFINITY, l = 0.f;
+    float* const bias_row = (float*)(sP + NPBUF * C::P_STAGE) + q4 * 96;
     for (int i = 0; i < nblk; ++i) {
       const int sb = i % NSBUF, pb = i % NPBUF;
+      if constexpr (BIAS) {
+        // bias_row[d]: rows q4 * 32 + lane and keys j of the block with distance base + d, d = 63 + lane - j
+        const int base = pos_first + q4 * 32 - (b_lo + i) * KB - (KB - 1);
+        const float* src = p.bias + (int64_t)head * p.window;
+        __syncwarp();
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+          const int dist = base + k * 32 + lane;
+          bias_row[k * 32 + lane] = dist >= 0 && dist < p.window ? src[dist] * 1.4426950408889634f : -INFINITY;
+        }
+        __syncwarp();
+      }
       if (!mbar_wait(&s_full[sb], (i / NSBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
       tc_fence_after();
       uint32_t sr[KB];
@@ -245,15 +261,11 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       const bool full_blk = key0 + KB - 1 <= pos_first && (p.window <= 0 || key0 >= pos_first + TR - p.window);
       const float* sf = (const float*)sr;
       float mx;
-      if (BIAS) {
-        constexpr float LOG2E = 1.4426950408889634f;
-        const float* br = p.bias + (int64_t)head * p.window + (qpos - key0);      // br[-j]: bias of key j of the block
+      if constexpr (BIAS) {
         mx = -INFINITY;
 #pragma unroll
         for (int j = 0; j < KB; ++j) {
-          const int kj = key0 + j;
-          const bool ok = full_blk || (row_ok && kj <= qpos && kj >= lo_key);
-          const float v = ok ? fmaf(br[-j], LOG2E, __uint_as_float(sr[j]) * p.scale_log2) : -INFINITY;
+          const float v = fmaf(__uint_as_float(sr[j]), p.scale_log2, bias_row[KB - 1 + lane - j]);
           sr[j] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
@@ -295,10 +307,11 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
           psum += a + b;
         }
       } else {
+        const float nm = m_ref == -INFINITY ? 0.f : -m_ref;        // nothing visible yet: every score is minus infinity, every weight 0
 #pragma unroll
         for (int j = 0; j < KB / 2; ++j) {
-          const float a = (m_ref == -INFINITY) ? 0.f : exp2f(__uint_as_float(sr[2 * j]) - m_ref);
-          const float b = (m_ref == -INFINITY) ? 0.f : exp2f(__uint_as_float(sr[2 * j + 1]) - m_ref);
+          const float a = exp2f(__uint_as_float(sr[2 * j]) + nm);
+          const float b = exp2f(__uint_as_float(sr[2 * j + 1]) + nm);
           __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
           pw[j] = *(uint32_t*)&h;
           float2 back = __bfloat1622float2(h);
@@ -417,7 +430,7 @@ int make_cache_map(CUtensorMap* m, const void* cache, int heads, int hd, int num
 template <int DK, int DV, bool SPLITP, bool BIAS>
 int launch_fa(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const FaParams& p, int NB, cudaStream_t s) {
   static MarySmemSlots smem_set = {};
-  constexpr int SMEM = FaCfg<DK, DV, SPLITP>::SMEM;
+  constexpr int SMEM = FaCfg<DK, DV, SPLITP, BIAS>::SMEM;
   if (int rc = mary_ensure_dyn_smem((const void*)fa_prefill_kernel<DK, DV, SPLITP, BIAS>, SMEM, &smem_set)) return rc;
   fa_prefill_kernel<DK, DV, SPLITP, BIAS><<<dim3(NB, p.Hq), NTHREADS, SMEM, s>>>(tq, tk, tv, p);
   MARY_CHECK_LAUNCH();

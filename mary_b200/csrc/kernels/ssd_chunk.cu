@@ -11,23 +11,27 @@
 // keeps 16 significant bits; sums and the carried state are 32-bit.  The logarithms c are summed in 64 bits and kept as two floats: their
 // differences stay exact however small the decays have become.
 //
-// One CTA = (32 value channels, head, sequence), four warps = (16 channels) x (half of the state's rows).  The state lives transposed in
-// the accumulator registers of mma.m16n8k16, [channel][state row]; read that way an accumulator IS the second operand of the product that
-// reads the state, so it never leaves the registers between chunks.  C, B and x of the next chunk are in flight while this one is worked on.
+// The products C_i . B_j of a chunk are the same for every head of a group and come from a kernel of their own (gram).  One CTA of the
+// recurrence = (32 value channels, head, sequence), eight warps = (16 channels) x (a quarter of the state's rows).  The state lives
+// transposed in the accumulator registers of mma.m16n8k16, [channel][state row]; read that way an accumulator IS the second operand of the
+// product that reads the state, so it never leaves the registers between chunks.  C, B and x of the next chunk are in flight while this
+// one is worked on.  Rows in shared memory are padded by 16 bytes, so the eight rows of a fragment fall on different banks and every
+// address of a loop is a base and a constant.
 #include "host_utils.h"
-#include "recurrent.cuh"
+#include "typed.cuh"
 
 using namespace mary;
 
 namespace {
 
 typedef __nv_bfloat16 bf16;
-constexpr int L = 64, PC = 32, NTH = 128;
+constexpr int L = 64, PC = 32, NTH = 256;
 
 struct ChunkParams {
   const bf16* xbc;                       // [T][C]: x [H P], B [G N], C [G N]
   const float* dt; const float* c_hi; const float* c_lo;      // [H][T]; c: log2 of the decay since the start of the token's chunk
   const float* skip; float* y; float* state;
+  float4* gram;                          // [chunk][G][10 blocks][2][32 lanes]: C_i . B_j as a lane's accumulators of two 16 x 8 tiles
   const int* q_start; const int* kv_len; const int* slots;
   int T, G, H, N, P, C;
 };
@@ -39,14 +43,19 @@ __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t a) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
 }
 __device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool in) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
 }
 __device__ __forceinline__ void cp4(uint32_t dst, const void* src, bool in) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(dst), "l"(src), "r"(in ? 4 : 0) : "memory");
+}
+__device__ __forceinline__ float pow2(float x) {            // x <= 0
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
 }
 // (a, b) as two bf16 pairs: rounded values and rounding errors
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
@@ -56,23 +65,76 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
   hi = *(const uint32_t*)&h;
   lo = *(const uint32_t*)&l;
 }
-// byte offset of a 16-byte piece in a tile whose rows have CH of them; rows are permuted so that eight rows of a column hit all banks
-template <int CH> __device__ __forceinline__ uint32_t at(int row, int piece) {
-  if constexpr (CH >= 8) return (uint32_t)(row * CH + (piece ^ (row & 7))) * 16;
-  else return (uint32_t)(row * CH + (piece ^ ((row >> 1) & 3))) * 16;
-}
+// the ten 16 x 16 blocks on and below the diagonal of a chunk's 64 x 64 token pairs
+__device__ __forceinline__ int blk_m(int b) { return b < 4 ? 3 : b < 7 ? 2 : b < 9 ? 1 : 0; }
+__device__ __forceinline__ int blk_j(int b) { return b < 4 ? b : b < 7 ? b - 4 : b < 9 ? b - 7 : 0; }
+// chunk c of a sequence whose rows start at row0: a place of its own among T / 64 + sequences places
+__device__ __forceinline__ int64_t chunk_place(int row0, int seq, int c) { return row0 / L + seq + c; }
 
 template <int NP> struct Lay {
-  static constexpr int TILE = L * NP * 2, X = L * PC * 2, M = L * L * 2;
+  static constexpr int ROW = NP * 2 + 16, XROW = PC * 2 + 16, MROW = L * 2 + 16;        // bytes
+  static constexpr int TILE = L * ROW, X = L * XROW, M = L * MROW;
   static constexpr int SC = 2 * TILE + X, STAGE = SC + 3 * L * 4;       // C, B, x, (dt, c_hi, c_lo)
-  static constexpr int M_AT = 2 * STAGE, XW_AT = M_AT + 2 * M, Y_AT = XW_AT + 2 * X, BYTES = Y_AT + L * PC * 4;
+  static constexpr int M_AT = 2 * STAGE, XW_AT = M_AT + 2 * M;
+  static constexpr int Y_AT = M_AT, Y = L * PC * 4;                     // three partial results, over what the products have read by then
+  static constexpr int BYTES = XW_AT + 2 * X;
+  static_assert(3 * Y <= 2 * M + 2 * X, "the partial results fit");
 };
 
+// 64 rows of B and C: piece k of row r, THREADS threads.  Rows past `rows` and state rows past N are zero.
+template <int NP, int THREADS>
+__device__ __forceinline__ void load_bc(uint32_t dst_c, uint32_t dst_b, const bf16* first_row, int64_t ld, int c_off, int N, int rows) {
+  constexpr int CN = NP / 8, STEP = THREADS / CN;
+  const int r0 = threadIdx.x / CN, k = threadIdx.x % CN;
+  const bool col = k * 8 < N;
+  const bf16* src = first_row + (col ? k * 8 : 0);
+  const uint32_t o = r0 * Lay<NP>::ROW + k * 16;
+#pragma unroll
+  for (int i = 0; i < L / STEP; ++i) {
+    const int r = r0 + i * STEP;
+    const bool in = col && r < rows;
+    const bf16* s = src + (in ? r * ld : 0);
+    cp16(dst_c + o + i * STEP * Lay<NP>::ROW, s + c_off, in);
+    cp16(dst_b + o + i * STEP * Lay<NP>::ROW, s, in);
+  }
+}
+
 template <int NP>
-__global__ void __launch_bounds__(NTH) ssd_chunk_kernel(const ChunkParams p) {
+__global__ void __launch_bounds__(128) ssd_gram_kernel(const ChunkParams p) {
   pdl_sync();
   using S = Lay<NP>;
-  constexpr int CN = NP / 8, NH = NP / 2, NT = NH / 8;      // 16-byte pieces per row of B / C; state rows and 8-row tiles of a warp
+  extern __shared__ __align__(128) uint8_t smem[];
+  const int seq = blockIdx.z, g = blockIdx.y, c = blockIdx.x, lane = threadIdx.x & 31;
+  const int row0 = p.q_start[seq], n = p.q_start[seq + 1] - row0;
+  if (c * L >= n) return;
+  const uint32_t sC = smem_u32(smem), sB = sC + S::TILE;
+  load_bc<NP, 128>(sC, sB, p.xbc + (int64_t)(row0 + c * L) * p.C + p.H * p.P + g * p.N, p.C, p.G * p.N, p.N, n - c * L);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  for (int b = threadIdx.x >> 5; b < 10; b += 4) {
+    float gm[2][4] = {};
+    const uint32_t ac = sC + (blk_m(b) * 16 + (lane & 15)) * S::ROW + (lane >> 4) * 16;
+    const uint32_t bc = sB + (blk_j(b) * 16 + (lane & 7) + ((lane >> 4) << 3)) * S::ROW + ((lane >> 3) & 1) * 16;
+#pragma unroll
+    for (int k = 0; k < NP / 16; ++k) {
+      uint32_t a[4], q[4];
+      ldsm4(a, ac + k * 32);
+      ldsm4(q, bc + k * 32);
+      mma(gm[0], a, q[0], q[1]);
+      mma(gm[1], a, q[2], q[3]);
+    }
+    float4* dst = p.gram + ((chunk_place(row0, seq, c) * p.G + g) * 10 + b) * 64 + lane;
+#pragma unroll
+    for (int t = 0; t < 2; ++t) dst[t * 32] = make_float4(gm[t][0], gm[t][1], gm[t][2], gm[t][3]);
+  }
+}
+
+template <int NP>
+__global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const ChunkParams p) {
+  pdl_sync();
+  using S = Lay<NP>;
+  constexpr int NH = NP / 4, NT = NH / 8;                   // state rows and 8-row tiles of a warp
   extern __shared__ __align__(128) uint8_t smem[];
   const uint32_t sm = smem_u32(smem);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pw = warp & 1, nw = warp >> 1;
@@ -96,22 +158,18 @@ __global__ void __launch_bounds__(NTH) ssd_chunk_kernel(const ChunkParams p) {
       st[t][2 * e + 1] = v.y;
     }
   const float skip = p.skip[h];
+  const bf16* bc_rows = p.xbc + (int64_t)row0 * p.C + inner + g * p.N;
+  const int xr = tid >> 2, xk = tid & 3;                    // x: one 16-byte piece per thread
+  const bf16* x_rows = p.xbc + (int64_t)row0 * p.C + h * p.P;
+  const bool x_col = p0 + xk * 8 < p.P;
+  const uint32_t x_at = xr * S::XROW + xk * 16;
 
   auto load = [&](int c) {                                  // chunk c -> stage c & 1
     const uint32_t s = sm + (c & 1) * S::STAGE;
     const int t0 = c * L;
-    for (int i = tid; i < L * CN; i += NTH) {
-      const int r = i / CN, k = i % CN;
-      const bool in = t0 + r < n && k * 8 < p.N;
-      const bf16* src = p.xbc + (int64_t)(row0 + (in ? t0 + r : 0)) * p.C + inner + g * p.N + (in ? k * 8 : 0);
-      cp16(s + at<CN>(r, k), src + p.G * p.N, in);          // C
-      cp16(s + S::TILE + at<CN>(r, k), src, in);            // B
-    }
-    for (int i = tid; i < L * (PC / 8); i += NTH) {
-      const int r = i / (PC / 8), k = i % (PC / 8);
-      const bool in = t0 + r < n && p0 + k * 8 < p.P;
-      cp16(s + 2 * S::TILE + at<PC / 8>(r, k), p.xbc + (int64_t)(row0 + (in ? t0 + r : 0)) * p.C + h * p.P + (in ? p0 + k * 8 : 0), in);
-    }
+    load_bc<NP, NTH>(s, s + S::TILE, bc_rows + (int64_t)t0 * p.C, p.C, p.G * p.N, p.N, n - t0);
+    const bool in = x_col && t0 + xr < n;
+    cp16(s + 2 * S::TILE + x_at, x_rows + (in ? (int64_t)(t0 + xr) * p.C + p0 + xk * 8 : 0), in);
     if (tid < L) {                                          // tokens past the end: no step, the decay of the last one
       const int64_t o = (int64_t)h * p.T + row0 + min(t0 + tid, n - 1);
       const uint32_t d = s + S::SC + tid * 4;
@@ -121,10 +179,23 @@ __global__ void __launch_bounds__(NTH) ssd_chunk_kernel(const ChunkParams p) {
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
+  auto gram = [&](int c, int b, float4 (&v)[2]) {
+    const float4* src = p.gram + ((chunk_place(row0, seq, c) * p.G + g) * 10 + b) * 64 + lane;
+    v[0] = src[0];
+    v[1] = src[32];
+  };
+  // this lane's places in the fragments
+  const uint32_t f_c = (lane & 15) * S::ROW + (nw * NH) * 2 + (lane >> 4) * 16;               // C, first operand
+  const uint32_t f_m = (nw * 16 + (lane & 15)) * S::MROW + (lane >> 4) * 16;                  // decayed products, first operand
+  const uint32_t f_x = (lane & 15) * S::XROW + (pw * 2 + (lane >> 4)) * 16;                   // x, second operand
+  const uint32_t f_w = ((lane & 7) + ((lane >> 4) << 3)) * S::XROW + (pw * 2 + ((lane >> 3) & 1)) * 16;      // weighted x, first operand
+  const uint32_t f_b = (lane & 15) * S::ROW + (nw * NH) * 2 + (lane >> 4) * 16;               // B, second operand
 
   const int chunks = (n + L - 1) / L;
   load(0);
   for (int c = 0; c < chunks; ++c) {
+    float4 gm[2];
+    gram(c, warp, gm);
     if (c + 1 < chunks) {
       load(c + 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
@@ -137,58 +208,45 @@ __global__ void __launch_bounds__(NTH) ssd_chunk_kernel(const ChunkParams p) {
     const float* dt = (const float*)(smem + stage + S::SC);
     const float *hi = dt + L, *lo = hi + L;
     const float hiL = hi[L - 1], loL = lo[L - 1];
-    // x weighted for the state update
-    for (int i = tid; i < L * (PC / 8); i += NTH) {
-      const int r = i / (PC / 8);
-      const uint32_t o = at<PC / 8>(r, i % (PC / 8));
-      const float w = exp2f((hiL - hi[r]) + (loL - lo[r])) * dt[r];
+    {                                                       // x weighted for the state update
+      const float w = pow2((hiL - hi[xr]) + (loL - lo[xr])) * dt[xr];
       float f[8];
-      unpack16(*(const uint4*)(smem + stage + 2 * S::TILE + o), f);
+      unpack16(*(const uint4*)(smem + stage + 2 * S::TILE + x_at), f);
       uint4 a, b;
       split2(f[0] * w, f[1] * w, a.x, b.x);
       split2(f[2] * w, f[3] * w, a.y, b.y);
       split2(f[4] * w, f[5] * w, a.z, b.z);
       split2(f[6] * w, f[7] * w, a.w, b.w);
-      *(uint4*)(smem + S::XW_AT + o) = a;
-      *(uint4*)(smem + S::XW_AT + S::X + o) = b;
+      *(uint4*)(smem + S::XW_AT + x_at) = a;
+      *(uint4*)(smem + S::XW_AT + S::X + x_at) = b;
     }
-    // decayed products of the chunk's tokens: the ten 16 x 16 blocks on and below the diagonal, shared out over the warps
-    {
-      constexpr int MT[10] = {3, 3, 2, 2, 3, 3, 2, 1, 0, 1}, JT[10] = {0, 2, 0, 2, 1, 3, 1, 1, 0, 0};
+    for (int b = warp; b < 10; b += 8) {                    // decayed products
+      const int mt = blk_m(b), jt = blk_j(b);
+      const int i0 = mt * 16 + lr;
+      const float hii[2] = {hi[i0], hi[i0 + 8]}, loi[2] = {lo[i0], lo[i0 + 8]};
 #pragma unroll
-      for (int b = 0; b < 10; ++b) {
-        if ((b & 3) != warp) continue;
-        const int mt = MT[b], jt = JT[b];
-        float gm[2][4] = {};
-#pragma unroll
-        for (int k = 0; k < NP / 16; ++k) {
-          uint32_t a[4], q[4];
-          ldsm4(a, sC + at<CN>(mt * 16 + (lane & 15), 2 * k + (lane >> 4)));
-          ldsm4(q, sB + at<CN>(jt * 16 + (lane & 7) + ((lane >> 4) << 3), 2 * k + ((lane >> 3) & 1)));
-          mma(gm[0], a, q[0], q[1]);
-          mma(gm[1], a, q[2], q[3]);
-        }
+      for (int t = 0; t < 2; ++t) {
+        const int j = jt * 16 + t * 8 + lc;
+        const float2 hj = *(const float2*)(hi + j), lj = *(const float2*)(lo + j), dj = *(const float2*)(dt + j);
+        const float gv[4] = {gm[t].x, gm[t].y, gm[t].z, gm[t].w};
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int i = mt * 16 + lr + 8 * e;
-          const float hii = hi[i], loi = lo[i];
-#pragma unroll
-          for (int t = 0; t < 2; ++t) {
-            const int j = jt * 16 + t * 8 + lc;
-            float w[2];
-#pragma unroll
-            for (int d = 0; d < 2; ++d)
-              w[d] = j + d <= i ? gm[t][2 * e + d] * (exp2f((hii - hi[j + d]) + (loi - lo[j + d])) * dt[j + d]) : 0.f;
-            uint32_t vh, vl;
-            split2(w[0], w[1], vh, vl);
-            const uint32_t o = at<L / 8>(i, jt * 2 + t) + (lane & 3) * 4;
-            *(uint32_t*)(smem + S::M_AT + o) = vh;
-            *(uint32_t*)(smem + S::M_AT + S::M + o) = vl;
+          float w0 = gv[2 * e] * (pow2((hii[e] - hj.x) + (loi[e] - lj.x)) * dj.x);
+          float w1 = gv[2 * e + 1] * (pow2((hii[e] - hj.y) + (loi[e] - lj.y)) * dj.y);
+          if (mt == jt) {
+            if (j > i0 + 8 * e) w0 = 0.f;
+            if (j + 1 > i0 + 8 * e) w1 = 0.f;
           }
+          uint32_t vh, vl;
+          split2(w0, w1, vh, vl);
+          uint8_t* d = smem + S::M_AT + (i0 + 8 * e) * S::MROW + j * 2;
+          *(uint32_t*)d = vh;
+          *(uint32_t*)(d + S::M) = vl;
         }
       }
+      if (b + 8 < 10) gram(c, b + 8, gm);
     }
-    // what the state before the chunk gives (this warp's half of its rows)
+    // what the state before the chunk gives (this warp's quarter of its rows), without the tokens' decay
     float y[4][2][4];
 #pragma unroll
     for (int mt = 0; mt < 4; ++mt)
@@ -203,105 +261,90 @@ __global__ void __launch_bounds__(NTH) ssd_chunk_kernel(const ChunkParams p) {
       for (int o = 0; o < 2; ++o)
 #pragma unroll
         for (int t = 0; t < 2; ++t) split2(st[2 * k + t][2 * o], st[2 * k + t][2 * o + 1], bh[o][t], bl[o][t]);
+      uint32_t a[4][4];
 #pragma unroll
-      for (int mt = 0; mt < 4; ++mt) {
-        uint32_t a[4];
-        ldsm4(a, sC + at<CN>(mt * 16 + (lane & 15), (nw * NH + k * 16) / 8 + (lane >> 4)));
+      for (int mt = 0; mt < 4; ++mt) ldsm4(a[mt], sC + f_c + mt * 16 * S::ROW + k * 32);
 #pragma unroll
-        for (int o = 0; o < 2; ++o) {
-          mma(y[mt][o], a, bh[o][0], bh[o][1]);
-          mma(y[mt][o], a, bl[o][0], bl[o][1]);
-        }
-      }
+      for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+        for (int o = 0; o < 2; ++o) mma(y[mt][o], a[mt], bh[o][0], bh[o][1]);
+#pragma unroll
+      for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+        for (int o = 0; o < 2; ++o) mma(y[mt][o], a[mt], bl[o][0], bl[o][1]);
     }
-#pragma unroll
-    for (int mt = 0; mt < 4; ++mt)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int i = mt * 16 + lr + 8 * e;
-        const float w = exp2f(hi[i] + lo[i]);
-#pragma unroll
-        for (int o = 0; o < 2; ++o) {
-          y[mt][o][2 * e] *= w;
-          y[mt][o][2 * e + 1] *= w;
-        }
-      }
     __syncthreads();
-    // tokens of the chunk among themselves: token blocks 0 and 3 on the first pair of warps, 1 and 2 on the second
-#pragma unroll
-    for (int mt = 0; mt < 4; ++mt) {
-      if ((mt == 0 || mt == 3) != (nw == 0)) continue;
-#pragma unroll
-      for (int k = 0; k <= mt; ++k) {
-        uint32_t a[4], b[4], q[4];
-        const uint32_t o = at<L / 8>(mt * 16 + (lane & 15), 2 * k + (lane >> 4));
-        ldsm4(a, sM + o);
-        ldsm4(b, sM + S::M + o);
-        ldsm4t(q, sX + at<PC / 8>(k * 16 + (lane & 15), pw * 2 + (lane >> 4)));
-        mma(y[mt][0], a, q[0], q[1]);
-        mma(y[mt][1], a, q[2], q[3]);
-        mma(y[mt][0], b, q[0], q[1]);
-        mma(y[mt][1], b, q[2], q[3]);
-      }
-    }
-    // the other half's token blocks to shared memory
-    auto y_at = [&](int i, int o) { return (float2*)(smem + S::Y_AT) + i * (PC / 2) + ((pw * 8 + o * 4 + (lane & 3)) ^ ((i & 3) << 2)); };
-#pragma unroll
-    for (int mt = 0; mt < 4; ++mt)
-      if ((mt < 2) != (nw == 0)) {
-#pragma unroll
-        for (int o = 0; o < 2; ++o)
-#pragma unroll
-          for (int e = 0; e < 2; ++e) *y_at(mt * 16 + lr + 8 * e, o) = make_float2(y[mt][o][2 * e], y[mt][o][2 * e + 1]);
-      }
     // state update
-    const float decay = exp2f(hiL + loL);
+    const float decay = pow2(hiL + loL);
 #pragma unroll
     for (int t = 0; t < NT; ++t)
 #pragma unroll
       for (int e = 0; e < 4; ++e) st[t][e] *= decay;
 #pragma unroll
     for (int k = 0; k < L / 16; ++k) {
-      uint32_t a[4], b[4];
-      const uint32_t o = at<PC / 8>(k * 16 + (lane & 7) + ((lane >> 4) << 3), pw * 2 + ((lane >> 3) & 1));
-      ldsm4t(a, sW + o);
-      ldsm4t(b, sW + S::X + o);
+      uint32_t a[4], b[4], q[NT / 2][4];
+      ldsm4t(a, sW + f_w + k * 16 * S::XROW);
+      ldsm4t(b, sW + S::X + f_w + k * 16 * S::XROW);
 #pragma unroll
-      for (int t = 0; t < NT; t += 2) {
-        uint32_t q[4];
-        ldsm4t(q, sB + at<CN>(k * 16 + (lane & 15), nw * NT + t + (lane >> 4)));
-        mma(st[t], a, q[0], q[1]);
-        mma(st[t + 1], a, q[2], q[3]);
-        mma(st[t], b, q[0], q[1]);
-        mma(st[t + 1], b, q[2], q[3]);
-      }
+      for (int t = 0; t < NT / 2; ++t) ldsm4t(q[t], sB + f_b + k * 16 * S::ROW + t * 32);
+#pragma unroll
+      for (int t = 0; t < NT; ++t) mma(st[t], a, q[t / 2][2 * (t & 1)], q[t / 2][2 * (t & 1) + 1]);
+#pragma unroll
+      for (int t = 0; t < NT; ++t) mma(st[t], b, q[t / 2][2 * (t & 1)], q[t / 2][2 * (t & 1) + 1]);
     }
-    float2 x[2][2][2];
+    // tokens of the chunk among themselves: token block nw, which this warp also finishes
+    float z[2][4] = {};
+    for (int k = 0; k <= nw; ++k) {
+      uint32_t a[4], b[4], q[4];
+      ldsm4(a, sM + f_m + k * 32);
+      ldsm4(b, sM + S::M + f_m + k * 32);
+      ldsm4t(q, sX + f_x + k * 16 * S::XROW);
+      mma(z[0], a, q[0], q[1]);
+      mma(z[1], a, q[2], q[3]);
+      mma(z[0], b, q[0], q[1]);
+      mma(z[1], b, q[2], q[3]);
+    }
+    const float own[2] = {pow2(hi[nw * 16 + lr] + lo[nw * 16 + lr]), pow2(hi[nw * 16 + lr + 8] + lo[nw * 16 + lr + 8])};
 #pragma unroll
-    for (int m = 0; m < 2; ++m)
+    for (int o = 0; o < 2; ++o)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float2 x = __bfloat1622float2(*(const __nv_bfloat162*)(smem + stage + 2 * S::TILE + (nw * 16 + lr + 8 * e) * S::XROW + (pw * 2 + o) * 16 + lc * 2));
+        z[o][2 * e] = fmaf(skip, x.x, z[o][2 * e]);
+        z[o][2 * e + 1] = fmaf(skip, x.y, z[o][2 * e + 1]);
+      }
+    __syncthreads();
+    // the other token blocks' partial results go to their warps
+    auto y_at = [&](int slot, int i, int o) {
+      return (float2*)(smem + S::Y_AT + slot * S::Y) + i * (PC / 2) + ((pw * 8 + o * 4 + (lane & 3)) ^ ((i & 3) << 2));
+    };
+    float mine[2][4];
+#pragma unroll
+    for (int mt = 0; mt < 4; ++mt) {
 #pragma unroll
       for (int o = 0; o < 2; ++o)
 #pragma unroll
-        for (int e = 0; e < 2; ++e)
-          x[m][o][e] = __bfloat1622float2(*(const __nv_bfloat162*)(smem + stage + 2 * S::TILE +
-                                                                   at<PC / 8>((nw * 2 + m) * 16 + lr + 8 * e, pw * 2 + o) + (lane & 3) * 4));
+        for (int e = 0; e < 2; ++e) {
+          if (mt == nw) {
+            mine[o][2 * e] = y[mt][o][2 * e];
+            mine[o][2 * e + 1] = y[mt][o][2 * e + 1];
+          } else {
+            *y_at((nw - mt - 1) & 3, mt * 16 + lr + 8 * e, o) = make_float2(y[mt][o][2 * e], y[mt][o][2 * e + 1]);
+          }
+        }
+    }
     __syncthreads();
 #pragma unroll
-    for (int mt = 0; mt < 4; ++mt) {
-      if ((mt < 2) != (nw == 0)) {
-        continue;
-      }
+    for (int e = 0; e < 2; ++e) {
+      const int i = nw * 16 + lr + 8 * e;
+      if (c * L + i >= n) continue;
+      float* dst = p.y + (int64_t)(row0 + c * L + i) * inner + h * p.P + p0 + pw * 16 + lc;
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int i = mt * 16 + lr + 8 * e;
-        if (c * L + i >= n) continue;
-        float* dst = p.y + (int64_t)(row0 + c * L + i) * inner + h * p.P + p0 + pw * 16 + lc;
-#pragma unroll
-        for (int o = 0; o < 2; ++o) {
-          const float2 v = *y_at(i, o), xv = x[mt & 1][o][e];
-          if (p0 + pw * 16 + o * 8 < p.P)
-            *(float2*)(dst + o * 8) = make_float2(fmaf(skip, xv.x, y[mt][o][2 * e] + v.x), fmaf(skip, xv.y, y[mt][o][2 * e + 1] + v.y));
-        }
+      for (int o = 0; o < 2; ++o) {
+        const float2 u = *y_at(0, i, o), v = *y_at(1, i, o), w = *y_at(2, i, o);
+        if (p0 + pw * 16 + o * 8 < p.P)
+          *(float2*)(dst + o * 8) = make_float2(fmaf(own[e], (mine[o][2 * e] + u.x) + (v.x + w.x), z[o][2 * e]),
+                                                fmaf(own[e], (mine[o][2 * e + 1] + u.y) + (v.y + w.y), z[o][2 * e + 1]));
       }
     }
   }
@@ -314,55 +357,110 @@ __global__ void __launch_bounds__(NTH) ssd_chunk_kernel(const ChunkParams p) {
     }
 }
 
-// silu(conv(xbc) + bias) in bf16: a thread takes four channels of four tokens
+// silu(conv(xbc) + bias) in bf16: a thread takes four channels of CB tokens, the rows it reads all requested before the first is used
+constexpr int CB = 16;
 template <int TAPS>
-__global__ void __launch_bounds__(256) ss_conv_kernel(const bf16* __restrict__ xbc, int64_t ldx, const bf16* __restrict__ w, const bf16* __restrict__ bias,
+__global__ void __launch_bounds__(128) ss_conv_kernel(const bf16* __restrict__ xbc, int64_t ldx, const bf16* __restrict__ w, const bf16* __restrict__ bias,
                                                       const bf16* __restrict__ ring_all, const int* __restrict__ q_start, const int* __restrict__ kv_len,
-                                                      const int* __restrict__ slots, bf16* __restrict__ out, int taps, int C) {
+                                                      const int* __restrict__ slots, bf16* __restrict__ out, int n_taps, int C) {
   pdl_sync();
-  const int seq = blockIdx.z, blk = blockIdx.y, ch = (blockIdx.x * 256 + threadIdx.x) * 4;
-  const int first = q_start[seq], end = q_start[seq + 1], rb = first + blk * 4;
+  const int taps = TAPS > 0 ? TAPS : n_taps;
+  const int seq = blockIdx.z, ch = (blockIdx.x * 128 + threadIdx.x) * 4;
+  const int first = q_start[seq], end = q_start[seq + 1], rb = first + blockIdx.y * CB;
   if (rb >= end || ch >= C) return;
-  const int pos = kv_len[seq] - (end - first) + blk * 4;
-  float y[4][4];
-  conv_block<bf16, TAPS, 4>(xbc, ldx, w, bias, ring_all + (int64_t)slots[seq] * taps * C, taps, C, ch, rb, first, end, pos, y);
+  const int pos = kv_len[seq] - (end - first) + blockIdx.y * CB;
+  const bf16* ring = ring_all + (int64_t)slots[seq] * taps * C;
+  float b[4];
+  load_e<bf16, 4>(bias + ch, b);
+  if constexpr (TAPS > 0) {
+    float v[TAPS + CB - 1][4];
 #pragma unroll
-  for (int t = 0; t < 4; ++t)
-    if (rb + t < end) store_e<bf16, 4>(out + (int64_t)(rb + t) * C + ch, y[t]);
-}
-
-// One thread per (chunk, head): step sizes and the summed logarithms of the decays, [H][T]
-__global__ void __launch_bounds__(128) ss_decay_kernel(const bf16* __restrict__ dt_in, int64_t ldx, const float* __restrict__ dt_bias,
-                                                       const float* __restrict__ a_log, const int* __restrict__ q_start, float* __restrict__ dt,
-                                                       float* __restrict__ c_hi, float* __restrict__ c_lo, int H, int T) {
-  pdl_sync();
-  const int h = blockIdx.x * 128 + threadIdx.x, seq = blockIdx.z;
-  const int t0 = q_start[seq] + blockIdx.y * L, t1 = min(t0 + L, q_start[seq + 1]);
-  if (h >= H || t0 >= t1) return;
-  const float bias = dt_bias[h], a = -expf(a_log[h]);
-  const int64_t o = (int64_t)h * T;
-  double c = 0.0;
-  for (int t = t0; t < t1; t += 8) {
-    float raw[8];
+    for (int r = 1 - TAPS; r < CB; ++r) {
+      const bf16* src = rb + r >= first ? xbc + (int64_t)(rb + r) * ldx + ch : ring + (int64_t)((pos + r + TAPS) % TAPS) * C + ch;
+      if (rb + r < end && pos + r >= 0) load_e<bf16, 4>(src, v[r + TAPS - 1]);
+      else
 #pragma unroll
-    for (int i = 0; i < 8; ++i) raw[i] = t + i < t1 ? __bfloat162float(dt_in[(int64_t)(t + i) * ldx + h]) : 0.f;
+        for (int e = 0; e < 4; ++e) v[r + TAPS - 1][e] = 0.f;
+    }
+    float wt[4][TAPS];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      if (t + i >= t1) break;
-      const float d = softplus_x(raw[i] + bias);
-      c += (double)(a * d) * 1.4426950408889634;
-      const float ch = (float)c;
-      dt[o + t + i] = d;
-      c_hi[o + t + i] = ch;
-      c_lo[o + t + i] = (float)(c - (double)ch);
+    for (int e = 0; e < 4; ++e)
+      load_e<bf16, TAPS>(w + (int64_t)(ch + e) * TAPS, wt[e]);
+#pragma unroll
+    for (int t = 0; t < CB; ++t) {
+      float y[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        y[e] = b[e];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) y[e] = fmaf(wt[e][j], v[t + j][e], y[e]);
+        y[e] = silu_t<bf16>(y[e]);
+      }
+      if (rb + t < end) store_e<bf16, 4>(out + (int64_t)(rb + t) * C + ch, y);
+    }
+  } else {
+    for (int t = 0; t < CB && rb + t < end; ++t) {
+      float y[4] = {b[0], b[1], b[2], b[3]};
+      for (int d = 0; d < taps; ++d) {                     // d tokens back
+        const int r = t - d;
+        float v[4];
+        if (rb + r >= first) load_e<bf16, 4>(xbc + (int64_t)(rb + r) * ldx + ch, v);
+        else if (pos + r >= 0) load_e<bf16, 4>(ring + (int64_t)((pos + r) % taps) * C + ch, v);
+        else break;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[e] = fmaf(__bfloat162float(w[(int64_t)(ch + e) * taps + taps - 1 - d]), v[e], y[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) y[e] = silu_t<bf16>(y[e]);
+      store_e<bf16, 4>(out + (int64_t)(rb + t) * C + ch, y);
     }
   }
 }
 
+// One warp per (chunk, head): step sizes and the summed logarithms of the decays, [H][T]; a lane takes two tokens
+__global__ void __launch_bounds__(256) ss_decay_kernel(const bf16* __restrict__ dt_in, int64_t ldx, const float* __restrict__ dt_bias,
+                                                       const float* __restrict__ a_log, const int* __restrict__ q_start, float* __restrict__ dt,
+                                                       float* __restrict__ c_hi, float* __restrict__ c_lo, int H, int T) {
+  pdl_sync();
+  const int h = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, seq = blockIdx.z;
+  const int t0 = q_start[seq] + blockIdx.y * L, t1 = min(t0 + L, q_start[seq + 1]);
+  if (h >= H || t0 >= t1) return;
+  const float bias = dt_bias[h], a = -expf(a_log[h]);
+  float d[2];
+  double c[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int t = t0 + 2 * lane + i;
+    d[i] = t < t1 ? softplus_x(__bfloat162float(dt_in[(int64_t)t * ldx + h]) + bias) : 0.f;
+    c[i] = (double)(a * d[i]) * 1.4426950408889634;
+  }
+  c[1] += c[0];
+  double before = c[1];                                // inclusive scan over the lanes, then what came before this lane
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const double v = __shfl_up_sync(0xffffffffu, before, o);
+    if (lane >= o) before += v;
+  }
+  before -= c[1];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int t = t0 + 2 * lane + i;
+    if (t >= t1) continue;
+    const double v = before + c[i];
+    const float hi = (float)v;
+    const int64_t o = (int64_t)h * T + t;
+    dt[o] = d[i];
+    c_hi[o] = hi;
+    c_lo[o] = (float)(v - (double)hi);
+  }
+}
+
 template <int NP>
-int launch_chunk(const ChunkParams& p, int S, cudaStream_t s) {
-  static MarySmemSlots slots = {};
-  if (int rc = mary_ensure_dyn_smem((const void*)ssd_chunk_kernel<NP>, Lay<NP>::BYTES, &slots)) return rc;
+int launch_chunk(const ChunkParams& p, int S, int max_q, cudaStream_t s) {
+  static MarySmemSlots slots[2] = {};
+  if (int rc = mary_ensure_dyn_smem((const void*)ssd_gram_kernel<NP>, 2 * Lay<NP>::TILE, &slots[0])) return rc;
+  if (int rc = mary_ensure_dyn_smem((const void*)ssd_chunk_kernel<NP>, Lay<NP>::BYTES, &slots[1])) return rc;
+  MARY_LAUNCH((ssd_gram_kernel<NP>), dim3((max_q + L - 1) / L, p.G, S), 128, 2 * Lay<NP>::TILE, s, p);
   MARY_LAUNCH((ssd_chunk_kernel<NP>), dim3((p.P + PC - 1) / PC, p.H, S), NTH, Lay<NP>::BYTES, s, p);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
@@ -378,12 +476,12 @@ MARY_API int mary_ss_conv_decay(const void* xbc, int64_t ldx, const void* taps_w
   if (S <= 0 || max_q <= 0) return MARY_OK;
   if (H < 1 || C < 1 || C % 4 || ldx % 4 || taps < 1 || S > 65535 || (((uintptr_t)xbc | (uintptr_t)ring | (uintptr_t)taps_w | (uintptr_t)xbc_out) & 7))
     return MARY_ERR_BAD_ARG;
-  if ((max_q + 3) / 4 > 65535) return MARY_ERR_BAD_ARG;
-  const dim3 grid((C / 4 + 255) / 256, (max_q + 3) / 4, S);
+  if ((max_q + CB - 1) / CB > 65535 || ((uintptr_t)taps_b & 7)) return MARY_ERR_BAD_ARG;
+  const dim3 grid((C / 4 + 127) / 128, (max_q + CB - 1) / CB, S);
   auto fn = taps == 4 ? ss_conv_kernel<4> : ss_conv_kernel<0>;
-  MARY_LAUNCH(fn, grid, 256, 0, s, (const bf16*)xbc, ldx, (const bf16*)taps_w, (const bf16*)taps_b, (const bf16*)ring, q_start, kv_len, slots,
+  MARY_LAUNCH(fn, grid, 128, 0, s, (const bf16*)xbc, ldx, (const bf16*)taps_w, (const bf16*)taps_b, (const bf16*)ring, q_start, kv_len, slots,
               (bf16*)xbc_out, taps, C);
-  MARY_LAUNCH(ss_decay_kernel, dim3((H + 127) / 128, (max_q + L - 1) / L, S), 128, 0, s, (const bf16*)dt_in, ldx, dt_bias, a_log, q_start, dt, c_hi, c_lo,
+  MARY_LAUNCH(ss_decay_kernel, dim3((H + 7) / 8, (max_q + L - 1) / L, S), 256, 0, s, (const bf16*)dt_in, ldx, dt_bias, a_log, q_start, dt, c_hi, c_lo,
               H, T);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
@@ -391,13 +489,18 @@ MARY_API int mary_ss_conv_decay(const void* xbc, int64_t ldx, const void* taps_w
 
 MARY_API int mary_ssd_chunk_supported(int N, int P) { return N >= 8 && N <= 256 && N % 8 == 0 && P >= 8 && P % 8 == 0; }
 
-// y [T, H P] f32; the state [slots][H][P][N] is read (zero for a portion that starts its sequence) and updated in place.
+MARY_API int64_t mary_ssd_chunk_scratch_floats(int T, int S, int G) { return ((int64_t)T / L + S + 1) * G * 10 * 64 * 4; }
+
+// y [T, H P] f32; the state [slots][H][P][N] is read (zero for a portion that starts its sequence) and updated in place.  scratch:
+// mary_ssd_chunk_scratch_floats(T, S, G) floats, 16-byte aligned.
 MARY_API int mary_ssd_chunk(const void* xbc, const float* dt, const float* c_hi, const float* c_lo, const float* skip, float* y, float* state,
-                            const int* q_start, const int* kv_len, const int* slots, int S, int T, int G, int H, int N, int P, cudaStream_t s) {
+                            float* scratch, const int* q_start, const int* kv_len, const int* slots, int S, int max_q, int T, int G, int H, int N, int P,
+                            cudaStream_t s) {
   if (S <= 0 || T <= 0) return MARY_OK;
-  if (G < 1 || H < 1 || H % G || H > 65535 || S > 65535 || !mary_ssd_chunk_supported(N, P) || ((uintptr_t)xbc & 15)) return MARY_ERR_BAD_ARG;
-  const ChunkParams p = {(const bf16*)xbc, dt, c_hi, c_lo, skip, y, state, q_start, kv_len, slots, T, G, H, N, P, H * P + 2 * G * N};
-  if (N <= 64) return launch_chunk<64>(p, S, s);
-  if (N <= 128) return launch_chunk<128>(p, S, s);
-  return launch_chunk<256>(p, S, s);
+  if (G < 1 || H < 1 || H % G || H > 65535 || S > 65535 || !mary_ssd_chunk_supported(N, P) || (((uintptr_t)xbc | (uintptr_t)scratch) & 15))
+    return MARY_ERR_BAD_ARG;
+  const ChunkParams p = {(const bf16*)xbc, dt, c_hi, c_lo, skip, y, state, (float4*)scratch, q_start, kv_len, slots, T, G, H, N, P, H * P + 2 * G * N};
+  if (N <= 64) return launch_chunk<64>(p, S, max_q, s);
+  if (N <= 128) return launch_chunk<128>(p, S, max_q, s);
+  return launch_chunk<256>(p, S, max_q, s);
 }

@@ -92,8 +92,8 @@ __global__ void __launch_bounds__(256) ss_prep_kernel(const T* __restrict__ xbc,
   }
 }
 
-// out[t, part] = rms(y[t, part] * silu(z[t, part])) * gain, one CTA per (token, part) of n values
-template <typename T>
+// out[t, part] = rms(y[t, part] * silu(z[t, part])) * gain, one CTA per (token, part) of n values; E values per access
+template <typename T, int E>
 __global__ void gated_part_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, int64_t ldz, const T* __restrict__ gain, T* __restrict__ out,
                                        int64_t ldo, int inner, int n, float eps) {
   pdl_sync();
@@ -102,27 +102,43 @@ __global__ void gated_part_norm_kernel(const float* __restrict__ y, const T* __r
   const int c0 = blockIdx.y * n;
   const float* yr = y + t * inner + c0;
   const T* zr = z + t * ldz + c0;
-  constexpr int KEEP = 8;                             // values a thread keeps between the two passes
-  float v[KEEP], ss = 0.f;
+  T* o = out + t * ldo + c0;
+  constexpr int KEEP = E == 1 ? 8 : 2;                // accesses a thread keeps between the two passes
+  const int step = blockDim.x * E;
+  float v[KEEP][E], ss = 0.f;
+  auto value = [&](int i, float (&u)[E]) {
+    float zv[E];
+    load_e<float, E>(yr + i, u);
+    load_e<T, E>(zr + i, zv);
 #pragma unroll
-  for (int j = 0; j < KEEP; ++j) {
-    const int i = threadIdx.x + j * blockDim.x;
-    v[j] = i < n ? yr[i] * silu_t<T>(to_f<T>(zr[i])) : 0.f;
-    ss = fmaf(v[j], v[j], ss);
-  }
-  for (int i = threadIdx.x + KEEP * blockDim.x; i < n; i += blockDim.x) {
-    const float u = yr[i] * silu_t<T>(to_f<T>(zr[i]));
-    ss = fmaf(u, u, ss);
+    for (int e = 0; e < E; ++e) {
+      u[e] *= silu_t<T>(zv[e]);
+      ss = fmaf(u[e], u[e], ss);
+    }
+  };
+  auto put = [&](int i, float (&u)[E], float inv) {
+    float g[E];
+    load_e<T, E>(gain + c0 + i, g);
+#pragma unroll
+    for (int e = 0; e < E; ++e) u[e] *= inv * g[e];
+    store_e<T, E>(o + i, u);
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j)
+    if (threadIdx.x * E + j * step < n) value(threadIdx.x * E + j * step, v[j]);
+  for (int i = threadIdx.x * E + KEEP * step; i < n; i += step) {
+    float u[E];
+    value(i, u);
   }
   const float inv = 1.0f / sqrtf(block_sum_x(ss, red) / n + eps);
-  T* o = out + t * ldo + c0;
 #pragma unroll
-  for (int j = 0; j < KEEP; ++j) {
-    const int i = threadIdx.x + j * blockDim.x;
-    if (i < n) o[i] = from_f<T>(v[j] * inv * to_f<T>(gain[c0 + i]));
+  for (int j = 0; j < KEEP; ++j)
+    if (threadIdx.x * E + j * step < n) put(threadIdx.x * E + j * step, v[j], inv);
+  for (int i = threadIdx.x * E + KEEP * step; i < n; i += step) {
+    float u[E];
+    value(i, u);
+    put(i, u, inv);
   }
-  for (int i = threadIdx.x + KEEP * blockDim.x; i < n; i += blockDim.x)
-    o[i] = from_f<T>(yr[i] * silu_t<T>(to_f<T>(zr[i])) * inv * to_f<T>(gain[c0 + i]));
 }
 
 struct SsStep {
@@ -241,7 +257,12 @@ MARY_API int mary_gated_part_norm(const float* y, const void* z, int64_t ldz, co
   const int n = inner / parts;
   int nt = (n + 7) / 8;
   nt = nt <= 32 ? 32 : (nt >= 512 ? 512 : (nt + 31) / 32 * 32);
-  BY_TYPE(f32, MARY_LAUNCH((gated_part_norm_kernel<T>), dim3(n_tok, parts), nt, 0, s, y, (const T*)z, ldz, (const T*)gain, (T*)out, ldo, inner, n, eps));
+  BY_TYPE(f32, {
+    const uintptr_t mask = 4 * sizeof(T) - 1;
+    const bool vec = n % 4 == 0 && ldz % 4 == 0 && ldo % 4 == 0 && !(((uintptr_t)z | (uintptr_t)gain | (uintptr_t)out) & mask) && !((uintptr_t)y & 15);
+    auto fn = vec ? gated_part_norm_kernel<T, 4> : gated_part_norm_kernel<T, 1>;
+    MARY_LAUNCH(fn, dim3(n_tok, parts), nt, 0, s, y, (const T*)z, ldz, (const T*)gain, (T*)out, ldo, inner, n, eps);
+  });
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }

@@ -38,7 +38,8 @@ declare("mary_rotate_heads", "pppfp" + "iiiiii" + "is")
 declare("mary_fill_shared_part", "pliplii" + "iis")
 declare("mary_ss_prep", "pl" + "pppppp" + "ppp" + "pppppp" + "iiiiiii" + "is")
 declare("mary_ss_conv_decay", "pl" + "pppppp" + "ppp" + "pppp" + "iiiiiis")
-declare("mary_ssd_chunk", "ppppppp" + "ppp" + "iiiiiis")
+declare("mary_ssd_chunk", "pppppppp" + "ppp" + "iiiiiiis")
+declare("mary_ssd_chunk_scratch_floats", "iii", ret64=True)
 declare("mary_ssd_chunk_supported", "ii")
 declare("mary_head_decay_scan", "pppppppp" + "p" + "ppp" + "illl" + "iiiis")
 declare("mary_gated_part_norm", "pplppl" + "iiifis")
@@ -461,8 +462,9 @@ def ssd_chunk(rows, dt, hi, lo, skip, state, meta, G, H, N, P):
     """The recurrence on the tensor cores, 64 tokens at a time: f32 ``[T, H * P]``."""
     T = rows.shape[0]
     y = _empty(T, H * P, dtype=torch.float32, device=rows.device)
-    check(lib().mary_ssd_chunk(_p(rows), _p(dt), _p(hi), _p(lo), _p(skip), _p(y), _p(state), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots),
-                               meta.num_seqs, T, G, H, N, P, _stream()), "ssd_chunk")
+    scratch = _empty(lib().mary_ssd_chunk_scratch_floats(T, meta.num_seqs, G), dtype=torch.float32, device=rows.device)
+    check(lib().mary_ssd_chunk(_p(rows), _p(dt), _p(hi), _p(lo), _p(skip), _p(y), _p(state), _p(scratch), _p(meta.q_start), _p(meta.kv_len),
+                               _p(meta.state_slots), meta.num_seqs, meta.max_q_len, T, G, H, N, P, _stream()), "ssd_chunk")
     return y
 
 

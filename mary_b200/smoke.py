@@ -62,6 +62,27 @@ def _recurrent_engine(dev):
     return out
 
 
+def _state_space_engine(dev):
+    """A Rokarax decoder (attention with a distance bias, state space, latent attention, a layer with shared keys) generating through the
+    scheduler, two sequences."""
+    from .models.registry import family_of, make_engine
+    from .models.rokarax import RokaraxConfig, RokaraxModel, init_random_
+    mlp = {"kind": "dense", "ff": 512}
+    att = dict(heads=8, kv_heads=2, dim=64, vdim=64, scale=0.1, bias_max=100.0, mask={"size": 70})
+    layers = [{"type": "attention", "mlp": mlp, "mixer": att},
+              {"type": "mamba2", "mlp": None, "mixer": dict(heads=8, vdim=64, state=128, groups=2, conv=4, norm_groups=2)},
+              {"type": "latent_attention", "mlp": mlp, "mixer": dict(
+                  heads=4, dim=128, rot_dim=64, vdim=128, q_rank=128, kv_rank=512, scale=0.07, mask={"size": 50},
+                  rot={"dims": 64, "base": 10000.0, "scaling": dict(factor=2.0, original=1024.0, fast=32.0, slow=1.0)})},
+              {"type": "attention", "mlp": mlp, "mixer": {**att, "kv_from": 0}}]
+    d = {"architecture": "Rokarax", "vocab": 1024, "width": 512, "norm": {"eps": 1e-6}, "embedding": {"scale": 8.0}, "layers": layers}
+    m = RokaraxModel(RokaraxConfig.from_json(d), dtype=torch.bfloat16, device=dev)
+    init_random_(m, 0)
+    out = make_engine(m, family_of(d), 512, 2, dev).generate([list(range(90)), [5, 4, 3]], 4)
+    assert all(len(o) == 4 for o in out)
+    return out
+
+
 def _lora_step(m, dev):
     from .train.trainer import LoraTrainer
     tr = LoraTrainer(m, rank=8, alpha=16.0, lr=1e-3)
@@ -80,9 +101,10 @@ def run_smoke() -> None:
     n = _flagship(dev)
     m, out = _gemma_engine(dev)
     rec = _recurrent_engine(dev)
+    ssm = _state_space_engine(dev)
     losses = _lora_step(m, dev)
     torch.cuda.synchronize()
     st = cuda.last_status()
     assert st == 0, f"kernel status {st}"
-    print(f"smoke ok: flagship emitted {n} tokens in 4 speculative steps; gemma {out}; tatizen {rec}; lora loss {losses[0]:.3f} -> {losses[1]:.3f}; "
+    print(f"smoke ok: flagship emitted {n} tokens in 4 speculative steps; gemma {out}; tatizen {rec}; rokarax {ssm}; lora loss {losses[0]:.3f} -> {losses[1]:.3f}; "
           f"{cuda.LAUNCHES} kernel launches")
