@@ -17,7 +17,11 @@ struct SsIo {
 };
 
 __device__ __forceinline__ float step_size(float raw, float bias) { return softplus_x(raw + bias); }
-__device__ __forceinline__ float step_decay(float a_log, float dt) { return expf(-expf(a_log) * dt); }
+// Decays close to 1 are multiplied over thousands of tokens, so theirs is the exponential with the smaller error there.
+__device__ __forceinline__ float step_decay(float a_log, float dt) {
+  const float x = -expf(a_log) * dt;
+  return x > -0.5f ? 1.0f + expm1f(x) : expf(x);
+}
 
 // One warp per (sequence, block of four tokens, item); items: G groups (B, C and the products B_j . C_i of the block), chunks of x
 // channels, chunks of 32 heads (step sizes and decays).  VEC: widths, pitch and addresses allow accesses of four values.
