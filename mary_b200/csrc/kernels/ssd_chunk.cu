@@ -46,6 +46,10 @@ __device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint3
   asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+__device__ __forceinline__ void mma_first(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {      // d = a b
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%10, %10, %10, %10};"
+      : "=f"(d[0]), "=f"(d[1]), "=f"(d[2]), "=f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1), "f"(0.f));
+}
 __device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool in) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
 }
@@ -76,27 +80,30 @@ template <int NP> struct Lay {
   static constexpr int TILE = L * ROW, X = L * XROW, M = L * MROW;
   static constexpr int SC = 2 * TILE + X, STAGE = SC + 3 * L * 4;       // C, B, x, (dt, c_hi, c_lo)
   static constexpr int M_AT = 2 * STAGE, XW_AT = M_AT + 2 * M;
-  static constexpr int Y_AT = M_AT, Y = L * PC * 4;                     // three partial results, over what the products have read by then
-  static constexpr int BYTES = XW_AT + 2 * X;
-  static_assert(3 * Y <= 2 * M + 2 * X, "the partial results fit");
+  static constexpr int Y_AT = M_AT, Y = L * PC * 4;                     // four partial results, over what the products have read by then
+  static constexpr int BYTES = M_AT + 4 * Y;
+  static_assert(2 * M + 2 * X <= 4 * Y, "the decayed products and the weighted x fit");
 };
 
-// 64 rows of B and C: piece k of row r, THREADS threads.  Rows past `rows` and state rows past N are zero.
+// 64 rows of B and C, THREADS threads; src: this thread's first piece of B.  Rows past `rows` and state rows past N are zero.
 template <int NP, int THREADS>
-__device__ __forceinline__ void load_bc(uint32_t dst_c, uint32_t dst_b, const bf16* first_row, int64_t ld, int c_off, int N, int rows) {
+__device__ __forceinline__ void load_bc(uint32_t dst_c, uint32_t dst_b, const bf16* src, int64_t ld, int c_off, bool col, int rows) {
   constexpr int CN = NP / 8, STEP = THREADS / CN;
   const int r0 = threadIdx.x / CN, k = threadIdx.x % CN;
-  const bool col = k * 8 < N;
-  const bf16* src = first_row + (col ? k * 8 : 0);
   const uint32_t o = r0 * Lay<NP>::ROW + k * 16;
+  const bf16* s = src;
 #pragma unroll
   for (int i = 0; i < L / STEP; ++i) {
-    const int r = r0 + i * STEP;
-    const bool in = col && r < rows;
-    const bf16* s = src + (in ? r * ld : 0);
-    cp16(dst_c + o + i * STEP * Lay<NP>::ROW, s + c_off, in);
-    cp16(dst_b + o + i * STEP * Lay<NP>::ROW, s, in);
+    const bool in = col && r0 + i * STEP < rows;
+    cp16(dst_c + o + i * STEP * Lay<NP>::ROW, in ? s + c_off : src, in);
+    cp16(dst_b + o + i * STEP * Lay<NP>::ROW, in ? s : src, in);
+    s += STEP * ld;
   }
+}
+template <int NP, int THREADS> __device__ __forceinline__ const bf16* first_piece(const bf16* row, int64_t ld, int N) {
+  constexpr int CN = NP / 8;
+  const int k = threadIdx.x % CN;
+  return row + (k * 8 < N ? (int64_t)(threadIdx.x / CN) * ld + k * 8 : 0);
 }
 
 template <int NP>
@@ -108,7 +115,9 @@ __global__ void __launch_bounds__(128) ssd_gram_kernel(const ChunkParams p) {
   const int row0 = p.q_start[seq], n = p.q_start[seq + 1] - row0;
   if (c * L >= n) return;
   const uint32_t sC = smem_u32(smem), sB = sC + S::TILE;
-  load_bc<NP, 128>(sC, sB, p.xbc + (int64_t)(row0 + c * L) * p.C + p.H * p.P + g * p.N, p.C, p.G * p.N, p.N, n - c * L);
+  const bf16* row = p.xbc + (int64_t)(row0 + c * L) * p.C + p.H * p.P + g * p.N;
+  const bool in = (int)(threadIdx.x / (NP / 8)) < n - c * L;
+  load_bc<NP, 128>(sC, sB, in ? first_piece<NP, 128>(row, p.C, p.N) : row, p.C, p.G * p.N, (threadIdx.x % (NP / 8)) * 8 < p.N, n - c * L);
   asm volatile("cp.async.commit_group;" ::: "memory");
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
@@ -158,32 +167,35 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
       st[t][2 * e + 1] = v.y;
     }
   const float skip = p.skip[h];
-  const bf16* bc_rows = p.xbc + (int64_t)row0 * p.C + inner + g * p.N;
-  const int xr = tid >> 2, xk = tid & 3;                    // x: one 16-byte piece per thread
-  const bf16* x_rows = p.xbc + (int64_t)row0 * p.C + h * p.P;
+  // what this thread copies of a chunk: pieces of B and C (rows bc_r, bc_r + STEP, ..), one piece of x, one token's step and decay
+  constexpr int CN = NP / 8;
+  const int bc_r = tid / CN;
+  const bool bc_col = tid % CN * 8 < p.N;
+  const bf16* bc_row = p.xbc + (int64_t)row0 * p.C + inner + g * p.N;
+  const int xr = tid >> 2, xk = tid & 3;
   const bool x_col = p0 + xk * 8 < p.P;
+  const bf16* x_row = p.xbc + (int64_t)row0 * p.C + h * p.P + (x_col ? p0 + xk * 8 : 0);
   const uint32_t x_at = xr * S::XROW + xk * 16;
+  const int64_t dt_at = (int64_t)h * p.T + row0;
 
   auto load = [&](int c) {                                  // chunk c -> stage c & 1
     const uint32_t s = sm + (c & 1) * S::STAGE;
-    const int t0 = c * L;
-    load_bc<NP, NTH>(s, s + S::TILE, bc_rows + (int64_t)t0 * p.C, p.C, p.G * p.N, p.N, n - t0);
-    const bool in = x_col && t0 + xr < n;
-    cp16(s + 2 * S::TILE + x_at, x_rows + (in ? (int64_t)(t0 + xr) * p.C + p0 + xk * 8 : 0), in);
+    const int t0 = c * L, left = n - t0;
+    const bf16* row = bc_row + (int64_t)t0 * p.C;
+    load_bc<NP, NTH>(s, s + S::TILE, bc_r < left ? first_piece<NP, NTH>(row, p.C, p.N) : row, p.C, p.G * p.N, bc_col, left);
+    const bool in = x_col && xr < left;
+    cp16(s + 2 * S::TILE + x_at, x_row + (int64_t)(in ? t0 + xr : t0) * p.C, in);
     if (tid < L) {                                          // tokens past the end: no step, the decay of the last one
-      const int64_t o = (int64_t)h * p.T + row0 + min(t0 + tid, n - 1);
+      const int64_t o = dt_at + min(t0 + tid, n - 1);
       const uint32_t d = s + S::SC + tid * 4;
-      cp4(d, p.dt + o, t0 + tid < n);
+      cp4(d, p.dt + o, tid < left);
       cp4(d + L * 4, p.c_hi + o, true);
       cp4(d + 2 * L * 4, p.c_lo + o, true);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  auto gram = [&](int c, int b, float4 (&v)[2]) {
-    const float4* src = p.gram + ((chunk_place(row0, seq, c) * p.G + g) * 10 + b) * 64 + lane;
-    v[0] = src[0];
-    v[1] = src[32];
-  };
+  const float4* gram_at = p.gram + (chunk_place(row0, seq, 0) * p.G + g) * 640 + lane;
+  float* y_at = p.y + (int64_t)(row0 + nw * 16 + lr) * inner + h * p.P + p0 + pw * 16 + lc;      // this lane's first result of a chunk
   // this lane's places in the fragments
   const uint32_t f_c = (lane & 15) * S::ROW + (nw * NH) * 2 + (lane >> 4) * 16;               // C, first operand
   const uint32_t f_m = (nw * 16 + (lane & 15)) * S::MROW + (lane >> 4) * 16;                  // decayed products, first operand
@@ -194,8 +206,7 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
   const int chunks = (n + L - 1) / L;
   load(0);
   for (int c = 0; c < chunks; ++c) {
-    float4 gm[2];
-    gram(c, warp, gm);
+    float4 gm[2] = {gram_at[warp * 64], gram_at[warp * 64 + 32]};
     if (c + 1 < chunks) {
       load(c + 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
@@ -244,16 +255,10 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
           *(uint32_t*)(d + S::M) = vl;
         }
       }
-      if (b + 8 < 10) gram(c, b + 8, gm);
+      if (b + 8 < 10) { gm[0] = gram_at[(b + 8) * 64]; gm[1] = gram_at[(b + 8) * 64 + 32]; }
     }
     // what the state before the chunk gives (this warp's quarter of its rows), without the tokens' decay
     float y[4][2][4];
-#pragma unroll
-    for (int mt = 0; mt < 4; ++mt)
-#pragma unroll
-      for (int o = 0; o < 2; ++o)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) y[mt][o][e] = 0.f;
 #pragma unroll
     for (int k = 0; k < NH / 16; ++k) {
       uint32_t bh[2][2], bl[2][2];                          // [channel octet][half of the k rows]
@@ -267,7 +272,10 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
 #pragma unroll
       for (int mt = 0; mt < 4; ++mt)
 #pragma unroll
-        for (int o = 0; o < 2; ++o) mma(y[mt][o], a[mt], bh[o][0], bh[o][1]);
+        for (int o = 0; o < 2; ++o) {
+          if (k == 0) mma_first(y[mt][o], a[mt], bh[o][0], bh[o][1]);
+          else mma(y[mt][o], a[mt], bh[o][0], bh[o][1]);
+        }
 #pragma unroll
       for (int mt = 0; mt < 4; ++mt)
 #pragma unroll
@@ -314,39 +322,32 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
         z[o][2 * e + 1] = fmaf(skip, x.y, z[o][2 * e + 1]);
       }
     __syncthreads();
-    // the other token blocks' partial results go to their warps
-    auto y_at = [&](int slot, int i, int o) {
-      return (float2*)(smem + S::Y_AT + slot * S::Y) + i * (PC / 2) + ((pw * 8 + o * 4 + (lane & 3)) ^ ((i & 3) << 2));
-    };
-    float mine[2][4];
+    // partial results of the four quarters meet in shared memory: token i, channel pair c2 at place c2 ^ 4 (i & 3) of its row
+    const int c2 = (pw * 8 + (lane & 3)) ^ ((lr & 3) << 2), c2_b = c2 ^ 4;
+    float2* part = (float2*)(smem + S::Y_AT + nw * S::Y) + lr * (PC / 2);
 #pragma unroll
-    for (int mt = 0; mt < 4; ++mt) {
+    for (int mt = 0; mt < 4; ++mt)
 #pragma unroll
-      for (int o = 0; o < 2; ++o)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          if (mt == nw) {
-            mine[o][2 * e] = y[mt][o][2 * e];
-            mine[o][2 * e + 1] = y[mt][o][2 * e + 1];
-          } else {
-            *y_at((nw - mt - 1) & 3, mt * 16 + lr + 8 * e, o) = make_float2(y[mt][o][2 * e], y[mt][o][2 * e + 1]);
-          }
-        }
-    }
+      for (int e = 0; e < 2; ++e) {
+        part[(mt * 16 + 8 * e) * (PC / 2) + c2] = make_float2(y[mt][0][2 * e], y[mt][0][2 * e + 1]);
+        part[(mt * 16 + 8 * e) * (PC / 2) + c2_b] = make_float2(y[mt][1][2 * e], y[mt][1][2 * e + 1]);
+      }
     __syncthreads();
+    const float2* sum = (const float2*)(smem + S::Y_AT) + (nw * 16 + lr) * (PC / 2);
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      const int i = nw * 16 + lr + 8 * e;
-      if (c * L + i >= n) continue;
-      float* dst = p.y + (int64_t)(row0 + c * L + i) * inner + h * p.P + p0 + pw * 16 + lc;
+      if (c * L + nw * 16 + lr + 8 * e >= n) continue;
 #pragma unroll
       for (int o = 0; o < 2; ++o) {
-        const float2 u = *y_at(0, i, o), v = *y_at(1, i, o), w = *y_at(2, i, o);
+        const int at = 8 * e * (PC / 2) + (o ? c2_b : c2);
+        const float2 u = sum[at], v = sum[at + S::Y / 8], w = sum[at + 2 * (S::Y / 8)], x = sum[at + 3 * (S::Y / 8)];
         if (p0 + pw * 16 + o * 8 < p.P)
-          *(float2*)(dst + o * 8) = make_float2(fmaf(own[e], (mine[o][2 * e] + u.x) + (v.x + w.x), z[o][2 * e]),
-                                                fmaf(own[e], (mine[o][2 * e + 1] + u.y) + (v.y + w.y), z[o][2 * e + 1]));
+          *(float2*)(y_at + (e ? 8 * (int64_t)inner : 0) + o * 8) =
+              make_float2(fmaf(own[e], (u.x + v.x) + (w.x + x.x), z[o][2 * e]), fmaf(own[e], (u.y + v.y) + (w.y + x.y), z[o][2 * e + 1]));
       }
     }
+    gram_at += p.G * 640;
+    y_at += L * (int64_t)inner;
   }
 #pragma unroll
   for (int t = 0; t < NT; ++t)
@@ -358,7 +359,7 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
 }
 
 // silu(conv(xbc) + bias) in bf16: a thread takes four channels of CB tokens, the rows it reads all requested before the first is used
-constexpr int CB = 16;
+constexpr int CB = 8;
 template <int TAPS>
 __global__ void __launch_bounds__(128) ss_conv_kernel(const bf16* __restrict__ xbc, int64_t ldx, const bf16* __restrict__ w, const bf16* __restrict__ bias,
                                                       const bf16* __restrict__ ring_all, const int* __restrict__ q_start, const int* __restrict__ kv_len,
