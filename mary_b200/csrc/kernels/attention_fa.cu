@@ -17,6 +17,7 @@
 //             in the un-swizzled K-major core-matrix layout, finally O / l to global memory.
 // Blocks of keys that no row of the tile can see (beyond the causal diagonal, before the window) are never loaded.
 // All waits are bounded; a wait that runs out sets the status word, frees TMEM and returns.
+#include "attention_form.cuh"
 #include "common.cuh"
 #include "host_utils.h"
 
@@ -34,11 +35,14 @@ constexpr float RESCALE_THRESHOLD = 8.0f;
 // weights keep 16 significant bits; two P V products per block.
 // BIAS: a bias by distance is added to the scaled score.  Every softmax warp copies the 95 values that its rows can meet in a block to
 // shared memory, minus infinity outside the window and after the query, so the bias is the mask as well.
-template <int DK, int DV, bool SPLITP, bool BIAS>
+// MAPS = 1 or 2 makes the kernel honour FaParams::f (0: plain attention).  With two maps (query and key rows [map 0 | map 1], DK each) the
+// tile walks its key blocks once per map, into accumulators of their own, and a row's thread forms the difference and its norm at the end.
+template <int DK, int DV, bool SPLITP, bool BIAS, int MAPS>
 struct FaCfg {
+  static constexpr int NM = MAPS == 2 ? 2 : 1;
   static constexpr int NCK = DK / CHUNK, NCV = DV / CHUNK;
   static constexpr int Q_CHUNK_BYTES = TR * 128;
-  static constexpr int Q_BYTES = NCK * Q_CHUNK_BYTES;
+  static constexpr int Q_BYTES = NM * NCK * Q_CHUNK_BYTES;
   static constexpr int K_CHUNK_BYTES = KB * 128, V_CHUNK_BYTES = KB * 128;
   static constexpr int K_STAGE = NCK * K_CHUNK_BYTES, V_STAGE = NCV * V_CHUNK_BYTES;
   static constexpr int STAGES = (DK + DV > 384) ? 2 : 3;
@@ -46,7 +50,8 @@ struct FaCfg {
   static constexpr int BIAS_BYTES = BIAS ? 4 * 96 * 4 : 0;
   static constexpr int P_STAGE = SPLITP ? 2 * P_BYTES : P_BYTES;
   static constexpr int SMEM = Q_BYTES + STAGES * (K_STAGE + V_STAGE) + NPBUF * P_STAGE + BIAS_BYTES + 1024 + 256;
-  static constexpr int TMEM_COLS = DV <= 128 ? 256 : 512;     // S: 2 x 64 columns at 0..127, O: DV columns at 128..
+  static constexpr int TMEM_COLS = 128 + NM * DV <= 256 ? 256 : 512;     // S: 2 x 64 columns at 0..127, O: DV columns per map at 128..
+  static_assert(128 + NM * DV <= 512 && !(BIAS && MAPS), "accumulator columns");
   static_assert(DK % CHUNK == 0 && DV % CHUNK == 0 && DV <= 256 && DK <= 256, "head dims: multiples of 64 up to 256");
   static_assert(SMEM <= 232448, "shared memory budget");
 };
@@ -60,8 +65,16 @@ struct FaParams {
   const float* bias;       // BIAS: [Hq][window] by distance, added to the scaled score
   const __nv_bfloat16* gate;   // rows of gate_ld elements, head h at h * DV: the output times its logistic function; or null
   int64_t gate_ld;
+  MaryAttnForm f;
   int* status;
 };
+
+// Two values at a time through the packed 32-bit pipes: a * b + c.
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(*(const uint64_t*)&a), "l"(*(const uint64_t*)&b), "l"(*(const uint64_t*)&c));
+  return *(float2*)&d;
+}
 
 __device__ __forceinline__ uint64_t fa_desc_kmajor_noswz(uint32_t addr, uint32_t lbo_bytes, uint32_t sbo_bytes) {
   return (uint64_t)((addr >> 4) & 0x3FFF) | ((uint64_t)(lbo_bytes >> 4) << 16) | ((uint64_t)(sbo_bytes >> 4) << 32) | (1ull << 46);
@@ -71,11 +84,12 @@ __device__ __forceinline__ uint64_t fa_desc_mnmajor_sw128(uint32_t addr, uint32_
          (2ull << 61);
 }
 
-template <int DK, int DV, bool SPLITP, bool BIAS>
+template <int DK, int DV, bool SPLITP, bool BIAS, int MAPS>
 __global__ void __launch_bounds__(NTHREADS, 1)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                   const __grid_constant__ CUtensorMap tm_v, const FaParams p) {
-  using C = FaCfg<DK, DV, SPLITP, BIAS>;
+  using C = FaCfg<DK, DV, SPLITP, BIAS, MAPS>;
+  constexpr int NM = C::NM;
   constexpr int STAGES = C::STAGES, NPBUF = C::NPBUF;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~uintptr_t(1023));
@@ -105,9 +119,11 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
   const int kvlen = p.kv_len[seq];
   const int pos_first = kvlen - (seq_tok1 - seq_tok0) + (tok0 - seq_tok0);   // position of the tile's first query token
   const int k_hi = pos_first + nrows;                                         // keys [0, k_hi) are visible to some row
-  const int k_lo = p.window > 0 ? max(0, pos_first - p.window + 1) : 0;
+  int k_lo = p.window > 0 ? max(0, pos_first - p.window + 1) : 0;
+  if constexpr (MAPS > 0) k_lo = max(k_lo, first_key(p.f, pos_first));
   const int b_lo = k_lo / KB, b_hi = (k_hi + KB - 1) / KB;
   const int nblk = max(0, b_hi - b_lo);
+  const int ntot = NM * nblk;                      // key blocks to go through, map after map
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -134,7 +150,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       const bool isK = warp == 0;
       if (isK && lane == 0) {
         mbar_expect_tx(q_full, C::Q_BYTES);
-        for (int c = 0; c < C::NCK; ++c) tma_load_2d(sQ + c * C::Q_CHUNK_BYTES, &tm_q, q_full, head * DK + c * CHUNK, tok0);
+        for (int c = 0; c < NM * C::NCK; ++c) tma_load_2d(sQ + c * C::Q_CHUNK_BYTES, &tm_q, q_full, head * NM * DK + c * CHUNK, tok0);
       }
       const int* pt = p.page_table + (int64_t)seq * p.max_pages;
       uint64_t* full = isK ? k_full : v_full;
@@ -145,7 +161,10 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       const int hd = isK ? DK : DV;
       const CUtensorMap* tm = isK ? &tm_k : &tm_v;
       int stage = 0; uint32_t phase = 0;
-      for (int b = b_lo; b < b_hi; ++b) {
+      for (int i = 0; i < ntot; ++i) {
+        const bool second = NM == 2 && i >= nblk;
+        const int b = b_lo + (second ? i - nblk : i);
+        const int row_head = isK ? kvh * NM + (second ? 1 : 0) : kvh;        // heads of hd values along a token's cache row
         int ok = 1;
         if (lane == 0) {
           ok = mbar_wait(&empty[stage], phase ^ 1, abort_flag, p.status, MARY_ERR_TIMEOUT_TMA) ? 1 : 0;
@@ -157,7 +176,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
           if (lane == 0) {
             const int key0 = b * KB;
             const int page = (key0 < kvlen) ? pt[key0 / KB] : pt[0];
-            tma_load_4d(ring + stage * stage_bytes, tm, &full[stage], 0, 0, kvh * nchunk, page);
+            tma_load_4d(ring + stage * stage_bytes, tm, &full[stage], 0, 0, row_head * nchunk, page);
           }
         } else
         // (KB / PAGE) pages x nchunk chunks operations of [16 tokens x 64 dims] (2 KB each), spread over the lanes
@@ -165,7 +184,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
           const int pg = op / nchunk, c = op % nchunk;
           const int key0 = b * KB + pg * PAGE;
           const int page = (key0 < kvlen) ? pt[key0 / PAGE] : pt[0];     // pages past the end: any valid page (masked)
-          tma_load_3d(ring + stage * stage_bytes + c * (KB * 128) + pg * (PAGE * 128), tm, &full[stage], kvh * hd + c * CHUNK, 0, page);
+          tma_load_3d(ring + stage * stage_bytes + c * (KB * 128) + pg * (PAGE * 128), tm, &full[stage], row_head * hd + c * CHUNK, 0, page);
         }
         __syncwarp();
         if (++stage == STAGES) { stage = 0; phase ^= 1; }
@@ -183,11 +202,12 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
         if (!mbar_wait(&k_full[stage], (i / STAGES) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_TMA)) return false;
         tc_fence_after();
         const uint32_t kb_addr = smem_u32(sK + stage * C::K_STAGE);
+        const uint32_t qm_addr = q_addr + (NM == 2 && i >= nblk ? C::NCK * C::Q_CHUNK_BYTES : 0);
 #pragma unroll
         for (int c = 0; c < C::NCK; ++c) {
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
-            umma_f16(tmem_S + sb * KB, umma_desc_sw128(q_addr + c * C::Q_CHUNK_BYTES + k * 32),
+            umma_f16(tmem_S + sb * KB, umma_desc_sw128(qm_addr + c * C::Q_CHUNK_BYTES + k * 32),
                      umma_desc_sw128(kb_addr + c * C::K_CHUNK_BYTES + k * 32), idesc_s, (c > 0 || k > 0) ? 1u : 0u);
           }
         }
@@ -196,29 +216,32 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
         return true;
       };
       if (!issue_qk(0)) goto done;
-      if (nblk > 1 && !issue_qk(1)) goto done;
-      for (int i = 0; i < nblk; ++i) {
+      if (ntot > 1 && !issue_qk(1)) goto done;
+      for (int i = 0; i < ntot; ++i) {
         const int pb = i % NPBUF, stage = i % STAGES;
         if (!mbar_wait(&v_full[stage], (i / STAGES) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_TMA)) goto done;
         if (!mbar_wait(&p_full[pb], (i / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
         tc_fence_after();
         const uint32_t vb_addr = smem_u32(sV + stage * C::V_STAGE);
+        const bool second = NM == 2 && i >= nblk;
+        const uint32_t om = tmem_O + (second ? DV : 0);
+        const int i0 = second ? nblk : 0;
 #pragma unroll
         for (int kk = 0; kk < KB / 16; ++kk) {
           // A = P[:, 16 keys] (K-major, no swizzle: the two 16-byte key chunks of one MMA TR*16 bytes apart, 8-row groups
           // 128 bytes apart); B = V^T of those keys (MN-major, 128B swizzle: 64-dim groups one chunk apart, 8-key groups 1 KB apart)
-          umma_f16(tmem_O, fa_desc_kmajor_noswz(p_addr + pb * C::P_STAGE + kk * 2 * (TR * 16), TR * 16, 128),
-                   fa_desc_mnmajor_sw128(vb_addr + kk * 16 * 128, C::V_CHUNK_BYTES, 1024), idesc_o, (i > 0 || kk > 0) ? 1u : 0u);
+          umma_f16(om, fa_desc_kmajor_noswz(p_addr + pb * C::P_STAGE + kk * 2 * (TR * 16), TR * 16, 128),
+                   fa_desc_mnmajor_sw128(vb_addr + kk * 16 * 128, C::V_CHUNK_BYTES, 1024), idesc_o, (i > i0 || kk > 0) ? 1u : 0u);
         }
         if constexpr (SPLITP) {
 #pragma unroll
           for (int kk = 0; kk < KB / 16; ++kk)
-            umma_f16(tmem_O, fa_desc_kmajor_noswz(p_addr + pb * C::P_STAGE + P_BYTES + kk * 2 * (TR * 16), TR * 16, 128),
+            umma_f16(om, fa_desc_kmajor_noswz(p_addr + pb * C::P_STAGE + P_BYTES + kk * 2 * (TR * 16), TR * 16, 128),
                      fa_desc_mnmajor_sw128(vb_addr + kk * 16 * 128, C::V_CHUNK_BYTES, 1024), idesc_o, 1u);
         }
         umma_commit(&v_empty[stage]);
         umma_commit(&pv_done[pb]);
-        if (i + 2 < nblk && !issue_qk(i + 2)) goto done;
+        if (i + 2 < ntot && !issue_qk(i + 2)) goto done;
       }
     }
   } else if (nblk > 0) {
@@ -227,12 +250,23 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
     const int r = q4 * 32 + lane;
     const bool row_ok = r < nrows;
     const int qpos = pos_first + r;
-    const int lo_key = p.window > 0 ? qpos - p.window + 1 : 0;
+    int lo_key = p.window > 0 ? qpos - p.window + 1 : 0;
+    float sl2 = p.scale_log2;                        // this row's factor on the raw scores
+    int full_from = p.window > 0 ? pos_first + TR - p.window : 0;      // blocks from this key on are inside every row's window and chunk
+    if constexpr (MAPS > 0) {
+      lo_key = max(lo_key, first_key(p.f, qpos));
+      sl2 *= query_temperature(p.f, qpos);
+      full_from = max(full_from, first_key(p.f, pos_first + TR - 1));
+    }
     const uint32_t lane_off = (uint32_t)(q4 * 32) << 16;
-    float m_ref = -INFINITY, l = 0.f;
+    float m_ref = -INFINITY, l = 0.f, l_first = 0.f;
     float* const bias_row = (float*)(sP + NPBUF * C::P_STAGE) + q4 * 96;
-    for (int i = 0; i < nblk; ++i) {
+    for (int i = 0; i < ntot; ++i) {
       const int sb = i % NSBUF, pb = i % NPBUF;
+      const bool second = NM == 2 && i >= nblk;
+      const int i0 = second ? nblk : 0;
+      const uint32_t om = tmem_O + (second ? DV : 0);
+      if (NM == 2 && i == nblk) { l_first = l; l = 0.f; m_ref = -INFINITY; }
       if constexpr (BIAS) {
         // bias_row[d]: rows q4 * 32 + lane and keys j of the block with distance base + d, d = 63 + lane - j
         const int base = pos_first + q4 * 32 - (b_lo + i) * KB - (KB - 1);
@@ -254,13 +288,42 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[sb]);
-      const int key0 = (b_lo + i) * KB;
+      const int key0 = (b_lo + i - i0) * KB;
       // A block that every row of the tile sees entirely (all blocks left of the diagonal band and inside the window) takes the
       // short path: no per-element mask, the maximum on the raw scores, one fused multiply-add and one exponential per element.
       // A thread owns one query row and walks its 64 scores in sequence, so this loop's instruction count bounds the block rate.
-      const bool full_blk = key0 + KB - 1 <= pos_first && (p.window <= 0 || key0 >= pos_first + TR - p.window);
-      const float* sf = (const float*)sr;
+      const bool full_blk = key0 + KB - 1 <= pos_first && key0 >= full_from && (MAPS == 0 || sl2 > 0.f);
       float mx;
+      if constexpr (MAPS > 0) {
+        if (p.f.cap > 0.f) {
+          // the capped score in units of log2: small arguments (all of a warp's) by the series of tanh, two scores at a time
+          float top = 0.f;
+#pragma unroll
+          for (int j = 0; j < KB; ++j) top = fmaxf(top, fabsf(__uint_as_float(sr[j])));
+          const float k = sl2 / (p.f.cap * 1.4426950408889634f);             // raw score -> argument of tanh
+          if (__all_sync(0xffffffffu, top * fabsf(k) <= 0.25f)) {
+            const float k2 = k * k, c1 = sl2, c3 = c1 * k2 * (-1.0f / 3.0f), c5 = c1 * k2 * k2 * (2.0f / 15.0f);
+            const float c7 = c1 * k2 * k2 * k2 * (-17.0f / 315.0f), c9 = c1 * k2 * k2 * k2 * k2 * (62.0f / 2835.0f);
+            const float2 zero = make_float2(0.f, 0.f);
+#pragma unroll
+            for (int j = 0; j < KB; j += 2) {
+              const float2 x = make_float2(__uint_as_float(sr[j]), __uint_as_float(sr[j + 1])), y = fma2(x, x, zero);
+              float2 q = fma2(y, make_float2(c9, c9), make_float2(c7, c7));
+              q = fma2(q, y, make_float2(c5, c5));
+              q = fma2(q, y, make_float2(c3, c3));
+              q = fma2(q, y, make_float2(c1, c1));
+              q = fma2(q, x, zero);
+              sr[j] = __float_as_uint(q.x);
+              sr[j + 1] = __float_as_uint(q.y);
+            }
+          } else {
+            const float c = p.f.cap * 1.4426950408889634f;
+#pragma unroll
+            for (int j = 0; j < KB; ++j) sr[j] = __float_as_uint(c * tanh_32(__uint_as_float(sr[j]) * k));
+          }
+        }
+      }
+      const float sc = MAPS > 0 && p.f.cap > 0.f ? 1.0f : sl2;               // factor on what `sr` now holds
       if constexpr (BIAS) {
         mx = -INFINITY;
 #pragma unroll
@@ -270,17 +333,17 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
           mx = fmaxf(mx, v);
         }
       } else if (full_blk) {
-        mx = sf[0];
+        mx = __uint_as_float(sr[0]);
 #pragma unroll
-        for (int j = 1; j < KB; ++j) mx = fmaxf(mx, sf[j]);
-        mx *= p.scale_log2;
+        for (int j = 1; j < KB; ++j) mx = fmaxf(mx, __uint_as_float(sr[j]));
+        mx *= sc;
       } else {
         mx = -INFINITY;
 #pragma unroll
         for (int j = 0; j < KB; ++j) {
           const int kj = key0 + j;
           const bool ok = row_ok && kj <= qpos && kj >= lo_key;
-          const float v = ok ? __uint_as_float(sr[j]) * p.scale_log2 : -INFINITY;
+          const float v = ok ? __uint_as_float(sr[j]) * sc : -INFINITY;
           sr[j] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
@@ -295,8 +358,8 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
         const float nm = -m_ref;
 #pragma unroll
         for (int j = 0; j < KB / 2; ++j) {
-          const float a = exp2f(fmaf(sf[2 * j], p.scale_log2, nm));
-          const float b = exp2f(fmaf(sf[2 * j + 1], p.scale_log2, nm));
+          const float a = exp2f(fmaf(__uint_as_float(sr[2 * j]), sc, nm));
+          const float b = exp2f(fmaf(__uint_as_float(sr[2 * j + 1]), sc, nm));
           __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
           pw[j] = *(uint32_t*)&h;
           if constexpr (SPLITP) {
@@ -325,19 +388,19 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
         }
       }
       l = l * corr + psum;
-      if (__any_sync(0xffffffffu, need && !first) && i > 0) {
+      if (__any_sync(0xffffffffu, need && !first) && i > i0) {
         // O may only be touched once the previous P V has completed
         if (!mbar_wait(&pv_done[(i - 1) % NPBUF], ((i - 1) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
         tc_fence_after();
 #pragma unroll 1
         for (int c0 = 0; c0 < DV; c0 += 32) {
           uint32_t o[32];
-          tmem_ld_32x32b_x32(tmem_O + lane_off + c0, o);
+          tmem_ld_32x32b_x32(om + lane_off + c0, o);
           tmem_ld_wait();
 #pragma unroll
           for (int j = 0; j < 32; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * corr);
 #pragma unroll
-          for (int j = 0; j < 32; j += 8) tmem_st_32x32b_x8(tmem_O + lane_off + c0 + j, o + j);
+          for (int j = 0; j < 32; j += 8) tmem_st_32x32b_x8(om + lane_off + c0 + j, o + j);
         }
         tmem_st_wait();
       }
@@ -360,9 +423,51 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       if (lane == 0) mbar_arrive(&p_full[pb]);
     }
     // ------------------------------------------------------------------ write out
-    if (!mbar_wait(&pv_done[(nblk - 1) % NPBUF], ((nblk - 1) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+    if (!mbar_wait(&pv_done[(ntot - 1) % NPBUF], ((ntot - 1) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
     tc_fence_after();
-    const float inv_l = l > 0.f ? 1.f / l : 0.f;
+    if constexpr (MAPS == 1) {
+      if (p.f.sink) l += exp2f(fmaf(p.f.sink[head], 1.4426950408889634f, -m_ref));
+    }
+    float inv_l = l > 0.f ? 1.f / l : 0.f;
+    if constexpr (NM == 2) {
+      // o = a0 - mix * a1 as w0 * O0 + w1 * O1, then the norm over the row's DV values
+      float w0 = l_first > 0.f ? 1.f / l_first : 0.f, w1 = -p.f.mix * inv_l, ss = 0.f;
+#pragma unroll 1
+      for (int c0 = 0; c0 < DV; c0 += 32) {
+        uint32_t a[32], b[32];
+        tmem_ld_32x32b_x32(tmem_O + lane_off + c0, a);
+        tmem_ld_32x32b_x32(tmem_O + lane_off + DV + c0, b);
+        tmem_ld_wait();
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+          const float v = fmaf(w1, __uint_as_float(b[j]), w0 * __uint_as_float(a[j]));
+          ss = fmaf(v, v, ss);
+        }
+      }
+      const float c = p.f.post * rsqrtf(ss / DV + p.f.eps);
+      w0 *= c;
+      w1 *= c;
+#pragma unroll 1
+      for (int c0 = 0; c0 < DV; c0 += 32) {
+        uint32_t a[32], b[32];
+        tmem_ld_32x32b_x32(tmem_O + lane_off + c0, a);
+        tmem_ld_32x32b_x32(tmem_O + lane_off + DV + c0, b);
+        tmem_ld_wait();
+        if (row_ok) {
+          uint4 w[4];
+          uint32_t* wp = (uint32_t*)w;
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            __nv_bfloat162 h = __floats2bfloat162_rn(fmaf(w1, __uint_as_float(b[2 * j]), w0 * __uint_as_float(a[2 * j])),
+                                                     fmaf(w1, __uint_as_float(b[2 * j + 1]), w0 * __uint_as_float(a[2 * j + 1])));
+            wp[j] = *(uint32_t*)&h;
+          }
+          uint4* dst = (uint4*)(p.out + (int64_t)(tok0 + r) * p.out_ld + head * DV + c0);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) dst[j] = w[j];
+        }
+      }
+    } else
 #pragma unroll 1
     for (int c0 = 0; c0 < DV; c0 += 32) {
       uint32_t o[32];
@@ -427,12 +532,12 @@ int make_cache_map(CUtensorMap* m, const void* cache, int heads, int hd, int num
   return r == CUDA_SUCCESS ? MARY_OK : MARY_ERR_CUDA;
 }
 
-template <int DK, int DV, bool SPLITP, bool BIAS>
+template <int DK, int DV, bool SPLITP, bool BIAS, int MAPS = 0>
 int launch_fa(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const FaParams& p, int NB, cudaStream_t s) {
   static MarySmemSlots smem_set = {};
-  constexpr int SMEM = FaCfg<DK, DV, SPLITP, BIAS>::SMEM;
-  if (int rc = mary_ensure_dyn_smem((const void*)fa_prefill_kernel<DK, DV, SPLITP, BIAS>, SMEM, &smem_set)) return rc;
-  fa_prefill_kernel<DK, DV, SPLITP, BIAS><<<dim3(NB, p.Hq), NTHREADS, SMEM, s>>>(tq, tk, tv, p);
+  constexpr int SMEM = FaCfg<DK, DV, SPLITP, BIAS, MAPS>::SMEM;
+  if (int rc = mary_ensure_dyn_smem((const void*)fa_prefill_kernel<DK, DV, SPLITP, BIAS, MAPS>, SMEM, &smem_set)) return rc;
+  fa_prefill_kernel<DK, DV, SPLITP, BIAS, MAPS><<<dim3(NB, p.Hq), NTHREADS, SMEM, s>>>(tq, tk, tv, p);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }
@@ -446,24 +551,34 @@ MARY_API int mary_attention_prefill_supported(int DK, int DV) {
   return (DK == 64 && DV == 64) || (DK == 128 && DV == 128) || (DK == 192 && DV == 128) || (DK == 256 && DV == 256);
 }
 
+// The same for two maps of DK values each.
+MARY_API int mary_attention_prefill_maps_supported(int DK, int DV) {
+  return (DK == 64 && DV == 64) || (DK == 64 && DV == 128) || (DK == 128 && DV == 128);
+}
+
 // q [T, Hq, DK] bf16 contiguous; kcache [pages, page_size (16 or 64), Hkv, DK] and vcache [.., Hkv, DV] bf16 with element strides per token
 // and per page (heads contiguous inside a token row); out [T, Hq, DV] bf16.  blk_seq / blk_tok0: NB tiles of at most 128 query
 // tokens that never cross a sequence.  Causal with the last query token of a sequence at position kv_len - 1; window > 0 keeps
 // keys (pos - window, pos].  out_ld: elements between the output rows of two tokens (0: Hq * DV; a multiple of 8).  split_p: softmax
 // weights with 16 significant bits.  bias [Hq][window] (or null; with split_p and equal widths only) is added to the scaled score by
-// distance, gate (or null; 16-byte aligned rows) multiplies the output by its logistic function.  Returns MARY_ERR_BAD_ARG for head dims without an instantiation.
+// distance, gate (or null; 16-byte aligned rows) multiplies the output by its logistic function.  form (or null; with split_p, without bias): see attention_form.cuh; with two
+// maps query and key rows have 2 DK values per head and T may exceed a row's pitch as form->q_ld says.  Returns MARY_ERR_BAD_ARG for head dims without an instantiation.
 MARY_API int mary_attention_prefill(const void* q, const void* kcache, const void* vcache, void* out, const int* page_table,
                                     const int* kv_len, const int* q_start, const int* blk_seq, const int* blk_tok0, int NB, int T, int Hq,
                                     int Hkv, int DK, int DV, int num_pages, int max_pages, int64_t k_tok_stride, int64_t k_page_stride,
                                     int64_t v_tok_stride, int64_t v_page_stride, int window, float scale, int page_size,
-                                    int64_t out_ld, int split_p, const float* bias, const void* gate, int64_t gate_ld, cudaStream_t s) {
+                                    int64_t out_ld, int split_p, const float* bias, const void* gate, int64_t gate_ld, const MaryAttnForm* form, cudaStream_t s) {
   if (NB <= 0) return MARY_OK;
-  if (!mary_attention_prefill_supported(DK, DV) || Hkv < 1 || Hq % Hkv || (page_size != PAGE && page_size != KB)) return MARY_ERR_BAD_ARG;
+  const int maps = form && form->maps == 2 ? 2 : 1;
+  if (form && (form->maps > 2 || !split_p || bias || (maps == 2 && (gate || form->sink)))) return MARY_ERR_BAD_ARG;
+  if (!(maps == 2 ? mary_attention_prefill_maps_supported(DK, DV) : mary_attention_prefill_supported(DK, DV)) || Hkv < 1 || Hq % Hkv || (page_size != PAGE && page_size != KB)) return MARY_ERR_BAD_ARG;
   if ((k_tok_stride * 2) % 16 || (k_page_stride * 2) % 16 || (v_tok_stride * 2) % 16 || (v_page_stride * 2) % 16) return MARY_ERR_BAD_ARG;
   CUtensorMap tq, tk, tv;
-  int rc = mary_make_tmap_2d(&tq, q, 4, (uint64_t)T, (uint64_t)Hq * DK, (uint64_t)Hq * DK, TR, CHUNK, 1);
+  const uint64_t q_ld = form && form->q_ld > 0 ? (uint64_t)form->q_ld : (uint64_t)Hq * maps * DK;
+  if (q_ld % 8 || ((uintptr_t)q & 15)) return MARY_ERR_BAD_ARG;
+  int rc = mary_make_tmap_2d(&tq, q, 4, (uint64_t)T, (uint64_t)Hq * maps * DK, q_ld, TR, CHUNK, 1);
   if (rc) return rc;
-  if ((rc = make_cache_map(&tk, kcache, Hkv, DK, num_pages, k_tok_stride, k_page_stride, page_size))) return rc;
+  if ((rc = make_cache_map(&tk, kcache, Hkv * maps, DK, num_pages, k_tok_stride, k_page_stride, page_size))) return rc;
   if ((rc = make_cache_map(&tv, vcache, Hkv, DV, num_pages, v_tok_stride, v_page_stride, page_size))) return rc;
   FaParams p;
   p.page_table = page_table; p.kv_len = kv_len; p.q_start = q_start; p.blk_seq = blk_seq; p.blk_tok0 = blk_tok0;
@@ -473,6 +588,18 @@ MARY_API int mary_attention_prefill(const void* q, const void* kcache, const voi
   if (p.out_ld % 8 || ((uintptr_t)out & 15) || gate_ld % 8 || ((uintptr_t)gate & 15)) return MARY_ERR_BAD_ARG;
   if (bias && (!split_p || DK != DV || window < 1)) return MARY_ERR_BAD_ARG;
   p.scale_log2 = scale * 1.4426950408889634f; p.status = mary_status_ptr();
+  p.f = form ? *form : MaryAttnForm{};
+  if (maps == 2) {
+    if (DV == 64) return launch_fa<64, 64, true, false, 2>(tq, tk, tv, p, NB, s);
+    if (DK == 64) return launch_fa<64, 128, true, false, 2>(tq, tk, tv, p, NB, s);
+    return launch_fa<128, 128, true, false, 2>(tq, tk, tv, p, NB, s);
+  }
+  if (form && (p.f.chunk > 0 || p.f.sink || p.f.temp_every > 0 || p.f.cap > 0.f)) {
+    if (DK == 64) return launch_fa<64, 64, true, false, 1>(tq, tk, tv, p, NB, s);
+    if (DK == 128) return launch_fa<128, 128, true, false, 1>(tq, tk, tv, p, NB, s);
+    if (DK == 192) return launch_fa<192, 128, true, false, 1>(tq, tk, tv, p, NB, s);
+    return launch_fa<256, 256, true, false, 1>(tq, tk, tv, p, NB, s);
+  }
   if (bias) {
     if (DK == 64) return launch_fa<64, 64, true, true>(tq, tk, tv, p, NB, s);
     if (DK == 128) return launch_fa<128, 128, true, true>(tq, tk, tv, p, NB, s);

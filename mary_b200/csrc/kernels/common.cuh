@@ -247,8 +247,15 @@ __device__ __forceinline__ float situ_f(float g, float u) {
   const float beta = 4.0f, lb = 25.0f;
   return beta * tanhf(g / beta) * (1.0f / (1.0f + __expf(-g))) * (lb * tanhf(u / lb));
 }
-// act: 0 = GeGLU(tanh), 1 = SwiGLU, 2 = SiTU
-__device__ __forceinline__ float glu_f(int act, float g, float u) {
+// gate capped from above, up clamped to both sides and shifted by one, logistic gate with slope 1.702
+__device__ __forceinline__ float clamped_glu_f(float g, float u, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+}
+// act: 0 = GeGLU(tanh), 1 = SwiGLU, 2 = SiTU, 3 = clamped (limit)
+__device__ __forceinline__ float glu_f(int act, float g, float u, float limit = 0.f) {
+  if (act == 3) return clamped_glu_f(g, u, limit);
   return act == 0 ? gelu_tanh_f(g) * u : (act == 1 ? silu_f(g) * u : situ_f(g, u));
 }
 

@@ -143,7 +143,8 @@ __global__ void norm_add_norm_kernel(const TI* __restrict__ a, const __nv_bfloat
   }
 }
 
-__global__ void glu_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out, int F, int64_t n, int act) {
+__global__ void glu_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out, int64_t ld, int F, int64_t n, int act,
+                           float limit) {
   pdl_sync();
   int64_t idx = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * 8;
   if (idx >= n) return;
@@ -157,9 +158,9 @@ __global__ void glu_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* 
 #pragma unroll
   for (int j = 0; j < 4; ++j) {
     float2 gf = __bfloat1622float2(gp[j]), uf = __bfloat1622float2(up[j]);
-    op[j] = __floats2bfloat162_rn(glu_f(act, gf.x, uf.x), glu_f(act, gf.y, uf.y));
+    op[j] = __floats2bfloat162_rn(glu_f(act, gf.x, uf.x, limit), glu_f(act, gf.y, uf.y, limit));
   }
-  *(uint4*)(out + idx) = o;
+  *(uint4*)(out + t * ld + f) = o;
 }
 
 __global__ void embed_kernel(const int* __restrict__ ids, const __nv_bfloat16* __restrict__ table, __nv_bfloat16* __restrict__ out,
@@ -303,12 +304,14 @@ MARY_API int mary_norm_add_norm(const void* a, int a_is_f32, const void* w_post,
   return MARY_OK;
 }
 
-MARY_API int mary_glu(const void* gu, void* out, int T, int F, int act, cudaStream_t s) {
+// ld: elements between output rows (0: F)
+MARY_API int mary_glu(const void* gu, void* out, int64_t ld, int T, int F, int act, float limit, cudaStream_t s) {
   if (T <= 0) return MARY_OK;
-  if (F % 8) return MARY_ERR_BAD_ARG;
+  if (ld <= 0) ld = F;
+  if (F % 8 || ld % 8 || ((uintptr_t)out & 15)) return MARY_ERR_BAD_ARG;
   int64_t n = (int64_t)T * F;
   int blocks = (int)((n / 8 + NT - 1) / NT);
-  MARY_LAUNCH(glu_kernel, blocks, NT, 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, F, n, act);
+  MARY_LAUNCH(glu_kernel, blocks, NT, 0, s, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ld, F, n, act, limit);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }

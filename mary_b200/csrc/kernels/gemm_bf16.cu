@@ -37,6 +37,7 @@ struct GemmParams {
   int tiles_r, tiles_c, split_k, k_blocks_per_split, k_blocks;
   int glu_offset;            // rows between the gate tile and the up tile of the weight operand (GLU only)
   int act;
+  float glu_limit;           // of the clamped GLU
   int epi;
   int swap;                  // 1: row operand = weights, D[i][j] -> out[j * ldo + i]
   int64_t ldo;
@@ -380,7 +381,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tm_r, const __grid_constant
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
           float a = __uint_as_float(r[j]) * p.alpha;
-          v[j] = GLU ? glu_f(p.act, a, __uint_as_float(r2[j]) * p.alpha) : a;
+          v[j] = GLU ? glu_f(p.act, a, __uint_as_float(r2[j]) * p.alpha, p.glu_limit) : a;
         }
         if (sk) {
           // add this K-slice into the tile's f32 accumulator in scratch (column-major, so a warp's 32 rows are contiguous:
@@ -440,7 +441,7 @@ int launch(const CUtensorMap& tr, const CUtensorMap& tc, const GemmParams& p, cu
 }  // namespace
 
 // out[M, N] (bf16, or f32 for epi 1/2) = alpha * X[M, K] * W[N, K]^T (+ bias[N]).
-//   glu != 0: W holds [gate (N rows) ; up (N rows)] and out = act(gate) * up, act = glu - 1 (0 GeGLU, 1 SwiGLU, 2 SiTU).
+//   glu != 0: W holds [gate (N rows) ; up (N rows)] and out = act(gate) * up, act = glu - 1 (0 GeGLU, 1 SwiGLU, 2 SiTU, 3 clamped by glu_limit).
 //   epi: 0 store bf16, 1 atomically add f32 into `out` (caller zeroes it; required when split_k > 1), 2 store f32.
 //   swap: -1 = choose automatically, 0 = activations are the row operand, 1 = weights are the row operand.
 // Leading dimensions are in elements; all of ldx, ldw must be multiples of 8 and the bases 16-byte aligned.
@@ -473,7 +474,7 @@ static int gemm_impl(const void* X, const void* W, void* out, int M, int N, int 
                      int64_t bsx, int64_t bsw, int64_t bso, const float* bias, float alpha, int glu, int epi, int split_k, int swap,
                      const uint64_t* rs_bufs, int rs_world, int rs_src, int rs_rpr, cudaStream_t stream, float* ws = nullptr,
                      int64_t ws_floats = 0, int* counters = nullptr, int n_counters = 0, bool stream_k = false,
-                     const int* g_tiles = nullptr, const int* g_meta = nullptr, int g_experts = 0, int g_nt = 0);
+                     const int* g_tiles = nullptr, const int* g_meta = nullptr, int g_experts = 0, int g_nt = 0, float glu_limit = 0.f);
 
 // Tells the GEMM launchers called next on THIS thread that their W operand holds constant model weights (1) or may have been
 // written by an earlier kernel of the stream (0, the default).  Only read when programmatic dependent launch is enabled.
@@ -500,7 +501,8 @@ MARY_API int mary_gemm_bf16_rs(const void* X, const void* W, int M, int N, int K
 static int gemm_impl(const void* X, const void* W, void* out, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldo, int batch,
                      int64_t bsx, int64_t bsw, int64_t bso, const float* bias, float alpha, int glu, int epi, int split_k, int swap,
                      const uint64_t* rs_bufs, int rs_world, int rs_src, int rs_rpr, cudaStream_t stream, float* ws, int64_t ws_floats,
-                     int* counters, int n_counters, bool stream_k, const int* g_tiles, const int* g_meta, int g_experts, int g_nt) {
+                     int* counters, int n_counters, bool stream_k, const int* g_tiles, const int* g_meta, int g_experts, int g_nt,
+                     float glu_limit) {
   if (M <= 0 || N <= 0 || K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || batch < 1) return MARY_ERR_BAD_ARG;
   if (split_k < 1) split_k = 1;
   const bool sk_epi = epi == EPI_SK_BF16 || epi == EPI_SK_F32;
@@ -518,6 +520,7 @@ static int gemm_impl(const void* X, const void* W, void* out, int M, int N, int 
   p.split_k = (p.k_blocks + p.k_blocks_per_split - 1) / p.k_blocks_per_split;
   p.glu_offset = N;
   p.act = glu ? glu - 1 : 0;
+  p.glu_limit = glu_limit;
   p.epi = epi;
   p.swap = use_swap ? 1 : 0;
   p.ldo = ldo;
@@ -642,9 +645,10 @@ static int gemm_impl(const void* X, const void* W, void* out, int M, int N, int 
 }
 
 MARY_API int mary_gemm_bf16(const void* X, const void* W, void* out, int M, int N, int K, int64_t ldx, int64_t ldw,
-                            int64_t ldo, const float* bias, float alpha, int glu, int epi, int split_k, int swap,
+                            int64_t ldo, const float* bias, float alpha, int glu, int epi, int split_k, int swap, float glu_limit,
                             cudaStream_t stream) {
-  return mary_gemm_bf16_batched(X, W, out, M, N, K, ldx, ldw, ldo, 1, 0, 0, 0, bias, alpha, glu, epi, split_k, swap, stream);
+  return gemm_impl(X, W, out, M, N, K, ldx, ldw, ldo, 1, 0, 0, 0, bias, alpha, glu, epi, split_k, swap, nullptr, 0, 0, 0, stream, nullptr, 0, nullptr,
+                   0, false, nullptr, nullptr, 0, 0, glu_limit);
 }
 
 // Grouped (mixture-of-experts) GEMM with unquantised expert weights: out[rows_pad, N] = X[rows_pad, K] * W[expert of the row's tile]^T,
@@ -655,10 +659,10 @@ MARY_API int mary_gemm_bf16(const void* X, const void* W, void* out, int M, int 
 // 128-row operand (nt must be 128), the expert's weights the column operand (prefill-sized batches; no GLU epilogue).
 MARY_API int mary_gemm_bf16_grouped(const void* X, const void* W, void* out, int rows_pad, int N, int K, int64_t ldx, int64_t ldw,
                                     int64_t ldo, int E, int64_t bsw, const int* tiles, const int* meta, int nt, int glu, int swap,
-                                    cudaStream_t stream) {
+                                    float glu_limit, cudaStream_t stream) {
   if (!tiles || !meta || E < 1 || (glu && !swap)) return MARY_ERR_BAD_ARG;
   return gemm_impl(X, W, out, rows_pad, N, K, ldx, ldw, ldo, 1, 0, bsw, 0, nullptr, 1.0f, glu, EPI_STORE_BF16, 1, swap ? 1 : 0, nullptr, 0, 0, 0,
-                   stream, nullptr, 0, nullptr, 0, false, tiles, meta, E, nt);
+                   stream, nullptr, 0, nullptr, 0, false, tiles, meta, E, nt, glu_limit);
 }
 
 // Split-K finished inside the kernel, without a zero-fill or a cast pass: out (bf16, or f32 when out_f32) = alpha * X W^T + bias

@@ -11,13 +11,9 @@ namespace {
 constexpr int BM = 64, BN = 64, BK = 16, NT = 256;
 
 template <typename TI, typename TO>
-__global__ void __launch_bounds__(NT) gemm_simt_kernel(const TI* __restrict__ X, const TI* __restrict__ W, TO* __restrict__ out, int M, int N, int K,
-                                                       int64_t ldx, int64_t ldw, int64_t ldo, float alpha, int accumulate, int64_t bsx, int64_t bsw,
-                                                       int64_t bso) {
-  pdl_sync();
-  X += blockIdx.z * bsx; W += blockIdx.z * bsw; out += blockIdx.z * bso;
+__device__ __forceinline__ void simt_tile(const TI* __restrict__ X, const TI* __restrict__ W, TO* __restrict__ out, int M, int N, int K, int64_t ldx,
+                                          int64_t ldw, int64_t ldo, float alpha, int accumulate, int m0, int n0) {
   __shared__ float sx[2][BK][BM + 4], sw[2][BK][BN + 4];
-  const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
   const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
   const int lk = threadIdx.x % BK, lr = threadIdx.x / BK;          // loader: one k, rows lr, lr + 16, ...
   float acc[4][4] = {};
@@ -69,6 +65,27 @@ __global__ void __launch_bounds__(NT) gemm_simt_kernel(const TI* __restrict__ X,
   }
 }
 
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(NT) gemm_simt_kernel(const TI* __restrict__ X, const TI* __restrict__ W, TO* __restrict__ out, int M, int N, int K,
+                                                       int64_t ldx, int64_t ldw, int64_t ldo, float alpha, int accumulate, int64_t bsx, int64_t bsw,
+                                                       int64_t bso) {
+  pdl_sync();
+  simt_tile<TI, TO>(X + blockIdx.z * bsx, W + blockIdx.z * bsw, out + blockIdx.z * bso, M, N, K, ldx, ldw, ldo, alpha, accumulate, blockIdx.y * BM,
+                    blockIdx.x * BN);
+}
+
+// Rows sorted into tiles of one expert each (tiles: {expert, first row, rows, -}, meta[0] of them in use): every tile times its expert's matrix.
+template <typename TI>
+__global__ void __launch_bounds__(NT) gemm_simt_grouped_kernel(const TI* __restrict__ X, const TI* __restrict__ W, TI* __restrict__ out, int N, int K,
+                                                               int64_t ldx, int64_t ldw, int64_t ldo, int E, int64_t bsw, const int* __restrict__ tiles,
+                                                               const int* __restrict__ meta) {
+  pdl_sync();
+  if ((int)blockIdx.y >= meta[0]) return;
+  const int* t = tiles + 4 * blockIdx.y;
+  const int e = min(max(t[0], 0), E - 1);
+  simt_tile<TI, TI>(X + (int64_t)t[1] * ldx, W + e * bsw, out + (int64_t)t[1] * ldo, min(t[2], BM), N, K, ldx, ldw, ldo, 1.0f, 0, 0, blockIdx.x * BN);
+}
+
 }  // namespace
 
 // `batch` products over strided views (element strides bsx / bsw / bso).  x_f32: X and W are f32 (else both bf16); out_f32: out is f32 (else bf16)
@@ -92,4 +109,18 @@ MARY_API int mary_gemm_simt_batched(const void* X, const void* W, void* out, int
 MARY_API int mary_gemm_simt(const void* X, const void* W, void* out, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldo, float alpha,
                             int accumulate, int x_f32, int out_f32, cudaStream_t s) {
   return mary_gemm_simt_batched(X, W, out, M, N, K, ldx, ldw, ldo, 1, 0, 0, 0, alpha, accumulate, x_f32, out_f32, s);
+}
+
+// out[r] = X[r] W[expert of r's tile]^T over the rows of a routing plan with tiles of at most 64 rows (`max_tiles` of them); X, W [E][N][K] (bsw elements
+// between experts) and out have one storage type.
+MARY_API int mary_gemm_simt_grouped(const void* X, const void* W, void* out, int N, int K, int64_t ldx, int64_t ldw, int64_t ldo, int E, int64_t bsw,
+                                    const int* tiles, const int* meta, int max_tiles, int f32, cudaStream_t s) {
+  if (max_tiles <= 0) return MARY_OK;
+  if (N <= 0 || K <= 0 || E < 1 || max_tiles > 65535) return MARY_ERR_BAD_ARG;
+  const dim3 grid((N + BN - 1) / BN, max_tiles);
+  using B = __nv_bfloat16;
+  if (f32) MARY_LAUNCH((gemm_simt_grouped_kernel<float>), grid, NT, 0, s, (const float*)X, (const float*)W, (float*)out, N, K, ldx, ldw, ldo, E, bsw, tiles, meta);
+  else MARY_LAUNCH((gemm_simt_grouped_kernel<B>), grid, NT, 0, s, (const B*)X, (const B*)W, (B*)out, N, K, ldx, ldw, ldo, E, bsw, tiles, meta);
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
 }

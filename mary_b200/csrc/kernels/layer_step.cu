@@ -106,6 +106,7 @@ __device__ __forceinline__ void warp_dot4(const __nv_bfloat16* __restrict__ w, i
 // mode 2: y[n] = silu(W[n] x) * (W[n + N] x)
 // mode 3: y[n] = alpha * W[n] x, y in f32   (what a post-norm consumes)
 // mode 4: y[n] = gelu_tanh(W[n] x) * (W[n + N] x)
+// mode 5: y[n] = clamped GLU of the same two with limit alpha
 __global__ void __launch_bounds__(LS_THREADS) step_matvec_kernel(const __nv_bfloat16* __restrict__ h, const __nv_bfloat16* __restrict__ gain,
                                                                  float eps, const __nv_bfloat16* __restrict__ w, int64_t ldw, int N, int K,
                                                                  const __nv_bfloat16* __restrict__ res, __nv_bfloat16* __restrict__ y, int mode,
@@ -116,8 +117,8 @@ __global__ void __launch_bounds__(LS_THREADS) step_matvec_kernel(const __nv_bflo
   stage_input(h, gain, eps, K, xs, red);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = LS_THREADS / 32;
   const int gw = blockIdx.x * nw + warp, tw = gridDim.x * nw;
-  if (mode == 2 || mode == 4) {
-    const int act = mode == 2 ? 1 : 0;
+  if (mode == 2 || mode >= 4) {
+    const int act = mode == 2 ? 1 : (mode == 4 ? 0 : 3);
     const int pw = rpw >= 2 ? 2 : 1;               // output rows per warp and pass (each is a gate row and an up row)
     for (int n0 = gw * pw; n0 < N; n0 += tw * pw) {
       const int rows[4] = {n0, n0 + N, n0 + 1, n0 + 1 + N};
@@ -125,8 +126,8 @@ __global__ void __launch_bounds__(LS_THREADS) step_matvec_kernel(const __nv_bflo
       float d[4];
       warp_dot4(w, ldw, rows, cnt, xs, K, d, gw);
       if (lane == 0) {
-        y[n0] = __float2bfloat16(glu_f(act, d[0], d[1]));           // on the f32 sums, as the GEMM's GLU epilogue does
-        if (cnt == 4) y[n0 + 1] = __float2bfloat16(glu_f(act, d[2], d[3]));
+        y[n0] = __float2bfloat16(glu_f(act, d[0], d[1], alpha));           // on the f32 sums, as the GEMM's GLU epilogue does
+        if (cnt == 4) y[n0 + 1] = __float2bfloat16(glu_f(act, d[2], d[3], alpha));
       }
     }
   } else {
@@ -285,15 +286,16 @@ __global__ void __launch_bounds__(LS_THREADS) step_attention_kernel(const __nv_b
 }
 }  // namespace
 
-// y[N] = f(W[N (or 2N), K] x) with the stage's folded neighbours (mode: 0 plain, 1 + residual, 2 SwiGLU over [gate; up] rows);
+// y[N] = f(W[N (or 2N), K] x) with the stage's folded neighbours (mode: 0 plain, 1 + residual, 2 SwiGLU over [gate; up] rows,
+// 3 f32 result, 4 GEGLU, 5 clamped GLU);
 // gain != null: x = rms(h) * gain, else x = h.
 MARY_API int mary_step_matvec(const void* h, const void* gain, float eps, const void* w, int64_t ldw, int N, int K, const void* res, void* y,
                               int mode, float alpha, cudaStream_t s) {
-  if (N <= 0 || K <= 0 || (K & 7) || (ldw & 7) || K > LS_MAX_H || mode < 0 || mode > 4 || (mode == 1 && !res)) return MARY_ERR_BAD_ARG;
+  if (N <= 0 || K <= 0 || (K & 7) || (ldw & 7) || K > LS_MAX_H || mode < 0 || mode > 5 || (mode == 1 && !res)) return MARY_ERR_BAD_ARG;
   // rows per warp and pass: as many as still give every SM a CTA (a narrow output with one row per warp fills the machine,
   // a wide one keeps four rows of loads in flight per warp)
   const int sms = mary_num_sms(), nw = LS_THREADS / 32;
-  int rpw = (mode == 2 || mode == 4) ? 2 : 4;
+  int rpw = (mode == 2 || mode >= 4) ? 2 : 4;
   while (rpw > 1 && (N + nw * rpw - 1) / (nw * rpw) < sms) rpw >>= 1;
   int grid = (N + nw * rpw - 1) / (nw * rpw);
   const int cap = 4 * sms;

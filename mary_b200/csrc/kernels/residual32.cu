@@ -102,12 +102,17 @@ __global__ void rmsnorm32_kernel(const float* __restrict__ x, const T* __restric
 }
 
 template <typename T>
-__global__ void glu_any_kernel(const T* __restrict__ gu, T* __restrict__ out, int F, int64_t n, int act) {
+__global__ void glu_any_kernel(const T* __restrict__ gu, T* __restrict__ out, int F, int64_t n, int act, float limit) {
   pdl_sync();
   const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n) return;
   const int64_t t = i / F, f = i % F;
   const float g = to_f<T>(gu[t * 2 * F + f]), u = to_f<T>(gu[t * 2 * F + F + f]);
+  if (act == 3) {
+    const float gl = fminf(g, limit), ul = fminf(fmaxf(u, -limit), limit);
+    out[i] = from_f<T>(gl * sigmoid_x(1.702f * gl) * (ul + 1.0f));
+    return;
+  }
   const float k0 = 0.7978845608028654f, k1 = 0.044715f;
   const float a = act == 0 ? 0.5f * g * (1.0f + tanhf(k0 * (g + k1 * g * g * g))) : silu_x(g);
   out[i] = from_f<T>(a * u);
@@ -295,12 +300,12 @@ MARY_API int mary_rmsnorm32(const float* x, const void* w, void* y, int T_, int 
   return MARY_OK;
 }
 
-// act: 0 = tanh-form GELU, 1 = SiLU; any F
-MARY_API int mary_glu_any(const void* gu, void* out, int T_, int F, int act, int f32, cudaStream_t s) {
+// act: 0 = tanh-form GELU, 1 = SiLU, 3 = clamped by `limit`; any F
+MARY_API int mary_glu_any(const void* gu, void* out, int T_, int F, int act, float limit, int f32, cudaStream_t s) {
   if (T_ <= 0) return MARY_OK;
-  if (act < 0 || act > 1) return MARY_ERR_BAD_ARG;
+  if (act < 0 || act > 3 || act == 2) return MARY_ERR_BAD_ARG;
   const int64_t n = (int64_t)T_ * F;
-  BY_TYPE(f32, MARY_LAUNCH((glu_any_kernel<T>), (unsigned)((n + NT - 1) / NT), NT, 0, s, (const T*)gu, (T*)out, F, n, act));
+  BY_TYPE(f32, MARY_LAUNCH((glu_any_kernel<T>), (unsigned)((n + NT - 1) / NT), NT, 0, s, (const T*)gu, (T*)out, F, n, act, limit));
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }

@@ -1,7 +1,7 @@
 // One CTA (256 threads) routes one token: softmax or sigmoid(+bias) scores, optional group-limited pre-selection, the k best
 // experts with ties going to the lower index, renormalised weights.  Shared by the stand-alone router kernel (select.cu) and
 // the fused route + dispatch kernel of the expert pipeline (ep_fused.cu).
-// Rules: sigmoid+bias selection with unbiased weights (src/models/k3/router.rs:9-15, src/models/inkling/routetopk.rs:112-260),
+// A bias is added to the scores for the choice only.  Rules: sigmoid+bias selection with unbiased weights (src/models/k3/router.rs:9-15, src/models/inkling/routetopk.rs:112-260),
 // softmax top-k with renormalisation (src/models/gemma/gemma4/layers.rs:269-325); the group-limited branch, which the
 // reference refuses (src/models/k3/router.rs:136-143), keeps the `topk_group` groups whose two best biased scores sum highest.
 //
@@ -60,8 +60,8 @@ __device__ __forceinline__ void router_block(const float* __restrict__ row, cons
     sum = 0.f;
 #pragma unroll
     for (int w = 0; w < 8; ++w) sum += S.red[w];
-    if (tid < E) { S.sc[tid] = e0 / sum; S.sel[tid] = e0 / sum; }
-    if (tid + 256 < E) { S.sc[tid + 256] = e1 / sum; S.sel[tid + 256] = e1 / sum; }
+    if (tid < E) { S.sc[tid] = e0 / sum; S.sel[tid] = e0 / sum + (bias ? bias[tid] : 0.f); }
+    if (tid + 256 < E) { S.sc[tid + 256] = e1 / sum; S.sel[tid + 256] = e1 / sum + (bias ? bias[tid + 256] : 0.f); }
   } else {
     if (tid < E) { const float sg = 1.0f / (1.0f + __expf(-v0)); S.sc[tid] = sg; S.sel[tid] = sg + (bias ? bias[tid] : 0.f); }
     if (tid + 256 < E) { const float sg = 1.0f / (1.0f + __expf(-v1)); S.sc[tid + 256] = sg; S.sel[tid + 256] = sg + (bias ? bias[tid + 256] : 0.f); }

@@ -69,7 +69,7 @@ __global__ void argmax_kernel(const float* __restrict__ logits, int64_t ld, int 
   }
 }
 
-// One warp per token.  mode 0: softmax over all experts, top-k, optional renormalisation.
+// One warp per token.  mode 0: softmax over all experts, selection on scores + bias (if any), optional renormalisation.
 // mode 1: scores = sigmoid(logit); selection on scores + bias, optionally limited to the `topk_group` best of
 // `n_group` groups (group score = sum of its two best biased scores); weights = unbiased scores of the chosen,
 // renormalised by (sum + 1e-20), times `scale`.  Ties resolve to the lower index.  A non-finite logit sets *flag.
@@ -102,7 +102,10 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, int64_t ld,
     }
     sum = warp_sum(sum);
 #pragma unroll
-    for (int j = 0; j < MAXE_PER_LANE; ++j) { if (sc[j] != -INFINITY) sc[j] /= sum; sel[j] = sc[j]; }
+    for (int j = 0; j < MAXE_PER_LANE; ++j) {
+      if (sc[j] != -INFINITY) sc[j] /= sum;
+      sel[j] = sc[j] + (bias && lane + 32 * j < E ? bias[lane + 32 * j] : 0.f);
+    }
   } else {
 #pragma unroll
     for (int j = 0; j < MAXE_PER_LANE; ++j) {

@@ -337,3 +337,140 @@ class StateSpaceMixer(nn.Module):
         for mine, theirs in ((self.w_out, "o"), (self.w_taps, "conv"), (self.b_taps, "conv.b"), (self.gain, "norm"), (self.a_log, "A_log"),
                              (self.dt_bias, "dt_bias"), (self.skip, "D")):
             mine.data.copy_(get(p + theirs))
+
+
+def stepped_frequencies(dims: int, base: float, factor: float | None = None, low: float = 0.0, high: float = 0.0, original: float = 0.0):
+    """Rotation frequencies ``[dims / 2]`` in f64.  With a ``factor``: wavelengths below ``original / high`` stay, those above ``original / low`` grow by
+    the factor, between them the two frequencies are blended linearly in ``original / wavelength``."""
+    f = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    if factor is None:
+        return f
+    turns = original * f / (2.0 * math.pi)
+    s = ((turns - low) / (high - low)) if high != low else torch.zeros_like(f)
+    return torch.where(turns > high, f, torch.where(turns < low, f / factor, (1.0 - s) * f / factor + s * f))
+
+
+class JoinedColumns:
+    """Several inputs side by side, every block from a multiple of 8 columns on, for one product with a matrix whose columns are laid out alike
+    (``[b0 | b1 | ..] [W0 | W1 | ..]^T``, the sum of the blocks' products); columns between blocks are zero on both sides."""
+
+    def __init__(self, blocks: dict[str, int]):
+        self.at, n = {}, 0
+        for name, cols in blocks.items():
+            self.at[name] = (n, cols)
+            n += pad8(cols)
+        self.cols, self.gaps = n, any(c % 8 for c in blocks.values())
+
+    def fill(self, weight, name: str, value) -> None:
+        a, n = self.at[name]
+        weight.data[:, a:a + n].copy_(value)
+
+    def buffer(self, rows: int, like):
+        return (torch.zeros if self.gaps else torch.empty)(rows, self.cols, dtype=like.dtype, device=like.device)
+
+    def part(self, buf, name: str):
+        a, n = self.at[name]
+        return buf[:, a:a + n]
+
+
+class CappedAttentionMixer(nn.Module):
+    """Causal attention without rotation: the query scaled by a temperature that grows with the logarithm of the position, the score capped by a
+    hyperbolic tangent, a learned sink per head in the sum of the weights.  Writes the heads' outputs; the output projection is the caller's."""
+
+    def __init__(self, width, heads, kv_heads, dk, dv, scale, cap, temperature, dtype, device):
+        super().__init__()
+        if dk > 640 or dv > 512:
+            raise ValueError(f"head widths {dk}/{dv} exceed what the kernels hold (640/512)")
+        self.heads, self.kv_heads, self.dk, self.dv, self.scale, self.cap, self.temperature = heads, kv_heads, dk, dv, scale, cap, temperature
+        self.proj = FusedProjection(dict(q=heads * dk, k=kv_heads * dk, v=kv_heads * dv))
+        self.w_in = param(self.proj.rows, width, dtype=dtype, device=device)
+        self.sink = param(heads, dtype=torch.float32, device=device)
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.dv
+
+    def kv_spec(self):
+        return self.kv_heads, self.dk, self.dv
+
+    def finish(self) -> None:
+        self.form = ops.AttentionForm(cap=self.cap, sink=self.sink.data, temperature=self.temperature)
+
+    def forward(self, x, meta, kc, vc, out):
+        y = ops.linear(x, self.w_in)
+        part = lambda n: self.proj.part(y, n)  # noqa: E731
+        ops.rotate_append(None, part("k"), part("v"), self.heads, self.kv_heads, self.dk, None, meta, kc, vc)
+        ops.attention_exact(part("q").unflatten(1, (self.heads, self.dk)), kc, vc, meta, self.scale, out=out, form=self.form)
+
+    def load(self, get, p: str) -> None:
+        for n in "qkv":
+            self.proj.fill(self.w_in, n, get(p + n))
+        self.sink.data.copy_(get(p + "sink"))
+
+
+class DifferentialAttentionMixer(nn.Module):
+    """Attention within chunks of the sequence as the difference of two softmax maps over the same values: query and key heads hold the maps side
+    by side (split-half rotation on the first dimensions of each), the second map enters with a learned weight, the result is normed per head.
+    Writes the heads' outputs; the output projection is the caller's."""
+
+    def __init__(self, width, heads, kv_heads, dk, dv, scale, chunk, freq, diff, eps, dtype, device):
+        super().__init__()
+        if dk > 640 or dv > 512:
+            raise ValueError(f"head widths {dk}/{dv} exceed what the kernels hold (640/512)")
+        self.heads, self.kv_heads, self.dk, self.dv, self.scale, self.chunk, self.diff, self.eps = heads, kv_heads, dk, dv, scale, chunk, diff, eps
+        self.proj = FusedProjection(dict(q=2 * heads * dk, k=2 * kv_heads * dk, v=kv_heads * dv))
+        self.w_in = param(self.proj.rows, width, dtype=dtype, device=device)
+        self.mix = nn.ParameterDict({n: param(dk, dtype=torch.float32, device=device) for n in ("lq1", "lk1", "lq2", "lk2")})
+        self.register_buffer("freq", freq.to(torch.float64).to(device), persistent=False)
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.dv
+
+    def kv_spec(self):
+        return self.kv_heads, 2 * self.dk, self.dv
+
+    def finish(self) -> None:
+        dot = lambda i: float((self.mix[f"lq{i}"].double() * self.mix[f"lk{i}"].double()).sum())  # noqa: E731
+        mix = math.exp(dot(1)) - math.exp(dot(2)) + self.diff
+        self.form = ops.AttentionForm(chunk=self.chunk, difference=(mix, 1.0 - self.diff, self.eps))
+
+    def forward(self, x, meta, kc, vc, out):
+        y = ops.linear(x, self.w_in)
+        part = lambda n: self.proj.part(y, n)  # noqa: E731
+        q = part("q")
+        ops.rotate_append(q, part("k"), part("v"), 2 * self.heads, 2 * self.kv_heads, self.dk, self.freq, meta, kc, vc)
+        ops.attention_exact(q.unflatten(1, (self.heads, 2 * self.dk)), kc, vc, meta, self.scale, out=out, form=self.form)
+
+    def load(self, get, p: str) -> None:
+        for n in "qkv":
+            self.proj.fill(self.w_in, n, get(p + n))
+        for n, v in self.mix.items():
+            v.data.copy_(get(p + n))
+
+
+class RoutedExperts(nn.Module):
+    """A mixture of GLU experts: softmax scores over all of them, the ``top`` best by score plus a correction, weighted by ``scale`` times the score.
+    The last ``identity`` router outputs stand for the input itself.  The result goes to ``ops.stream_step``, which sums it up."""
+
+    def __init__(self, width, experts, identity, ff, top, scale, act, limit, dtype, device):
+        super().__init__()
+        if experts + identity > 512 or not 1 <= top <= min(32, experts + identity):
+            raise ValueError(f"{top} of {experts} + {identity} experts: the router holds 512 and chooses up to 32")
+        self.experts, self.identity, self.ff, self.top, self.scale, self.act, self.limit = experts, identity, ff, top, scale, act, limit
+        kw = dict(dtype=dtype, device=device)
+        self.w_router = param(experts + identity, width, **kw)
+        self.correction = param(experts + identity, dtype=torch.float32, device=device)
+        self.w_gu, self.w_down = param(experts, 2 * ff, width, **kw), param(experts, width, ff, **kw)
+
+    def forward(self, x):
+        idx, w = ops.router_topk(ops.linear_f32(x, self.w_router), self.top, "softmax", self.correction, scale=self.scale, renorm=False)
+        return ops.expert_outputs(x, idx, w, self.w_gu, self.w_down, self.act, self.limit)
+
+    def load(self, get, p: str) -> None:
+        self.w_router.data.copy_(get(p + "router"))
+        self.correction.data.copy_(get(p + "correction"))
+        for e in range(self.experts):
+            self.w_gu.data[e, :self.ff].copy_(get(f"{p}e{e}.gate"))
+            self.w_gu.data[e, self.ff:].copy_(get(f"{p}e{e}.up"))
+            self.w_down.data[e].copy_(get(f"{p}e{e}.down"))

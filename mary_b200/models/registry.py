@@ -45,6 +45,14 @@ def _load_rokarax(d, loader, device, dtype):
     return model
 
 
+def _load_nipurax(d, loader, device, dtype):
+    from .nipurax.config import NipuraxConfig
+    from .nipurax.model import NipuraxModel, load_into
+    model = NipuraxModel(NipuraxConfig.from_json(d), loader.shape("bigram")[0], dtype=dtype, device=device)
+    load_into(model, loader)
+    return model
+
+
 def _load_mistral(d, loader, device, dtype):
     from .mistral.model import MistralConfig, MistralModel, load_into
     model = MistralModel(MistralConfig.from_hf(d), dtype=dtype, device=device)
@@ -65,6 +73,8 @@ FAMILIES = [
            kernels=_DENSE_KERNELS + ("attention_general", "residual32", "linear_attention", "recurrent_scan")),
     Family("rokarax", lambda d: d.get("architecture") == "Rokarax", _load_rokarax, page_size=64, f32_on_gpu=True,
            kernels=_DENSE_KERNELS + ("attention_general", "attention_mla", "residual32", "linear_attention", "recurrent_scan", "latent", "state_space", "ssd_chunk")),
+    Family("nipurax", lambda d: d.get("architecture") == "Nipurax", _load_nipurax, page_size=64, f32_on_gpu=True,
+           kernels=_DENSE_KERNELS + ("attention_general", "residual32", "parallel_stream", "moe", "expert_step")),
     Family("gemma4", lambda d: str(d.get("model_type", "")).startswith("gemma4"), _load_gemma4),
     Family("mistral", lambda d: d.get("model_type") in ("mistral", "ministral", "qwen3", "mistral3"), _load_mistral),
 ]

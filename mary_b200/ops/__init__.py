@@ -6,6 +6,7 @@ from __future__ import annotations
 import torch
 
 from . import reference as ref
+from .attention_form import AttentionForm  # noqa: F401
 
 
 def _cuda(x) -> bool:
@@ -172,11 +173,15 @@ def glu(gate_up, act: str = "geglu"):
     return {"geglu": ref.geglu, "swiglu": ref.swiglu, "situ": ref.situ}[act](gate_up[..., :F], gate_up[..., F:])
 
 
-def linear_glu(x, w_gu, act: str = "geglu"):
-    """``act(x @ gate^T) * (x @ up^T)`` with ``w_gu = [gate; up]``; fused into the GEMM epilogue on the GPU."""
+def linear_glu(x, w_gu, act: str = "geglu", limit: float = 0.0, out=None):
+    """``act(x @ gate^T) * (x @ up^T)`` with ``w_gu = [gate; up]``; fused into the GEMM epilogue on the GPU.  ``clamped``: gate at most
+    ``limit``, up within it, ``g * sigmoid(1.702 g) * (u + 1)``.  ``out``: a row view that receives the result."""
     if _cuda(x):
-        return _k().linear_glu(x, w_gu, act)
-    return glu(ref.linear(x, w_gu), act)
+        return _k().linear_glu(x, w_gu, act, limit, out)
+    y = ref.linear(x, w_gu)
+    F = y.shape[-1] // 2
+    y = ref.clamped_glu(y[..., :F], y[..., F:], limit).to(x.dtype) if act == "clamped" else glu(y, act)
+    return y if out is None else out.copy_(y)
 
 
 def embed(ids, table, scale=1.0):
@@ -198,7 +203,7 @@ def router_topk(logits, k, mode="softmax", bias=None, n_group=1, topk_group=1, s
     if _cuda(logits):
         return _k().router_topk(logits, k, mode, bias, n_group, topk_group, scale, renorm)
     if mode == "softmax":
-        return ref.router_softmax_topk(logits, k, renorm)
+        return ref.router_softmax_topk(logits, k, renorm, bias, scale)
     return ref.router_sigmoid_topk(logits, bias, k, n_group, topk_group, scale, renorm)
 
 
@@ -270,13 +275,14 @@ def qk_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vca
     return f(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps)
 
 
-def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, bias=None, gate=None):
+def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, bias=None, gate=None, form=None):
     """Causal paged attention whose scores, softmax weights and sums stay in 32 bits, for any head widths: ``[T, Hq * DV]``.  ``window``: keys
     at most ``window - 1`` positions back (0: all); ``bias [Hq, window]`` f32 is added to the scaled score by distance; ``gate [T, Hq * DV]``
-    multiplies the result by its logistic function before it is rounded."""
+    multiplies the result by its logistic function before it is rounded.  ``form`` (an ``AttentionForm``; no window, bias or gate then): chunks,
+    capped scores, sinks, query temperature, the difference of two maps; ``q`` may be a row view of a projection."""
     if _cuda(q):
-        return _h().attention_exact(q, kcache, vcache, meta, scale, out, window, bias, gate)
-    o = ref.attention_exact(q, kcache, vcache, meta, scale, window, bias, gate)
+        return _h().attention_exact(q, kcache, vcache, meta, scale, out, window, bias, gate, form)
+    o = ref.attention_exact(q, kcache, vcache, meta, scale, window, bias, gate, form)
     if out is None:
         return o
     out.copy_(o)
@@ -337,3 +343,38 @@ def gated_delta_attention(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, rin
     the convolutions by absolute position, ``state`` is laid out as above."""
     f = _h().gated_delta_attention if _cuda(x) else ref.gated_delta_attention
     return f(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, ring, state, meta, HK, H, dk, dv, eps, out_scale, out)
+
+
+# --------------------------------------------------------------------------- parallel sublayers, routed experts, token pairs
+def _pl():
+    from . import cuda_parallel
+    return cuda_parallel
+
+
+def embed_pairs(ids, table, pairs, mul_prev: int, mul_cur: int, last, meta, x0=None, x1=None):
+    """Residual stream ``table[id] + pairs[(previous id * mul_prev + id * mul_cur) mod (len(pairs) - 1)]`` in f32, the last row of ``pairs`` for a
+    sequence's first token.  ``last [slots, 1]`` int32 keeps a sequence's newest token between steps; ``x0``, ``x1``: row views that receive
+    copies in the activation type."""
+    f = _pl().embed_pairs if _cuda(table) else ref.embed_pairs
+    return f(ids, table, pairs, mul_prev, mul_cur, last, meta, x0, x1)
+
+
+def rotate_append(q, k, v, n_q, n_kv, dk, freq, meta, kcache, vcache) -> None:
+    """Rotate ``q`` (row views of one projection: ``n_q`` heads of ``dk``) in place and ``k`` (``n_kv`` heads) into the cache, ``v`` into the cache.
+    ``freq``: f64 frequencies of the pairs ``(i, i + len(freq))``, ``None`` for no rotation (then ``q`` may be None)."""
+    f = _pl().rotate_append if _cuda(k) else ref.rotate_append
+    return f(q, k, v, n_q, n_kv, dk, freq, meta, kcache, vcache)
+
+
+def expert_outputs(x, idx, w, gate_up, down, act: str, limit: float = 0.0):
+    """The routed experts of a batch (``gate_up [E, 2 F, W]``, ``down [E, W, F]``; entries with an index of ``E`` or more stand for ``x`` itself) in
+    the form that ``stream_step`` sums up."""
+    f = _pl().expert_outputs if _cuda(x) else ref.expert_outputs
+    return f(x, idx, w, gate_up, down, act, limit)
+
+
+def stream_step(h, a=None, m: float = 1.0, routed=None, vec=None, keep: bool = True, gains=(), eps: float = 0.0, copy=None):
+    """``h <- keep h + m (a + sum of the routed experts) + vec`` on a 32-bit stream, in place; returns ``rms(h) * gain`` in the activation type for
+    every one of ``gains`` (at most two).  ``copy``: a row view that receives ``h``."""
+    f = _pl().stream_step if _cuda(h) else ref.stream_step
+    return f(h, a, m, routed, vec, keep, gains, eps, copy)

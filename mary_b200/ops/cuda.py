@@ -14,11 +14,11 @@ from ..utils.canary import empty as _empty
 
 _SIG = {
     # name: argument codes — p pointer, i int32, l int64, f float, s stream
-    "mary_gemm_bf16": "pppiiilllpfiiiis",
+    "mary_gemm_bf16": "pppiiilllpfiiiifs",
     "mary_rmsnorm": "pippiillfs",
     "mary_add_rmsnorm": "pipppiifs",
     "mary_norm_add_norm": "pippppiiffs",
-    "mary_glu": "ppiiis",
+    "mary_glu": "ppliiifs",
     "mary_embed": "pppiifis",
     "mary_qk_norm_rope_append": "piiippipppppp" + "fils",
     "mary_short_conv": "ppppiiis",
@@ -115,7 +115,7 @@ def _bf16(t):
 
 # --------------------------------------------------------------------------- GEMM
 def gemm(x, w, out=None, bias=None, alpha: float = 1.0, glu: str | None = None, epi: str = "bf16", split_k: int = 1,
-         swap: int = -1):
+         swap: int = -1, limit: float = 0.0):
     """``out[M, N] = alpha * x[M, K] @ w[N, K]^T``.  ``glu``: ``w = [gate; up]`` (2N rows) and the epilogue writes
     ``act(gate) * up``.  ``epi``: ``"bf16"`` store, ``"f32"`` store, ``"red"`` accumulate into a zeroed f32 ``out``."""
     _bf16(x), _bf16(w)
@@ -128,9 +128,9 @@ def gemm(x, w, out=None, bias=None, alpha: float = 1.0, glu: str | None = None, 
     e = {"bf16": 0, "red": 1, "f32": 2}[epi]
     if out is None:
         out = (torch.zeros if e == 1 else torch.empty)(M, N, dtype=torch.bfloat16 if e == 0 else torch.float32, device=x.device)
-    g = 0 if glu is None else {"geglu": 1, "swiglu": 2, "situ": 3}[glu]
+    g = 0 if glu is None else {"geglu": 1, "swiglu": 2, "situ": 3, "clamped": 4}[glu]
     rc = lib().mary_gemm_bf16(_p(x), _p(w), _p(out), M, N, K, x.stride(0), w.stride(0), out.stride(0), _p(bias), alpha, g, e,
-                              split_k, swap, _stream())
+                              split_k, swap, limit, _stream())
     check(rc, "gemm_bf16")
     return out
 
@@ -258,17 +258,20 @@ def linear_f32(x, w, split_k: int | None = None, alpha: float = 1.0):
         return gemm_splitk(x, w, 0 if split_k is None else sk, f32=True, alpha=alpha) if sk > 1 else gemm(x, w, alpha=alpha, epi="f32")
 
 
-def linear_glu(x, w_gu, act: str = "geglu"):
+def linear_glu(x, w_gu, act: str = "geglu", limit: float = 0.0, out=None):
+    """``out``: a row view that receives the result (its rows 16-byte aligned where the product is)."""
     M = x.shape[0]
     if x.dtype == torch.float32 or x.shape[1] % 8 or w_gu.shape[0] % 16:
         from .cuda_hybrid import glu_any
-        return glu_any(linear(x, w_gu), act)
-    if M == 1 and act in ("geglu", "swiglu") and x.shape[1] <= 8192 and w_gu.numel() * 2 <= MATVEC_GLU_MAX_BYTES and w_gu.stride(0) % 8 == 0:
-        return step_matvec(x, w_gu, mode=act)
-    with static_weights:
-        if M <= 128:
-            return gemm(x, w_gu, glu=act)
-        return glu(gemm(x, w_gu), act)
+        y = glu_any(linear(x, w_gu), act, limit)
+    elif M == 1 and act in ("geglu", "swiglu", "clamped") and x.shape[1] <= 8192 and w_gu.numel() * 2 <= MATVEC_GLU_MAX_BYTES and w_gu.stride(0) % 8 == 0:
+        return step_matvec(x, w_gu, mode=act, alpha=limit if act == "clamped" else 1.0, out=out)
+    else:
+        with static_weights:
+            if M <= 128:
+                return gemm(x, w_gu, out=out, glu=act, limit=limit)
+            y = glu(gemm(x, w_gu), act, limit, out)
+    return y if out is None or out is y else out.copy_(y)
 
 
 # --------------------------------------------------------------------------- norms and friends
@@ -297,10 +300,13 @@ def norm_add_norm(a, w_post, h, w_next, eps=1e-6, scalar=1.0):
     return xo, h
 
 
-def glu(gate_up, act="geglu"):
+def glu(gate_up, act="geglu", limit: float = 0.0, out=None):
     T, F2 = gate_up.shape
-    out = _empty(T, F2 // 2, dtype=torch.bfloat16, device=gate_up.device)
-    check(lib().mary_glu(_p(gate_up.contiguous()), _p(out), T, F2 // 2, {"geglu": 0, "swiglu": 1, "situ": 2}[act], _stream()), "glu")
+    ld = 0 if out is None else out.stride(0)
+    if out is None:
+        out = _empty(T, F2 // 2, dtype=torch.bfloat16, device=gate_up.device)
+    check(lib().mary_glu(_p(gate_up.contiguous()), _p(out), ld, T, F2 // 2, {"geglu": 0, "swiglu": 1, "situ": 2, "clamped": 3}[act], limit, _stream()),
+          "glu")
     return out
 
 
@@ -353,7 +359,7 @@ def _q_blocks(meta, rq: int, group: str | None = None):
     return cache[key]
 
 
-declare("mary_paged_attention_decode", "ppppppppp" + "iii" + "llll" + "iiiiii" + "ff" + "pl" + "ppls")
+declare("mary_paged_attention_decode", "ppppppppp" + "iii" + "llll" + "iiiiii" + "ff" + "pl" + "pplpis")
 
 
 DECODE_TARGET_CTAS = 2368      # CTAs the decode attention kernel aims for when it picks the number of kv splits (16 per SM)
@@ -364,13 +370,44 @@ def _gate(gate):
     return (None, 0) if gate is None else (_p(gate), gate.stride(0))
 
 
-def _paged_attention_decode(q, kcache, vcache, meta, scale, window, softcap, nsplit, out=None, group=None, bias=None, gate=None):
-    """Decode-shaped batches (few rows per kv head, equal K and V widths of 64/128/256): the bandwidth-oriented kernel.  ``bias``, ``gate``: see
-    ``ops.attention_exact``."""
+class _Form(ctypes.Structure):
+    """``MaryAttnForm`` of ``csrc/kernels/attention_form.cuh``."""
+    _fields_ = [("sink", ctypes.c_void_p), ("q_ld", ctypes.c_int64), ("chunk", ctypes.c_int32), ("maps", ctypes.c_int32),
+                ("temp_every", ctypes.c_int32), ("temp_coef", ctypes.c_float), ("cap", ctypes.c_float), ("mix", ctypes.c_float), ("post", ctypes.c_float),
+                ("eps", ctypes.c_float)]
+
+
+def form_struct(form, q):
+    """The C form of an ``AttentionForm`` (or None) for queries ``q [T, Hq, width]`` whose rows may have a pitch."""
+    if form is None and q.is_contiguous():
+        return None
+    assert q.stride(2) == 1 and q.stride(1) == q.shape[2]
+    s = _Form(q_ld=q.stride(0), maps=1)
+    if form is not None:
+        s.chunk, s.cap, s.maps = form.chunk, form.cap, form.maps
+        if form.sink is not None:
+            assert form.sink.dtype == torch.float32 and form.sink.is_contiguous() and form.sink.shape == (q.shape[1],)
+            s.sink = form.sink.data_ptr()
+        if form.temperature is not None:
+            s.temp_coef, s.temp_every = form.temperature
+        if form.difference is not None:
+            s.mix, s.post, s.eps = form.difference
+    return s
+
+
+def _form_p(s):
+    return None if s is None else ctypes.addressof(s)
+
+
+def _paged_attention_decode(q, kcache, vcache, meta, scale, window, softcap, nsplit, out=None, group=None, bias=None, gate=None, form=None):
+    """Decode-shaped batches (few rows per kv head, equal K and V widths of 64/128/256): the bandwidth-oriented kernel.  ``bias``, ``gate``, ``form``:
+    see ``ops.attention_exact``."""
     T, Hq, D = q.shape
-    Hkv = kcache.shape[2]
+    Hkv, DV = kcache.shape[2], vcache.shape[3]
     G = Hq // Hkv
-    cap = 4 if D == 256 else 8
+    maps = 1 if form is None else form.maps
+    D //= maps
+    cap = 4 if D == 256 or maps == 2 else 8
     rq = max(1, min(cap // G, meta.max_q_len))
     blk_seq, blk_q0, NB = _q_blocks(meta, rq, group)
     if nsplit is None:
@@ -379,16 +416,20 @@ def _paged_attention_decode(q, kcache, vcache, meta, scale, window, softcap, nsp
         nsplit = max(1, min(want, 32, span // 64))
     ld = 0                                        # ``out``: a row view [T, Hq * D] of any pitch
     if out is None:
-        out = _empty(T, Hq, D, dtype=torch.bfloat16, device=q.device)
+        out = _empty(T, Hq, DV, dtype=torch.bfloat16, device=q.device)
     else:
         ld = out.stride(0)
     scratch = None
-    if nsplit > 1:
-        scratch = _empty(lib().mary_paged_attention_scratch_floats(NB, Hkv, nsplit, D), dtype=torch.float32, device=q.device)
-    check(lib().mary_paged_attention_decode(_p(q.contiguous()), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len),
+    if nsplit > 1 or maps == 2:
+        scratch = _empty(lib().mary_paged_attention_scratch_floats(NB, Hkv, nsplit, DV), dtype=torch.float32, device=q.device)
+    if form is None:
+        q = q.contiguous()
+    fs = form_struct(form, q)
+    check(lib().mary_paged_attention_decode(_p(q), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len),
                                             _p(meta.q_start), _p(blk_seq), _p(blk_q0), NB, meta.page_table.shape[1], meta.page_size,
                                             kcache.stride(1), kcache.stride(0), vcache.stride(1), vcache.stride(0), Hq, Hkv, D, rq,
-                                            nsplit, window, scale, softcap, _p(scratch), ld, _p(bias), *_gate(gate), _stream()), "paged_attention_decode")
+                                            nsplit, window, scale, softcap, _p(scratch), ld, _p(bias), *_gate(gate), _form_p(fs), DV, _stream()),
+          "paged_attention_decode")
     return out
 
 
@@ -477,25 +518,27 @@ def gqa_decode_tc(q, kcache, vcache, meta, scale, window=0, softcap=0.0, nsplit=
     return out
 
 
-declare("mary_attention_prefill", "ppppppppp" + "iiiiiiii" + "llll" + "ifi" + "li" + "ppls")
+declare("mary_attention_prefill", "ppppppppp" + "iiiiiiii" + "llll" + "ifi" + "li" + "pplps")
+declare("mary_attention_prefill_maps_supported", "ii")
 declare("mary_attention_prefill_supported", "ii")
 PREFILL_MIN_ROWS = 48     # mean query tokens per sequence from which the 128-row tensor-core tiles pay off
 
 
-def attention_prefill(q, kcache, vcache, meta, scale, window=0, out=None, split_p: bool = False, group=None, bias=None, gate=None):
+def attention_prefill(q, kcache, vcache, meta, scale, window=0, out=None, split_p: bool = False, group=None, bias=None, gate=None, form=None):
     """Causal / sliding-window attention of whole query blocks on the tensor cores (``csrc/kernels/attention_fa.cu``):
     ``q[T, Hq, DK]``, caches ``[pages, page, Hkv, D]``; 128 query tokens of one head per CTA.  A cache with 64-token pages is
     streamed with one TMA operation per 64-key stage; a cache with smaller pages is first regrouped into 64-token pages (one
     gather, small beside the attention arithmetic) when the host knows the sequence lengths.
     ``split_p`` keeps 16 significant bits of the softmax weights; ``out`` may be a row view ``[T, Hq * DV]``; ``group``: see ``_q_blocks``; ``bias`` (with
-    ``split_p``), ``gate``: see ``ops.attention_exact``."""
+    ``split_p``), ``gate``, ``form`` (with ``split_p``): see ``ops.attention_exact``."""
     T, Hq, DK = q.shape
     Hkv, DV = kcache.shape[2], vcache.shape[-1]
+    DK //= 1 if form is None else form.maps
     ps = meta.page_size
     assert kcache.shape[1] == ps
     if ps in (16, 32) and meta.kv_lens_host is not None:
         pick, meta = meta.repage(64)
-        kcache = kcache[pick].view(-1, 64, Hkv, DK)
+        kcache = kcache[pick].view(-1, 64, Hkv, kcache.shape[3])
         vcache = vcache[pick].view(-1, 64, Hkv, DV)
         ps = 64
     assert ps in (16, 64)
@@ -505,10 +548,13 @@ def attention_prefill(q, kcache, vcache, meta, scale, window=0, out=None, split_
         out = _empty(T, Hq, DV, dtype=torch.bfloat16, device=q.device)
     else:
         ld = out.stride(0)
-    check(lib().mary_attention_prefill(_p(q.contiguous()), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len),
+    if form is None:
+        q = q.contiguous()
+    fs = form_struct(form, q)
+    check(lib().mary_attention_prefill(_p(q), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len),
                                        _p(meta.q_start), _p(blk_seq), _p(blk_tok0), NB, T, Hq, Hkv, DK, DV, kcache.shape[0],
                                        meta.page_table.shape[1], kcache.stride(1), kcache.stride(0), vcache.stride(1), vcache.stride(0),
-                                       int(window), float(scale), ps, ld, int(split_p), _p(bias), *_gate(gate), _stream()), "attention_prefill")
+                                       int(window), float(scale), ps, ld, int(split_p), _p(bias), *_gate(gate), _form_p(fs), _stream()), "attention_prefill")
     return out
 
 
@@ -747,14 +793,14 @@ declare("mary_step_matvec", "ppfpliippi" + "fs")
 declare("mary_step_attention", "pppppppppp" + "iiiilffp" + "s")
 
 
-def step_matvec(h, w, gain=None, eps: float = 1e-6, res=None, mode: str = "plain", alpha: float = 1.0):
+def step_matvec(h, w, gain=None, eps: float = 1e-6, res=None, mode: str = "plain", alpha: float = 1.0, out=None):
     """One-token matrix-vector stage of the fused layer step: ``W x`` (``plain``), ``res + W x`` (``residual``), ``act(W_gate x) * (W_up x)``
-    over ``w = [gate; up]`` (``swiglu`` / ``geglu``) or ``alpha * W x`` as f32 (``f32``), with ``x = rms(h) * gain`` when ``gain`` is given,
+    over ``w = [gate; up]`` (``swiglu`` / ``geglu`` / ``clamped`` with limit ``alpha``) or ``alpha * W x`` as f32 (``f32``), with ``x = rms(h) * gain`` when ``gain`` is given,
     else ``x = h``.  ``h [1, K]`` -> ``[1, N]``."""
-    m = {"plain": 0, "residual": 1, "swiglu": 2, "f32": 3, "geglu": 4}[mode]
+    m = {"plain": 0, "residual": 1, "swiglu": 2, "f32": 3, "geglu": 4, "clamped": 5}[mode]
     K = h.shape[-1]
-    N = w.shape[0] // 2 if m in (2, 4) else w.shape[0]
-    y = _empty(1, N, dtype=torch.float32 if m == 3 else torch.bfloat16, device=h.device)
+    N = w.shape[0] // 2 if m in (2, 4, 5) else w.shape[0]
+    y = _empty(1, N, dtype=torch.float32 if m == 3 else torch.bfloat16, device=h.device) if out is None else out
     check(lib().mary_step_matvec(_p(h), _p(gain), eps, _p(w), w.stride(0), N, K, _p(res), _p(y), m, alpha, _stream()), "step_matvec")
     return y
 

@@ -4,6 +4,7 @@ Each wrapper serves bf16 and 32-bit activations (the kernels are instantiated fo
 given.  Nothing here converts a 32-bit product to a reduced-precision mode."""
 from __future__ import annotations
 
+import numpy as np
 import torch
 
 from ..utils.canary import empty as _empty
@@ -14,9 +15,10 @@ declare("mary_gemm_simt", "pppiiilllfiiis")
 declare("mary_embed32", "ppppiifiis")
 declare("mary_post_norm_add", "plppppiifis")
 declare("mary_rmsnorm32", "pppiifis")
-declare("mary_glu_any", "ppiiiis")
+declare("mary_glu_any", "ppiiifis")
 declare("mary_qk_norm_append", "ppp" + "liiii" + "pppppp" + "fil" + "is")
-declare("mary_attention_general", "ppppppppp" + "iii" + "lllll" + "iiiiiii" + "fpplpis")
+declare("mary_attention_general", "ppppppppp" + "iii" + "lllll" + "iiiiiii" + "fpplppis")
+declare("mary_map_difference", "pplpiiifffis")
 declare("mary_attention_general_rows", "i")
 declare("mary_attention_general_scratch_floats", "iiiii", ret64=True)
 declare("mary_channel_decay", "pli" + "ppp" + "iifis")
@@ -100,10 +102,11 @@ def rmsnorm32(h, w, eps):
     return y
 
 
-def glu_any(gate_up, act: str):
+def glu_any(gate_up, act: str, limit: float = 0.0):
     T, F2 = gate_up.shape
     out = _empty(T, F2 // 2, dtype=gate_up.dtype, device=gate_up.device)
-    check(lib().mary_glu_any(_p(gate_up.contiguous()), _p(out), T, F2 // 2, {"geglu": 0, "swiglu": 1}[act], _f32(gate_up), _stream()), "glu_any")
+    check(lib().mary_glu_any(_p(gate_up.contiguous()), _p(out), T, F2 // 2, {"geglu": 0, "swiglu": 1, "clamped": 3}[act], limit, _f32(gate_up),
+                             _stream()), "glu_any")
     return out
 
 
@@ -121,12 +124,16 @@ def qk_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vca
 DECODE_ROWS = K.DECODE_GROUP_ROWS         # sequences with at most this many query tokens take the decode kernel, the others the prefill kernel
 
 
-def attention_general(q, kcache, vcache, meta, scale, out, group=None, nsplit=None, window: int = 0, bias=None, gate=None):
+def attention_general(q, kcache, vcache, meta, scale, out, group=None, nsplit=None, window: int = 0, bias=None, gate=None, form=None):
     """Any head widths, group size and storage type; ``group`` restricts the call to ``"prefill"`` or ``"decode"`` sequences.  ``bias``,
-    ``gate``: see ``ops.attention_exact``."""
+    ``gate``, ``form``: see ``ops.attention_exact``."""
     T, Hq, DK = q.shape
     Hkv, DV = kcache.shape[2], vcache.shape[3]
     G = Hq // Hkv
+    fs, result = K.form_struct(form, q), out
+    if form is not None and form.maps == 2:           # the kernel counts (head, map) pairs and leaves both maps' outputs in 32 bits
+        Hq, Hkv, DK = 2 * Hq, 2 * Hkv, DK // 2
+        out = _empty(T, Hq * DV, dtype=torch.float32, device=q.device)
     rq = max(1, min(lib().mary_attention_general_rows(G), meta.max_q_len))
     blk_seq, blk_q0, NB = K._q_blocks(meta, rq, group)
     if NB == 0:
@@ -141,27 +148,48 @@ def attention_general(q, kcache, vcache, meta, scale, out, group=None, nsplit=No
     check(lib().mary_attention_general(_p(q), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len), _p(meta.q_start), _p(blk_seq),
                                        _p(blk_q0), NB, meta.page_table.shape[1], meta.page_size, kcache.stride(1), kcache.stride(0), vcache.stride(1),
                                        vcache.stride(0), out.stride(0), Hq, Hkv, DK, DV, rq, nsplit, window, scale, _p(bias), *K._gate(gate), _p(scratch),
-                                       _f32(q), _stream()), "attention_general")
-    return out
+                                       K._form_p(fs), _f32(q), _stream()), "attention_general")
+    if out is not result:
+        rows = None if group is None else _group_rows(meta, group)
+        check(lib().mary_map_difference(_p(out), _p(result), result.stride(0), _p(rows), T if rows is None else rows.numel(), Hq // 2, DV,
+                                        *form.difference, _f32(q), _stream()), "map_difference")
+    return result
 
 
-def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, bias=None, gate=None):
+def _group_rows(meta, group: str):
+    """The rows of the batch that belong to a group of sequences (int32, memoised)."""
+    memo = meta.__dict__.setdefault("_cache", {})
+    key = ("rows", group)
+    if key not in memo:
+        q = meta.q_lens_host
+        pick = np.repeat((q > DECODE_ROWS) == (group == "prefill"), q)
+        memo[key] = torch.from_numpy(np.nonzero(pick)[0].astype(np.int32)).to(meta.positions.device, non_blocking=True)
+    return memo[key]
+
+
+def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, bias=None, gate=None, form=None):
     """Causal attention with scores, softmax weights and sums in 32 bits: the tensor-core prefill kernel with two-term weights for
     sequences that bring more than ``DECODE_ROWS`` tokens, the bandwidth-oriented decode kernel for the others, the general kernel for
     32-bit tensors and for head shapes those have no instantiation for.  ``out`` may be a row view ``[T, Hq * DV]``."""
     T, Hq, DK = q.shape
     Hkv, DV = kcache.shape[2], vcache.shape[3]
-    assert q.is_contiguous() and kcache.is_contiguous() and vcache.stride(3) == 1 and kcache.shape[1] == meta.page_size
+    assert (q.is_contiguous() or form is not None) and kcache.is_contiguous() and vcache.stride(3) == 1 and kcache.shape[1] == meta.page_size
     assert bias is None or (bias.is_contiguous() and bias.shape == (Hq, window) and bias.dtype == torch.float32)
     assert gate is None or gate.dtype == q.dtype
     if out is None:
         out = _empty(T, Hq * DV, dtype=q.dtype, device=q.device)
     assert out.stride(1) == 1
-    bf16 = q.dtype == torch.bfloat16 and DK == DV and vcache.is_contiguous()
-    kw = dict(window=window, bias=bias, gate=gate)
-    aligned = all(t is None or (t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0) for t in (out, gate))
-    fast_prefill = bf16 and DK in (64, 128, 256) and meta.page_size in (16, 64) and aligned
-    fast_decode = bf16 and DK in (64, 128, 256) and Hq // Hkv <= (4 if DK == 256 else 8)
+    kw = dict(window=window, bias=bias, gate=gate, form=form)
+    aligned = all(t is None or (t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0) for t in (out, gate, q))
+    bf16 = q.dtype == torch.bfloat16 and vcache.is_contiguous()
+    if form is not None and form.maps == 2:
+        bf16 = bf16 and bool(lib().mary_attention_prefill_maps_supported(DK // 2, DV))
+        fast_prefill = bf16 and meta.page_size in (16, 64) and aligned
+        fast_decode = bf16 and Hq // Hkv <= 4 and aligned
+    else:
+        bf16 = bf16 and DK == DV and DK in (64, 128, 256)
+        fast_prefill = bf16 and meta.page_size in (16, 64) and aligned
+        fast_decode = bf16 and Hq // Hkv <= (4 if DK == 256 else 8) and (q.is_contiguous() or aligned)
     if not (fast_prefill or fast_decode):
         return attention_general(q, kcache, vcache, meta, scale, out, **kw)
     if meta.max_q_len > DECODE_ROWS:
@@ -171,7 +199,7 @@ def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, b
             attention_general(q, kcache, vcache, meta, scale, out, "prefill", **kw)
     if K._q_blocks(meta, 1, "decode")[2]:
         if fast_decode:
-            K._paged_attention_decode(q, kcache, vcache, meta, scale, window, 0.0, None, out=out, group="decode", bias=bias, gate=gate)
+            K._paged_attention_decode(q, kcache, vcache, meta, scale, window, 0.0, None, out=out, group="decode", bias=bias, gate=gate, form=form)
         else:
             attention_general(q, kcache, vcache, meta, scale, out, "decode", **kw)
     return out

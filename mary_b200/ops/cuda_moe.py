@@ -124,17 +124,17 @@ def experts_forward(x, idx, w, ex, shared=None, nt: int | None = None):
     return unpermute(y, plan, w, T, k, shared)
 
 
-declare("mary_gemm_bf16_grouped", "ppp" + "iii" + "lll" + "i" + "l" + "pp" + "iii" + "s")
+declare("mary_gemm_bf16_grouped", "ppp" + "iii" + "lll" + "i" + "l" + "pp" + "iii" + "fs")
 
 
-def grouped_gemm_bf16(xg, w, plan: Plan, n_out: int, glu: str | None, swap: bool = True):
+def grouped_gemm_bf16(xg, w, plan: Plan, n_out: int, glu: str | None, swap: bool = True, limit: float = 0.0):
     """``out[r] = act_glu(xg[r] @ w[expert of r's tile]^T)`` over the plan's padded rows; ``w [E, n_out or 2 n_out, K]`` unquantised.
     ``swap=False`` (plans with 128-row tiles, no GLU): tokens as the 128-row tensor-core operand, for prefill-sized batches."""
     E, _, K = w.shape
     out = _empty(plan.max_rows, n_out, dtype=torch.bfloat16, device=xg.device)
-    g = 0 if glu is None else {"geglu": 1, "swiglu": 2, "situ": 3}[glu]
+    g = 0 if glu is None else {"geglu": 1, "swiglu": 2, "situ": 3, "clamped": 4}[glu]
     check(lib().mary_gemm_bf16_grouped(_p(xg), _p(w), _p(out), plan.max_rows, n_out, K, xg.stride(0), w.stride(1), out.stride(0), E,
-                                       w.stride(0), _p(plan.tiles), _p(plan.meta), plan.nt, g, int(swap), _stream()), "gemm_bf16_grouped")
+                                       w.stride(0), _p(plan.tiles), _p(plan.meta), plan.nt, g, int(swap), limit, _stream()), "gemm_bf16_grouped")
     return out
 
 

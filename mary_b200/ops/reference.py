@@ -143,13 +143,14 @@ def argmax_first(logits):
 
 
 # --------------------------------------------------------------------------- MoE
-def router_softmax_topk(logits, k: int, renorm: bool = True):
-    """Softmax router: probabilities over all experts, top-k (ties -> lower index), renormalised."""
+def router_softmax_topk(logits, k: int, renorm: bool = True, bias=None, scale: float = 1.0):
+    """Softmax router: probabilities over all experts, top-k of them plus ``bias`` (ties -> lower index), weights without it, renormalised."""
     p = torch.softmax(logits.float(), dim=-1)
-    w, idx = topk_first(p, k)
+    idx = topk_first(p if bias is None else p + bias.float(), k)[1]
+    w = p.gather(-1, idx.long())
     if renorm:
         w = w / w.sum(-1, keepdim=True)
-    return idx.int(), w
+    return idx.int(), w * scale
 
 
 def topk_first(scores, k: int):
@@ -341,7 +342,44 @@ def gated_delta_attention(x, taps_w, b_in, a_in, a_log, dt_bias, gate, gain, rin
     return out
 
 
-def attention_exact(q, kcache, vcache, meta, scale, window: int = 0, bias=None, gate=None):
+def _attention_form(q, kcache, vcache, meta, scale, f):
+    """One map of ``attention_exact`` with an ``AttentionForm``: f32 ``[T, Hq, DV]``."""
+    T, Hq, _ = q.shape
+    G = Hq // kcache.shape[2]
+    out = torch.empty(T, Hq, vcache.shape[3])
+    qs, kl = meta.q_start.tolist(), meta.kv_len.tolist()
+    for s in range(meta.num_seqs):
+        rows = slice(qs[s], qs[s + 1])
+        K = gather_pages(kcache, meta.page_table[s], kl[s]).float().repeat_interleave(G, 1)
+        V = gather_pages(vcache, meta.page_table[s], kl[s]).float().repeat_interleave(G, 1)
+        pos, kpos = meta.positions[rows].long(), torch.arange(kl[s])
+        Q = q[rows].float()
+        if f.temperature is not None:
+            Q = Q * (1.0 + f.temperature[0] * torch.log((pos + 1).div(f.temperature[1], rounding_mode="floor").float() + 1.0))[:, None, None]
+        sc = torch.einsum("nhd,lhd->hnl", Q, K) * scale
+        if f.cap > 0:
+            sc = f.cap * torch.tanh(sc / f.cap)
+        seen = kpos[None] <= pos[:, None]
+        if f.chunk > 0:
+            seen &= kpos[None] >= (pos // f.chunk * f.chunk)[:, None]
+        sc = sc.masked_fill(~seen[None], float("-inf"))
+        if f.sink is not None:
+            sc = torch.cat([sc, f.sink.float()[:, None, None].expand(-1, sc.shape[1], 1)], -1)
+        out[rows] = torch.einsum("hnl,lhd->nhd", torch.softmax(sc, -1)[..., :kl[s]], V)
+    return out
+
+
+def attention_exact(q, kcache, vcache, meta, scale, window: int = 0, bias=None, gate=None, form=None):
+    if form is not None:
+        assert window == 0 and bias is None and gate is None
+        d = q.shape[2] // form.maps
+        o = [_attention_form(q[..., m * d:(m + 1) * d], kcache[..., m * d:(m + 1) * d], vcache, meta, scale, form) for m in range(form.maps)]
+        y = o[0]
+        if form.difference is not None:
+            mix, post, eps = form.difference
+            y = y - mix * o[1]
+            y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps) * post
+        return y.reshape(q.shape[0], -1).to(q.dtype)
     rel = None if bias is None else bias[None].expand(q.shape[0], -1, -1)
     o = paged_attention(q.float(), kcache, vcache, meta, scale, window, rel_bias=rel).reshape(q.shape[0], -1)
     return (o if gate is None else o * torch.sigmoid(gate.float())).to(q.dtype)
@@ -409,3 +447,69 @@ def state_space(xbc, taps_w, taps_b, dt_in, dt_bias, a_log, skip, z, gain, norm_
     y = ((y + skip[:, None] * x).reshape(T, H * P) * F.silu(z.float())).view(T, norm_parts, -1)
     out.copy_((y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, H * P) * gain.float())
     return out
+
+
+# --------------------------------------------------------------------------- parallel sublayers, routed experts, token pairs
+def embed_pairs(ids, table, pairs, mul_prev: int, mul_cur: int, last, meta, x0=None, x1=None):
+    ids, buckets = ids.long(), pairs.shape[0] - 1
+    row = torch.empty_like(ids)
+    for rows, slot, pos in _portions(meta):
+        t = ids[rows]
+        prev = torch.cat([last[slot].long().view(1), t[:-1]])
+        row[rows] = (prev * mul_prev + t * mul_cur) % buckets
+        if pos == 0:
+            row[rows.start] = buckets
+        last[slot] = t[-1].to(torch.int32)
+    h = table[ids].float() + pairs[row].float()
+    for x in (x0, x1):
+        if x is not None:
+            x.copy_(h)
+    return h
+
+
+def rotate_halves(x, positions, freq):
+    """``x [T, H, D]``: dimensions ``i`` and ``i + n`` turn by ``position * freq[i]`` (``n`` f64 frequencies), the others stay."""
+    n = freq.numel()
+    ang = (positions.double()[:, None] * freq.double()[None])[:, None]
+    c, s = ang.cos().float(), ang.sin().float()
+    u, v = x[..., :n].float(), x[..., n:2 * n].float()
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:].float()], -1).to(x.dtype)
+
+
+def rotate_append(q, k, v, n_q, n_kv, dk, freq, meta, kcache, vcache):
+    T = k.shape[0]
+    k = k.reshape(T, n_kv, dk)
+    if freq is not None:
+        q.copy_(rotate_halves(q.reshape(T, n_q, dk), meta.positions, freq).reshape(T, -1))
+        k = rotate_halves(k, meta.positions, freq)
+    kv_append(k.reshape(T, *kcache.shape[2:]), v.reshape(T, *vcache.shape[2:]), kcache, vcache, meta.slot_mapping)
+
+
+def clamped_glu(g, u, limit: float):
+    g, u = g.float().clamp(max=limit), u.float().clamp(-limit, limit)
+    return g * torch.sigmoid(1.702 * g) * (u + 1.0)
+
+
+def expert_outputs(x, idx, w, gate_up, down, act: str, limit: float = 0.0):
+    E, F2, _ = gate_up.shape
+    out = torch.zeros(x.shape[0], down.shape[1])
+    for e in range(E):
+        t, j = torch.nonzero(idx == e, as_tuple=True)
+        if t.numel():
+            y = linear(x[t], gate_up[e])
+            h = (clamped_glu(y[:, :F2 // 2], y[:, F2 // 2:], limit) if act == "clamped" else {"geglu": geglu, "swiglu": swiglu}[act](y[:, :F2 // 2], y[:, F2 // 2:]))
+            out.index_add_(0, t, linear(h.to(x.dtype), down[e]).float() * w[t, j][:, None])
+    return out + (w * (idx >= E)).sum(-1, keepdim=True) * x.float()
+
+
+def stream_step(h, a, m, routed, vec, keep, gains, eps, copy):
+    s = torch.zeros_like(h) if a is None else a.float()
+    s = m * (s if routed is None else s + routed)
+    if keep:
+        s = s + h
+    if vec is not None:
+        s = s + vec.float()
+    h.copy_(s)
+    if copy is not None:
+        copy.copy_(h)
+    return [rmsnorm32(h, g, eps) for g in gains]
