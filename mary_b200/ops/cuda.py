@@ -421,7 +421,7 @@ def _paged_attention_decode(q, kcache, vcache, meta, scale, window, softcap, nsp
         ld = out.stride(0)
     scratch = None
     if nsplit > 1 or maps == 2:
-        scratch = _empty(lib().mary_paged_attention_scratch_floats(NB, Hkv, nsplit, DV), dtype=torch.float32, device=q.device)
+        scratch = _empty(lib().mary_paged_attention_scratch_floats(NB, Hkv, max(nsplit, maps), DV), dtype=torch.float32, device=q.device)
     if form is None:
         q = q.contiguous()
     fs = form_struct(form, q)
