@@ -1,5 +1,6 @@
-"""Throughput of the hybrid decoders (Tatizen, Rokarax) beside the dense decoder of equal size (the Mistral shell), prefill and decode, on
-one GPU.
+"""Throughput of the decoders with a 32-bit residual stream beside the closest decoder of equal size, prefill and decode, on one GPU: Tatizen and
+Rokarax beside the dense decoder (the Mistral shell), Nipurax beside the decoder with routed bf16 experts next to a dense feed-forward (the
+Gemma shell).
 
 Random weights of the named sizes; every step streams weights and caches far larger than L2.  Prefill: whole prompts through
 ``model.greedy`` (logits of the last rows).  Decode: the fixed-batch decoder replaying one CUDA graph per step over caches and states
@@ -18,6 +19,10 @@ PAGE = 64
 # heads with windows of 1024 positions, state space layers of twice the width in heads of 64 with 128 state rows, latents of 512 + 64
 SIZES = {"2k": (2048, 8192, (16, 4), 8, (16, 8)), "4k": (4096, 12288, (32, 8), 16, (32, 16))}
 LAYERS, VOCAB, WINDOW = 8, 32768, 1024
+# Nipurax: the same width and attention heads, every layer with experts, experts per token, their width and the shared one's; two of six layers
+# run twice, so that eight layer runs stand beside the other decoder's eight layers
+EXPERTS = {"2k": (32, 4, 1024, 2048), "4k": (32, 4, 1536, 4096)}
+IDENTITY, CHUNK = 4, 2048
 CASES = [("prefill", 1, 4096), ("prefill", 8, 512), ("decode", 1, 2048), ("decode", 32, 2048), ("decode", 128, 2048)]
 
 
@@ -44,6 +49,23 @@ def dense_config(size: str):
     return MistralConfig(LAYERS, W, F, H, G, 128, VOCAB, qk_norm=True, name=f"dense-{size}")
 
 
+def nipurax_config(size: str):
+    from .nipurax.config import CappedSpec, DifferentialSpec, ExpertsSpec, GLUSpec, LayerSpec, LoopSpec, NipuraxConfig, PairsSpec, RotationSpec
+    (W, _, (H, G), _, _), (E, top, F, FS) = SIZES[size], EXPERTS[size]
+    moe = ExpertsSpec(E, IDENTITY, top, 2.0, GLUSpec(F, 7.0), GLUSpec(FS, 7.0))
+    cap = LayerSpec(CappedSpec(H, G, 128, 128, 128 ** -0.5, 30.0, 0.1, 1024), moe)
+    dif = LayerSpec(DifferentialSpec(H, G, 64, 128, 0.125, CHUNK, 0.3, RotationSpec(64, 1e6, 8.0, 1.0, 4.0, 2048.0)), moe)
+    return NipuraxConfig(VOCAB, W, 1e-5, 0.3, PairsSpec(65521, 31, 7), LoopSpec(2, 4, 2), [cap, dif] * 3, name=f"nipurax-{size}")
+
+
+def routed_config(size: str):
+    from .gemma4.config import Gemma4TextConfig
+    (W, _, (H, G), _, _), (E, top, F, FS) = SIZES[size], EXPERTS[size]
+    return Gemma4TextConfig(hidden_size=W, num_hidden_layers=LAYERS, num_attention_heads=H, num_key_value_heads=G, head_dim=128, intermediate_size=FS,
+                            vocab_size=VOCAB, layer_types=["full_attention"] * LAYERS, enable_moe_block=True, num_experts=E, top_k_experts=top,
+                            moe_intermediate_size=F)
+
+
 def make_model(kind: str, size: str, dev):
     kw = dict(dtype=torch.bfloat16, device=dev)
     if kind == "tatizen":
@@ -52,6 +74,14 @@ def make_model(kind: str, size: str, dev):
     elif kind == "rokarax":
         from .rokarax.model import RokaraxModel, init_random_
         m = RokaraxModel(rokarax_config(size), **kw)
+    elif kind == "nipurax":
+        from .nipurax.model import NipuraxModel, init_random_
+        m = NipuraxModel(nipurax_config(size), **kw)
+    elif kind == "routed":
+        from .gemma4.model import Gemma4Model
+        from .gemma4.weights import init_random_
+        m = Gemma4Model(routed_config(size), **kw)
+        m.trunk = m.hidden
     else:
         from .mistral.model import MistralModel, init_random_
         m = MistralModel(dense_config(size), **kw)
@@ -66,7 +96,8 @@ def make_cache(m, batch: int, tokens: int, dev) -> PagedKVCache:
         t.normal_()
     for layer in c.state:
         for t in layer.values():
-            t.normal_(0.0, 0.02)
+            if t.is_floating_point():
+                t.normal_(0.0, 0.02)
     return c
 
 
@@ -107,7 +138,7 @@ def run(design: str, sizes, cases, steps: int, warmup: int, trace: bool = False)
     dev = torch.device("cuda", 0)
     out = []
     for size in sizes:
-        for kind in (design, "dense"):
+        for kind in (design, "routed" if design == "nipurax" else "dense"):
             m = make_model(kind, size, dev)
             for what, batch, n in cases:
                 # dependent launch: a decode step is a chain of short kernels and gains from it; a prefill step loses (the waiting blocks of
@@ -140,5 +171,5 @@ def run(design: str, sizes, cases, steps: int, warmup: int, trace: bool = False)
     status = K.last_status()
     if status:
         raise RuntimeError(f"kernel status {status}")
-    return {"metric": f"tokens/s, {design} beside the dense decoder of equal size", "unit": "tokens/s", "layers": LAYERS, "dtype": "bf16",
+    return {"metric": f"tokens/s, {design} beside the {'routed' if design == 'nipurax' else 'dense'} decoder of equal size", "unit": "tokens/s", "layers": LAYERS, "dtype": "bf16",
             "data": "synthetic", "steps": steps, "warmup": max(warmup, 3), "cases": out}

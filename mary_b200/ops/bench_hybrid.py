@@ -1,5 +1,5 @@
 """Micro-benchmarks of the kernels of decoders with recurrent layers, beside the like kernels of the dense decoders
-(``python -m mary_b200.ops.bench_kernels hybrid`` and ``rokarax``).  Fractions: bytes against the measured copy bandwidth, tensor-core products against
+(``python -m mary_b200.ops.bench_kernels hybrid``, ``rokarax`` and ``nipurax``).  Fractions: bytes against the measured copy bandwidth, tensor-core products against
 the measured cuBLAS rate, the recurrences (32-bit multiply-adds on the CUDA cores) against the nominal 128 multiply-adds per SM and clock."""
 from __future__ import annotations
 
@@ -214,5 +214,86 @@ def run_rokarax(width: int = 4096, heads: int = 32, kv_heads: int = 8, window: i
         ar, h, hb, xb = torch.randn(B, width, device="cuda"), torch.randn(B, width, device="cuda"), torch.randn(B, width, **bf), torch.randn(B, width, **bf)
         add("add_rmsnorm", case, lambda: K.add_rmsnorm(xb, hb, norm.w, 1e-5), nbytes=B * width * 8, like="dense decoder")
         add("dyt_add", case, lambda: H.dyt_add(ar, norm, h, norm), nbytes=B * width * 14)
+    assert K.last_status() == 0
+    return add.rows
+
+
+def run_nipurax(width: int = 2048, heads: int = 16, kv_heads: int = 4, experts: int = 32, top: int = 4, ff: int = 1024, chunk: int = 2048) -> list[dict]:
+    """The kernels of the Nipurax decoder: capped attention with a sink and differential attention beside the plain ones, routed experts with the
+    clamped GLU beside those of the decoder with a GEGLU, the row kernels."""
+    from ..models.mixers import stepped_frequencies
+    from . import AttentionForm
+    from . import cuda as K
+    from . import cuda_hybrid as H
+    from . import cuda_moe as M
+    from . import cuda_parallel as P
+    add = _Table()
+    tf = add.tf
+    bf = dict(dtype=torch.bfloat16, device="cuda")
+    D = 128
+    cap = AttentionForm(cap=30.0, sink=torch.zeros(heads, device="cuda"), temperature=(0.1, 1024))
+    dif = AttentionForm(chunk=chunk, difference=(0.4, 0.7, 1e-5))
+    freq = stepped_frequencies(64, 1e6, 8.0, 1.0, 4.0, 2048.0).cuda()
+    gu, down = torch.randn(experts, 2 * ff, width, **bf) * 0.02, torch.randn(experts, width, ff, **bf) * 0.02
+    gain, vec = torch.ones(width, **bf), torch.ones(width, **bf)
+
+    def rows(T, case):
+        x = torch.randn(T, width, **bf)
+        lg = torch.randn(T, experts + 4, device="cuda")
+        corr = torch.zeros(experts + 4, device="cuda")
+        idx, w = K.router_topk(lg[:, :experts].contiguous(), top, "softmax")
+        add("router_topk", case, lambda: K.router_topk(lg, top, "softmax", corr, scale=2.0, renorm=False), nbytes=T * (experts + 4) * 4.0)
+        n = T * top
+        used = min(n, experts) if n < experts else experts
+        wb, fl = used * 3.0 * ff * width * 2, 6.0 * n * ff * width
+        add("experts, decoder with GEGLU", case, lambda: M.experts_forward_bf16(x, idx, w, gu, down, "geglu"), fl, tf, wb, like="routed decoder")
+        add("experts, clamped", case, lambda: P.expert_outputs(x, idx, w, gu, down, "clamped", 7.0), fl, tf, wb)
+        r = P.expert_outputs(x, idx, w, gu, down, "clamped", 7.0)
+        a, h, hb = torch.randn(T, width, device="cuda"), torch.randn(T, width, device="cuda"), torch.randn(T, width, **bf)
+        add("add_rmsnorm", case, lambda: K.add_rmsnorm(x, hb, gain, 1e-5), nbytes=T * width * 8, like="routed decoder")
+        add("norm_add_norm", case, lambda: K.norm_add_norm(a, gain, hb, gain, 1e-5), nbytes=T * width * 10, like="routed decoder")
+        per = 4 if r.sum is not None else 2 * top
+        add("stream_step, experts", case, lambda: P.stream_step(h, a, 0.3, r, None, True, (gain, gain), 1e-5, None), nbytes=T * width * (16.0 + per))
+        add("stream_step, pass", case, lambda: P.stream_step(h, a, 1.0, None, vec, False, (gain, gain), 1e-5, None), nbytes=T * width * 12.0)
+
+    for B, q in ((1, 4096), (8, 512)):
+        case, T = f"{B} x {q} tokens", B * q
+        m = _meta(B, q, q)
+        n_in = (heads + 2 * kv_heads) * D
+        y = torch.randn(T, n_in, **bf)
+        pq, pk, pv = y.split([heads * D, kv_heads * D, kv_heads * D], 1)
+        kc = torch.randn(m.page_table.numel(), 64, kv_heads, D, **bf)
+        vc, out = torch.randn_like(kc), torch.empty(T, heads * D, **bf)
+        Q = torch.randn(T, heads, D, **bf)
+        fl = 4.0 * heads * D * T * (q + 1) / 2
+        add("attention_prefill", case, lambda: K.attention_prefill(Q, kc, vc, m, 0.05), fl, tf, like="routed decoder")
+        add("  split_p", case, lambda: H.attention_exact(Q, kc, vc, m, 0.05, out=out), fl, tf)
+        add("  capped, sink, temperature", case, lambda: H.attention_exact(Q, kc, vc, m, 0.05, out=out, form=cap), fl, tf)
+        keys = sum(i % chunk + 1 for i in range(q)) / q
+        add("difference of maps (64 / 128)", case, lambda: H.attention_exact(Q, kc, vc, m, 0.05, out=out, form=dif), heads * T * keys * (4.0 * 64 + 4.0 * 128), tf)
+        inv, g = torch.ones(D // 2, device="cuda"), torch.ones(D, **bf)
+        add("qk_norm_rope_append", case, lambda: K.qk_norm_rope_append(y, heads, kv_heads, D, g, g, False, inv, m, kc, vc, 1e-5), nbytes=T * n_in * 4,
+            like="routed decoder")
+        add("rotate_append", case, lambda: P.rotate_append(pq, pk, pv, 2 * heads, 2 * kv_heads, 64, freq, m, kc, vc), nbytes=T * n_in * 4)
+        add("append", case, lambda: P.rotate_append(None, pk, pv, heads, kv_heads, D, None, m, kc, vc), nbytes=T * 2 * kv_heads * D * 4)
+        rows(T, case)
+    for B in (1, 32, 128):
+        case, ctx = f"{B} x 1 token", 2048
+        m = _meta(B, 1, ctx)
+        n_in = (heads + 2 * kv_heads) * D
+        y = torch.randn(B, n_in, **bf)
+        pq, pk, pv = y.split([heads * D, kv_heads * D, kv_heads * D], 1)
+        kc = torch.randn(m.page_table.numel(), 64, kv_heads, D, **bf)
+        vc, Q = torch.randn_like(kc), torch.randn(B, heads, D, **bf)
+        out = torch.empty(B, heads * D, **bf)
+        nb = 2.0 * B * ctx * kv_heads * D * 2
+        add("paged_attention_decode", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1), nbytes=nb, like="routed decoder")
+        add("  capped, sink, temperature", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1, out=out, form=cap), nbytes=nb)
+        add("difference of maps (64 / 128)", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1, out=out, form=dif), nbytes=nb)
+        inv, g = torch.ones(D // 2, device="cuda"), torch.ones(D, **bf)
+        add("qk_norm_rope_append", case, lambda: K.qk_norm_rope_append(y, heads, kv_heads, D, g, g, False, inv, m, kc, vc, 1e-5), nbytes=B * n_in * 4,
+            like="routed decoder")
+        add("rotate_append", case, lambda: P.rotate_append(pq, pk, pv, 2 * heads, 2 * kv_heads, 64, freq, m, kc, vc), nbytes=B * n_in * 4)
+        rows(B, case)
     assert K.last_status() == 0
     return add.rows

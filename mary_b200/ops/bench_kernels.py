@@ -571,6 +571,9 @@ if __name__ == "__main__":
     if what == "rokarax":
         from .bench_hybrid import run_rokarax
         run_rokarax(*nums)
+    if what == "nipurax":
+        from .bench_hybrid import run_nipurax
+        run_nipurax(*nums)
     if what == "moeprefill":
         bench_moeprefill(*nums)
     if what == "bf16moe":
