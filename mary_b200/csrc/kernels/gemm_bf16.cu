@@ -267,6 +267,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tm_r, const __grid_constant
       const uint32_t idesc = idesc_bf16(BM, BN);
       int stage = 0; uint32_t phase = 0;
       int it = 0;
+      if (g_tiles) pdl_wait();             // the walk over the tiles reads the routing plan, which the previous kernel may still be writing
       WorkIter<LEAN> iter(p);
       WorkItem w;
       for (; iter.next(w); ++it) {
