@@ -69,13 +69,6 @@ struct FaParams {
   int* status;
 };
 
-// Two values at a time through the packed 32-bit pipes: a * b + c.
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-  uint64_t d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(*(const uint64_t*)&a), "l"(*(const uint64_t*)&b), "l"(*(const uint64_t*)&c));
-  return *(float2*)&d;
-}
-
 __device__ __forceinline__ uint64_t fa_desc_kmajor_noswz(uint32_t addr, uint32_t lbo_bytes, uint32_t sbo_bytes) {
   return (uint64_t)((addr >> 4) & 0x3FFF) | ((uint64_t)(lbo_bytes >> 4) << 16) | ((uint64_t)(sbo_bytes >> 4) << 32) | (1ull << 46);
 }
@@ -296,31 +289,12 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       float mx;
       if constexpr (MAPS > 0) {
         if (p.f.cap > 0.f) {
-          // the capped score in units of log2: small arguments (all of a warp's) by the series of tanh, two scores at a time
-          float top = 0.f;
+          float v[KB];
 #pragma unroll
-          for (int j = 0; j < KB; ++j) top = fmaxf(top, fabsf(__uint_as_float(sr[j])));
-          const float k = sl2 / (p.f.cap * 1.4426950408889634f);             // raw score -> argument of tanh
-          if (__all_sync(0xffffffffu, top * fabsf(k) <= 0.25f)) {
-            const float k2 = k * k, c1 = sl2, c3 = c1 * k2 * (-1.0f / 3.0f), c5 = c1 * k2 * k2 * (2.0f / 15.0f);
-            const float c7 = c1 * k2 * k2 * k2 * (-17.0f / 315.0f), c9 = c1 * k2 * k2 * k2 * k2 * (62.0f / 2835.0f);
-            const float2 zero = make_float2(0.f, 0.f);
+          for (int j = 0; j < KB; ++j) v[j] = __uint_as_float(sr[j]);
+          cap_scores<KB>(v, sl2, p.f.cap);
 #pragma unroll
-            for (int j = 0; j < KB; j += 2) {
-              const float2 x = make_float2(__uint_as_float(sr[j]), __uint_as_float(sr[j + 1])), y = fma2(x, x, zero);
-              float2 q = fma2(y, make_float2(c9, c9), make_float2(c7, c7));
-              q = fma2(q, y, make_float2(c5, c5));
-              q = fma2(q, y, make_float2(c3, c3));
-              q = fma2(q, y, make_float2(c1, c1));
-              q = fma2(q, x, zero);
-              sr[j] = __float_as_uint(q.x);
-              sr[j + 1] = __float_as_uint(q.y);
-            }
-          } else {
-            const float c = p.f.cap * 1.4426950408889634f;
-#pragma unroll
-            for (int j = 0; j < KB; ++j) sr[j] = __float_as_uint(c * tanh_32(__uint_as_float(sr[j]) * k));
-          }
+          for (int j = 0; j < KB; ++j) sr[j] = __float_as_uint(v[j]);
         }
       }
       const float sc = MAPS > 0 && p.f.cap > 0.f ? 1.0f : sl2;               // factor on what `sr` now holds
@@ -597,7 +571,7 @@ MARY_API int mary_attention_prefill(const void* q, const void* kcache, const voi
   if (form && (p.f.chunk > 0 || p.f.sink || p.f.temp_every > 0 || p.f.cap > 0.f)) {
     if (DK == 64) return launch_fa<64, 64, true, false, 1>(tq, tk, tv, p, NB, s);
     if (DK == 128) return launch_fa<128, 128, true, false, 1>(tq, tk, tv, p, NB, s);
-    if (DK == 192) return launch_fa<192, 128, true, false, 1>(tq, tk, tv, p, NB, s);
+    if (DK == 192) return MARY_ERR_BAD_ARG;
     return launch_fa<256, 256, true, false, 1>(tq, tk, tv, p, NB, s);
   }
   if (bias) {

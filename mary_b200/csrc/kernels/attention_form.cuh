@@ -39,6 +39,41 @@ __device__ __forceinline__ float tanh_32(float x) {
   if (a <= 0.5f) return tanh_series(x);
   return copysignf(1.0f - __fdividef(2.0f, __expf(2.0f * fminf(a, 20.0f)) + 1.0f), x);
 }
+// Two values at a time through the packed 32-bit pipes: a * b + c.
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(*(const uint64_t*)&a), "l"(*(const uint64_t*)&b), "l"(*(const uint64_t*)&c));
+  return *(float2*)&d;
+}
+
+// N raw scores of a lane's row -> cap * tanh(score * scale / cap) in units of log2, given scale_log2 = scale * log2(e).  Where no score of the
+// warp is beyond a quarter of the cap (lanes that hold no scores: `held` false) the series of tanh to the ninth power is exact to 32 bits.
+template <int N>
+__device__ __forceinline__ void cap_scores(float (&s)[N], float scale_log2, float cap, bool held = true) {
+  float top = 0.f;
+#pragma unroll
+  for (int j = 0; j < N; ++j) top = fmaxf(top, fabsf(s[j]));
+  const float c = cap * 1.4426950408889634f, k = scale_log2 / c;                // raw score -> argument of tanh
+  if (__all_sync(0xffffffffu, !held || top * fabsf(k) <= 0.25f)) {
+    const float k2 = k * k, c1 = scale_log2, c3 = c1 * k2 * (-1.0f / 3.0f), c5 = c1 * k2 * k2 * (2.0f / 15.0f);
+    const float c7 = c1 * k2 * k2 * k2 * (-17.0f / 315.0f), c9 = c1 * k2 * k2 * k2 * k2 * (62.0f / 2835.0f);
+    const float2 zero = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < N; j += 2) {
+      const float2 x = make_float2(s[j], s[j + 1]), y = fma2(x, x, zero);
+      float2 q = fma2(y, make_float2(c9, c9), make_float2(c7, c7));
+      q = fma2(q, y, make_float2(c5, c5));
+      q = fma2(q, y, make_float2(c3, c3));
+      q = fma2(q, y, make_float2(c1, c1));
+      q = fma2(q, x, zero);
+      s[j] = q.x;
+      s[j + 1] = q.y;
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < N; ++j) s[j] = c * tanh_32(s[j] * k);
+  }
+}
 __device__ __forceinline__ float cap_score(float s, float cap) { return cap > 0.f ? cap * tanh_32(s / cap) : s; }
 
 }  // namespace mary

@@ -19,6 +19,11 @@
 //            its lanes 0-15: scale, optional soft-cap, causal / sliding-window mask, running max with lazy rescale of O, P to
 //            shared memory; at the end O / l to global, or f32 partials when the key range is split.
 // Every wait is bounded and reports through the status word.
+//
+// MAPS = 1 and 2 are the forms with exact softmax weights (P as the sum of two bf16 values) and what attention_form.cuh lists, over 32- or
+// 64-token pages.  Two maps of 64 dims each (key and query rows [map 0 | map 1]) are rows of ONE tile: a row of map m holds its query in
+// chunk m and zeros in the other, so Q K^T over the whole key row is the score of its map; rows of map 0 are 0 .. 31, of map 1 32 .. 63.
+#include "attention_form.cuh"
 #include "common.cuh"
 #include "host_utils.h"
 
@@ -34,7 +39,7 @@ constexpr float RESCALE_THRESHOLD = 8.0f;
 constexpr int AHEAD = 1;                          // blocks by which Q K^T leads P V
 constexpr float LOG2E = 1.4426950408889634f;
 
-template <int D, int PAGE>
+template <int D, int PAGE, int MAPS>
 struct GCfg {
   static constexpr int NCH = D / CHUNK;
   static constexpr int Q_CHUNK_BYTES = TR * 128;                  // 8 KB
@@ -44,12 +49,14 @@ struct GCfg {
   static constexpr int PPB = 32 / PAGE;                           // pages per pipeline stage: a stage always holds KB = 32 keys
   static constexpr int KB = PAGE * PPB;
   static constexpr int STAGE_BYTES = 2 * PAGE_BYTES * PPB;        // [page of the stage][K page | V page]
-  static constexpr int STAGES = D == 256 ? 5 : 5;
-  static constexpr int P_BYTES = TR * KB * 2;
+  static constexpr int STAGES = MAPS > 0 ? 4 : 5;                 // two CTAs of D = 128 share an SM
+  static constexpr int P_HALF = TR * KB * 2;                      // rounded weights; with MAPS > 0 their rounding errors behind them
+  static constexpr int P_BYTES = MAPS > 0 ? 2 * P_HALF : P_HALF;
   static constexpr int SMEM = Q_BYTES + STAGES * STAGE_BYTES + NPBUF * P_BYTES + 1024 + 256;
   static constexpr int TMEM_COLS = D <= 128 ? 256 : 512;          // S: 3 x PAGE columns at 0..95, O: D columns at 128..
   static_assert(D % CHUNK == 0 && D <= 256 && (PAGE == 16 || PAGE == 32), "head dim 64..256 in chunks of 64, pages of 16 or 32 tokens");
   static_assert(NSBUF * KB <= 128 && SMEM <= 232448, "budget");
+  static_assert(MAPS < 2 || D == 2 * CHUNK, "two maps: one 64-dim chunk each");
 };
 
 struct GqaParams {
@@ -60,6 +67,9 @@ struct GqaParams {
   int max_pages, Hq, Hkv, G, RQ, nsplit, window;
   float scale, softcap;
   int* status;
+  int page;                // tokens per page (MAPS > 0: 32 or 64)
+  int64_t out_ld;          // elements between the output rows of two tokens
+  MaryAttnForm f;
 };
 
 __device__ __forceinline__ void tma_load_5d(void* dst, const CUtensorMap* m, uint64_t* bar, int x, int y, int z, int w, int v) {
@@ -80,12 +90,12 @@ __device__ __forceinline__ uint64_t desc_mnmajor_sw128(uint32_t addr, uint32_t l
          (2ull << 61);
 }
 
-template <int D, int PAGE>
+template <int D, int PAGE, int MAPS>
 __global__ void __launch_bounds__(NTHREADS, 1)
 gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                      const GqaParams p) {
   pdl_sync();
-  using C = GCfg<D, PAGE>;
+  using C = GCfg<D, PAGE, MAPS>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
@@ -112,8 +122,10 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   const int qlen = q_end - p.q_start[seq];
   const int pos0 = kvlen - qlen + (tok0 - p.q_start[seq]);           // position of the block's first query token
   const int k_hi = pos0 + nq;                                         // keys [k_lo, k_hi) are visible to some row
-  const int k_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
-  constexpr int KB = GCfg<D, PAGE>::KB, PPB = GCfg<D, PAGE>::PPB;
+  int k_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+  if constexpr (MAPS > 0) k_lo = max(k_lo, first_key(p.f, pos0));
+  constexpr int KB = C::KB, PPB = C::PPB;
+  constexpr int MR = MAPS == 2 ? TR / 2 : TR;                         // rows of one map
   const int blk_first = k_lo / KB;
   const int nblk_total = (k_hi + KB - 1) / KB - blk_first;
   const int n_pages = (k_hi + PAGE - 1) / PAGE;                       // pages of this sequence that hold visible keys
@@ -138,7 +150,9 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     const int box_rows = p.G * p.RQ;
     for (int i = threadIdx.x; i < C::NCH * (TR - box_rows) * 8; i += NTHREADS) {
       const int c = i / ((TR - box_rows) * 8), rem = i % ((TR - box_rows) * 8);
-      *(uint4*)(sQ + c * C::Q_CHUNK_BYTES + (box_rows + rem / 8) * 128 + (rem % 8) * 16) = make_uint4(0u, 0u, 0u, 0u);
+      int row = box_rows + rem / 8;
+      if (MAPS == 2 && c == 1 && row < MR + box_rows) row -= box_rows;     // chunk 1 is filled from row MR on: 0 .. MR - 1 and the rest are zero
+      *(uint4*)(sQ + c * C::Q_CHUNK_BYTES + row * 128 + (rem % 8) * 16) = make_uint4(0u, 0u, 0u, 0u);
     }
     fence_proxy_async();
   }
@@ -153,7 +167,8 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     if (nblk > 0 && lane == 0) {
       // the box holds G * RQ rows; rows of tokens past the block's end belong to other sequences (or are zero fill) and stay unused
       mbar_expect_tx(q_full, (uint32_t)(C::NCH * p.G * p.RQ * 128));
-      for (int c = 0; c < C::NCH; ++c) tma_load_3d(sQ + c * C::Q_CHUNK_BYTES, &tm_q, q_full, c * CHUNK, kvh * p.G, tok0);
+      for (int c = 0; c < C::NCH; ++c)
+        tma_load_3d(sQ + c * C::Q_CHUNK_BYTES + (MAPS == 2 ? c * MR * 128 : 0), &tm_q, q_full, c * CHUNK, kvh * p.G, tok0);
       const int* pt = p.page_table + (int64_t)seq * p.max_pages;
       int stage = 0; uint32_t phase = 0;
       for (int b = b_lo; b < b_hi; ++b) {
@@ -163,9 +178,15 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
 #pragma unroll
         for (int pp = 0; pp < PPB; ++pp) {
           const int pi = b * PPB + pp;
-          const int page = pt[pi < n_pages ? pi : b * PPB];       // a page past the visible keys repeats the block's first page (masked)
-          tma_load_5d(st + pp * 2 * C::PAGE_BYTES, &tm_k, &k_full[stage], 0, 0, 0, kvh, page);
-          tma_load_5d(st + pp * 2 * C::PAGE_BYTES + C::PAGE_BYTES, &tm_v, &k_full[stage], 0, 0, 0, kvh, page);
+          int page, tok = 0;
+          if constexpr (MAPS > 0) {
+            page = pt[b * KB / p.page];
+            tok = b * KB % p.page;
+          } else {
+            page = pt[pi < n_pages ? pi : b * PPB];               // a page past the visible keys repeats the block's first page (masked)
+          }
+          tma_load_5d(st + pp * 2 * C::PAGE_BYTES, &tm_k, &k_full[stage], 0, tok, 0, kvh, page);
+          tma_load_5d(st + pp * 2 * C::PAGE_BYTES + C::PAGE_BYTES, &tm_v, &k_full[stage], 0, tok, 0, kvh, page);
         }
         if (++stage == C::STAGES) { stage = 0; phase ^= 1; }
       }
@@ -217,6 +238,9 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           umma_f16(tmem_O, desc_kmajor_noswz(p_addr + pb * C::P_BYTES + kk * 2 * (TR * 16), TR * 16, 128),
                    desc_mnmajor_sw128(st_addr + pp * 2 * C::PAGE_BYTES + C::PAGE_BYTES + in_page * 128, C::PAGE_CHUNK_BYTES, 1024), idesc_o,
                    (i > 0 || kk > 0) ? 1u : 0u);
+          if constexpr (MAPS > 0)
+            umma_f16(tmem_O, desc_kmajor_noswz(p_addr + pb * C::P_BYTES + C::P_HALF + kk * 2 * (TR * 16), TR * 16, 128),
+                     desc_mnmajor_sw128(st_addr + pp * 2 * C::PAGE_BYTES + C::PAGE_BYTES + in_page * 128, C::PAGE_CHUNK_BYTES, 1024), idesc_o, 1u);
         }
         umma_commit(&k_empty[stage]);       // the stage may be overwritten once PV has read it
         umma_commit(&pv_done[pb]);
@@ -226,10 +250,17 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     // ------------------------------------------------------------------ softmax warps: 16 query rows per warp
     const int q4 = warp & 3;
     const int r = q4 * 16 + (lane & 15);            // accumulator row held by this lane (lanes 16-31 hold nothing)
-    const bool row_ok = lane < 16 && r < nrows;
-    const int qpos = pos0 + r / p.G;
+    const int rm = r % MR;                          // row within its map
+    const bool row_ok = lane < 16 && rm < nrows;
+    const int qpos = pos0 + rm / p.G;
     const uint32_t lane_off = (uint32_t)(q4 * 32) << 16;
-    const float sc2 = p.scale * LOG2E;
+    float sc2 = p.scale * LOG2E;
+    int lo_key = 0, full_from = 0;
+    if constexpr (MAPS > 0) {
+      sc2 *= query_temperature(p.f, qpos);
+      lo_key = first_key(p.f, qpos);
+      full_from = first_key(p.f, pos0 + nq - 1);
+    }
     float m_ref = -INFINITY, l = 0.f;
     for (int i = 0; i < nblk; ++i) {
       const int sb = i % NSBUF, pb = i & 1;
@@ -245,23 +276,34 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       // A block that every row sees entirely (all but the last of a decode step and the window's edge) takes the short path: no
       // per-element mask, the maximum on the raw scores, one fused multiply-add and one exponential per element.  A row's scores
       // are processed by ONE lane in sequence, so the instruction count of this loop is the kernel's cycle time.
-      const bool full_blk = p.softcap <= 0.f && key0 + KB - 1 <= pos0 && (p.window <= 0 || pos0 + nq - 1 - key0 < p.window);
-      const float* sf = (const float*)sr;
+      const bool full_blk = p.softcap <= 0.f && key0 + KB - 1 <= pos0 && (p.window <= 0 || pos0 + nq - 1 - key0 < p.window) && key0 >= full_from &&
+                            (MAPS == 0 || sc2 > 0.f);
+      float sf[KB];
+#pragma unroll
+      for (int j = 0; j < KB; ++j) sf[j] = __uint_as_float(sr[j]);
+      float sc = sc2;                                // factor on what sf holds
+      if constexpr (MAPS > 0) {
+        if (p.f.cap > 0.f) {
+          sc = 1.f;
+          cap_scores<KB>(sf, sc2, p.f.cap, lane < 16);
+        }
+      }
       float sv[KB];
       float mx;
       if (full_blk) {
         mx = sf[0];
 #pragma unroll
         for (int j = 1; j < KB; ++j) mx = fmaxf(mx, sf[j]);
-        mx *= sc2;
+        mx *= sc;
       } else {
         mx = -INFINITY;
 #pragma unroll
         for (int j = 0; j < KB; ++j) {
           const int kp = key0 + j;
-          const bool ok = row_ok && kp <= qpos && (p.window <= 0 || qpos - kp < p.window);
+          const bool ok = row_ok && kp <= qpos && (p.window <= 0 || qpos - kp < p.window) && kp >= lo_key;
           float x = sf[j];
-          if (p.softcap > 0.f) x = p.softcap * tanhf(x * p.scale / p.softcap) * LOG2E;
+          if constexpr (MAPS > 0) x *= sc;
+          else if (p.softcap > 0.f) x = p.softcap * tanhf(x * p.scale / p.softcap) * LOG2E;
           else x *= sc2;
           sv[j] = ok ? x : -INFINITY;
           mx = fmaxf(mx, sv[j]);
@@ -273,16 +315,21 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       const bool first = (m_ref == -INFINITY);
       float corr = 1.f;
       if (need) { corr = first ? 0.f : exp2f(m_ref - mx); m_ref = mx; }
-      uint32_t pw[KB / 2];
+      uint32_t pw[KB / 2], pl[MAPS > 0 ? KB / 2 : 1];
       float psum = 0.f;
       if (full_blk) {
         const float nm = -m_ref;
 #pragma unroll
         for (int j = 0; j < KB / 2; ++j) {
-          const float a = exp2f(fmaf(sf[2 * j], sc2, nm));
-          const float b = exp2f(fmaf(sf[2 * j + 1], sc2, nm));
+          const float a = exp2f(fmaf(sf[2 * j], sc, nm));
+          const float b = exp2f(fmaf(sf[2 * j + 1], sc, nm));
           __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
           pw[j] = *(uint32_t*)&h;
+          if constexpr (MAPS > 0) {
+            const float2 back = __bfloat1622float2(h);
+            __nv_bfloat162 lo = __floats2bfloat162_rn(a - back.x, b - back.y);
+            pl[j] = *(uint32_t*)&lo;
+          }
           psum += a + b;
         }
       } else {
@@ -293,7 +340,13 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
           pw[j] = *(uint32_t*)&h;
           float2 back = __bfloat1622float2(h);
-          psum += back.x + back.y;
+          if constexpr (MAPS > 0) {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(a - back.x, b - back.y);
+            pl[j] = *(uint32_t*)&lo;
+            psum += a + b;
+          } else {
+            psum += back.x + back.y;
+          }
         }
       }
       l = l * corr + psum;
@@ -322,6 +375,11 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
 #pragma unroll
         for (int c = 0; c < KB / 8; ++c)
           *(uint4*)(sP + pb * C::P_BYTES + c * (TR * 16) + r * 16) = make_uint4(pw[4 * c], pw[4 * c + 1], pw[4 * c + 2], pw[4 * c + 3]);
+        if constexpr (MAPS > 0) {
+#pragma unroll
+          for (int c = 0; c < KB / 8; ++c)
+            *(uint4*)(sP + pb * C::P_BYTES + C::P_HALF + c * (TR * 16) + r * 16) = make_uint4(pl[4 * c], pl[4 * c + 1], pl[4 * c + 2], pl[4 * c + 3]);
+        }
       }
       fence_proxy_async();       // make the generic-proxy writes of P visible to the tensor core
       tc_fence_before();
@@ -331,16 +389,21 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     // ------------------------------------------------------------------ write out
     if (!mbar_wait(&pv_done[(nblk - 1) & 1], ((nblk - 1) >> 1) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
     tc_fence_after();
-    const float inv_l = l > 0.f ? 1.f / l : 0.f;
-    const int tq = tok0 + r / p.G, head = kvh * p.G + r % p.G;
+    const int tq = tok0 + rm / p.G, head = kvh * p.G + rm % p.G;
+    const bool whole = MAPS < 2 && p.nsplit == 1;          // nothing to merge
+    float inv_l = l;
+    if constexpr (MAPS == 1) {
+      if (p.f.sink && whole && row_ok) inv_l += exp2f(fmaf(p.f.sink[head], LOG2E, -m_ref));
+    }
+    inv_l = inv_l > 0.f ? 1.f / inv_l : 0.f;
 #pragma unroll 1
     for (int c0 = 0; c0 < D; c0 += 32) {
       uint32_t o[32];
       tmem_ld_32x32b_x32(tmem_O + lane_off + c0, o);
       tmem_ld_wait();
       if (row_ok) {
-        if (p.nsplit == 1) {
-          __nv_bfloat16* dst = p.out + ((int64_t)tq * p.Hq + head) * D + c0;
+        if (whole) {
+          __nv_bfloat16* dst = p.out + (int64_t)tq * p.out_ld + head * D + c0;
           uint4 w[4];
           uint32_t* wp = (uint32_t*)w;
 #pragma unroll
@@ -357,14 +420,14 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         }
       }
     }
-    if (row_ok && p.nsplit > 1) {
+    if (row_ok && !whole) {
       float* ml = p.part_ml + ((((int64_t)nb * p.Hkv + kvh) * p.nsplit + split) * TR + r) * 2;
       ml[0] = m_ref; ml[1] = l;
     }
-  } else if (warp >= 2 && p.nsplit > 1) {
+  } else if (warp >= 2 && (p.nsplit > 1 || MAPS == 2)) {
     // an empty split still has to publish neutral partials
     const int r = (warp & 3) * 16 + (lane & 15);
-    if (lane < 16 && r < nrows) {
+    if (lane < 16 && r % MR < nrows) {
       float* ml = p.part_ml + ((((int64_t)nb * p.Hkv + kvh) * p.nsplit + split) * TR + r) * 2;
       ml[0] = -INFINITY; ml[1] = 0.f;
     }
@@ -402,18 +465,76 @@ __global__ void gqa_tc_combine_kernel(const GqaParams p, int D) {
   }
 }
 
+// The same with the sink (one map), or for the difference of two maps: out = rms(o0 - mix * o1) * post.  128 threads.
+template <int D, int MAPS>
+__global__ void __launch_bounds__(128) gqa_tc_combine_form_kernel(const GqaParams p) {
+  pdl_sync();
+  constexpr int E = D / 128;
+  __shared__ float red[4];
+  const int nb = blockIdx.x, kvh = blockIdx.y, r = blockIdx.z;
+  const int seq = p.blk_seq[nb], tok0 = p.blk_q0[nb];
+  const int nq = min(p.RQ, p.q_start[seq + 1] - tok0);
+  if (r >= nq * p.G) return;
+  const int tq = tok0 + r / p.G, head = kvh * p.G + r % p.G;
+  float y[E];
+#pragma unroll
+  for (int e = 0; e < E; ++e) y[e] = 0.f;
+#pragma unroll
+  for (int map = 0; map < MAPS; ++map) {
+    const int64_t base = (((int64_t)nb * p.Hkv + kvh) * p.nsplit) * TR + map * (TR / 2) + r;
+    float mm = -INFINITY, ll = 0.f, acc[E];
+#pragma unroll
+    for (int e = 0; e < E; ++e) acc[e] = 0.f;
+    for (int s = 0; s < p.nsplit; ++s) mm = fmaxf(mm, p.part_ml[(base + (int64_t)s * TR) * 2]);
+    for (int s = 0; s < p.nsplit; ++s) {
+      const int64_t pi = base + (int64_t)s * TR;
+      const float ms = p.part_ml[pi * 2];
+      if (ms == -INFINITY) continue;
+      const float c = exp2f(ms - mm);
+      ll = fmaf(p.part_ml[pi * 2 + 1], c, ll);
+#pragma unroll
+      for (int e = 0; e < E; ++e) acc[e] = fmaf(p.part_o[pi * D + threadIdx.x + 128 * e], c, acc[e]);
+    }
+    float norm = 0.f;
+    if (MAPS == 1 && p.f.sink) {
+      const float sk = p.f.sink[head] * LOG2E, top = fmaxf(mm, sk), c = exp2f(mm - top);
+      norm = c / fmaf(ll, c, exp2f(sk - top));
+    } else if (ll > 0.f) norm = 1.f / ll;
+    if (map == 1) norm *= -p.f.mix;
+#pragma unroll
+    for (int e = 0; e < E; ++e) y[e] = fmaf(acc[e], norm, y[e]);
+  }
+  float c = 1.f;
+  if constexpr (MAPS == 2) {
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e) ss = fmaf(y[e], y[e], ss);
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    c = p.f.post * rsqrtf((red[0] + red[1] + red[2] + red[3]) / D + p.f.eps);
+  }
+#pragma unroll
+  for (int e = 0; e < E; ++e) p.out[(int64_t)tq * p.out_ld + head * D + threadIdx.x + 128 * e] = __float2bfloat16(y[e] * c);
+}
+
 typedef CUresult (*PFN_encode)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
                                const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-template <int D, int PAGE>
+template <int D, int PAGE, int MAPS = 0>
 int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const GqaParams& p, int NB, cudaStream_t s) {
-  using C = GCfg<D, PAGE>;
+  using C = GCfg<D, PAGE, MAPS>;
   static MarySmemSlots smem_set = {};
-  if (int rc = mary_ensure_dyn_smem((const void*)gqa_decode_tc_kernel<D, PAGE>, C::SMEM, &smem_set)) return rc;
-  MARY_LAUNCH((gqa_decode_tc_kernel<D, PAGE>), dim3(NB, p.Hkv, p.nsplit), NTHREADS, C::SMEM, s, tq, tk, tv, p);
+  if (int rc = mary_ensure_dyn_smem((const void*)gqa_decode_tc_kernel<D, PAGE, MAPS>, C::SMEM, &smem_set)) return rc;
+  MARY_LAUNCH((gqa_decode_tc_kernel<D, PAGE, MAPS>), dim3(NB, p.Hkv, p.nsplit), NTHREADS, C::SMEM, s, tq, tk, tv, p);
   MARY_CHECK_LAUNCH();
-  if (p.nsplit > 1) {
+  if constexpr (MAPS > 0) {
+    if (p.nsplit > 1 || MAPS == 2) {
+      MARY_LAUNCH((gqa_tc_combine_form_kernel<D, MAPS>), dim3(NB, p.Hkv, p.RQ * p.G), 128, 0, s, p);
+      MARY_CHECK_LAUNCH();
+    }
+  } else if (p.nsplit > 1) {
     MARY_LAUNCH(gqa_tc_combine_kernel, dim3(NB, p.Hkv, p.RQ * p.G), 128, 0, s, p, D);
     MARY_CHECK_LAUNCH();
   }
@@ -425,29 +546,39 @@ int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, 
 MARY_API int64_t mary_gqa_tc_scratch_floats(int NB, int Hkv, int nsplit, int D) {
   return nsplit > 1 ? (int64_t)NB * Hkv * nsplit * TR * (D + 2) : 0;
 }
+// The forms: 32- or 64-token pages; one map of D = 128 or 256, or two maps in key rows of D = 128 (values as wide).
+MARY_API int mary_gqa_tc_form_supported(int D, int page_size, int G, int RQ, int maps) {
+  return ((D == 128 || (D == 256 && maps == 1)) && (page_size == 32 || page_size == 64) && G >= 1 && RQ >= 1 && G * RQ <= (maps == 2 ? TR / 2 : TR)) ? 1 : 0;
+}
 MARY_API int mary_gqa_tc_supported(int D, int page_size, int G, int RQ) {
   return ((D == 128 || D == 256) && (page_size == 16 || page_size == 32) && G >= 1 && RQ >= 1 && G * RQ <= TR && G <= 256 && RQ <= 256) ? 1 : 0;
 }
 
 // q [T, Hq, D] bf16; K / V caches [pages, page_size, Hkv, D] bf16, contiguous; out [T, Hq, D] bf16.  blk_seq / blk_q0: NB blocks of at
-// most RQ query tokens of one sequence (q0 is a global token row).  G = Hq / Hkv heads share a kv head; G * RQ <= 64.
+// most RQ query tokens of one sequence (q0 is a global token row).  G = Hq / Hkv heads share a kv head; G * RQ <= 64.  form (or null):
+// exact softmax weights and what attention_form.cuh lists, see mary_gqa_tc_form_supported; its two maps need scratch for any nsplit (ask for 2).
+// out_ld: elements between the output rows of two tokens (0: Hq * D).
 MARY_API int mary_gqa_decode_tc(const void* q, const void* kc, const void* vc, void* out, const int* page_table, const int* kv_len,
                                 const int* q_start, const int* blk_seq, const int* blk_q0, int NB, int T, int num_pages, int max_pages,
                                 int page_size, int Hq, int Hkv, int D, int RQ, int nsplit, int window, float scale, float softcap,
-                                float* scratch, cudaStream_t s) {
+                                float* scratch, const MaryAttnForm* form, int64_t out_ld, cudaStream_t s) {
   if (NB <= 0) return MARY_OK;
   if (Hkv < 1 || Hq % Hkv) return MARY_ERR_BAD_ARG;
   const int G = Hq / Hkv;
-  if (!mary_gqa_tc_supported(D, page_size, G, RQ)) return MARY_ERR_BAD_ARG;
+  const int maps = form ? (form->maps == 2 ? 2 : 1) : 0;
+  if (maps ? !mary_gqa_tc_form_supported(D, page_size, G, RQ, maps) || softcap > 0.f : !mary_gqa_tc_supported(D, page_size, G, RQ)) return MARY_ERR_BAD_ARG;
+  const int64_t q_ld = form && form->q_ld > 0 ? form->q_ld : (int64_t)Hq * D;
+  if (out_ld <= 0) out_ld = (int64_t)Hq * D;
+  if (q_ld % 8 || out_ld % 8 || ((uintptr_t)out & 15) || (maps == 2 && form->sink)) return MARY_ERR_BAD_ARG;
   if (nsplit < 1) nsplit = 1;
-  if (nsplit > 1 && !scratch) return MARY_ERR_BAD_ARG;
+  if ((nsplit > 1 || maps == 2) && !scratch) return MARY_ERR_BAD_ARG;
   PFN_encode enc = (PFN_encode)mary_encode_fn();
   if (!enc) return MARY_ERR_CUDA;
   CUtensorMap tq, tk, tv;
   {
     // q as [tokens][heads][D]: the box takes one 64-dim chunk of the G heads of a kv head for RQ consecutive tokens
     cuuint64_t dims[3] = {(cuuint64_t)D, (cuuint64_t)Hq, (cuuint64_t)T};
-    cuuint64_t strides[2] = {(cuuint64_t)D * 2, (cuuint64_t)Hq * D * 2};
+    cuuint64_t strides[2] = {(cuuint64_t)D * 2, (cuuint64_t)q_ld * 2};
     cuuint32_t box[3] = {CHUNK, (cuuint32_t)G, (cuuint32_t)RQ};
     cuuint32_t estr[3] = {1, 1, 1};
     if (((uintptr_t)q & 15) || enc(&tq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(q), dims, strides, box, estr,
@@ -460,7 +591,7 @@ MARY_API int mary_gqa_decode_tc(const void* q, const void* kc, const void* vc, v
     const void* base = which ? vc : kc;
     cuuint64_t dims[5] = {CHUNK, (cuuint64_t)page_size, (cuuint64_t)(D / CHUNK), (cuuint64_t)Hkv, (cuuint64_t)num_pages};
     cuuint64_t strides[4] = {(cuuint64_t)Hkv * D * 2, CHUNK * 2, (cuuint64_t)D * 2, (cuuint64_t)page_size * Hkv * D * 2};
-    cuuint32_t box[5] = {CHUNK, (cuuint32_t)page_size, (cuuint32_t)(D / CHUNK), 1, 1};
+    cuuint32_t box[5] = {CHUNK, (cuuint32_t)(page_size < 32 ? page_size : 32), (cuuint32_t)(D / CHUNK), 1, 1};
     cuuint32_t estr[5] = {1, 1, 1, 1, 1};
     if (((uintptr_t)base & 15) || enc(which ? &tv : &tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 5, const_cast<void*>(base), dims, strides, box, estr,
                                       CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
@@ -473,6 +604,10 @@ MARY_API int mary_gqa_decode_tc(const void* q, const void* kc, const void* vc, v
   p.part_ml = scratch ? scratch + (int64_t)NB * Hkv * nsplit * TR * D : nullptr;
   p.max_pages = max_pages; p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.RQ = RQ; p.nsplit = nsplit; p.window = window;
   p.scale = scale; p.softcap = softcap; p.status = mary_status_ptr();
+  p.page = page_size; p.out_ld = out_ld;
+  p.f = form ? *form : MaryAttnForm{};
+  if (maps == 2) return launch<128, 32, 2>(tq, tk, tv, p, NB, s);
+  if (maps == 1) return D == 128 ? launch<128, 32, 1>(tq, tk, tv, p, NB, s) : launch<256, 32, 1>(tq, tk, tv, p, NB, s);
   if (D == 128) return page_size == 16 ? launch<128, 16>(tq, tk, tv, p, NB, s) : launch<128, 32>(tq, tk, tv, p, NB, s);
   return page_size == 16 ? launch<256, 16>(tq, tk, tv, p, NB, s) : launch<256, 32>(tq, tk, tv, p, NB, s);
 }

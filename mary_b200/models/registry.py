@@ -74,7 +74,7 @@ FAMILIES = [
     Family("rokarax", lambda d: d.get("architecture") == "Rokarax", _load_rokarax, page_size=64, f32_on_gpu=True,
            kernels=_DENSE_KERNELS + ("attention_general", "attention_mla", "residual32", "linear_attention", "recurrent_scan", "latent", "state_space", "ssd_chunk")),
     Family("nipurax", lambda d: d.get("architecture") == "Nipurax", _load_nipurax, page_size=64, f32_on_gpu=True,
-           kernels=_DENSE_KERNELS + ("attention_general", "residual32", "parallel_stream", "moe", "expert_step")),
+           kernels=_DENSE_KERNELS + ("attention_general", "attention_gqa_tc", "residual32", "parallel_stream", "moe", "expert_step")),
     Family("gemma4", lambda d: str(d.get("model_type", "")).startswith("gemma4"), _load_gemma4),
     Family("mistral", lambda d: d.get("model_type") in ("mistral", "ministral", "qwen3", "mistral3"), _load_mistral),
 ]

@@ -169,8 +169,8 @@ def _group_rows(meta, group: str):
 
 def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, bias=None, gate=None, form=None):
     """Causal attention with scores, softmax weights and sums in 32 bits: the tensor-core prefill kernel with two-term weights for
-    sequences that bring more than ``DECODE_ROWS`` tokens, the bandwidth-oriented decode kernel for the others, the general kernel for
-    32-bit tensors and for head shapes those have no instantiation for.  ``out`` may be a row view ``[T, Hq * DV]``."""
+    sequences that bring more than ``DECODE_ROWS`` tokens, the bandwidth-oriented decode kernel for the others (its tensor-core twin where that takes
+    the ``form``), the general kernel for 32-bit tensors and for head shapes those have no instantiation for.  ``out`` may be a row view ``[T, Hq * DV]``."""
     T, Hq, DK = q.shape
     Hkv, DV = kcache.shape[2], vcache.shape[3]
     assert (q.is_contiguous() or form is not None) and kcache.is_contiguous() and vcache.stride(3) == 1 and kcache.shape[1] == meta.page_size
@@ -190,6 +190,8 @@ def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, b
         bf16 = bf16 and DK == DV and DK in (64, 128, 256)
         fast_prefill = bf16 and meta.page_size in (16, 64) and aligned
         fast_decode = bf16 and Hq // Hkv <= (4 if DK == 256 else 8) and (q.is_contiguous() or aligned)
+    tc_decode = form is not None and aligned and window == 0 and bias is None and gate is None and K.gqa_tc_form_supported(q, kcache, vcache, meta, form)
+    fast_decode = fast_decode or tc_decode
     if not (fast_prefill or fast_decode):
         return attention_general(q, kcache, vcache, meta, scale, out, **kw)
     if meta.max_q_len > DECODE_ROWS:
@@ -198,7 +200,9 @@ def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, b
         else:
             attention_general(q, kcache, vcache, meta, scale, out, "prefill", **kw)
     if K._q_blocks(meta, 1, "decode")[2]:
-        if fast_decode:
+        if tc_decode:
+            K.gqa_decode_tc(q, kcache, vcache, meta, scale, out=out, group="decode", form=form)
+        elif fast_decode:
             K._paged_attention_decode(q, kcache, vcache, meta, scale, window, 0.0, None, out=out, group="decode", bias=bias, gate=gate, form=form)
         else:
             attention_general(q, kcache, vcache, meta, scale, out, "decode", **kw)
