@@ -12,7 +12,7 @@
 //             it and does not wait for the P V of that block;
 //   warp 1    MMA: S[128 x 64] = Q K^T into one of two TMEM buffers (issued two blocks ahead), O[128 x DV] += P V with
 //             V^T read from the V stage as an MN-major B operand and P from shared memory;
-//   warps 2-5 softmax: thread r owns row r (TMEM lane r): tcgen05.ld of S, scale, causal / window mask, running maximum
+//   warps 2-5 (with attention forms also 7-10, two threads per row) softmax: thread r owns row r (TMEM lane r): tcgen05.ld of S, scale, causal / window mask, running maximum
 //             with lazy rescale of O (only when the maximum grows by more than 2^8), P written to shared memory as bf16
 //             in the un-swizzled K-major core-matrix layout, finally O / l to global memory.
 // Blocks of keys that no row of the tile can see (beyond the causal diagonal, before the window) are never loaded.
@@ -28,7 +28,6 @@ namespace {
 constexpr int PAGE = 16, KB = 64, TR = 128, CHUNK = 64;
 constexpr int NSBUF = 2;
 constexpr int P_BYTES = TR * KB * 2;              // 16 KB
-constexpr int NTHREADS = 224;
 constexpr float RESCALE_THRESHOLD = 8.0f;
 
 // SPLITP: P is handed to the tensor cores as the sum of two bf16 values (rounded value and rounding error), so that the softmax
@@ -47,9 +46,14 @@ struct FaCfg {
   static constexpr int K_STAGE = NCK * K_CHUNK_BYTES, V_STAGE = NCV * V_CHUNK_BYTES;
   static constexpr int STAGES = (DK + DV > 384) ? 2 : 3;
   static constexpr int NPBUF = (SPLITP && DK + DV > 256) ? 1 : 2;
+  // threads that share a query row, each with half of its scores (MAPS > 0, where shared memory has room for what they exchange): the row's
+  // softmax is the longest chain of the kernel, and one warp per scheduler cannot hide its own latencies
+  static constexpr int HW = (MAPS > 0 && NM * DK <= 128 && DV <= 128) ? 2 : 1;
+  static constexpr int NTHREADS = 96 + 128 * HW;
+  static constexpr int XCH_BYTES = HW == 2 ? 2 * 2 * TR * 4 : 0;
   static constexpr int BIAS_BYTES = BIAS ? 4 * 96 * 4 : 0;
   static constexpr int P_STAGE = SPLITP ? 2 * P_BYTES : P_BYTES;
-  static constexpr int SMEM = Q_BYTES + STAGES * (K_STAGE + V_STAGE) + NPBUF * P_STAGE + BIAS_BYTES + 1024 + 256;
+  static constexpr int SMEM = Q_BYTES + STAGES * (K_STAGE + V_STAGE) + NPBUF * P_STAGE + BIAS_BYTES + XCH_BYTES + 1024 + 256;
   static constexpr int TMEM_COLS = 128 + NM * DV <= 256 ? 256 : 512;     // S: 2 x 64 columns at 0..127, O: DV columns per map at 128..
   static_assert(128 + NM * DV <= 512 && !(BIAS && MAPS), "accumulator columns");
   static_assert(DK % CHUNK == 0 && DV % CHUNK == 0 && DV <= 256 && DK <= 256, "head dims: multiples of 64 up to 256");
@@ -78,11 +82,11 @@ __device__ __forceinline__ uint64_t fa_desc_mnmajor_sw128(uint32_t addr, uint32_
 }
 
 template <int DK, int DV, bool SPLITP, bool BIAS, int MAPS>
-__global__ void __launch_bounds__(NTHREADS, 1)
+__global__ void __launch_bounds__((FaCfg<DK, DV, SPLITP, BIAS, MAPS>::NTHREADS), 1)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                   const __grid_constant__ CUtensorMap tm_v, const FaParams p) {
   using C = FaCfg<DK, DV, SPLITP, BIAS, MAPS>;
-  constexpr int NM = C::NM;
+  constexpr int NM = C::NM, HW = C::HW;
   constexpr int STAGES = C::STAGES, NPBUF = C::NPBUF;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~uintptr_t(1023));
@@ -90,7 +94,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
   uint8_t* sK = sQ + C::Q_BYTES;
   uint8_t* sV = sK + STAGES * C::K_STAGE;
   uint8_t* sP = sV + STAGES * C::V_STAGE;
-  uint64_t* bars = (uint64_t*)(sP + NPBUF * C::P_STAGE + C::BIAS_BYTES);
+  uint64_t* bars = (uint64_t*)(sP + NPBUF * C::P_STAGE + C::BIAS_BYTES + C::XCH_BYTES);
   uint64_t* q_full = bars;                 // 1
   uint64_t* k_full = q_full + 1;           // [STAGES]
   uint64_t* k_empty = k_full + STAGES;
@@ -104,7 +108,8 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
   volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int nb = blockIdx.x, head = blockIdx.y;
+  // all heads of the last tiles of the batch first: they see the most keys, and short tiles are left to fill the end of the launch
+  const int nb = gridDim.y - 1 - blockIdx.y, head = blockIdx.x;
   const int kvh = head / (p.Hq / p.Hkv);
   const int seq = p.blk_seq[nb], tok0 = p.blk_tok0[nb];          // tok0: index into the flattened token axis
   const int seq_tok0 = p.q_start[seq], seq_tok1 = p.q_start[seq + 1];
@@ -121,8 +126,8 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
     for (int s = 0; s < STAGES; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
-    for (int b = 0; b < NSBUF; ++b) { mbar_init(&s_full[b], 1); mbar_init(&s_empty[b], 4); }
-    for (int b = 0; b < NPBUF; ++b) { mbar_init(&p_full[b], 4); mbar_init(&pv_done[b], 1); }
+    for (int b = 0; b < NSBUF; ++b) { mbar_init(&s_full[b], 1); mbar_init(&s_empty[b], 4 * HW); }
+    for (int b = 0; b < NPBUF; ++b) { mbar_init(&p_full[b], 4 * HW); mbar_init(&pv_done[b], 1); }
     *abort_flag = 0;
     fence_barrier_init();
     tma_prefetch_desc(&tm_q);
@@ -238,9 +243,27 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       }
     }
   } else if (nblk > 0) {
-    // ------------------------------------------------------------------ softmax warps: thread = query row
+    // ------------------------------------------------------------------ softmax warps (2-5, and 7-10 when two threads share a row): thread = query row, or half of its scores
     const int q4 = warp & 3;                         // the TMEM lane group this warp may access
     const int r = q4 * 32 + lane;
+    constexpr int KC = KB / HW;                      // scores of a block that a thread holds
+    const int half = HW == 2 && warp > 6 ? 1 : 0, cb = half * KC;
+    float* const xch = (float*)(sP + NPBUF * C::P_STAGE + C::BIAS_BYTES);       // [2][2][TR]
+    // A wait that ran out must be seen by the whole warp, and a partner warp that stands at the pair's barrier must be let go: it finds
+    // the abort flag raised and leaves as well.
+    auto wait = [&](uint64_t* bar, uint32_t parity) -> bool {
+      const bool ok = mbar_wait(bar, parity, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA);
+      if constexpr (HW == 2) {
+        if (__all_sync(0xffffffffu, ok)) return true;
+        asm volatile("bar.arrive %0, 64;" ::"r"(1 + q4) : "memory");
+        return false;
+      }
+      return ok;
+    };
+    auto meet = [&]() -> bool {                      // the two warps of the pair
+      asm volatile("bar.sync %0, 64;" ::"r"(1 + q4) : "memory");
+      return !__any_sync(0xffffffffu, *abort_flag != 0);
+    };
     const bool row_ok = r < nrows;
     const int qpos = pos_first + r;
     int lo_key = p.window > 0 ? qpos - p.window + 1 : 0;
@@ -272,11 +295,11 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
         }
         __syncwarp();
       }
-      if (!mbar_wait(&s_full[sb], (i / NSBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+      if (!wait(&s_full[sb], (i / NSBUF) & 1)) goto done;
       tc_fence_after();
-      uint32_t sr[KB];
-      tmem_ld_32x32b_x32(tmem_S + lane_off + sb * KB, sr);
-      tmem_ld_32x32b_x32(tmem_S + lane_off + sb * KB + 32, sr + 32);
+      uint32_t sr[KC];
+      tmem_ld_32x32b_x32(tmem_S + lane_off + sb * KB + cb, sr);
+      if constexpr (HW == 1) tmem_ld_32x32b_x32(tmem_S + lane_off + sb * KB + 32, sr + 32);
       tmem_ld_wait();
       tc_fence_before();
       __syncwarp();
@@ -289,12 +312,12 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       float mx;
       if constexpr (MAPS > 0) {
         if (p.f.cap > 0.f) {
-          float v[KB];
+          float v[KC];
 #pragma unroll
-          for (int j = 0; j < KB; ++j) v[j] = __uint_as_float(sr[j]);
-          cap_scores<KB>(v, sl2, p.f.cap);
+          for (int j = 0; j < KC; ++j) v[j] = __uint_as_float(sr[j]);
+          cap_scores<KC>(v, sl2, p.f.cap);
 #pragma unroll
-          for (int j = 0; j < KB; ++j) sr[j] = __float_as_uint(v[j]);
+          for (int j = 0; j < KC; ++j) sr[j] = __float_as_uint(v[j]);
         }
       }
       const float sc = MAPS > 0 && p.f.cap > 0.f ? 1.0f : sl2;               // factor on what `sr` now holds
@@ -309,29 +332,35 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       } else if (full_blk) {
         mx = __uint_as_float(sr[0]);
 #pragma unroll
-        for (int j = 1; j < KB; ++j) mx = fmaxf(mx, __uint_as_float(sr[j]));
+        for (int j = 1; j < KC; ++j) mx = fmaxf(mx, __uint_as_float(sr[j]));
         mx *= sc;
       } else {
         mx = -INFINITY;
 #pragma unroll
-        for (int j = 0; j < KB; ++j) {
-          const int kj = key0 + j;
+        for (int j = 0; j < KC; ++j) {
+          const int kj = key0 + cb + j;
           const bool ok = row_ok && kj <= qpos && kj >= lo_key;
           const float v = ok ? __uint_as_float(sr[j]) * sc : -INFINITY;
           sr[j] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
       }
+      if constexpr (HW == 2) {
+        float* x = xch + (i & 1) * 2 * TR;
+        x[half * TR + r] = mx;
+        if (!meet()) goto done;
+        mx = fmaxf(mx, x[(half ^ 1) * TR + r]);
+      }
       const bool need = mx > m_ref + RESCALE_THRESHOLD;
       const bool first = (m_ref == -INFINITY);
       float corr = 1.f;
       if (need) { corr = first ? 0.f : exp2f(m_ref - mx); m_ref = mx; }
-      uint32_t pw[KB / 2], pl[SPLITP ? KB / 2 : 1];
+      uint32_t pw[KC / 2], pl[SPLITP ? KC / 2 : 1];
       float psum = 0.f;
       if (full_blk && !BIAS) {
         const float nm = -m_ref;
 #pragma unroll
-        for (int j = 0; j < KB / 2; ++j) {
+        for (int j = 0; j < KC / 2; ++j) {
           const float a = exp2f(fmaf(__uint_as_float(sr[2 * j]), sc, nm));
           const float b = exp2f(fmaf(__uint_as_float(sr[2 * j + 1]), sc, nm));
           __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
@@ -346,7 +375,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       } else {
         const float nm = m_ref == -INFINITY ? 0.f : -m_ref;        // nothing visible yet: every score is minus infinity, every weight 0
 #pragma unroll
-        for (int j = 0; j < KB / 2; ++j) {
+        for (int j = 0; j < KC / 2; ++j) {
           const float a = exp2f(__uint_as_float(sr[2 * j]) + nm);
           const float b = exp2f(__uint_as_float(sr[2 * j + 1]) + nm);
           __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
@@ -364,10 +393,10 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       l = l * corr + psum;
       if (__any_sync(0xffffffffu, need && !first) && i > i0) {
         // O may only be touched once the previous P V has completed
-        if (!mbar_wait(&pv_done[(i - 1) % NPBUF], ((i - 1) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+        if (!wait(&pv_done[(i - 1) % NPBUF], ((i - 1) / NPBUF) & 1)) goto done;
         tc_fence_after();
 #pragma unroll 1
-        for (int c0 = 0; c0 < DV; c0 += 32) {
+        for (int c0 = half * (DV / HW); c0 < (half + 1) * (DV / HW); c0 += 32) {
           uint32_t o[32];
           tmem_ld_32x32b_x32(om + lane_off + c0, o);
           tmem_ld_wait();
@@ -380,16 +409,16 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       }
       if (i >= NPBUF) {
         // this P buffer was last read by the P V of block i - NPBUF
-        if (!mbar_wait(&pv_done[pb], ((i - NPBUF) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+        if (!wait(&pv_done[pb], ((i - NPBUF) / NPBUF) & 1)) goto done;
       }
       // P (bf16) -> shared memory: chunk c holds keys 8c..8c+7 of every row, 16 bytes per row
 #pragma unroll
-      for (int c = 0; c < KB / 8; ++c)
-        *(uint4*)(sP + pb * C::P_STAGE + c * (TR * 16) + r * 16) = make_uint4(pw[4 * c], pw[4 * c + 1], pw[4 * c + 2], pw[4 * c + 3]);
+      for (int c = 0; c < KC / 8; ++c)
+        *(uint4*)(sP + pb * C::P_STAGE + (cb / 8 + c) * (TR * 16) + r * 16) = make_uint4(pw[4 * c], pw[4 * c + 1], pw[4 * c + 2], pw[4 * c + 3]);
       if constexpr (SPLITP) {
 #pragma unroll
-        for (int c = 0; c < KB / 8; ++c)
-          *(uint4*)(sP + pb * C::P_STAGE + P_BYTES + c * (TR * 16) + r * 16) = make_uint4(pl[4 * c], pl[4 * c + 1], pl[4 * c + 2], pl[4 * c + 3]);
+        for (int c = 0; c < KC / 8; ++c)
+          *(uint4*)(sP + pb * C::P_STAGE + P_BYTES + (cb / 8 + c) * (TR * 16) + r * 16) = make_uint4(pl[4 * c], pl[4 * c + 1], pl[4 * c + 2], pl[4 * c + 3]);
       }
       fence_proxy_async();       // make the generic-proxy writes of P visible to the tensor core
       tc_fence_before();
@@ -397,8 +426,18 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       if (lane == 0) mbar_arrive(&p_full[pb]);
     }
     // ------------------------------------------------------------------ write out
-    if (!mbar_wait(&pv_done[(ntot - 1) % NPBUF], ((ntot - 1) / NPBUF) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
+    if (!wait(&pv_done[(ntot - 1) % NPBUF], ((ntot - 1) / NPBUF) & 1)) goto done;
     tc_fence_after();
+    if constexpr (HW == 2) {
+      // the other half's sums (buffers of the block loop that nobody reads any more after the first meeting)
+      if (!meet()) goto done;
+      xch[half * TR + r] = l;
+      xch[(2 + half) * TR + r] = l_first;
+      if (!meet()) goto done;
+      l += xch[(half ^ 1) * TR + r];
+      l_first += xch[(2 + (half ^ 1)) * TR + r];
+    }
+    const int o_lo = half * (DV / HW), o_hi = o_lo + DV / HW;      // value columns of this thread
     if constexpr (MAPS == 1) {
       if (p.f.sink) l += exp2f(fmaf(p.f.sink[head], 1.4426950408889634f, -m_ref));
     }
@@ -407,7 +446,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       // o = a0 - mix * a1 as w0 * O0 + w1 * O1, then the norm over the row's DV values
       float w0 = l_first > 0.f ? 1.f / l_first : 0.f, w1 = -p.f.mix * inv_l, ss = 0.f;
 #pragma unroll 1
-      for (int c0 = 0; c0 < DV; c0 += 32) {
+      for (int c0 = o_lo; c0 < o_hi; c0 += 32) {
         uint32_t a[32], b[32];
         tmem_ld_32x32b_x32(tmem_O + lane_off + c0, a);
         tmem_ld_32x32b_x32(tmem_O + lane_off + DV + c0, b);
@@ -418,11 +457,17 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
           ss = fmaf(v, v, ss);
         }
       }
+      if constexpr (HW == 2) {
+        if (!meet()) goto done;
+        xch[half * TR + r] = ss;
+        if (!meet()) goto done;
+        ss += xch[(half ^ 1) * TR + r];
+      }
       const float c = p.f.post * rsqrtf(ss / DV + p.f.eps);
       w0 *= c;
       w1 *= c;
 #pragma unroll 1
-      for (int c0 = 0; c0 < DV; c0 += 32) {
+      for (int c0 = o_lo; c0 < o_hi; c0 += 32) {
         uint32_t a[32], b[32];
         tmem_ld_32x32b_x32(tmem_O + lane_off + c0, a);
         tmem_ld_32x32b_x32(tmem_O + lane_off + DV + c0, b);
@@ -443,7 +488,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       }
     } else
 #pragma unroll 1
-    for (int c0 = 0; c0 < DV; c0 += 32) {
+    for (int c0 = o_lo; c0 < o_hi; c0 += 32) {
       uint32_t o[32];
       tmem_ld_32x32b_x32(tmem_O + lane_off + c0, o);
       tmem_ld_wait();
@@ -511,7 +556,7 @@ int launch_fa(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& t
   static MarySmemSlots smem_set = {};
   constexpr int SMEM = FaCfg<DK, DV, SPLITP, BIAS, MAPS>::SMEM;
   if (int rc = mary_ensure_dyn_smem((const void*)fa_prefill_kernel<DK, DV, SPLITP, BIAS, MAPS>, SMEM, &smem_set)) return rc;
-  fa_prefill_kernel<DK, DV, SPLITP, BIAS, MAPS><<<dim3(NB, p.Hq), NTHREADS, SMEM, s>>>(tq, tk, tv, p);
+  fa_prefill_kernel<DK, DV, SPLITP, BIAS, MAPS><<<dim3(p.Hq, NB), FaCfg<DK, DV, SPLITP, BIAS, MAPS>::NTHREADS, SMEM, s>>>(tq, tk, tv, p);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }
@@ -543,6 +588,7 @@ MARY_API int mary_attention_prefill(const void* q, const void* kcache, const voi
                                     int64_t v_tok_stride, int64_t v_page_stride, int window, float scale, int page_size,
                                     int64_t out_ld, int split_p, const float* bias, const void* gate, int64_t gate_ld, const MaryAttnForm* form, cudaStream_t s) {
   if (NB <= 0) return MARY_OK;
+  if (NB > 65535) return MARY_ERR_BAD_ARG;
   const int maps = form && form->maps == 2 ? 2 : 1;
   if (form && (form->maps > 2 || !split_p || bias || (maps == 2 && (gate || form->sink)))) return MARY_ERR_BAD_ARG;
   if (!(maps == 2 ? mary_attention_prefill_maps_supported(DK, DV) : mary_attention_prefill_supported(DK, DV)) || Hkv < 1 || Hq % Hkv || (page_size != PAGE && page_size != KB)) return MARY_ERR_BAD_ARG;

@@ -83,6 +83,26 @@ def _state_space_engine(dev):
     return out
 
 
+def _routed_engine(dev):
+    """A Nipurax decoder (capped attention with sinks, differential attention, routed experts, a loop over two layers) generating through the
+    scheduler, two sequences."""
+    from .models.nipurax import NipuraxConfig, NipuraxModel, init_random_
+    from .models.registry import family_of, make_engine
+    mlp = {"kind": "moe", "expert": {"ff": 256, "limit": 2.0}, "shared": {"ff": 384, "limit": 2.0},
+           "router": {"experts": 8, "identity": 2, "top": 3, "scale": 2.0}}
+    cap = {"type": "attention_2", "mlp": mlp, "mixer": dict(heads=8, kv_heads=2, dim=128, vdim=128, scale=0.09, softcap=30.0,
+                                                            q_temp={"coef": 0.2, "every": 32})}
+    dif = {"type": "attention", "mlp": mlp, "mixer": dict(heads=4, kv_heads=2, dim=64, vdim=128, scale=0.12, mask={"size": 48}, diff=0.3, rot={
+        "dims": 32, "base": 10000.0, "scaling": dict(factor=4.0, low=1.0, high=4.0, original=1024.0)})}
+    d = {"architecture": "Nipurax", "vocab": 1024, "width": 512, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "layers": [cap, dif, cap],
+         "embedding": {"bigram": {"buckets": 1021, "mul_prev": 17, "mul_cur": 3}}, "loop": {"start": 0, "stop": 2, "times": 2}}
+    m = NipuraxModel(NipuraxConfig.from_json(d), dtype=torch.bfloat16, device=dev)
+    init_random_(m, 0)
+    out = make_engine(m, family_of(d), 512, 2, dev).generate([list(range(90)), [5, 4, 3]], 4)
+    assert all(len(o) == 4 for o in out)
+    return out
+
+
 def _lora_step(m, dev):
     from .train.trainer import LoraTrainer
     tr = LoraTrainer(m, rank=8, alpha=16.0, lr=1e-3)
@@ -102,9 +122,10 @@ def run_smoke() -> None:
     m, out = _gemma_engine(dev)
     rec = _recurrent_engine(dev)
     ssm = _state_space_engine(dev)
+    moe = _routed_engine(dev)
     losses = _lora_step(m, dev)
     torch.cuda.synchronize()
     st = cuda.last_status()
     assert st == 0, f"kernel status {st}"
-    print(f"smoke ok: flagship emitted {n} tokens in 4 speculative steps; gemma {out}; tatizen {rec}; rokarax {ssm}; lora loss {losses[0]:.3f} -> {losses[1]:.3f}; "
+    print(f"smoke ok: flagship emitted {n} tokens in 4 speculative steps; gemma {out}; tatizen {rec}; rokarax {ssm}; nipurax {moe}; lora loss {losses[0]:.3f} -> {losses[1]:.3f}; "
           f"{cuda.LAUNCHES} kernel launches")
