@@ -140,6 +140,7 @@ class MoEFFN(nn.Module):
         self.e_local = E // par.ep_size
         self.e0 = par.ep_rank * self.e_local
         self.ep_layer = None                             # parallel.ep.EPLayer in all-to-all mode
+        self.routed_scale = c.routed_scaling_factor if c.router == "sigmoid" else 1.0      # softmax weights are used as they are
         self.w_router = _P(E, c.hidden_size, dtype=dtype, device=device)
         self.router_bias = nn.Parameter(torch.zeros(E, dtype=torch.float32, device=device), requires_grad=False) \
             if c.router == "sigmoid" else None
@@ -155,7 +156,7 @@ class MoEFFN(nn.Module):
         c = self.c
         logits = ops.linear_f32(x, self.w_router)
         return ops.router_topk(logits, c.num_experts_per_tok, c.router, self.router_bias, c.n_group, c.topk_group,
-                               c.routed_scaling_factor, c.norm_topk_prob)
+                               self.routed_scale, c.norm_topk_prob)
 
     FUSED_MAX_ROWS = 512      # decode-sized batches take the four-launch pipeline; larger ones the planned path with 128-row tiles
 
@@ -196,7 +197,7 @@ class MoEFFN(nn.Module):
         """``h += ffn(x)`` and the next block's normed input through the four-launch pipeline.  Returns ``(x_next | None, h)``."""
         c, par = self.c, self.par
         logits = ops.linear_f32(x, self.w_router)
-        router = dict(mode=c.router, bias=self.router_bias, n_group=c.n_group, topk_group=c.topk_group, scale=c.routed_scaling_factor,
+        router = dict(mode=c.router, bias=self.router_bias, n_group=c.n_group, topk_group=c.topk_group, scale=self.routed_scale,
                       renorm=c.norm_topk_prob)
         add = ops.linear(ops.linear_glu(x, self.shared.w_gu, c.act), self.shared.w_down) if self.shared is not None else None
         if fm.local_only and par.ep_size > 1:
