@@ -15,6 +15,7 @@ from ..runtime.kv_cache import PagedKVCache
 from ..runtime.spec_decode import SpecDecoder
 
 PAGE = 64
+PAGES = {"routed": 16}             # a decoder whose family is served with other pages
 # width, feed-forward, attention (heads, kv heads), linear heads, delta (value heads, q/k heads); head widths 128.  Rokarax: the same attention
 # heads with windows of 1024 positions, state space layers of twice the width in heads of 64 with 128 state rows, latents of 512 + 64
 SIZES = {"2k": (2048, 8192, (16, 4), 8, (16, 8)), "4k": (4096, 12288, (32, 8), 16, (32, 16))}
@@ -90,8 +91,8 @@ def make_model(kind: str, size: str, dev):
     return m
 
 
-def make_cache(m, batch: int, tokens: int, dev) -> PagedKVCache:
-    c = PagedKVCache.for_model(m, num_pages=batch * ((tokens + PAGE - 1) // PAGE), page_size=PAGE, device=dev, num_slots=batch)
+def make_cache(m, batch: int, tokens: int, dev, page: int = PAGE) -> PagedKVCache:
+    c = PagedKVCache.for_model(m, num_pages=batch * ((tokens + page - 1) // page), page_size=page, device=dev, num_slots=batch)
     for t in [*c.k, *c.v]:
         t.normal_()
     for layer in c.state:
@@ -116,8 +117,9 @@ def timed(fn, steps: int, warmup: int) -> float:
 
 def prefill_step(m, cache, batch: int, n: int, dev):
     ids = torch.randint(0, VOCAB, (batch * n,), dtype=torch.int32, device=dev)
-    table = np.arange(batch * ((n + PAGE - 1) // PAGE), dtype=np.int32).reshape(batch, -1)
-    meta = BatchMeta.build([n] * batch, [n] * batch, table, PAGE, dev, np.arange(batch, dtype=np.int32))
+    page = cache.page_size
+    table = np.arange(batch * ((n + page - 1) // page), dtype=np.int32).reshape(batch, -1)
+    meta = BatchMeta.build([n] * batch, [n] * batch, table, page, dev, np.arange(batch, dtype=np.int32))
     rows = torch.arange(batch, device=dev) * n + n - 1
 
     def run():
@@ -146,7 +148,7 @@ def run(design: str, sizes, cases, steps: int, warmup: int, trace: bool = False)
                 K.set_pdl(what == "decode")
                 tokens = n if what == "prefill" else n + max(steps, 1) + max(warmup, 3) + 64
                 tokens = (tokens + PAGE - 1) // PAGE * PAGE
-                cache = make_cache(m, batch, tokens, dev)
+                cache = make_cache(m, batch, tokens, dev, PAGES.get(kind, PAGE))
                 if trace:
                     from ..utils.trace import Tracer
                     step = prefill_step(m, cache, batch, n, dev) if what == "prefill" else None

@@ -287,7 +287,9 @@ def run_nipurax(width: int = 2048, heads: int = 16, kv_heads: int = 4, experts: 
         vc, Q = torch.randn_like(kc), torch.randn(B, heads, D, **bf)
         out = torch.empty(B, heads * D, **bf)
         nb = 2.0 * B * ctx * kv_heads * D * 2
-        add("paged_attention_decode", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1), nbytes=nb, like="routed decoder")
+        m16, k16, v16 = _meta(B, 1, ctx, 16), kc.view(-1, 16, kv_heads, D), vc.view(-1, 16, kv_heads, D)
+        add("gqa_decode_tc", case, lambda: K.gqa_decode_tc(Q, k16, v16, m16, 0.1), nbytes=nb, like="routed decoder")
+        add("paged_attention_decode", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1), nbytes=nb)
         add("  capped, sink, temperature", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1, out=out, form=cap), nbytes=nb)
         add("difference of maps (64 / 128)", case, lambda: H.attention_exact(Q, kc, vc, m, 0.1, out=out, form=dif), nbytes=nb)
         inv, g = torch.ones(D // 2, device="cuda"), torch.ones(D, **bf)
