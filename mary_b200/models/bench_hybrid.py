@@ -55,8 +55,8 @@ def nipurax_config(size: str):
     (W, _, (H, G), _, _), (E, top, F, FS) = SIZES[size], EXPERTS[size]
     moe = ExpertsSpec(E, IDENTITY, top, 2.0, GLUSpec(F, 7.0), GLUSpec(FS, 7.0))
     cap = LayerSpec(CappedSpec(H, G, 128, 128, 128 ** -0.5, 30.0, 0.1, 1024), moe)
-    dif = LayerSpec(DifferentialSpec(H, G, 64, 128, 0.125, CHUNK, 0.3, RotationSpec(64, 1e6, 8.0, 1.0, 4.0, 2048.0)), moe)
-    return NipuraxConfig(VOCAB, W, 1e-5, 0.3, PairsSpec(65521, 31, 7), LoopSpec(2, 4, 2), [cap, dif] * 3, name=f"nipurax-{size}")
+    dif = LayerSpec(DifferentialSpec(H, G, 64, 128, 0.125, CHUNK, 0.2, RotationSpec(64, 5e5, 4.0, 1.0, 8.0, 4096.0)), moe)
+    return NipuraxConfig(VOCAB, W, 1e-5, 0.25, PairsSpec(65521, 36313, 27191), LoopSpec(2, 4, 2), [cap, dif] * 3, name=f"nipurax-{size}")
 
 
 def routed_config(size: str):

@@ -233,7 +233,7 @@ def run_nipurax(width: int = 2048, heads: int = 16, kv_heads: int = 4, experts: 
     D = 128
     cap = AttentionForm(cap=30.0, sink=torch.zeros(heads, device="cuda"), temperature=(0.1, 1024))
     dif = AttentionForm(chunk=chunk, difference=(0.4, 0.7, 1e-5))
-    freq = stepped_frequencies(64, 1e6, 8.0, 1.0, 4.0, 2048.0).cuda()
+    freq = stepped_frequencies(64, 5e5, 4.0, 1.0, 8.0, 4096.0).cuda()
     gu, down = torch.randn(experts, 2 * ff, width, **bf) * 0.02, torch.randn(experts, width, ff, **bf) * 0.02
     gain, vec = torch.ones(width, **bf), torch.ones(width, **bf)
 
