@@ -29,7 +29,8 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr", "-Xptxas", "-v",
 ]
 # Files whose arithmetic also serves 32-bit models keep the exact divide, square root and exponential; all others use the fast forms.
-EXACT_MATH = {"linear_attention", "recurrent_scan", "residual32", "parallel_stream", "gemm_simt", "attention_general", "latent", "state_space", "ssd_chunk"}
+EXACT_MATH = {"linear_attention", "recurrent_scan", "residual32", "parallel_stream", "gemm_simt", "attention_general", "latent", "state_space", "ssd_chunk",
+              "hyper_streams"}
 
 
 def _stamp(paths, extra=""):

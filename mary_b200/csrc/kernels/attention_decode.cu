@@ -275,7 +275,7 @@ attn_decode_kernel(const DecParams p) {
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < R * MAPS * DV; i += blockDim.x) {
+  for (int i = threadIdx.x; i < R * MAPS * DV; i += blockDim.x) {        // whole warps: DV is a multiple of 32
     const int r = i / DV, d = i % DV;
     float mm = -INFINITY;
 #pragma unroll
@@ -290,7 +290,9 @@ attn_decode_kernel(const DecParams p) {
     }
     if (MAPS == 1 && p.nsplit == 1) {
       const int tq = row0 + r / p.G, h = kvh * p.G + r % p.G;
-      p.out[(int64_t)tq * p.out_ld + (int64_t)h * DV + d] = gated(p, acc * weight_norm(p, FORM, h, mm, ll), tq, h * DV + d);
+      float x = acc * weight_norm(p, FORM, h, mm, ll);
+      if constexpr (FORM) x = turned_back_lane(p.f, x, tq, d, DV, true);
+      p.out[(int64_t)tq * p.out_ld + (int64_t)h * DV + d] = gated(p, x, tq, h * DV + d);
     } else {
       const int64_t pi = (((int64_t)nb * p.Hkv + kvh) * p.nsplit + split) * MAXR + r;
       p.part_o[pi * DV + d] = acc;
@@ -319,7 +321,8 @@ __global__ void attn_decode_combine_kernel(const DecParams p, int D) {
       acc += p.part_o[pi * D + d] * c;
     }
     const int tq = row0 + r / p.G, h = kvh * p.G + r % p.G;
-    p.out[(int64_t)tq * p.out_ld + (int64_t)h * D + d] = gated(p, acc * weight_norm(p, true, h, mm, ll), tq, h * D + d);
+    const float x = turned_back_lane(p.f, acc * weight_norm(p, true, h, mm, ll), tq, d, D, true);      // whole warps: D is a multiple of 32
+    p.out[(int64_t)tq * p.out_ld + (int64_t)h * D + d] = gated(p, x, tq, h * D + d);
   }
 }
 
@@ -423,13 +426,13 @@ static int decode_run(const void* q, const void* kc, const void* vc, const float
   p.part_ml = scratch ? scratch + (int64_t)NB * Hkv * p.nsplit * MAXR * DV : nullptr;
   const int R = RQ * p.G;
   if (p.f.maps == 2) {
-    if (bias || gate || p.f.sink || R > 4) return MARY_ERR_BAD_ARG;
+    if (bias || gate || p.f.sink || p.f.turn || R > 4) return MARY_ERR_BAD_ARG;
     if (D == 64 && DV == 64) return R <= 2 ? launch_maps<64, 64, 2>(p, NB, s) : launch_maps<64, 64, 4>(p, NB, s);
     if (D == 64 && DV == 128) return R <= 2 ? launch_maps<64, 128, 2>(p, NB, s) : launch_maps<64, 128, 4>(p, NB, s);
     if (D == 128 && DV == 128) return R <= 2 ? launch_maps<128, 128, 2>(p, NB, s) : launch_maps<128, 128, 4>(p, NB, s);
     return MARY_ERR_BAD_ARG;
   }
-  const bool fm = form && (p.f.chunk > 0 || p.f.sink || p.f.temp_every > 0 || p.f.cap > 0.f);
+  const bool fm = form && (p.f.chunk > 0 || p.f.sink || p.f.temp_every > 0 || p.f.cap > 0.f || p.f.turn);
   if (D == 256) { if (R <= 2) return launch<256, 2>(p, NB, fm, s); if (R <= 4) return launch<256, 4>(p, NB, fm, s); return MARY_ERR_BAD_ARG; }
   if (D == 128) { if (R <= 4) return launch<128, 4>(p, NB, fm, s); if (R <= 8) return launch<128, 8>(p, NB, fm, s); return MARY_ERR_BAD_ARG; }
   if (D == 64) { if (R <= 4) return launch<64, 4>(p, NB, fm, s); if (R <= 8) return launch<64, 8>(p, NB, fm, s); return MARY_ERR_BAD_ARG; }

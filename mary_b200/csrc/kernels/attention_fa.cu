@@ -511,6 +511,18 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
             }
           }
         }
+        if constexpr (MAPS == 1) {
+          if (p.f.turn) {
+            const float4* cs = (const float4*)(p.f.turn + ((int64_t)(tok0 + r) * DV + c0) / 2);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+              const float4 c = cs[j];
+              float* x = (float*)o + 4 * j;
+              const float2 a = turned_back(make_float2(c.x, c.y), x[0], x[1]), b = turned_back(make_float2(c.z, c.w), x[2], x[3]);
+              x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y;
+            }
+          }
+        }
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           __nv_bfloat162 h = __floats2bfloat162_rn(__uint_as_float(o[2 * j]) * inv_l, __uint_as_float(o[2 * j + 1]) * inv_l);
@@ -590,7 +602,7 @@ MARY_API int mary_attention_prefill(const void* q, const void* kcache, const voi
   if (NB <= 0) return MARY_OK;
   if (NB > 65535) return MARY_ERR_BAD_ARG;
   const int maps = form && form->maps == 2 ? 2 : 1;
-  if (form && (form->maps > 2 || !split_p || bias || (maps == 2 && (gate || form->sink)))) return MARY_ERR_BAD_ARG;
+  if (form && (form->maps > 2 || !split_p || bias || (maps == 2 && (gate || form->sink || form->turn)) || (form->turn && (gate || ((uintptr_t)form->turn & 15))))) return MARY_ERR_BAD_ARG;
   if (!(maps == 2 ? mary_attention_prefill_maps_supported(DK, DV) : mary_attention_prefill_supported(DK, DV)) || Hkv < 1 || Hq % Hkv || (page_size != PAGE && page_size != KB)) return MARY_ERR_BAD_ARG;
   if ((k_tok_stride * 2) % 16 || (k_page_stride * 2) % 16 || (v_tok_stride * 2) % 16 || (v_page_stride * 2) % 16) return MARY_ERR_BAD_ARG;
   CUtensorMap tq, tk, tv;
@@ -614,7 +626,7 @@ MARY_API int mary_attention_prefill(const void* q, const void* kcache, const voi
     if (DK == 64) return launch_fa<64, 128, true, false, 2>(tq, tk, tv, p, NB, s);
     return launch_fa<128, 128, true, false, 2>(tq, tk, tv, p, NB, s);
   }
-  if (form && (p.f.chunk > 0 || p.f.sink || p.f.temp_every > 0 || p.f.cap > 0.f)) {
+  if (form && (p.f.chunk > 0 || p.f.sink || p.f.temp_every > 0 || p.f.cap > 0.f || p.f.turn)) {
     if (DK == 64) return launch_fa<64, 64, true, false, 1>(tq, tk, tv, p, NB, s);
     if (DK == 128) return launch_fa<128, 128, true, false, 1>(tq, tk, tv, p, NB, s);
     if (DK == 192) return MARY_ERR_BAD_ARG;

@@ -1,11 +1,12 @@
 // What a call of the attention kernels may ask for beyond causal softmax attention with a window: chunks, capped scores, a sink, a query
-// temperature by position, and the difference of two softmax maps over the same values.
+// temperature by position, the difference of two softmax maps over the same values, and a rotation of the result by the query's position.
 #pragma once
 #include "common.cuh"
 
 // Passed by host pointer to the launchers (null: none of it).  Two maps: the query and key rows of a head are [map 0 | map 1], both maps read
 // the head's values, and the result is rms(a0 - mix * a1) * post over the value width.
 struct MaryAttnForm {
+  const float2* turn;    // [T][DV / 2] (cosine, sine): pair (2 m, 2 m + 1) of every head's result at token row t is turned back by that angle; or null
   const float* sink;     // [Hq]: a learned score per head that enters the sum of weights only; or null
   int64_t q_ld;          // elements between the query rows of two tokens (0: contiguous)
   int chunk;             // > 0: a query sees the keys of its own chunk of this many positions, counted from position 0
@@ -22,6 +23,17 @@ __device__ __forceinline__ float query_temperature(const MaryAttnForm& f, int po
   return f.temp_every > 0 ? fmaf(f.temp_coef, logf((float)((pos + 1) / f.temp_every + 1)), 1.0f) : 1.0f;
 }
 __device__ __forceinline__ int first_key(const MaryAttnForm& f, int pos) { return f.chunk > 0 ? pos / f.chunk * f.chunk : 0; }
+
+// The result's pair (a, b) turned back by the angle of cs.
+__device__ __forceinline__ float2 turned_back(float2 cs, float a, float b) { return make_float2(fmaf(a, cs.x, b * cs.y), fmaf(b, cs.x, -a * cs.y)); }
+// The same where neighbouring lanes hold neighbouring columns: every lane of the warp calls it with its value of token row t, column d of a head.
+__device__ __forceinline__ float turned_back_lane(const MaryAttnForm& f, float v, int64_t t, int d, int DV, bool in) {
+  if (!f.turn) return v;
+  const float other = __shfl_xor_sync(0xffffffffu, v, 1);
+  if (!in) return v;
+  const float2 cs = f.turn[t * (DV / 2) + d / 2];
+  return fmaf(v, cs.x, (d & 1 ? -other : other) * cs.y);
+}
 
 // tanh in 32 bits whatever the compiler's math mode (its fast tanh has 11 bits): the power series for small arguments, elsewhere
 // 1 - 2 / (exp(2 |x|) + 1), whose result is at least 0.46 there, so the subtraction loses nothing.

@@ -151,8 +151,11 @@ __global__ void __launch_bounds__(WARPS * 32) attn_general_kernel(const GenParam
       const int h = query_head(p, kvh, g0 + rr % gc), col = h * p.DV;
       const float inv = finish_scale(p, h, m[r], l[r]);
 #pragma unroll
-      for (int v = 0; v < NV; ++v)
-        if (lane + 32 * v < p.DV) store_out<T>(p, o[r][v] * inv, row, col + lane + 32 * v);
+      for (int v = 0; v < NV; ++v) {
+        const bool in = lane + 32 * v < p.DV;
+        const float x = turned_back_lane(p.f, o[r][v] * inv, row, lane + 32 * v, p.DV, in);
+        if (in) store_out<T>(p, x, row, col + lane + 32 * v);
+      }
     } else {
       const int64_t pi = (((int64_t)nb * gridDim.y + blockIdx.y) * p.nsplit + split) * ROWS + rr;
 #pragma unroll
@@ -170,7 +173,9 @@ __global__ void attn_general_combine_kernel(const GenParams p) {
   const int gc = min(p.GC, p.G - g0);
   const int seq = p.blk_seq[nb], row0 = p.blk_q0[nb];
   const int R = min(p.RQ, p.q_start[seq + 1] - row0) * gc;
-  for (int i = threadIdx.x; i < R * p.DV; i += blockDim.x) {
+  for (int i0 = 0; i0 < R * p.DV; i0 += blockDim.x) {              // whole warps go through it together
+    const bool in = i0 + (int)threadIdx.x < R * p.DV;
+    const int i = in ? i0 + threadIdx.x : 0;
     const int r = i / p.DV, d = i % p.DV;
     const int64_t base = (((int64_t)nb * gridDim.y + blockIdx.y) * p.nsplit) * ROWS + r;
     float mm = -INFINITY;
@@ -184,7 +189,8 @@ __global__ void attn_general_combine_kernel(const GenParams p) {
       acc += p.part_o[pi * p.DV + d] * c;
     }
     const int h = query_head(p, kvh, g0 + r % gc);
-    store_out<T>(p, acc * finish_scale(p, h, mm, ll), row0 + r / gc, h * p.DV + d);
+    const float x = turned_back_lane(p.f, acc * finish_scale(p, h, mm, ll), row0 + r / gc, d, p.DV, in);
+    if (in) store_out<T>(p, x, row0 + r / gc, h * p.DV + d);
   }
 }
 
@@ -253,7 +259,7 @@ MARY_API int mary_attention_general(const void* q, const void* kc, const void* v
   p.f = form ? *form : MaryAttnForm{};
   if (p.f.maps < 1) p.f.maps = 1;
   if (p.f.q_ld <= 0) p.f.q_ld = (int64_t)Hq * DK;
-  if (p.f.maps > 2 || Hkv % p.f.maps || (p.f.maps == 2 && (gate || bias || p.f.sink)) || (bias && p.f.chunk)) return MARY_ERR_BAD_ARG;
+  if (p.f.maps > 2 || Hkv % p.f.maps || (p.f.maps == 2 && (gate || bias || p.f.sink || p.f.turn)) || (p.f.turn && (DV & 1)) || (bias && p.f.chunk)) return MARY_ERR_BAD_ARG;
   p.GC = p.G < ROWS ? p.G : ROWS;
   p.gchunks = (p.G + p.GC - 1) / p.GC;
   if (RQ < 1 || RQ * p.GC > ROWS || (nsplit > 1 && !scratch)) return MARY_ERR_BAD_ARG;

@@ -406,6 +406,18 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           __nv_bfloat16* dst = p.out + (int64_t)tq * p.out_ld + head * D + c0;
           uint4 w[4];
           uint32_t* wp = (uint32_t*)w;
+          if constexpr (MAPS == 1) {
+            if (p.f.turn) {
+              const float4* cs = (const float4*)(p.f.turn + ((int64_t)tq * D + c0) / 2);
+#pragma unroll
+              for (int j = 0; j < 8; ++j) {
+                const float4 c = cs[j];
+                float* x = (float*)o + 4 * j;
+                const float2 a = turned_back(make_float2(c.x, c.y), x[0], x[1]), b = turned_back(make_float2(c.z, c.w), x[2], x[3]);
+                x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y;
+              }
+            }
+          }
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             __nv_bfloat162 h = __floats2bfloat162_rn(__uint_as_float(o[2 * j]) * inv_l, __uint_as_float(o[2 * j + 1]) * inv_l);
@@ -505,6 +517,10 @@ __global__ void __launch_bounds__(128) gqa_tc_combine_form_kernel(const GqaParam
     for (int e = 0; e < E; ++e) y[e] = fmaf(acc[e], norm, y[e]);
   }
   float c = 1.f;
+  if constexpr (MAPS == 1) {
+#pragma unroll
+    for (int e = 0; e < E; ++e) y[e] = turned_back_lane(p.f, y[e], tq, threadIdx.x + 128 * e, D, true);
+  }
   if constexpr (MAPS == 2) {
     float ss = 0.f;
 #pragma unroll
@@ -569,7 +585,7 @@ MARY_API int mary_gqa_decode_tc(const void* q, const void* kc, const void* vc, v
   if (maps ? !mary_gqa_tc_form_supported(D, page_size, G, RQ, maps) || softcap > 0.f : !mary_gqa_tc_supported(D, page_size, G, RQ)) return MARY_ERR_BAD_ARG;
   const int64_t q_ld = form && form->q_ld > 0 ? form->q_ld : (int64_t)Hq * D;
   if (out_ld <= 0) out_ld = (int64_t)Hq * D;
-  if (q_ld % 8 || out_ld % 8 || ((uintptr_t)out & 15) || (maps == 2 && form->sink)) return MARY_ERR_BAD_ARG;
+  if (q_ld % 8 || out_ld % 8 || ((uintptr_t)out & 15) || (maps == 2 && (form->sink || form->turn)) || (form && ((uintptr_t)form->turn & 15))) return MARY_ERR_BAD_ARG;
   if (nsplit < 1) nsplit = 1;
   if ((nsplit > 1 || maps == 2) && !scratch) return MARY_ERR_BAD_ARG;
   PFN_encode enc = (PFN_encode)mary_encode_fn();

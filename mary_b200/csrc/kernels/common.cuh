@@ -243,6 +243,8 @@ __device__ __forceinline__ float gelu_tanh_f(float x) {
   return 0.5f * x * (1.0f + tanhf(k0 * (x + k1 * x * x * x)));
 }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
+// The tanh form of GELU as x times the logistic function of twice its argument: nothing cancels, whatever the compiler's math mode.
+__device__ __forceinline__ float gelu_sigmoid_f(float x) { return x / (1.0f + __expf(-1.5957691216057308f * (x + 0.044715f * x * x * x))); }
 __device__ __forceinline__ float situ_f(float g, float u) {
   const float beta = 4.0f, lb = 25.0f;
   return beta * tanhf(g / beta) * (1.0f / (1.0f + __expf(-g))) * (lb * tanhf(u / lb));

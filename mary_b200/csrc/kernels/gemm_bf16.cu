@@ -38,6 +38,7 @@ struct GemmParams {
   int glu_offset;            // rows between the gate tile and the up tile of the weight operand (GLU only)
   int act;
   float glu_limit;           // of the clamped GLU
+  int un_act, un_cols;       // > 0: an activation (1 tanh-form GELU, 2 SiLU) of the first un_cols output features, on the f32 sums
   int epi;
   int swap;                  // 1: row operand = weights, D[i][j] -> out[j * ldo + i]
   int64_t ldo;
@@ -171,7 +172,7 @@ struct Cfg {
 // 128-row tiles, two accumulators of BN columns); without swap they are the column operand and the two
 // BN-row tiles are... handled by launching the swapped roles only: GLU without swap is expressed by the host
 // as two B tiles, see launch code.  To keep one device code path, GLU always means "two row-operand tiles".
-template <int BN, bool GLU, int LEAN_MODE>          // 0: every path; 1: decode-shaped launches only; 2: the same with the short pipeline
+template <int BN, bool GLU, int LEAN_MODE>          // 0: every path; 1: decode-shaped launches only; 2: the same with the short pipeline; 3: 1 with an activation
 __global__ void __launch_bounds__(NTHREADS, 1)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap tm_r, const __grid_constant__ CUtensorMap tm_c, const GemmParams p) {
   constexpr bool LEAN = LEAN_MODE != 0;
@@ -316,6 +317,17 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tm_r, const __grid_constant
       const bool sk = sk_epi && w.nseg > 1;             // a tile computed by one CTA alone is stored directly
       const int tile = w.tile;
       float* slot = sk ? p.ws + (int64_t)tile * (BM * BN) : nullptr;      // the tile's f32 accumulator (zero between calls)
+      // the activation of finished sums, columns tc * BN + c0 .. of this thread's row
+      auto activate = [&](int c0, float* v) {
+        if constexpr (!GLU && (LEAN_MODE == 0 || LEAN_MODE == 3)) {
+          if (p.un_act == 0) return;
+          const int left = swap ? (i < p.un_cols ? 32 : 0) : p.un_cols - (tc * BN + c0);
+          if (left <= 0) return;
+#pragma unroll
+          for (int j = 0; j < 32; ++j)
+            if (j < left) v[j] = p.un_act == 1 ? gelu_sigmoid_f(v[j]) : silu_f(v[j]);
+        }
+      };
       // stores 32 finished values of this thread's row (columns tc * BN + c0 ..) in the requested form
       auto emit = [&](int c0, const float* v, int epi) {
         const int j0 = tc * BN + c0;
@@ -390,6 +402,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tm_r, const __grid_constant
 #pragma unroll
           for (int j = 0; j < 32; ++j) atomicAdd(slot + (c0 + j) * BM + q * 32 + lane, v[j]);
         } else {
+          activate(c0, v);
           emit(c0, v, final_epi);
         }
       }
@@ -412,6 +425,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tm_r, const __grid_constant
             for (int j = 0; j < 32; ++j) v[j] = __ldcg(a + j * BM);
 #pragma unroll
             for (int j = 0; j < 32; ++j) __stcg(a + j * BM, 0.f);          // the accumulator is left zero for the next call
+            activate(c0, v);
             emit(c0, v, final_epi);
           }
           if (threadIdx.x == 64) p.counters[tile] = 0;
@@ -475,7 +489,8 @@ static int gemm_impl(const void* X, const void* W, void* out, int M, int N, int 
                      int64_t bsx, int64_t bsw, int64_t bso, const float* bias, float alpha, int glu, int epi, int split_k, int swap,
                      const uint64_t* rs_bufs, int rs_world, int rs_src, int rs_rpr, cudaStream_t stream, float* ws = nullptr,
                      int64_t ws_floats = 0, int* counters = nullptr, int n_counters = 0, bool stream_k = false,
-                     const int* g_tiles = nullptr, const int* g_meta = nullptr, int g_experts = 0, int g_nt = 0, float glu_limit = 0.f);
+                     const int* g_tiles = nullptr, const int* g_meta = nullptr, int g_experts = 0, int g_nt = 0, float glu_limit = 0.f,
+                     int un_act = 0, int un_cols = 0);
 
 // Tells the GEMM launchers called next on THIS thread that their W operand holds constant model weights (1) or may have been
 // written by an earlier kernel of the stream (0, the default).  Only read when programmatic dependent launch is enabled.
@@ -503,7 +518,8 @@ static int gemm_impl(const void* X, const void* W, void* out, int M, int N, int 
                      int64_t bsx, int64_t bsw, int64_t bso, const float* bias, float alpha, int glu, int epi, int split_k, int swap,
                      const uint64_t* rs_bufs, int rs_world, int rs_src, int rs_rpr, cudaStream_t stream, float* ws, int64_t ws_floats,
                      int* counters, int n_counters, bool stream_k, const int* g_tiles, const int* g_meta, int g_experts, int g_nt,
-                     float glu_limit) {
+                     float glu_limit, int un_act, int un_cols) {
+  if (un_act < 0 || un_act > 2 || (un_act && (glu || bias || (epi != EPI_STORE_BF16 && epi != EPI_SK_BF16)))) return MARY_ERR_BAD_ARG;
   if (M <= 0 || N <= 0 || K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || batch < 1) return MARY_ERR_BAD_ARG;
   if (split_k < 1) split_k = 1;
   const bool sk_epi = epi == EPI_SK_BF16 || epi == EPI_SK_F32;
@@ -522,6 +538,8 @@ static int gemm_impl(const void* X, const void* W, void* out, int M, int N, int 
   p.glu_offset = N;
   p.act = glu ? glu - 1 : 0;
   p.glu_limit = glu_limit;
+  p.un_act = un_act;
+  p.un_cols = un_cols;
   p.epi = epi;
   p.swap = use_swap ? 1 : 0;
   p.ldo = ldo;
@@ -615,6 +633,13 @@ static int gemm_impl(const void* X, const void* W, void* out, int M, int N, int 
         default: return launch<128, true, 1>(tr, tc, p, stream);
       }
     }
+    if (un_act) {
+      switch (bn) {
+        case 32: return launch<32, false, 3>(tr, tc, p, stream);
+        case 64: return launch<64, false, 3>(tr, tc, p, stream);
+        default: return launch<128, false, 3>(tr, tc, p, stream);
+      }
+    }
     if (g_short_pipeline) {
       switch (bn) {
         case 32: return launch<32, false, 2>(tr, tc, p, stream);
@@ -650,6 +675,14 @@ MARY_API int mary_gemm_bf16(const void* X, const void* W, void* out, int M, int 
                             cudaStream_t stream) {
   return gemm_impl(X, W, out, M, N, K, ldx, ldw, ldo, 1, 0, 0, 0, bias, alpha, glu, epi, split_k, swap, nullptr, 0, 0, 0, stream, nullptr, 0, nullptr,
                    0, false, nullptr, nullptr, 0, 0, glu_limit);
+}
+
+// out = act(X W^T) on the first un_cols output features (act: 1 tanh-form GELU, 2 SiLU), X W^T on the others; bf16.  ws null: no split of K, else
+// stream-K as mary_gemm_bf16_splitk with split_k = 0.
+MARY_API int mary_gemm_bf16_act(const void* X, const void* W, void* out, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldo, int act, int un_cols,
+                                float* ws, int64_t ws_floats, int* counters, int n_counters, cudaStream_t stream) {
+  return gemm_impl(X, W, out, M, N, K, ldx, ldw, ldo, 1, 0, 0, 0, nullptr, 1.0f, 0, ws ? EPI_SK_BF16 : EPI_STORE_BF16, 1, -1, nullptr, 0, 0, 0, stream,
+                   ws, ws_floats, counters, n_counters, ws != nullptr, nullptr, nullptr, 0, 0, 0.f, act, un_cols);
 }
 
 // Grouped (mixture-of-experts) GEMM with unquantised expert weights: out[rows_pad, N] = X[rows_pad, K] * W[expert of the row's tile]^T,

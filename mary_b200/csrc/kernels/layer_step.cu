@@ -107,17 +107,18 @@ __device__ __forceinline__ void warp_dot4(const __nv_bfloat16* __restrict__ w, i
 // mode 3: y[n] = alpha * W[n] x, y in f32   (what a post-norm consumes)
 // mode 4: y[n] = gelu_tanh(W[n] x) * (W[n + N] x)
 // mode 5: y[n] = clamped GLU of the same two with limit alpha
+// mode 6, 7: y[n] = gelu_tanh (6) or silu (7) of W[n] x for n < act_rows, W[n] x for the others
 __global__ void __launch_bounds__(LS_THREADS) step_matvec_kernel(const __nv_bfloat16* __restrict__ h, const __nv_bfloat16* __restrict__ gain,
                                                                  float eps, const __nv_bfloat16* __restrict__ w, int64_t ldw, int N, int K,
                                                                  const __nv_bfloat16* __restrict__ res, __nv_bfloat16* __restrict__ y, int mode,
-                                                                 int rpw, float alpha) {
+                                                                 int rpw, float alpha, int act_rows) {
   pdl_sync();
   extern __shared__ float xs[];
   __shared__ float red[32];
   stage_input(h, gain, eps, K, xs, red);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = LS_THREADS / 32;
   const int gw = blockIdx.x * nw + warp, tw = gridDim.x * nw;
-  if (mode == 2 || mode >= 4) {
+  if (mode == 2 || mode == 4 || mode == 5) {
     const int act = mode == 2 ? 1 : (mode == 4 ? 0 : 3);
     const int pw = rpw >= 2 ? 2 : 1;               // output rows per warp and pass (each is a gate row and an up row)
     for (int n0 = gw * pw; n0 < N; n0 += tw * pw) {
@@ -139,6 +140,7 @@ __global__ void __launch_bounds__(LS_THREADS) step_matvec_kernel(const __nv_bflo
       if (lane < cnt) {
         float v = lane == 0 ? d[0] : (lane == 1 ? d[1] : (lane == 2 ? d[2] : d[3]));
         if (mode == 3) { ((float*)y)[n0 + lane] = alpha * v; continue; }
+        if (mode >= 6 && n0 + lane < act_rows) v = mode == 6 ? gelu_sigmoid_f(v) : silu_f(v);
         if (mode == 1) v = __bfloat162float(res[n0 + lane]) + __bfloat162float(__float2bfloat16(v));
         y[n0 + lane] = __float2bfloat16(v);
       }
@@ -287,21 +289,21 @@ __global__ void __launch_bounds__(LS_THREADS) step_attention_kernel(const __nv_b
 }  // namespace
 
 // y[N] = f(W[N (or 2N), K] x) with the stage's folded neighbours (mode: 0 plain, 1 + residual, 2 SwiGLU over [gate; up] rows,
-// 3 f32 result, 4 GEGLU, 5 clamped GLU);
+// 3 f32 result, 4 GEGLU, 5 clamped GLU, 6 / 7 GELU / SiLU of the first act_rows rows);
 // gain != null: x = rms(h) * gain, else x = h.
 MARY_API int mary_step_matvec(const void* h, const void* gain, float eps, const void* w, int64_t ldw, int N, int K, const void* res, void* y,
-                              int mode, float alpha, cudaStream_t s) {
-  if (N <= 0 || K <= 0 || (K & 7) || (ldw & 7) || K > LS_MAX_H || mode < 0 || mode > 5 || (mode == 1 && !res)) return MARY_ERR_BAD_ARG;
+                              int mode, float alpha, int act_rows, cudaStream_t s) {
+  if (N <= 0 || K <= 0 || (K & 7) || (ldw & 7) || K > LS_MAX_H || mode < 0 || mode > 7 || (mode == 1 && !res)) return MARY_ERR_BAD_ARG;
   // rows per warp and pass: as many as still give every SM a CTA (a narrow output with one row per warp fills the machine,
   // a wide one keeps four rows of loads in flight per warp)
   const int sms = mary_num_sms(), nw = LS_THREADS / 32;
-  int rpw = (mode == 2 || mode >= 4) ? 2 : 4;
+  int rpw = (mode == 2 || mode == 4 || mode == 5) ? 2 : 4;
   while (rpw > 1 && (N + nw * rpw - 1) / (nw * rpw) < sms) rpw >>= 1;
   int grid = (N + nw * rpw - 1) / (nw * rpw);
   const int cap = 4 * sms;
   if (grid > cap) grid = cap;
   MARY_LAUNCH(step_matvec_kernel, grid, LS_THREADS, (size_t)K * sizeof(float), s, (const __nv_bfloat16*)h, (const __nv_bfloat16*)gain, eps,
-              (const __nv_bfloat16*)w, ldw, N, K, (const __nv_bfloat16*)res, (__nv_bfloat16*)y, mode, rpw, alpha);
+              (const __nv_bfloat16*)w, ldw, N, K, (const __nv_bfloat16*)res, (__nv_bfloat16*)y, mode, rpw, alpha, act_rows);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }

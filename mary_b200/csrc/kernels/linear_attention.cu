@@ -266,6 +266,51 @@ __global__ void __launch_bounds__(NT) decay_step_kernel(const T* __restrict__ q,
   finish_head<T>(so, red, gate + row + (int64_t)h * io.DV, gain, y + (int64_t)t * ldy + (int64_t)h * io.DV, io.DV, io.eps, io.out_scale);
 }
 
+// Linear attention with a constant decay per head.  The norm spans the heads of a token: the CTA that finishes the token's last head norms the row
+// and gates it, y = rms(o) * gain * sigmoid(gate).
+template <typename T, int NR4>
+__global__ void __launch_bounds__(NT) lightning_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v,
+                                                            const T* __restrict__ gate, int64_t ld, const float* __restrict__ decay,
+                                                            const T* __restrict__ gain, T* __restrict__ y, int64_t ldy, float* __restrict__ rows,
+                                                            int* __restrict__ arrived, StepIo io) {
+  pdl_sync();
+  constexpr int DKP = NR4 * 32;
+  extern __shared__ __align__(16) float sm[];
+  float *sq = sm, *sk = sq + DKP, *sv = sk + DKP, *so = sv + io.DV;
+  __shared__ float red[32];
+  __shared__ int last;
+  const int seq = blockIdx.x, h = blockIdx.y, t = io.q_start[seq], inner = io.H * io.DV;
+  const bool fresh = io.positions[t] == 0;
+  float* state = io.state + ((int64_t)io.slots[seq] * io.H + h) * io.DV * io.DKS;
+  float4 st[NR4];
+  load_cols<NR4>(st, state, threadIdx.x >> 3, io.DV, io.DKS, fresh, threadIdx.x & 7);
+  const int64_t row = (int64_t)t * ld;
+  for (int c = threadIdx.x; c < DKP; c += NT) {
+    sq[c] = c < io.DK ? to_f<T>(q[row + h * io.DK + c]) : 0.f;
+    sk[c] = c < io.DK ? to_f<T>(k[row + h * io.DK + c]) : 0.f;
+  }
+  for (int c = threadIdx.x; c < io.DV; c += NT) sv[c] = to_f<T>(v[row + h * io.DV + c]);
+  __syncthreads();
+  step_columns<NR4, DECAY_HEAD>(st, state, io.DV, io.DKS, fresh, sq, sk, nullptr, decay[h], 1.f, sv, so);
+  __syncthreads();
+  float* yr = rows + (int64_t)seq * inner;
+  for (int c = threadIdx.x; c < io.DV; c += NT) yr[h * io.DV + c] = so[c];
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    last = atomicAdd(arrived + seq, 1) == io.H - 1;
+    if (last) arrived[seq] = 0;
+  }
+  __syncthreads();
+  if (!last) return;
+  __threadfence();
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < inner; i += NT) { const float x = __ldcg(yr + i); ss = fmaf(x, x, ss); }
+  const float inv = 1.0f / sqrtf(block_sum_x(ss, red) / inner + io.eps);
+  T* o = y + (int64_t)t * ldy;
+  for (int i = threadIdx.x; i < inner; i += NT) o[i] = from_f<T>(__ldcg(yr + i) * inv * to_f<T>(gain[i]) * sigmoid_t<T>(to_f<T>(gate[row + i])));
+}
+
 template <typename T, int NR4>
 __global__ void __launch_bounds__(NT) delta_step_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, T* __restrict__ ring_all,
                                                         int taps, const T* __restrict__ b_in, const T* __restrict__ a_in,
@@ -408,6 +453,20 @@ MARY_API int mary_delta_step(const void* x, int64_t ldx, const void* taps_w, voi
   const StepIo io = {q_start, positions, slots, state, H, HK, DK, DV, (DK + 3) / 4 * 4, eps, out_scale};
   BY_TYPE(f32, BY_WIDTH(DK, MARY_LAUNCH((delta_step_kernel<T, NR4>), dim3(S, H), NT, (2 * NR4 * 32 + 2 * DV) * 4, s, (const T*)x, ldx, (const T*)taps_w, (T*)ring,
                                         taps, (const T*)b_in, (const T*)a_in, a_log, dt_bias, (const T*)gate, (const T*)gain, (T*)y, ldy, io)));
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
+}
+
+// One token of each of S sequences of linear attention with a constant decay per head (decay [H]): recurrence, norm of the whole row, gate.  q, k, v,
+// gate: columns of projection rows with pitch ld; rows: scratch [S, H DV]; arrived: S counters, zero before and after.
+MARY_API int mary_lightning_step(const void* q, const void* k, const void* v, const void* gate, int64_t ld, const float* decay, const void* gain, void* y,
+                                 int64_t ldy, float* state, float* rows, int* arrived, const int* q_start, const int* positions, const int* slots, int S,
+                                 int H, int DK, int DV, float eps, int f32, cudaStream_t s) {
+  if (S <= 0) return MARY_OK;
+  if (H < 1 || H > 65535 || DK < 1 || DK > 256 || DV < 1 || DV > 4096 || !rows || !arrived) return MARY_ERR_BAD_ARG;
+  const StepIo io = {q_start, positions, slots, state, H, H, DK, DV, (DK + 3) / 4 * 4, eps, 1.f};
+  BY_TYPE(f32, BY_WIDTH(DK, MARY_LAUNCH((lightning_step_kernel<T, NR4>), dim3(S, H), NT, (2 * NR4 * 32 + 2 * DV) * 4, s, (const T*)q, (const T*)k,
+                                        (const T*)v, (const T*)gate, ld, decay, (const T*)gain, (T*)y, ldy, rows, arrived, io)));
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }

@@ -1,35 +1,16 @@
 // Row kernels of decoders with parallel sublayers around a 32-bit residual stream, for bf16 and for 32-bit activations: token plus
-// token-pair embedding, rotation of queries and keys by split halves with cache append, and the residual step that adds the sublayers'
+// token-pair embedding, rotation of queries and keys by split halves with cache append, rotation of queries, keys and values by neighbouring
+// pairs with norms and cache append, and the residual step that adds the sublayers'
 // outputs (the weighted rows of routed experts among them) and norms the new stream for whatever reads it next.  One CTA per token; any
 // width; norms, sums and angles in exact 32-bit (angles: reduced in 64-bit) arithmetic.
 #include "host_utils.h"
-#include "typed.cuh"
+#include "routed.cuh"
 
 using namespace mary;
 
 namespace {
 
 constexpr int NT = 256;
-
-// E values of storage type T, 16-byte aligned when E = 8.
-template <typename T, int E> __device__ __forceinline__ void load_v(const T* p, float (&f)[E]) {
-  if constexpr (E == 8 && sizeof(T) == 2) unpack16(*(const uint4*)p, f);
-  else if constexpr (E == 8) {
-    *(float4*)f = *(const float4*)p;
-    *(float4*)(f + 4) = *(const float4*)(p + 4);
-  } else {
-    f[0] = to_f<T>(p[0]);
-  }
-}
-template <typename T, int E> __device__ __forceinline__ void store_v(T* p, const float (&f)[E]) {
-  if constexpr (E == 8 && sizeof(T) == 2) *(uint4*)p = pack16(f);
-  else if constexpr (E == 8) {
-    *(float4*)p = *(const float4*)f;
-    *(float4*)(p + 4) = *(const float4*)(f + 4);
-  } else {
-    p[0] = from_f<T>(f[0]);
-  }
-}
 
 // h[t] = table[id] + pairs[(prev * mul_prev + id * mul_cur) mod buckets], the extra row `buckets` for the first token of a sequence; copies
 // in the activation type to x0 and x1 (or null).  last[slot] keeps a sequence's newest token between steps: the CTA of a sequence's
@@ -134,16 +115,90 @@ __global__ void __launch_bounds__(NT) rotate_append_kernel(T* __restrict__ q, co
   }
 }
 
-constexpr int MAXK = 32;
+// turn[t][i] = (cos, sin) of positions[t] * freq[i], times gain; angles reduced in 64 bits
+__global__ void turn_table_kernel(const int* __restrict__ positions, const double* __restrict__ freq, int n, float gain, float2* __restrict__ turn,
+                                  int64_t total) {
+  pdl_sync();
+  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total) return;
+  const double a = positions[i / n] * freq[i % n], two_pi = 6.283185307179586;
+  float s, c;
+  sincosf((float)(a - rint(a / two_pi) * two_pi), &s, &c);
+  turn[i] = make_float2(c * gain, s * gain);
+}
 
-// Where the weighted outputs of a token's routed experts come from: padded rows (row_of[t * k + j], y) or their finished sum; entries whose
-// expert index is n_experts or more stand for the normed input x itself.
-template <typename T> struct Routed {
-  const T* y; int64_t ldy; const int* row_of;
-  const float* sum;
-  const int* idx; const float* w; const T* x;
-  int k, n_experts;
+struct TurnIo {
+  const float2* turn; int n;             // queries and keys: pairs 2 i, 2 i + 1 for i < n, the dimensions behind them stay
+  const float2* vturn; int vn;           // values (vn = 0: not turned)
+  const float* temp;                     // [nq] or null
+  int nq, nk, D, DV;
+  float eps;                             // < 0: no norm
 };
+
+// One warp per head in turn: query heads are turned, divided by their root mean square, multiplied by temp and written back; key heads the
+// same without temp into the cache, value heads turned into the cache.  A lane holds NU units of 2 P neighbouring values.
+template <typename T, int P, int NU>
+__global__ void __launch_bounds__(NT) turn_norm_append_kernel(T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int64_t ld, TurnIo io,
+                                                              const int64_t* __restrict__ slots, T* __restrict__ kc, T* __restrict__ vc,
+                                                              int64_t n_slots, int* __restrict__ status) {
+  pdl_sync();
+  constexpr int E = 2 * P;
+  const int64_t t = blockIdx.x, slot = slots[t];
+  const bool ok = slot >= 0 && slot < n_slots;
+  if (!ok && threadIdx.x == 0) atomicCAS(status, 0, (int)MARY_ERR_BOUNDS);       // a slot outside the cache: recorded, no write
+  const int lane = threadIdx.x & 31;
+  for (int h = threadIdx.x >> 5; h < io.nq + 2 * io.nk; h += NT / 32) {
+    const bool is_q = h < io.nq, is_v = h >= io.nq + io.nk;
+    const int hk = h - io.nq - (is_v ? io.nk : 0), D = is_v ? io.DV : io.D, n = is_v ? io.vn : io.n;
+    if (!is_q && !ok) continue;
+    const T* src = is_q ? q + t * ld + h * D : (is_v ? v : k) + t * ld + hk * D;
+    T* dst = is_q ? q + t * ld + h * D : (is_v ? vc : kc) + (slot * io.nk + hk) * D;
+    const float2* turn = (is_v ? io.vturn : io.turn) + t * n;
+    float f[NU][E], ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < NU; ++u) {
+      const int c = (u * 32 + lane) * E;
+      if constexpr (P > 1) {
+        if (c < D) load_e<T, E>(src + c, f[u]);
+      } else {
+        f[u][0] = c < D ? to_f<T>(src[c]) : 0.f;
+        f[u][1] = c + 1 < D ? to_f<T>(src[c + 1]) : 0.f;
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < NU; ++u) {
+      const int c = (u * 32 + lane) * E;
+      if (c >= D) break;
+#pragma unroll
+      for (int p = 0; p < P; ++p) {
+        float &a = f[u][2 * p], &b = f[u][2 * p + 1];
+        if (c / 2 + p < n) {
+          const float2 cs = turn[c / 2 + p];
+          const float x = a * cs.x - b * cs.y, y = b * cs.x + a * cs.y;
+          a = x;
+          b = y;
+        }
+        ss = fmaf(a, a, fmaf(b, b, ss));
+      }
+    }
+    float m = 1.f;
+    if (!is_v && io.eps >= 0.f) m = 1.0f / sqrtf(warp_sum(ss) / D + io.eps);
+    if (is_q && io.temp) m *= io.temp[h];
+#pragma unroll
+    for (int u = 0; u < NU; ++u) {
+      const int c = (u * 32 + lane) * E;
+      if (c >= D) break;
+#pragma unroll
+      for (int j = 0; j < E; ++j) f[u][j] *= m;
+      if constexpr (P > 1) store_e<T, E>(dst + c, f[u]);
+      else {
+        dst[c] = from_f<T>(f[u][0]);
+        if (c + 1 < D) dst[c + 1] = from_f<T>(f[u][1]);
+      }
+    }
+  }
+}
+
 template <typename T> struct Follow {              // what reads the new stream: up to two norms of it, or a plain copy
   const T* w1; T* x1; const T* w2; T* x2;
   T* copy; int64_t ld;
@@ -155,49 +210,22 @@ __global__ void __launch_bounds__(NT) stream_step_kernel(const float* __restrict
                                                          float* __restrict__ h, int keep, Follow<T> f, int H, float eps) {
   pdl_sync();
   extern __shared__ float row[];
-  __shared__ float red[32], weight[MAXK], self_sh;
-  __shared__ int src[MAXK], n_src;
+  __shared__ float red[32];
+  __shared__ RoutedRows list;
   const int64_t t = blockIdx.x;
   if (r.k > 0) {
-    if (threadIdx.x == 0) {
-      float self = 0.f;
-      int n = 0;
-      for (int j = 0; j < r.k; ++j) {
-        const float w = r.w[t * r.k + j];
-        if (r.idx[t * r.k + j] >= r.n_experts) self += w;
-        else if (r.y) {
-          const int s = r.row_of[t * r.k + j];
-          if (s >= 0) { src[n] = s; weight[n++] = w; }
-        }
-      }
-      n_src = n;
-      self_sh = self;
-    }
+    if (threadIdx.x == 0) list_routed(r, t, list);
     __syncthreads();
   }
-  const float self = r.k > 0 ? self_sh : 0.f;
-  const int ns = r.k > 0 ? n_src : 0;
+  const float self = r.k > 0 ? list.self : 0.f;
+  const int ns = r.k > 0 ? list.n : 0;
   float ss = 0.f;
   for (int i = threadIdx.x * E; i < H; i += NT * E) {
     float s[E], g[E];
 #pragma unroll
     for (int j = 0; j < E; ++j) s[j] = 0.f;
     if (a) load_v<float, E>(a + t * lda + i, s);
-    if (r.sum) {
-      load_v<float, E>(r.sum + t * H + i, g);
-#pragma unroll
-      for (int j = 0; j < E; ++j) s[j] += g[j];
-    }
-    for (int e = 0; e < ns; ++e) {
-      load_v<T, E>(r.y + src[e] * r.ldy + i, g);
-#pragma unroll
-      for (int j = 0; j < E; ++j) s[j] = fmaf(weight[e], g[j], s[j]);
-    }
-    if (self != 0.f) {
-      load_v<T, E>(r.x + t * H + i, g);
-#pragma unroll
-      for (int j = 0; j < E; ++j) s[j] = fmaf(self, g[j], s[j]);
-    }
+    add_routed<T, E>(r, list, ns, self, t, i, H, s);
 #pragma unroll
     for (int j = 0; j < E; ++j) s[j] *= m;
     if (keep) {
@@ -278,13 +306,42 @@ MARY_API int mary_rotate_append(void* q, const void* k, const void* v, int64_t l
   return MARY_OK;
 }
 
-// a [T] rows of lda f32 (or null).  k > 0: routed experts, see Routed (y with row_of, or sum [T, H], or neither when every entry stands for x).
+// turn [T, n, 2] f32: cosine and sine of positions[t] * freq[i], times gain.
+MARY_API int mary_turn_table(const int* positions, const double* freq, int n, float gain, float* turn, int T_, cudaStream_t s) {
+  if (T_ <= 0 || n == 0) return MARY_OK;
+  if (n < 0) return MARY_ERR_BAD_ARG;
+  const int64_t total = (int64_t)T_ * n;
+  MARY_LAUNCH(turn_table_kernel, (unsigned)((total + NT - 1) / NT), NT, 0, s, positions, freq, n, gain, (float2*)turn, total);
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
+}
+
+// q, k, v: columns of projection rows with pitch ld (q is replaced in place).  turn [T, n, 2], vturn [T, vn, 2]: tables as above (n or vn = 0: not
+// turned); temp [nq] (or null): factors of the query heads; eps < 0: no norm of queries and keys.  kc [slots][nk][D], vc [slots][nk][DV].
+MARY_API int mary_turn_norm_append(void* q, const void* k, const void* v, int64_t ld, int nq, int nk, int D, int DV, const float* turn, int n,
+                                   const float* vturn, int vn, const float* temp, const int64_t* slots, void* kc, void* vc, float eps, int T_,
+                                   int64_t n_slots, int f32, cudaStream_t s) {
+  if (T_ <= 0) return MARY_OK;
+  if (nq < 1 || nk < 1 || D < 1 || DV < 1 || D > 640 || DV > 640 || n < 0 || 2 * n > D || vn < 0 || 2 * vn > DV) return MARY_ERR_BAD_ARG;
+  const TurnIo io = {(const float2*)turn, n, (const float2*)vturn, vn, temp, nq, nk, D, DV, eps};
+  const bool vec = D % 4 == 0 && DV % 4 == 0 && ld % 4 == 0 && aligned16({q, k, v, kc, vc});
+  const int widest = D > DV ? D : DV;
+  BY_TYPE(f32, {
+    auto fn = !vec ? turn_norm_append_kernel<T, 1, 10>
+                   : (widest <= 128 ? turn_norm_append_kernel<T, 2, 1> : (widest <= 256 ? turn_norm_append_kernel<T, 2, 2> : turn_norm_append_kernel<T, 2, 5>));
+    MARY_LAUNCH(fn, T_, NT, 0, s, (T*)q, (const T*)k, (const T*)v, ld, io, slots, (T*)kc, (T*)vc, n_slots, mary_status_ptr());
+  });
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
+}
+
+// a [T] rows of lda f32 (or null).  k > 0: routed experts, see routed.cuh (y with row_of, or sum [T, H], or neither when every entry stands for x).
 // w1 / x1, w2 / x2: norm gains and [T, H] results (x1 null: no norm; x2 null: one norm); copy: rows of ldc elements or null.
 MARY_API int mary_stream_step(const float* a, int64_t lda, float m, const void* y, int64_t ldy, const int* row_of, const float* sum, const int* idx,
                               const float* w, const void* x, int k, int n_experts, const void* vec, float* h, int keep, const void* w1, void* x1,
                               const void* w2, void* x2, void* copy, int64_t ldc, int T_, int H, float eps, int f32, cudaStream_t s) {
   if (T_ <= 0) return MARY_OK;
-  if (k < 0 || k > MAXK || (k > 0 && (!idx || !w || !x || (y && !row_of))) || (x1 && !w1) || (x2 && (!w2 || !x1))) return MARY_ERR_BAD_ARG;
+  if (k < 0 || k > ROUTED_MAX || (k > 0 && (!idx || !w || !x || (y && !row_of))) || (x1 && !w1) || (x2 && (!w2 || !x1))) return MARY_ERR_BAD_ARG;
   const bool wide = H % 8 == 0 && lda % 4 == 0 && ldy % 8 == 0 && ldc % 8 == 0 && aligned16({a, y, sum, x, vec, h, w1, x1, w2, x2, copy});
   const size_t sm = (size_t)H * 4;
   static MarySmemSlots smem_set[4] = {};

@@ -52,7 +52,7 @@ __device__ __forceinline__ f2 mul2(f2 a, f2 b) {
 
 struct ScanParams {
   const void* q; const void* k; const void* v;      // token rows of ldq / ldk / ldv elements; q, k head h / rep, v head h
-  const float* decay;                               // [T, H * DK] per channel, or [T, H] per head
+  const float* decay;                               // [T, H * DK] per channel (lda floats between tokens; 0: the same for all), or [T, H] per head
   const float* beta;                                // [T, H] (decay per head, delta rule)
   const float* pairs;                               // [T, HK, 8] (delta rule): k_j . k_i and k_j . q_i of the row's block of four;
                                                     // [T, HK, 4] (decay per head): k_j . q_i
@@ -60,7 +60,7 @@ struct ScanParams {
   float* out;                                       // [T, H * DV]
   float* state;                                     // [slots][H][DV][DKS]
   const int* q_start; const int* kv_len; const int* slots;
-  int64_t ldq, ldk, ldv;
+  int64_t ldq, ldk, ldv, lda;
   int H, HK, rep, DK, DV, DKS;
   float q_scale;
 };
@@ -109,12 +109,12 @@ __global__ void __launch_bounds__(NT) scan_kernel(const ScanParams p) {
   const TI* qp = (const TI*)p.q + (int64_t)(row0 + my_t) * p.ldq + (int64_t)hk * p.DK + my_c * E;
   const TI* kp = (const TI*)p.k + (int64_t)(row0 + my_t) * p.ldk + (int64_t)hk * p.DK + my_c * E;
   const TI* vp = (const TI*)p.v + (int64_t)(row0 + my_t) * p.ldv + (int64_t)h * p.DV + blockIdx.x * COLS + my_c;
-  const float* ap = BLOCKS ? p.decay + (int64_t)(row0 + lane) * p.H + h : p.decay + ((int64_t)(row0 + my_t) * p.H + h) * p.DK + my_c * EA;
+  const float* ap = BLOCKS ? p.decay + (int64_t)(row0 + lane) * p.H + h : p.decay + (int64_t)(row0 + my_t) * p.lda + (int64_t)h * p.DK + my_c * EA;
   const float* bp = BLOCKS ? p.beta + (int64_t)(row0 + lane) * p.H + h : nullptr;
   constexpr int NP = DELTA ? 2 : 1;
   const float4* pp = BLOCKS ? (const float4*)p.pairs + ((int64_t)(row0 + lane) * p.HK + hk) * NP : nullptr;
   const float skip = MODE == DECAY_HEAD ? p.skip[h] : 0.f;
-  const int64_t step_q = CT * p.ldq, step_k = CT * p.ldk, step_v = CT * p.ldv, step_a = (int64_t)CT * p.H * (BLOCKS ? 1 : p.DK);
+  const int64_t step_q = CT * p.ldq, step_k = CT * p.ldk, step_v = CT * p.ldv, step_a = CT * (BLOCKS ? (int64_t)p.H : p.lda);
   const int ch_left = p.DK - my_c * E, ch_left_a = p.DK - my_c * EA, col_left = p.DV - blockIdx.x * COLS - my_c;
 
   Reg<TI, E> rq[NVQ], rk[NVQ];
@@ -377,20 +377,20 @@ int dispatch(const ScanParams& p, int S, cudaStream_t s) {
 template <typename TI, int MODE>
 int entry(const ScanParams& p, int S, cudaStream_t s) {
   constexpr int E = Pack<TI>::N;
-  const bool vec = p.DK % E == 0 && p.DK % 4 == 0 && p.ldq % E == 0 && p.ldk % E == 0 && !(((uintptr_t)p.q | (uintptr_t)p.k | (uintptr_t)p.decay) & 15);
+  const bool vec = p.DK % E == 0 && p.DK % 4 == 0 && p.ldq % E == 0 && p.ldk % E == 0 && p.lda % 4 == 0 && !(((uintptr_t)p.q | (uintptr_t)p.k | (uintptr_t)p.decay) & 15);
   return vec ? dispatch<TI, MODE, true>(p, S, s) : dispatch<TI, MODE, false>(p, S, s);
 }
 
 }  // namespace
 
-// q, k, v: bf16, or f32 when x_f32; the state [slots][H][DV][DK rounded up to 4] is updated in place.  S sequences, rows
+// q, k, v: bf16, or f32 when x_f32; decay [T] rows of lda floats (0: one row for all tokens); the state [slots][H][DV][DK rounded up to 4] is updated in place.  S sequences, rows
 // q_start[s] .. q_start[s+1].
-MARY_API int mary_decay_scan(const void* q, const void* k, const void* v, const float* decay, float* out, float* state, const int* q_start,
+MARY_API int mary_decay_scan(const void* q, const void* k, const void* v, const float* decay, int64_t lda, float* out, float* state, const int* q_start,
                              const int* kv_len, const int* slots, int S, int64_t ldq, int64_t ldk, int64_t ldv, int H, int DK, int DV,
                              float q_scale, int x_f32, cudaStream_t s) {
   if (S <= 0) return MARY_OK;
   if (H < 1 || DK < 1 || DK > 256 || DV < 1 || S > 65535 || H > 65535) return MARY_ERR_BAD_ARG;
-  ScanParams p = {q, k, v, decay, nullptr, nullptr, nullptr, out, state, q_start, kv_len, slots, ldq, ldk, ldv, H, H, 1, DK, DV, (DK + 3) / 4 * 4, q_scale};
+  ScanParams p = {q, k, v, decay, nullptr, nullptr, nullptr, out, state, q_start, kv_len, slots, ldq, ldk, ldv, lda, H, H, 1, DK, DV, (DK + 3) / 4 * 4, q_scale};
   return x_f32 ? entry<float, DECAY_CHANNEL>(p, S, s) : entry<__nv_bfloat16, DECAY_CHANNEL>(p, S, s);
 }
 
@@ -401,7 +401,7 @@ MARY_API int mary_delta_scan(const float* q, const float* k, const float* v, con
                              int HK, int H, int DK, int DV, float q_scale, cudaStream_t s) {
   if (S <= 0) return MARY_OK;
   if (HK < 1 || H < 1 || H % HK || DK < 1 || DK > 256 || DV < 1 || S > 65535 || H > 65535 || ((uintptr_t)pairs & 15)) return MARY_ERR_BAD_ARG;
-  ScanParams p = {q, k, v, decay, beta, pairs, nullptr, out, state, q_start, kv_len, slots, ldq, ldk, ldv, H, HK, H / HK, DK, DV, (DK + 3) / 4 * 4, q_scale};
+  ScanParams p = {q, k, v, decay, beta, pairs, nullptr, out, state, q_start, kv_len, slots, ldq, ldk, ldv, 0, H, HK, H / HK, DK, DV, (DK + 3) / 4 * 4, q_scale};
   return entry<float, DECAY_DELTA>(p, S, s);
 }
 
@@ -412,6 +412,6 @@ MARY_API int mary_head_decay_scan(const float* q, const float* k, const float* v
                                   int64_t ldq, int64_t ldk, int64_t ldv, int G, int H, int DK, int DV, cudaStream_t s) {
   if (S <= 0) return MARY_OK;
   if (G < 1 || H < 1 || H % G || DK < 1 || DK > 256 || DV < 1 || S > 65535 || H > 65535 || ((uintptr_t)pairs & 15)) return MARY_ERR_BAD_ARG;
-  ScanParams p = {q, k, v, decay, beta, pairs, skip, out, state, q_start, kv_len, slots, ldq, ldk, ldv, H, G, H / G, DK, DV, (DK + 3) / 4 * 4, 1.f};
+  ScanParams p = {q, k, v, decay, beta, pairs, skip, out, state, q_start, kv_len, slots, ldq, ldk, ldv, 0, H, G, H / G, DK, DV, (DK + 3) / 4 * 4, 1.f};
   return entry<float, DECAY_HEAD>(p, S, s);
 }

@@ -118,6 +118,23 @@ __global__ void glu_any_kernel(const T* __restrict__ gu, T* __restrict__ out, in
   out[i] = from_f<T>(a * u);
 }
 
+// y = act(y) in place on the first n columns of rows with pitch ld.  act: 0 = tanh-form GELU, 1 = SiLU
+template <typename T>
+__global__ void act_rows_kernel(T* __restrict__ y, int64_t ld, int n, int64_t total, int act) {
+  pdl_sync();
+  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total) return;
+  T* p = y + i / n * ld + i % n;
+  const float g = to_f<T>(*p), k0 = 0.7978845608028654f, k1 = 0.044715f;
+  *p = from_f<T>(act == 0 ? 0.5f * g * (1.0f + tanhf(k0 * (g + k1 * g * g * g))) : silu_x(g));
+}
+
+__global__ void soft_cap_kernel(float* __restrict__ x, int64_t n, float cap) {
+  pdl_sync();
+  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) x[i] = cap * tanhf(x[i] / cap);
+}
+
 // One warp per (token, head) of a projection row: RMS norm of query and key heads (gains optional), queries to qo, keys and values
 // to their cache slots.  Keys are DK wide, values DV wide; q / k / v are row views of one projection with pitch ld.
 template <typename T>
@@ -306,6 +323,25 @@ MARY_API int mary_glu_any(const void* gu, void* out, int T_, int F, int act, flo
   if (act < 0 || act > 3 || act == 2) return MARY_ERR_BAD_ARG;
   const int64_t n = (int64_t)T_ * F;
   BY_TYPE(f32, MARY_LAUNCH((glu_any_kernel<T>), (unsigned)((n + NT - 1) / NT), NT, 0, s, (const T*)gu, (T*)out, F, n, act, limit));
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
+}
+
+// act: 0 = tanh-form GELU, 1 = SiLU, in place on the first n columns of T rows with pitch ld
+MARY_API int mary_act_rows(void* y, int64_t ld, int T_, int n, int act, int f32, cudaStream_t s) {
+  if (T_ <= 0 || n <= 0) return MARY_OK;
+  if (act < 0 || act > 1 || ld < n) return MARY_ERR_BAD_ARG;
+  const int64_t total = (int64_t)T_ * n;
+  BY_TYPE(f32, MARY_LAUNCH((act_rows_kernel<T>), (unsigned)((total + NT - 1) / NT), NT, 0, s, (T*)y, ld, n, total, act));
+  MARY_CHECK_LAUNCH();
+  return MARY_OK;
+}
+
+// x = cap * tanh(x / cap), n contiguous f32 values in place
+MARY_API int mary_soft_cap(float* x, int64_t n, float cap, cudaStream_t s) {
+  if (n <= 0) return MARY_OK;
+  if (!(cap > 0.f)) return MARY_ERR_BAD_ARG;
+  MARY_LAUNCH(soft_cap_kernel, (unsigned)((n + NT - 1) / NT), NT, 0, s, x, n, cap);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }

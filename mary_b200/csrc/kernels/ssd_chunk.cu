@@ -33,7 +33,9 @@ struct ChunkParams {
   const float* skip; float* y; float* state;
   float4* gram;                          // [chunk][G][10 blocks][2][32 lanes]: C_i . B_j as a lane's accumulators of two 16 x 8 tiles
   const int* q_start; const int* kv_len; const int* slots;
-  int T, G, H, N, P, C;
+  int T, G, H, N, P;
+  int64_t C;                             // elements between the rows of two tokens
+  int per_head;                          // 1: decays that are the same for all tokens, dt, c_hi and c_lo [H][64] by place in the chunk
 };
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t a) {
@@ -176,7 +178,7 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
   const bool x_col = p0 + xk * 8 < p.P;
   const bf16* x_row = p.xbc + (int64_t)row0 * p.C + h * p.P + (x_col ? p0 + xk * 8 : 0);
   const uint32_t x_at = xr * S::XROW + xk * 16;
-  const int64_t dt_at = (int64_t)h * p.T + row0;
+  const int64_t dt_at = p.per_head ? (int64_t)h * L : (int64_t)h * p.T + row0;
 
   auto load = [&](int c) {                                  // chunk c -> stage c & 1
     const uint32_t s = sm + (c & 1) * S::STAGE;
@@ -186,7 +188,7 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
     const bool in = x_col && xr < left;
     cp16(s + 2 * S::TILE + x_at, x_row + (int64_t)(in ? t0 + xr : t0) * p.C, in);
     if (tid < L) {                                          // tokens past the end: no step, the decay of the last one
-      const int64_t o = dt_at + min(t0 + tid, n - 1);
+      const int64_t o = dt_at + (p.per_head ? min(tid, left - 1) : min(t0 + tid, n - 1));
       const uint32_t d = s + S::SC + tid * 4;
       cp4(d, p.dt + o, tid < left);
       cp4(d + L * 4, p.c_hi + o, true);
@@ -492,16 +494,29 @@ MARY_API int mary_ssd_chunk_supported(int N, int P) { return N >= 8 && N <= 256 
 
 MARY_API int64_t mary_ssd_chunk_scratch_floats(int T, int S, int G) { return ((int64_t)T / L + S + 1) * G * 10 * 64 * 4; }
 
+static int chunk_run(const ChunkParams& p, int S, int max_q, cudaStream_t s) {
+  if (S <= 0 || p.T <= 0) return MARY_OK;
+  if (p.G < 1 || p.H < 1 || p.H % p.G || p.H > 65535 || S > 65535 || !mary_ssd_chunk_supported(p.N, p.P) || p.C % 8 ||
+      (((uintptr_t)p.xbc | (uintptr_t)p.gram) & 15))
+    return MARY_ERR_BAD_ARG;
+  if (p.N <= 64) return launch_chunk<64>(p, S, max_q, s);
+  if (p.N <= 128) return launch_chunk<128>(p, S, max_q, s);
+  return launch_chunk<256>(p, S, max_q, s);
+}
+
 // y [T, H P] f32; the state [slots][H][P][N] is read (zero for a portion that starts its sequence) and updated in place.  scratch:
 // mary_ssd_chunk_scratch_floats(T, S, G) floats, 16-byte aligned.
 MARY_API int mary_ssd_chunk(const void* xbc, const float* dt, const float* c_hi, const float* c_lo, const float* skip, float* y, float* state,
                             float* scratch, const int* q_start, const int* kv_len, const int* slots, int S, int max_q, int T, int G, int H, int N, int P,
                             cudaStream_t s) {
-  if (S <= 0 || T <= 0) return MARY_OK;
-  if (G < 1 || H < 1 || H % G || H > 65535 || S > 65535 || !mary_ssd_chunk_supported(N, P) || (((uintptr_t)xbc | (uintptr_t)scratch) & 15))
-    return MARY_ERR_BAD_ARG;
-  const ChunkParams p = {(const bf16*)xbc, dt, c_hi, c_lo, skip, y, state, (float4*)scratch, q_start, kv_len, slots, T, G, H, N, P, H * P + 2 * G * N};
-  if (N <= 64) return launch_chunk<64>(p, S, max_q, s);
-  if (N <= 128) return launch_chunk<128>(p, S, max_q, s);
-  return launch_chunk<256>(p, S, max_q, s);
+  return chunk_run({(const bf16*)xbc, dt, c_hi, c_lo, skip, y, state, (float4*)scratch, q_start, kv_len, slots, T, G, H, N, P, H * P + 2 * G * N, 0}, S, max_q, s);
+}
+
+// Linear attention with one constant decay per head, S_t = d S_{t-1} + k_t v_t^T, y_t = S_t^T q_t: the same chunks with q, k, v for C, B, x.  vkq:
+// rows of ld elements [v: H P | k: H N | q: H N]; one, c_hi, c_lo, zero [H][64]: step size 1, log2 of d^1 .. d^64 as two floats, no skip.
+MARY_API int mary_lightning_chunk(const void* vkq, int64_t ld, const float* one, const float* c_hi, const float* c_lo, const float* zero, float* y,
+                                  float* state, float* scratch, const int* q_start, const int* kv_len, const int* slots, int S, int max_q, int T, int H,
+                                  int N, int P, cudaStream_t s) {
+  if (ld < (int64_t)H * (P + 2 * N)) return MARY_ERR_BAD_ARG;
+  return chunk_run({(const bf16*)vkq, one, c_hi, c_lo, zero, y, state, (float4*)scratch, q_start, kv_len, slots, T, H, H, N, P, ld, 1}, S, max_q, s);
 }

@@ -96,8 +96,9 @@ __global__ void __launch_bounds__(256) ss_prep_kernel(const T* __restrict__ xbc,
   }
 }
 
-// out[t, part] = rms(y[t, part] * silu(z[t, part])) * gain, one CTA per (token, part) of n values; E values per access
-template <typename T, int E>
+// out[t, part] = rms(y[t, part] * silu(z[t, part])) * gain, one CTA per (token, part) of n values; E values per access.  NORM_FIRST: rms(y[t, part])
+// * gain * sigmoid(z[t, part]) instead
+template <typename T, int E, bool NORM_FIRST>
 __global__ void gated_part_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, int64_t ldz, const T* __restrict__ gain, T* __restrict__ out,
                                        int64_t ldo, int inner, int n, float eps) {
   pdl_sync();
@@ -113,10 +114,10 @@ __global__ void gated_part_norm_kernel(const float* __restrict__ y, const T* __r
   auto value = [&](int i, float (&u)[E]) {
     float zv[E];
     load_e<float, E>(yr + i, u);
-    load_e<T, E>(zr + i, zv);
+    if constexpr (!NORM_FIRST) load_e<T, E>(zr + i, zv);
 #pragma unroll
     for (int e = 0; e < E; ++e) {
-      u[e] *= silu_t<T>(zv[e]);
+      if constexpr (!NORM_FIRST) u[e] *= silu_t<T>(zv[e]);
       ss = fmaf(u[e], u[e], ss);
     }
   };
@@ -125,6 +126,11 @@ __global__ void gated_part_norm_kernel(const float* __restrict__ y, const T* __r
     load_e<T, E>(gain + c0 + i, g);
 #pragma unroll
     for (int e = 0; e < E; ++e) u[e] *= inv * g[e];
+    if constexpr (NORM_FIRST) {
+      load_e<T, E>(zr + i, g);
+#pragma unroll
+      for (int e = 0; e < E; ++e) u[e] *= sigmoid_t<T>(g[e]);
+    }
     store_e<T, E>(o + i, u);
   };
 #pragma unroll
@@ -254,8 +260,9 @@ MARY_API int mary_ss_prep(const void* xbc, int64_t ldx, const void* taps_w, cons
   return MARY_OK;
 }
 
+// norm_first = 0: rms(y * silu(z)) * gain, 1: rms(y) * gain * sigmoid(z), in `parts` equal parts of a row
 MARY_API int mary_gated_part_norm(const float* y, const void* z, int64_t ldz, const void* gain, void* out, int64_t ldo, int n_tok, int inner, int parts,
-                                  float eps, int f32, cudaStream_t s) {
+                                  float eps, int norm_first, int f32, cudaStream_t s) {
   if (n_tok <= 0) return MARY_OK;
   if (parts < 1 || inner % parts || parts > 65535) return MARY_ERR_BAD_ARG;
   const int n = inner / parts;
@@ -264,7 +271,8 @@ MARY_API int mary_gated_part_norm(const float* y, const void* z, int64_t ldz, co
   BY_TYPE(f32, {
     const uintptr_t mask = 4 * sizeof(T) - 1;
     const bool vec = n % 4 == 0 && ldz % 4 == 0 && ldo % 4 == 0 && !(((uintptr_t)z | (uintptr_t)gain | (uintptr_t)out) & mask) && !((uintptr_t)y & 15);
-    auto fn = vec ? gated_part_norm_kernel<T, 4> : gated_part_norm_kernel<T, 1>;
+    auto fn = norm_first ? (vec ? gated_part_norm_kernel<T, 4, true> : gated_part_norm_kernel<T, 1, true>)
+                         : (vec ? gated_part_norm_kernel<T, 4, false> : gated_part_norm_kernel<T, 1, false>);
     MARY_LAUNCH(fn, dim3(n_tok, parts), nt, 0, s, y, (const T*)z, ldz, (const T*)gain, (T*)out, ldo, inner, n, eps);
   });
   MARY_CHECK_LAUNCH();

@@ -63,6 +63,26 @@ template <typename T, int E> __device__ __forceinline__ void store_e(T* p, const
   }
 }
 
+// E values, one 16-byte access of bf16 or two of f32 when E = 8, see load_e otherwise.
+template <typename T, int E> __device__ __forceinline__ void load_v(const T* p, float (&f)[E]) {
+  if constexpr (E == 8 && sizeof(T) == 2) unpack16(*(const uint4*)p, f);
+  else if constexpr (E == 8) {
+    *(float4*)f = *(const float4*)p;
+    *(float4*)(f + 4) = *(const float4*)(p + 4);
+  } else {
+    load_e<T, E>(p, f);
+  }
+}
+template <typename T, int E> __device__ __forceinline__ void store_v(T* p, const float (&f)[E]) {
+  if constexpr (E == 8 && sizeof(T) == 2) *(uint4*)p = pack16(f);
+  else if constexpr (E == 8) {
+    *(float4*)p = *(const float4*)f;
+    *(float4*)(p + 4) = *(const float4*)(f + 4);
+  } else {
+    store_e<T, E>(p, f);
+  }
+}
+
 // Exact forms (these files are compiled without fast math): logistic function, SiLU, softplus and the log of the logistic function.
 __device__ __forceinline__ float sigmoid_x(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float silu_x(float x) { return x / (1.0f + expf(-x)); }
@@ -78,6 +98,10 @@ template <typename T> __device__ __forceinline__ float exp_t(float x) {
 template <typename T> __device__ __forceinline__ float silu_t(float x) {
   if constexpr (sizeof(T) == 4) return silu_x(x);
   else return __fdividef(x, 1.0f + __expf(-x));
+}
+template <typename T> __device__ __forceinline__ float sigmoid_t(float x) {
+  if constexpr (sizeof(T) == 4) return sigmoid_x(x);
+  else return __fdividef(1.0f, 1.0f + __expf(-x));
 }
 template <typename T> __device__ __forceinline__ float log_sigmoid_t(float x) {
   if constexpr (sizeof(T) == 4) return log_sigmoid_x(x);

@@ -449,28 +449,191 @@ class DifferentialAttentionMixer(nn.Module):
             v.data.copy_(get(p + n))
 
 
-class RoutedExperts(nn.Module):
-    """A mixture of GLU experts: softmax scores over all of them, the ``top`` best by score plus a correction, weighted by ``scale`` times the score.
-    The last ``identity`` router outputs stand for the input itself.  The result goes to ``ops.stream_step``, which sums it up."""
+class TurnedAttentionMixer(nn.Module):
+    """Causal attention in which values are rotated as well: queries and keys turned by neighbouring pairs on their first dimensions and then divided by
+    their root mean square, a learned temperature per head, scores capped by a hyperbolic tangent, a sink of score 0 without a value; values enter the
+    cache turned by their position, and the result is turned back by the query's.  Writes the heads' outputs; the output projection is the
+    caller's."""
 
-    def __init__(self, width, experts, identity, ff, top, scale, act, limit, dtype, device):
+    def __init__(self, width, heads, kv_heads, dk, dv, scale, cap, freq, gain, vfreq, eps, dtype, device):
+        """``freq`` (f64) and ``gain``: as ``yarn_frequencies`` gives them; ``vfreq``: frequencies of the value pairs."""
+        super().__init__()
+        if dk > 640 or dv > 512 or 2 * vfreq.numel() != dv:
+            raise ValueError(f"head widths {dk}/{dv}: the kernels hold 640/512, and values are turned in pairs")
+        self.heads, self.kv_heads, self.dk, self.dv, self.scale, self.cap, self.gain, self.eps = heads, kv_heads, dk, dv, scale, cap, gain, eps
+        self.proj = FusedProjection(dict(q=heads * dk, k=kv_heads * dk, v=kv_heads * dv))
+        self.w_in = param(self.proj.rows, width, dtype=dtype, device=device)
+        self.temp = param(heads, dtype=torch.float32, device=device)
+        for name, f in (("freq", freq), ("vfreq", vfreq)):
+            self.register_buffer(name, f.to(torch.float64).to(device), persistent=False)
+        self.register_buffer("sink", torch.zeros(heads, dtype=torch.float32, device=device), persistent=False)
+        self.table_key = (tuple(freq.tolist()), gain, tuple(vfreq.tolist()))
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.dv
+
+    def kv_spec(self):
+        return self.kv_heads, self.dk, self.dv
+
+    def tables(self, meta):
+        """Cosines and sines of the batch's positions for queries and keys and for values; the same for every mixer with this ``table_key``."""
+        return ops.turn_table(meta.positions, self.freq, self.gain) if self.freq.numel() else None, ops.turn_table(meta.positions, self.vfreq)
+
+    def forward(self, x, meta, kc, vc, tables, out):
+        y = ops.linear(x, self.w_in)
+        part = lambda n: self.proj.part(y, n)  # noqa: E731
+        q, (turn, vturn) = part("q"), tables
+        ops.turn_norm_append(q, part("k"), part("v"), self.heads, self.kv_heads, self.dk, turn, vturn, self.temp, meta, kc, vc, self.eps)
+        ops.attention_exact(q.unflatten(1, (self.heads, self.dk)), kc, vc, meta, self.scale, out=out,
+                            form=ops.AttentionForm(cap=self.cap, sink=self.sink, turn=vturn))
+
+    def load(self, get, p: str) -> None:
+        for n in "qkv":
+            self.proj.fill(self.w_in, n, get(p + n))
+        self.temp.data.copy_(get(p + "temp"))
+
+
+class HeadDecays(nn.Module):
+    """One constant decay per head in the forms that the kernels take: ``head [H]``, ``channel [H * dk]`` and, for chunks of 64 tokens, ``chunk [4, H, 64]``: a step
+    size of one, log2 of ``d ** 1 .. d ** 64`` as two floats, a skip of zero."""
+
+    def __init__(self, decays, dk: int, device):
+        super().__init__()
+        d = torch.tensor(decays, dtype=torch.float64)
+        if bool((d < 0.0).any()) or bool((d > 1.0).any()):
+            raise ValueError(f"decays {list(decays)} outside 0 .. 1")
+        c = torch.log2(d).clamp(min=-1e4)[:, None] * torch.arange(1, 65, dtype=torch.float64)       # 2 ** -1e4 is zero in 32 bits
+        hi = c.float()
+        chunk = torch.stack([torch.ones_like(hi), hi, (c - hi.double()).float(), torch.zeros_like(hi)])
+        for name, t in (("head", d.float()), ("channel", d.float().repeat_interleave(dk)), ("chunk", chunk)):
+            self.register_buffer(name, t.contiguous().to(device), persistent=False)
+
+
+class LightningMixer(nn.Module):
+    """Linear attention with one constant decay per head, SiLU on queries, keys and values; the read-out of all heads normed together and gated by a
+    logistic function of the input.  Writes the gated row; the output projection is the caller's."""
+
+    def __init__(self, width, heads, dk, dv, decays, eps, dtype, device):
+        super().__init__()
+        if dk > 256 or dv > 4096:
+            raise ValueError(f"recurrent widths {dk}/{dv} exceed what the kernels hold (256/4096)")
+        if len(decays) != heads:
+            raise ValueError(f"{len(decays)} decays for {heads} heads")
+        self.heads, self.dk, self.dv, self.eps = heads, dk, dv, eps
+        self.proj = FusedProjection(dict(v=heads * dv, k=heads * dk, q=heads * dk, g=heads * dv))
+        self.w_in = param(self.proj.rows, width, dtype=dtype, device=device)
+        self.norm = param(heads * dv, dtype=dtype, device=device)
+        self.decays = HeadDecays(decays, dk, device)
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.dv
+
+    def state_spec(self):
+        return {"S": (state_shape(self.heads, self.dk, self.dv), torch.float32)}
+
+    def forward(self, x, meta, state, out):
+        y = ops.linear_act(x, self.w_in, "silu", cols=self.proj.at["g"][0])
+        part = lambda n: self.proj.part(y, n)  # noqa: E731
+        ops.lightning_attention(y, part("q"), part("k"), part("v"), part("g"), self.decays, self.norm, state["S"], meta, self.heads, self.dk, self.dv,
+                                self.eps, out)
+
+    def load(self, get, p: str) -> None:
+        for n in self.proj.at:
+            self.proj.fill(self.w_in, n, get(p + n))
+        self.norm.data.copy_(get(p + "norm"))
+
+
+class DenseMLP(nn.Module):
+    """``down(act(up x))`` as f32."""
+
+    def __init__(self, width: int, ff: int, act: str, dtype, device):
+        super().__init__()
+        self.act = act
+        self.w_up, self.w_down = param(ff, width, dtype=dtype, device=device), param(width, ff, dtype=dtype, device=device)
+
+    def forward(self, x):
+        return ops.linear_f32(ops.linear_act(x, self.w_up, self.act), self.w_down)
+
+    def load(self, get, p: str) -> None:
+        self.w_up.data.copy_(get(p + "up"))
+        self.w_down.data.copy_(get(p + "down"))
+
+
+class StreamWeights(nn.Module):
+    """How one sublayer reads from and writes to ``n`` residual streams: its input ``sum_s read[s] x_s``, then ``x_t <- sum_s mix[s, t] x_s + write[t] y``.
+    A single stream without weights of its own is the plain residual sum."""
+
+    def __init__(self, n: int, device):
+        super().__init__()
+        self.read, self.write, self.mix = (param(*shape, dtype=torch.float32, device=device) for shape in ((n,), (n,), (n, n)))
+
+    def plain(self) -> None:
+        for p in (self.read, self.write, self.mix):
+            p.data.fill_(1.0)
+
+    def load(self, get, p: str) -> None:
+        for mine, theirs in ((self.read, "in"), (self.write, "out"), (self.mix, "mix")):
+            mine.data.copy_(get(p + theirs))
+
+
+class RoutedExperts(nn.Module):
+    """A mixture of GLU experts: softmax scores over all of them, the ``top`` best by score plus a correction (``correction`` False: by score), weighted by
+    ``scale`` times the score, or with ``renorm`` by the softmax over the chosen ones.  The last ``identity`` scores stand for the input itself; ``extra`` more
+    router rows give logits of their own.  The result goes to ``ops.stream_step`` or ``ops.mix_streams``, which sums it up."""
+
+    def __init__(self, width, experts, identity, ff, top, scale, act, limit, dtype, device, renorm: bool = False, correction: bool = True, extra: int = 0):
         super().__init__()
         if experts + identity > 512 or not 1 <= top <= min(32, experts + identity):
             raise ValueError(f"{top} of {experts} + {identity} experts: the router holds 512 and chooses up to 32")
         self.experts, self.identity, self.ff, self.top, self.scale, self.act, self.limit = experts, identity, ff, top, scale, act, limit
         kw = dict(dtype=dtype, device=device)
-        self.w_router = param(experts + identity, width, **kw)
-        self.correction = param(experts + identity, dtype=torch.float32, device=device)
+        self.renorm, self.scores = renorm, experts + identity
+        self.w_router = param(experts + identity + extra, width, **kw)
+        self.correction = param(experts + identity, dtype=torch.float32, device=device) if correction else None
         self.w_gu, self.w_down = param(experts, 2 * ff, width, **kw), param(experts, width, ff, **kw)
 
-    def forward(self, x):
-        idx, w = ops.router_topk(ops.linear_f32(x, self.w_router), self.top, "softmax", self.correction, scale=self.scale, renorm=False)
+    def forward(self, x, z=None):
+        """``z``: the router's logits where the caller has them already."""
+        z = ops.linear_f32(x, self.w_router) if z is None else z
+        idx, w = ops.router_topk(z[:, :self.scores], self.top, "softmax", self.correction, scale=self.scale, renorm=self.renorm)
         return ops.expert_outputs(x, idx, w, self.w_gu, self.w_down, self.act, self.limit)
 
     def load(self, get, p: str) -> None:
-        self.w_router.data.copy_(get(p + "router"))
-        self.correction.data.copy_(get(p + "correction"))
+        self.w_router.data[:self.scores].copy_(get(p + "router"))
+        if self.correction is not None:
+            self.correction.data.copy_(get(p + "correction"))
         for e in range(self.experts):
             self.w_gu.data[e, :self.ff].copy_(get(f"{p}e{e}.gate"))
             self.w_gu.data[e, self.ff:].copy_(get(f"{p}e{e}.up"))
             self.w_down.data[e].copy_(get(f"{p}e{e}.down"))
+
+
+class SharedRoutedExperts(nn.Module):
+    """Routed experts weighted by the softmax over the chosen ones, beside a shared expert that a logistic gate per token (its logit is one more row of
+    the router) multiplies.  The shared expert may be absent."""
+
+    def __init__(self, width, experts, ff, top, act, limit, shared_ff, shared_limit, dtype, device):
+        super().__init__()
+        self.act, self.shared_ff, self.shared_limit = act, shared_ff, shared_limit
+        self.routed = RoutedExperts(width, experts, 0, ff, top, 1.0, act, limit, dtype, device, renorm=True, correction=False, extra=1 if shared_ff else 0)
+        self.w_shared = self.w_down = None
+        if shared_ff:
+            self.w_shared, self.w_down = param(2 * shared_ff, width, dtype=dtype, device=device), param(width, shared_ff, dtype=dtype, device=device)
+
+    def forward(self, x):
+        """``(shared expert's output f32 or None, its gate's logits [T] or None, routed experts)`` as ``ops.mix_streams`` takes them."""
+        z = ops.linear_f32(x, self.routed.w_router)
+        routed = self.routed(x, z)
+        if self.w_shared is None:
+            return None, None, routed
+        return ops.linear_f32(ops.linear_glu(x, self.w_shared, self.act, self.shared_limit), self.w_down), z[:, self.routed.scores], routed
+
+    def load(self, get, p: str) -> None:
+        self.routed.load(get, p)
+        if self.w_shared is not None:
+            self.routed.w_router.data[self.routed.scores:].copy_(get(p + "shared.sg"))
+            self.w_shared.data[:self.shared_ff].copy_(get(p + "shared.gate"))
+            self.w_shared.data[self.shared_ff:].copy_(get(p + "shared.up"))
+            self.w_down.data.copy_(get(p + "shared.down"))

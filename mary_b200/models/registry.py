@@ -53,6 +53,14 @@ def _load_nipurax(d, loader, device, dtype):
     return model
 
 
+def _load_kivezen(d, loader, device, dtype):
+    from .kivezen.config import KivezenConfig
+    from .kivezen.model import KivezenModel, load_into
+    model = KivezenModel(KivezenConfig.from_json(d), dtype=dtype, device=device)
+    load_into(model, loader)
+    return model
+
+
 def _load_mistral(d, loader, device, dtype):
     from .mistral.model import MistralConfig, MistralModel, load_into
     model = MistralModel(MistralConfig.from_hf(d), dtype=dtype, device=device)
@@ -75,6 +83,9 @@ FAMILIES = [
            kernels=_DENSE_KERNELS + ("attention_general", "attention_mla", "residual32", "linear_attention", "recurrent_scan", "latent", "state_space", "ssd_chunk")),
     Family("nipurax", lambda d: d.get("architecture") == "Nipurax", _load_nipurax, page_size=64, f32_on_gpu=True,
            kernels=_DENSE_KERNELS + ("attention_general", "attention_gqa_tc", "residual32", "parallel_stream", "moe", "expert_step")),
+    Family("kivezen", lambda d: d.get("architecture") == "Kivezen", _load_kivezen, page_size=64, f32_on_gpu=True,
+           kernels=_DENSE_KERNELS + ("attention_general", "attention_gqa_tc", "residual32", "linear_attention", "recurrent_scan", "state_space", "ssd_chunk",
+                                     "parallel_stream", "hyper_streams", "moe", "expert_step")),
     Family("gemma4", lambda d: str(d.get("model_type", "")).startswith("gemma4"), _load_gemma4),
     Family("mistral", lambda d: d.get("model_type") in ("mistral", "ministral", "qwen3", "mistral3"), _load_mistral),
 ]

@@ -173,6 +173,17 @@ def glu(gate_up, act: str = "geglu"):
     return {"geglu": ref.geglu, "swiglu": ref.swiglu, "situ": ref.situ}[act](gate_up[..., :F], gate_up[..., F:])
 
 
+def linear_act(x, w, act: str, cols: int | None = None):
+    """``act(x @ w^T)``, the activation (``gelu``: tanh form, or ``silu``) on the first ``cols`` outputs only (None: all of them)."""
+    cols = w.shape[0] if cols is None else cols
+    return _k().linear_act(x, w, act, cols) if _cuda(x) else ref.linear_act(x, w, act, cols)
+
+
+def soft_cap(x, cap: float):
+    """``cap * tanh(x / cap)`` of f32 values, in place."""
+    return _h().soft_cap(x, cap) if _cuda(x) else x.copy_(cap * torch.tanh(x / cap))
+
+
 def linear_glu(x, w_gu, act: str = "geglu", limit: float = 0.0, out=None):
     """``act(x @ gate^T) * (x @ up^T)`` with ``w_gu = [gate; up]``; fused into the GEMM epilogue on the GPU.  ``clamped``: gate at most
     ``limit``, up within it, ``g * sigmoid(1.702 g) * (u + 1)``.  ``out``: a row view that receives the result."""
@@ -279,7 +290,7 @@ def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, b
     """Causal paged attention whose scores, softmax weights and sums stay in 32 bits, for any head widths: ``[T, Hq * DV]``.  ``window``: keys
     at most ``window - 1`` positions back (0: all); ``bias [Hq, window]`` f32 is added to the scaled score by distance; ``gate [T, Hq * DV]``
     multiplies the result by its logistic function before it is rounded.  ``form`` (an ``AttentionForm``; no window, bias or gate then): chunks,
-    capped scores, sinks, query temperature, the difference of two maps; ``q`` may be a row view of a projection."""
+    capped scores, sinks, query temperature, the difference of two maps, a rotation of the result; ``q`` may be a row view of a projection."""
     if _cuda(q):
         return _h().attention_exact(q, kcache, vcache, meta, scale, out, window, bias, gate, form)
     o = ref.attention_exact(q, kcache, vcache, meta, scale, window, bias, gate, form)
@@ -328,6 +339,13 @@ def state_space(xbc, taps_w, taps_b, dt_in, dt_bias, a_log, skip, z, gain, norm_
     return f(xbc, taps_w, taps_b, dt_in, dt_bias, a_log, skip, z, gain, norm_parts, ring, state, meta, G, H, N, P, eps, out)
 
 
+def lightning_attention(y, q, k, v, gate, decays, gain, state, meta, H, dk, dv, eps, out):
+    """``S <- d_h S + k v^T``, ``o = S^T q`` per head with constant decays (``models.mixers.HeadDecays``); then ``rms(o) * gain * sigmoid(gate)``, the
+    norm over the whole row, into ``out [T, H * dv]``.  ``q``, ``k``, ``v``, ``gate``: columns of the projection rows ``y``.  ``state`` as below."""
+    f = _h().lightning_attention if _cuda(q) else ref.lightning_attention
+    return f(y, q, k, v, gate, decays, gain, state, meta, H, dk, dv, eps, out)
+
+
 def decayed_linear_attention(q, k, v, gate, low, a2, a2_bias, inv_tau, gain, state, meta, H, dk, dv, eps, out_scale, out):
     """``S <- diag(alpha) S + k v^T``, ``o = S^T q`` per head with ``alpha = sigmoid(low a2^T + a2_bias) ** inv_tau`` per key channel and
     ``q`` scaled by ``dk ** -0.5``; then ``rms(o) * gain * silu(gate) * out_scale`` into ``out [T, H * dv]``.  Continues from and updates
@@ -364,6 +382,32 @@ def rotate_append(q, k, v, n_q, n_kv, dk, freq, meta, kcache, vcache) -> None:
     ``freq``: f64 frequencies of the pairs ``(i, i + len(freq))``, ``None`` for no rotation (then ``q`` may be None)."""
     f = _pl().rotate_append if _cuda(k) else ref.rotate_append
     return f(q, k, v, n_q, n_kv, dk, freq, meta, kcache, vcache)
+
+
+def turn_table(positions, freq, gain: float = 1.0):
+    """Cosine and sine of ``positions[t] * freq[i]`` times ``gain``: f32 ``[T, n, 2]`` (``freq``: f64, angles reduced in 64 bits)."""
+    return _pl().turn_table(positions, freq, gain) if _cuda(positions) else ref.turn_table(positions, freq, gain)
+
+
+def turn_norm_append(q, k, v, n_q, n_kv, dk, turn, vturn, temp, meta, kcache, vcache, eps) -> None:
+    """Queries (``n_q`` heads of ``dk``) in place and keys (``n_kv`` heads) into the cache, their pairs ``2 i, 2 i + 1`` turned by the table ``turn`` (dimensions
+    beyond it stay), then divided by their root mean square per head (``eps`` None: not), queries times ``temp [n_q]`` (or None); values turned by ``vturn`` (or
+    None) into the cache.  ``q``, ``k``, ``v``: row views of one projection."""
+    f = _pl().turn_norm_append if _cuda(k) else ref.turn_norm_append
+    return f(q, k, v, n_q, n_kv, dk, turn, vturn, temp, meta, kcache, vcache, eps)
+
+
+def embed_streams(ids, table, n: int, weights, gain, eps):
+    """``n`` residual streams that all start as the token's row of the embedding table, and the first sublayer's input: ``(xs [T, n, width] f32,
+    rms(sum_s weights[s] xs[s]) * gain)``."""
+    return (_pl() if _cuda(table) else ref).embed_streams(ids, table, n, weights, gain, eps)
+
+
+def mix_streams(xs, mix, out, a, gate, routed, weights, gain, eps, keep: bool = True):
+    """The step between two sublayers of a residual of several streams: ``y = a * sigmoid(gate) + routed experts`` (``a``: f32 rows or None, ``gate [T]`` f32
+    or None, ``routed``: from ``expert_outputs`` or None), ``xs[t] <- sum_s mix[s, t] xs[s] + out[t] y`` in place (``keep`` False: left undefined); returns
+    ``rms(sum_t weights[t] xs[t]) * gain`` in the activation type."""
+    return (_pl() if _cuda(xs) else ref).mix_streams(xs, mix, out, a, gate, routed, weights, gain, eps, keep)
 
 
 def expert_outputs(x, idx, w, gate_up, down, act: str, limit: float = 0.0):

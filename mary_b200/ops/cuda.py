@@ -258,6 +258,33 @@ def linear_f32(x, w, split_k: int | None = None, alpha: float = 1.0):
         return gemm_splitk(x, w, 0 if split_k is None else sk, f32=True, alpha=alpha) if sk > 1 else gemm(x, w, alpha=alpha, epi="f32")
 
 
+declare("mary_gemm_bf16_act", "pppiiilllii" + "plpis")
+
+
+def linear_act(x, w, act: str, cols: int):
+    """The activation (``gelu`` or ``silu``) is applied to the f32 sums in the epilogue, except on the CUDA-core paths."""
+    M, K = x.shape
+    N = w.shape[0]
+    if x.dtype == torch.float32 or K % 8 or x.stride(0) % 8 or w.stride(0) % 8:
+        from .cuda_hybrid import act_rows, gemm_simt
+        return act_rows(gemm_simt(x, w), act, cols)
+    if M == 1 and K <= 8192 and N * K * 2 <= MATVEC_MAX_BYTES and w.stride(1) == 1:
+        return step_matvec(x, w, mode=act, act_rows=cols)
+    out = _empty(M, N, dtype=torch.bfloat16, device=x.device)
+    code = {"gelu": 1, "silu": 2}[act]
+    ws = cnt = None
+    if _auto_split_k(M, N, K) > 1:
+        ws, cnt = _sk_workspace(x.device)
+    sk = (None, 0, None, 0) if ws is None else (_p(ws), ws.numel(), _p(cnt), cnt.numel())
+    args = lambda *sk: (_p(x), _p(w), _p(out), M, N, K, x.stride(0), w.stride(0), out.stride(0), code, cols, *sk, _stream())  # noqa: E731
+    with static_weights:
+        rc = lib().mary_gemm_bf16_act(*args(*sk))
+        if rc != 0 and ws is not None:             # more tiles than the scratch holds: without the split
+            rc = lib().mary_gemm_bf16_act(*args(None, 0, None, 0))
+    check(rc, "gemm_bf16_act")
+    return out
+
+
 def linear_glu(x, w_gu, act: str = "geglu", limit: float = 0.0, out=None):
     """``out``: a row view that receives the result (its rows 16-byte aligned where the product is)."""
     M = x.shape[0]
@@ -372,7 +399,7 @@ def _gate(gate):
 
 class _Form(ctypes.Structure):
     """``MaryAttnForm`` of ``csrc/kernels/attention_form.cuh``."""
-    _fields_ = [("sink", ctypes.c_void_p), ("q_ld", ctypes.c_int64), ("chunk", ctypes.c_int32), ("maps", ctypes.c_int32),
+    _fields_ = [("turn", ctypes.c_void_p), ("sink", ctypes.c_void_p), ("q_ld", ctypes.c_int64), ("chunk", ctypes.c_int32), ("maps", ctypes.c_int32),
                 ("temp_every", ctypes.c_int32), ("temp_coef", ctypes.c_float), ("cap", ctypes.c_float), ("mix", ctypes.c_float), ("post", ctypes.c_float),
                 ("eps", ctypes.c_float)]
 
@@ -388,6 +415,9 @@ def form_struct(form, q):
         if form.sink is not None:
             assert form.sink.dtype == torch.float32 and form.sink.is_contiguous() and form.sink.shape == (q.shape[1],)
             s.sink = form.sink.data_ptr()
+        if form.turn is not None:
+            assert form.turn.dtype == torch.float32 and form.turn.is_contiguous() and form.turn.shape[0] == q.shape[0]
+            s.turn = form.turn.data_ptr()
         if form.temperature is not None:
             s.temp_coef, s.temp_every = form.temperature
         if form.difference is not None:
@@ -809,19 +839,20 @@ def mla_unabsorb_o(o_lat, w_uv, H):
 
 
 # ------------------------------------------------------------------------------------------------- one-token decoder layer step
-declare("mary_step_matvec", "ppfpliippi" + "fs")
+declare("mary_step_matvec", "ppfpliippi" + "fis")
 declare("mary_step_attention", "pppppppppp" + "iiiilffp" + "s")
 
 
-def step_matvec(h, w, gain=None, eps: float = 1e-6, res=None, mode: str = "plain", alpha: float = 1.0, out=None):
+def step_matvec(h, w, gain=None, eps: float = 1e-6, res=None, mode: str = "plain", alpha: float = 1.0, out=None, act_rows: int = 0):
     """One-token matrix-vector stage of the fused layer step: ``W x`` (``plain``), ``res + W x`` (``residual``), ``act(W_gate x) * (W_up x)``
-    over ``w = [gate; up]`` (``swiglu`` / ``geglu`` / ``clamped`` with limit ``alpha``) or ``alpha * W x`` as f32 (``f32``), with ``x = rms(h) * gain`` when ``gain`` is given,
+    over ``w = [gate; up]`` (``swiglu`` / ``geglu`` / ``clamped`` with limit ``alpha``) or ``alpha * W x`` as f32 (``f32``) or ``W x`` with an
+    activation of its first ``act_rows`` values (``gelu`` / ``silu``), with ``x = rms(h) * gain`` when ``gain`` is given,
     else ``x = h``.  ``h [1, K]`` -> ``[1, N]``."""
-    m = {"plain": 0, "residual": 1, "swiglu": 2, "f32": 3, "geglu": 4, "clamped": 5}[mode]
+    m = {"plain": 0, "residual": 1, "swiglu": 2, "f32": 3, "geglu": 4, "clamped": 5, "gelu": 6, "silu": 7}[mode]
     K = h.shape[-1]
     N = w.shape[0] // 2 if m in (2, 4, 5) else w.shape[0]
     y = _empty(1, N, dtype=torch.float32 if m == 3 else torch.bfloat16, device=h.device) if out is None else out
-    check(lib().mary_step_matvec(_p(h), _p(gain), eps, _p(w), w.stride(0), N, K, _p(res), _p(y), m, alpha, _stream()), "step_matvec")
+    check(lib().mary_step_matvec(_p(h), _p(gain), eps, _p(w), w.stride(0), N, K, _p(res), _p(y), m, alpha, act_rows, _stream()), "step_matvec")
     return y
 
 

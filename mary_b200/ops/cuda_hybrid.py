@@ -16,6 +16,10 @@ declare("mary_embed32", "ppppiifiis")
 declare("mary_post_norm_add", "plppppiifis")
 declare("mary_rmsnorm32", "pppiifis")
 declare("mary_glu_any", "ppiiifis")
+declare("mary_act_rows", "pliiiis")
+declare("mary_soft_cap", "plfs")
+declare("mary_lightning_chunk", "pl" + "ppppppp" + "ppp" + "iiiiiis")
+declare("mary_lightning_step", "pppplpppl" + "ppp" + "ppp" + "iiiifis")
 declare("mary_qk_norm_append", "ppp" + "liiii" + "pppppp" + "fil" + "is")
 declare("mary_attention_general", "ppppppppp" + "iii" + "lllll" + "iiiiiii" + "fpplppis")
 declare("mary_map_difference", "pplpiiifffis")
@@ -25,7 +29,7 @@ declare("mary_channel_decay", "pli" + "ppp" + "iifis")
 declare("mary_delta_prep", "pl" + "pppppp" + "ppp" + "pppppp" + "iiiiiii" + "is")
 declare("mary_conv_history", "plpppp" + "iiiis")
 declare("mary_gated_head_norm", "pplppl" + "iiiffis")
-declare("mary_decay_scan", "pppppp" + "ppp" + "illl" + "iiifis")
+declare("mary_decay_scan", "pppplpp" + "ppp" + "illl" + "iiifis")
 declare("mary_delta_scan", "pppppppp" + "ppp" + "illl" + "iiiifs")
 declare("mary_decay_step", "ppppp" + "li" + "ppfp" + "plfp" + "ppp" + "iiiiffis")
 declare("mary_delta_step", "plppi" + "pppppp" + "plp" + "ppp" + "iiiiiffis")
@@ -44,7 +48,7 @@ declare("mary_ssd_chunk", "pppppppp" + "ppp" + "iiiiiiis")
 declare("mary_ssd_chunk_scratch_floats", "iii", ret64=True)
 declare("mary_ssd_chunk_supported", "ii")
 declare("mary_head_decay_scan", "pppppppp" + "p" + "ppp" + "illl" + "iiiis")
-declare("mary_gated_part_norm", "pplppl" + "iiifis")
+declare("mary_gated_part_norm", "pplppl" + "iiifiis")
 declare("mary_ss_step", "plppp" + "pppp" + "pp" + "ipl" + "ppp" + "ppp" + "iiiiiifis")
 
 
@@ -108,6 +112,19 @@ def glu_any(gate_up, act: str, limit: float = 0.0):
     check(lib().mary_glu_any(_p(gate_up.contiguous()), _p(out), T, F2 // 2, {"geglu": 0, "swiglu": 1, "clamped": 3}[act], limit, _f32(gate_up),
                              _stream()), "glu_any")
     return out
+
+
+def act_rows(y, act: str, cols: int):
+    """The activation in place on the first ``cols`` columns."""
+    py, ld = _rows(y)
+    check(lib().mary_act_rows(py, ld, y.shape[0], cols, {"gelu": 0, "silu": 1}[act], _f32(y), _stream()), "act_rows")
+    return y
+
+
+def soft_cap(x, cap: float):
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    check(lib().mary_soft_cap(_p(x), x.numel(), cap, _stream()), "soft_cap")
+    return x
 
 
 def qk_norm_append(q, k, v, n_q, n_kv, dk, dv, q_gain, k_gain, meta, kcache, vcache, eps):
@@ -221,11 +238,13 @@ def channel_decay(low, a2, bias, inv_tau: float):
 
 
 def decay_scan(q, k, v, decay, state, meta, H, dk, dv, q_scale):
-    """Decayed linear attention over the portions of a batch; the state of every sequence's slot is read and updated.  f32 ``[T, H, dv]``."""
+    """Decayed linear attention over the portions of a batch; the state of every sequence's slot is read and updated.  f32 ``[T, H, dv]``.  ``decay``: a
+    row of channel decays per token, or a single one for all of them."""
     T = q.shape[0]
     out = _empty(T, H, dv, dtype=torch.float32, device=q.device)
     (pq, lq), (pk, lk), (pv, lv) = _rows(q), _rows(k), _rows(v)
-    check(lib().mary_decay_scan(pq, pk, pv, _p(decay), _p(out), _p(state), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots), meta.num_seqs,
+    lda = 0 if decay.dim() == 1 else decay.stride(0)
+    check(lib().mary_decay_scan(pq, pk, pv, _p(decay), lda, _p(out), _p(state), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots), meta.num_seqs,
                                 lq, lk, lv, H, dk, dv, q_scale, _f32(q), _stream()), "decay_scan")
     return out
 
@@ -500,9 +519,10 @@ def ssd_chunk(rows, dt, hi, lo, skip, state, meta, G, H, N, P):
     return y
 
 
-def gated_part_norm(y, z, gain, parts, eps, out):
+def gated_part_norm(y, z, gain, parts, eps, out, norm_first: bool = False):
     (pz, ldz), (po, ldo) = _rows(z), _rows(out)
-    check(lib().mary_gated_part_norm(_p(y), pz, ldz, _p(gain), po, ldo, y.shape[0], y.shape[1], parts, eps, _f32(z), _stream()), "gated_part_norm")
+    check(lib().mary_gated_part_norm(_p(y), pz, ldz, _p(gain), po, ldo, y.shape[0], y.shape[1], parts, eps, int(norm_first), _f32(z), _stream()),
+          "gated_part_norm")
     return out
 
 
@@ -526,3 +546,34 @@ def state_space(xbc, taps_w, taps_b, dt_in, dt_bias, a_log, skip, z, gain, norm_
     x, b, c, dt, decay, pairs = ss_prep(xbc, taps_w, taps_b, ring, dt_in, dt_bias, a_log, meta, G, H, N, P)
     conv_history(xbc, ring, meta, taps, taps_w.shape[0])
     return gated_part_norm(head_decay_scan(x, b, c, dt, decay, pairs, skip, state, meta, G, H, N, P), z, gain, norm_parts, eps, out)
+
+
+# --------------------------------------------------------------------------- linear attention with one constant decay per head
+def lightning_chunk(y_in, decays, state, meta, H, dk, dv):
+    """The recurrence on the tensor cores, 64 tokens at a time, over projection rows that start with ``[v | k | q]``: f32 ``[T, H * dv]``."""
+    T = y_in.shape[0]
+    o = _empty(T, H * dv, dtype=torch.float32, device=y_in.device)
+    scratch = _empty(lib().mary_ssd_chunk_scratch_floats(T, meta.num_seqs, H), dtype=torch.float32, device=y_in.device)
+    one, hi, lo, zero = (_p(t) for t in decays.chunk)
+    py, ld = _rows(y_in)
+    check(lib().mary_lightning_chunk(py, ld, one, hi, lo, zero, _p(o), _p(state), _p(scratch), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots),
+                                     meta.num_seqs, meta.max_q_len, T, H, dk, dv, _stream()), "lightning_chunk")
+    return o
+
+
+def lightning_attention(y_in, q, k, v, gate, decays, gain, state, meta, H, dk, dv, eps, out):
+    (pq, ld), (po, ldo) = _rows(q), _rows(out)
+    assert all(t.stride(0) == ld for t in (k, v, gate))
+    if meta.max_q_len == 1:
+        S = meta.num_seqs
+        rows = _empty(S, H * dv, dtype=torch.float32, device=q.device)
+        check(lib().mary_lightning_step(pq, _p(k), _p(v), _p(gate), ld, _p(decays.head), _p(gain), po, ldo, _p(state), _p(rows),
+                                        _p(_arrival_counters(q.device, S)), _p(meta.q_start), _p(meta.positions), _p(meta.state_slots), S, H, dk, dv, eps,
+                                        _f32(q), _stream()), "lightning_step")
+        return out
+    if (q.dtype == torch.bfloat16 and lib().mary_ssd_chunk_supported(dk, dv) and ld % 8 == 0 and y_in.data_ptr() % 16 == 0
+            and v.data_ptr() == y_in.data_ptr() and k.data_ptr() == v.data_ptr() + H * dv * 2 and q.data_ptr() == k.data_ptr() + H * dk * 2):
+        o = lightning_chunk(y_in, decays, state, meta, H, dk, dv)
+    else:
+        o = decay_scan(q, k, v, decays.channel, state, meta, H, dk, dv, 1.0).view(-1, H * dv)
+    return gated_part_norm(o, gate, gain, 1, eps, out, norm_first=True)

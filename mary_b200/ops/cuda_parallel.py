@@ -15,6 +15,9 @@ from .cuda_moe import grouped_gemm_bf16, moe_plan
 declare("mary_embed_pairs", "ppp" + "llip" + "pppp" + "ppp" + "liiiis")
 declare("mary_rotate_append", "ppp" + "liiiii" + "ppp" + "pp" + "ilis")
 declare("mary_stream_step", "plf" + "plp" + "pppp" + "ii" + "ppi" + "ppppp" + "liifis")
+declare("mary_mix_streams", "ppi" + "plpl" + "plpppppii" + "ppp" + "ii" + "ppp" + "iifis")
+declare("mary_turn_table", "ppifpis")
+declare("mary_turn_norm_append", "ppp" + "liiii" + "pipip" + "ppp" + "filis")
 declare("mary_gather_rows", "plpiipis")
 declare("mary_expert_glu", "plpiiiplpiiifs")
 declare("mary_expert_down", "pppiiiplpiis")
@@ -40,6 +43,25 @@ def rotate_append(q, k, v, n_q, n_kv, dk, freq, meta, kcache, vcache):
     assert freq is None or freq.dtype == torch.float64
     check(lib().mary_rotate_append(_p(q), pk, pv, ld, n_q, n_kv, dk, v.shape[1], n, _p(freq), _p(meta.positions), _p(meta.slot_mapping), _p(kcache),
                                    _p(vcache), k.shape[0], kcache.shape[0] * kcache.shape[1], _f32(k), _stream()), "rotate_append")
+
+
+def turn_table(positions, freq, gain: float):
+    T, n = positions.shape[0], freq.numel()
+    assert freq.dtype == torch.float64 and positions.dtype == torch.int32
+    out = _empty(T, n, 2, dtype=torch.float32, device=positions.device)
+    check(lib().mary_turn_table(_p(positions), _p(freq), n, gain, _p(out), T, _stream()), "turn_table")
+    return out
+
+
+def turn_norm_append(q, k, v, n_q, n_kv, dk, turn, vturn, temp, meta, kcache, vcache, eps):
+    T = q.shape[0]
+    (pq, ld), (pk, l2), (pv, l3) = _rows(q), _rows(k), _rows(v)
+    assert ld == l2 == l3 and kcache.is_contiguous() and vcache.is_contiguous() and kcache.dtype == q.dtype
+    table = lambda t: (None, 0) if t is None else (_p(t), t.shape[1])  # noqa: E731
+    assert all(t is None or (t.is_contiguous() and t.dtype == torch.float32 and t.shape[0] == T) for t in (turn, vturn))
+    check(lib().mary_turn_norm_append(pq, pk, pv, ld, n_q, n_kv, dk, vcache.shape[3], *table(turn), *table(vturn), _p(temp), _p(meta.slot_mapping),
+                                      _p(kcache), _p(vcache), -1.0 if eps is None else eps, T, kcache.shape[0] * kcache.shape[1], _f32(q), _stream()),
+          "turn_norm_append")
 
 
 # --------------------------------------------------------------------------- routed experts
@@ -116,6 +138,36 @@ def expert_outputs(x, idx, w, gate_up, down, act: str, limit: float = 0.0) -> Ro
 
 
 # --------------------------------------------------------------------------- the residual step
+def _routed_args(r, like):
+    """The arguments that describe routed experts to a kernel (see ``csrc/kernels/routed.cuh``)."""
+    if r is None:
+        return None, 0, None, None, None, None, None, 0, 0
+    assert r.x.is_contiguous() and r.x.dtype == like.dtype and (r.y is None or r.y.dtype == like.dtype)
+    return (_p(r.y), 0 if r.y is None else r.y.stride(0), _p(r.row_of), _p(r.sum), _p(r.idx), _p(r.w), _p(r.x), r.idx.shape[1], r.n_experts)
+
+
+def embed_streams(ids, table, n: int, weights, gain, eps):
+    ids = ids.to(torch.int32)
+    T, H = ids.shape[0], table.shape[1]
+    xs = _empty(T, n, H, dtype=torch.float32, device=table.device)
+    x = _empty(T, H, dtype=table.dtype, device=table.device)
+    check(lib().mary_mix_streams(_p(ids), _p(table), table.shape[0], None, 0, None, 0, *_routed_args(None, x), None, None, _p(xs), n, 1, _p(weights),
+                                 _p(gain), _p(x), T, H, eps, _f32(table), _stream()), "embed_streams")
+    return xs, x
+
+
+def mix_streams(xs, mix, out, a, gate, routed, weights, gain, eps, keep: bool):
+    T, n, H = xs.shape
+    x = _empty(T, H, dtype=gain.dtype, device=xs.device)
+    pa, lda = (None, 0) if a is None else _rows(a)
+    assert xs.dtype == torch.float32 and xs.is_contiguous() and (a is None or a.dtype == torch.float32)
+    assert gate is None or (gate.dtype == torch.float32 and gate.dim() == 1 and gate.shape[0] == T)
+    assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (mix, out, weights)) and mix.shape == (n, n)
+    check(lib().mary_mix_streams(None, None, 0, pa, lda, _p(gate), 0 if gate is None else gate.stride(0), *_routed_args(routed, x), _p(mix), _p(out), _p(xs), n,
+                                 int(keep), _p(weights), _p(gain), _p(x), T, H, eps, _f32(x), _stream()), "mix_streams")
+    return x
+
+
 def stream_step(h, a, m, routed, vec, keep, gains, eps, copy):
     T, H = h.shape
     like = next(t for t in (*gains, copy) if t is not None)
@@ -123,14 +175,9 @@ def stream_step(h, a, m, routed, vec, keep, gains, eps, copy):
     xs = [_empty(T, H, dtype=like.dtype, device=h.device) for _ in gains]
     pa, lda = (None, 0) if a is None else _rows(a)
     assert h.dtype == torch.float32 and h.is_contiguous() and (a is None or a.dtype == torch.float32) and len(gains) <= 2
-    r = routed
-    if r is not None:
-        assert r.x.is_contiguous() and r.x.dtype == like.dtype and (r.y is None or r.y.dtype == like.dtype)
     pc, ldc = (None, 0) if copy is None else _rows(copy)
     g = list(gains) + [None] * (2 - len(gains))
     x = xs + [None] * (2 - len(gains))
-    check(lib().mary_stream_step(pa, lda, m, *((None, 0, None, None, None, None, None, 0, 0) if r is None else
-                                               (_p(r.y), 0 if r.y is None else r.y.stride(0), _p(r.row_of), _p(r.sum), _p(r.idx), _p(r.w), _p(r.x),
-                                                r.idx.shape[1], r.n_experts)),
+    check(lib().mary_stream_step(pa, lda, m, *_routed_args(routed, like),
                                  _p(vec), _p(h), int(keep), _p(g[0]), _p(x[0]), _p(g[1]), _p(x[1]), pc, ldc, T, H, eps, f32, _stream()), "stream_step")
     return xs

@@ -366,7 +366,7 @@ def _attention_form(q, kcache, vcache, meta, scale, f):
         if f.sink is not None:
             sc = torch.cat([sc, f.sink.float()[:, None, None].expand(-1, sc.shape[1], 1)], -1)
         out[rows] = torch.einsum("hnl,lhd->nhd", torch.softmax(sc, -1)[..., :kl[s]], V)
-    return out
+    return out if f.turn is None else _turn_pairs(out, f.turn, -1.0)
 
 
 def attention_exact(q, kcache, vcache, meta, scale, window: int = 0, bias=None, gate=None, form=None):
@@ -483,6 +483,67 @@ def rotate_append(q, k, v, n_q, n_kv, dk, freq, meta, kcache, vcache):
         q.copy_(rotate_halves(q.reshape(T, n_q, dk), meta.positions, freq).reshape(T, -1))
         k = rotate_halves(k, meta.positions, freq)
     kv_append(k.reshape(T, *kcache.shape[2:]), v.reshape(T, *vcache.shape[2:]), kcache, vcache, meta.slot_mapping)
+
+
+def turn_table(positions, freq, gain: float):
+    a = positions.double()[:, None] * freq.double()[None]
+    return (torch.stack([a.cos(), a.sin()], -1).float() * gain).contiguous()
+
+
+def _turn_pairs(x, turn, sign: float = 1.0):
+    """``x [T, H, D]`` f32: the pair ``2 i, 2 i + 1`` turned by entry ``i`` of the table ``[T, n, 2]``, backwards with ``sign`` -1; the other dimensions stay."""
+    n = turn.shape[1]
+    c, s = turn[:, None, :, 0], sign * turn[:, None, :, 1]
+    u, v = x[..., 0:2 * n:2], x[..., 1:2 * n:2]
+    return torch.cat([torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2), x[..., 2 * n:]], -1)
+
+
+def turn_norm_append(q, k, v, n_q, n_kv, dk, turn, vturn, temp, meta, kcache, vcache, eps):
+    T = k.shape[0]
+    y = []
+    for z, n in ((q, n_q), (k, n_kv)):
+        z = z.reshape(T, n, dk).float()
+        z = z if turn is None else _turn_pairs(z, turn)
+        y.append(z if eps is None else z / torch.sqrt(z.pow(2).mean(-1, keepdim=True) + eps))
+    vv = v.reshape(T, n_kv, -1).float()
+    vv = vv if vturn is None else _turn_pairs(vv, vturn)
+    q.copy_((y[0] if temp is None else y[0] * temp.float()[:, None]).reshape(T, -1))
+    kv_append(y[1].to(kcache.dtype), vv.to(vcache.dtype), kcache, vcache, meta.slot_mapping)
+
+
+def linear_act(x, w, act: str, cols: int):
+    y = linear(x, w).float()
+    y[:, :cols] = F.gelu(y[:, :cols], approximate="tanh") if act == "gelu" else F.silu(y[:, :cols])
+    return y.to(x.dtype)
+
+
+def embed_streams(ids, table, n: int, weights, gain, eps):
+    e = table[ids.long()].float()
+    return e[:, None].repeat(1, n, 1), rmsnorm32(e * weights.sum(), gain, eps)
+
+
+def mix_streams(xs, mix, out, a, gate, routed, weights, gain, eps, keep):
+    y = 0.0
+    if a is not None:
+        y = a.float() if gate is None else a.float() * torch.sigmoid(gate)[:, None]
+    if routed is not None:
+        y = y + routed
+    xs.copy_(torch.einsum("tsw,so->tow", xs, mix) + out[:, None] * y[:, None])
+    return rmsnorm32(torch.einsum("tsw,s->tw", xs, weights), gain, eps)
+
+
+def lightning_attention(y, q, k, v, gate, decays, gain, state, meta, H, dk, dv, eps, out):
+    T = q.shape[0]
+    q, k, v = q.reshape(T, H, dk).float(), k.reshape(T, H, dk).float(), v.reshape(T, H, dv).float()
+    o = torch.empty(T, H, dv)
+    for rows, slot, pos in _portions(meta):
+        S = state[slot, :, :, :dk] * (0.0 if pos == 0 else 1.0)                  # [H, dv, dk]
+        for t in range(rows.start, rows.stop):
+            S = S * decays.head[:, None, None] + v[t][:, :, None] * k[t][:, None, :]
+            o[t] = (S * q[t][:, None, :]).sum(-1)
+        state[slot, :, :, :dk] = S
+    out.copy_(rmsnorm32(o.reshape(T, H * dv), gain.float(), eps) * torch.sigmoid(gate.float()))
+    return out
 
 
 def clamped_glu(g, u, limit: float):
