@@ -63,14 +63,16 @@ def ramp_frequencies(dims: int, base: float, scaling: dict | None):
     return out, 0.1 * math.log(scaling["factor"]) + 1.0
 
 
-def rotate_pairs(x, freq, gain: float = 1.0, sign: float = 1.0):
-    """``x [T, H, D]``: dimensions ``2 i`` and ``2 i + 1`` turn by ``sign * position * freq[i]``; dimensions beyond the pairs stay."""
-    y = x.clone()
+def rotate_pairs(x, freq, gain: float = 1.0, sign: float = 1.0, start: int = 0):
+    """``x [T, H, D]``, its first row at position ``start``: dimensions ``2 i`` and ``2 i + 1`` turn by ``sign * position * freq[i]``; dimensions beyond the
+    pairs stay."""
+    y, n = x.clone(), 2 * len(freq)
+    f = torch.tensor(freq, dtype=torch.float64)
     for t in range(x.shape[0]):
-        for i, f in enumerate(freq):
-            c, s = math.cos(t * f) * gain, math.sin(sign * t * f) * gain
-            u, v = x[t, :, 2 * i], x[t, :, 2 * i + 1]
-            y[t, :, 2 * i], y[t, :, 2 * i + 1] = u * c - v * s, v * c + u * s
+        a = sign * (start + t) * f
+        c, s = torch.cos(a) * gain, torch.sin(a) * gain
+        u, v = x[t, :, 0:n:2], x[t, :, 1:n:2]
+        y[t, :, 0:n:2], y[t, :, 1:n:2] = u * c - v * s, v * c + u * s
     return y
 
 

@@ -1,0 +1,463 @@
+"""The Kivezen decoder and the mechanisms it is made of against the plain float64 oracle, on the host path and on the CUDA path (32-bit and
+bf16): each mechanism alone, whole prompts, token-by-token decoding, portions, mixed batches, reuse of pages and state slots."""
+import math
+import random
+
+import pytest
+import torch
+
+from mary_b200 import ops
+from mary_b200.models.mixers import HeadDecays, SharedRoutedExperts, state_shape, yarn_frequencies
+from mary_b200.models.registry import FAMILIES, make_engine
+from mary_b200.oracle import kivezen as oracle
+from mary_b200.runtime.batch import BatchMeta
+from mary_b200.runtime.kv_cache import PagedKVCache
+
+from kivezen_cases import CONFIGS, SCALING, attention, build, config, dense, lightning, moe, random_weights
+from paged_cases import Paged, bf16, error, prompt, schedule
+
+FAMILY = next(f for f in FAMILIES if f.name == "kivezen")
+TARGETS = [pytest.param(("cpu", torch.float32), id="cpu"), pytest.param(("cuda", torch.float32), id="cuda-f32", marks=pytest.mark.gpu),
+           pytest.param(("cuda", torch.bfloat16), id="cuda-bf16", marks=pytest.mark.gpu)]
+
+
+@pytest.fixture(params=TARGETS)
+def target(request):
+    return request.param
+
+
+def tol(target, f32=2e-5, b16=1.5e-2):
+    return f32 if target[1] == torch.float32 else b16
+
+
+def rand(g, *shape):
+    return bf16(torch.randn(*shape, generator=g))
+
+
+# --------------------------------------------------------------------------- residual streams
+@pytest.mark.parametrize("width", [8, 50, 72, 333, 2056])
+@pytest.mark.parametrize("n", [1, 2, 3, 4, 6, 8, 11, 16])
+def test_streams_start_as_the_embedding_and_mix(target, width, n):
+    """The mix matrix is not symmetric, every weight differs; all streams are formed from the old ones; rows wider than the streams; a gate of every sign."""
+    dev, dt = target
+    g = torch.Generator().manual_seed(width + n)
+    T, V, eps = 5, 40, 1e-2
+    table, gains = rand(g, V, width), rand(g, 3, width)
+    ids = torch.randint(0, V, (T,), generator=g)
+    read, write, mix = torch.randn(3, n, generator=g), torch.randn(n, generator=g), torch.randn(n, n, generator=g)
+    a, gate = torch.randn(T, width + 8, generator=g)[:, :width], 3.0 * torch.randn(T, 2, generator=g)
+    put = lambda x: x.to(dev, dt)  # noqa: E731
+    xs, x = ops.embed_streams(ids.int().to(dev), put(table), n, read[0].to(dev), put(gains[0]), eps)
+    want = torch.stack([table[ids].double()] * n)
+    assert torch.equal(xs.cpu().double(), want.transpose(0, 1)) and x.dtype == dt
+    assert error(x, oracle.rms(oracle.streams_in(want, read[0].double()), gains[0].double(), eps)) < tol(target, 1e-6, 4e-3)
+    for step, (gated, keep) in enumerate(((True, True), (False, False))):
+        y = a.double() * (oracle.sigmoid(gate[:, 1:].double()) if gated else 1.0)
+        want = oracle.streams_out(want, y, mix.double(), write.double())
+        x = ops.mix_streams(xs, mix.to(dev), write.to(dev), a.to(dev), gate.to(dev)[:, 1] if gated else None, None, read[step + 1].to(dev),
+                            put(gains[step + 1]), eps, keep=keep)
+        if keep:
+            assert error(xs, want.transpose(0, 1)) < 1e-6
+        assert x.dtype == dt and error(x, oracle.rms(oracle.streams_in(want, read[step + 1].double()), gains[step + 1].double(), eps)) < tol(target, 2e-6, 4e-3)
+
+
+# --------------------------------------------------------------------------- rotation
+@pytest.mark.parametrize("rot", [(64, 1e4, dict(factor=4.0, original=4096.0, fast=32.0, slow=1.0)), (16, 1e6, dict(factor=2.5, original=300.0, fast=9.0, slow=2.0)),
+                                 (2, 100.0, dict(factor=5.0, original=64.0, fast=0.2, slow=0.1)), (24, 50.0, SCALING), (12, 300.0, None),
+                                 (8, 10.0, dict(factor=2.0, original=40.0, fast=3.0, slow=3.0)), (0, 10.0, None)], ids=str)
+def test_rotation_frequencies(rot):
+    dims, base, scaling = rot
+    freq, gain = yarn_frequencies(dims, base, **(scaling or {}))
+    want, want_gain = oracle.ramp_frequencies(dims, base, scaling)
+    assert gain == pytest.approx(want_gain, rel=1e-12) and torch.allclose(freq, torch.tensor(want, dtype=torch.float64), rtol=1e-12)
+
+
+@pytest.mark.parametrize("shape", [(3, 2, 20, 12, 28), (4, 1, 64, 64, 64), (2, 2, 17, 6, 34), (8, 2, 128, 96, 128), (5, 1, 24, 0, 40), (2, 1, 640, 64, 512),
+                                   (3, 1, 200, 200, 72), (1, 1, 2, 2, 2)], ids=str)
+def test_turned_and_normed_into_the_cache(target, shape):
+    """Positions into the thousands: the angle keeps its digits.  The norm counts the dimensions that are not turned and the factor of cosine and sine."""
+    dev, dt = target
+    H, G, D, rot, E = shape
+    g = torch.Generator().manual_seed(D)
+    freq, gain = oracle.ramp_frequencies(rot, 900.0, None if rot == 0 else dict(factor=3.0, original=90.0, fast=6.0, slow=0.5))
+    vfreq = [900.0 ** (-2.0 * m / E) for m in range(E // 2)]
+    n, start, ld, eps = 10, 5000, (H + G) * D + G * E, 0.05
+    y, temp = rand(g, n, ld + (-ld % 8) + 8), torch.randn(H, generator=g)
+    pool = Paged(64, 160, device=dev)
+    pool.step({0: start})
+    meta = pool.step({0: n})
+    kc, vc = torch.zeros(160, 64, G, D, dtype=dt, device=dev), torch.zeros(160, 64, G, E, dtype=dt, device=dev)
+    rows = y.clone().to(dev, dt)
+    q, k, v = rows[:, :H * D], rows[:, H * D:(H + G) * D], rows[:, (H + G) * D:ld]
+    table = lambda f, s: ops.turn_table(meta.positions, torch.tensor(f, dtype=torch.float64, device=dev), s) if f else None  # noqa: E731
+    ops.turn_norm_append(q, k, v, H, G, D, table(freq, gain), table(vfreq, 1.0), temp.to(dev), meta, kc, vc, eps)
+
+    turned = lambda x, heads, f, s=1.0: oracle.rotate_pairs(x.double().view(n, heads, -1), f, s, start=start)  # noqa: E731
+    slots = meta.slot_mapping.long().cpu()
+    want_q = oracle.rms(turned(y[:, :H * D], H, freq, gain), 1.0, eps) * temp.double()[:, None]
+    assert error(q, want_q.reshape(n, -1)) < tol(target, 2e-6, 3e-3)
+    assert error(kc.view(-1, G, D).cpu()[slots], oracle.rms(turned(y[:, H * D:(H + G) * D], G, freq, gain), 1.0, eps)) < tol(target, 2e-6, 3e-3)
+    assert error(vc.view(-1, G, E).cpu()[slots], turned(y[:, (H + G) * D:ld], G, vfreq)) < tol(target, 2e-6, 3e-3)
+    assert torch.equal(rows[:, ld:].cpu().float(), y[:, ld:]) and float(kc.float().abs().sum(-1).gt(0).sum()) == n * G
+
+
+# --------------------------------------------------------------------------- attention
+def unit(g, n, heads, d):
+    """Rows as the cache holds them: unit root mean square."""
+    x = torch.randn(n, heads, d, generator=g)
+    return bf16(x / x.pow(2).mean(-1, keepdim=True).sqrt())
+
+
+HEADS = [(6, 2, 64, 64), (4, 4, 32, 48), (8, 1, 128, 128), (12, 2, 96, 40), (2, 2, 256, 256), (20, 1, 16, 24), (3, 1, 17, 34), (16, 2, 128, 128), (10, 1, 64, 64),
+         (8, 2, 256, 256), (4, 2, 128, 64), (6, 2, 64, 32), (4, 1, 192, 128), (2, 1, 20, 2)]
+
+
+@pytest.mark.parametrize("heads", HEADS, ids=str)
+@pytest.mark.parametrize("page, scale, cap", [(16, 1.0, 40.0), (64, 4.0, 5.0), (64, 0.5, 30.0), (64, 8.0, 20.0)])
+def test_attention_with_cap_and_turned_result(target, heads, page, scale, cap):
+    """Scores well inside the cap, around it and far beyond it, in prompts, portions and decoding; the result turned back by the query's own position."""
+    dev, dt = target
+    H, G, D, E = heads
+    g = torch.Generator().manual_seed(H * D + E)
+    lengths = {0: 150, 1: 1, 2: 77}
+    q, k, v = ({s: unit(g, n, hh, d) for s, n in lengths.items()} for hh, d in ((H, D), (G, D), (G, E)))
+    scale *= D ** -0.5
+    freq = [50.0 ** (-2.0 * m / E) for m in range(E // 2)]
+    ones = torch.ones(H, dtype=torch.float64)
+    want = {s: oracle.rotate_pairs(oracle.attend(q[s].double(), k[s].double(), v[s].double(), scale, ones, cap), freq, sign=-1.0).reshape(n, H * E)
+            for s, n in lengths.items()}
+    pool = Paged(page, device=dev)
+    kc, vc = torch.zeros(96, page, G, D, dtype=dt, device=dev), torch.zeros(96, page, G, E, dtype=dt, device=dev)
+    sink, freq = torch.zeros(H, device=dev), torch.tensor(freq, dtype=torch.float64, device=dev)
+    for step in schedule(lengths, random.Random(1)):
+        meta = pool.step({s: n for s, (_, n) in step.items()})
+        take = lambda x: torch.cat([x[s][a:a + n] for s, (a, n) in step.items()]).to(dev, dt)  # noqa: E731
+        ops.ref.kv_append(take(k), take(v), kc, vc, meta.slot_mapping)
+        rows = torch.cat([take(q).flatten(1), take(q).flatten(1)[:, :8]], 1)               # a pitch wider than the queries
+        rows = torch.cat([rows, torch.zeros_like(rows[:, :-rows.shape[1] % 8])], 1)
+        out = ops.rows_buffer(rows.shape[0], H * E + 24, rows)
+        out.fill_(7.0)
+        form = ops.AttentionForm(cap=cap, sink=sink, turn=ops.turn_table(meta.positions, freq))
+        ops.attention_exact(rows[:, :H * D].unflatten(1, (H, D)), kc, vc, meta, scale, out=out[:, :H * E], form=form)
+        assert error(out[:, :H * E], torch.cat([want[s][a:a + n] for s, (a, n) in step.items()])) < tol(target, 2e-5, 5e-3)
+        assert bool((out[:, H * E:] == 7.0).all())
+
+
+@pytest.mark.parametrize("heads", [(4, 2, 64, 64), (8, 1, 128, 128), (4, 1, 40, 24), (4, 2, 128, 64)], ids=str)
+@pytest.mark.parametrize("decoded", [False, True])
+def test_a_far_key_and_the_sink_stand_out(target, heads, decoded):
+    """Among hundreds of keys one far back wins by its score alone: at the first position, at page borders, within a page and the query's own.  Where every
+    score is far below zero, the sink takes the weight and the result is small."""
+    dev, dt = target
+    H, G, D, E = heads
+    page, T = 64, 450
+    g = torch.Generator().manual_seed(3)
+    v = rand(g, T, G, E)
+    freq = torch.tensor([30.0 ** (-2.0 * m / E) for m in range(E // 2)], dtype=torch.float64)
+    for j in (0, 1, 63, 64, 127, 384, T - 1, 300, None):
+        k, q = bf16(0.05 * torch.randn(T, G, D, generator=g)), bf16(0.05 * torch.randn(T, H, D, generator=g))
+        if j is None:                                            # every key points away from the last query
+            k += 1.0
+            q[T - 1] = -6.0 / D
+        else:
+            k[j] = rand(g, G, D)
+            q[T - 1] = bf16(2.0 * k[j].repeat_interleave(H // G, 0))
+        s = torch.einsum("hd,khd->hk", q[T - 1].double(), k.double().repeat_interleave(H // G, 1)) * 2.0
+        s = oracle.soft_cap(s, 14.0)
+        p = torch.softmax(torch.cat([s, torch.zeros(H, 1, dtype=torch.float64)], 1), -1)[:, :T]
+        assert (p.sum(1) < 0.2).all() if j is None else (p[:, j] > 0.98).all()
+        o = torch.einsum("hk,khd->hd", p, v.double().repeat_interleave(H // G, 1))
+        want = oracle.rotate_pairs(o[None], freq.tolist(), sign=-1.0, start=T - 1)[0]
+        kc, vc = (torch.full((16, page, G, d), 0.25, dtype=dt, device=dev) for d in (D, E))
+        pool = Paged(page, 16, device=dev, seed=j or 0)
+        at = 0
+        for n in ([T - 1, 1] if decoded else [T]):
+            meta = pool.step({0: n})
+            ops.ref.kv_append(k[at:at + n].to(dev, dt), v[at:at + n].to(dev, dt), kc, vc, meta.slot_mapping)
+            at += n
+        form = ops.AttentionForm(cap=14.0, sink=torch.zeros(H, device=dev), turn=ops.turn_table(meta.positions, freq.to(dev)))
+        out = ops.attention_exact(q[T - n:].to(dev, dt), kc, vc, meta, 2.0, form=form).view(-1, H, E)[-1]
+        assert (out.double().cpu() - want).abs().max() < tol(target, 1e-5, 2e-2), j
+
+
+# --------------------------------------------------------------------------- lightning attention
+@pytest.mark.parametrize("shape", [(3, 20, 28), (2, 64, 64), (4, 128, 128), (1, 13, 9), (2, 200, 40), (2, 256, 64), (5, 8, 8), (2, 96, 24)], ids=str)
+@pytest.mark.parametrize("cut", ["whole", "portions", "ones"])
+def test_lightning_attention(target, shape, cut):
+    """Decays of 0, close to 1 and 1; sequences of unequal lengths and portions across chunks of 64; slots that others used before; a norm over all heads."""
+    dev, dt = target
+    H, D, E = shape
+    g = torch.Generator().manual_seed(H * D + E)
+    decay = [0.9, 1.0, 0.999, 0.0, 0.3][:H]
+    lengths = {0: 200, 1: 1, 2: 67} if cut != "ones" else {0: 40, 1: 1, 2: 25}
+    eps, C = 1e-3, H * E
+    x = {s: rand(g, n, 2 * H * D + 2 * C) for s, n in lengths.items()}                  # v, k, q (already activated), g
+    gain = rand(g, C)
+    want = {}
+    for s, n in lengths.items():
+        v, k, q, z = x[s].double().split([C, H * D, H * D, C], 1)
+        o = oracle.decayed_sums(q.view(n, H, D), k.view(n, H, D), v.view(n, H, E), decay).reshape(n, C)
+        want[s] = oracle.rms(o, gain.double(), eps) * oracle.sigmoid(z)
+    pool = Paged(64, device=dev, slots=4)
+    state = torch.full((4, *state_shape(H, D, E)), 3.0, device=dev)
+    decays = HeadDecays(decay, D, dev)
+    steps = {"whole": [{s: (0, n) for s, n in lengths.items()}], "portions": schedule(lengths, random.Random(4), (1, 2, 3, 17, 63, 64, 65, 70)),
+             "ones": schedule(lengths, random.Random(5), (1,))}[cut]
+    pad = lambda n: (n + 7) // 8 * 8  # noqa: E731
+    for step in steps:
+        meta = pool.step({s: n for s, (_, n) in step.items()})
+        rows = torch.cat([x[s][a:a + n] for s, (a, n) in step.items()])
+        y = torch.zeros(rows.shape[0], pad(C) + 2 * pad(H * D) + pad(C), dtype=dt, device=dev)
+        parts, at = [], 0
+        for piece in rows.split([C, H * D, H * D, C], 1):
+            parts.append(y[:, at:at + piece.shape[1]])
+            parts[-1].copy_(piece)
+            at += pad(piece.shape[1])
+        out = ops.rows_buffer(rows.shape[0], C + 24, y)
+        out.fill_(7.0)
+        v, k, q, z = parts
+        ops.lightning_attention(y, q, k, v, z, decays, gain.to(dev, dt), state, meta, H, D, E, eps, out[:, :C])
+        assert error(out[:, :C], torch.cat([want[s][a:a + n] for s, (a, n) in step.items()])) < tol(target, 2e-5, 8e-3)
+        assert bool((out[:, C:] == 7.0).all())
+
+
+def test_a_write_far_back_is_still_in_the_state(target):
+    """One key of hundreds meets the last query; what it wrote has decayed exactly as often as there were tokens since, over chunks and portions."""
+    dev, dt = target
+    H, D, E, T = 2, 64, 64, 400
+    for j in (0, 63, 64, 65, 127, 300, T - 1):
+        for sizes in ([T], [T - 1, 1], [65, 200, T - 265], [1] * 3 + [T - 3]):
+            y = torch.zeros(T, 2 * H * D + 2 * H * E)
+            v, k, q, z = y.split([H * E, H * D, H * D, H * E], 1)
+            v.copy_(rand(torch.Generator().manual_seed(j), T, H * E))
+            k[j], q[T - 1], z[:] = 1.0, 1.0, 50.0
+            decay, gain = (0.98, 0.995), torch.ones(H * E)
+            o = torch.cat([D * decay[h] ** (T - 1 - j) * v[j, h * E:(h + 1) * E].double() for h in range(H)])
+            want = oracle.rms(o, 1.0, 1e-6)
+            pool, state, at = Paged(64, device=dev), torch.full((6, *state_shape(H, D, E)), 3.0, device=dev), 0
+            for n in sizes:
+                meta = pool.step({0: n})
+                yy = y[at:at + n].to(dev, dt)
+                vv, kk, qq, zz = yy.split([H * E, H * D, H * D, H * E], 1)
+                out = torch.empty(n, H * E, dtype=dt, device=dev)
+                ops.lightning_attention(yy, qq, kk, vv, zz, HeadDecays(decay, D, dev), gain.to(dev, dt), state, meta, H, D, E, 1e-6, out)
+                at += n
+            assert error(out[-1], want) < tol(target, 2e-4, 5e-3), (j, sizes)
+
+
+# --------------------------------------------------------------------------- feed-forward
+@pytest.mark.parametrize("shape", [(64, 24), (72, 13), (50, 16), (256, 520), (1024, 96), (4096, 64)], ids=str)
+@pytest.mark.parametrize("T", [1, 5, 130, 300])
+@pytest.mark.parametrize("act", ["gelu", "silu"])
+def test_products_with_an_activation(target, shape, T, act):
+    """Matrix-vector products, weights as the row operand, split sums and prompts; large arguments of both signs; only the first columns activated."""
+    dev, dt = target
+    W, F = shape
+    g = torch.Generator().manual_seed(W + T)
+    x, w = rand(g, T, W), bf16(4.0 * torch.randn(F, W, generator=g) * W ** -0.5)
+    f = {"gelu": oracle.gelu, "silu": oracle.silu}[act]
+    z = x.double() @ w.double().T
+    for cols in (None, F // 3, 0):
+        n = F if cols is None else cols
+        y = ops.linear_act(x.to(dev, dt), w.to(dev, dt), act, cols)
+        assert y.dtype == dt and error(y, torch.cat([f(z[:, :n]), z[:, n:]], 1)) < tol(target, 1e-5, 8e-3)
+
+
+def test_soft_cap(target):
+    dev, _ = target
+    x = torch.cat([torch.linspace(-200.0, 200.0, 999), torch.tensor([0.0, 1e-6, -1e-6])])
+    y = ops.soft_cap(x.clone().to(dev)[None], 7.0)[0]
+    assert torch.allclose(y.double().cpu(), oracle.soft_cap(x.double(), 7.0), rtol=2e-6, atol=1e-12)
+
+
+@pytest.mark.parametrize("router", [(5, 3), (1, 1), (7, 7), (16, 2), (12, 6), (40, 4)], ids=str)
+@pytest.mark.parametrize("size", [(64, 24, 40), (72, 13, 0), (50, 16, 9), (256, 64, 128)], ids=str)
+@pytest.mark.parametrize("T", [1, 3, 40, 700])
+def test_experts_and_the_gated_shared_one(target, router, size, T):
+    """From one token to hundreds per expert; weights are the softmax over the chosen only; the shared expert's gate is one number per token."""
+    dev, dt = target
+    (E, top), (W, F, FS) = router, size
+    g = torch.Generator().manual_seed(T + W)
+    w = {"router": rand(g, E, W)}
+    for n, f in [(f"e{e}", F) for e in range(E)] + ([("shared", FS)] if FS else []):
+        w.update({f"{n}.gate": bf16(torch.randn(f, W, generator=g) * W ** -0.5), f"{n}.up": bf16(torch.randn(f, W, generator=g) * W ** -0.5),
+                  f"{n}.down": bf16(torch.randn(W, f, generator=g) * f ** -0.5)})
+    if FS:
+        w["shared.sg"] = bf16(2.0 * torch.randn(1, W, generator=g) * W ** -0.5)
+    wd = {k: v.double() for k, v in w.items()}
+    c = {"kind": "moe", "router": {"experts": E, "top": top}, "expert": {"limit": 0.8}, "shared": {"limit": 0.5} if FS else None}
+    x = bf16(0.3 * torch.randn(4 * T, W, generator=g))
+    if E > top:                                      # tokens without a close call between the last chosen and the next
+        s = (x @ w["router"].T).sort(-1, descending=True).values
+        x = x[(s[:, top - 1] - s[:, top]).sort(descending=True).indices]
+    x = x[:T]
+    want = oracle.feed_forward(x.double(), c, wd, "")
+    m = SharedRoutedExperts(W, E, F, top, "clamped", 0.8, FS, 0.5, dt, dev)
+    m.load(lambda n: w[n], "")
+    xs, one = torch.ones(T, 1, W, device=dev), torch.ones(1, device=dev)
+    gain = torch.ones(W, dtype=dt, device=dev)
+    y = ops.mix_streams(xs, torch.zeros(1, 1, device=dev), one, *m(x.to(dev, dt)), one, gain, 1e-5)
+    assert error(xs[:, 0], want) < tol(target, 2e-5, 1.2e-2)
+    assert error(y, oracle.rms(xs[:, 0].double().cpu(), 1.0, 1e-5)) < tol(target, 1e-6, 4e-3)
+
+
+# --------------------------------------------------------------------------- the model through the engine
+def engine(name, target, tokens=1024, seqs=4, seed=0, **kw):
+    cfg = CONFIGS[name] if isinstance(name, str) else name
+    w = random_weights(cfg, seed)
+    m = build(cfg, w, *target)
+    return cfg, w, make_engine(m, FAMILY, tokens, seqs, target[0], **kw)
+
+
+def close(target, got, want, f32=2e-4, b16=6e-2):
+    """Rows agree.  With 16-bit activations a token now and then falls on the other side of a close call between two experts (few of them, and a
+    different expert is not a different text); in 32 bits none does."""
+    d = (got.double().cpu() - want.double()).pow(2).mean(-1).sqrt() / want.double().pow(2).mean().sqrt()
+    if target[1] == torch.float32:
+        assert float(d.max()) < f32
+    else:
+        assert float((d > b16).double().mean()) <= 0.25 and float(d.median()) < b16 / 2 and float(d.max()) < 0.8
+
+
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_whole_prompt_and_layers(target, name):
+    cfg, w, eng = engine(name, target)
+    ids = prompt(cfg, 140)
+    logits, streams = oracle.run(cfg, w, ids)
+    s = eng.open_sequence()
+    close(target, eng.feed([(s, ids, range(len(ids)))]), logits)
+    eng.close_sequence(s)
+    s = eng.open_sequence()
+    eng.cache.alloc.extend(s, len(ids))
+    table, lens = eng.cache.alloc.page_table([s])
+    meta = BatchMeta.build([len(ids)], lens, table, eng.cache.page_size, target[0], eng.cache.alloc.slots([s]))
+    with torch.no_grad():
+        states = eng.model.layer_states(torch.tensor(ids, dtype=torch.int32, device=target[0]), meta, eng.cache)
+    assert len(states) == len(streams) == len(eng.model.runs)
+    for i in range(len(states)):
+        close(target, states[i], streams[i], 1e-4)
+
+
+@pytest.mark.parametrize("name", list(CONFIGS))
+@pytest.mark.parametrize("cut", ["ones", "twos", "changing"])
+def test_portions_and_decoding(target, name, cut):
+    cfg, w, eng = engine(name, target)
+    ids = prompt(cfg, 140, 3)
+    logits, _ = oracle.run(cfg, w, ids)
+    sizes = {"ones": [1] * 140, "twos": [2] * 70, "changing": [63, 1, 1, 2, 30, 3, 17, 9, 8, 1, 1, 1, 3]}[cut]
+    s, at, got = eng.open_sequence(), 0, []
+    for n in sizes:
+        got.append(eng.feed([(s, ids[at:at + n], range(n))]))
+        at += n
+    assert at == 140
+    close(target, torch.cat(got), logits)
+
+
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_mixed_batches_pages_and_slots_reused(target, name):
+    """More requests than slots and more tokens than the pool over time: portions of some beside single tokens of others; every logit
+    equals the request's own, whatever ran beside it and whoever used its pages and slot before."""
+    cfg, w, eng = engine(name, target, tokens=512, seqs=3)
+    rng = random.Random(7)
+    todo = [prompt(cfg, n, n) for n in (150, 3, 64, 65, 100, 128, 1, 70, 90)]
+    want = [oracle.run(cfg, w, p)[0] for p in todo]
+    queue, live, got = list(range(len(todo))), {}, {i: [] for i in range(len(todo))}
+    while queue or live:
+        while queue and len(live) < 3 and sum(-(-len(todo[i]) // 64) for i in [*live, queue[0]]) <= 8:
+            live[queue.pop(0)] = [eng.open_sequence(), 0]
+        step = [i for i in live if rng.random() < 0.75] or list(live)[:1]
+        entries = []
+        for i in step:
+            n = min(rng.choice((1, 1, 1, 2, 9, 33, 64)), len(todo[i]) - live[i][1])
+            entries.append((live[i][0], todo[i][live[i][1]:live[i][1] + n], range(n)))
+        out = eng.feed(entries)
+        k = 0
+        for i, (_, t, _) in zip(step, entries):
+            got[i].append(out[k:k + len(t)])
+            k += len(t)
+            live[i][1] += len(t)
+        for i in step:
+            if live[i][1] == len(todo[i]):
+                eng.close_sequence(live.pop(i)[0])
+    close(target, torch.cat([torch.cat(got[i]) for i in range(len(todo))]), torch.cat(want))
+    assert eng.cache.alloc.free_pages == 8
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dt", [torch.float32, torch.bfloat16], ids=str)
+def test_long_prompts(dt):
+    """Prompts of more than a thousand tokens, whole and in long portions, time after time over the same pages and slots."""
+    target = ("cuda", dt)
+    layers = [lightning((0.999, 0.9), 64, 64, moe(4, 2, 64, 1.0, (64, 1.0))), attention(4, 2, 64, 64, 32, 0.2, 6.0, 1e4, dict(factor=4.0, original=300.0, fast=30.0, slow=1.0))]
+    cfg, w, eng = engine(config(layers, vocab=64, width=128, loop=(0, 2, 2)), target, tokens=6400)
+    ids = prompt(cfg, 1100, 2)
+    logits, _ = oracle.run(cfg, w, ids)
+    for sizes in ([1100], [800, 300], [1100], [833, 1, 266]):
+        s, at, got = eng.open_sequence(), 0, []
+        for n in sizes:
+            got.append(eng.feed([(s, ids[at:at + n], range(n))]))
+            at += n
+        close(target, torch.cat(got), logits)
+        eng.close_sequence(s)
+
+
+def test_long_decoding(target):
+    cfg = config([attention(4, 2, 64, 64, 32, 0.2, 6.0, mlp=moe(3, 2)), lightning((0.99, 0.5), 64, 24, mlp=None)], vocab=97, width=64, loop=(0, 1, 2))
+    cfg, w, eng = engine(cfg, target)
+    n = 400 if target[0] == "cuda" else 150
+    ids = prompt(cfg, n, 1)
+    logits, _ = oracle.run(cfg, w, ids)
+    s = eng.open_sequence()
+    got = [eng.feed([(s, ids[:5], [4])])] + [eng.feed([(s, [t], [0])]) for t in ids[5:]]
+    close(target, torch.cat(got), logits[4:])
+
+
+def greedy_of(target, logits, ids):
+    """How far the chosen tokens' logits lie below the best ones: nothing but rounding (16 bits: a close call of a router now and then)."""
+    at = logits[torch.arange(len(ids)), torch.tensor(ids)]
+    gap = logits.max(-1).values - at
+    if target[1] == torch.float32:
+        assert float(gap.max()) <= 2e-3
+    else:
+        assert float((gap > 0.25).double().mean()) <= 0.25
+
+
+@pytest.mark.parametrize("name", ["mixed", "tensor", "plain"])
+def test_greedy_generation_through_the_scheduler(target, name):
+    """Prompts of unequal lengths, more of them than are served together, chunked prefill: every generated token is the oracle's arg-max of
+    the text before it (within rounding where two logits are as good as equal)."""
+    cfg, w, eng = engine(name, target, tokens=768, seqs=3, prefill_chunk=50)
+    prompts = [prompt(cfg, n, n) for n in (5, 120, 1, 64, 33)]
+    outs = eng.generate(prompts, 12)
+    for p, o in zip(prompts, outs):
+        assert len(o) == 12
+        greedy_of(target, oracle.run(cfg, w, p + o)[0][len(p) - 1:len(p) + 11], o)
+    assert eng.cache.alloc.free_pages == 12
+
+
+@pytest.mark.parametrize("graph", [False, True])
+@pytest.mark.parametrize("name", ["mixed", "tensor"])
+def test_fixed_batch_decoder(target, graph, name):
+    from mary_b200.runtime.spec_decode import SpecDecoder
+    cfg, w, eng = engine(name, target)
+    m = eng.model
+    cache = PagedKVCache.for_model(m, num_pages=9, page_size=64, device=target[0], num_slots=3)
+    dec = SpecDecoder(m, cache, 3, max_len=192, device=target[0], use_graph=graph)
+    prompts = [prompt(cfg, 70, i) for i in range(3)]
+    toks = [[int(t)] for t in dec.prefill(prompts, chunk=48)]
+    dec.capture()
+    for _ in range(10):
+        dec.step()
+        for b, t in enumerate(dec.emitted[:, 0].tolist()):
+            toks[b].append(t)
+    for p, o in zip(prompts, toks):
+        greedy_of(target, oracle.run(cfg, w, p + o)[0][69:80], o)
+
+
+def test_gain_of_the_scaled_rotation():
+    """Both cosine and sine grow with the logarithm of the factor, so it is seen where only part of a head is turned."""
+    _, gain = oracle.ramp_frequencies(8, 100.0, SCALING)
+    assert gain == pytest.approx(0.1 * math.log(3.0) + 1.0)
+    x = torch.ones(1, 1, 12, dtype=torch.float64)
+    y = oracle.rms(oracle.rotate_pairs(x, [1.0] * 4, gain), 1.0, 0.0)[0, 0]
+    assert float(y[0] / y[11]) == pytest.approx(gain) and dense(3)["ff"] == 3
