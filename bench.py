@@ -125,8 +125,8 @@ def main():
                          "of this package's kernels); both: the product arm, then the library arm on the same GPUs, and vs_baseline = ours / library")
     ap.add_argument("--library-steps", type=int, default=4, help="timed steps of the library arm (after 2 warm-up steps)")
     ap.add_argument("--library-limit", type=float, default=240.0, help="seconds after which a stalled library arm is abandoned")
-    ap.add_argument("--model", default="k3", choices=["k3", "inkling", "gemma12b", "tiny", "tatizen", "rokarax", "nipurax"],
-                    help="k3 is the headline; the others time the remaining workload configurations with the same harness; tatizen, rokarax, nipurax: prefill "
+    ap.add_argument("--model", default="k3", choices=["k3", "inkling", "gemma12b", "tiny", "tatizen", "rokarax", "nipurax", "kivezen"],
+                    help="k3 is the headline; the others time the remaining workload configurations with the same harness; tatizen, rokarax, nipurax, kivezen: prefill "
                          "and decode of that decoder beside the closest one of equal size, at two sizes, on one GPU")
     ap.add_argument("--ep", default="auto", choices=["auto", "replicated", "a2a"],
                     help="expert parallel layout for N > 1: replicated tokens + tensor-parallel attention + reduction, or home-rank "
@@ -158,7 +158,7 @@ def main():
     if args.impl == "reference":
         return reference_arm(args)
     W = max(args.warmup, 3)
-    if args.model in ("tatizen", "rokarax", "nipurax"):
+    if args.model in ("tatizen", "rokarax", "nipurax", "kivezen"):
         return hybrid_bench(args, W)
     # a benchmark that stops making progress must end by itself: dump the stacks and exit after the limit
     import faulthandler

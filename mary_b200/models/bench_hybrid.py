@@ -1,5 +1,5 @@
 """Throughput of the decoders with a 32-bit residual stream beside the closest decoder of equal size, prefill and decode, on one GPU: Tatizen and
-Rokarax beside the dense decoder (the Mistral shell), Nipurax beside the decoder with routed bf16 experts next to a dense feed-forward (the
+Rokarax beside the dense decoder (the Mistral shell), Nipurax and Kivezen beside the decoder with routed bf16 experts next to a dense feed-forward (the
 Gemma shell).
 
 Random weights of the named sizes; every step streams weights and caches far larger than L2.  Prefill: whole prompts through
@@ -24,6 +24,8 @@ LAYERS, VOCAB, WINDOW = 8, 32768, 1024
 # run twice, so that eight layer runs stand beside the other decoder's eight layers
 EXPERTS = {"2k": (32, 4, 1024, 2048), "4k": (32, 4, 1536, 4096)}
 IDENTITY, CHUNK = 4, 2048
+# Kivezen: the same experts, attention and linear attention in turn, four residual streams, the same loop
+STREAMS, BESIDE_ROUTED = 4, ("nipurax", "kivezen")
 CASES = [("prefill", 1, 4096), ("prefill", 8, 512), ("decode", 1, 2048), ("decode", 32, 2048), ("decode", 128, 2048)]
 
 
@@ -59,6 +61,15 @@ def nipurax_config(size: str):
     return NipuraxConfig(VOCAB, W, 1e-5, 0.25, PairsSpec(65521, 36313, 27191), LoopSpec(2, 4, 2), [cap, dif] * 3, name=f"nipurax-{size}")
 
 
+def kivezen_config(size: str):
+    from .kivezen.config import AttentionSpec, ExpertsSpec, GLUSpec, KivezenConfig, LayerSpec, LightningSpec, LoopSpec, RotationSpec
+    (W, _, (H, G), _, _), (E, top, F, FS) = SIZES[size], EXPERTS[size]
+    moe = ExpertsSpec(E, top, GLUSpec(F, 7.0), GLUSpec(FS, 7.0))
+    att = LayerSpec(AttentionSpec(H, G, 128, 128, 128 ** -0.5, 30.0, RotationSpec(128, 1e5, 4.0, 4096.0, 32.0, 1.0)), moe)
+    lin = LayerSpec(LightningSpec(H, 128, 128, [2.0 ** (-8.0 * (h + 1) / H / 2 ** (h % 3)) for h in range(H)]), moe)
+    return KivezenConfig(VOCAB, W, 1e-5, 30.0, STREAMS, LoopSpec(2, 4, 2), [lin, att] * 3, name=f"kivezen-{size}")
+
+
 def routed_config(size: str):
     from .gemma4.config import Gemma4TextConfig
     (W, _, (H, G), _, _), (E, top, F, FS) = SIZES[size], EXPERTS[size]
@@ -78,6 +89,9 @@ def make_model(kind: str, size: str, dev):
     elif kind == "nipurax":
         from .nipurax.model import NipuraxModel, init_random_
         m = NipuraxModel(nipurax_config(size), **kw)
+    elif kind == "kivezen":
+        from .kivezen.model import KivezenModel, init_random_
+        m = KivezenModel(kivezen_config(size), **kw)
     elif kind == "routed":
         from .gemma4.model import Gemma4Model
         from .gemma4.weights import init_random_
@@ -137,10 +151,10 @@ def decode_step(m, cache, batch: int, ctx: int, tokens: int, dev):
 
 def run(design: str, sizes, cases, steps: int, warmup: int, trace: bool = False) -> dict:
     from ..ops import cuda as K
-    dev = torch.device("cuda", 0)
+    dev, beside = torch.device("cuda", 0), "routed" if design in BESIDE_ROUTED else "dense"
     out = []
     for size in sizes:
-        for kind in (design, "routed" if design == "nipurax" else "dense"):
+        for kind in (design, beside):
             m = make_model(kind, size, dev)
             for what, batch, n in cases:
                 # dependent launch: a decode step is a chain of short kernels and gains from it; a prefill step loses (the waiting blocks of
@@ -173,5 +187,5 @@ def run(design: str, sizes, cases, steps: int, warmup: int, trace: bool = False)
     status = K.last_status()
     if status:
         raise RuntimeError(f"kernel status {status}")
-    return {"metric": f"tokens/s, {design} beside the {'routed' if design == 'nipurax' else 'dense'} decoder of equal size", "unit": "tokens/s", "layers": LAYERS, "dtype": "bf16",
+    return {"metric": f"tokens/s, {design} beside the {beside} decoder of equal size", "unit": "tokens/s", "layers": LAYERS, "dtype": "bf16",
             "data": "synthetic", "steps": steps, "warmup": max(warmup, 3), "cases": out}

@@ -1,5 +1,5 @@
 """Micro-benchmarks of the kernels of decoders with recurrent layers, beside the like kernels of the dense decoders
-(``python -m mary_b200.ops.bench_kernels hybrid``, ``rokarax`` and ``nipurax``).  Fractions: bytes against the measured copy bandwidth, tensor-core products against
+(``python -m mary_b200.ops.bench_kernels hybrid``, ``rokarax``, ``nipurax`` and ``kivezen``).  Fractions: bytes against the measured copy bandwidth, tensor-core products against
 the measured cuBLAS rate, the recurrences (32-bit multiply-adds on the CUDA cores) against the nominal 128 multiply-adds per SM and clock."""
 from __future__ import annotations
 
@@ -296,6 +296,120 @@ def run_nipurax(width: int = 2048, heads: int = 16, kv_heads: int = 4, experts: 
         add("qk_norm_rope_append", case, lambda: K.qk_norm_rope_append(y, heads, kv_heads, D, g, g, False, inv, m, kc, vc, 1e-5), nbytes=B * n_in * 4,
             like="routed decoder")
         add("rotate_append", case, lambda: P.rotate_append(pq, pk, pv, 2 * heads, 2 * kv_heads, 64, freq, m, kc, vc), nbytes=B * n_in * 4)
+        rows(B, case)
+    assert K.last_status() == 0
+    return add.rows
+
+
+def run_kivezen(width: int = 2048, heads: int = 16, kv_heads: int = 4, experts: int = 32, top: int = 4, ff: int = 1024, streams: int = 4) -> list[dict]:
+    """The kernels of the Kivezen decoder: attention with a cap and turned values beside the plain one, lightning attention beside the Mamba-2 chunks and
+    steps and the decayed linear attention, the mixing of the residual streams beside the row kernels of the routed decoder, products with an
+    activation beside plain ones."""
+    from ..models.mixers import HeadDecays, state_shape, yarn_frequencies
+    from . import AttentionForm
+    from . import cuda as K
+    from . import cuda_hybrid as H
+    from . import cuda_moe as M
+    from . import cuda_parallel as P
+    add = _Table()
+    tf = add.tf
+    bf = dict(dtype=torch.bfloat16, device="cuda")
+    D = 128
+    C = heads * D
+    sink = torch.zeros(heads, device="cuda")
+    freq = yarn_frequencies(D, 1e5, 4.0, 4096.0, 32.0, 1.0)[0].cuda()
+    gu, down = torch.randn(experts, 2 * ff, width, **bf) * 0.02, torch.randn(experts, width, ff, **bf) * 0.02
+    gain, row_gain = torch.ones(width, **bf), torch.ones(C, **bf)
+    read, mix = torch.ones(streams, device="cuda"), torch.eye(streams, device="cuda")
+    decays = HeadDecays([1.0 - 2.0 ** -(4 + h % 8) for h in range(heads)], D, "cuda")
+    # the like recurrence of Rokarax at the same width: heads of 64 with 128 state rows shared by all
+    SH = C // 64
+    ones = torch.ones(SH, device="cuda")
+
+    def rows(T, case):
+        x = torch.randn(T, width, **bf)
+        z = torch.randn(T, experts + 1, device="cuda")
+        idx, w = K.router_topk(z[:, :experts], top, "softmax")
+        n = T * top
+        used = min(n, experts)
+        wb, fl = used * 3.0 * ff * width * 2, 6.0 * n * ff * width
+        add("experts, decoder with GEGLU", case, lambda: M.experts_forward_bf16(x, idx, w, gu, down, "geglu"), fl, tf, wb, like="routed decoder")
+        add("experts, clamped", case, lambda: P.expert_outputs(x, idx, w, gu, down, "clamped", 7.0), fl, tf, wb)
+        r = P.expert_outputs(x, idx, w, gu, down, "clamped", 7.0)
+        a, hb, xs = torch.randn(T, width, device="cuda"), torch.randn(T, width, **bf), torch.randn(T, streams, width, device="cuda")
+        add("add_rmsnorm", case, lambda: K.add_rmsnorm(x, hb, gain, 1e-5), nbytes=T * width * 8, like="routed decoder")
+        add("norm_add_norm", case, lambda: K.norm_add_norm(a, gain, hb, gain, 1e-5), nbytes=T * width * 10, like="routed decoder")
+        add("mix_streams", case, lambda: P.mix_streams(xs, mix, read, a, None, None, read, gain, 1e-5, True), nbytes=T * width * (8.0 * streams + 6))
+        per = 4 if r.sum is not None else 2 * top
+        add("mix_streams, experts", case, lambda: P.mix_streams(xs, mix, read, a, z[:, experts], r, read, gain, 1e-5, True),
+            nbytes=T * width * (8.0 * streams + 6 + per))
+        w_up, w_in = torch.randn(4 * width, width, **bf) * 0.02, torch.randn(4 * C, width, **bf) * 0.02
+        for name, wt, fn, like in (("linear", w_up, lambda: K.linear(x, w_up), "both decoders"), ("linear, gelu", w_up, lambda: K.linear_act(x, w_up, "gelu", 4 * width), None),
+                                   ("linear, silu on 3 of 4 parts", w_in, lambda: K.linear_act(x, w_in, "silu", 3 * C), None)):
+            add(name, case, fn, 2.0 * T * wt.numel(), tf, 2.0 * (wt.numel() + T * width + T * wt.shape[0]), like=like)
+
+    for B, q in ((1, 4096), (8, 512)):
+        case, T = f"{B} x {q} tokens", B * q
+        m = _meta(B, q, q)
+        n_in = (heads + 2 * kv_heads) * D
+        y = torch.randn(T, n_in, **bf)
+        pq, pk, pv = y.split([heads * D, kv_heads * D, kv_heads * D], 1)
+        kc = torch.randn(m.page_table.numel(), 64, kv_heads, D, **bf)
+        vc, out = torch.randn_like(kc), torch.empty(T, C, **bf)
+        Q = torch.randn(T, heads, D, **bf)
+        turn = P.turn_table(m.positions, freq, 1.0)
+        fl = 4.0 * heads * D * T * (q + 1) / 2
+        add("attention_prefill", case, lambda: K.attention_prefill(Q, kc, vc, m, 0.05), fl, tf, like="routed decoder")
+        add("  capped, sink", case, lambda: H.attention_exact(Q, kc, vc, m, 0.05, out=out, form=AttentionForm(cap=30.0, sink=sink)), fl, tf)
+        add("  capped, sink, turned", case, lambda: H.attention_exact(Q, kc, vc, m, 0.05, out=out, form=AttentionForm(cap=30.0, sink=sink, turn=turn)), fl, tf)
+        inv, g = torch.ones(D // 2, device="cuda"), torch.ones(D, **bf)
+        add("qk_norm_rope_append", case, lambda: K.qk_norm_rope_append(y, heads, kv_heads, D, g, g, False, inv, m, kc, vc, 1e-5), nbytes=T * n_in * 4,
+            like="routed decoder")
+        add("turn_table", case, lambda: P.turn_table(m.positions, freq, 1.0), nbytes=T * D * 4.0)
+        add("turn_norm_append", case, lambda: P.turn_norm_append(pq, pk, pv, heads, kv_heads, D, turn, turn, sink, m, kc, vc, 1e-5), nbytes=T * (n_in * 4 + D * 8.0))
+        yl = torch.randn(T, 4 * C, **bf)
+        pv, pk, pq, pg = yl.split([C] * 4, 1)
+        S = torch.zeros(B, *state_shape(heads, D, D), device="cuda")
+        fl = 2.0 * T * heads * (2 * D * D + 64 * D + 32 * D)
+        add("lightning_chunk", case, lambda: H.lightning_chunk(yl, decays, S, m, heads, D, D), fl, tf, T * C * 10.0)
+        o = H.lightning_chunk(yl, decays, S, m, heads, D, D)
+        add("norm, gate", case, lambda: H.gated_part_norm(o, pg, row_gain, 1, 1e-5, out, norm_first=True), nbytes=T * C * 8.0)
+        xbc = torch.randn(T, C + 256, **bf)
+        S2 = torch.zeros(B, *state_shape(SH, 128, 64), device="cuda")
+        hi = (-0.02 * (torch.arange(T, device="cuda") % 64 + 1.0)).expand(SH, T).contiguous()
+        dt, lo = torch.ones_like(hi), torch.zeros_like(hi)
+        add("ssd_chunk (Mamba-2)", case, lambda: H.ssd_chunk(xbc, dt, hi, lo, ones, S2, m, 1, SH, 128, 64), 2.0 * T * SH * (2 * 128 * 64 + 32 * 64) + 2.0 * T * 64 * 128, tf,
+            T * (C * 6.0 + 512), like="rokarax")
+        add("decay_scan", case, lambda: H.decay_scan(pq, pk, pv, decays.channel, S, m, heads, D, D, 1.0), 5.0 * T * C * D, F32_TFLOPS, T * C * 10.0, like="tatizen")
+        rows(T, case)
+    for B in (1, 32, 128):
+        case, ctx = f"{B} x 1 token", 2048
+        m = _meta(B, 1, ctx)
+        n_in = (heads + 2 * kv_heads) * D
+        y = torch.randn(B, n_in, **bf)
+        pq, pk, pv = y.split([heads * D, kv_heads * D, kv_heads * D], 1)
+        kc = torch.randn(m.page_table.numel(), 64, kv_heads, D, **bf)
+        vc, Q = torch.randn_like(kc), torch.randn(B, heads, D, **bf)
+        out = torch.empty(B, C, **bf)
+        turn = P.turn_table(m.positions, freq, 1.0)
+        nb = 2.0 * B * ctx * kv_heads * D * 2
+        m16, k16, v16 = _meta(B, 1, ctx, 16), kc.view(-1, 16, kv_heads, D), vc.view(-1, 16, kv_heads, D)
+        add("gqa_decode_tc", case, lambda: K.gqa_decode_tc(Q, k16, v16, m16, 0.1), nbytes=nb, like="routed decoder")
+        add("  capped, sink, turned", case, lambda: H.attention_exact(Q, kc, vc, m, 0.05, out=out, form=AttentionForm(cap=30.0, sink=sink, turn=turn)), nbytes=nb)
+        inv, g = torch.ones(D // 2, device="cuda"), torch.ones(D, **bf)
+        add("qk_norm_rope_append", case, lambda: K.qk_norm_rope_append(y, heads, kv_heads, D, g, g, False, inv, m, kc, vc, 1e-5), nbytes=B * n_in * 4,
+            like="routed decoder")
+        add("turn_table", case, lambda: P.turn_table(m.positions, freq, 1.0), nbytes=B * D * 4.0)
+        add("turn_norm_append", case, lambda: P.turn_norm_append(pq, pk, pv, heads, kv_heads, D, turn, turn, sink, m, kc, vc, 1e-5), nbytes=B * (n_in * 4 + D * 8.0))
+        yl = torch.randn(B, 4 * C, **bf)
+        pv, pk, pq, pg = yl.split([C] * 4, 1)
+        S = torch.zeros(B, *state_shape(heads, D, D), device="cuda")
+        add("lightning_step", case, lambda: H.lightning_attention(yl, pq, pk, pv, pg, decays, row_gain, S, m, heads, D, D, 1e-5, out), nbytes=B * C * D * 8.0)
+        a2, b2, hg = torch.randn(C, 16, **bf), torch.randn(C, **bf), torch.ones(D, **bf)
+        yd = torch.randn(B, 4 * C + 16, **bf)
+        dq, dk, dv, dg, low = yd.split([C, C, C, C, 16], 1)
+        add("decay_step", case, lambda: H.decayed_linear_attention(dq, dk, dv, dg, low, a2, b2, 1 / 16, hg, S, m, heads, D, D, 1e-5, 1.0, out),
+            nbytes=B * C * D * 8.0, like="tatizen")
         rows(B, case)
     assert K.last_status() == 0
     return add.rows

@@ -574,6 +574,9 @@ if __name__ == "__main__":
     if what == "nipurax":
         from .bench_hybrid import run_nipurax
         run_nipurax(*nums)
+    if what == "kivezen":
+        from .bench_hybrid import run_kivezen
+        run_kivezen(*nums)
     if what == "moeprefill":
         bench_moeprefill(*nums)
     if what == "bf16moe":

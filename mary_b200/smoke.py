@@ -103,6 +103,24 @@ def _routed_engine(dev):
     return out
 
 
+def _streams_engine(dev):
+    """A Kivezen decoder (four residual streams, lightning attention, attention with turned values, gated shared expert, a loop over two layers) generating
+    through the scheduler, two sequences."""
+    from .models.kivezen import KivezenConfig, KivezenModel, init_random_
+    from .models.registry import family_of, make_engine
+    moe = {"kind": "moe", "expert": {"ff": 256, "limit": 2.0}, "shared": {"ff": 384, "limit": 1.5}, "router": {"experts": 8, "top": 2}}
+    lin = {"type": "lightning", "mlp": {"kind": "dense", "ff": 768}, "mixer": dict(heads=4, dim=128, vdim=64, decay=[0.5, 0.9, 0.97, 0.995])}
+    att = {"type": "attention", "mlp": moe, "mixer": dict(heads=8, kv_heads=2, dim=128, vdim=128, scale=0.09, softcap=20.0, rot={
+        "dims": 96, "base": 50000.0, "scaling": dict(factor=4.0, original=1024.0, fast=32.0, slow=1.0)})}
+    d = {"architecture": "Kivezen", "vocab": 1024, "width": 512, "norm": {"eps": 1e-6}, "logit_softcap": 20.0, "streams": 4, "layers": [lin, att, lin],
+         "loop": {"start": 0, "stop": 2, "times": 2}}
+    m = KivezenModel(KivezenConfig.from_json(d), dtype=torch.bfloat16, device=dev)
+    init_random_(m, 0)
+    out = make_engine(m, family_of(d), 512, 2, dev).generate([list(range(90)), [5, 4, 3]], 4)
+    assert all(len(o) == 4 for o in out)
+    return out
+
+
 def _lora_step(m, dev):
     from .train.trainer import LoraTrainer
     tr = LoraTrainer(m, rank=8, alpha=16.0, lr=1e-3)
@@ -123,9 +141,10 @@ def run_smoke() -> None:
     rec = _recurrent_engine(dev)
     ssm = _state_space_engine(dev)
     moe = _routed_engine(dev)
+    hyper = _streams_engine(dev)
     losses = _lora_step(m, dev)
     torch.cuda.synchronize()
     st = cuda.last_status()
     assert st == 0, f"kernel status {st}"
-    print(f"smoke ok: flagship emitted {n} tokens in 4 speculative steps; gemma {out}; tatizen {rec}; rokarax {ssm}; nipurax {moe}; lora loss {losses[0]:.3f} -> {losses[1]:.3f}; "
+    print(f"smoke ok: flagship emitted {n} tokens in 4 speculative steps; gemma {out}; tatizen {rec}; rokarax {ssm}; nipurax {moe}; kivezen {hyper}; lora loss {losses[0]:.3f} -> {losses[1]:.3f}; "
           f"{cuda.LAUNCHES} kernel launches")
