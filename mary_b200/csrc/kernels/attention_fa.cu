@@ -582,6 +582,11 @@ MARY_API int mary_attention_prefill_supported(int DK, int DV) {
   return (DK == 64 && DV == 64) || (DK == 128 && DV == 128) || (DK == 192 && DV == 128) || (DK == 256 && DV == 256);
 }
 
+// The same with an attention form of one map.
+MARY_API int mary_attention_prefill_form_supported(int DK, int DV) {
+  return (DK == 64 && DV == 64) || (DK == 128 && DV == 128) || (DK == 128 && DV == 64) || (DK == 256 && DV == 256);
+}
+
 // The same for two maps of DK values each.
 MARY_API int mary_attention_prefill_maps_supported(int DK, int DV) {
   return (DK == 64 && DV == 64) || (DK == 64 && DV == 128) || (DK == 128 && DV == 128);
@@ -603,7 +608,9 @@ MARY_API int mary_attention_prefill(const void* q, const void* kcache, const voi
   if (NB > 65535) return MARY_ERR_BAD_ARG;
   const int maps = form && form->maps == 2 ? 2 : 1;
   if (form && (form->maps > 2 || !split_p || bias || (maps == 2 && (gate || form->sink || form->turn)) || (form->turn && (gate || ((uintptr_t)form->turn & 15))))) return MARY_ERR_BAD_ARG;
-  if (!(maps == 2 ? mary_attention_prefill_maps_supported(DK, DV) : mary_attention_prefill_supported(DK, DV)) || Hkv < 1 || Hq % Hkv || (page_size != PAGE && page_size != KB)) return MARY_ERR_BAD_ARG;
+  const bool formed = form && maps == 1 && (form->chunk > 0 || form->sink || form->temp_every > 0 || form->cap > 0.f || form->turn);
+  if (!(maps == 2 ? mary_attention_prefill_maps_supported(DK, DV)
+                  : formed ? mary_attention_prefill_form_supported(DK, DV) : mary_attention_prefill_supported(DK, DV)) || Hkv < 1 || Hq % Hkv || (page_size != PAGE && page_size != KB)) return MARY_ERR_BAD_ARG;
   if ((k_tok_stride * 2) % 16 || (k_page_stride * 2) % 16 || (v_tok_stride * 2) % 16 || (v_page_stride * 2) % 16) return MARY_ERR_BAD_ARG;
   CUtensorMap tq, tk, tv;
   const uint64_t q_ld = form && form->q_ld > 0 ? (uint64_t)form->q_ld : (uint64_t)Hq * maps * DK;
@@ -626,10 +633,10 @@ MARY_API int mary_attention_prefill(const void* q, const void* kcache, const voi
     if (DK == 64) return launch_fa<64, 128, true, false, 2>(tq, tk, tv, p, NB, s);
     return launch_fa<128, 128, true, false, 2>(tq, tk, tv, p, NB, s);
   }
-  if (form && (p.f.chunk > 0 || p.f.sink || p.f.temp_every > 0 || p.f.cap > 0.f || p.f.turn)) {
+  if (formed) {
+    if (DK == 128 && DV == 64) return launch_fa<128, 64, true, false, 1>(tq, tk, tv, p, NB, s);
     if (DK == 64) return launch_fa<64, 64, true, false, 1>(tq, tk, tv, p, NB, s);
     if (DK == 128) return launch_fa<128, 128, true, false, 1>(tq, tk, tv, p, NB, s);
-    if (DK == 192) return MARY_ERR_BAD_ARG;
     return launch_fa<256, 256, true, false, 1>(tq, tk, tv, p, NB, s);
   }
   if (bias) {

@@ -39,21 +39,23 @@ constexpr float RESCALE_THRESHOLD = 8.0f;
 constexpr int AHEAD = 1;                          // blocks by which Q K^T leads P V
 constexpr float LOG2E = 1.4426950408889634f;
 
-template <int D, int PAGE, int MAPS>
+template <int D, int PAGE, int MAPS, int DV>
 struct GCfg {
   static constexpr int NCH = D / CHUNK;
   static constexpr int Q_CHUNK_BYTES = TR * 128;                  // 8 KB
   static constexpr int Q_BYTES = NCH * Q_CHUNK_BYTES;
   static constexpr int PAGE_CHUNK_BYTES = PAGE * 128;             // one 64-dim chunk of one page
-  static constexpr int PAGE_BYTES = NCH * PAGE_CHUNK_BYTES;       // K (or V) page
+  static constexpr int PAGE_BYTES = NCH * PAGE_CHUNK_BYTES;       // K page
+  static constexpr int KV_BYTES = PAGE_BYTES + DV / CHUNK * PAGE_CHUNK_BYTES;      // K page and V page
   static constexpr int PPB = 32 / PAGE;                           // pages per pipeline stage: a stage always holds KB = 32 keys
   static constexpr int KB = PAGE * PPB;
-  static constexpr int STAGE_BYTES = 2 * PAGE_BYTES * PPB;        // [page of the stage][K page | V page]
+  static constexpr int STAGE_BYTES = KV_BYTES * PPB;              // [page of the stage][K page | V page]
   static constexpr int STAGES = MAPS > 0 ? 4 : 5;                 // two CTAs of D = 128 share an SM
   static constexpr int P_HALF = TR * KB * 2;                      // rounded weights; with MAPS > 0 their rounding errors behind them
   static constexpr int P_BYTES = MAPS > 0 ? 2 * P_HALF : P_HALF;
   static constexpr int SMEM = Q_BYTES + STAGES * STAGE_BYTES + NPBUF * P_BYTES + 1024 + 256;
-  static constexpr int TMEM_COLS = D <= 128 ? 256 : 512;          // S: 3 x PAGE columns at 0..95, O: D columns at 128..
+  static constexpr int TMEM_COLS = D <= 128 ? 256 : 512;          // S: 3 x PAGE columns at 0..95, O: DV columns at 128..
+  static_assert(DV % CHUNK == 0 && DV <= D && (DV == D || MAPS == 1), "value widths");
   static_assert(D % CHUNK == 0 && D <= 256 && (PAGE == 16 || PAGE == 32), "head dim 64..256 in chunks of 64, pages of 16 or 32 tokens");
   static_assert(NSBUF * KB <= 128 && SMEM <= 232448, "budget");
   static_assert(MAPS < 2 || D == 2 * CHUNK, "two maps: one 64-dim chunk each");
@@ -90,12 +92,12 @@ __device__ __forceinline__ uint64_t desc_mnmajor_sw128(uint32_t addr, uint32_t l
          (2ull << 61);
 }
 
-template <int D, int PAGE, int MAPS>
+template <int D, int PAGE, int MAPS, int DV>
 __global__ void __launch_bounds__(NTHREADS, 1)
 gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                      const GqaParams p) {
   pdl_sync();
-  using C = GCfg<D, PAGE, MAPS>;
+  using C = GCfg<D, PAGE, MAPS, DV>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
@@ -161,7 +163,7 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
   const uint32_t tmem_S = tmem_base;            // NSBUF x PAGE columns
-  const uint32_t tmem_O = tmem_base + 128;      // D columns
+  const uint32_t tmem_O = tmem_base + 128;      // DV columns
 
   if (warp == 0) {
     if (nblk > 0 && lane == 0) {
@@ -185,8 +187,8 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           } else {
             page = pt[pi < n_pages ? pi : b * PPB];               // a page past the visible keys repeats the block's first page (masked)
           }
-          tma_load_5d(st + pp * 2 * C::PAGE_BYTES, &tm_k, &k_full[stage], 0, tok, 0, kvh, page);
-          tma_load_5d(st + pp * 2 * C::PAGE_BYTES + C::PAGE_BYTES, &tm_v, &k_full[stage], 0, tok, 0, kvh, page);
+          tma_load_5d(st + pp * C::KV_BYTES, &tm_k, &k_full[stage], 0, tok, 0, kvh, page);
+          tma_load_5d(st + pp * C::KV_BYTES + C::PAGE_BYTES, &tm_v, &k_full[stage], 0, tok, 0, kvh, page);
         }
         if (++stage == C::STAGES) { stage = 0; phase ^= 1; }
       }
@@ -194,7 +196,7 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   } else if (warp == 1) {
     if (elect_one() && nblk > 0) {
       const uint32_t idesc_s = idesc_bf16(TR, PAGE);            // one page of keys per instruction
-      const uint32_t idesc_o = idesc_bf16(TR, D) | (1u << 16);           // B operand MN-major
+      const uint32_t idesc_o = idesc_bf16(TR, DV) | (1u << 16);           // B operand MN-major
       if (!mbar_wait(q_full, 0, abort_flag, p.status, MARY_ERR_TIMEOUT_TMA)) goto done;
       const uint32_t q_addr = smem_u32(sQ), p_addr = smem_u32(sP);
       auto issue_qk = [&](int i) -> bool {        // i = block index relative to b_lo
@@ -210,7 +212,7 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
 #pragma unroll
             for (int k = 0; k < 4; ++k) {
               umma_f16(tmem_S + sb * KB + pp * PAGE, umma_desc_sw128(q_addr + c * C::Q_CHUNK_BYTES + k * 32),
-                       umma_desc_sw128(kb_addr + pp * 2 * C::PAGE_BYTES + c * C::PAGE_CHUNK_BYTES + k * 32), idesc_s, (c > 0 || k > 0) ? 1u : 0u);
+                       umma_desc_sw128(kb_addr + pp * C::KV_BYTES + c * C::PAGE_CHUNK_BYTES + k * 32), idesc_s, (c > 0 || k > 0) ? 1u : 0u);
             }
           }
         }
@@ -236,11 +238,11 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           // B = V^T of those keys from their V page (MN-major, 128B swizzle: 64-dim groups one chunk apart, 8-key groups 1 KB apart)
           const int pp = kk * 16 / PAGE, in_page = kk * 16 % PAGE;
           umma_f16(tmem_O, desc_kmajor_noswz(p_addr + pb * C::P_BYTES + kk * 2 * (TR * 16), TR * 16, 128),
-                   desc_mnmajor_sw128(st_addr + pp * 2 * C::PAGE_BYTES + C::PAGE_BYTES + in_page * 128, C::PAGE_CHUNK_BYTES, 1024), idesc_o,
+                   desc_mnmajor_sw128(st_addr + pp * C::KV_BYTES + C::PAGE_BYTES + in_page * 128, C::PAGE_CHUNK_BYTES, 1024), idesc_o,
                    (i > 0 || kk > 0) ? 1u : 0u);
           if constexpr (MAPS > 0)
             umma_f16(tmem_O, desc_kmajor_noswz(p_addr + pb * C::P_BYTES + C::P_HALF + kk * 2 * (TR * 16), TR * 16, 128),
-                     desc_mnmajor_sw128(st_addr + pp * 2 * C::PAGE_BYTES + C::PAGE_BYTES + in_page * 128, C::PAGE_CHUNK_BYTES, 1024), idesc_o, 1u);
+                     desc_mnmajor_sw128(st_addr + pp * C::KV_BYTES + C::PAGE_BYTES + in_page * 128, C::PAGE_CHUNK_BYTES, 1024), idesc_o, 1u);
         }
         umma_commit(&k_empty[stage]);       // the stage may be overwritten once PV has read it
         umma_commit(&pv_done[pb]);
@@ -355,7 +357,7 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         if (!mbar_wait(&pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, abort_flag, p.status, MARY_ERR_TIMEOUT_MMA)) goto done;
         tc_fence_after();
 #pragma unroll 1
-        for (int c0 = 0; c0 < D; c0 += 32) {
+        for (int c0 = 0; c0 < DV; c0 += 32) {
           uint32_t o[32];
           tmem_ld_32x32b_x32(tmem_O + lane_off + c0, o);
           tmem_ld_wait();
@@ -397,18 +399,18 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     }
     inv_l = inv_l > 0.f ? 1.f / inv_l : 0.f;
 #pragma unroll 1
-    for (int c0 = 0; c0 < D; c0 += 32) {
+    for (int c0 = 0; c0 < DV; c0 += 32) {
       uint32_t o[32];
       tmem_ld_32x32b_x32(tmem_O + lane_off + c0, o);
       tmem_ld_wait();
       if (row_ok) {
         if (whole) {
-          __nv_bfloat16* dst = p.out + (int64_t)tq * p.out_ld + head * D + c0;
+          __nv_bfloat16* dst = p.out + (int64_t)tq * p.out_ld + head * DV + c0;
           uint4 w[4];
           uint32_t* wp = (uint32_t*)w;
           if constexpr (MAPS == 1) {
             if (p.f.turn) {
-              const float4* cs = (const float4*)(p.f.turn + ((int64_t)tq * D + c0) / 2);
+              const float4* cs = (const float4*)(p.f.turn + ((int64_t)tq * DV + c0) / 2);
 #pragma unroll
               for (int j = 0; j < 8; ++j) {
                 const float4 c = cs[j];
@@ -426,7 +428,7 @@ gqa_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
 #pragma unroll
           for (int j = 0; j < 4; ++j) ((uint4*)dst)[j] = w[j];
         } else {
-          float* dst = p.part_o + ((((int64_t)nb * p.Hkv + kvh) * p.nsplit + split) * TR + r) * D + c0;
+          float* dst = p.part_o + ((((int64_t)nb * p.Hkv + kvh) * p.nsplit + split) * TR + r) * DV + c0;
 #pragma unroll
           for (int j = 0; j < 32; j += 4) *(float4*)(dst + j) = make_float4(__uint_as_float(o[j]), __uint_as_float(o[j + 1]), __uint_as_float(o[j + 2]), __uint_as_float(o[j + 3]));
         }
@@ -477,11 +479,12 @@ __global__ void gqa_tc_combine_kernel(const GqaParams p, int D) {
   }
 }
 
-// The same with the sink (one map), or for the difference of two maps: out = rms(o0 - mix * o1) * post.  128 threads.
+// The same with the sink (one map), or for the difference of two maps: out = rms(o0 - mix * o1) * post.  D: width of the values.
+template <int D> constexpr int COMBINE_THREADS = D < 128 ? D : 128;
 template <int D, int MAPS>
-__global__ void __launch_bounds__(128) gqa_tc_combine_form_kernel(const GqaParams p) {
+__global__ void __launch_bounds__(COMBINE_THREADS<D>) gqa_tc_combine_form_kernel(const GqaParams p) {
   pdl_sync();
-  constexpr int E = D / 128;
+  constexpr int N = COMBINE_THREADS<D>, E = D / N;
   __shared__ float red[4];
   const int nb = blockIdx.x, kvh = blockIdx.y, r = blockIdx.z;
   const int seq = p.blk_seq[nb], tok0 = p.blk_q0[nb];
@@ -505,7 +508,7 @@ __global__ void __launch_bounds__(128) gqa_tc_combine_form_kernel(const GqaParam
       const float c = exp2f(ms - mm);
       ll = fmaf(p.part_ml[pi * 2 + 1], c, ll);
 #pragma unroll
-      for (int e = 0; e < E; ++e) acc[e] = fmaf(p.part_o[pi * D + threadIdx.x + 128 * e], c, acc[e]);
+      for (int e = 0; e < E; ++e) acc[e] = fmaf(p.part_o[pi * D + threadIdx.x + N * e], c, acc[e]);
     }
     float norm = 0.f;
     if (MAPS == 1 && p.f.sink) {
@@ -519,7 +522,7 @@ __global__ void __launch_bounds__(128) gqa_tc_combine_form_kernel(const GqaParam
   float c = 1.f;
   if constexpr (MAPS == 1) {
 #pragma unroll
-    for (int e = 0; e < E; ++e) y[e] = turned_back_lane(p.f, y[e], tq, threadIdx.x + 128 * e, D, true);
+    for (int e = 0; e < E; ++e) y[e] = turned_back_lane(p.f, y[e], tq, threadIdx.x + N * e, D, true);
   }
   if constexpr (MAPS == 2) {
     float ss = 0.f;
@@ -531,23 +534,23 @@ __global__ void __launch_bounds__(128) gqa_tc_combine_form_kernel(const GqaParam
     c = p.f.post * rsqrtf((red[0] + red[1] + red[2] + red[3]) / D + p.f.eps);
   }
 #pragma unroll
-  for (int e = 0; e < E; ++e) p.out[(int64_t)tq * p.out_ld + head * D + threadIdx.x + 128 * e] = __float2bfloat16(y[e] * c);
+  for (int e = 0; e < E; ++e) p.out[(int64_t)tq * p.out_ld + head * D + threadIdx.x + N * e] = __float2bfloat16(y[e] * c);
 }
 
 typedef CUresult (*PFN_encode)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
                                const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-template <int D, int PAGE, int MAPS = 0>
+template <int D, int PAGE, int MAPS = 0, int DV = D>
 int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const GqaParams& p, int NB, cudaStream_t s) {
-  using C = GCfg<D, PAGE, MAPS>;
+  using C = GCfg<D, PAGE, MAPS, DV>;
   static MarySmemSlots smem_set = {};
-  if (int rc = mary_ensure_dyn_smem((const void*)gqa_decode_tc_kernel<D, PAGE, MAPS>, C::SMEM, &smem_set)) return rc;
-  MARY_LAUNCH((gqa_decode_tc_kernel<D, PAGE, MAPS>), dim3(NB, p.Hkv, p.nsplit), NTHREADS, C::SMEM, s, tq, tk, tv, p);
+  if (int rc = mary_ensure_dyn_smem((const void*)gqa_decode_tc_kernel<D, PAGE, MAPS, DV>, C::SMEM, &smem_set)) return rc;
+  MARY_LAUNCH((gqa_decode_tc_kernel<D, PAGE, MAPS, DV>), dim3(NB, p.Hkv, p.nsplit), NTHREADS, C::SMEM, s, tq, tk, tv, p);
   MARY_CHECK_LAUNCH();
   if constexpr (MAPS > 0) {
     if (p.nsplit > 1 || MAPS == 2) {
-      MARY_LAUNCH((gqa_tc_combine_form_kernel<D, MAPS>), dim3(NB, p.Hkv, p.RQ * p.G), 128, 0, s, p);
+      MARY_LAUNCH((gqa_tc_combine_form_kernel<DV, MAPS>), dim3(NB, p.Hkv, p.RQ * p.G), COMBINE_THREADS<DV>, 0, s, p);
       MARY_CHECK_LAUNCH();
     }
   } else if (p.nsplit > 1) {
@@ -562,9 +565,9 @@ int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, 
 MARY_API int64_t mary_gqa_tc_scratch_floats(int NB, int Hkv, int nsplit, int D) {
   return nsplit > 1 ? (int64_t)NB * Hkv * nsplit * TR * (D + 2) : 0;
 }
-// The forms: 32- or 64-token pages; one map of D = 128 or 256, or two maps in key rows of D = 128 (values as wide).
-MARY_API int mary_gqa_tc_form_supported(int D, int page_size, int G, int RQ, int maps) {
-  return ((D == 128 || (D == 256 && maps == 1)) && (page_size == 32 || page_size == 64) && G >= 1 && RQ >= 1 && G * RQ <= (maps == 2 ? TR / 2 : TR)) ? 1 : 0;
+// The forms: 32- or 64-token pages; one map of D = 128 or 256, or two maps in key rows of D = 128 (values as wide); one map of 128 with values of 64.
+MARY_API int mary_gqa_tc_form_supported(int D, int DV, int page_size, int G, int RQ, int maps) {
+  return ((DV == D || (D == 128 && DV == 64 && maps == 1)) && (D == 128 || (D == 256 && maps == 1)) && (page_size == 32 || page_size == 64) && G >= 1 && RQ >= 1 && G * RQ <= (maps == 2 ? TR / 2 : TR)) ? 1 : 0;
 }
 MARY_API int mary_gqa_tc_supported(int D, int page_size, int G, int RQ) {
   return ((D == 128 || D == 256) && (page_size == 16 || page_size == 32) && G >= 1 && RQ >= 1 && G * RQ <= TR && G <= 256 && RQ <= 256) ? 1 : 0;
@@ -573,18 +576,19 @@ MARY_API int mary_gqa_tc_supported(int D, int page_size, int G, int RQ) {
 // q [T, Hq, D] bf16; K / V caches [pages, page_size, Hkv, D] bf16, contiguous; out [T, Hq, D] bf16.  blk_seq / blk_q0: NB blocks of at
 // most RQ query tokens of one sequence (q0 is a global token row).  G = Hq / Hkv heads share a kv head; G * RQ <= 64.  form (or null):
 // exact softmax weights and what attention_form.cuh lists, see mary_gqa_tc_form_supported; its two maps need scratch for any nsplit (ask for 2).
-// out_ld: elements between the output rows of two tokens (0: Hq * D).
+// out_ld: elements between the output rows of two tokens (0: Hq * DV).  DV: width of the values (0: D).
 MARY_API int mary_gqa_decode_tc(const void* q, const void* kc, const void* vc, void* out, const int* page_table, const int* kv_len,
                                 const int* q_start, const int* blk_seq, const int* blk_q0, int NB, int T, int num_pages, int max_pages,
                                 int page_size, int Hq, int Hkv, int D, int RQ, int nsplit, int window, float scale, float softcap,
-                                float* scratch, const MaryAttnForm* form, int64_t out_ld, cudaStream_t s) {
+                                float* scratch, const MaryAttnForm* form, int64_t out_ld, int DV, cudaStream_t s) {
   if (NB <= 0) return MARY_OK;
+  if (DV <= 0) DV = D;
   if (Hkv < 1 || Hq % Hkv) return MARY_ERR_BAD_ARG;
   const int G = Hq / Hkv;
   const int maps = form ? (form->maps == 2 ? 2 : 1) : 0;
-  if (maps ? !mary_gqa_tc_form_supported(D, page_size, G, RQ, maps) || softcap > 0.f : !mary_gqa_tc_supported(D, page_size, G, RQ)) return MARY_ERR_BAD_ARG;
+  if (maps ? !mary_gqa_tc_form_supported(D, DV, page_size, G, RQ, maps) || softcap > 0.f : DV != D || !mary_gqa_tc_supported(D, page_size, G, RQ)) return MARY_ERR_BAD_ARG;
   const int64_t q_ld = form && form->q_ld > 0 ? form->q_ld : (int64_t)Hq * D;
-  if (out_ld <= 0) out_ld = (int64_t)Hq * D;
+  if (out_ld <= 0) out_ld = (int64_t)Hq * DV;
   if (q_ld % 8 || out_ld % 8 || ((uintptr_t)out & 15) || (maps == 2 && (form->sink || form->turn)) || (form && ((uintptr_t)form->turn & 15))) return MARY_ERR_BAD_ARG;
   if (nsplit < 1) nsplit = 1;
   if ((nsplit > 1 || maps == 2) && !scratch) return MARY_ERR_BAD_ARG;
@@ -605,9 +609,10 @@ MARY_API int mary_gqa_decode_tc(const void* q, const void* kc, const void* vc, v
   for (int which = 0; which < 2; ++which) {
     // cache as [pages][kv heads][chunks][tokens][64 dims]: the box is one page of one kv head, chunk-major
     const void* base = which ? vc : kc;
-    cuuint64_t dims[5] = {CHUNK, (cuuint64_t)page_size, (cuuint64_t)(D / CHUNK), (cuuint64_t)Hkv, (cuuint64_t)num_pages};
-    cuuint64_t strides[4] = {(cuuint64_t)Hkv * D * 2, CHUNK * 2, (cuuint64_t)D * 2, (cuuint64_t)page_size * Hkv * D * 2};
-    cuuint32_t box[5] = {CHUNK, (cuuint32_t)(page_size < 32 ? page_size : 32), (cuuint32_t)(D / CHUNK), 1, 1};
+    const int w = which ? DV : D;
+    cuuint64_t dims[5] = {CHUNK, (cuuint64_t)page_size, (cuuint64_t)(w / CHUNK), (cuuint64_t)Hkv, (cuuint64_t)num_pages};
+    cuuint64_t strides[4] = {(cuuint64_t)Hkv * w * 2, CHUNK * 2, (cuuint64_t)w * 2, (cuuint64_t)page_size * Hkv * w * 2};
+    cuuint32_t box[5] = {CHUNK, (cuuint32_t)(page_size < 32 ? page_size : 32), (cuuint32_t)(w / CHUNK), 1, 1};
     cuuint32_t estr[5] = {1, 1, 1, 1, 1};
     if (((uintptr_t)base & 15) || enc(which ? &tv : &tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 5, const_cast<void*>(base), dims, strides, box, estr,
                                       CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
@@ -617,12 +622,13 @@ MARY_API int mary_gqa_decode_tc(const void* q, const void* kc, const void* vc, v
   GqaParams p;
   p.page_table = page_table; p.kv_len = kv_len; p.q_start = q_start; p.blk_seq = blk_seq; p.blk_q0 = blk_q0;
   p.out = (__nv_bfloat16*)out; p.part_o = scratch;
-  p.part_ml = scratch ? scratch + (int64_t)NB * Hkv * nsplit * TR * D : nullptr;
+  p.part_ml = scratch ? scratch + (int64_t)NB * Hkv * nsplit * TR * DV : nullptr;
   p.max_pages = max_pages; p.Hq = Hq; p.Hkv = Hkv; p.G = G; p.RQ = RQ; p.nsplit = nsplit; p.window = window;
   p.scale = scale; p.softcap = softcap; p.status = mary_status_ptr();
   p.page = page_size; p.out_ld = out_ld;
   p.f = form ? *form : MaryAttnForm{};
   if (maps == 2) return launch<128, 32, 2>(tq, tk, tv, p, NB, s);
+  if (maps == 1 && DV != D) return launch<128, 32, 1, 64>(tq, tk, tv, p, NB, s);
   if (maps == 1) return D == 128 ? launch<128, 32, 1>(tq, tk, tv, p, NB, s) : launch<256, 32, 1>(tq, tk, tv, p, NB, s);
   if (D == 128) return page_size == 16 ? launch<128, 16>(tq, tk, tv, p, NB, s) : launch<128, 32>(tq, tk, tv, p, NB, s);
   return page_size == 16 ? launch<256, 16>(tq, tk, tv, p, NB, s) : launch<256, 32>(tq, tk, tv, p, NB, s);

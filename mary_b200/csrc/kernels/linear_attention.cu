@@ -304,11 +304,24 @@ __global__ void __launch_bounds__(NT) lightning_step_kernel(const T* __restrict_
   __syncthreads();
   if (!last) return;
   __threadfence();
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < inner; i += NT) { const float x = __ldcg(yr + i); ss = fmaf(x, x, ss); }
-  const float inv = 1.0f / sqrtf(block_sum_x(ss, red) / inner + io.eps);
   T* o = y + (int64_t)t * ldy;
-  for (int i = threadIdx.x; i < inner; i += NT) o[i] = from_f<T>(__ldcg(yr + i) * inv * to_f<T>(gain[i]) * sigmoid_t<T>(to_f<T>(gate[row + i])));
+  const T* gr = gate + row;
+  auto put = [&](int i, float x, float inv) { o[i] = from_f<T>(x * inv * to_f<T>(gain[i]) * sigmoid_t<T>(to_f<T>(gr[i]))); };
+  constexpr int KEEP = 16;                             // values a thread keeps between the two passes, all requested before the first is used
+  float held[KEEP], ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int i = threadIdx.x + j * NT;
+    held[j] = i < inner ? __ldcg(yr + i) : 0.f;
+  }
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) ss = fmaf(held[j], held[j], ss);
+  for (int i = threadIdx.x + KEEP * NT; i < inner; i += NT) { const float x = __ldcg(yr + i); ss = fmaf(x, x, ss); }
+  const float inv = 1.0f / sqrtf(block_sum_x(ss, red) / inner + io.eps);
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j)
+    if ((int)threadIdx.x + j * NT < inner) put(threadIdx.x + j * NT, held[j], inv);
+  for (int i = threadIdx.x + KEEP * NT; i < inner; i += NT) put(i, __ldcg(yr + i), inv);
 }
 
 template <typename T, int NR4>

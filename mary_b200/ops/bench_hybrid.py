@@ -362,6 +362,9 @@ def run_kivezen(width: int = 2048, heads: int = 16, kv_heads: int = 4, experts: 
         add("attention_prefill", case, lambda: K.attention_prefill(Q, kc, vc, m, 0.05), fl, tf, like="routed decoder")
         add("  capped, sink", case, lambda: H.attention_exact(Q, kc, vc, m, 0.05, out=out, form=AttentionForm(cap=30.0, sink=sink)), fl, tf)
         add("  capped, sink, turned", case, lambda: H.attention_exact(Q, kc, vc, m, 0.05, out=out, form=AttentionForm(cap=30.0, sink=sink, turn=turn)), fl, tf)
+        half, half_turn = vc.view(-1, 64, kv_heads, D // 2)[:kc.shape[0]].contiguous(), turn[:, :D // 4].contiguous()
+        add("  .., values of 64", case, lambda: H.attention_exact(Q, kc, half, m, 0.05, out=out[:, :C // 2], form=AttentionForm(cap=30.0, sink=sink, turn=half_turn)),
+            0.75 * fl, tf)
         inv, g = torch.ones(D // 2, device="cuda"), torch.ones(D, **bf)
         add("qk_norm_rope_append", case, lambda: K.qk_norm_rope_append(y, heads, kv_heads, D, g, g, False, inv, m, kc, vc, 1e-5), nbytes=T * n_in * 4,
             like="routed decoder")
@@ -396,6 +399,9 @@ def run_kivezen(width: int = 2048, heads: int = 16, kv_heads: int = 4, experts: 
         m16, k16, v16 = _meta(B, 1, ctx, 16), kc.view(-1, 16, kv_heads, D), vc.view(-1, 16, kv_heads, D)
         add("gqa_decode_tc", case, lambda: K.gqa_decode_tc(Q, k16, v16, m16, 0.1), nbytes=nb, like="routed decoder")
         add("  capped, sink, turned", case, lambda: H.attention_exact(Q, kc, vc, m, 0.05, out=out, form=AttentionForm(cap=30.0, sink=sink, turn=turn)), nbytes=nb)
+        half, half_turn = vc.view(-1, 64, kv_heads, D // 2)[:kc.shape[0]].contiguous(), turn[:, :D // 4].contiguous()
+        add("  .., values of 64", case, lambda: H.attention_exact(Q, kc, half, m, 0.05, out=out[:, :C // 2], form=AttentionForm(cap=30.0, sink=sink, turn=half_turn)),
+            nbytes=0.75 * nb)
         inv, g = torch.ones(D // 2, device="cuda"), torch.ones(D, **bf)
         add("qk_norm_rope_append", case, lambda: K.qk_norm_rope_append(y, heads, kv_heads, D, g, g, False, inv, m, kc, vc, 1e-5), nbytes=B * n_in * 4,
             like="routed decoder")

@@ -506,7 +506,7 @@ def paged_attention_decode_q8(q, kcache, vcache, meta, scale, window=0, softcap=
     return out
 
 
-declare("mary_gqa_decode_tc", "ppppppppp" + "iiiiiiiiiii" + "ffppls")
+declare("mary_gqa_decode_tc", "ppppppppp" + "iiiiiiiiiii" + "ffpplis")
 declare("mary_gqa_tc_supported", "iiii")
 declare("mary_gqa_tc_scratch_floats", "iiii", ret64=True)
 
@@ -525,15 +525,15 @@ def gqa_tc_supported(q, kcache, meta) -> bool:
     return bool(lib().mary_gqa_tc_supported(D, meta.page_size, G, rq)) and kcache.shape[1] == meta.page_size
 
 
-declare("mary_gqa_tc_form_supported", "iiiii")
+declare("mary_gqa_tc_form_supported", "iiiiii")
 
 
 def gqa_tc_form_supported(q, kcache, vcache, meta, form) -> bool:
-    """Whether the tensor-core decode kernel takes this ``AttentionForm`` (32- or 64-token pages, one map of 128 or 256 dims, or two of 64 with
-    values of 128)."""
+    """Whether the tensor-core decode kernel takes this ``AttentionForm`` (32- or 64-token pages, one map of 128 or 256 dims with values as
+    wide, one of 128 with values of 64, or two of 64 with values of 128)."""
     G = q.shape[1] // kcache.shape[2]
-    return (q.dtype == torch.bfloat16 and kcache.shape == vcache.shape and kcache.is_contiguous() and vcache.is_contiguous()
-            and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and bool(lib().mary_gqa_tc_form_supported(q.shape[2], meta.page_size, G, 1, form.maps)))
+    return (q.dtype == torch.bfloat16 and kcache.shape[:3] == vcache.shape[:3] and kcache.is_contiguous() and vcache.is_contiguous()
+            and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and bool(lib().mary_gqa_tc_form_supported(q.shape[2], vcache.shape[3], meta.page_size, G, 1, form.maps)))
 
 
 def gqa_decode_tc(q, kcache, vcache, meta, scale, window=0, softcap=0.0, nsplit=None, out=None, group=None, form=None):
@@ -541,7 +541,7 @@ def gqa_decode_tc(q, kcache, vcache, meta, scale, window=0, softcap=0.0, nsplit=
     tile, K and V pages arrive by TMA, split-KV partials are merged by a second kernel.  ``form`` (see ``ops.attention_exact``; ``q`` and ``out`` may
     then be row views): exact softmax weights."""
     T, Hq, D = q.shape
-    Hkv = kcache.shape[2]
+    Hkv, DV = kcache.shape[2], vcache.shape[3]
     G = Hq // Hkv
     maps = 1 if form is None else form.maps
     rq = max(1, min(64 // maps // G, meta.max_q_len, 8 if group == "decode" else 64))
@@ -551,25 +551,26 @@ def gqa_decode_tc(q, kcache, vcache, meta, scale, window=0, softcap=0.0, nsplit=
         span = meta.max_kv_len if window <= 0 else min(meta.max_kv_len, window + rq)
         nsplit = max(1, min(want, 32, span // (4 * min(meta.page_size, 32))))
     if out is None:
-        out = _empty(T, Hq, D, dtype=torch.bfloat16, device=q.device)
+        out = _empty(T, Hq, DV, dtype=torch.bfloat16, device=q.device)
         ld = 0
     else:
         ld = out.stride(0)
     scratch = None
     if nsplit > 1 or maps == 2:
-        scratch = _empty(lib().mary_gqa_tc_scratch_floats(NB, Hkv, max(nsplit, maps), D), dtype=torch.float32, device=q.device)
+        scratch = _empty(lib().mary_gqa_tc_scratch_floats(NB, Hkv, max(nsplit, maps), DV), dtype=torch.float32, device=q.device)
     if form is None:
         q = q.contiguous()
     fs = form_struct(form, q)
-    assert vcache.is_contiguous() and vcache.shape == kcache.shape
+    assert vcache.is_contiguous() and vcache.shape[:3] == kcache.shape[:3]
     check(lib().mary_gqa_decode_tc(_p(q), _p(kcache), _p(vcache), _p(out), _p(meta.page_table), _p(meta.kv_len), _p(meta.q_start),
                                    _p(blk_seq), _p(blk_q0), NB, T, kcache.shape[0], meta.page_table.shape[1], meta.page_size, Hq, Hkv, D, rq,
-                                   nsplit, window, scale, softcap, _p(scratch), _form_p(fs), ld, _stream()), "gqa_decode_tc")
+                                   nsplit, window, scale, softcap, _p(scratch), _form_p(fs), ld, DV, _stream()), "gqa_decode_tc")
     return out
 
 
 declare("mary_attention_prefill", "ppppppppp" + "iiiiiiii" + "llll" + "ifi" + "li" + "pplps")
 declare("mary_attention_prefill_maps_supported", "ii")
+declare("mary_attention_prefill_form_supported", "ii")
 declare("mary_attention_prefill_supported", "ii")
 PREFILL_MIN_ROWS = 48     # mean query tokens per sequence from which the 128-row tensor-core tiles pay off
 

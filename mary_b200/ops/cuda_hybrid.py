@@ -204,9 +204,9 @@ def attention_exact(q, kcache, vcache, meta, scale, out=None, window: int = 0, b
         fast_prefill = bf16 and meta.page_size in (16, 64) and aligned
         fast_decode = bf16 and Hq // Hkv <= 4 and aligned
     else:
-        bf16 = bf16 and DK == DV and DK in (64, 128, 256)
-        fast_prefill = bf16 and meta.page_size in (16, 64) and aligned
-        fast_decode = bf16 and Hq // Hkv <= (4 if DK == 256 else 8) and (q.is_contiguous() or aligned)
+        equal = DK == DV and DK in (64, 128, 256)
+        fast_prefill = bf16 and (bool(lib().mary_attention_prefill_form_supported(DK, DV)) if form is not None else equal) and meta.page_size in (16, 64) and aligned
+        fast_decode = bf16 and equal and Hq // Hkv <= (4 if DK == 256 else 8) and (q.is_contiguous() or aligned)
     tc_decode = form is not None and aligned and window == 0 and bias is None and gate is None and K.gqa_tc_form_supported(q, kcache, vcache, meta, form)
     fast_decode = fast_decode or tc_decode
     if not (fast_prefill or fast_decode):
