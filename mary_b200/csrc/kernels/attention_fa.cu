@@ -426,6 +426,18 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       if (lane == 0) mbar_arrive(&p_full[pb]);
     }
     // ------------------------------------------------------------------ write out
+    const int o_lo = half * (DV / HW), o_hi = o_lo + DV / HW;      // value columns of this thread
+    const bool turned = MAPS == 1 && p.f.turn && row_ok;
+    float4 cs[MAPS == 1 ? 8 : 1];                                  // angles of the next 32 columns, requested ahead of their use
+    auto load_turn = [&](int c0) {
+      if constexpr (MAPS == 1) {
+        if (!turned) return;
+        const float4* src = (const float4*)(p.f.turn + ((int64_t)(tok0 + r) * DV + c0) / 2);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) cs[j] = __ldg(src + j);
+      }
+    };
+    load_turn(o_lo);
     if (!wait(&pv_done[(ntot - 1) % NPBUF], ((ntot - 1) / NPBUF) & 1)) goto done;
     tc_fence_after();
     if constexpr (HW == 2) {
@@ -437,7 +449,6 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
       l += xch[(half ^ 1) * TR + r];
       l_first += xch[(2 + (half ^ 1)) * TR + r];
     }
-    const int o_lo = half * (DV / HW), o_hi = o_lo + DV / HW;      // value columns of this thread
     if constexpr (MAPS == 1) {
       if (p.f.sink) l += exp2f(fmaf(p.f.sink[head], 1.4426950408889634f, -m_ref));
     }
@@ -512,15 +523,14 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constan
           }
         }
         if constexpr (MAPS == 1) {
-          if (p.f.turn) {
-            const float4* cs = (const float4*)(p.f.turn + ((int64_t)(tok0 + r) * DV + c0) / 2);
+          if (turned) {
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-              const float4 c = cs[j];
               float* x = (float*)o + 4 * j;
-              const float2 a = turned_back(make_float2(c.x, c.y), x[0], x[1]), b = turned_back(make_float2(c.z, c.w), x[2], x[3]);
+              const float2 a = turned_back(make_float2(cs[j].x, cs[j].y), x[0], x[1]), b = turned_back(make_float2(cs[j].z, cs[j].w), x[2], x[3]);
               x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y;
             }
+            if (c0 + 32 < o_hi) load_turn(c0 + 32);
           }
         }
 #pragma unroll

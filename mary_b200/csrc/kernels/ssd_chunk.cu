@@ -17,6 +17,10 @@
 // product that reads the state, so it never leaves the registers between chunks.  C, B and x of the next chunk are in flight while this
 // one is worked on.  Rows in shared memory are padded by 16 bytes, so the eight rows of a fragment fall on different banks and every
 // address of a loop is a base and a constant.
+//
+// Where heads and sequences leave most of the machine without work, a sequence is cut into segments of whole chunks: a first pass takes every
+// segment but the last through the state update alone, from a state of zero, and the pass proper starts each segment from what the earlier
+// ones left, S <- d S + E with a segment's end state E and its whole decay d.
 #include "host_utils.h"
 #include "typed.cuh"
 
@@ -35,6 +39,9 @@ struct ChunkParams {
   const int* q_start; const int* kv_len; const int* slots;
   int T, G, H, N, P;
   int64_t C;                             // elements between the rows of two tokens
+  int segs;                              // segments per sequence
+  float* seg_state;                      // segs > 1: [S][segs][H][P][NS]: the state before the portion, then the end states of segments 0 .. segs - 2
+  float* seg_log;                        // [S][segs][H]: log2 of the decay over segment 0 .. segs - 2
   int per_head;                          // 1: decays that are the same for all tokens, dt, c_hi and c_lo [H][64] by place in the chunk
 };
 
@@ -87,8 +94,8 @@ template <int NP> struct Lay {
   static_assert(2 * M + 2 * X <= 4 * Y, "the decayed products and the weighted x fit");
 };
 
-// 64 rows of B and C, THREADS threads; src: this thread's first piece of B.  Rows past `rows` and state rows past N are zero.
-template <int NP, int THREADS>
+// 64 rows of B (and of C: WITH_C), THREADS threads; src: this thread's first piece of B.  Rows past `rows` and state rows past N are zero.
+template <int NP, int THREADS, bool WITH_C = true>
 __device__ __forceinline__ void load_bc(uint32_t dst_c, uint32_t dst_b, const bf16* src, int64_t ld, int c_off, bool col, int rows) {
   constexpr int CN = NP / 8, STEP = THREADS / CN;
   const int r0 = threadIdx.x / CN, k = threadIdx.x % CN;
@@ -97,7 +104,7 @@ __device__ __forceinline__ void load_bc(uint32_t dst_c, uint32_t dst_b, const bf
 #pragma unroll
   for (int i = 0; i < L / STEP; ++i) {
     const bool in = col && r0 + i * STEP < rows;
-    cp16(dst_c + o + i * STEP * Lay<NP>::ROW, in ? s + c_off : src, in);
+    if constexpr (WITH_C) cp16(dst_c + o + i * STEP * Lay<NP>::ROW, in ? s + c_off : src, in);
     cp16(dst_b + o + i * STEP * Lay<NP>::ROW, in ? s : src, in);
     s += STEP * ld;
   }
@@ -141,7 +148,8 @@ __global__ void __launch_bounds__(128) ssd_gram_kernel(const ChunkParams p) {
   }
 }
 
-template <int NP>
+// STATE_ONLY: the first pass over segments.
+template <int NP, bool STATE_ONLY>
 __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const ChunkParams p) {
   pdl_sync();
   using S = Lay<NP>;
@@ -149,12 +157,19 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
   extern __shared__ __align__(128) uint8_t smem[];
   const uint32_t sm = smem_u32(smem);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pw = warp & 1, nw = warp >> 1;
-  const int seq = blockIdx.z, h = blockIdx.y, p0 = blockIdx.x * PC, g = h / (p.H / p.G), inner = p.H * p.P;
+  const int per_seq = STATE_ONLY ? p.segs - 1 : p.segs;
+  const int seq = blockIdx.z / per_seq, seg = blockIdx.z % per_seq, h = blockIdx.y, p0 = blockIdx.x * PC, g = h / (p.H / p.G), inner = p.H * p.P;
   const int row0 = p.q_start[seq], n = p.q_start[seq + 1] - row0;
   if (n <= 0) return;
   const bool fresh = p.kv_len[seq] == n;
   const int NS = (p.N + 3) / 4 * 4;
+  const int chunks = (n + L - 1) / L, seg_chunks = (chunks + p.segs - 1) / p.segs;
+  const int c_lo = min(chunks, seg * seg_chunks), c_hi = min(chunks, c_lo + seg_chunks);
+  if (!STATE_ONLY && c_lo >= c_hi) return;
   float* state = p.state + ((int64_t)p.slots[seq] * p.H + h) * p.P * NS;
+  float* seg_at = p.segs > 1 ? p.seg_state + ((int64_t)seq * p.segs * p.H + h) * p.P * NS : nullptr;      // entry 0 of this head
+  const int64_t seg_step = (int64_t)p.H * p.P * NS;
+  const float* seg_log = p.segs > 1 ? p.seg_log + (int64_t)seq * p.segs * p.H + h : nullptr;
   const int lr = lane >> 2, lc = (lane & 3) * 2;            // row and first column of an accumulator tile held by this lane
   // S^T: tile t = state rows nw NH + 8 t .., channels p0 + 16 pw ..
   float st[NT][4];
@@ -164,7 +179,21 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
     for (int e = 0; e < 2; ++e) {
       const int ch = p0 + pw * 16 + lr + 8 * e, r = nw * NH + t * 8 + lc;
       float2 v = make_float2(0.f, 0.f);
-      if (!fresh && ch < p.P && r < p.N) v = *(const float2*)(state + (int64_t)ch * NS + r);
+      if (ch < p.P && r < p.N) {
+        const int64_t at = (int64_t)ch * NS + r;
+        if constexpr (STATE_ONLY) {
+          if (seg == 0) *(float2*)(seg_at + at) = fresh ? v : *(const float2*)(state + at);
+        } else if (p.segs > 1) {
+          v = *(const float2*)(seg_at + at);
+          for (int j = 0; j < seg; ++j) {
+            const float d = pow2(seg_log[j * p.H]);
+            const float2 end = *(const float2*)(seg_at + (j + 1) * seg_step + at);
+            v = make_float2(fmaf(v.x, d, end.x), fmaf(v.y, d, end.y));
+          }
+        } else if (!fresh) {
+          v = *(const float2*)(state + at);
+        }
+      }
       st[t][2 * e] = v.x;
       st[t][2 * e + 1] = v.y;
     }
@@ -184,7 +213,7 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
     const uint32_t s = sm + (c & 1) * S::STAGE;
     const int t0 = c * L, left = n - t0;
     const bf16* row = bc_row + (int64_t)t0 * p.C;
-    load_bc<NP, NTH>(s, s + S::TILE, bc_r < left ? first_piece<NP, NTH>(row, p.C, p.N) : row, p.C, p.G * p.N, bc_col, left);
+    load_bc<NP, NTH, !STATE_ONLY>(s, s + S::TILE, bc_r < left ? first_piece<NP, NTH>(row, p.C, p.N) : row, p.C, p.G * p.N, bc_col, left);
     const bool in = x_col && xr < left;
     cp16(s + 2 * S::TILE + x_at, x_row + (int64_t)(in ? t0 + xr : t0) * p.C, in);
     if (tid < L) {                                          // tokens past the end: no step, the decay of the last one
@@ -205,11 +234,16 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
   const uint32_t f_w = ((lane & 7) + ((lane >> 4) << 3)) * S::XROW + (pw * 2 + ((lane >> 3) & 1)) * 16;      // weighted x, first operand
   const uint32_t f_b = (lane & 15) * S::ROW + (nw * NH) * 2 + (lane >> 4) * 16;               // B, second operand
 
-  const int chunks = (n + L - 1) / L;
-  load(0);
-  for (int c = 0; c < chunks; ++c) {
-    float4 gm[2] = {gram_at[warp * 64], gram_at[warp * 64 + 32]};
-    if (c + 1 < chunks) {
+  double seg_sum = 0.0;
+  if (c_lo < c_hi) load(c_lo);
+  if constexpr (!STATE_ONLY) {
+    gram_at += (int64_t)c_lo * p.G * 640;
+    y_at += (int64_t)c_lo * L * inner;
+  }
+  for (int c = c_lo; c < c_hi; ++c) {
+    float4 gm[2];
+    if constexpr (!STATE_ONLY) { gm[0] = gram_at[warp * 64]; gm[1] = gram_at[warp * 64 + 32]; }
+    if (c + 1 < c_hi) {
       load(c + 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
@@ -233,6 +267,7 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
       *(uint4*)(smem + S::XW_AT + x_at) = a;
       *(uint4*)(smem + S::XW_AT + S::X + x_at) = b;
     }
+    if constexpr (!STATE_ONLY)
     for (int b = warp; b < 10; b += 8) {                    // decayed products
       const int mt = blk_m(b), jt = blk_j(b);
       const int i0 = mt * 16 + lr;
@@ -261,6 +296,7 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
     }
     // what the state before the chunk gives (this warp's quarter of its rows), without the tokens' decay
     float y[4][2][4];
+    if constexpr (!STATE_ONLY)
 #pragma unroll
     for (int k = 0; k < NH / 16; ++k) {
       uint32_t bh[2][2], bl[2][2];                          // [channel octet][half of the k rows]
@@ -301,6 +337,11 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
       for (int t = 0; t < NT; ++t) mma(st[t], a, q[t / 2][2 * (t & 1)], q[t / 2][2 * (t & 1) + 1]);
 #pragma unroll
       for (int t = 0; t < NT; ++t) mma(st[t], b, q[t / 2][2 * (t & 1)], q[t / 2][2 * (t & 1) + 1]);
+    }
+    if constexpr (STATE_ONLY) {
+      seg_sum += (double)hiL + (double)loL;
+      __syncthreads();
+      continue;
     }
     // tokens of the chunk among themselves: token block nw, which this warp also finishes
     float z[2][4] = {};
@@ -350,6 +391,12 @@ __global__ void __launch_bounds__(NTH, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
     }
     gram_at += p.G * 640;
     y_at += L * (int64_t)inner;
+  }
+  if constexpr (STATE_ONLY) {
+    state = seg_at + (seg + 1) * seg_step;
+    if (p0 == 0 && tid == 0) p.seg_log[((int64_t)seq * p.segs + seg) * p.H + h] = (float)seg_sum;
+  } else if (c_hi < chunks) {
+    return;
   }
 #pragma unroll
   for (int t = 0; t < NT; ++t)
@@ -458,13 +505,27 @@ __global__ void __launch_bounds__(256) ss_decay_kernel(const bf16* __restrict__ 
   }
 }
 
+// Segments per sequence: as many as the machine has room for beside what heads and sequences fill, of eight chunks or more.
+int chunk_segments(int S, int max_q, int H, int N, int P) {
+  const int64_t blocks = (int64_t)((P + PC - 1) / PC) * H * S, room = (int64_t)mary_num_sms() * (N <= 128 ? 2 : 1);
+  int segs = (int)(room / blocks);
+  const int most = (max_q + L - 1) / L / 8;
+  segs = segs < most ? segs : most;
+  segs = segs < 16 ? segs : 16;
+  return segs > 1 && (int64_t)S * segs <= 65535 ? segs : 1;
+}
+int64_t gram_floats(int T, int S, int G) { return ((int64_t)T / L + S + 1) * G * 10 * 64 * 4; }
+
 template <int NP>
 int launch_chunk(const ChunkParams& p, int S, int max_q, cudaStream_t s) {
-  static MarySmemSlots slots[2] = {};
+  static MarySmemSlots slots[3] = {};
   if (int rc = mary_ensure_dyn_smem((const void*)ssd_gram_kernel<NP>, 2 * Lay<NP>::TILE, &slots[0])) return rc;
-  if (int rc = mary_ensure_dyn_smem((const void*)ssd_chunk_kernel<NP>, Lay<NP>::BYTES, &slots[1])) return rc;
+  if (int rc = mary_ensure_dyn_smem((const void*)ssd_chunk_kernel<NP, false>, Lay<NP>::BYTES, &slots[1])) return rc;
+  if (int rc = mary_ensure_dyn_smem((const void*)ssd_chunk_kernel<NP, true>, Lay<NP>::BYTES, &slots[2])) return rc;
+  const int cols = (p.P + PC - 1) / PC;
   MARY_LAUNCH((ssd_gram_kernel<NP>), dim3((max_q + L - 1) / L, p.G, S), 128, 2 * Lay<NP>::TILE, s, p);
-  MARY_LAUNCH((ssd_chunk_kernel<NP>), dim3((p.P + PC - 1) / PC, p.H, S), NTH, Lay<NP>::BYTES, s, p);
+  if (p.segs > 1) MARY_LAUNCH((ssd_chunk_kernel<NP, true>), dim3(cols, p.H, S * (p.segs - 1)), NTH, Lay<NP>::BYTES, s, p);
+  MARY_LAUNCH((ssd_chunk_kernel<NP, false>), dim3(cols, p.H, S * p.segs), NTH, Lay<NP>::BYTES, s, p);
   MARY_CHECK_LAUNCH();
   return MARY_OK;
 }
@@ -492,10 +553,16 @@ MARY_API int mary_ss_conv_decay(const void* xbc, int64_t ldx, const void* taps_w
 
 MARY_API int mary_ssd_chunk_supported(int N, int P) { return N >= 8 && N <= 256 && N % 8 == 0 && P >= 8 && P % 8 == 0; }
 
-MARY_API int64_t mary_ssd_chunk_scratch_floats(int T, int S, int G) { return ((int64_t)T / L + S + 1) * G * 10 * 64 * 4; }
+MARY_API int64_t mary_ssd_chunk_scratch_floats(int T, int S, int max_q, int G, int H, int N, int P) {
+  const int segs = chunk_segments(S, max_q, H, N, P);
+  return gram_floats(T, S, G) + (segs > 1 ? (int64_t)S * segs * H * ((int64_t)P * ((N + 3) / 4 * 4) + 1) : 0);
+}
 
-static int chunk_run(const ChunkParams& p, int S, int max_q, cudaStream_t s) {
+static int chunk_run(ChunkParams p, int S, int max_q, cudaStream_t s) {
   if (S <= 0 || p.T <= 0) return MARY_OK;
+  p.segs = chunk_segments(S, max_q, p.H, p.N, p.P);
+  p.seg_state = (float*)p.gram + gram_floats(p.T, S, p.G);
+  p.seg_log = p.seg_state + (int64_t)S * p.segs * p.H * p.P * ((p.N + 3) / 4 * 4);
   if (p.G < 1 || p.H < 1 || p.H % p.G || p.H > 65535 || S > 65535 || !mary_ssd_chunk_supported(p.N, p.P) || p.C % 8 ||
       (((uintptr_t)p.xbc | (uintptr_t)p.gram) & 15))
     return MARY_ERR_BAD_ARG;
@@ -505,11 +572,11 @@ static int chunk_run(const ChunkParams& p, int S, int max_q, cudaStream_t s) {
 }
 
 // y [T, H P] f32; the state [slots][H][P][N] is read (zero for a portion that starts its sequence) and updated in place.  scratch:
-// mary_ssd_chunk_scratch_floats(T, S, G) floats, 16-byte aligned.
+// mary_ssd_chunk_scratch_floats(T, S, max_q, G, H, N, P) floats, 16-byte aligned.
 MARY_API int mary_ssd_chunk(const void* xbc, const float* dt, const float* c_hi, const float* c_lo, const float* skip, float* y, float* state,
                             float* scratch, const int* q_start, const int* kv_len, const int* slots, int S, int max_q, int T, int G, int H, int N, int P,
                             cudaStream_t s) {
-  return chunk_run({(const bf16*)xbc, dt, c_hi, c_lo, skip, y, state, (float4*)scratch, q_start, kv_len, slots, T, G, H, N, P, H * P + 2 * G * N, 0}, S, max_q, s);
+  return chunk_run({(const bf16*)xbc, dt, c_hi, c_lo, skip, y, state, (float4*)scratch, q_start, kv_len, slots, T, G, H, N, P, H * P + 2 * G * N, 1, nullptr, nullptr, 0}, S, max_q, s);
 }
 
 // Linear attention with one constant decay per head, S_t = d S_{t-1} + k_t v_t^T, y_t = S_t^T q_t: the same chunks with q, k, v for C, B, x.  vkq:
@@ -518,5 +585,5 @@ MARY_API int mary_lightning_chunk(const void* vkq, int64_t ld, const float* one,
                                   float* state, float* scratch, const int* q_start, const int* kv_len, const int* slots, int S, int max_q, int T, int H,
                                   int N, int P, cudaStream_t s) {
   if (ld < (int64_t)H * (P + 2 * N)) return MARY_ERR_BAD_ARG;
-  return chunk_run({(const bf16*)vkq, one, c_hi, c_lo, zero, y, state, (float4*)scratch, q_start, kv_len, slots, T, H, H, N, P, ld, 1}, S, max_q, s);
+  return chunk_run({(const bf16*)vkq, one, c_hi, c_lo, zero, y, state, (float4*)scratch, q_start, kv_len, slots, T, H, H, N, P, ld, 1, nullptr, nullptr, 1}, S, max_q, s);
 }

@@ -45,7 +45,7 @@ declare("mary_fill_shared_part", "pliplii" + "iis")
 declare("mary_ss_prep", "pl" + "pppppp" + "ppp" + "pppppp" + "iiiiiii" + "is")
 declare("mary_ss_conv_decay", "pl" + "pppppp" + "ppp" + "pppp" + "iiiiiis")
 declare("mary_ssd_chunk", "pppppppp" + "ppp" + "iiiiiiis")
-declare("mary_ssd_chunk_scratch_floats", "iii", ret64=True)
+declare("mary_ssd_chunk_scratch_floats", "iiiiiii", ret64=True)
 declare("mary_ssd_chunk_supported", "ii")
 declare("mary_head_decay_scan", "pppppppp" + "p" + "ppp" + "illl" + "iiiis")
 declare("mary_gated_part_norm", "pplppl" + "iiifiis")
@@ -513,7 +513,7 @@ def ssd_chunk(rows, dt, hi, lo, skip, state, meta, G, H, N, P):
     """The recurrence on the tensor cores, 64 tokens at a time: f32 ``[T, H * P]``."""
     T = rows.shape[0]
     y = _empty(T, H * P, dtype=torch.float32, device=rows.device)
-    scratch = _empty(lib().mary_ssd_chunk_scratch_floats(T, meta.num_seqs, G), dtype=torch.float32, device=rows.device)
+    scratch = _empty(lib().mary_ssd_chunk_scratch_floats(T, meta.num_seqs, meta.max_q_len, G, H, N, P), dtype=torch.float32, device=rows.device)
     check(lib().mary_ssd_chunk(_p(rows), _p(dt), _p(hi), _p(lo), _p(skip), _p(y), _p(state), _p(scratch), _p(meta.q_start), _p(meta.kv_len),
                                _p(meta.state_slots), meta.num_seqs, meta.max_q_len, T, G, H, N, P, _stream()), "ssd_chunk")
     return y
@@ -553,7 +553,7 @@ def lightning_chunk(y_in, decays, state, meta, H, dk, dv):
     """The recurrence on the tensor cores, 64 tokens at a time, over projection rows that start with ``[v | k | q]``: f32 ``[T, H * dv]``."""
     T = y_in.shape[0]
     o = _empty(T, H * dv, dtype=torch.float32, device=y_in.device)
-    scratch = _empty(lib().mary_ssd_chunk_scratch_floats(T, meta.num_seqs, H), dtype=torch.float32, device=y_in.device)
+    scratch = _empty(lib().mary_ssd_chunk_scratch_floats(T, meta.num_seqs, meta.max_q_len, H, H, dk, dv), dtype=torch.float32, device=y_in.device)
     one, hi, lo, zero = (_p(t) for t in decays.chunk)
     py, ld = _rows(y_in)
     check(lib().mary_lightning_chunk(py, ld, one, hi, lo, zero, _p(o), _p(state), _p(scratch), _p(meta.q_start), _p(meta.kv_len), _p(meta.state_slots),

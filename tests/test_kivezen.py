@@ -221,6 +221,32 @@ def test_lightning_attention(target, shape, cut):
         assert bool((out[:, C:] == 7.0).all())
 
 
+def test_long_prompts_with_few_heads(target):
+    """Thousands of tokens beside short portions and single tokens, begun and continued: where heads are few, a long portion is worked on in several places at
+    once, each from the state that the places before it leave."""
+    dev, dt = target
+    H, D, E, eps = 2, 64, 32, 1e-3
+    decay, g = (0.9995, 0.97), torch.Generator().manual_seed(8)
+    lengths = {0: 2700, 1: 1600, 2: 41, 3: 2}
+    x = {s: rand(g, n, 2 * H * (D + E)) for s, n in lengths.items()}
+    gain, want = rand(g, H * E), {}
+    for s, n in lengths.items():
+        v, k, q, z = x[s].double().split([H * E, H * D, H * D, H * E], 1)
+        o = oracle.decayed_sums(q.view(n, H, D), k.view(n, H, D), v.view(n, H, E), decay).reshape(n, H * E)
+        want[s] = oracle.rms(o, gain.double(), eps) * oracle.sigmoid(z)
+    pool, state = Paged(64, device=dev, slots=4), torch.full((4, *state_shape(H, D, E)), 3.0, device=dev)
+    at = dict.fromkeys(lengths, 0)
+    for step in ({0: 1500, 2: 40, 3: 1}, {1: 1600}, {0: 1200, 2: 1, 3: 1}):
+        meta = pool.step(step)
+        y = torch.cat([x[s][at[s]:at[s] + n] for s, n in step.items()]).to(dev, dt)
+        v, k, q, z = y.split([H * E, H * D, H * D, H * E], 1)
+        out = torch.empty(y.shape[0], H * E, dtype=dt, device=dev)
+        ops.lightning_attention(y, q, k, v, z, HeadDecays(decay, D, dev), gain.to(dev, dt), state, meta, H, D, E, eps, out)
+        assert error(out, torch.cat([want[s][at[s]:at[s] + n] for s, n in step.items()])) < tol(target, 5e-5, 8e-3)
+        for s, n in step.items():
+            at[s] += n
+
+
 def test_a_write_far_back_is_still_in_the_state(target):
     """One key of hundreds meets the last query; what it wrote has decayed exactly as often as there were tokens since, over chunks and portions."""
     dev, dt = target
